@@ -28,8 +28,8 @@ NVCC = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
               "-Xcompiler", "-fPIC", "-Xcompiler", "-Wall", "--expt-relaxed-constexpr",
               "-diag-suppress", "177", "-diag-suppress", "550"]
-# sources listed here are compiled without --use_fast_math (none at present: the RoPE table is built by torch ops)
-NO_FAST_MATH: set = set()
+# sources compiled without --use_fast_math: their exponentials, tanh and divisions feed routers, norms and recurrences
+NO_FAST_MATH: set = {"attention_simt.cu", "gemm_f32.cu", "mlstm.cu", "mlstm_tc5.cu", "moe.cu", "stream_norm.cu"}
 
 
 def _newer(src: str, dst: str, deps: List[str]) -> bool:
@@ -46,12 +46,39 @@ def _run(cmd: List[str]) -> str:
     return r.stdout + r.stderr
 
 
-def build_kernels(force=False, verbose=False) -> str:
+# Kernel sources of one model family, for a process that serves only that family from a tree without built libraries: they link
+# into a library of their own (`libtelb_kernels-<family>.so`) in a fraction of the time of the whole set.
+KERNEL_SETS = {
+    "dimesun": ["attention_decode_tc5.cu", "attention_simt.cu", "attention_tc5.cu", "attention_tc5_extra.cu", "elementwise.cu", "gemm_f32.cu",
+                "gemm_skinny_tc5.cu", "gemm_tc5.cu", "mlstm.cu", "mlstm_tc5.cu", "moe.cu", "nvfp4_host.cu", "stream_norm.cu"],
+}
+
+
+def kernel_library(family: str = "") -> str:
+    return os.path.join(LIBDIR, f"libtelb_kernels-{family}.so" if family else "libtelb_kernels.so")
+
+
+def ensure_built(model_type: str) -> str:
+    """Build what a model family needs if the tree holds no built libraries: the runtime module and, when the whole kernel library is
+    absent, the family's own (or the whole one for families without a list).  Returns the family whose library serves, or ""."""
+    import glob
+    if not glob.glob(os.path.join(LIBDIR, "_telb_runtime*.so")):
+        build_runtime()
+    if os.path.exists(kernel_library()):
+        return ""
+    family = model_type if model_type in KERNEL_SETS else ""
+    if not os.path.exists(kernel_library(family)):
+        build_kernels(family=family)
+    return family
+
+
+def build_kernels(force=False, verbose=False, family: str = "") -> str:
+    """Compile and link the kernel library: every source, or those of one family (``KERNEL_SETS``)."""
     kdir = os.path.join(CSRC, "kernels")
     os.makedirs(BUILD, exist_ok=True)
     os.makedirs(LIBDIR, exist_ok=True)
     headers = [os.path.join(kdir, f) for f in os.listdir(kdir) if f.endswith((".h", ".cuh", ".inc"))]
-    srcs = sorted(f for f in os.listdir(kdir) if f.endswith(".cu"))
+    srcs = sorted(KERNEL_SETS[family] if family else (f for f in os.listdir(kdir) if f.endswith(".cu")))
     objs, jobs = [], []
     for f in srcs:
         src, obj = os.path.join(kdir, f), os.path.join(BUILD, f[:-3] + ".o")
@@ -66,7 +93,7 @@ def build_kernels(force=False, verbose=False) -> str:
             for out in ex.map(_run, jobs):
                 if verbose and out.strip():
                     print(out)
-    lib = os.path.join(LIBDIR, "libtelb_kernels.so")
+    lib = kernel_library(family)
     if jobs or not os.path.exists(lib):
         # link beside the target and rename: a process (or a snapshot of the tree) never sees a half-written library
         _run([NVCC, "-shared", "-o", lib + ".tmp"] + objs + ["-lcudart_static", "-lpthread", "-ldl", "-lrt"])

@@ -118,6 +118,8 @@ def init_random_weights(model: nn.Module, seed: int = 0, std: float = 0.02) -> n
             mod.quantize_from(ws)
         elif isinstance(mod, LinearBase):
             mod.weight.data.copy_(_randn_chunked(tuple(mod.weight.shape), g, std, mod.weight.device).to(mod.weight.dtype))
+            if hasattr(mod, "zero_padding"):
+                mod.zero_padding()
         elif isinstance(mod, nn.Embedding):
             mod.weight.data.copy_(_randn_chunked(tuple(mod.weight.shape), g, std, mod.weight.device).to(mod.weight.dtype))
     for name, mod in model.named_modules():

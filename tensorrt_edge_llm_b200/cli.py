@@ -26,6 +26,7 @@ COMMANDS = {
     "tts": ("tensorrt_edge_llm_b200.commands.tts", "Text to speech from a request file (talker, code predictor, vocoder)"),
     "multistage": ("tensorrt_edge_llm_b200.commands.multistage", "Run requests through a multi-stage graph"),
     "action": ("tensorrt_edge_llm_b200.commands.action", "Vision-language-action inference: reasoning text + trajectory"),
+    "trace": ("tensorrt_edge_llm_b200.commands.trace", "Replay steps of given token ids and write logits"),
     "bench": ("tensorrt_edge_llm_b200.benchmarks.llm_bench", "Offline benchmark writing report.json"),
 }
 

@@ -4,7 +4,8 @@ Counterpart of the reference's ``examples/cpp/llm_inference.cpp`` with the reque
 ``docs/source/user_guide/format/input-format.md`` (``examples/cpp/common/requestFileParser.cpp``): top-level sampling
 defaults (``temperature top_p top_k sampling_seed max_generate_length num_logprobs logit_bias guided_decoding
 apply_chat_template add_generation_prompt enable_thinking batch_size``) and per-request ``messages`` with overrides
-(``sampling_seed logit_bias num_logprobs guided_decoding stop disable_spec_decode``).  ``--dump-profile`` prints the
+(``sampling_seed logit_bias num_logprobs guided_decoding stop disable_spec_decode``).  A request may give ``input_ids`` instead of
+``messages``; a file of such requests runs without a tokenizer.  ``--dump-profile`` prints the
 stage timings and peak device memory."""
 from __future__ import annotations
 
@@ -46,9 +47,12 @@ def parse_request_file(body: Dict[str, Any]) -> List[Dict[str, Any]]:
     top_lp = int(body.get("num_logprobs", 0))
     out = []
     for i, r in enumerate(body["requests"]):
-        if not isinstance(r, dict) or not isinstance(r.get("messages"), list) or not r["messages"]:
-            raise RequestFileError(f"requests[{i}] needs a non-empty 'messages' array")
-        for m in r["messages"]:
+        ids = r.get("input_ids") if isinstance(r, dict) else None
+        if ids is not None and (not isinstance(ids, list) or not ids or any(not isinstance(t, int) or t < 0 for t in ids)):
+            raise RequestFileError(f"requests[{i}]: input_ids is a non-empty list of token ids")
+        if ids is None and (not isinstance(r, dict) or not isinstance(r.get("messages"), list) or not r["messages"]):
+            raise RequestFileError(f"requests[{i}] needs a non-empty 'messages' array (or 'input_ids')")
+        for m in r.get("messages") or []:
             if m.get("role") not in ("system", "user", "assistant", "tool") or "content" not in m:
                 raise RequestFileError(f"requests[{i}]: every message needs a role and content")
         n_lp = int(r.get("num_logprobs", top_lp))
@@ -61,7 +65,7 @@ def parse_request_file(body: Dict[str, Any]) -> List[Dict[str, Any]]:
         bias = r.get("logit_bias", body.get("logit_bias"))
         stop = r.get("stop", [])
         out.append({
-            "messages": r["messages"],
+            "messages": r.get("messages") or [], "input_ids": ids,
             "temperature": float(body.get("temperature", 1.0)), "top_p": float(body.get("top_p", 0.8)), "top_k": int(body.get("top_k", 50)),
             "seed": int(r.get("sampling_seed", body.get("sampling_seed", 42))),
             "max_tokens": int(body.get("max_generate_length", 256)),
@@ -118,7 +122,7 @@ def run_requests(llm, template, requests: List[Dict[str, Any]], multimodal=None)
     for r in requests:
         render = (lambda msgs, r=r: template.apply(msgs, r["add_generation_prompt"], None, r["enable_thinking"])) if r["apply_chat_template"] \
             else _text_of
-        prompt = _with_media(llm, multimodal, r["messages"], render)
+        prompt = r["input_ids"] if r.get("input_ids") else _with_media(llm, multimodal, r["messages"], render)
         sp = SamplingParams(max_tokens=r["max_tokens"], temperature=r["temperature"], top_k=r["top_k"], top_p=r["top_p"], seed=r["seed"],
                             logprobs=r["num_logprobs"] if r["num_logprobs"] > 0 else None, logit_bias=r["logit_bias"], guided=r["guided"],
                             context_cache_lookup=r["cache_lookup"], context_cache_commit=r["cache_commit"],
@@ -149,6 +153,7 @@ def main(argv=None) -> int:
     p.add_argument("--draft-model", "--draftModel", default=None)
     p.add_argument("--dump-profile", "--dumpProfile", action="store_true")
     p.add_argument("--device", default=None)
+    p.add_argument("--dtype", default=None, choices=["bfloat16", "float16", "float32"], help="compute type instead of the checkpoint's own")
     a = p.parse_args(argv)
     from .. import profiling as prof
     from ..chat_template import ChatTemplate
@@ -162,10 +167,12 @@ def main(argv=None) -> int:
         return 1
     try:
         tok = rt.Tokenizer.load_from_hf(a.model_dir)
-    except Exception as e:       # a checkpoint without tokenizer files can still run token-id free text through the fallback below
-        print(f"no tokenizer in {a.model_dir}: {e}", file=sys.stderr)
-        return 1
-    llm = LLM(a.model_dir, device=a.device, max_batch_size=a.max_batch_size, tokenizer=tok, draft_model=a.draft_model)
+    except Exception as e:       # requests given as token ids need no tokenizer
+        if any(not r["input_ids"] for r in requests):
+            print(f"no tokenizer in {a.model_dir}: {e}", file=sys.stderr)
+            return 1
+        tok = None
+    llm = LLM(a.model_dir, device=a.device, max_batch_size=a.max_batch_size, tokenizer=tok, draft_model=a.draft_model, dtype=a.dtype)
     prof.set_profiling_enabled(a.dump_profile)
     mon = prof.MemoryMonitor().start() if a.dump_profile else None
     try:

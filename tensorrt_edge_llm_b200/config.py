@@ -37,6 +37,7 @@ AWQ_GROUP = 128
 LAYER_ATTENTION = "attention"
 LAYER_MAMBA = "mamba"
 LAYER_GDN = "gdn"
+LAYER_MLSTM = "mlstm"
 LAYER_MLP = "mlp"
 LAYER_MOE = "moe"
 
@@ -175,6 +176,83 @@ class GdnConfig:
         return 2 * self.key_dim + self.value_dim
 
 
+def pad_head(dim: int, multiples=(64, 128, 256)) -> int:
+    """Head size the kernels see: the next of ``multiples``, beyond them the next multiple of 64.  The extra features come from zero
+    projection rows, so they change no product; norms over a head divide by the real size."""
+    for m in multiples:
+        if dim <= m:
+            return m
+    return (dim + 63) // 64 * 64
+
+
+@dataclass
+class MlstmConfig:
+    """Matrix-memory LSTM mixer geometry."""
+
+    num_heads: int = 8
+    head_k_dim: int = 128
+    head_v_dim: int = 128
+    gate_cap: float = 15.0           # gate pre-activations pass cap * tanh(x / cap)
+
+    @property
+    def k_pad(self) -> int:
+        return pad_head(self.head_k_dim)
+
+    @property
+    def v_pad(self) -> int:
+        return (self.head_v_dim + 127) // 128 * 128
+
+
+@dataclass
+class AttentionConfig:
+    """Geometry of one attention layer in stacks whose layers differ from one another."""
+
+    num_heads: int = 8
+    num_kv_heads: int = 8
+    head_dim: int = 128              # query / key size
+    v_head_dim: int = 128
+    rotary_dim: int = 128            # leading features of a head that rotate (rotate-half pairs)
+    rope_theta: float = 10000.0
+    scale: float = 0.0               # multiplies q·k
+    chunk: int = 0                   # > 0: position i sees j <= i only inside its own block of `chunk` positions
+    zero_sink: bool = False          # the softmax denominator holds one more term, exp(0), without a value
+
+    @property
+    def pad(self) -> int:
+        """One padded size serves keys and values: they share the pages of the cache."""
+        return pad_head(max(self.head_dim, self.v_head_dim))
+
+
+@dataclass
+class MoeConfig:
+    """Mixture-of-experts block of one layer in stacks whose layers differ from one another."""
+
+    num_experts: int = 8
+    top_k: int = 2
+    intermediate_size: int = 64
+    limit: float = 7.0               # clamped gated unit: gate <= limit, |up| <= limit
+    alpha: float = 1.702             # gate * sigmoid(alpha * gate) * (up + 1)
+
+    @property
+    def inter_pad(self) -> int:
+        return (self.intermediate_size + 63) // 64 * 64
+
+
+@dataclass
+class LayerConfig:
+    """One layer of a stack described layer by layer: its mixer and its feed-forward (None = none)."""
+
+    kind: str = LAYER_ATTENTION
+    attention: Optional[AttentionConfig] = None
+    mlstm: Optional[MlstmConfig] = None
+    moe: Optional[MoeConfig] = None
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "LayerConfig":
+        sub = lambda c, v: c(**v) if isinstance(v, dict) else v
+        return cls(d["kind"], sub(AttentionConfig, d.get("attention")), sub(MlstmConfig, d.get("mlstm")), sub(MoeConfig, d.get("moe")))
+
+
 @dataclass
 class ModelConfig:
     """Architecture description of a decoder (dense, MoE or hybrid)."""
@@ -232,6 +310,14 @@ class ModelConfig:
     mlp_types: List[str] = field(default_factory=list)     # "mlp" / "moe" / "none" per layer
     mamba: Optional[MambaConfig] = None
     gdn: Optional[GdnConfig] = None
+    # Stacks described layer by layer.  `layer_specs` holds the distinct layers; the stack executes layer *runs*: layers
+    # loop_start .. loop_stop - 1 run loop_times times in a row with the same weights.  Every run has its own cache or state, so
+    # `num_hidden_layers` and `layer_types` count runs.
+    layer_specs: List[LayerConfig] = field(default_factory=list)
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 1
+    residual_mult: float = 1.0              # the residual stream advances by this multiple of a layer's output
     diffusion: Optional[DiffusionConfig] = None      # block-diffusion checkpoints (model_type "diffusion_gemma")
     # draft heads
     draft_type: Optional[str] = None        # "eagle3" / "mtp"
@@ -314,6 +400,23 @@ class ModelConfig:
     def compute_dtype(self) -> torch.dtype:
         return {"bfloat16": torch.bfloat16, "float16": torch.float16,
                 "float32": torch.float32}[self.dtype]
+
+    @property
+    def layer_run_ids(self) -> List[int]:
+        """Index into ``layer_specs`` of every layer run, in execution order."""
+        n = len(self.layer_specs)
+        if self.loop_stop <= self.loop_start:
+            return list(range(n))
+        body = list(range(self.loop_start, self.loop_stop))
+        return list(range(self.loop_start)) + body * self.loop_times + list(range(self.loop_stop, n))
+
+    def kv_geometry(self) -> Optional[List[tuple]]:
+        """``(kv heads, head size)`` of every attention layer's cache when the layers carry their own geometry, else ``None`` (the
+        model-wide sizes apply)."""
+        if not self.layer_specs:
+            return None
+        specs = [self.layer_specs[i] for i in self.layer_run_ids]
+        return [(sp.attention.num_kv_heads, sp.attention.pad) for sp in specs if sp.kind == LAYER_ATTENTION]
 
     def kv_donor(self, layer_idx: int) -> int:
         """The layer whose KV cache ``layer_idx`` attends over, or -1 when it writes and reads its own."""
@@ -398,6 +501,8 @@ class ModelConfig:
             d["mamba"] = MambaConfig(**d["mamba"])
         if isinstance(d.get("gdn"), dict):
             d["gdn"] = GdnConfig(**d["gdn"])
+        if d.get("layer_specs"):
+            d["layer_specs"] = [LayerConfig.from_dict(x) if isinstance(x, dict) else x for x in d["layer_specs"]]
         if isinstance(d.get("diffusion"), dict):
             d["diffusion"] = DiffusionConfig(**d["diffusion"])
         known = {f.name for f in dataclasses.fields(cls)}
@@ -407,6 +512,8 @@ class ModelConfig:
     @classmethod
     def from_hf_dict(cls, hf: Dict[str, Any], quant: Optional[QuantConfig] = None,
                      has_qk_norm: Optional[bool] = None) -> "ModelConfig":
+        if str(hf.get("architecture", "")) == "Dimesun":
+            return _parse_dimesun(cls, hf, quant)
         llm = hf.get("text_config", hf)
         model_type = llm.get("model_type", hf.get("model_type", "llama"))
         heads = int(llm["num_attention_heads"])
@@ -507,7 +614,8 @@ class ModelConfig:
         return cfg
 
     @classmethod
-    def from_pretrained(cls, model_dir: str, mapping: Optional[Mapping] = None) -> "ModelConfig":
+    def from_pretrained(cls, model_dir: str, mapping: Optional[Mapping] = None, dtype: Optional[str] = None) -> "ModelConfig":
+        """``dtype`` overrides the compute type that the checkpoint names."""
         hf = load_config_dict(model_dir)
         gen_path = os.path.join(model_dir, "generation_config.json")
         if hf.get("model_type") == "diffusion_gemma" and os.path.exists(gen_path) and "generation_config" not in hf:
@@ -517,6 +625,10 @@ class ModelConfig:
         cfg = cls.from_hf_dict(hf, quant=quant, has_qk_norm=_detect_qk_norm(model_dir, hf))
         if mapping is not None:
             cfg.mapping = mapping
+        if dtype is not None:
+            if dtype not in ("bfloat16", "float16", "float32"):
+                raise ValueError(f"unknown compute type {dtype!r}")
+            cfg.dtype = dtype
         return cfg
 
 
@@ -659,6 +771,51 @@ def _parse_gemma(llm: Dict[str, Any], n_layers: int) -> Dict[str, Any]:
     if llm.get("attn_logit_softcapping"):
         raise ValueError("attention logit soft-capping (Gemma 2) is not supported by the attention kernels")
     return out
+
+
+def _parse_dimesun(cls, hf: Dict[str, Any], quant: Optional["QuantConfig"]) -> "ModelConfig":
+    """Dimesun: parallel layers (one norm, mixer and experts side by side) listed one by one, mLSTM or chunked attention as the mixer,
+    an optional loop over a span of the layers, fp32 residual stream, tied embeddings."""
+    specs: List[LayerConfig] = []
+    for i, entry in enumerate(hf["layers"]):
+        m, f, kind = entry["mixer"], entry.get("mlp"), str(entry["type"])
+        spec = LayerConfig(kind=kind)
+        if kind == LAYER_MLSTM:
+            spec.mlstm = MlstmConfig(num_heads=int(m["heads"]), head_k_dim=int(m["dim"]), head_v_dim=int(m["vdim"]), gate_cap=float(m["gate_cap"]))
+        elif kind == LAYER_ATTENTION:
+            rot = m.get("rot") or {}
+            spec.attention = AttentionConfig(
+                num_heads=int(m["heads"]), num_kv_heads=int(m["kv_heads"]), head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]),
+                rotary_dim=int(rot.get("dims", 0)), rope_theta=float(rot.get("base", 10000.0)), scale=float(m["scale"]),
+                chunk=int((m.get("mask") or {}).get("size", 0)), zero_sink=True)
+            a = spec.attention
+            if a.num_heads % a.num_kv_heads or a.rotary_dim % 2 or a.rotary_dim > a.head_dim:
+                raise ValueError(f"layer {i}: query heads must be a multiple of the KV heads, and the rotary size even and within the head")
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        if f:
+            if f.get("kind", "moe") != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+            spec.moe = MoeConfig(num_experts=int(f["router"]["experts"]), top_k=int(f["router"]["top"]), intermediate_size=int(f["expert"]["ff"]),
+                                 limit=float(f["expert"]["limit"]))
+            if not 0 < spec.moe.top_k <= spec.moe.num_experts:
+                raise ValueError(f"layer {i}: a token uses between one and all of the experts")
+        specs.append(spec)
+    loop = hf.get("loop") or {}
+    start, stop, times = int(loop.get("start", 0)), int(loop.get("stop", 0)), int(loop.get("times", 1))
+    if loop and not (0 <= start < stop <= len(specs) and times >= 1):
+        raise ValueError("the loop must span layers of the stack and run at least once")
+    attn = next((sp.attention for sp in specs if sp.attention), AttentionConfig(1, 1, 64, 64))
+    probe = cls(layer_specs=specs, loop_start=start, loop_stop=stop, loop_times=times, num_hidden_layers=1, layer_types=[LAYER_ATTENTION])
+    runs = [specs[i] for i in probe.layer_run_ids]
+    torch_dtype = str(hf.get("torch_dtype", hf.get("dtype", "bfloat16"))).replace("torch.", "")
+    return cls(model_type="dimesun", vocab_size=int(hf["vocab"]), hidden_size=int(hf["width"]), intermediate_size=0,
+               num_hidden_layers=len(runs), num_attention_heads=attn.num_heads, num_key_value_heads=attn.num_kv_heads, head_dim=attn.pad,
+               rms_norm_eps=float(hf["norm"]["eps"]), rope_theta=attn.rope_theta, tie_word_embeddings=True,
+               dtype=torch_dtype if torch_dtype in ("bfloat16", "float16", "float32") else "bfloat16",
+               layer_types=[sp.kind for sp in runs], mlp_types=[LAYER_MOE if sp.moe else "none" for sp in runs],
+               layer_specs=specs, loop_start=start, loop_stop=stop, loop_times=times, residual_mult=float(hf["residual_mult"]),
+               quant=quant or QuantConfig(), bos_token_id=hf.get("bos_token_id"), eos_token_id=hf.get("eos_token_id"))
 
 
 def _parse_dspark(llm: dict, hf: dict) -> dict:
@@ -867,6 +1024,25 @@ def tiny_llama_config(**over: Any) -> ModelConfig:
     base = dict(model_type="llama", vocab_size=32000, hidden_size=256, intermediate_size=688,
                 num_hidden_layers=2, num_attention_heads=4, num_key_value_heads=2, head_dim=64,
                 rms_norm_eps=1e-6, rope_theta=1e4, dtype="float32", max_position_embeddings=2048)
+    base.update(over)
+    return ModelConfig(**base)
+
+
+def dimesun_config(layers: int = 12, hidden: int = 2048, vocab: int = 131072, heads: int = 16, experts: int = 64, top_k: int = 4, inter: int = 768,
+                   chunk: int = 2048, **over: Any) -> ModelConfig:
+    """Dimesun at the sizes of a small production model: every third layer chunked attention (``heads`` query heads, four per KV
+    head, d 128), the others mLSTM (``heads`` heads, 128 x 128), all with experts; no loop unless given."""
+    specs = []
+    for i in range(layers):
+        moe = MoeConfig(experts, top_k, inter, 7.0)
+        if i % 3 == 2:
+            specs.append(LayerConfig(LAYER_ATTENTION, attention=AttentionConfig(heads, max(heads // 4, 1), 128, 128, 128, 1e6, 128 ** -0.5, chunk, True),
+                                     moe=moe))
+        else:
+            specs.append(LayerConfig(LAYER_MLSTM, mlstm=MlstmConfig(heads, 128, 128, 15.0), moe=moe))
+    base = dict(model_type="dimesun", vocab_size=vocab, hidden_size=hidden, intermediate_size=0, num_hidden_layers=layers,
+                num_attention_heads=heads, num_key_value_heads=max(heads // 4, 1), head_dim=128, rms_norm_eps=1e-6, tie_word_embeddings=True,
+                layer_types=[sp.kind for sp in specs], mlp_types=[LAYER_MOE] * layers, layer_specs=specs, residual_mult=0.5)
     base.update(over)
     return ModelConfig(**base)
 

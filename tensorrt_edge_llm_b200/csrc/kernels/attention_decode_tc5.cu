@@ -39,6 +39,7 @@ struct DecParams {
     int max_pages, page_size;
     int hq, hkv, group;
     int splits, total_tokens, window;
+    int chunk;                      // chunked mask: a token sees only keys of its own `chunk`-token block (0 = none)
     int num_seqs, num_items;        // items = sequences x KV heads x splits, walked by persistent CTAs
     float scale_log2;
     const float* sinks;             // [Hq] fp32 per-head sink logits (natural-log units), or null
@@ -94,6 +95,7 @@ __device__ __forceinline__ DecItem decode_item(const DecParams& p, int item) {
     const int kv_end = it.past + it.qlen;
     int tile_lo = 0;
     if (p.window > 0) tile_lo = max(0, it.past - p.window + 1) / kDecTile;
+    if (p.chunk > 0) tile_lo = max(tile_lo, it.past / p.chunk * p.chunk / kDecTile);
     const int tile_hi = (kv_end + kDecTile - 1) / kDecTile;
     const int per = (tile_hi - tile_lo + p.splits - 1) / p.splits;
     it.j0 = tile_lo + it.split * per;
@@ -374,10 +376,16 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
             if (it.qlen <= 0) continue;
             const int ncol = it.qlen * p.group;         // live columns (<= NC)
             float m_used[NC], l_part[NC];
+            int key_lo[NC];                             // first key of the column's block (chunked mask)
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
                 m_used[c] = -INFINITY;
                 l_part[c] = 0.f;
+                key_lo[c] = 0;
+            }
+            if (p.chunk > 0) {
+#pragma unroll
+                for (int c = 0; c < NC; ++c) key_lo[c] = (it.past + (c >> gshift)) / p.chunk * p.chunk;
             }
             const uint32_t o_addr = lane_addr + kOCol + (ig & 1) * 16;
             for (int j = 0; j < it.ntiles && ok; ++j, ++jg) {
@@ -402,6 +410,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
                         const int qi = c >> gshift;
                         bool vis = tk <= it.past + qi;
                         if (p.window > 0) vis = vis && tk > it.past + qi - p.window;
+                        vis = vis && tk >= key_lo[c];
                         s[c] = vis ? __uint_as_float(raw[c]) * scale_log2 : -INFINITY;
                         const float wm = warp_max_f32(s[c]);
                         if (lane == c) red[(warp - 2) * 16 + c] = wm;
@@ -613,7 +622,7 @@ extern "C" int telb_paged_attention_decode_traced(const void* q, const void* kv_
                                                   int total_tokens, int max_q_len, int num_pages, int max_pages, int page_size,
                                                   int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                                                   long long ws_floats, int is_bf16, int* status, unsigned long long* trace,
-                                                  const float* sinks, cudaStream_t stream);
+                                                  const float* sinks, int chunk, cudaStream_t stream);
 
 // Decode-shaped steps only: max_q_len * (Hq/Hkv) <= 16.  Same tensors as telb_paged_attention.
 extern "C" int telb_paged_attention_decode(const void* q, const void* kv_layer, void* out, const int* q_start,
@@ -623,14 +632,14 @@ extern "C" int telb_paged_attention_decode(const void* q, const void* kv_layer, 
                                            long long ws_floats, int is_bf16, int* status, cudaStream_t stream) {
     return telb_paged_attention_decode_traced(q, kv_layer, out, q_start, q_len, past_len, page_table, num_seqs, total_tokens, max_q_len,
                                               num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16,
-                                              status, nullptr, nullptr, stream);
+                                              status, nullptr, nullptr, 0, stream);
 }
 
 static int decode_impl(const void* q, const void* kv_layer, void* out, void* oq, void* osf, const float* ogs, const int* q_start,
                        const int* q_len, const int* past_len, const int* page_table, int num_seqs, int total_tokens, int max_q_len,
                        int num_pages, int max_pages, int page_size, int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                        long long ws_floats, int is_bf16, int* status, unsigned long long* trace, const float* sinks, const float* kv_scales,
-                       cudaStream_t stream);
+                       int chunk, cudaStream_t stream);
 
 // Same call with a timeline buffer (3 x 64 x 4 u64, zeroed by the caller) filled by the first CTA.
 extern "C" int telb_paged_attention_decode_traced(const void* q, const void* kv_layer, void* out, const int* q_start,
@@ -638,9 +647,9 @@ extern "C" int telb_paged_attention_decode_traced(const void* q, const void* kv_
                                                   int total_tokens, int max_q_len, int num_pages, int max_pages, int page_size,
                                                   int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                                                   long long ws_floats, int is_bf16, int* status, unsigned long long* trace,
-                                                  const float* sinks, cudaStream_t stream) {
+                                                  const float* sinks, int chunk, cudaStream_t stream) {
     return decode_impl(q, kv_layer, out, nullptr, nullptr, nullptr, q_start, q_len, past_len, page_table, num_seqs, total_tokens, max_q_len,
-                       num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, trace, sinks, nullptr, stream);
+                       num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, trace, sinks, nullptr, chunk, stream);
 }
 
 // Decode attention whose output is written as NVFP4 only (packed codes out_xq [T, Hq * D / 2], atom-layout scales out_sf over
@@ -653,7 +662,7 @@ extern "C" int telb_paged_attention_decode_quant(const void* q, const void* kv_l
                                                  int is_bf16, int* status, const float* sinks, cudaStream_t stream) {
     if (!out_xq || !out_sf || !out_global_scale) return fail("telb_paged_attention_decode_quant: output buffers and scale are required");
     return decode_impl(q, kv_layer, nullptr, out_xq, out_sf, out_global_scale, q_start, q_len, past_len, page_table, num_seqs, total_tokens,
-                       max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, nullptr, sinks, nullptr, stream);
+                       max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, nullptr, sinks, nullptr, 0, stream);
 }
 
 // Decode attention over FP8 (E4M3) cache pages read in place: `q8` is the query tensor cast to E4M3 [T, Hq, D], `kv_layer` the
@@ -670,14 +679,14 @@ extern "C" int telb_paged_attention_decode_fp8(const void* q8, const void* kv_la
     if (out_xq && (!out_sf || !out_global_scale)) return fail("telb_paged_attention_decode_fp8: NVFP4 output needs its scale buffers");
     return decode_impl(q8, kv_layer, out, out_xq, out_sf, out_global_scale, q_start, q_len, past_len, page_table, num_seqs, total_tokens,
                        max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, nullptr,
-                       sinks, kv_scales, stream);
+                       sinks, kv_scales, 0, stream);
 }
 
 static int decode_impl(const void* q, const void* kv_layer, void* out, void* oq, void* osf, const float* ogs, const int* q_start,
                        const int* q_len, const int* past_len, const int* page_table, int num_seqs, int total_tokens, int max_q_len,
                        int num_pages, int max_pages, int page_size, int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                        long long ws_floats, int is_bf16, int* status, unsigned long long* trace, const float* sinks, const float* kv_scales,
-                       cudaStream_t stream) {
+                       int chunk, cudaStream_t stream) {
     if (num_seqs <= 0 || total_tokens <= 0) return 0;
     if (d != 128) return fail("telb_paged_attention_decode: head_dim must be 128");
     if (page_size != 64 && page_size != 128) return fail("telb_paged_attention_decode: page size must be 64 or 128");
@@ -704,6 +713,7 @@ static int decode_impl(const void* q, const void* kv_layer, void* out, void* oq,
     p.group = group;
     p.total_tokens = total_tokens;
     p.window = window;
+    p.chunk = chunk > 0 ? chunk : 0;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.status = status;
     p.trace = trace;

@@ -1,0 +1,121 @@
+// Paged grouped-query attention on the CUDA cores, for the element type and head sizes that the tcgen05 kernels do not take
+// (fp32 caches, heads wider than 256).  Same tensors and masks as the tile kernel of attention_tc5_extra.cu: causal, sliding
+// window, chunked (a row sees only keys of its own `chunk`-token block, counted from position 0) and sink logits.
+//
+// One warp per (token, query head): 32 keys at a time, one key per lane for the scores, then one slice of the head per lane for
+// the weighted values, with a running maximum.  Everything after the loads is fp32.
+#include "host_utils.h"
+#include "tc5_common.cuh"
+
+namespace telb {
+
+struct SimtAttnParams {
+    const void* q;
+    const void* kv;
+    void* out;
+    const int* q_start;
+    const int* past_len;
+    const int* seq_ids;
+    const int* page_table;
+    int tokens, max_pages, page_size, hq, hkv, d, window, chunk;
+    float scale;
+    const float* sinks;
+};
+
+template <typename T, int E>                             // E: head features per lane, d <= 32 E
+__global__ void __launch_bounds__(128) attn_simt_kernel(const __grid_constant__ SimtAttnParams p) {
+    pdl_prologue();
+    extern __shared__ float s_q[];                       // [4 warps][d]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const long long wid = (long long)blockIdx.x * 4 + warp;
+    if (wid >= (long long)p.tokens * p.hq) return;
+    const int t = (int)(wid / p.hq), h = (int)(wid - (long long)t * p.hq);
+    const int kvh = h / (p.hq / p.hkv);
+    const int seq = p.seq_ids[t];
+    const int pos = p.past_len[seq] + (t - p.q_start[seq]);
+    const T* q = reinterpret_cast<const T*>(p.q) + ((size_t)t * p.hq + h) * p.d;
+    float* sq = s_q + warp * p.d;
+    for (int i = lane; i < p.d; i += 32) sq[i] = Cvt<T>::to_f(q[i]);
+    __syncwarp();
+    int lo = 0;
+    if (p.window > 0) lo = max(lo, pos - p.window + 1);
+    if (p.chunk > 0) lo = max(lo, pos / p.chunk * p.chunk);
+    const T* kv = reinterpret_cast<const T*>(p.kv);
+    const int* pages = p.page_table + (size_t)seq * p.max_pages;
+    float m = p.sinks ? p.sinks[h] : -INFINITY;
+    float l = p.sinks ? 1.f : 0.f;
+    float acc[E];
+#pragma unroll
+    for (int e = 0; e < E; ++e) acc[e] = 0.f;
+    for (int j0 = lo; j0 <= pos; j0 += 32) {
+        const int j = j0 + lane;
+        const int page = j <= pos ? pages[j / p.page_size] : -1;
+        const size_t krow = page < 0 ? 0 : (((size_t)page * 2) * p.hkv + kvh) * p.page_size + j % p.page_size;
+        float s = -INFINITY;
+        if (page >= 0) {
+            const T* k = kv + krow * p.d;
+            float dot = 0.f;
+            for (int i = 0; i < p.d; ++i) dot = fmaf(sq[i], Cvt<T>::to_f(k[i]), dot);
+            s = dot * p.scale;
+        }
+        float mx = s;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float m_new = fmaxf(m, mx);
+        if (m_new == -INFINITY) continue;
+        const float f = m == -INFINITY ? 0.f : expf(m - m_new);
+        const float e_s = s == -INFINITY ? 0.f : expf(s - m_new);
+        float sum = e_s;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+        l = l * f + sum;
+        m = m_new;
+#pragma unroll
+        for (int e = 0; e < E; ++e) acc[e] *= f;
+        const int cnt = min(32, pos - j0 + 1);
+        for (int jj = 0; jj < cnt; ++jj) {
+            const float w = __shfl_sync(0xffffffffu, e_s, jj);
+            const unsigned long long row = __shfl_sync(0xffffffffu, (unsigned long long)krow, jj);
+            const T* v = kv + ((size_t)row + (size_t)p.hkv * p.page_size) * p.d;
+#pragma unroll
+            for (int e = 0; e < E; ++e)
+                if (e * 32 + lane < p.d) acc[e] = fmaf(w, Cvt<T>::to_f(v[e * 32 + lane]), acc[e]);
+        }
+    }
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+    T* out = reinterpret_cast<T*>(p.out) + ((size_t)t * p.hq + h) * p.d;
+#pragma unroll
+    for (int e = 0; e < E; ++e)
+        if (e * 32 + lane < p.d) out[e * 32 + lane] = Cvt<T>::from_f(acc[e] * inv);
+}
+
+template <typename T>
+static int launch_simt(const SimtAttnParams& p, cudaStream_t stream) {
+    const long long warps = (long long)p.tokens * p.hq;
+    const dim3 grid((unsigned)((warps + 3) / 4));
+    const size_t smem = (size_t)4 * p.d * sizeof(float);
+#define TELB_SIMT(E_) TELB_LAUNCH("attn_simt_kernel", (attn_simt_kernel<T, E_>), grid, dim3(128), smem, stream, p)
+    if (p.d <= 64) TELB_SIMT(2);
+    else if (p.d <= 128) TELB_SIMT(4);
+    else if (p.d <= 256) TELB_SIMT(8);
+    else if (p.d <= 512) TELB_SIMT(16);
+    else TELB_SIMT(32);
+#undef TELB_SIMT
+    TELB_CHECK_LAUNCH("attn_simt_kernel");
+    return 0;
+}
+
+}  // namespace telb
+
+using namespace telb;
+
+extern "C" int telb_paged_attention_simt(const void* q, const void* kv_layer, void* out, const int* q_start, const int* past_len, const int* seq_ids,
+                                         const int* page_table, int total_tokens, int max_pages, int page_size, int hq, int hkv, int d, float scale,
+                                         int window, int chunk, const float* sinks, int dtype, cudaStream_t stream) {
+    if (total_tokens <= 0) return 0;
+    if (d > 1024) return fail("telb_paged_attention_simt: head_dim must be at most 1024");
+    if (hkv <= 0 || hq % hkv) return fail("telb_paged_attention_simt: Hq must be a multiple of Hkv");
+    SimtAttnParams p{q, kv_layer, out, q_start, past_len, seq_ids, page_table, total_tokens, max_pages, page_size, hq, hkv, d, window, chunk, scale, sinks};
+    if (dtype == 2) return launch_simt<float>(p, stream);
+    return dtype == 1 ? launch_simt<__nv_bfloat16>(p, stream) : launch_simt<__half>(p, stream);
+}

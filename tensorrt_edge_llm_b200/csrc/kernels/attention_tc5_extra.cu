@@ -29,6 +29,7 @@ struct AttnParams {
     int splits;
     int total_tokens;
     int window;                // sliding window, 0 = none, -1 = no causal mask (every row sees every cached and new token)
+    int chunk;                 // chunked mask: a row sees only keys of its own `chunk`-token block, counted from position 0; 0 = none
     float scale_log2;          // softmax scale * log2(e)
     const float* sinks;        // [Hq] fp32 per-head sink logits (natural-log units) joining every row's softmax denominator, or null
     // Skip-softmax (BLASST tile vote): skip_thr[seq] = log2(lambda) of the sequence (lambda = S / length, -inf = dense), or null.
@@ -199,17 +200,17 @@ extern "C" int telb_paged_attention(const void* q, const void* kv_layer, void* o
                                     const int* tree_mask, int mask_words, int num_seqs, int total_tokens,
                                     int max_q_len, int num_pages, int max_pages, int page_size, int hq, int hkv, int d,
                                     float scale, int window, int splits, float* ws, long long ws_floats, int is_bf16,
-                                    int* status, const float* sinks, const float* skip_thr, int* skip_stats, cudaStream_t stream) {
+                                    int* status, const float* sinks, const float* skip_thr, int* skip_stats, int chunk, cudaStream_t stream) {
     if (num_seqs <= 0 || total_tokens <= 0) return 0;
-    if (sinks == nullptr && skip_thr == nullptr && d != 256)
+    const int group = hkv > 0 ? hq / hkv : 0;
+    if (sinks == nullptr && skip_thr == nullptr && chunk <= 0 && d != 256 && group > 0 && 128 % group == 0)
         return telb_paged_attention_dense(q, kv_layer, out, q_start, q_len, past_len, page_table, tree_mask, mask_words, num_seqs,
                                           total_tokens, max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits,
                                           ws, ws_floats, is_bf16, status, stream);
     if (d != 64 && d != 128 && d != 256) return fail("telb_paged_attention: head_dim must be 64, 128 or 256");
     if (page_size != 64 && page_size != 128) return fail("telb_paged_attention: page size must be 64 or 128");
-    if (hq % hkv) return fail("telb_paged_attention: Hq must be a multiple of Hkv");
-    const int group = hq / hkv;
-    if (group > 128 || (128 % group)) return fail("telb_paged_attention: GQA ratio must divide 128");
+    if (hkv <= 0 || hq % hkv) return fail("telb_paged_attention: Hq must be a multiple of Hkv");
+    if (group > 128) return fail("telb_paged_attention: at most 128 query heads per KV head");
     AttnParams p{};
     p.out = out;
     p.q_start = q_start;
@@ -226,6 +227,7 @@ extern "C" int telb_paged_attention(const void* q, const void* kv_layer, void* o
     p.tq = 128 / group;
     p.total_tokens = total_tokens;
     p.window = window;
+    p.chunk = chunk > 0 ? chunk : 0;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.out_bf16 = is_bf16;
     p.sinks = sinks;

@@ -790,6 +790,11 @@ extern "C" int telb_rope_kv_write(const void* qkv, void* q_out, void* kv_layer, 
                                   int max_pages, float eps, int is_bf16, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (d % 2 || d > 512) return fail("telb_rope_kv_write: head_dim must be even and <= 512");
+    if (is_bf16 == 2) {                                  // fp32 rows and cache
+        TELB_LAUNCH("rope_kv_write_kernel", (rope_kv_write_kernel<float>), dim3(tokens, hq + 2 * hkv), dim3(d / 2), 0, stream, (const float*)qkv, (float*)q_out, (float*)kv_layer, cos_sin, positions, seq_ids, q_start, past_len, page_table, kv_offsets, (const float*)q_norm_w, (const float*)k_norm_w, hq, hkv, d, rot_dim, page_size, max_pages, eps);
+        TELB_CHECK_LAUNCH("rope_kv_write_kernel");
+        return 0;
+    }
     if (rot_dim == d && d == 128 && tokens >= 1024) {
         const int blocks = (tokens + 3) / 4;             // 4 warps = 4 tokens per block
         DISPATCH_T(is_bf16, {

@@ -20,6 +20,7 @@ struct GemmParams {
     const void* residual;
     int feat_on_lane;
     int out_bf16;
+    int out_f32;        // 16-bit operands, but the fp32 sums are stored as they are (bias is fp32 then; no residual)
     float* ws;
     int* counters;
     int* status;
@@ -214,6 +215,34 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, const float 
             cptr[o] = Cvt<T>::from_f(x);
         }
     }
+}
+
+// The same chunk stored in fp32 (row-major or transposed output, fp32 bias).
+__device__ __forceinline__ void epilogue_store_f32(const GemmParams& p, const float (&v)[32], int row, int col0, int ncols_valid) {
+    float* cptr = reinterpret_cast<float*>(p.c);
+    const float* bptr = reinterpret_cast<const float*>(p.bias);
+    const float a_lane = (p.alpha && p.feat_on_lane) ? __ldg(&p.alpha[row]) : 1.f;
+    const float b_lane = (bptr && p.feat_on_lane) ? __ldg(&bptr[row]) : 0.f;
+    float o[32];
+#pragma unroll
+    for (int j = 0; j < 32; ++j) {
+        o[j] = v[j];
+        if (p.feat_on_lane) {
+            o[j] = o[j] * a_lane + b_lane;
+        } else if (j < ncols_valid) {
+            if (p.alpha) o[j] *= p.alpha[col0 + j];
+            if (bptr) o[j] += __ldg(&bptr[col0 + j]);
+        }
+    }
+    float* dst = cptr + row * p.ldc_lane + col0 * p.ldc_col;
+    if (p.ldc_col == 1 && ncols_valid == 32 && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {
+#pragma unroll
+        for (int q = 0; q < 8; ++q) reinterpret_cast<float4*>(dst)[q] = make_float4(o[4 * q], o[4 * q + 1], o[4 * q + 2], o[4 * q + 3]);
+        return;
+    }
+#pragma unroll
+    for (int j = 0; j < 32; ++j)
+        if (j < ncols_valid) dst[(long long)j * p.ldc_col] = o[j];
 }
 
 // A full 32-column chunk of one accumulator row → 64 bytes of 16-bit output, with the per-column
@@ -424,7 +453,8 @@ __device__ __forceinline__ void gemm_epilogue_role(const GemmParams& p, uint32_t
                 const int col0 = b0 + c * 32;
                 int nvalid = min(min(32, BN - c * 32), p.rows_b - col0);
                 if (row_ok && nvalid > 0) {
-                    if (p.out_bf16) epilogue_store<__nv_bfloat16>(pt, v, out_row, col0, nvalid);
+                    if (p.out_f32) epilogue_store_f32(pt, v, out_row, col0, nvalid);
+                    else if (p.out_bf16) epilogue_store<__nv_bfloat16>(pt, v, out_row, col0, nvalid);
                     else epilogue_store<__half>(pt, v, out_row, col0, nvalid);
                 }
             }
@@ -492,7 +522,8 @@ __device__ __forceinline__ void gemm_epilogue_role(const GemmParams& p, uint32_t
                     const int col0 = b0 + c * 32;
                     int nvalid = min(ncol, p.rows_b - col0);
                     if (row_ok && nvalid > 0) {
-                        if (p.out_bf16) epilogue_store<__nv_bfloat16>(pt, v, row, col0, nvalid);
+                        if (p.out_f32) epilogue_store_f32(pt, v, row, col0, nvalid);
+                        else if (p.out_bf16) epilogue_store<__nv_bfloat16>(pt, v, row, col0, nvalid);
                         else epilogue_store<__half>(pt, v, row, col0, nvalid);
                     }
                 }

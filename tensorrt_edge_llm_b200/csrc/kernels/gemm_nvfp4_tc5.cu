@@ -276,12 +276,8 @@ extern "C" int telb_gemm_nvfp4_wide_launch(const void* xq, const void* x_sf, con
                                            const void* params_blob, int pair, cudaStream_t stream);
 
 // Number of 64-element K groups the scale buffers are padded to (whole 256-element stages).
-extern "C" int telb_nvfp4_k64_pad(int k) { return ((k + 255) / 256) * 4; }
-
-// Bytes of an atom-layout scale buffer for `rows` x `k`.
-extern "C" long long telb_nvfp4_sf_bytes(long long rows, int k) {
-    return ((rows + 127) / 128) * (long long)telb_nvfp4_k64_pad(k) * 512;
-}
+extern "C" int telb_nvfp4_k64_pad(int k);
+extern "C" long long telb_nvfp4_sf_bytes(long long rows, int k);
 
 extern "C" int telb_nvfp4_swizzle_scales(const void* sf_rowmajor, void* sf_atoms, long long rows, int k,
                                          cudaStream_t stream) {

@@ -44,6 +44,7 @@ struct SkinnyParams {
     const float* alpha;              // [n_out] or null
     const void* residual;            // [m_tok, n_out] or null
     int out_bf16;
+    int out_f32;                     // store the fp32 sums (out and bias are fp32 then; no residual, no collective)
     const uint8_t* sf_w;             // NVFP4 scale atoms of the weights / activations
     const uint8_t* sf_x;
     int sf_k64;
@@ -381,7 +382,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
     float alpha = 1.f, bias = 0.f;
     if (feat_ok) {                                   // static per-feature constants: fetch while the MMAs run
         if (p.alpha) alpha = __ldg(&p.alpha[feat]);
-        if (p.bias) bias = Cvt<T>::to_f(reinterpret_cast<const T*>(p.bias)[feat]);
+        if (p.bias) bias = p.out_f32 ? __ldg(reinterpret_cast<const float*>(p.bias) + feat) : Cvt<T>::to_f(reinterpret_cast<const T*>(p.bias)[feat]);
     }
     if (is_epi) {
         s_alpha[lrow] = alpha;
@@ -438,6 +439,10 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
                     v[i] = v[i] * s_alpha[fg + i] + s_bias[fg + i];
                     if (resp) v[i] += Cvt<T>::to_f(resp[o + i]);
                 }
+                if (p.out_f32) {
+                    *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.out) + o) = make_float4(v[0], v[1], v[2], v[3]);
+                    continue;
+                }
                 uint2 u;
                 u.x = Cvt<T>::pack2(v[0], v[1]);
                 u.y = Cvt<T>::pack2(v[2], v[3]);
@@ -465,7 +470,8 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
                         float v = (have_acc ? __uint_as_float(r[j]) : 0.f) * alpha + bias;
                         const size_t o = (size_t)tok * p.n_out + feat;
                         if (resp) v += Cvt<T>::to_f(resp[o]);
-                        outp[o] = Cvt<T>::from_f(v);
+                        if (p.out_f32) reinterpret_cast<float*>(p.out)[o] = v;
+                        else outp[o] = Cvt<T>::from_f(v);
                     }
                 }
             }
@@ -528,7 +534,11 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
                         if (resp) v[i] += Cvt<T>::to_f(resp[o + i]);
                     }
                 }
-                if (vec_out && f0 + 3 < p.n_out) {
+                if (p.out_f32) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i)
+                        if (f0 + i < p.n_out) reinterpret_cast<float*>(p.out)[o + i] = v[i];
+                } else if (vec_out && f0 + 3 < p.n_out) {
                     uint2 u;
                     u.x = Cvt<T>::pack2(v[0], v[1]);
                     u.y = Cvt<T>::pack2(v[2], v[3]);
@@ -673,7 +683,7 @@ struct SkinnySwiglu {
 static int gemm_skinny_impl(int kind, const void* x, const void* x_sf, const void* w, const void* w_sf, void* out, int M,
                             int N, int K, const float* alpha, const void* bias, const void* residual, int is_bf16,
                             int* status, int force_ranks, const TelbGemmFusion* fusion, int group, cudaStream_t stream,
-                            const SkinnySwiglu* sw = nullptr) {
+                            const SkinnySwiglu* sw = nullptr, int out_f32 = 0) {
     if (M <= 0 || N <= 0 || K <= 0) return 0;
     if (sw && (M > 64 || N % 128 || residual)) return fail("telb_gemm_skinny: the SwiGLU epilogue needs M <= 64, N % 128 == 0 and no residual");
     if (M > 128) return fail("telb_gemm_skinny: M must be <= 128");
@@ -693,6 +703,7 @@ static int gemm_skinny_impl(int kind, const void* x, const void* x_sf, const voi
     p.alpha = alpha;
     p.residual = residual;
     p.out_bf16 = is_bf16;
+    p.out_f32 = out_f32;
     p.status = status;
     if (sw) {
         p.sw_xq = sw->xq;
@@ -753,6 +764,12 @@ extern "C" int telb_gemm_skinny_fused(int kind, const void* x, const void* x_sf,
                                       int* status, int force_ranks, const TelbGemmFusion* fusion, cudaStream_t stream) {
     if (kind != 0 && kind != 1) return fail("telb_gemm_skinny_fused: kind must be 0 (16-bit) or 1 (NVFP4)");
     return gemm_skinny_impl(kind, x, x_sf, w, w_sf, out, M, N, K, alpha, bias, residual, is_bf16, status, force_ranks, fusion, 0, stream);
+}
+
+// 16-bit operands, fp32 result and bias (M <= 128).
+extern "C" int telb_gemm_skinny_f32out(const void* x, const void* w, float* out, int M, int N, int K, const float* bias, int is_bf16,
+                                       int* status, cudaStream_t stream) {
+    return gemm_skinny_impl(0, x, nullptr, w, nullptr, out, M, N, K, nullptr, bias, nullptr, is_bf16, status, 0, nullptr, 0, stream, nullptr, 1);
 }
 
 // Decode-size gate/up projection with SwiGLU + NVFP4 quantisation in the epilogue (M <= 64): w holds 2 * inter rows in which

@@ -183,6 +183,9 @@ extern "C" int telb_gemm_skinny_fused(int kind, const void* x, const void* x_sf,
                                       int N, int K, const float* alpha, const void* bias, const void* residual, int is_bf16,
                                       int* status, int force_ranks, const telb::TelbGemmFusion* fusion, cudaStream_t stream);
 
+extern "C" int telb_gemm_skinny_f32out(const void* x, const void* w, float* out, int M, int N, int K, const float* bias, int is_bf16,
+                                       int* status, cudaStream_t stream);
+
 extern "C" const char* telb_last_error() { return g_last_error; }
 
 // out[M,N] = x[M,K] · w[N,K]^T  (16-bit row-major operands, K % 8 == 0).
@@ -192,7 +195,7 @@ extern "C" const char* telb_last_error() { return g_last_error; }
 static int gemm_f16_impl(const void* x, const void* w, void* out, int M, int N, int K, const void* bias,
                          const float* alpha, const void* residual, int is_bf16, void* ws, long long ws_bytes,
                          int* counters, int n_counters, int* status, int mode, int force_splits,
-                         const TelbGemmFusion* fusion, cudaStream_t stream) {
+                         const TelbGemmFusion* fusion, cudaStream_t stream, int out_f32 = 0) {
     if (M <= 0 || N <= 0 || K <= 0) return 0;
     if (fusion && fusion->rs_world > 1 && residual) return fail("telb_gemm_f16: reduce-scatter epilogue takes no residual");
     if (K % 8) return fail("telb_gemm_f16: K must be a multiple of 8");
@@ -201,6 +204,8 @@ static int gemm_f16_impl(const void* x, const void* w, void* out, int M, int N, 
     if (fusion && M <= 128 && (fusion->rs_world <= 1 || N % 4 == 0))
         return telb_gemm_skinny_fused(0, x, nullptr, w, nullptr, out, M, N, K, alpha, bias, residual, is_bf16, status, 0, fusion, stream);
     if (fusion) mode = 1;         // otherwise the fused collectives run in the large-M layout
+    if (mode == 0 && M <= 128 && out_f32)
+        return telb_gemm_skinny_f32out(x, w, (float*)out, M, N, K, (const float*)bias, is_bf16, status, stream);
     if (mode == 0 && M <= 128)
         return telb_gemm_skinny(0, x, nullptr, w, nullptr, out, M, N, K, alpha, bias, residual, is_bf16, status, 0, stream);
     const CUtensorMapDataType dt = is_bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
@@ -214,6 +219,7 @@ static int gemm_f16_impl(const void* x, const void* w, void* out, int M, int N, 
     p.alpha = alpha;
     p.residual = residual;
     p.out_bf16 = is_bf16;
+    p.out_f32 = out_f32;
     p.ws = static_cast<float*>(ws);
     p.counters = counters;
     p.status = status;
@@ -266,6 +272,12 @@ extern "C" int telb_gemm_f16(const void* x, const void* w, void* out, int M, int
                          force_splits, nullptr, stream);
 }
 
+// 16-bit operands, fp32 result (routers, gate pre-activations, logits): out[M,N] fp32 = x · wᵀ + bias (fp32 or null).
+extern "C" int telb_gemm_f16_f32out(const void* x, const void* w, float* out, int M, int N, int K, const float* bias, int is_bf16,
+                                    int* status, cudaStream_t stream) {
+    return gemm_f16_impl(x, w, out, M, N, K, bias, nullptr, nullptr, is_bf16, nullptr, 0, nullptr, 0, status, 0, 0, nullptr, stream, 1);
+}
+
 // Same GEMM with a tensor-parallel collective fused in (see TelbGemmFusion): reduce-scatter epilogue
 // and / or all-gather prologue.  `out` is unused by the reduce-scatter form.
 extern "C" int telb_gemm_f16_fused(const void* x, const void* w, void* out, int M, int N, int K, const void* bias,
@@ -298,12 +310,11 @@ extern "C" int telb_gemm_f16_grouped(const void* x, const void* w, void* out, in
     p.tile_expert = tile_expert;
     p.group_rows_b = N;
     const int bn = N >= 256 && N % 256 == 0 ? 256 : 128;
-    if (N % bn) return fail("telb_gemm_f16_grouped: N must be a multiple of 128");
     CUtensorMap ta, tb;
     if (make_tmap_2d(&ta, dt, 2, x, rows_pad, K, (uint64_t)K * 2, kBM, kBK, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
     if (make_tmap_2d(&tb, dt, 2, w, (uint64_t)experts * N, K, (uint64_t)K * 2, bn, kBK, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
     p.tiles_a = rows_pad / kBM;
-    p.tiles_b = N / bn;
+    p.tiles_b = (N + bn - 1) / bn;      // a partial last tile reads into the next expert's rows and does not store those columns
     p.splits = 1;
     p.kb_per_split = p.kb_total;
     return bn == 256 ? launch_gemm<256, 4>(ta, tb, p, stream) : launch_gemm<128, 6>(ta, tb, p, stream);

@@ -2,6 +2,8 @@
 //
 //   moe_route          softmax over E router logits → top-k (ties → lower index) → optional renormalise
 //                      (sigmoid + group-limited top-k for DeepSeek/Nemotron-style routers)
+//   moe_route_chosen   top-k over fp32 logits, softmax over the chosen ones
+//   clamped_glu        clamped gated activation between the two expert GEMMs
 //   moe_align          per-expert counts → 128-row padded segment offsets → destination row of every
 //                      (token, k) slot → expert id of every 128-row tile (-1 = unused tile)
 //   moe_gather_quant   copy each routed token row to its destination row, quantising to NVFP4 on the way
@@ -114,6 +116,79 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, float* __restrict
             topk_w[(size_t)t * top_k + r] = my_w[r] * inv * scaling;
             topk_idx[(size_t)t * top_k + r] = my_i[r];
         }
+    }
+}
+
+// Router whose weights are the softmax over the chosen logits only: the `top_k` largest logits (ties → lower index), one warp per
+// token.  The logits are fp32 rows `ld` apart (they may be columns of a wider projection).  experts <= 1024.
+__global__ void moe_route_chosen_kernel(const float* __restrict__ logits, int ld, float* __restrict__ topk_w, int* __restrict__ topk_idx,
+                                        int tokens, int experts, int top_k) {
+    pdl_prologue();
+    const int lane = threadIdx.x & 31;
+    const int t = (int)((blockIdx.x * (long long)blockDim.x + threadIdx.x) >> 5);
+    if (t >= tokens) return;
+    const float* row = logits + (size_t)t * ld;
+    unsigned taken = 0;                                  // bit i: expert lane + 32 i is chosen
+    float first = 0.f, sum = 0.f, my = 0.f;              // lane r keeps the exponential of pick r
+    int my_i = 0;
+    for (int r = 0; r < top_k; ++r) {
+        float best = -INFINITY;
+        int bi = 0x7fffffff;
+        for (int i = 0; lane + 32 * i < experts; ++i) {
+            const float v = row[lane + 32 * i];
+            if (!((taken >> i) & 1u) && (v > best || bi == 0x7fffffff)) { best = v; bi = lane + 32 * i; }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+            if (oi != 0x7fffffff && (ov > best || (ov == best && oi < bi) || bi == 0x7fffffff)) { best = ov; bi = oi; }
+        }
+        if (r == 0) first = best;
+        const float e = expf(best - first);
+        sum += e;
+        if (lane == r) { my = e; my_i = bi; }
+        if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
+    }
+    if (lane < top_k) {
+        topk_w[(size_t)t * top_k + lane] = my / sum;
+        topk_idx[(size_t)t * top_k + lane] = my_i;
+    }
+}
+
+// Clamped gated unit over [gate I | up I] rows of the padded expert layout (or plain rows): with g = min(gate, limit) and
+// u = clamp(up, ±limit), out = g · σ(alpha g) · (u + 1).  Rows that hold no routed token are skipped.
+template <typename T>
+__global__ void clamped_glu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, const int* __restrict__ tile_rows, int rows, int inter,
+                                   float limit, float alpha) {
+    pdl_prologue();
+    const int groups = inter >> 3;
+    const long long total = (long long)rows * groups;
+    for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+        const int r = (int)(i / groups), c = (int)(i - (long long)r * groups) * 8;
+        if (tile_rows && (r & 127) >= tile_rows[r >> 7]) continue;
+        const T* src = gate_up + (size_t)r * 2 * inter + c;
+        float y[8];
+        alignas(16) T gv[8];
+        alignas(16) T uv[8];
+        constexpr int kVec = 16 / sizeof(T);
+#pragma unroll
+        for (int q = 0; q < 8 / kVec; ++q) {
+            *reinterpret_cast<uint4*>(gv + q * kVec) = *reinterpret_cast<const uint4*>(src + q * kVec);
+            *reinterpret_cast<uint4*>(uv + q * kVec) = *reinterpret_cast<const uint4*>(src + inter + q * kVec);
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const float g = fminf(Cvt<T>::to_f(gv[j]), limit);
+            const float u = fminf(fmaxf(Cvt<T>::to_f(uv[j]), -limit), limit);
+            y[j] = g / (1.f + expf(-alpha * g)) * (u + 1.f);
+        }
+        alignas(16) T ov[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ov[j] = Cvt<T>::from_f(y[j]);
+#pragma unroll
+        for (int q = 0; q < 8 / kVec; ++q)
+            *reinterpret_cast<uint4*>(out + (size_t)r * inter + c + q * kVec) = *reinterpret_cast<const uint4*>(ov + q * kVec);
     }
 }
 
@@ -273,6 +348,36 @@ extern "C" int telb_moe_route(const void* logits, float* topk_w, int* topk_idx, 
     return 0;
 }
 
+extern "C" int telb_moe_route_chosen(const float* logits, int ld, float* topk_w, int* topk_idx, int tokens, int experts, int top_k,
+                                     cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (top_k > 32 || top_k > experts || experts > 1024) return fail("telb_moe_route_chosen: top_k <= 32, experts <= 1024");
+    TELB_LAUNCH("moe_route_chosen_kernel", moe_route_chosen_kernel, dim3((tokens + 3) / 4), dim3(128), 0, stream, logits, ld, topk_w, topk_idx, tokens,
+                experts, top_k);
+    TELB_CHECK_LAUNCH("moe_route_chosen_kernel");
+    return 0;
+}
+
+// dtype: 0 fp16, 1 bf16, 2 fp32.  tile_rows (rows in use of every 128-row tile) may be null.
+extern "C" int telb_clamped_glu(const void* gate_up, void* out, const int* tile_rows, int rows, int inter, float limit, float alpha, int dtype,
+                                cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (inter % 8) return fail("telb_clamped_glu: the width must be a multiple of 8");
+    const long long total = (long long)rows * (inter / 8);
+    const long long blocks = (total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16;
+    if (dtype == 2)
+        TELB_LAUNCH("clamped_glu_kernel", (clamped_glu_kernel<float>), dim3((unsigned)blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out,
+                    tile_rows, rows, inter, limit, alpha);
+    else if (dtype == 1)
+        TELB_LAUNCH("clamped_glu_kernel", (clamped_glu_kernel<__nv_bfloat16>), dim3((unsigned)blocks), dim3(256), 0, stream,
+                    (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, tile_rows, rows, inter, limit, alpha);
+    else
+        TELB_LAUNCH("clamped_glu_kernel", (clamped_glu_kernel<__half>), dim3((unsigned)blocks), dim3(256), 0, stream, (const __half*)gate_up, (__half*)out,
+                    tile_rows, rows, inter, limit, alpha);
+    TELB_CHECK_LAUNCH("clamped_glu_kernel");
+    return 0;
+}
+
 extern "C" int telb_moe_align(const int* topk_idx, int* dst_row, int* tile_expert, int* counts_out, int slots, int experts,
                               int expert_lo, int expert_hi, int max_tiles, cudaStream_t stream) {
     if (experts > 4096) return fail("telb_moe_align: too many experts");
@@ -285,7 +390,7 @@ extern "C" int telb_moe_align(const int* topk_idx, int* dst_row, int* tile_exper
 extern "C" int telb_moe_gather(const void* x, const int* dst_row, void* out16, void* xq, void* sf, const float* global_scale,
                                int slots, int top_k, int hidden, int is_bf16, cudaStream_t stream) {
     if (slots <= 0) return 0;
-    if (hidden % 16) return fail("telb_moe_gather: hidden must be a multiple of 16");
+    if (hidden % (out16 ? 8 : 16)) return fail("telb_moe_gather: hidden must be a multiple of 16 (8 for a plain copy)");
     const int k64 = telb_nvfp4_k64_pad(hidden);
     if (is_bf16)
         TELB_LAUNCH("moe_gather_kernel", (moe_gather_kernel<__nv_bfloat16>), dim3(slots), dim3(128), 0, stream, (const __nv_bfloat16*)x,

@@ -30,7 +30,7 @@ def _ensure_builtin():
     from .models.default import CausalLM
     for t in ("llama", "qwen2", "qwen3", "mistral", "phi3", "gemma", "default"):
         _REGISTRY[t] = CausalLM
-    from .models import qwen3_moe, nemotron_h, eagle3, eagle4, mtp, gemma, diffusion_gemma, dflash, dflash2, lilicorr, dspark, tts  # noqa: F401  (register themselves)
+    from .models import qwen3_moe, nemotron_h, eagle3, eagle4, mtp, gemma, diffusion_gemma, dflash, dflash2, lilicorr, dspark, tts, dimesun  # noqa: F401  (register themselves)
 
 
 def model_class_for(cfg: ModelConfig):
@@ -71,12 +71,15 @@ class AutoModel:
         return model
 
     @staticmethod
-    def from_pretrained(model_dir: str, mapping: Optional[Mapping] = None, comm=None, device="cpu"):
+    def from_pretrained(model_dir: str, mapping: Optional[Mapping] = None, comm=None, device="cpu", dtype: Optional[str] = None):
+        """``dtype`` ("bfloat16" | "float16" | "float32") overrides the compute type the checkpoint names."""
         from .checkpoint.artifacts import is_artifact_dir, load_artifacts
         from .checkpoint.loader import load_weights
         if is_artifact_dir(model_dir):          # prepared by `trtedge build`: load the rank's tensors as stored
+            if dtype is not None:
+                raise ValueError("prepared weights keep the compute type they were prepared in")
             return load_artifacts(model_dir, mapping, comm, device)
-        cfg = ModelConfig.from_pretrained(model_dir, mapping)
+        cfg = ModelConfig.from_pretrained(model_dir, mapping, dtype)
         cls = model_class_for(cfg)
         model = cls(cfg, comm)
         load_weights(model, model_dir)

@@ -23,7 +23,7 @@ from .. import ops
 from ..config import ModelConfig
 from ..ops.meta import StepMeta
 from ..parallel.comm import LocalComm
-from .linear import NVFP4Linear, TPMode, make_linear
+from .linear import HeadLinear, NVFP4Linear, TPMode, make_linear
 
 
 class RMSNorm(nn.Module):
@@ -152,6 +152,31 @@ class Attention(nn.Module):
             # decode step into an NVFP4 projection: the attention epilogue quantises for it
             return self.o_proj(ops.cuda_ops().paged_attention_quant(q, kv_layer, meta, self.scale, self.sliding_window, gs, sinks=sinks))
         o = ops.paged_attention(q, kv_layer, meta, self.scale, self.sliding_window, sinks)
+        return self.o_proj(o.reshape(o.shape[0], -1))
+
+
+class LayerAttention(nn.Module):
+    """Attention with a geometry of its own (``AttentionConfig``): key and value sizes that may differ, partial rotary, a score scale,
+    chunked causal masking and a zero sink.  Heads are padded to a size the kernels take and share the paged cache layout; cos / sin
+    tables come from the model per (base, rotary size)."""
+
+    def __init__(self, cfg: ModelConfig, spec, prefix: str):
+        super().__init__()
+        self.spec, self.prefix = spec, prefix
+        h, d = cfg.hidden_size, spec.pad
+        self.qkv_proj = HeadLinear(h, 0, out_heads=[(spec.num_heads, spec.head_dim, d), (spec.num_kv_heads, spec.head_dim, d),
+                                                    (spec.num_kv_heads, spec.v_head_dim, d)],
+                                   sources=["q_proj", "k_proj", "v_proj"], dtype=cfg.compute_dtype)
+        self.o_proj = HeadLinear(0, h, in_heads=(spec.num_heads, spec.v_head_dim, d), dtype=cfg.compute_dtype)
+        if spec.zero_sink:
+            self.register_buffer("sinks", torch.zeros(spec.num_heads, dtype=torch.float32), persistent=False)
+        else:
+            self.sinks = None
+
+    def forward(self, x: torch.Tensor, meta: StepMeta, kv_layer: torch.Tensor, cos_sin: torch.Tensor) -> torch.Tensor:
+        sp = self.spec
+        q = ops.rope_kv_write(self.qkv_proj(x), kv_layer, meta, cos_sin, sp.num_heads, sp.num_kv_heads, sp.pad)
+        o = ops.paged_attention(q, kv_layer, meta, sp.scale, None, self.sinks, chunk=sp.chunk)
         return self.o_proj(o.reshape(o.shape[0], -1))
 
 

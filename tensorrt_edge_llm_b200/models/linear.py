@@ -125,6 +125,60 @@ class Linear(LinearBase):
         return ops.linear(x, self.weight, self.bias)
 
 
+class HeadLinear(Linear):
+    """Linear whose features are attention or recurrence heads padded to the size the kernels work on.
+
+    ``out_heads``: one ``(heads, real size, padded size)`` per source module (its checkpoint rows are ``heads x real``);
+    ``in_heads``: the same for the input features.  Padding rows and columns are zero, so padded features are zeros on the
+    way out and ignored on the way in."""
+
+    def __init__(self, in_features: int, out_features: int, out_heads=None, in_heads=None, sources=None, dtype=torch.bfloat16):
+        self.out_heads, self.in_heads = out_heads, in_heads
+        n_in = in_features if in_heads is None else in_heads[0] * in_heads[2]
+        outs = [out_features] if out_heads is None else [h * pad for h, _, pad in out_heads]
+        super().__init__(n_in, outs, dtype=dtype, sources=sources)
+
+    def _pad_in(self, w: torch.Tensor) -> torch.Tensor:
+        if self.in_heads is None:
+            return w
+        h, real, pad = self.in_heads
+        return torch.nn.functional.pad(w.reshape(w.shape[0], h, real), (0, pad - real)).reshape(w.shape[0], h * pad)
+
+    def load_from(self, tensors):
+        parts = []
+        for i, t in enumerate(tensors):
+            w = self._pad_in(t["weight"])
+            if self.out_heads is not None:
+                h, real, pad = self.out_heads[i]
+                w = torch.nn.functional.pad(w.reshape(h, real, -1), (0, 0, 0, pad - real)).reshape(h * pad, -1)
+            parts.append(w)
+        self.weight.data.copy_(torch.cat(parts, 0).to(self.weight.dtype))
+
+    @torch.no_grad()
+    def zero_padding(self) -> None:
+        """Clear the padding of a weight that was drawn at random."""
+        w = self.weight.data
+        if self.in_heads is not None:
+            h, real, pad = self.in_heads
+            w.view(w.shape[0], h, pad)[:, :, real:] = 0
+        r0 = 0
+        for h, real, pad in self.out_heads or ():
+            w[r0:r0 + h * pad].view(h, pad, -1)[:, real:] = 0
+            r0 += h * pad
+
+
+class Fp32OutLinear(Linear):
+    """Linear with 16-bit operands whose fp32 sums leave as they are: routers, gate pre-activations, logits.  Several small
+    projections of one input stack into one product (``sources`` may live in different modules)."""
+
+    def __init__(self, in_features: int, out_features, sources=None, bias: bool = False, dtype=torch.bfloat16):
+        super().__init__(in_features, out_features, dtype=dtype, sources=sources)
+        self.bias = nn.Parameter(torch.zeros(self.out_features, dtype=torch.float32), requires_grad=False) if bias else None
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return ops.linear_f32(x, self.weight, self.bias)
+
+
 class NVFP4Linear(LinearBase):
     """NVFP4 weights (E2M1 pairs, E4M3 scale per 16 inputs, fp32 ``weight_scale_2``).
 

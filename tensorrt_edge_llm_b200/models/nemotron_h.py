@@ -20,11 +20,11 @@ import torch
 from torch import nn
 
 from .. import ops
-from ..config import LAYER_ATTENTION, LAYER_GDN, LAYER_MAMBA, LAYER_MLP, LAYER_MOE, ModelConfig
+from ..config import LAYER_ATTENTION, LAYER_GDN, LAYER_MAMBA, LAYER_MLP, LAYER_MLSTM, LAYER_MOE, ModelConfig
 from ..model import register_model
 from ..ops.meta import StepMeta
 from .default import MLP, Attention, CausalLM, RMSNorm
-from .linear import TPMode, make_linear
+from .linear import HeadLinear, TPMode, make_linear
 
 
 class RecurrentState:
@@ -33,6 +33,8 @@ class RecurrentState:
     def __init__(self, cfg: ModelConfig, seats: int, device, dtype):
         tp = cfg.tp_size
         self.conv, self.ssm, self.gdn = {}, {}, {}
+        self.mlstm, self.mlstm_norm = {}, {}      # matrix memory; normaliser and running maximum
+        runs = cfg.layer_run_ids if cfg.layer_specs else None
         for i, t in enumerate(cfg.layer_types):
             if t == LAYER_MAMBA:
                 m = cfg.mamba
@@ -44,11 +46,16 @@ class RecurrentState:
                 self.conv[i] = torch.zeros(seats, g.conv_dim // tp, g.conv_kernel - 1, dtype=dtype, device=device)
                 self.gdn[i] = torch.zeros(seats, g.num_v_heads // tp, g.head_k_dim, g.head_v_dim, dtype=torch.float32, device=device)
 
+            elif t == LAYER_MLSTM:
+                m = cfg.layer_specs[runs[i]].mlstm
+                self.mlstm[i] = torch.zeros(seats, m.num_heads, m.k_pad, m.v_pad, dtype=torch.float32, device=device)
+                self.mlstm_norm[i] = torch.zeros(seats, m.num_heads, m.k_pad + 1, dtype=torch.float32, device=device)
+
     def bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for d in (self.conv, self.ssm, self.gdn) for t in d.values())
+        return sum(t.numel() * t.element_size() for t in self.pools())
 
     def pools(self):
-        for d in (self.conv, self.ssm, self.gdn):
+        for d in (self.conv, self.ssm, self.gdn, self.mlstm, self.mlstm_norm):
             yield from d.values()
 
     # ---- replay data -------------------------------------------------------------------------------------------------
@@ -246,6 +253,46 @@ class GatedDeltaNetMixer(nn.Module):
         t = qkv.shape[0]
         ops.gated_delta_rule(q.reshape(t, self.hk, g.head_k_dim), k.reshape(t, self.hk, g.head_k_dim), v.reshape(t, self.hv, g.head_v_dim),
                              a, b, self.A_log, self.dt_bias, state.gdn[layer_idx], meta)
+
+
+class MLstmMixer(nn.Module):
+    """Matrix-memory LSTM: q, k, v and the output gate from one product; the log input and forget gates arrive as fp32 columns of the
+    layer's fp32 projection (``gates``: input gates of all heads, then forget gates); state in fp32 rows indexed by seat.  Head norm
+    and output gate are part of the recurrent op."""
+
+    def __init__(self, cfg: ModelConfig, spec, prefix: str):
+        super().__init__()
+        self.spec, self.prefix, self.eps = spec, prefix, cfg.rms_norm_eps
+        h, n, dt = cfg.hidden_size, spec.num_heads, cfg.compute_dtype
+        self.qkvg_proj = HeadLinear(h, 0, out_heads=[(n, spec.head_k_dim, spec.k_pad), (n, spec.head_k_dim, spec.k_pad),
+                                                     (n, spec.head_v_dim, spec.v_pad), (n, spec.head_v_dim, spec.v_pad)],
+                                    sources=["q_proj", "k_proj", "v_proj", "g_proj"], dtype=dt)
+        self.o_proj = HeadLinear(0, h, in_heads=(n, spec.head_v_dim, spec.v_pad), dtype=dt)
+        self.out_norm = nn.Parameter(torch.ones(n * spec.v_pad, dtype=torch.float32), requires_grad=False)
+
+    @torch.no_grad()
+    def load_checkpoint(self, fetch) -> bool:
+        w = fetch(f"{self.prefix}.head_norm.weight")
+        if w is not None:
+            sp = self.spec
+            self.out_norm.zero_()
+            self.out_norm.view(sp.num_heads, sp.v_pad)[:, :sp.head_v_dim] = w.float().reshape(sp.num_heads, sp.head_v_dim)
+        return False        # the projections are loaded by the generic path
+
+    def forward(self, x, gates, meta: StepMeta, state: RecurrentState, run: int):
+        qkvg = self.qkvg_proj(x)
+        if state.record is not None:
+            state.record[run] = (qkvg, gates)
+        return self.o_proj(self._recur(qkvg, gates, meta, state, run))
+
+    def _recur(self, qkvg, gates, meta, state, run):
+        sp = self.spec
+        return ops.mlstm(qkvg, gates, self.out_norm, state.mlstm[run], state.mlstm_norm[run], meta, sp.head_k_dim ** -0.5, sp.gate_cap,
+                         self.eps, sp.head_v_dim)
+
+    @torch.no_grad()
+    def replay(self, saved, rows: torch.Tensor, meta: StepMeta, state: RecurrentState, run: int) -> None:
+        self._recur(*(t.index_select(0, rows) for t in saved), meta, state, run)
 
 
 class HybridLayer(nn.Module):

@@ -273,6 +273,70 @@ class MoEBlock(nn.Module):
         return out.to(x.dtype)
 
 
+class RoutedRows:
+    """What the experts of a step produced, before the weighted sum: rows in expert order with the tables that lead back to the tokens.
+    The kernel that advances the residual stream takes the sum itself (``ops.stream_norm``)."""
+
+    __slots__ = ("y", "ws", "weights")
+
+    def __init__(self, y, ws, weights):
+        self.y, self.ws, self.weights = y, ws, weights
+
+
+class ClampedExperts(nn.Module):
+    """Experts with a clamped gated unit (``MoeConfig``) and a router whose weights are the softmax over the chosen logits.  The fp32
+    logits come from the layer (its fp32 projection), the weighted sum is left to the consumer."""
+
+    def __init__(self, cfg: ModelConfig, spec, prefix: str):
+        super().__init__()
+        self.spec, self.prefix = spec, prefix
+        self.hidden = cfg.hidden_size
+        e, i, dt = spec.num_experts, spec.inter_pad, cfg.compute_dtype
+        # rows of an expert: gate, then up; the intermediate size is padded with zero rows / columns (a zero gate gives a zero unit)
+        self.w13 = nn.Parameter(torch.zeros(e * 2 * i, cfg.hidden_size, dtype=dt), requires_grad=False)
+        self.w2 = nn.Parameter(torch.zeros(e * cfg.hidden_size, i, dtype=dt), requires_grad=False)
+
+    @torch.no_grad()
+    def load_checkpoint(self, fetch) -> bool:
+        sp, h = self.spec, self.hidden
+        w13 = self.w13.data.view(sp.num_experts, 2, sp.inter_pad, h)
+        w2 = self.w2.data.view(sp.num_experts, h, sp.inter_pad)
+        found = False
+        for e in range(sp.num_experts):
+            g, u, d = (fetch(f"{self.prefix}.experts.{e}.{n}_proj.weight") for n in ("gate", "up", "down"))
+            if g is None:
+                continue
+            found = True
+            w13[e, 0, :sp.intermediate_size] = g.to(w13.dtype)
+            w13[e, 1, :sp.intermediate_size] = u.to(w13.dtype)
+            w2[e, :, :sp.intermediate_size] = d.to(w2.dtype)
+        return found
+
+    @torch.no_grad()
+    def random_init(self, gen: torch.Generator, std: float = 0.02) -> None:
+        sp = self.spec
+        dev = self.w13.device
+        g = torch.Generator(device=dev).manual_seed(int(torch.randint(0, 2 ** 31 - 1, (1,), generator=gen)))
+        w13 = self.w13.data.view(sp.num_experts, 2, sp.inter_pad, self.hidden)
+        w2 = self.w2.data.view(sp.num_experts, self.hidden, sp.inter_pad)
+        for e in range(sp.num_experts):
+            w13[e].normal_(0.0, std, generator=g)[:, sp.intermediate_size:] = 0
+            w2[e].normal_(0.0, std, generator=g)[:, sp.intermediate_size:] = 0
+
+    def forward(self, x: torch.Tensor, logits: torch.Tensor):
+        """``x`` ``[T, hidden]`` and fp32 router logits ``[T, experts]`` (may be a column slice) → :class:`RoutedRows`."""
+        sp = self.spec
+        w, idx = ops.moe_route_chosen(logits, sp.top_k)
+        if not x.is_cuda:
+            return ops.ref.clamped_experts(x, self.w13.view(sp.num_experts, -1, self.hidden), self.w2.view(sp.num_experts, self.hidden, -1), w, idx,
+                                           sp.limit, sp.alpha)
+        cu = ops.cuda_ops()
+        ws = cu.moe_align(idx, sp.num_experts, 0, sp.num_experts)
+        h1 = cu.gemm_grouped(cu.moe_gather(x, ws, sp.top_k, None), self.w13, ws, sp.num_experts)
+        y = cu.gemm_grouped(cu.clamped_glu(h1, sp.limit, sp.alpha, ws), self.w2, ws, sp.num_experts)
+        return RoutedRows(y, ws, w)
+
+
 class MoEDecoderLayer(nn.Module):
     def __init__(self, cfg: ModelConfig, layer_idx: int):
         super().__init__()

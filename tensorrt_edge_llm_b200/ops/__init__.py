@@ -140,10 +140,46 @@ def rope_q(q, kv_layer, meta, cos_sin, num_q_heads, head_dim, q_norm_w=None, eps
     return ref.rope_q(q, meta, cos_sin, num_q_heads, head_dim, q_norm_w, eps)
 
 
-def paged_attention(q, kv_layer, meta, scale, sliding_window=None, sinks=None, causal=True):
+def paged_attention(q, kv_layer, meta, scale, sliding_window=None, sinks=None, causal=True, chunk=0):
+    """``chunk`` > 0: row at position ``i`` sees only keys ``j`` with ``j // chunk == i // chunk`` (and ``j <= i``)."""
     if q.is_cuda:
-        return cuda_ops().paged_attention(q, kv_layer, meta, scale, sliding_window, sinks, causal=causal)
-    return ref.paged_attention(q, kv_layer, meta, scale, sliding_window, sinks, causal=causal)
+        return cuda_ops().paged_attention(q, kv_layer, meta, scale, sliding_window, sinks, causal=causal, chunk=chunk)
+    return ref.paged_attention(q, kv_layer, meta, scale, sliding_window, sinks, causal=causal, chunk=chunk)
+
+
+def linear_f32(x, weight, bias=None):
+    """``x · weightᵀ (+ bias)`` with the fp32 sums as the result."""
+    if x.is_cuda:
+        return cuda_ops().gemm_f32out(x, weight, bias)
+    y = x.float() @ weight.float().t()
+    return y if bias is None else y + bias.float()
+
+
+def stream_norm(stream, weight, eps, *, delta=None, routed=None, mult=1.0, step=None, offset=0.0, ids=None, table=None, dtype=None):
+    """Advance the fp32 residual stream and normalise it for the next layer: returns ``(stream, h)``.
+
+    ``stream`` (or ``table[ids]`` when it is ``None``) ``+ mult * (delta + routed) + step``; ``h`` is its RMS norm times
+    ``offset + weight`` in the activation type (``None`` without ``weight``).  ``routed`` is a mixture block's output: a dense tensor,
+    or :class:`models.qwen3_moe.RoutedRows`, whose weighted sum the kernel takes itself."""
+    t = ids if stream is None else stream
+    if t.is_cuda:
+        return cuda_ops().stream_norm(stream, weight, eps, delta, routed, mult, step, offset, ids, table, dtype)
+    return ref.stream_norm(stream, weight, eps, delta, routed, mult, step, offset, ids, table, dtype)
+
+
+def moe_route_chosen(logits, top_k):
+    """The ``top_k`` largest fp32 logits per row and the softmax over them: ``(weights, indices)``."""
+    if logits.is_cuda:
+        return cuda_ops().moe_route_chosen(logits, top_k)
+    return ref.moe_route_chosen(logits, top_k)
+
+
+def mlstm(qkvg, gates, norm_w, state, norm_state, meta, scale, cap, eps, dv_real):
+    """Matrix-memory LSTM over packed ``[q | k | v | g]`` rows with head norm and output gate: ``[T, heads · dv]``.  ``state``
+    ``[seats, heads, dk, dv]`` and ``norm_state`` ``[seats, heads, dk + 1]`` (normaliser, running maximum) are advanced in place."""
+    if qkvg.is_cuda:
+        return cuda_ops().mlstm(qkvg, gates, norm_w, state, norm_state, meta, scale, cap, eps, dv_real)
+    return ref.mlstm(qkvg, gates, norm_w, state, norm_state, meta, scale, cap, eps, dv_real)
 
 
 def kv_fp8_prepare(kv_layer, meta, scales, dtype, window=0):

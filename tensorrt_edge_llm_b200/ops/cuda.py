@@ -17,6 +17,7 @@ from .meta import StepMeta
 
 _LIB_PATH = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "_lib", "libtelb_kernels.so")
 _lib: Optional[ctypes.CDLL] = None
+KERNEL_FAMILY = ""       # a family whose own kernel library (build.KERNEL_SETS) serves this process when the whole one is not built
 
 c_int, c_ll, c_float, c_vp = ctypes.c_int, ctypes.c_longlong, ctypes.c_float, ctypes.c_void_p
 
@@ -28,6 +29,11 @@ def lib() -> ctypes.CDLL:
         # cpp/kernels/cuteDslModuleLoader.cpp:178): the named library "fails to load" deterministically
         if os.environ.get("TELB_TEST_FAIL_KERNEL_LIBRARY", "") in ("1", os.path.basename(_LIB_PATH)):
             raise RuntimeError(f"native kernel library {_LIB_PATH} failed to load (TELB_TEST_FAIL_KERNEL_LIBRARY is set)")
+        if KERNEL_FAMILY and not os.path.exists(_LIB_PATH):
+            from ..build import kernel_library
+            _lib = ctypes.CDLL(kernel_library(KERNEL_FAMILY))
+            _lib.telb_last_error.restype = ctypes.c_char_p
+            return _lib
         if not os.path.exists(_LIB_PATH):
             raise RuntimeError(f"native kernel library not built: {_LIB_PATH} (run `python -m tensorrt_edge_llm_b200.build`)")
         _lib = ctypes.CDLL(_LIB_PATH)
@@ -86,6 +92,11 @@ def _is_bf16(t: torch.Tensor) -> int:
     if t.dtype == torch.float16:
         return 0
     raise TypeError(f"CUDA kernels take fp16 / bf16 activations, got {t.dtype}")
+
+
+def _dtype_code(t: torch.Tensor) -> int:
+    """0 fp16, 1 bf16, 2 fp32: the kernels that also run in 32 bits."""
+    return 2 if t.dtype == torch.float32 else _is_bf16(t)
 
 
 class Workspace:
@@ -228,6 +239,10 @@ def gemm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = N
     n = weight.shape[0]
     if weight.dtype != x.dtype:
         raise TypeError(f"gemm: activation {x.dtype} and weight {weight.dtype} differ")
+    if x.dtype == torch.float32:                  # true fp32 on the CUDA cores (the tensor cores have no fp32 operands)
+        if alpha is not None or residual is not None:
+            raise TypeError("gemm: the fp32 product takes no column scale and no residual")
+        return gemm_f32out(x2, weight, bias, out).reshape(*lead, n)
     if k % 8:
         # rows must be 16-byte multiples for the TMA descriptors: zero columns up to the next multiple of 8 change nothing
         # (patch embeddings with 3 · 14 · 14 = 588 inputs are the case in practice; the padded copies are made per call)
@@ -243,6 +258,54 @@ def gemm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = N
                                _p(ws.counters), c_int(ws.counters.numel()), _p(ws.status), c_int(mode), c_int(splits),
                                _stream()), "gemm")
     return out.reshape(*lead, n)
+
+
+def gemm_f32out(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[M,N]`` fp32 ``= x · weightᵀ (+ bias)``: tensor-core product of 16-bit operands, or the fp32 kernel for fp32 operands.
+    ``bias`` is fp32."""
+    x2 = x if x.is_contiguous() else x.contiguous()
+    m, k = x2.shape
+    n = weight.shape[0]
+    if weight.dtype != x.dtype or (bias is not None and bias.dtype != torch.float32):
+        raise TypeError(f"gemm_f32out: activation {x.dtype}, weight {weight.dtype}, bias {None if bias is None else bias.dtype}")
+    if out is None:
+        out = torch.empty(m, n, dtype=torch.float32, device=x.device)
+    if x.dtype == torch.float32:
+        _check(lib().telb_gemm_f32(_p(x2), _p(weight), _p(out), c_int(m), c_int(n), c_int(k), _p(bias), _stream()), "gemm_f32")
+        return out
+    if k % 8:
+        pad = 8 - k % 8
+        x2, weight = torch.nn.functional.pad(x2, (0, pad)), torch.nn.functional.pad(weight, (0, pad))
+        k += pad
+    _check(lib().telb_gemm_f16_f32out(_p(x2), _p(weight), _p(out), c_int(m), c_int(n), c_int(k), _p(bias), c_int(_is_bf16(x)),
+                                      _p(Workspace.get(x.device).status), _stream()), "gemm_f16_f32out")
+    return out
+
+
+def stream_norm(stream, weight, eps: float, delta, routed, mult: float, step, offset: float, ids, table, dtype):
+    """See :func:`ops.stream_norm`; ``routed`` carries expert rows (``y``, routing tables ``ws``, weights)."""
+    if stream is None:
+        t, width, dev = ids.numel(), table.shape[1], table.device
+        ids = ids.to(torch.int32).contiguous()
+        if table.dtype != dtype:
+            raise TypeError(f"stream_norm: embedding table {table.dtype}, activations {dtype}")
+    else:
+        (t, width), dev = stream.shape, stream.device
+        ids = table = None
+    for d in (delta, None if routed is None else routed.y):
+        if d is not None and d.dtype != dtype:
+            raise TypeError(f"stream_norm: update {d.dtype}, activations {dtype}")
+    x = torch.empty(t, width, dtype=torch.float32, device=dev)
+    h = None if weight is None else torch.empty(t, width, dtype=dtype, device=dev)
+    y = ws = w = None
+    if routed is not None:
+        y, ws, w = routed.y, routed.ws, routed.weights
+    code = 2 if dtype == torch.float32 else int(dtype == torch.bfloat16)
+    _check(lib().telb_stream_norm(
+        _p(ids), _p(table), c_int(table.shape[0] if table is not None else 0), _p(stream), _p(delta.contiguous() if delta is not None else None), _p(y),
+        _p(ws.dst_row if ws is not None else None), _p(w), c_int(w.shape[1] if w is not None else 0), c_int(y.shape[1] if y is not None else 0),
+        c_float(mult), _p(step), _p(weight), c_float(offset), c_float(eps), _p(x), _p(h), c_int(t), c_int(width), c_int(code), _stream()), "stream_norm")
+    return x, h
 
 
 def rope_table(inv_freq: torch.Tensor, attention_factor: float, max_pos: int, device) -> torch.Tensor:
@@ -280,7 +343,7 @@ def rope_kv_write(qkv, kv_layer, meta: StepMeta, cos_sin, num_q_heads, num_kv_he
         _p(qkv), _p(q), _p(kv_layer), _p(cos_sin), _p(positions), _p(meta.seq_ids), _p(meta.q_start),
         _p(meta.past_len), _p(meta.page_table), _p(meta.kv_offsets), _p(q_norm_w), _p(k_norm_w), c_int(t),
         c_int(num_q_heads), c_int(num_kv_heads), c_int(head_dim), c_int(cos_sin.shape[-1]), c_int(meta.page_size),
-        c_int(meta.page_table.shape[1]), c_float(eps), c_int(_is_bf16(qkv)), _stream()), "rope_kv_write")
+        c_int(meta.page_table.shape[1]), c_float(eps), c_int(_dtype_code(qkv)), _stream()), "rope_kv_write")
     return q
 
 
@@ -357,30 +420,36 @@ def paged_attention_decode_fp8(q8: torch.Tensor, kv_layer: torch.Tensor, meta: S
     return out if out_scale is None else QuantActs(xq, sf, (t, hq * d), out_dtype)
 
 
-def _attn_splits(meta: StepMeta, hkv: int, group: int) -> int:
+def _visible_len(meta: StepMeta, chunk: int) -> int:
+    """Most keys one row of the step can see."""
+    return min(meta.max_seq_len, chunk) if chunk > 0 else meta.max_seq_len
+
+
+def _attn_splits(meta: StepMeta, hkv: int, group: int, chunk: int = 0) -> int:
     tq = 128 // group
     qtiles = (meta.max_q_len + tq - 1) // tq
     ctas = meta.num_seqs * hkv * qtiles
     if ctas >= 148 or meta.max_q_len > 4 * tq:
         return 1
-    kv_tiles = max(1, (meta.max_seq_len + 63) // 64)
+    kv_tiles = max(1, (_visible_len(meta, chunk) + 63) // 64)
     return max(1, min((2 * 148 + ctas - 1) // ctas, kv_tiles, 32))
 
 
-def _decode_splits(meta: StepMeta, hkv: int) -> int:
+def _decode_splits(meta: StepMeta, hkv: int, chunk: int = 0) -> int:
     ctas = meta.num_seqs * hkv
     if ctas >= 148:
         return 1
-    tiles = max(1, (meta.max_seq_len + 127) // 128)
+    tiles = max(1, (_visible_len(meta, chunk) + 127) // 128)
     return max(1, min((148 + ctas - 1) // ctas, tiles, 32))
 
 
 def paged_attention(q, kv_layer, meta: StepMeta, scale, sliding_window=None, sinks=None, splits: Optional[int] = None,
                     kernel: Optional[str] = None, trace: Optional[torch.Tensor] = None, causal: bool = True,
-                    skip_thr: Optional[torch.Tensor] = None, skip_stats: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    skip_thr: Optional[torch.Tensor] = None, skip_stats: Optional[torch.Tensor] = None, chunk: int = 0) -> torch.Tensor:
     """Paged GQA attention.  Decode-shaped steps (``max_q_len * Hq/Hkv <= 16``, head_dim 128, causal)
     run the token-major XQA-style kernel; everything else the row-major tile kernel.
-    ``kernel`` forces ``"decode"`` or ``"tile"``; ``causal=False`` lets every row see every token of its sequence."""
+    ``kernel`` forces ``"decode"`` or ``"tile"``; ``causal=False`` lets every row see every token of its sequence; ``chunk`` > 0 limits
+    a row to the keys of its own ``chunk``-token block.  fp32 rows and head sizes without a tensor-core form run on the CUDA cores."""
     if not causal:
         sliding_window, kernel = -1, "tile"
     if sinks is not None:
@@ -390,8 +459,16 @@ def paged_attention(q, kv_layer, meta: StepMeta, scale, sliding_window=None, sin
     hkv = kv_layer.shape[2]
     group = hq // hkv
     out = torch.empty_like(q)
-    ws = Workspace.get(q.device)
     tm = meta.tree_mask
+    if q.dtype == torch.float32 or d not in (64, 128, 256):
+        if tm is not None or not causal or skip_thr is not None or meta.skip_thr is not None:
+            raise ValueError("fp32 / odd-sized attention covers causal, windowed and chunked masks only")
+        _check(lib().telb_paged_attention_simt(
+            _p(q), _p(kv_layer), _p(out), _p(meta.q_start), _p(meta.past_len), _p(meta.seq_ids), _p(meta.page_table), c_int(t),
+            c_int(meta.page_table.shape[1]), c_int(meta.page_size), c_int(hq), c_int(hkv), c_int(d), c_float(scale), c_int(sliding_window or 0),
+            c_int(chunk), _p(sinks), c_int(_dtype_code(q)), _stream()), "paged_attention_simt")
+        return out
+    ws = Workspace.get(q.device)
     decode_ok = (tm is None and d == 128 and meta.max_q_len * group <= 16 and 16 % group == 0)
     if skip_thr is None:
         skip_thr = meta.skip_thr            # per-sequence skip-softmax thresholds of the step (prefill-size steps only)
@@ -404,22 +481,22 @@ def paged_attention(q, kv_layer, meta: StepMeta, scale, sliding_window=None, sin
         if not decode_ok:
             raise ValueError("step is not decode-shaped")
         if splits is None:
-            splits = _decode_splits(meta, hkv)
+            splits = _decode_splits(meta, hkv, chunk)
         _check(lib().telb_paged_attention_decode_traced(
             _p(q), _p(kv_layer), _p(out), _p(meta.q_start), _p(meta.q_len), _p(meta.past_len), _p(meta.page_table),
             c_int(meta.num_seqs), c_int(t), c_int(meta.max_q_len), c_int(kv_layer.shape[0]), c_int(meta.page_table.shape[1]),
             c_int(meta.page_size), c_int(hq), c_int(hkv), c_int(d), c_float(scale), c_int(sliding_window or 0), c_int(splits),
-            _p(ws.attn_ws), c_ll(ws.attn_ws.numel()), c_int(_is_bf16(q)), _p(ws.status), _p(trace), _p(sinks), _stream()),
+            _p(ws.attn_ws), c_ll(ws.attn_ws.numel()), c_int(_is_bf16(q)), _p(ws.status), _p(trace), _p(sinks), c_int(chunk), _stream()),
             "paged_attention_decode", 2 if splits > 1 else 1)
         return out
     if splits is None:
-        splits = _attn_splits(meta, hkv, group)
+        splits = _attn_splits(meta, hkv, group, chunk)
     _check(lib().telb_paged_attention(
         _p(q), _p(kv_layer), _p(out), _p(meta.q_start), _p(meta.q_len), _p(meta.past_len), _p(meta.page_table),
         _p(tm), c_int(tm.shape[1] if tm is not None else 0), c_int(meta.num_seqs), c_int(t), c_int(meta.max_q_len),
         c_int(kv_layer.shape[0]), c_int(meta.page_table.shape[1]), c_int(meta.page_size), c_int(hq), c_int(hkv),
         c_int(d), c_float(scale), c_int(sliding_window or 0), c_int(splits), _p(ws.attn_ws), c_ll(ws.attn_ws.numel()),
-        c_int(_is_bf16(q)), _p(ws.status), _p(sinks), _p(skip_thr), _p(skip_stats), _stream()), "paged_attention", 2 if splits > 1 else 1)
+        c_int(_is_bf16(q)), _p(ws.status), _p(sinks), _p(skip_thr), _p(skip_stats), c_int(chunk), _stream()), "paged_attention", 2 if splits > 1 else 1)
     return out
 
 
@@ -748,6 +825,28 @@ def moe_route_softmax_topk(logits, top_k, renormalize=True, bias=None, sigmoid=F
     return w, idx
 
 
+def moe_route_chosen(logits: torch.Tensor, top_k: int):
+    """Top-k of fp32 logits (rows may be a column slice of a wider tensor) and the softmax over the chosen ones."""
+    if logits.dtype != torch.float32 or logits.stride(1) != 1:
+        raise TypeError("moe_route_chosen takes fp32 rows")
+    t, e = logits.shape
+    w = torch.empty(t, top_k, dtype=torch.float32, device=logits.device)
+    idx = torch.empty(t, top_k, dtype=torch.int32, device=logits.device)
+    _check(lib().telb_moe_route_chosen(_p(logits), c_int(logits.stride(0)), _p(w), _p(idx), c_int(t), c_int(e), c_int(top_k), _stream()),
+           "moe_route_chosen")
+    return w, idx
+
+
+def clamped_glu(gate_up: torch.Tensor, limit: float, alpha: float, ws: Optional["MoeWorkspace"] = None) -> torch.Tensor:
+    """Clamped gated unit over ``[gate | up]`` rows; with ``ws`` the rows of the padded expert layout that hold no token are skipped."""
+    rows, two = gate_up.shape
+    out = torch.empty(rows, two // 2, dtype=gate_up.dtype, device=gate_up.device)
+    tile_rows = c_vp(ws.tile_expert.data_ptr() + 4 * ws.max_tiles) if ws is not None else c_vp(0)
+    _check(lib().telb_clamped_glu(_p(gate_up), _p(out), tile_rows, c_int(rows), c_int(two // 2), c_float(limit), c_float(alpha),
+                                  c_int(_dtype_code(gate_up)), _stream()), "clamped_glu")
+    return out
+
+
 class MoeWorkspace:
     """Routing tables of one MoE call over the padded row space (every expert segment is a multiple
     of 128 rows, so a 128-row tile belongs to exactly one expert)."""
@@ -776,8 +875,9 @@ def moe_gather(x: torch.Tensor, ws: MoeWorkspace, top_k: int, quant_scale: Optio
     t, h = x.shape
     if quant_scale is None:
         out = torch.empty(ws.rows_pad, h, dtype=x.dtype, device=x.device)
+        # a plain copy: an fp32 row travels as twice as many 16-bit elements
         _check(lib().telb_moe_gather(_p(x), _p(ws.dst_row), _p(out), c_vp(0), c_vp(0), c_vp(0), c_int(t * top_k), c_int(top_k),
-                                     c_int(h), c_int(_is_bf16(x)), _stream()), "moe_gather")
+                                     c_int(h * x.element_size() // 2), c_int(1), _stream()), "moe_gather")
         return out
     L = lib()
     L.telb_nvfp4_sf_bytes.restype = c_ll
@@ -804,6 +904,10 @@ def gemm_grouped(x, weight, ws: MoeWorkspace, experts_local: int, alpha=None, bi
     n = weight.shape[0] // experts_local
     k = weight.shape[1]
     out = torch.empty(ws.rows_pad, n, dtype=x.dtype, device=x.device)
+    if x.dtype == torch.float32:
+        _check(lib().telb_gemm_f32_grouped(_p(x), _p(weight), _p(out), c_int(ws.rows_pad), c_int(n), c_int(k), _p(ws.tile_expert), _p(bias),
+                                           _stream()), "gemm_f32_grouped")
+        return out
     _check(lib().telb_gemm_f16_grouped(_p(x), _p(weight), _p(out), c_int(ws.rows_pad), c_int(n), c_int(k), c_int(experts_local),
                                        _p(ws.tile_expert), _p(alpha), _p(bias), c_int(_is_bf16(x)), _p(wsx.status), _stream()),
            "gemm_f16_grouped")
@@ -908,6 +1012,55 @@ def gated_delta_rule(q, k, v, a, b, A_log, dt_bias, state, meta: StepMeta):
                                        _p(dt_bias.float().contiguous()), _p(state), _p(out), _p(meta.q_start), _p(meta.q_len),
                                        _p(meta.past_len), _p(meta.slot_ids), c_int(meta.num_seqs), c_int(q.shape[1]), c_int(v.shape[1]),
                                        c_int(q.shape[2]), c_int(v.shape[2]), c_int(_is_bf16(q)), _stream()), "gated_delta_rule")
+    return out
+
+
+class MlstmParams(ctypes.Structure):
+    """Host mirror of ``MlstmParams`` (``csrc/kernels/mlstm_common.cuh``)."""
+    _fields_ = [(n, c_vp) for n in ("qkvg", "gates", "state", "norm_state", "norm_w", "out", "o32", "n_next", "q_start", "q_len", "past_len",
+                                    "slot_ids", "status")] + \
+               [(n, c_int) for n in ("ld", "ldg", "heads", "dk", "dv", "k_off", "v_off", "g_off", "dv_real")] + \
+               [(n, c_float) for n in ("scale", "cap", "eps")]
+
+
+MLSTM_TC_MIN_Q = 16      # steps whose longest sequence has at least this many new rows take the chunked tensor-core kernel
+
+
+def mlstm(qkvg, gates, norm_w, state, norm_state, meta: StepMeta, scale: float, cap: float, eps: float, dv_real: int,
+          kernel: Optional[str] = None) -> torch.Tensor:
+    """See :func:`ops.mlstm`.  Steps of one row per sequence run the fused decode kernel, longer ones the chunked tensor-core kernel
+    (16-bit rows) or the row-by-row walk; ``kernel`` forces ``"decode"``, ``"chunk"`` or ``"scan"``."""
+    qkvg = qkvg.contiguous()
+    t = qkvg.shape[0]
+    _, n, dk, dv = state.shape
+    assert state.dtype == norm_state.dtype == norm_w.dtype == gates.dtype == torch.float32
+    assert state.is_contiguous() and norm_state.is_contiguous() and gates.stride(1) == 1
+    assert qkvg.shape[1] == 2 * n * (dk + dv) and norm_state.shape[1:] == (n, dk + 1) and norm_w.numel() == n * dv and gates.shape[1] >= 2 * n
+    chunk_ok = qkvg.dtype != torch.float32 and dk in (64, 128) and dv % 128 == 0
+    if kernel is None:
+        if meta.max_q_len == 1 and dv <= 1024:
+            kernel = "decode"
+        else:
+            kernel = "chunk" if chunk_ok and meta.max_q_len >= MLSTM_TC_MIN_Q else "scan"
+    if (kernel == "decode" and meta.max_q_len != 1) or (kernel == "chunk" and not chunk_ok):
+        raise ValueError(f"the {kernel} kernel does not cover this step")
+    out = torch.empty(t, n * dv, dtype=qkvg.dtype, device=qkvg.device)
+    o32 = nn = None
+    if kernel == "scan" or (kernel == "chunk" and dv != 128):
+        o32 = torch.empty(t, n, dv, dtype=torch.float32, device=qkvg.device)
+        nn = torch.empty(meta.num_seqs, n, dk + 1, dtype=torch.float32, device=qkvg.device)
+    ptr = lambda x: None if x is None else _p(x).value
+    p = MlstmParams(*[ptr(x) for x in (qkvg, gates, state, norm_state, norm_w, out, o32, nn, meta.q_start, meta.q_len, meta.past_len,
+                                       meta.slot_ids, Workspace.get(qkvg.device).status)],
+                    qkvg.shape[1], gates.stride(0), n, dk, dv, n * dk, 2 * n * dk, n * (2 * dk + dv), dv_real, scale, cap, eps)
+    code = _dtype_code(qkvg)
+    L, ref_p = lib(), ctypes.byref(p)
+    if kernel == "decode":
+        _check(L.telb_mlstm_decode(ref_p, c_int(meta.num_seqs), c_int(code), _stream()), "mlstm_decode")
+    elif kernel == "chunk":
+        _check(L.telb_mlstm_chunk(ref_p, c_int(meta.num_seqs), c_int(t), c_int(code), _stream()), "mlstm_chunk", 1 if dv == 128 else 2)
+    else:
+        _check(L.telb_mlstm_scan(ref_p, c_int(meta.num_seqs), c_int(t), c_int(code), _stream()), "mlstm_scan", 2)
     return out
 
 

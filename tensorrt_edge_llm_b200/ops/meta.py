@@ -67,8 +67,9 @@ def build_step_meta(q_lens: Sequence[int], past_lens: Sequence[int], page_table:
                     page_size: int, slot_ids: Optional[Sequence[int]] = None,
                     logits_all: bool = False, device="cpu",
                     positions: Optional[Sequence[int]] = None,
-                    tree_mask: Optional[torch.Tensor] = None) -> StepMeta:
-    """Host-side construction of a :class:`StepMeta` (the Python twin of the native builder)."""
+                    tree_mask: Optional[torch.Tensor] = None, logits_rows: Optional[Sequence[int]] = None) -> StepMeta:
+    """Host-side construction of a :class:`StepMeta` (the Python twin of the native builder).  Logits are computed for the last row of
+    every sequence, for all rows (``logits_all``) or for the listed packed rows (``logits_rows``)."""
     n = len(q_lens)
     q_start = [0]
     for q in q_lens:
@@ -84,7 +85,9 @@ def build_step_meta(q_lens: Sequence[int], past_lens: Sequence[int], page_table:
         pos_t = positions.to(device=device, dtype=torch.int32).reshape(-1)
     elif positions is not None:
         pos = [int(x) for x in positions]
-    if logits_all:
+    if logits_rows is not None:
+        lidx = [int(r) for r in logits_rows]
+    elif logits_all:
         lidx = list(range(t))
     else:
         lidx = [q_start[i + 1] - 1 for i in range(n)]

@@ -259,7 +259,8 @@ def gather_kv(kv_layer: torch.Tensor, page_table_row: torch.Tensor, length: int,
 
 
 def paged_attention(q: torch.Tensor, kv_layer: torch.Tensor, meta: StepMeta, scale: float,
-                    sliding_window: Optional[int] = None, sinks: Optional[torch.Tensor] = None, causal: bool = True) -> torch.Tensor:
+                    sliding_window: Optional[int] = None, sinks: Optional[torch.Tensor] = None, causal: bool = True,
+                    chunk: int = 0) -> torch.Tensor:
     """Causal GQA attention of the step's rows over the paged cache (which already holds this
     step's keys/values).  Row ``i`` of a sequence sees cache slots ``[0, past + i]``
     (bottom-right aligned causal mask), optionally limited to a sliding window, or the tree
@@ -291,6 +292,8 @@ def paged_attention(q: torch.Tensor, kv_layer: torch.Tensor, meta: StepMeta, sca
             allowed = cols <= past + rows
         if sliding_window is not None and causal:
             allowed = allowed & (cols > past + rows - sliding_window)
+        if chunk:
+            allowed = allowed & (torch.div(cols, chunk, rounding_mode="floor") == torch.div(past + rows, chunk, rounding_mode="floor"))
         sc = sc.masked_fill(~allowed[None], float("-inf"))
         if sinks is not None:
             sink = sinks.float().view(hq, 1, 1).expand(hq, ql, 1)
@@ -551,6 +554,74 @@ def gated_delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch
             H = H + ki[:, :, None] * delta[:, None, :]
             out[i] = torch.einsum("hkv,hk->hv", H, qi).to(v.dtype)
         state[slot] = H.to(state.dtype)
+    return out
+
+
+def mlstm(qkvg: torch.Tensor, gates: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, norm_state: torch.Tensor, meta: StepMeta,
+          scale: float, cap: float, eps: float, dv_real: int) -> torch.Tensor:
+    """Matrix-memory LSTM, row by row in fp32 (see ``csrc/kernels/mlstm.cu`` for the equations).  Head sizes are those of ``state``."""
+    t = qkvg.shape[0]
+    _, n, dk, dv = state.shape
+    q, k, v, g = qkvg.float().split([n * dk, n * dk, n * dv, n * dv], dim=-1)
+    q, k, v = q.reshape(t, n, dk) * scale, k.reshape(t, n, dk), v.reshape(t, n, dv)
+    log_i = cap * torch.tanh(gates[:, :n] / cap)
+    log_f = F.logsigmoid(cap * torch.tanh(gates[:, n:2 * n] / cap))
+    o = torch.zeros(t, n, dv)
+    for s in range(meta.num_seqs):
+        r0, ql, past, slot = int(meta.q_start[s]), int(meta.q_len[s]), int(meta.past_len[s]), int(meta.slot_ids[s])
+        S = state[slot].clone() if past > 0 else torch.zeros(n, dk, dv)
+        nm = norm_state[slot].clone() if past > 0 else torch.zeros(n, dk + 1)
+        nv, m = nm[:, :dk], nm[:, dk]
+        for i in range(r0, r0 + ql):
+            m_new = torch.maximum(log_f[i] + m, log_i[i])
+            keep, add = torch.exp(log_f[i] + m - m_new), torch.exp(log_i[i] - m_new)
+            S = keep[:, None, None] * S + add[:, None, None] * k[i][:, :, None] * v[i][:, None, :]
+            nv = keep[:, None] * nv + add[:, None] * k[i]
+            m = m_new
+            den = torch.maximum((nv * q[i]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+            o[i] = torch.einsum("hkv,hk->hv", S, q[i]) / den[:, None]
+        state[slot] = S
+        norm_state[slot] = torch.cat([nv, m[:, None]], dim=-1)
+    o = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / dv_real + eps)
+    return (o.reshape(t, n * dv) * norm_w.float() * torch.sigmoid(g)).to(qkvg.dtype)
+
+
+# ------------------------------------------------------------------------------------------
+# parallel blocks: fp32 residual stream, experts with a clamped unit
+
+
+def stream_norm(stream, weight, eps, delta, routed, mult, step, offset, ids, table, dtype):
+    x = table[ids.long()].float() if stream is None else stream
+    for d in (delta, routed):
+        if d is not None:
+            x = x + mult * d.float()
+    if step is not None:
+        x = x + step
+    if weight is None:
+        return x, None
+    h = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * (offset + weight.float())
+    return x, h.to(dtype)
+
+
+def moe_route_chosen(logits: torch.Tensor, top_k: int):
+    order = torch.argsort(logits.float(), dim=-1, descending=True, stable=True)[:, :top_k]
+    return torch.softmax(logits.float().gather(1, order), dim=-1), order.to(torch.int32)
+
+
+def clamped_glu(gate_up: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+    g, u = gate_up.float().chunk(2, dim=-1)
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return (g * torch.sigmoid(alpha * g) * (u + 1)).to(gate_up.dtype)
+
+
+def clamped_experts(x, w13, w2, weights, idx, limit, alpha):
+    """Weighted sum of the chosen experts' outputs: ``w13 [E, 2I, H]`` (gate rows, then up rows), ``w2 [E, H, I]``."""
+    out = torch.zeros(x.shape[0], x.shape[1], dtype=torch.float32)
+    for e in range(w13.shape[0]):
+        rows, slot = (idx == e).nonzero(as_tuple=True)
+        if rows.numel():
+            a = clamped_glu(linear(x[rows], w13[e]), limit, alpha)
+            out.index_add_(0, rows, linear(a, w2[e]).float() * weights[rows, slot][:, None])
     return out
 
 

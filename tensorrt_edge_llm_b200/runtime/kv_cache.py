@@ -88,7 +88,18 @@ class KVCacheManager:
             if cfg.head_dim % 16:
                 raise ValueError("an FP8 KV cache needs a head_dim that is a multiple of 16")
             self.dtype = torch.float8_e4m3fn
-        self.pool = torch.zeros(self.num_layers, num_pages, 2, hkv, page_size, cfg.head_dim, dtype=self.dtype, device=device)
+        # Stacks whose attention layers have sizes of their own: one tensor per layer, all indexed by the same page table (the pool
+        # tensor is empty then and only names the device, the type and the page count).
+        self._layer_pools: Optional[List[torch.Tensor]] = None
+        geometry, head_dim = (cfg.kv_geometry() if num_layers is None else None), cfg.head_dim
+        if geometry is not None:
+            if self.kv_fp8:
+                raise ValueError("FP8 pages are not built for stacks with per-layer attention sizes")
+            if len(set(geometry)) > 1:
+                self._layer_pools = [torch.zeros(num_pages, 2, h, page_size, d, dtype=self.dtype, device=device) for h, d in geometry]
+            elif geometry:
+                hkv, head_dim = geometry[0]
+        self.pool = torch.zeros(0 if self._layer_pools else self.num_layers, num_pages, 2, hkv, page_size, head_dim, dtype=self.dtype, device=device)
         # hybrid models: model layer index → attention pool index, plus the recurrent state pools
         self._attn_index = {}
         for i, t in enumerate(cfg.layer_types):
@@ -113,10 +124,13 @@ class KVCacheManager:
 
     def kv_layer(self, model_layer: int) -> torch.Tensor:
         """KV pool of attention layer ``model_layer`` (index into the model's layer list)."""
-        return self.pool[self._attn_index[model_layer]]
+        i = self._attn_index[model_layer]
+        return self._layer_pools[i] if self._layer_pools else self.pool[i]
 
     @property
     def bytes_per_token(self) -> int:
+        if self._layer_pools:
+            return sum(t[0, :, :, 0].numel() * t.element_size() for t in self._layer_pools)
         return self.pool[:, 0, :, :, 0].numel() * self.pool.element_size()
 
     def capacity_tokens(self, seat: int) -> int:

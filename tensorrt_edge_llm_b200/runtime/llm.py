@@ -54,14 +54,19 @@ class LLM:
                  enable_prefix_cache: bool = False, scheduling: Optional[dict] = None, draft_model=None, speculative=None,
                  context_cache_max_records: int = 4096, context_cache_max_snapshots: int = 64,
                  embedding_quantization: Optional[str] = None, tp_mirror=None, mapping: Optional[Mapping] = None,
-                 kv_cache_dtype: Optional[str] = None):
+                 kv_cache_dtype: Optional[str] = None, dtype: Optional[str] = None):
+        """``dtype``: compute type to load the checkpoint in instead of the one it names ("bfloat16" | "float16" | "float32"; 32-bit
+        models run on the CPU, and on the GPU where every layer of the family has fp32 kernels)."""
         if device is None:
             device = "cuda" if torch.cuda.is_available() else "cpu"
         self.device = torch.device(device)
         if isinstance(model, ModelConfig):
+            if dtype is not None:
+                model = dataclasses.replace(model, dtype=dtype)
             self.model = AutoModel.from_config(model, comm=comm, device=self.device, random_init=random_init_seed)
         else:
-            self.model = AutoModel.from_pretrained(model, comm=comm, device=self.device, **({"mapping": mapping} if mapping else {}))
+            self.model = AutoModel.from_pretrained(model, comm=comm, device=self.device, **({"mapping": mapping} if mapping else {}),
+                                                   **({"dtype": dtype} if dtype else {}))
         self.cfg = self.model.cfg
         if embedding_quantization:                  # "fp8" | "nvfp4": the token table is stored quantised, rows expand on lookup
             from ..models.embedding import quantize_embedding

@@ -70,14 +70,14 @@ class ModelRunner:
 
     # ---- eager ragged step -----------------------------------------------------------------
     def _meta(self, seats: Sequence[int], q_lens: Sequence[int], logits_all=False, tree_mask=None,
-              positions=None) -> StepMeta:
+              positions=None, logits_rows=None) -> StepMeta:
         past = [self.kv.lengths[s] for s in seats]
         for s, q, p in zip(seats, q_lens, past):
             if p == 0:
                 self.rope_delta.pop(s, None)          # a fresh sequence on this seat
             self.kv.reserve(s, p + q)
         meta = build_step_meta(q_lens, past, self.kv.table_rows(seats), self.kv.page_size, slot_ids=seats,
-                               logits_all=logits_all, device=self.device, tree_mask=tree_mask, positions=positions)
+                               logits_all=logits_all, device=self.device, tree_mask=tree_mask, positions=positions, logits_rows=logits_rows)
         table = getattr(self.model.cfg, "skip_softmax_prefill_table", None)
         if table and tree_mask is None and max(q_lens, default=0) > 1:
             # skip-softmax deployment: every sequence of a prefill-size step votes with the threshold of its own length
@@ -91,9 +91,9 @@ class ModelRunner:
 
     @torch.no_grad()
     def step(self, seats: Sequence[int], token_lists: Sequence[Sequence[int]], logits_all=False,
-             commit=True, tree_mask=None, positions=None) -> torch.Tensor:
+             commit=True, tree_mask=None, positions=None, logits_rows=None) -> torch.Tensor:
         """Run one ragged step; returns logits ``[L, V]`` (last row of each sequence unless
-        ``logits_all``).  KV lengths advance by the rows fed when ``commit``."""
+        ``logits_all`` or an explicit list of packed rows, ``logits_rows``).  KV lengths advance by the rows fed when ``commit``."""
         q_lens = [len(t) for t in token_lists]
         for s in seats:
             if self.kv.lengths[s] == 0:
@@ -101,7 +101,7 @@ class ModelRunner:
         if positions is None and self.rope_delta and any(self.rope_delta.get(s) for s in seats):
             # sequences whose prompt held images: text positions run ahead of / behind the cache length by a fixed offset
             positions = [self.kv.lengths[s] + self.rope_delta.get(s, 0) + j for s, q in zip(seats, q_lens) for j in range(q)]
-        meta = self._meta(seats, q_lens, logits_all, tree_mask, positions)
+        meta = self._meta(seats, q_lens, logits_all, tree_mask, positions, logits_rows)
         flat = [t for ts in token_lists for t in ts]
         if self.device.type == "cuda":
             host = torch.tensor(flat, dtype=torch.int32).pin_memory()
@@ -500,11 +500,15 @@ class _DecodeGraph:
         self._load_state(seats, first_tokens)
         if self.graph is None:
             # warm up once eagerly (allocator, lazy kernels), restore state, then capture
+            recurrent = self.r.kv.recurrent
+            saved = recurrent.snapshot(seats) if recurrent is not None else None      # the warm-up step advances the state rows
             s = torch.cuda.Stream(device=self.r.device)
             s.wait_stream(torch.cuda.current_stream(self.r.device))
             with torch.cuda.stream(s):
                 self._body()
             torch.cuda.current_stream(self.r.device).wait_stream(s)
+            if saved is not None:
+                recurrent.restore(seats, saved)
             self._load_state(seats, first_tokens)
             from ..ops import cuda as _cu
             before = _cu.LAUNCHES
