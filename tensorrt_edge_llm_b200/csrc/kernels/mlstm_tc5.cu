@@ -238,6 +238,16 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_constan
             fence_proxy_async_smem();
             mbar_arrive(s_ready);
         }
+        // gate pre-activations are fetched one chunk ahead: nothing else covers their latency at the head of a chunk
+        float raw_i = 0.f, raw_f = 0.f;
+        auto fetch_gates = [&](int c) {
+            if (c * kMlL + r < ql) {
+                const float* g = p.gates + ((size_t)t_first + (size_t)c * kMlL + r) * p.ldg + h;
+                raw_i = g[0];
+                raw_f = g[p.heads];
+            }
+        };
+        fetch_gates(0);
         for (int c = 0; c < nchunks; ++c) {
             const uint32_t par = (uint32_t)c & 1u;
             const int len = min(kMlL, ql - c * kMlL);
@@ -246,8 +256,8 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_constan
             // ---- gates, cumulative log forget gate and running maximum (base 2) ----
             float f = 0.f, gi = -INFINITY;
             if (valid) {
-                gi = mlstm_input_gate(p.gates[t * p.ldg + h], p.cap) * kLog2e;
-                f = mlstm_forget_gate(p.gates[t * p.ldg + p.heads + h], p.cap) * kLog2e;
+                gi = mlstm_input_gate(raw_i, p.cap) * kLog2e;
+                f = mlstm_forget_gate(raw_f, p.cap) * kLog2e;
             }
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -334,25 +344,37 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_constan
                 fence_proxy_async_smem();
                 mbar_arrive(p_full);
             }
+            fetch_gates(c + 1);
+            uint4 gate_row[FUSED ? kMlV / 8 : 1];          // output-gate row, fetched under the products
+            if constexpr (FUSED) {
+                const uint4* gp = reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(p.qkvg) + t * p.ld + p.g_off + h * p.dv);
+#pragma unroll
+                for (int i = 0; i < kMlV / 8; ++i) gate_row[i] = valid ? gp[i] : make_uint4(0, 0, 0, 0);
+            }
             const float inv = 1.f / (fmaxf(fabsf(den), exp2f(-(f + b))) + kMlstmEps);
             // ---- Sᵀ ← e^{m_prev − B_end} Sᵀ (row r), under the P·V product ----
             if (ok) {
                 const float dec = exp2f(m_prev - b_end);
 #pragma unroll 1
-                for (int c16 = 0; c16 < DK / 16; ++c16) {
-                    uint32_t v[16];
+                for (int c16 = 0; c16 < DK / 16; c16 += 2) {
+                    uint32_t v[16], w[16];
                     tmem_ld_x16(lane_addr + kColS + c16 * 16, v);
+                    tmem_ld_x16(lane_addr + kColS + c16 * 16 + 16, w);
                     tmem_ld_wait();
 #pragma unroll
-                    for (int i = 0; i < 16; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * dec);
+                    for (int i = 0; i < 16; ++i) {
+                        v[i] = __float_as_uint(__uint_as_float(v[i]) * dec);
+                        w[i] = __float_as_uint(__uint_as_float(w[i]) * dec);
+                    }
                     tmem_st_x16(lane_addr + kColS + c16 * 16, v);
+                    tmem_st_x16(lane_addr + kColS + c16 * 16 + 16, w);
                 }
                 tmem_st_wait();
             }
             wait(y_bar, par);
             if (ok) {
                 // ---- (wV): high half in place, low half over P_hi (row r is this thread's own) ----
-#pragma unroll 1
+#pragma unroll 4
                 for (int c8 = 0; c8 < kMlV / 8; ++c8) {
                     const uint32_t off = (c8 >> 3) * 16384 + row_off + (((c8 & 7) ^ (r & 7)) << 4);
                     const uint4 vu = *reinterpret_cast<const uint4*>(sV + off);
@@ -373,42 +395,44 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_constan
                 if constexpr (FUSED) {
                     float ss = 0.f;
 #pragma unroll 1
-                    for (int c8 = 0; c8 < kMlV / 8; ++c8) {
-                        uint32_t ya[8], yi[8];
-                        tmem_ld_x8(lane_addr + kColG + c8 * 8, ya);
-                        tmem_ld_x8(lane_addr + kColYI + c8 * 8, yi);
+                    for (int c32 = 0; c32 < kMlV / 32; ++c32) {
+                        uint32_t ya[32], yi[32];
+                        tmem_ld_x32(lane_addr + kColG + c32 * 32, ya);
+                        tmem_ld_x32(lane_addr + kColYI + c32 * 32, yi);
                         tmem_ld_wait();
+                        float part[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-                        for (int i = 0; i < 8; ++i) {
+                        for (int i = 0; i < 32; ++i) {
                             const float o = __uint_as_float(ya[i]) * inv + __uint_as_float(yi[i]) * inter;
-                            ss = fmaf(o, o, ss);
+                            part[i & 3] = fmaf(o, o, part[i & 3]);
                         }
+                        ss += (part[0] + part[1]) + (part[2] + part[3]);
                     }
                     const float rn = 1.f / sqrtf(ss / p.dv_real + p.eps);
-                    const T* gp = reinterpret_cast<const T*>(p.qkvg) + t * p.ld + p.g_off + h * p.dv;
                     const float* nw = p.norm_w + h * p.dv;
                     T* op = reinterpret_cast<T*>(p.out) + (t * p.heads + h) * p.dv;
-#pragma unroll 1
-                    for (int c8 = 0; c8 < kMlV / 8; ++c8) {
-                        uint32_t ya[8], yi[8];
-                        tmem_ld_x8(lane_addr + kColG + c8 * 8, ya);
-                        tmem_ld_x8(lane_addr + kColYI + c8 * 8, yi);
+#pragma unroll
+                    for (int c16 = 0; c16 < kMlV / 16; ++c16) {
+                        uint32_t ya[16], yi[16];
+                        tmem_ld_x16(lane_addr + kColG + c16 * 16, ya);
+                        tmem_ld_x16(lane_addr + kColYI + c16 * 16, yi);
                         tmem_ld_wait();
-                        if (valid) {
-                            const uint4 gu = *reinterpret_cast<const uint4*>(gp + c8 * 8);
-                            const T* ge = reinterpret_cast<const T*>(&gu);
-                            const float4 w0 = *reinterpret_cast<const float4*>(nw + c8 * 8), w1 = *reinterpret_cast<const float4*>(nw + c8 * 8 + 4);
+#pragma unroll
+                        for (int q = 0; q < 2; ++q) {
+                            const T* ge = reinterpret_cast<const T*>(&gate_row[c16 * 2 + q]);
+                            const float4 w0 = *reinterpret_cast<const float4*>(nw + c16 * 16 + q * 8), w1 = *reinterpret_cast<const float4*>(nw + c16 * 16 + q * 8 + 4);
                             const float w8[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
                             float o[8];
 #pragma unroll
                             for (int i = 0; i < 8; ++i)
-                                o[i] = (__uint_as_float(ya[i]) * inv + __uint_as_float(yi[i]) * inter) * rn * w8[i] / (1.f + expf(-Cvt<T>::to_f(ge[i])));
+                                o[i] = __fdividef((__uint_as_float(ya[q * 8 + i]) * inv + __uint_as_float(yi[q * 8 + i]) * inter) * rn * w8[i],
+                                                  1.f + __expf(-Cvt<T>::to_f(ge[i])));
                             uint4 ou;
                             ou.x = Cvt<T>::pack2(o[0], o[1]);
                             ou.y = Cvt<T>::pack2(o[2], o[3]);
                             ou.z = Cvt<T>::pack2(o[4], o[5]);
                             ou.w = Cvt<T>::pack2(o[6], o[7]);
-                            *reinterpret_cast<uint4*>(op + c8 * 8) = ou;
+                            if (valid) *reinterpret_cast<uint4*>(op + c16 * 16 + q * 8) = ou;
                         }
                     }
                 } else {
@@ -434,14 +458,19 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_constan
             if (ok && r < DK) {
                 const uint8_t* kc = sK + (r >> 6) * 16384 + (r & 7) * 2;
                 const int unit = (r & 63) >> 3;
-                float acc = 0.f;
-#pragma unroll 8
-                for (int s = 0; s < kMlL; ++s) {
-                    const T k = *reinterpret_cast<const T*>(kc + (s >> 3) * 1024 + (s & 7) * 128 + ((unit ^ (s & 7)) << 4));
-                    const float w = sW[s];
-                    acc += w == 0.f ? 0.f : w * Cvt<T>::to_f(k);
+                float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+                for (int s8 = 0; s8 < kMlL / 8; ++s8) {
+                    const float4 w0 = *reinterpret_cast<const float4*>(sW + s8 * 8), w1 = *reinterpret_cast<const float4*>(sW + s8 * 8 + 4);
+                    const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {
+                        const T k = *reinterpret_cast<const T*>(kc + s8 * 1024 + i * 128 + ((unit ^ i) << 4));
+                        acc[i] = w[i] == 0.f ? acc[i] : fmaf(w[i], Cvt<T>::to_f(k), acc[i]);
+                    }
                 }
-                sN[r] = sN[r] * exp2f(m_prev - b_end) + acc;
+                const float sum = ((acc[0] + acc[1]) + (acc[2] + acc[3])) + ((acc[4] + acc[5]) + (acc[6] + acc[7]));
+                sN[r] = sN[r] * exp2f(m_prev - b_end) + sum;
             }
             if (ok) mbar_arrive(k_done);
             m_prev = f_end + b_end;
@@ -449,7 +478,7 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_constan
             wait(s_bar, par);
             if (!ok) continue;                             // leaves at the next barrier (or with the loop)
             const bool last = c == nchunks - 1;
-#pragma unroll 1
+#pragma unroll 4
             for (int c8 = 0; c8 < DK / 8; ++c8) {
                 uint32_t u8[8];
                 tmem_ld_x8(lane_addr + kColS + c8 * 8, u8);
