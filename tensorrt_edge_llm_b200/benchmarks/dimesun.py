@@ -151,13 +151,13 @@ def kernel_pairs(device) -> list:
         for m in ours + theirs:
             m.random_init(gen)
         x = [rnd(t, s["hidden"]).to(dt) for _ in range(2)]
-        lg = [rnd(t, s["experts"]) for _ in range(2)]
+        rw, rb = rnd(s["experts"], s["hidden"]).to(dt), rnd(s["experts"])
         stream = rnd(t, s["hidden"])
         w = torch.zeros(s["hidden"], device=device)
         two = (lambda fn: _graph_time(fn, 2)) if decode else (lambda fn: _time(lambda i: fn(i % 2), 10))
 
         def block(i):
-            r = ours[i](x[i], lg[i])
+            r = ours[i](x[i], cu.gemm_f32out(x[i], rw, rb))
             return cu.stream_norm(stream, w, 1e-6, x[i], r, 0.5, None, 1.0, None, None, dt)
 
         def like(i):
@@ -166,8 +166,8 @@ def kernel_pairs(device) -> list:
         hit = min(s["experts"], t * s["top_k"])
         wb, mf = hit * 3 * s["hidden"] * s["inter"] * 2, 6.0 * t * s["top_k"] * s["hidden"] * s["inter"]
         hb = t * s["hidden"] * 2
-        add(f"experts + stream update + norm, {label}", two(block), wb + 8 * hb, mf, "Qwen3-style experts (with router) + add + norm", two(like), wb + 6 * hb, mf)
-        del ours, theirs, x, lg
+        add(f"experts (with router) + stream update + norm, {label}", two(block), wb + 8 * hb, mf, "Qwen3-style experts (with router) + add + norm", two(like), wb + 6 * hb, mf)
+        del ours, theirs, x
     return rows
 
 
