@@ -62,13 +62,15 @@ def ensure_built(model_type: str) -> str:
     """Build what a model family needs if the tree holds no built libraries: the runtime module and, when the whole kernel library is
     absent, the family's own (or the whole one for families without a list).  Returns the family whose library serves, or ""."""
     import glob
-    if not glob.glob(os.path.join(LIBDIR, "_telb_runtime*.so")):
-        build_runtime()
-    if os.path.exists(kernel_library()):
-        return ""
-    family = model_type if model_type in KERNEL_SETS else ""
-    if not os.path.exists(kernel_library(family)):
-        build_kernels(family=family)
+    family = "" if os.path.exists(kernel_library()) or model_type not in KERNEL_SETS else model_type
+    with cf.ThreadPoolExecutor(max_workers=2) as ex:
+        jobs = []
+        if not glob.glob(os.path.join(LIBDIR, "_telb_runtime*.so")):
+            jobs.append(ex.submit(build_runtime))
+        if not os.path.exists(kernel_library(family)):
+            jobs.append(ex.submit(build_kernels, family=family))
+        for j in jobs:
+            j.result()
     return family
 
 
@@ -110,6 +112,7 @@ def build_runtime(force=False, verbose=False) -> str:
         return ""
     import pybind11
     os.makedirs(BUILD, exist_ok=True)
+    os.makedirs(LIBDIR, exist_ok=True)
     headers = [os.path.join(rdir, f) for f in os.listdir(rdir) if f.endswith((".h", ".hpp", ".inc"))]
     inc = ["-I" + pybind11.get_include(), "-I" + sysconfig.get_paths()["include"], "-I" + rdir]
     cxx = shutil.which("g++") or "g++"
