@@ -195,6 +195,42 @@ LLMEngineConfig LLMEngineConfig::from_runtime_config(const Json& root) {
     i(gd, "head_k_dim", c.gdn_head_k_dim);
     i(gd, "head_v_dim", c.gdn_head_v_dim);
     i(gd, "conv_kernel", c.gdn_conv_kernel);
+    const Json& specs = m["layer_specs"];
+    if (specs.is_array() && !specs.items().empty()) {
+        const auto& list = specs.items();
+        const int n = static_cast<int>(list.size());
+        auto pad_head = [](int d) { return d <= 64 ? 64 : d <= 128 ? 128 : d <= 256 ? 256 : (d + 63) / 64 * 64; };
+        auto add_run = [&](const Json& spec) {
+            long long kv = 0, state = 0;
+            int heads = 0, k = 0, v = 0;
+            if (spec["attention"].is_object()) {
+                const Json& a = spec["attention"];
+                i(a, "num_kv_heads", heads);
+                i(a, "head_dim", k);
+                i(a, "v_head_dim", v);
+                kv = 2LL * heads * pad_head(std::max(k, v));
+            } else if (spec["mlstm"].is_object()) {
+                const Json& a = spec["mlstm"];
+                i(a, "num_heads", heads);
+                i(a, "head_k_dim", k);
+                i(a, "head_v_dim", v);
+                k = pad_head(k);
+                state = 1LL * heads * (1LL * k * ((v + 127) / 128 * 128) + k + 1);
+            }
+            c.run_kv_elements.push_back(kv);
+            c.run_state_values.push_back(state);
+        };
+        int start = 0, stop = 0, times = 1;
+        i(m, "loop_start", start);
+        i(m, "loop_stop", stop);
+        i(m, "loop_times", times);
+        stop = std::min(stop, n);
+        if (start < 0 || stop <= start) start = stop = n, times = 0;
+        for (int l = 0; l < start; ++l) add_run(list[l]);
+        for (int t = 0; t < times; ++t)
+            for (int l = start; l < stop; ++l) add_run(list[l]);
+        for (int l = stop; l < n; ++l) add_run(list[l]);
+    }
     s(m, "draft_type", c.draft_type);
     s(m, "dflash_projector_type", c.dflash_projector_type);
     i(m, "draft_vocab_size", c.draft_vocab_size);
@@ -229,7 +265,7 @@ bool LLMEngineConfig::is_hybrid() const {
 
 int LLMEngineConfig::num_recurrent_layers() const {
     int n = 0;
-    for (const auto& t : layer_types) n += (t == "mamba" || t == "gdn") ? 1 : 0;
+    for (const auto& t : layer_types) n += (t == "mamba" || t == "gdn" || t == "mlstm") ? 1 : 0;
     return n;
 }
 
@@ -245,6 +281,11 @@ static int element_bytes(const std::string& dtype) { return dtype == "float32" ?
 
 long long LLMEngineConfig::kv_bytes_per_token() const {
     const int eb = (kv_cache_dtype == "auto" || kv_cache_dtype.empty() || kv_cache_dtype == "model") ? element_bytes(dtype) : element_bytes(kv_cache_dtype);
+    if (!run_kv_elements.empty()) {
+        long long n = 0;
+        for (const long long e : run_kv_elements) n += e;
+        return n * eb;
+    }
     const int kvh = std::max(1, num_kv_heads / std::max(1, world_size));
     return 2LL * num_attention_layers() * kvh * head_dim * eb;
 }
@@ -256,6 +297,7 @@ long long LLMEngineConfig::kv_pool_bytes() const {
 
 long long LLMEngineConfig::recurrent_state_bytes_per_seat() const {
     long long total = 0;
+    for (const long long v : run_state_values) total += 4 * v;
     const int eb = element_bytes(dtype), tp = std::max(1, world_size);
     for (const auto& t : layer_types) {
         if (t == "mamba") {
@@ -283,6 +325,7 @@ std::string LLMEngineConfig::validate() const {
     if (num_experts > 0 && (num_experts_per_tok <= 0 || num_experts_per_tok > num_experts)) return "num_experts_per_tok must be in 1..num_experts";
     for (const auto& t : layer_types) {
         if (t == "mamba" && (mamba_num_heads <= 0 || mamba_d_state <= 0)) return "a mamba layer needs the mamba section";
+        if (t == "mlstm" && run_state_values.size() != layer_types.size()) return "mlstm layers need their layer_specs";
         if (t == "gdn" && (gdn_num_v_heads <= 0 || gdn_head_k_dim <= 0)) return "a gdn layer needs the gdn section";
     }
     if (draft_type == "dflash" && dflash_block_size < 2) return "a block draft needs dflash_block_size >= 2";

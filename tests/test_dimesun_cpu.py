@@ -42,6 +42,21 @@ def test_config_runs_and_round_trip():
     assert not ModelConfig.from_hf_dict(cases.CONFIGS["attention_only"]()).is_hybrid
 
 
+@pytest.mark.parametrize("name", sorted(cases.CONFIGS))
+def test_native_engine_config_sizes(name):
+    """The native configuration derives the cache and state sizes that the Python managers allocate."""
+    from tensorrt_edge_llm_b200.checkpoint.artifacts import runtime_config_dict
+    from tensorrt_edge_llm_b200.runtime import native as rt
+    from tensorrt_edge_llm_b200.runtime.kv_cache import KVCacheManager
+    cfg = ModelConfig.from_hf_dict(cases.CONFIGS[name]())
+    c = rt.LLMEngineConfig.from_runtime_config(json.dumps(runtime_config_dict(cfg, 2, 64, 128, 1), default=str))
+    kv = KVCacheManager(cfg, 2, 64, max_seats=1, max_pages_per_seq=2)
+    state = 0 if kv.recurrent is None else kv.recurrent.bytes()
+    assert c.validate() == "" and c.is_hybrid() == cfg.is_hybrid and c.num_attention_layers() == cfg.num_attn_layers
+    assert c.kv_bytes_per_token() == kv.bytes_per_token
+    assert c.recurrent_state_bytes_per_seat() == state
+
+
 @pytest.mark.parametrize("change", ["mixer", "mlp", "loop", "rot"])
 def test_config_refuses_what_it_does_not_know(change):
     hf = cases.CONFIGS["mixed"]()
