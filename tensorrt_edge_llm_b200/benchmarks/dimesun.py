@@ -132,13 +132,15 @@ def kernel_pairs(device) -> list:
         qq = [rnd(t, n, d).to(dt) for _ in range(sets)]
         sinks = torch.zeros(n, device=device)
         for chunk in (s["chunk"], 512):
+            # the counterpart sees as many keys: plain causal attention over the same rows cut into sequences of one chunk each
             vis = sum((p % chunk) + 1 for ql, p0 in zip(q_lens, past) for p in range(p0, p0 + ql))
-            full = sum(p + 1 for ql, p0 in zip(q_lens, past) for p in range(p0, p0 + ql))
-            us = timer(lambda i: cu.paged_attention(qq[i], kv[i], meta, d ** -0.5, None, sinks, chunk=chunk))
-            us_full = timer(lambda i: cu.paged_attention(qq[i], kv[i], meta, d ** -0.5, None, None))
-            kvb = (lambda keys: keys * kvh * d * 4) if decode else (lambda keys: t * kvh * d * 4)
-            add(f"chunked attention (chunk {chunk}, sink), {label}", us, 2 * io + kvb(vis), 4.0 * vis * n * d, "causal attention", us_full,
-                2 * io + kvb(full), 4.0 * full * n * d)
+            cut = [(min(chunk, ql - c), p0 % chunk) for ql, p0 in zip(q_lens, past) for c in range(0, ql, chunk)]
+            like = _meta([c for c, _ in cut], [p for _, p in cut], device)
+            us = timer(lambda i: cu.paged_attention(qq[i], kv[i], meta, d ** -0.5, None, sinks, chunk=chunk, fp32_weights=True))
+            us_like = timer(lambda i: cu.paged_attention(qq[i], kv[i], like, d ** -0.5, None, None))
+            kvb = (vis if decode else t) * kvh * d * 4
+            add(f"chunked attention (chunk {chunk}, sink, fp32 weights), {label}", us, 2 * io + kvb, 4.0 * vis * n * d,
+                f"causal attention, {len(cut)} sequences of the chunk", us_like, 2 * io + kvb, 4.0 * vis * n * d)
         del kv, qq
         # ---- experts, the stream kernel, the fp32-output product ----
         cfg = dimesun_config(3, s["hidden"], s["vocab"], n, s["experts"], s["top_k"], s["inter"], s["chunk"])

@@ -216,6 +216,7 @@ class AttentionConfig:
     scale: float = 0.0               # multiplies q·k
     chunk: int = 0                   # > 0: position i sees j <= i only inside its own block of `chunk` positions
     zero_sink: bool = False          # the softmax denominator holds one more term, exp(0), without a value
+    fp32_weights: bool = False       # softmax weights keep fp32 precision in the weighted sum of 16-bit values
 
     @property
     def pad(self) -> int:
@@ -787,7 +788,7 @@ def _parse_dimesun(cls, hf: Dict[str, Any], quant: Optional["QuantConfig"]) -> "
             spec.attention = AttentionConfig(
                 num_heads=int(m["heads"]), num_kv_heads=int(m["kv_heads"]), head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]),
                 rotary_dim=int(rot.get("dims", 0)), rope_theta=float(rot.get("base", 10000.0)), scale=float(m["scale"]),
-                chunk=int((m.get("mask") or {}).get("size", 0)), zero_sink=True)
+                chunk=int((m.get("mask") or {}).get("size", 0)), zero_sink=True, fp32_weights=True)
             a = spec.attention
             if a.num_heads % a.num_kv_heads or a.rotary_dim % 2 or a.rotary_dim > a.head_dim:
                 raise ValueError(f"layer {i}: query heads must be a multiple of the KV heads, and the rotary size even and within the head")
@@ -1036,7 +1037,7 @@ def dimesun_config(layers: int = 12, hidden: int = 2048, vocab: int = 131072, he
     for i in range(layers):
         moe = MoeConfig(experts, top_k, inter, 7.0)
         if i % 3 == 2:
-            specs.append(LayerConfig(LAYER_ATTENTION, attention=AttentionConfig(heads, max(heads // 4, 1), 128, 128, 128, 1e6, 128 ** -0.5, chunk, True),
+            specs.append(LayerConfig(LAYER_ATTENTION, attention=AttentionConfig(heads, max(heads // 4, 1), 128, 128, 128, 1e6, 128 ** -0.5, chunk, True, True),
                                      moe=moe))
         else:
             specs.append(LayerConfig(LAYER_MLSTM, mlstm=MlstmConfig(heads, 128, 128, 15.0), moe=moe))

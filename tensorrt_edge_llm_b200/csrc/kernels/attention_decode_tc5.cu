@@ -39,6 +39,9 @@ struct DecParams {
     int max_pages, page_size;
     int hq, hkv, group;
     int splits, total_tokens, window;
+    // 1: probabilities enter P·V as a high and a low 16-bit half (fp32 weights to 2^-17); the two P buffers then hold the halves of one
+    // tile instead of two tiles
+    int split_p;
     int chunk;                      // chunked mask: a token sees only keys of its own `chunk`-token block (0 = none)
     int num_seqs, num_items;        // items = sequences x KV heads x splits, walked by persistent CTAs
     float scale_log2;
@@ -327,13 +330,19 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
                     const int stage = cp.jg % VS;
                     // A = Vᵀ: 64-wide d chunks are kChunkBytes apart (leading offset), 8-token groups 1024 B apart
                     const uint64_t dv = smem_desc_sw128_mn(s_v + stage * kKvBytes, kChunkBytes, 1024);
-                    const uint64_t dp = smem_desc_sw128(s_p + (cp.jg & 1) * kPBytes);
+                    const uint64_t dp = smem_desc_sw128(s_p + (p.split_p ? 0 : (cp.jg & 1)) * kPBytes);
                     const uint32_t d_o = tmem_base + kOCol + (cp.ig & 1) * 16;
 #pragma unroll
                     for (int k = 0; k < kDecTile / kMmaK; ++k) {    // 16 (32) tokens per MMA: 2048 (4096) B of V rows, 32 B of a P row
                         const uint64_t da_ = dv + (uint64_t)((k * kMmaK * 128) >> 4), db_ = dp + (uint64_t)(((k >> 2) * (kDecN * 128)) >> 4) + 2 * (k & 3);
                         if constexpr (KV8) umma_f8(d_o, da_, db_, idesc_o, (cp.j > 0 || k > 0) ? 1u : 0u);
                         else umma_f16(d_o, da_, db_, idesc_o, (cp.j > 0 || k > 0) ? 1u : 0u);
+                    }
+                    if (!KV8 && p.split_p) {
+#pragma unroll
+                        for (int k = 0; k < kDecTile / kMmaK; ++k)
+                            umma_f16(d_o, dv + (uint64_t)((k * kMmaK * 128) >> 4),
+                                     dp + (uint64_t)((kPBytes + (k >> 2) * (kDecN * 128)) >> 4) + 2 * (k & 3), idesc_o, 1u);
                     }
                     umma_commit(&v_empty[stage]);
                     umma_commit(&p_free[cp.jg & 1]);
@@ -439,6 +448,9 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
                 // P buffer b is free once the P·V two tiles back has completed.  This wait is taken for every use of the
                 // buffer, so its parity is exact; it also pins how far the tensor pipe can lag behind this warp.
                 if (!mbar_wait(&p_free[b], ((jg >> 1) & 1) ^ 1, abort_flag, p.status, kStatusEpilogueTimeout)) { ok = false; break; }
+                // split probabilities: both buffers belong to this tile, so the previous tile's P·V must have read them
+                if (p.split_p && jg > 0 &&
+                    !mbar_wait(&p_free[b ^ 1], ((jg - 1) >> 1) & 1, abort_flag, p.status, kStatusEpilogueTimeout)) { ok = false; break; }
                 if (j > 0 && any_need) {
                     // O may only be rescaled after the previous tile's P·V has landed: that is the next completion of the
                     // other P buffer's barrier (a parity wait on a barrier polled only now and then could alias).
@@ -456,7 +468,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
                 // Pᵀ[c][token]: row c is 128 tokens = two 128-byte swizzled chunks of 64 tokens.  Dead columns hold the
                 // zeros written at start-up.
                 // one 128-byte span of row c holds kSpan tokens; element bytes kEB
-                uint8_t* pbase = s_p + b * kPBytes + (r / kSpan) * (kDecN * 128);
+                uint8_t* pbase = s_p + (p.split_p ? 0 : b) * kPBytes + (r / kSpan) * (kDecN * 128);
                 const int tl = r % kSpan;
                 constexpr int kPer16 = 16 / kEB;               // tokens per 16-byte swizzle unit
 #pragma unroll
@@ -468,10 +480,12 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
                         l_part[c] += e;
                         if constexpr (KV8) *dst = __nv_cvt_float_to_fp8(e * 256.f, __NV_SATFINITE, __NV_E4M3);
                         else *reinterpret_cast<T*>(dst) = Cvt<T>::from_f(e);
+                        if (!KV8 && p.split_p) *reinterpret_cast<T*>(dst + kPBytes) = Cvt<T>::from_f(e - Cvt<T>::to_f(Cvt<T>::from_f(e)));
                     } else if (c < kDecN) {
                         // a shorter sequence may follow a longer one in this CTA: clear columns it no longer uses
                         if constexpr (KV8) *dst = 0;
                         else *reinterpret_cast<T*>(dst) = Cvt<T>::from_f(0.f);
+                        if (!KV8 && p.split_p) *reinterpret_cast<T*>(dst + kPBytes) = Cvt<T>::from_f(0.f);
                     }
                 }
                 fence_proxy_async_smem();
@@ -622,7 +636,7 @@ extern "C" int telb_paged_attention_decode_traced(const void* q, const void* kv_
                                                   int total_tokens, int max_q_len, int num_pages, int max_pages, int page_size,
                                                   int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                                                   long long ws_floats, int is_bf16, int* status, unsigned long long* trace,
-                                                  const float* sinks, int chunk, cudaStream_t stream);
+                                                  const float* sinks, int chunk, int split_p, cudaStream_t stream);
 
 // Decode-shaped steps only: max_q_len * (Hq/Hkv) <= 16.  Same tensors as telb_paged_attention.
 extern "C" int telb_paged_attention_decode(const void* q, const void* kv_layer, void* out, const int* q_start,
@@ -632,14 +646,14 @@ extern "C" int telb_paged_attention_decode(const void* q, const void* kv_layer, 
                                            long long ws_floats, int is_bf16, int* status, cudaStream_t stream) {
     return telb_paged_attention_decode_traced(q, kv_layer, out, q_start, q_len, past_len, page_table, num_seqs, total_tokens, max_q_len,
                                               num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16,
-                                              status, nullptr, nullptr, 0, stream);
+                                              status, nullptr, nullptr, 0, 0, stream);
 }
 
 static int decode_impl(const void* q, const void* kv_layer, void* out, void* oq, void* osf, const float* ogs, const int* q_start,
                        const int* q_len, const int* past_len, const int* page_table, int num_seqs, int total_tokens, int max_q_len,
                        int num_pages, int max_pages, int page_size, int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                        long long ws_floats, int is_bf16, int* status, unsigned long long* trace, const float* sinks, const float* kv_scales,
-                       int chunk, cudaStream_t stream);
+                       int chunk, int split_p, cudaStream_t stream);
 
 // Same call with a timeline buffer (3 x 64 x 4 u64, zeroed by the caller) filled by the first CTA.
 extern "C" int telb_paged_attention_decode_traced(const void* q, const void* kv_layer, void* out, const int* q_start,
@@ -647,9 +661,9 @@ extern "C" int telb_paged_attention_decode_traced(const void* q, const void* kv_
                                                   int total_tokens, int max_q_len, int num_pages, int max_pages, int page_size,
                                                   int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                                                   long long ws_floats, int is_bf16, int* status, unsigned long long* trace,
-                                                  const float* sinks, int chunk, cudaStream_t stream) {
+                                                  const float* sinks, int chunk, int split_p, cudaStream_t stream) {
     return decode_impl(q, kv_layer, out, nullptr, nullptr, nullptr, q_start, q_len, past_len, page_table, num_seqs, total_tokens, max_q_len,
-                       num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, trace, sinks, nullptr, chunk, stream);
+                       num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, trace, sinks, nullptr, chunk, split_p, stream);
 }
 
 // Decode attention whose output is written as NVFP4 only (packed codes out_xq [T, Hq * D / 2], atom-layout scales out_sf over
@@ -662,7 +676,7 @@ extern "C" int telb_paged_attention_decode_quant(const void* q, const void* kv_l
                                                  int is_bf16, int* status, const float* sinks, cudaStream_t stream) {
     if (!out_xq || !out_sf || !out_global_scale) return fail("telb_paged_attention_decode_quant: output buffers and scale are required");
     return decode_impl(q, kv_layer, nullptr, out_xq, out_sf, out_global_scale, q_start, q_len, past_len, page_table, num_seqs, total_tokens,
-                       max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, nullptr, sinks, nullptr, 0, stream);
+                       max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, nullptr, sinks, nullptr, 0, 0, stream);
 }
 
 // Decode attention over FP8 (E4M3) cache pages read in place: `q8` is the query tensor cast to E4M3 [T, Hq, D], `kv_layer` the
@@ -679,14 +693,14 @@ extern "C" int telb_paged_attention_decode_fp8(const void* q8, const void* kv_la
     if (out_xq && (!out_sf || !out_global_scale)) return fail("telb_paged_attention_decode_fp8: NVFP4 output needs its scale buffers");
     return decode_impl(q8, kv_layer, out, out_xq, out_sf, out_global_scale, q_start, q_len, past_len, page_table, num_seqs, total_tokens,
                        max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, nullptr,
-                       sinks, kv_scales, 0, stream);
+                       sinks, kv_scales, 0, 0, stream);
 }
 
 static int decode_impl(const void* q, const void* kv_layer, void* out, void* oq, void* osf, const float* ogs, const int* q_start,
                        const int* q_len, const int* past_len, const int* page_table, int num_seqs, int total_tokens, int max_q_len,
                        int num_pages, int max_pages, int page_size, int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                        long long ws_floats, int is_bf16, int* status, unsigned long long* trace, const float* sinks, const float* kv_scales,
-                       int chunk, cudaStream_t stream) {
+                       int chunk, int split_p, cudaStream_t stream) {
     if (num_seqs <= 0 || total_tokens <= 0) return 0;
     if (d != 128) return fail("telb_paged_attention_decode: head_dim must be 128");
     if (page_size != 64 && page_size != 128) return fail("telb_paged_attention_decode: page size must be 64 or 128");
@@ -714,6 +728,7 @@ static int decode_impl(const void* q, const void* kv_layer, void* out, void* oq,
     p.total_tokens = total_tokens;
     p.window = window;
     p.chunk = chunk > 0 ? chunk : 0;
+    p.split_p = split_p ? 1 : 0;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.status = status;
     p.trace = trace;

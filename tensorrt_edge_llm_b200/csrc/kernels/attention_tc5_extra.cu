@@ -29,6 +29,7 @@ struct AttnParams {
     int splits;
     int total_tokens;
     int window;                // sliding window, 0 = none, -1 = no causal mask (every row sees every cached and new token)
+    int split_p;               // 1: probabilities enter P·V as a high and a low 16-bit half (fp32 weights to 2^-17); the two P buffers hold one tile then
     int chunk;                 // chunked mask: a row sees only keys of its own `chunk`-token block, counted from position 0; 0 = none
     float scale_log2;          // softmax scale * log2(e)
     const float* sinks;        // [Hq] fp32 per-head sink logits (natural-log units) joining every row's softmax denominator, or null
@@ -200,10 +201,10 @@ extern "C" int telb_paged_attention(const void* q, const void* kv_layer, void* o
                                     const int* tree_mask, int mask_words, int num_seqs, int total_tokens,
                                     int max_q_len, int num_pages, int max_pages, int page_size, int hq, int hkv, int d,
                                     float scale, int window, int splits, float* ws, long long ws_floats, int is_bf16,
-                                    int* status, const float* sinks, const float* skip_thr, int* skip_stats, int chunk, cudaStream_t stream) {
+                                    int* status, const float* sinks, const float* skip_thr, int* skip_stats, int chunk, int split_p, cudaStream_t stream) {
     if (num_seqs <= 0 || total_tokens <= 0) return 0;
     const int group = hkv > 0 ? hq / hkv : 0;
-    if (sinks == nullptr && skip_thr == nullptr && chunk <= 0 && d != 256 && group > 0 && 128 % group == 0)
+    if (sinks == nullptr && skip_thr == nullptr && chunk <= 0 && !split_p && d != 256 && group > 0 && 128 % group == 0)
         return telb_paged_attention_dense(q, kv_layer, out, q_start, q_len, past_len, page_table, tree_mask, mask_words, num_seqs,
                                           total_tokens, max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits,
                                           ws, ws_floats, is_bf16, status, stream);
@@ -228,6 +229,7 @@ extern "C" int telb_paged_attention(const void* q, const void* kv_layer, void* o
     p.total_tokens = total_tokens;
     p.window = window;
     p.chunk = chunk > 0 ? chunk : 0;
+    p.split_p = split_p ? 1 : 0;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.out_bf16 = is_bf16;
     p.sinks = sinks;

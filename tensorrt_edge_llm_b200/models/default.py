@@ -176,7 +176,7 @@ class LayerAttention(nn.Module):
     def forward(self, x: torch.Tensor, meta: StepMeta, kv_layer: torch.Tensor, cos_sin: torch.Tensor) -> torch.Tensor:
         sp = self.spec
         q = ops.rope_kv_write(self.qkv_proj(x), kv_layer, meta, cos_sin, sp.num_heads, sp.num_kv_heads, sp.pad)
-        o = ops.paged_attention(q, kv_layer, meta, sp.scale, None, self.sinks, chunk=sp.chunk)
+        o = ops.paged_attention(q, kv_layer, meta, sp.scale, None, self.sinks, chunk=sp.chunk, fp32_weights=sp.fp32_weights)
         return self.o_proj(o.reshape(o.shape[0], -1))
 
 

@@ -140,10 +140,11 @@ def rope_q(q, kv_layer, meta, cos_sin, num_q_heads, head_dim, q_norm_w=None, eps
     return ref.rope_q(q, meta, cos_sin, num_q_heads, head_dim, q_norm_w, eps)
 
 
-def paged_attention(q, kv_layer, meta, scale, sliding_window=None, sinks=None, causal=True, chunk=0):
-    """``chunk`` > 0: row at position ``i`` sees only keys ``j`` with ``j // chunk == i // chunk`` (and ``j <= i``)."""
+def paged_attention(q, kv_layer, meta, scale, sliding_window=None, sinks=None, causal=True, chunk=0, fp32_weights=False):
+    """``chunk`` > 0: row at position ``i`` sees only keys ``j`` with ``j // chunk == i // chunk`` (and ``j <= i``).
+    ``fp32_weights``: the softmax weights keep fp32 precision in the weighted sum of 16-bit values."""
     if q.is_cuda:
-        return cuda_ops().paged_attention(q, kv_layer, meta, scale, sliding_window, sinks, causal=causal, chunk=chunk)
+        return cuda_ops().paged_attention(q, kv_layer, meta, scale, sliding_window, sinks, causal=causal, chunk=chunk, fp32_weights=fp32_weights)
     return ref.paged_attention(q, kv_layer, meta, scale, sliding_window, sinks, causal=causal, chunk=chunk)
 
 

@@ -445,11 +445,13 @@ def _decode_splits(meta: StepMeta, hkv: int, chunk: int = 0) -> int:
 
 def paged_attention(q, kv_layer, meta: StepMeta, scale, sliding_window=None, sinks=None, splits: Optional[int] = None,
                     kernel: Optional[str] = None, trace: Optional[torch.Tensor] = None, causal: bool = True,
-                    skip_thr: Optional[torch.Tensor] = None, skip_stats: Optional[torch.Tensor] = None, chunk: int = 0) -> torch.Tensor:
+                    skip_thr: Optional[torch.Tensor] = None, skip_stats: Optional[torch.Tensor] = None, chunk: int = 0,
+                    fp32_weights: bool = False) -> torch.Tensor:
     """Paged GQA attention.  Decode-shaped steps (``max_q_len * Hq/Hkv <= 16``, head_dim 128, causal)
     run the token-major XQA-style kernel; everything else the row-major tile kernel.
     ``kernel`` forces ``"decode"`` or ``"tile"``; ``causal=False`` lets every row see every token of its sequence; ``chunk`` > 0 limits
-    a row to the keys of its own ``chunk``-token block.  fp32 rows and head sizes without a tensor-core form run on the CUDA cores."""
+    a row to the keys of its own ``chunk``-token block; ``fp32_weights`` feeds the probabilities to the 16-bit P·V product as high + low
+    halves.  fp32 rows and head sizes without a tensor-core form run on the CUDA cores."""
     if not causal:
         sliding_window, kernel = -1, "tile"
     if sinks is not None:
@@ -486,7 +488,7 @@ def paged_attention(q, kv_layer, meta: StepMeta, scale, sliding_window=None, sin
             _p(q), _p(kv_layer), _p(out), _p(meta.q_start), _p(meta.q_len), _p(meta.past_len), _p(meta.page_table),
             c_int(meta.num_seqs), c_int(t), c_int(meta.max_q_len), c_int(kv_layer.shape[0]), c_int(meta.page_table.shape[1]),
             c_int(meta.page_size), c_int(hq), c_int(hkv), c_int(d), c_float(scale), c_int(sliding_window or 0), c_int(splits),
-            _p(ws.attn_ws), c_ll(ws.attn_ws.numel()), c_int(_is_bf16(q)), _p(ws.status), _p(trace), _p(sinks), c_int(chunk), _stream()),
+            _p(ws.attn_ws), c_ll(ws.attn_ws.numel()), c_int(_is_bf16(q)), _p(ws.status), _p(trace), _p(sinks), c_int(chunk), c_int(int(fp32_weights)), _stream()),
             "paged_attention_decode", 2 if splits > 1 else 1)
         return out
     if splits is None:
@@ -496,7 +498,7 @@ def paged_attention(q, kv_layer, meta: StepMeta, scale, sliding_window=None, sin
         _p(tm), c_int(tm.shape[1] if tm is not None else 0), c_int(meta.num_seqs), c_int(t), c_int(meta.max_q_len),
         c_int(kv_layer.shape[0]), c_int(meta.page_table.shape[1]), c_int(meta.page_size), c_int(hq), c_int(hkv),
         c_int(d), c_float(scale), c_int(sliding_window or 0), c_int(splits), _p(ws.attn_ws), c_ll(ws.attn_ws.numel()),
-        c_int(_is_bf16(q)), _p(ws.status), _p(sinks), _p(skip_thr), _p(skip_stats), c_int(chunk), _stream()), "paged_attention", 2 if splits > 1 else 1)
+        c_int(_is_bf16(q)), _p(ws.status), _p(sinks), _p(skip_thr), _p(skip_stats), c_int(chunk), c_int(int(fp32_weights)), _stream()), "paged_attention", 2 if splits > 1 else 1)
     return out
 
 
