@@ -123,6 +123,9 @@ class CheckpointReader:
     def get(self, name: str) -> torch.Tensor:
         return self._open(self._where[name]).get(name)
 
+    def shape(self, name: str) -> List[int]:
+        return self._open(self._where[name]).info(name)[1]
+
     def close(self):
         for f in self._files.values():
             f.close()

@@ -38,6 +38,7 @@ LAYER_ATTENTION = "attention"
 LAYER_MAMBA = "mamba"
 LAYER_GDN = "gdn"
 LAYER_MLSTM = "mlstm"
+LAYER_CHANNEL_DELTA = "channel_delta"
 LAYER_MLP = "mlp"
 LAYER_MOE = "moe"
 
@@ -217,11 +218,85 @@ class AttentionConfig:
     chunk: int = 0                   # > 0: position i sees j <= i only inside its own block of `chunk` positions
     zero_sink: bool = False          # the softmax denominator holds one more term, exp(0), without a value
     fp32_weights: bool = False       # softmax weights keep fp32 precision in the weighted sum of 16-bit values
+    unit_qk: bool = False            # queries and keys divided by their root mean square over the head, without a weight
+    temp_coef: float = 0.0           # query temperature: q times 1 + coef * ln(floor((position + 1) / every) + 1)
+    temp_every: float = 1.0
 
     @property
     def pad(self) -> int:
         """One padded size serves keys and values: they share the pages of the cache."""
         return pad_head(max(self.head_dim, self.v_head_dim))
+
+    @property
+    def cache_planes(self) -> int:
+        return 2                     # keys, values
+
+
+@dataclass
+class LatentConfig:
+    """Latent attention: all heads read one cached row per token, ``[latent | rotated key part]``; per-head keys and values are linear
+    in the latent."""
+
+    num_heads: int = 8
+    head_dim: int = 128              # query / key features without rotation
+    rot_dim: int = 64                # rotated query / key features (interleaved pairs); the key part is shared by the heads
+    v_head_dim: int = 128
+    rank: int = 512                  # size of the latent
+    rope_theta: float = 10000.0
+    scale: float = 0.0               # multiplies q·k
+
+    @property
+    def k_pad(self) -> int:
+        return (self.head_dim + 63) // 64 * 64
+
+    @property
+    def rot_pad(self) -> int:
+        return (self.rot_dim + 63) // 64 * 64
+
+    @property
+    def v_pad(self) -> int:
+        return (self.v_head_dim + 63) // 64 * 64
+
+    @property
+    def rank_pad(self) -> int:
+        return (self.rank + 63) // 64 * 64
+
+    num_kv_heads = 1                 # the cache holds one row per token
+
+    @property
+    def pad(self) -> int:
+        """Elements of a cached row."""
+        return self.rank_pad + self.rot_pad
+
+    @property
+    def cache_planes(self) -> int:
+        return 1                     # keys and values come from the same row
+
+
+@dataclass
+class ChannelDeltaConfig:
+    """Delta-rule mixer with one decay per head and key channel, short convolutions on q, k and v and a gated head norm."""
+
+    num_heads: int = 8
+    num_kv_heads: int = 8            # heads of q and k; head h uses floor(h / (num_heads / num_kv_heads))
+    head_k_dim: int = 128
+    head_v_dim: int = 128
+    conv_kernel: int = 4
+    decay_rank: int = 128            # inner size of the two-step projection behind the decays
+    gate_rank: int = 128             # the same for the output gate
+
+    @property
+    def k_pad(self) -> int:
+        return pad_head(self.head_k_dim, (32, 64, 128, 256))
+
+    @property
+    def v_pad(self) -> int:
+        return pad_head(self.head_v_dim, (32, 64, 128, 256))
+
+    @property
+    def conv_dim(self) -> int:
+        """Channels of the packed q | k | v rows."""
+        return 2 * self.num_kv_heads * self.k_pad + self.num_heads * self.v_pad
 
 
 @dataclass
@@ -247,11 +322,20 @@ class LayerConfig:
     attention: Optional[AttentionConfig] = None
     mlstm: Optional[MlstmConfig] = None
     moe: Optional[MoeConfig] = None
+    latent: Optional[LatentConfig] = None              # kind "attention" over cached latents
+    delta: Optional[ChannelDeltaConfig] = None
+    ff: int = 0                                        # dense gated feed-forward of this size
+
+    @property
+    def cached(self):
+        """Geometry of the rows this layer keeps in the paged cache, or None."""
+        return self.attention or self.latent
 
     @classmethod
     def from_dict(cls, d: Dict[str, Any]) -> "LayerConfig":
         sub = lambda c, v: c(**v) if isinstance(v, dict) else v
-        return cls(d["kind"], sub(AttentionConfig, d.get("attention")), sub(MlstmConfig, d.get("mlstm")), sub(MoeConfig, d.get("moe")))
+        return cls(d["kind"], sub(AttentionConfig, d.get("attention")), sub(MlstmConfig, d.get("mlstm")), sub(MoeConfig, d.get("moe")),
+                   sub(LatentConfig, d.get("latent")), sub(ChannelDeltaConfig, d.get("delta")), int(d.get("ff", 0)))
 
 
 @dataclass
@@ -319,6 +403,8 @@ class ModelConfig:
     loop_stop: int = 0
     loop_times: int = 1
     residual_mult: float = 1.0              # the residual stream advances by this multiple of a layer's output
+    embedding_mult: float = 1.0             # looked-up embedding rows times this enter the residual stream
+    logits_mult: float = 1.0                # logits are this multiple of the head's output
     diffusion: Optional[DiffusionConfig] = None      # block-diffusion checkpoints (model_type "diffusion_gemma")
     # draft heads
     draft_type: Optional[str] = None        # "eagle3" / "mtp"
@@ -417,7 +503,11 @@ class ModelConfig:
         if not self.layer_specs:
             return None
         specs = [self.layer_specs[i] for i in self.layer_run_ids]
-        return [(sp.attention.num_kv_heads, sp.attention.pad) for sp in specs if sp.kind == LAYER_ATTENTION]
+        return [(sp.cached.num_kv_heads, sp.cached.pad) for sp in specs if sp.kind == LAYER_ATTENTION]
+
+    def kv_planes(self) -> List[int]:
+        """Cached planes per attention layer of such a stack: 2 (keys, values) or 1 (latent rows)."""
+        return [self.layer_specs[i].cached.cache_planes for i in self.layer_run_ids if self.layer_specs[i].kind == LAYER_ATTENTION]
 
     def kv_donor(self, layer_idx: int) -> int:
         """The layer whose KV cache ``layer_idx`` attends over, or -1 when it writes and reads its own."""
@@ -515,6 +605,8 @@ class ModelConfig:
                      has_qk_norm: Optional[bool] = None) -> "ModelConfig":
         if str(hf.get("architecture", "")) == "Dimesun":
             return _parse_dimesun(cls, hf, quant)
+        if str(hf.get("architecture", "")) == "Debonex":
+            return _parse_debonex(cls, hf, quant)
         llm = hf.get("text_config", hf)
         model_type = llm.get("model_type", hf.get("model_type", "llama"))
         heads = int(llm["num_attention_heads"])
@@ -623,6 +715,8 @@ class ModelConfig:
             with open(gen_path, "r", encoding="utf-8") as f:
                 hf["generation_config"] = json.load(f)
         quant = parse_quant_config(model_dir, hf)
+        if hf.get("architecture") == "Debonex":
+            _add_projection_ranks(model_dir, hf)
         cfg = cls.from_hf_dict(hf, quant=quant, has_qk_norm=_detect_qk_norm(model_dir, hf))
         if mapping is not None:
             cfg.mapping = mapping
@@ -817,6 +911,67 @@ def _parse_dimesun(cls, hf: Dict[str, Any], quant: Optional["QuantConfig"]) -> "
                layer_types=[sp.kind for sp in runs], mlp_types=[LAYER_MOE if sp.moe else "none" for sp in runs],
                layer_specs=specs, loop_start=start, loop_stop=stop, loop_times=times, residual_mult=float(hf["residual_mult"]),
                quant=quant or QuantConfig(), bos_token_id=hf.get("bos_token_id"), eos_token_id=hf.get("eos_token_id"))
+
+
+def _add_projection_ranks(model_dir: str, hf: Dict[str, Any]) -> None:
+    """Debonex: the inner sizes of the two-step projections stand in the checkpoint's tensor shapes only; note them on the mixers."""
+    from .checkpoint.safetensors_io import CheckpointReader
+    reader = CheckpointReader(model_dir)
+    for i, entry in enumerate(hf["layers"]):
+        for key, name in (("decay_rank", "a1"), ("gate_rank", "g1")):
+            if f"l{i}.mix.{name}" in reader:
+                entry["mixer"].setdefault(key, reader.shape(f"l{i}.mix.{name}")[0])
+
+
+def _parse_debonex(cls, hf: Dict[str, Any], quant: Optional["QuantConfig"]) -> "ModelConfig":
+    """Debonex: pre-norm layers listed one by one; channel-decay delta rule, latent attention or attention with unit queries and keys and
+    a query temperature as the mixer, dense gated feed-forwards, element-wise tanh norms, fp32 residual stream."""
+    specs: List[LayerConfig] = []
+    for i, entry in enumerate(hf["layers"]):
+        m, f, kind = entry["mixer"], entry.get("mlp"), str(entry["type"])
+        spec = LayerConfig(kind=LAYER_ATTENTION)
+        if kind == "channel_delta":
+            spec.kind = LAYER_CHANNEL_DELTA
+            spec.delta = d = ChannelDeltaConfig(
+                num_heads=int(m["heads"]), num_kv_heads=int(m["kv_heads"]), head_k_dim=int(m["dim"]), head_v_dim=int(m["vdim"]),
+                conv_kernel=int(m["conv"]), decay_rank=int(m.get("decay_rank", m["vdim"])), gate_rank=int(m.get("gate_rank", m["vdim"])))
+            if d.num_heads % d.num_kv_heads or d.conv_kernel < 1:
+                raise ValueError(f"layer {i}: heads must be a multiple of the q / k heads, and the convolution needs a tap")
+        elif kind == "latent_attention":
+            rot = m.get("rot") or {}
+            spec.latent = LatentConfig(num_heads=int(m["heads"]), head_dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), v_head_dim=int(m["vdim"]),
+                                       rank=int(m["kv_rank"]), rope_theta=float(rot.get("base", 10000.0)), scale=float(m["scale"]))
+            if spec.latent.rot_dim % 2 or int(rot.get("dims", spec.latent.rot_dim)) != spec.latent.rot_dim:
+                raise ValueError(f"layer {i}: the whole rotated part turns, in pairs")
+        elif kind == "attention":
+            temp = m.get("q_temp") or {}
+            spec.attention = a = AttentionConfig(
+                num_heads=int(m["heads"]), num_kv_heads=int(m["kv_heads"]), head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]), rotary_dim=0,
+                scale=float(m["scale"]), fp32_weights=True, unit_qk=True, temp_coef=float(temp.get("coef", 0.0)),
+                temp_every=float(temp.get("every", 1)))
+            if a.num_heads % a.num_kv_heads or a.temp_every <= 0:
+                raise ValueError(f"layer {i}: query heads must be a multiple of the KV heads, and the temperature's step positive")
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        if f:
+            if f.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+            spec.ff = int(f["ff"])
+        specs.append(spec)
+    torch_dtype = str(hf.get("torch_dtype", hf.get("dtype", "bfloat16"))).replace("torch.", "")
+    base = dict(vocab_size=int(hf["vocab"]), hidden_size=int(hf["width"]), rms_norm_eps=float(hf["norm"]["eps"]),
+                dtype=torch_dtype if torch_dtype in ("bfloat16", "float16", "float32") else "bfloat16",
+                embedding_mult=float((hf.get("embedding") or {}).get("scale", 1.0)), logits_mult=float(hf.get("logit_scale", 1.0)),
+                quant=quant or QuantConfig(), bos_token_id=hf.get("bos_token_id"), eos_token_id=hf.get("eos_token_id"))
+    return cls(**base, **_debonex_stack(specs))
+
+
+def _debonex_stack(specs: List[LayerConfig]) -> Dict[str, Any]:
+    """Model-wide fields that follow from the layers."""
+    attn = next((sp.cached for sp in specs if sp.cached), AttentionConfig(1, 1, 64, 64))
+    return dict(model_type="debonex", intermediate_size=max((sp.ff for sp in specs), default=0), num_hidden_layers=len(specs),
+                num_attention_heads=attn.num_heads, num_key_value_heads=attn.num_kv_heads, head_dim=attn.pad, hidden_act="gelu_tanh",
+                layer_types=[sp.kind for sp in specs], mlp_types=[LAYER_MLP if sp.ff else "none" for sp in specs], layer_specs=specs)
 
 
 def _parse_dspark(llm: dict, hf: dict) -> dict:
@@ -1046,6 +1201,24 @@ def dimesun_config(layers: int = 12, hidden: int = 2048, vocab: int = 131072, he
                 layer_types=[sp.kind for sp in specs], mlp_types=[LAYER_MOE] * layers, layer_specs=specs, residual_mult=0.5)
     base.update(over)
     return ModelConfig(**base)
+
+
+def debonex_config(layers: int = 12, hidden: int = 2048, vocab: int = 32768, heads: int = 16, inter: int = 6144, rank: int = 512,
+                   **over: Any) -> ModelConfig:
+    """Debonex at the sizes of a small production model: of every four layers two delta-rule mixers (``heads`` heads, 128 x 128), one
+    latent attention (128 + 64 query / key features, latent ``rank``) and one attention layer (four query heads per KV head, d 128)."""
+    specs = []
+    for i in range(layers):
+        if i % 4 == 1:
+            specs.append(LayerConfig(LAYER_ATTENTION, latent=LatentConfig(heads, 128, 64, 128, rank, 1e4, 192 ** -0.5), ff=inter))
+        elif i % 4 == 3:
+            specs.append(LayerConfig(LAYER_ATTENTION, attention=AttentionConfig(heads, max(heads // 4, 1), 128, 128, 0, 1e4, 128 ** -0.5, fp32_weights=True,
+                                                                                unit_qk=True, temp_coef=0.1, temp_every=2048), ff=inter))
+        else:
+            specs.append(LayerConfig(LAYER_CHANNEL_DELTA, delta=ChannelDeltaConfig(heads, heads, 128, 128, 4, 128, 128), ff=inter))
+    base = dict(vocab_size=vocab, hidden_size=hidden, rms_norm_eps=1e-6, embedding_mult=2.0, logits_mult=1.0)
+    base.update(over)
+    return ModelConfig(**{**_debonex_stack(specs), **base})
 
 
 def hybrid_nemotron_config(**over: Any) -> ModelConfig:

@@ -2,6 +2,8 @@
 // (fp32 caches, heads wider than 256).  Same tensors and masks as the tile kernel of attention_tc5_extra.cu: causal, sliding
 // window, chunked (a row sees only keys of its own `chunk`-token block, counted from position 0) and sink logits.
 //
+// Latent rows (one plane, one row per token that serves as key and, with its first dv features, as value) are covered as well.
+//
 // One warp per (token, query head): 32 keys at a time, one key per lane for the scores, then one slice of the head per lane for
 // the weighted values, with a running maximum.  Everything after the loads is fp32.
 #include "host_utils.h"
@@ -18,11 +20,12 @@ struct SimtAttnParams {
     const int* seq_ids;
     const int* page_table;
     int tokens, max_pages, page_size, hq, hkv, d, window, chunk;
+    int dv, planes;              // value features; 2 = key and value planes, 1 = values are the first dv features of the keys
     float scale;
     const float* sinks;
 };
 
-template <typename T, int E>                             // E: head features per lane, d <= 32 E
+template <typename T, int E>                             // E: value features per lane, dv <= 32 E
 __global__ void __launch_bounds__(128) attn_simt_kernel(const __grid_constant__ SimtAttnParams p) {
     pdl_prologue();
     extern __shared__ float s_q[];                       // [4 warps][d]
@@ -42,6 +45,7 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(const __grid_constant__ 
     if (p.chunk > 0) lo = max(lo, pos / p.chunk * p.chunk);
     const T* kv = reinterpret_cast<const T*>(p.kv);
     const int* pages = p.page_table + (size_t)seq * p.max_pages;
+    const size_t v_rows = p.planes == 2 ? (size_t)p.hkv * p.page_size : 0;
     float m = p.sinks ? p.sinks[h] : -INFINITY;
     float l = p.sinks ? 1.f : 0.f;
     float acc[E];
@@ -50,7 +54,7 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(const __grid_constant__ 
     for (int j0 = lo; j0 <= pos; j0 += 32) {
         const int j = j0 + lane;
         const int page = j <= pos ? pages[j / p.page_size] : -1;
-        const size_t krow = page < 0 ? 0 : (((size_t)page * 2) * p.hkv + kvh) * p.page_size + j % p.page_size;
+        const size_t krow = page < 0 ? 0 : (((size_t)page * p.planes) * p.hkv + kvh) * p.page_size + j % p.page_size;
         float s = -INFINITY;
         if (page >= 0) {
             const T* k = kv + krow * p.d;
@@ -76,17 +80,17 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(const __grid_constant__ 
         for (int jj = 0; jj < cnt; ++jj) {
             const float w = __shfl_sync(0xffffffffu, e_s, jj);
             const unsigned long long row = __shfl_sync(0xffffffffu, (unsigned long long)krow, jj);
-            const T* v = kv + ((size_t)row + (size_t)p.hkv * p.page_size) * p.d;
+            const T* v = kv + ((size_t)row + v_rows) * p.d;
 #pragma unroll
             for (int e = 0; e < E; ++e)
-                if (e * 32 + lane < p.d) acc[e] = fmaf(w, Cvt<T>::to_f(v[e * 32 + lane]), acc[e]);
+                if (e * 32 + lane < p.dv) acc[e] = fmaf(w, Cvt<T>::to_f(v[e * 32 + lane]), acc[e]);
         }
     }
     const float inv = l > 0.f ? 1.f / l : 0.f;
-    T* out = reinterpret_cast<T*>(p.out) + ((size_t)t * p.hq + h) * p.d;
+    T* out = reinterpret_cast<T*>(p.out) + ((size_t)t * p.hq + h) * p.dv;
 #pragma unroll
     for (int e = 0; e < E; ++e)
-        if (e * 32 + lane < p.d) out[e * 32 + lane] = Cvt<T>::from_f(acc[e] * inv);
+        if (e * 32 + lane < p.dv) out[e * 32 + lane] = Cvt<T>::from_f(acc[e] * inv);
 }
 
 template <typename T>
@@ -95,10 +99,10 @@ static int launch_simt(const SimtAttnParams& p, cudaStream_t stream) {
     const dim3 grid((unsigned)((warps + 3) / 4));
     const size_t smem = (size_t)4 * p.d * sizeof(float);
 #define TELB_SIMT(E_) TELB_LAUNCH("attn_simt_kernel", (attn_simt_kernel<T, E_>), grid, dim3(128), smem, stream, p)
-    if (p.d <= 64) TELB_SIMT(2);
-    else if (p.d <= 128) TELB_SIMT(4);
-    else if (p.d <= 256) TELB_SIMT(8);
-    else if (p.d <= 512) TELB_SIMT(16);
+    if (p.dv <= 64) TELB_SIMT(2);
+    else if (p.dv <= 128) TELB_SIMT(4);
+    else if (p.dv <= 256) TELB_SIMT(8);
+    else if (p.dv <= 512) TELB_SIMT(16);
     else TELB_SIMT(32);
 #undef TELB_SIMT
     TELB_CHECK_LAUNCH("attn_simt_kernel");
@@ -115,7 +119,18 @@ extern "C" int telb_paged_attention_simt(const void* q, const void* kv_layer, vo
     if (total_tokens <= 0) return 0;
     if (d > 1024) return fail("telb_paged_attention_simt: head_dim must be at most 1024");
     if (hkv <= 0 || hq % hkv) return fail("telb_paged_attention_simt: Hq must be a multiple of Hkv");
-    SimtAttnParams p{q, kv_layer, out, q_start, past_len, seq_ids, page_table, total_tokens, max_pages, page_size, hq, hkv, d, window, chunk, scale, sinks};
+    SimtAttnParams p{q, kv_layer, out, q_start, past_len, seq_ids, page_table, total_tokens, max_pages, page_size, hq, hkv, d, window, chunk, d, 2, scale, sinks};
+    if (dtype == 2) return launch_simt<float>(p, stream);
+    return dtype == 1 ? launch_simt<__nv_bfloat16>(p, stream) : launch_simt<__half>(p, stream);
+}
+
+// Causal latent attention: q [T, Hq, row] against cached rows [pages, 1, 1, P, row]; out [T, Hq, dv], dv <= row.
+extern "C" int telb_latent_attention_simt(const void* q, const void* kv_layer, void* out, const int* q_start, const int* past_len, const int* seq_ids,
+                                          const int* page_table, int total_tokens, int max_pages, int page_size, int hq, int row, int dv, float scale,
+                                          int dtype, cudaStream_t stream) {
+    if (total_tokens <= 0) return 0;
+    if (dv > 1024 || dv > row || row > 2048) return fail("telb_latent_attention_simt: at most 1024 latent features");
+    SimtAttnParams p{q, kv_layer, out, q_start, past_len, seq_ids, page_table, total_tokens, max_pages, page_size, hq, 1, row, 0, 0, dv, 1, scale, nullptr};
     if (dtype == 2) return launch_simt<float>(p, stream);
     return dtype == 1 ? launch_simt<__nv_bfloat16>(p, stream) : launch_simt<__half>(p, stream);
 }

@@ -66,9 +66,28 @@ gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, float*
     }
 }
 
+// out[t, i] = gelu(in[t, i]) * in[t, inter + i], tanh form, for the models whose products above feed it.
+__global__ void __launch_bounds__(256) geglu_f32_kernel(const float* __restrict__ in, float* __restrict__ out, long long rows, int inter) {
+    pdl_prologue();
+    const long long n = rows * inter;
+    for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
+        const long long r = i / inter;
+        const float x = in[r * 2 * inter + i - r * inter], u = in[r * 2 * inter + inter + i - r * inter];
+        out[i] = 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x))) * u;
+    }
+}
+
 }  // namespace telb
 
 using namespace telb;
+
+extern "C" int telb_geglu_f32(const float* in, float* out, long long rows, int inter, cudaStream_t stream) {
+    if (rows <= 0 || inter <= 0) return 0;
+    const long long blocks = (rows * inter + 255) / 256;
+    TELB_LAUNCH("geglu_f32_kernel", geglu_f32_kernel, dim3((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0, stream, in, out, rows, inter);
+    TELB_CHECK_LAUNCH("geglu_f32_kernel");
+    return 0;
+}
 
 extern "C" int telb_gemm_f32(const float* x, const float* w, float* out, int M, int N, int K, const float* bias, cudaStream_t stream) {
     if (M <= 0 || N <= 0 || K <= 0) return 0;

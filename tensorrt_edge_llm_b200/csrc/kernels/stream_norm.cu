@@ -1,10 +1,11 @@
 // The fp32 residual stream of parallel blocks.  A parallel layer normalises once, both sublayers read that row, and the stream
 // advances by x += mult * (mixer + feed-forward).  One kernel does everything that lies between two layers:
 //
-//   source      x = table[id] (first call) or the running fp32 stream
+//   source      x = table_mult * table[id] (first call) or the running fp32 stream
 //   update      x += mult * (a + Σ_k w[t,k] · y[dst_row[t,k]])      a: mixer output, the sum: combine of the routed experts
 //   step        x += step                                            one vector for all rows (start of a pass of a looped stack)
-//   norm        h = x / sqrt(mean(x²) + eps) * (offset + weight)     written in the activation type for the next GEMMs
+//   norm        h = x / sqrt(mean(x²) + eps) * (offset + weight)     written in the activation type for the next GEMMs, or
+//               h = tanh(alpha x) * weight + bias                    with a scalar alpha: no statistics, no reduction
 //
 // so neither the combined expert output nor the sum of the two sublayers ever goes to memory, and the stream itself is read and
 // written once per layer.  The stream, the norm and the weights stay fp32; `offset` 1 serves weights that are stored around zero.
@@ -27,6 +28,9 @@ struct StreamParams {
     const float* step;       // [width] or null
     const float* weight;     // [width] or null (no norm)
     float offset, eps;
+    const float* alpha;      // scalar: element-wise tanh norm, or null
+    const float* bias;       // [width], with alpha
+    float table_mult;
     float* x_out;            // [T, width]
     void* h;                 // [T, width] or null
     int width;
@@ -74,6 +78,8 @@ __global__ void __launch_bounds__(kStreamThreads) stream_norm_kernel(const __gri
         if (p.ids) {
             const int id = min(max(p.ids[t], 0), p.vocab - 1);
             load4(reinterpret_cast<const T*>(p.table) + (size_t)id * p.width + c, x[e]);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) x[e][i] *= p.table_mult;
         } else {
             load4(p.x_in + t * p.width + c, x[e]);
         }
@@ -103,14 +109,19 @@ __global__ void __launch_bounds__(kStreamThreads) stream_norm_kernel(const __gri
         for (int i = 0; i < 4; ++i) ss += x[e][i] * x[e][i];
     }
     if (!p.h) return;
+    float inv = 0.f, alpha = 0.f;
+    if (p.alpha) {
+        alpha = *p.alpha;
+    } else {
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
-    __syncthreads();
-    float tot = 0.f;
+        for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        if ((tid & 31) == 0) red[tid >> 5] = ss;
+        __syncthreads();
+        float tot = 0.f;
 #pragma unroll
-    for (int w = 0; w < kStreamThreads / 32; ++w) tot += red[w];
-    const float inv = 1.f / sqrtf(tot / p.width + p.eps);
+        for (int w = 0; w < kStreamThreads / 32; ++w) tot += red[w];
+        inv = 1.f / sqrtf(tot / p.width + p.eps);
+    }
     T* h = reinterpret_cast<T*>(p.h) + t * p.width;
 #pragma unroll
     for (int e = 0; e < E; ++e) {
@@ -118,8 +129,15 @@ __global__ void __launch_bounds__(kStreamThreads) stream_norm_kernel(const __gri
         if (c >= p.width) break;
         float g[4];
         load4(p.weight + c, g);
+        if (p.alpha) {
+            float b[4];
+            load4(p.bias + c, b);
 #pragma unroll
-        for (int i = 0; i < 4; ++i) g[i] = x[e][i] * inv * (p.offset + g[i]);
+            for (int i = 0; i < 4; ++i) g[i] = fmaf(tanhf(alpha * x[e][i]), g[i], b[i]);
+        } else {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) g[i] = x[e][i] * inv * (p.offset + g[i]);
+        }
         if constexpr (sizeof(T) == 4) {
             *reinterpret_cast<float4*>(h + c) = make_float4(g[0], g[1], g[2], g[3]);
         } else {
@@ -152,12 +170,14 @@ using namespace telb;
 // dtype: 0 fp16, 1 bf16, 2 fp32 (of table, a, y and h; the stream, step and weight are fp32).
 extern "C" int telb_stream_norm(const int* ids, const void* table, int vocab, const float* x_in, const void* a, const void* y, const int* dst_row,
                                 const float* topk_w, int top_k, int ldy, float mult, const float* step, const float* weight, float offset,
-                                float eps, float* x_out, void* h, int tokens, int width, int dtype, cudaStream_t stream) {
+                                float eps, const float* alpha, const float* bias, float table_mult, float* x_out, void* h, int tokens,
+                                int width, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (width % 4 || width > 16 * 1024) return fail("telb_stream_norm: width must be a multiple of 4 and at most 16384");
     if (y && (top_k > kStreamMaxTopK || ldy % 4)) return fail("telb_stream_norm: top_k <= 32 and an expert row pitch that is a multiple of 4");
     if (!ids && !x_in) return fail("telb_stream_norm: ids or a stream is needed");
-    StreamParams p{ids, table, vocab, x_in, a, y, dst_row, topk_w, top_k, ldy, mult, step, weight, offset, eps, x_out, h, width};
+    if (alpha && weight && !bias) return fail("telb_stream_norm: the tanh norm has a bias");
+    StreamParams p{ids, table, vocab, x_in, a, y, dst_row, topk_w, top_k, ldy, mult, step, weight, offset, eps, alpha, bias, table_mult, x_out, h, width};
     if (dtype == 2) return launch_stream<float>(p, tokens, stream);
     return dtype == 1 ? launch_stream<__nv_bfloat16>(p, tokens, stream) : launch_stream<__half>(p, tokens, stream);
 }

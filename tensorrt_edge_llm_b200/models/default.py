@@ -23,7 +23,7 @@ from .. import ops
 from ..config import ModelConfig
 from ..ops.meta import StepMeta
 from ..parallel.comm import LocalComm
-from .linear import HeadLinear, NVFP4Linear, TPMode, make_linear
+from .linear import HeadLinear, NVFP4Linear, SplitHeadLinear, TPMode, make_linear
 
 
 class RMSNorm(nn.Module):
@@ -157,12 +157,13 @@ class Attention(nn.Module):
 
 class LayerAttention(nn.Module):
     """Attention with a geometry of its own (``AttentionConfig``): key and value sizes that may differ, partial rotary, a score scale,
-    chunked causal masking and a zero sink.  Heads are padded to a size the kernels take and share the paged cache layout; cos / sin
-    tables come from the model per (base, rotary size)."""
+    chunked causal masking and a zero sink; or, without rotary, unit queries and keys and a query temperature.  Heads are padded to a
+    size the kernels take and share the paged cache layout; the model hands in the position table (cos / sin per (base, rotary size),
+    or the temperature per position)."""
 
     def __init__(self, cfg: ModelConfig, spec, prefix: str):
         super().__init__()
-        self.spec, self.prefix = spec, prefix
+        self.spec, self.prefix, self.eps = spec, prefix, cfg.rms_norm_eps
         h, d = cfg.hidden_size, spec.pad
         self.qkv_proj = HeadLinear(h, 0, out_heads=[(spec.num_heads, spec.head_dim, d), (spec.num_kv_heads, spec.head_dim, d),
                                                     (spec.num_kv_heads, spec.v_head_dim, d)],
@@ -173,11 +174,67 @@ class LayerAttention(nn.Module):
         else:
             self.sinks = None
 
-    def forward(self, x: torch.Tensor, meta: StepMeta, kv_layer: torch.Tensor, cos_sin: torch.Tensor) -> torch.Tensor:
+    def forward(self, x: torch.Tensor, meta: StepMeta, kv_layer: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
         sp = self.spec
-        q = ops.rope_kv_write(self.qkv_proj(x), kv_layer, meta, cos_sin, sp.num_heads, sp.num_kv_heads, sp.pad)
+        if sp.unit_qk:
+            q = ops.unit_kv_write(self.qkv_proj(x), kv_layer, meta, table, sp.num_heads, sp.num_kv_heads, sp.pad, sp.head_dim, self.eps)
+        else:
+            q = ops.rope_kv_write(self.qkv_proj(x), kv_layer, meta, table, sp.num_heads, sp.num_kv_heads, sp.pad)
         o = ops.paged_attention(q, kv_layer, meta, sp.scale, None, self.sinks, chunk=sp.chunk, fp32_weights=sp.fp32_weights)
         return self.o_proj(o.reshape(o.shape[0], -1))
+
+
+class LatentAttention(nn.Module):
+    """Latent attention (``LatentConfig``).  One product gives the queries (unrotated | rotated part, each padded per head), the latent and
+    the rotated key part; ``ops.latent_write`` normalises the latent, turns the rotated parts and stores one row per token.  Attention
+    reads those rows directly with the key expansion folded into the query and the value expansion applied to the result (few rows
+    per sequence), or expands keys and values of the step's sequences first (prompt portions); see ``ops.latent_attention``."""
+
+    def __init__(self, cfg: ModelConfig, spec, prefix: str):
+        super().__init__()
+        self.spec, self.prefix, self.eps = spec, prefix, cfg.rms_norm_eps
+        h, n, dt = cfg.hidden_size, spec.num_heads, cfg.compute_dtype
+        self.in_proj = SplitHeadLinear(h, [(n, spec.head_dim, spec.k_pad), (n, spec.rot_dim, spec.rot_pad), (1, spec.rank, spec.rank_pad),
+                                           (1, spec.rot_dim, spec.rot_pad)], [2, 2], sources=["q_proj", "kv_down_proj"], dtype=dt)
+        # keys and values of all heads from a latent: rows [heads x k_pad | heads x v_pad]
+        self.kv_up_proj = HeadLinear(0, 0, out_heads=[(n, spec.head_dim, spec.k_pad), (n, spec.v_head_dim, spec.v_pad)],
+                                     in_heads=(1, spec.rank, spec.rank_pad), sources=["k_up_proj", "v_up_proj"], dtype=dt)
+        self.o_proj = HeadLinear(0, h, in_heads=(n, spec.v_head_dim, spec.v_pad), dtype=dt)
+        self.latent_norm = nn.Parameter(torch.ones(spec.rank_pad, dtype=torch.float32), requires_grad=False)
+        self._key_up_t: Optional[torch.Tensor] = None
+
+    @torch.no_grad()
+    def load_checkpoint(self, fetch) -> bool:
+        w = fetch(f"{self.prefix}.latent_norm.weight")
+        if w is not None:
+            self.latent_norm.zero_()
+            self.latent_norm[:self.spec.rank] = w.float()
+        return False        # the projections are loaded by the generic path
+
+    def finalize(self):
+        """Key expansion with its axes exchanged, ``[heads, rank_pad, k_pad]``: carries a query into latent space."""
+        sp = self.spec
+        w = self.kv_up_proj.weight[:sp.num_heads * sp.k_pad].view(sp.num_heads, sp.k_pad, sp.rank_pad)
+        self._key_up_t = w.transpose(1, 2).contiguous()
+
+    def forward(self, x: torch.Tensor, meta: StepMeta, kv_layer: torch.Tensor, cos_sin: torch.Tensor) -> torch.Tensor:
+        q = ops.latent_write(self.in_proj(x), kv_layer, meta, cos_sin, self.latent_norm, self.spec, self.eps)
+        if self._key_up_t is None or self._key_up_t.device != x.device:
+            self.finalize()
+        return self.o_proj(ops.latent_attention(q, kv_layer, meta, self.kv_up_proj.weight, self._key_up_t, self.spec))
+
+
+class GatedMLP(nn.Module):
+    """``down(act(gate x) * up x)`` with a size of its own (tanh-form gelu); the inner size is padded to what the kernels take."""
+
+    def __init__(self, cfg: ModelConfig, size: int):
+        super().__init__()
+        pad = (1, size, (size + 63) // 64 * 64)
+        self.gate_up_proj = HeadLinear(cfg.hidden_size, 0, out_heads=[pad, pad], sources=["gate_proj", "up_proj"], dtype=cfg.compute_dtype)
+        self.down_proj = HeadLinear(0, cfg.hidden_size, in_heads=pad, dtype=cfg.compute_dtype)
+
+    def forward(self, x):
+        return self.down_proj(ops.geglu(self.gate_up_proj(x), True))
 
 
 class MLP(nn.Module):

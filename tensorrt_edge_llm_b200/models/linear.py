@@ -179,6 +179,70 @@ class Fp32OutLinear(Linear):
         return ops.linear_f32(x, self.weight, self.bias)
 
 
+class StackedRankLinear(Linear):
+    """Outer halves of several low-rank projections whose inner rows lie side by side in one tensor: ``y_i = W_i · inner_i``.
+
+    The weights stack to one block matrix ``[sum(outs), sum(padded ranks)]`` whose rows of part ``i`` are zero outside the columns of
+    inner part ``i``, so every product reads the packed inner rows as they are.  ``forward`` returns one tensor per part: the first
+    with fp32 results; the others in the activation type at prefill sizes, and as columns of one fp32 product at decode sizes
+    (one launch instead of several).  ``ranks`` / ``out_heads``: ``(heads, real, padded)`` per part."""
+
+    ONE_PRODUCT_ROWS = 128
+
+    def __init__(self, ranks, out_heads, sources, dtype=torch.bfloat16):
+        self.ranks, self.out_heads = ranks, out_heads
+        super().__init__(sum(p for _, _, p in ranks), [h * p for h, _, p in out_heads], dtype=dtype, sources=sources)
+        self.weight.data.zero_()
+
+    def _blocks(self):
+        """``(row offset, column offset)`` of every part."""
+        r = c = 0
+        for (_, _, rank), n in zip(self.ranks, self.out_sizes):
+            yield r, c
+            r, c = r + n, c + rank
+
+    def load_from(self, tensors):
+        self.weight.data.zero_()
+        for t, (r, c), (heads, real, pad), (_, rank, _) in zip(tensors, self._blocks(), self.out_heads, self.ranks):
+            w = torch.nn.functional.pad(t["weight"].reshape(heads, real, rank), (0, 0, 0, pad - real)).reshape(heads * pad, rank)
+            self.weight.data[r:r + heads * pad, c:c + rank] = w.to(self.weight.dtype)
+
+    @torch.no_grad()
+    def zero_padding(self) -> None:
+        w = self.weight.data.clone()
+        self.weight.data.zero_()
+        for (r, c), (heads, real, pad), (_, rank, _) in zip(self._blocks(), self.out_heads, self.ranks):
+            self.weight.data[r:r + heads * pad].view(heads, pad, -1)[:, :real, c:c + rank] = w[r:r + heads * pad].view(heads, pad, -1)[:, :real, c:c + rank]
+
+    def forward(self, x: torch.Tensor):
+        if x.shape[0] <= self.ONE_PRODUCT_ROWS:
+            return ops.linear_f32(x, self.weight).split(self.out_sizes, dim=-1)
+        parts, r = [], 0
+        for n in self.out_sizes:
+            w = self.weight[r:r + n]
+            parts.append(ops.linear(x, w) if r else ops.linear_f32(x, w))
+            r += n
+        return tuple(parts)
+
+
+class SplitHeadLinear(HeadLinear):
+    """:class:`HeadLinear` whose checkpoint tensors interleave parts of a head: source ``i`` holds, head by head, the rows of the
+    ``parts[i]`` consecutive entries of ``out_heads``; they leave as separate column blocks."""
+
+    def __init__(self, in_features: int, out_heads, parts, sources, dtype=torch.bfloat16):
+        self.parts = parts
+        super().__init__(in_features, 0, out_heads=out_heads, sources=sources, dtype=dtype)
+
+    def load_from(self, tensors):
+        split, i = [], 0
+        for t, n in zip(tensors, self.parts):
+            group = self.out_heads[i:i + n]
+            w = t["weight"].reshape(group[0][0], sum(real for _, real, _ in group), -1)
+            split += [{"weight": p.reshape(-1, w.shape[-1])} for p in w.split([real for _, real, _ in group], dim=1)]
+            i += n
+        super().load_from(split)
+
+
 class NVFP4Linear(LinearBase):
     """NVFP4 weights (E2M1 pairs, E4M3 scale per 16 inputs, fp32 ``weight_scale_2``).
 

@@ -20,11 +20,11 @@ import torch
 from torch import nn
 
 from .. import ops
-from ..config import LAYER_ATTENTION, LAYER_GDN, LAYER_MAMBA, LAYER_MLP, LAYER_MLSTM, LAYER_MOE, ModelConfig
+from ..config import LAYER_ATTENTION, LAYER_CHANNEL_DELTA, LAYER_GDN, LAYER_MAMBA, LAYER_MLP, LAYER_MLSTM, LAYER_MOE, ModelConfig
 from ..model import register_model
 from ..ops.meta import StepMeta
 from .default import MLP, Attention, CausalLM, RMSNorm
-from .linear import HeadLinear, TPMode, make_linear
+from .linear import Fp32OutLinear, HeadLinear, StackedRankLinear, TPMode, make_linear
 
 
 class RecurrentState:
@@ -34,6 +34,7 @@ class RecurrentState:
         tp = cfg.tp_size
         self.conv, self.ssm, self.gdn = {}, {}, {}
         self.mlstm, self.mlstm_norm = {}, {}      # matrix memory; normaliser and running maximum
+        self.delta = {}                           # channel-decay delta rule
         runs = cfg.layer_run_ids if cfg.layer_specs else None
         for i, t in enumerate(cfg.layer_types):
             if t == LAYER_MAMBA:
@@ -50,12 +51,16 @@ class RecurrentState:
                 m = cfg.layer_specs[runs[i]].mlstm
                 self.mlstm[i] = torch.zeros(seats, m.num_heads, m.k_pad, m.v_pad, dtype=torch.float32, device=device)
                 self.mlstm_norm[i] = torch.zeros(seats, m.num_heads, m.k_pad + 1, dtype=torch.float32, device=device)
+            elif t == LAYER_CHANNEL_DELTA:
+                d = cfg.layer_specs[runs[i]].delta
+                self.conv[i] = torch.zeros(seats, d.conv_dim, d.conv_kernel - 1, dtype=dtype, device=device)
+                self.delta[i] = torch.zeros(seats, d.num_heads, d.k_pad, d.v_pad, dtype=torch.float32, device=device)
 
     def bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in self.pools())
 
     def pools(self):
-        for d in (self.conv, self.ssm, self.gdn, self.mlstm, self.mlstm_norm):
+        for d in (self.conv, self.ssm, self.gdn, self.mlstm, self.mlstm_norm, self.delta):
             yield from d.values()
 
     # ---- replay data -------------------------------------------------------------------------------------------------
@@ -289,6 +294,68 @@ class MLstmMixer(nn.Module):
         sp = self.spec
         return ops.mlstm(qkvg, gates, self.out_norm, state.mlstm[run], state.mlstm_norm[run], meta, sp.head_k_dim ** -0.5, sp.gate_cap,
                          self.eps, sp.head_v_dim)
+
+    @torch.no_grad()
+    def replay(self, saved, rows: torch.Tensor, meta: StepMeta, state: RecurrentState, run: int) -> None:
+        self._recur(*(t.index_select(0, rows) for t in saved), meta, state, run)
+
+
+class ChannelDeltaMixer(nn.Module):
+    """Delta rule with one decay per head and key channel.  q, k and v come from one product; the inner rows of the two low-rank
+    projections (decays, output gate) from a second, their outer halves and the step sizes with fp32 results.  Short convolutions,
+    unit norms, decays, recurrence, head norm and output gate are one op over the step's rows (``ops.channel_delta``)."""
+
+    def __init__(self, cfg: ModelConfig, spec, prefix: str):
+        super().__init__()
+        self.spec, self.prefix, self.eps = spec, prefix, cfg.rms_norm_eps
+        h, n, nk, dt = cfg.hidden_size, spec.num_heads, spec.num_kv_heads, cfg.compute_dtype
+        self.qkv_proj = HeadLinear(h, 0, out_heads=[(nk, spec.head_k_dim, spec.k_pad), (nk, spec.head_k_dim, spec.k_pad),
+                                                    (n, spec.head_v_dim, spec.v_pad)], sources=["q_proj", "k_proj", "v_proj"], dtype=dt)
+        ranks = [(1, r, (r + 7) // 8 * 8) for r in (spec.decay_rank, spec.gate_rank)]
+        self.rank_proj = HeadLinear(h, 0, out_heads=ranks, sources=["decay_in_proj", "gate_in_proj"], dtype=dt)
+        self.up_proj = StackedRankLinear(ranks, [(n, spec.head_k_dim, spec.k_pad), (n, spec.head_v_dim, spec.v_pad)],
+                                         sources=["decay_out_proj", "gate_out_proj"], dtype=dt)
+        self.beta_proj = Fp32OutLinear(h, [n], dtype=dt)
+        self.o_proj = HeadLinear(0, h, in_heads=(n, spec.head_v_dim, spec.v_pad), dtype=dt)
+        self.conv_weight = nn.Parameter(torch.zeros(spec.conv_dim, spec.conv_kernel, dtype=dt), requires_grad=False)
+        self.a_log = nn.Parameter(torch.zeros(n, dtype=torch.float32), requires_grad=False)
+        self.decay_bias = nn.Parameter(torch.zeros(n * spec.k_pad, dtype=torch.float32), requires_grad=False)
+        self.norm_weight = nn.Parameter(torch.ones(spec.v_pad, dtype=torch.float32), requires_grad=False)
+
+    def _heads(self, t: torch.Tensor, heads: int, real: int, pad: int) -> torch.Tensor:
+        """``[heads * real, ...]`` checkpoint rows with every head padded by zero rows."""
+        t = t.reshape(heads, real, -1)
+        return torch.nn.functional.pad(t, (0, 0, 0, pad - real)).reshape(heads * pad, -1)
+
+    @torch.no_grad()
+    def load_checkpoint(self, fetch) -> bool:
+        sp = self.spec
+        sizes = ((sp.num_kv_heads, sp.head_k_dim, sp.k_pad), (sp.num_kv_heads, sp.head_k_dim, sp.k_pad), (sp.num_heads, sp.head_v_dim, sp.v_pad))
+        taps = [fetch(f"{self.prefix}.{n}_conv") for n in "qkv"]
+        if any(t is None for t in taps):
+            return False
+        self.conv_weight.copy_(torch.cat([self._heads(t, *z) for t, z in zip(taps, sizes)]).to(self.conv_weight.dtype))
+        self.decay_bias.copy_(self._heads(fetch(f"{self.prefix}.dt_bias").float(), sp.num_heads, sp.head_k_dim, sp.k_pad)[:, 0])
+        self.norm_weight.zero_()
+        self.norm_weight[:sp.head_v_dim] = fetch(f"{self.prefix}.head_norm.weight").float()
+        return False        # the projections and a_log are loaded by the generic path
+
+    @torch.no_grad()
+    def random_init(self, gen, std=0.02):
+        self.conv_weight.copy_((torch.randn(self.conv_weight.shape, generator=gen) * 0.3).to(self.conv_weight.dtype))
+        self.a_log.copy_(torch.rand(self.spec.num_heads, generator=gen))
+        self.decay_bias.copy_(torch.rand(self.decay_bias.shape, generator=gen) - 4.0)
+
+    def forward(self, x, meta: StepMeta, state: RecurrentState, run: int):
+        qkv, beta = self.qkv_proj(x), self.beta_proj(x)
+        decay, gate = self.up_proj(self.rank_proj(x))
+        if state.record is not None:
+            state.record[run] = (qkv, decay, gate, beta)
+        return self.o_proj(self._recur(qkv, decay, gate, beta, meta, state, run))
+
+    def _recur(self, qkv, decay, gate, beta, meta, state, run):
+        return ops.channel_delta(qkv, decay, gate, beta, self.conv_weight, self.a_log, self.decay_bias, self.norm_weight, state.conv[run],
+                                 state.delta[run], meta, self.spec, self.eps)
 
     @torch.no_grad()
     def replay(self, saved, rows: torch.Tensor, meta: StepMeta, state: RecurrentState, run: int) -> None:

@@ -156,16 +156,19 @@ def linear_f32(x, weight, bias=None):
     return y if bias is None else y + bias.float()
 
 
-def stream_norm(stream, weight, eps, *, delta=None, routed=None, mult=1.0, step=None, offset=0.0, ids=None, table=None, dtype=None):
+def stream_norm(stream, weight, eps, *, delta=None, routed=None, mult=1.0, step=None, offset=0.0, ids=None, table=None, dtype=None,
+                alpha=None, bias=None, table_mult=1.0):
     """Advance the fp32 residual stream and normalise it for the next layer: returns ``(stream, h)``.
 
-    ``stream`` (or ``table[ids]`` when it is ``None``) ``+ mult * (delta + routed) + step``; ``h`` is its RMS norm times
-    ``offset + weight`` in the activation type (``None`` without ``weight``).  ``routed`` is a mixture block's output: a dense tensor,
-    or :class:`models.qwen3_moe.RoutedRows`, whose weighted sum the kernel takes itself."""
+    ``stream`` (or ``table[ids] * table_mult`` when it is ``None``) ``+ mult * (delta + routed) + step``; ``h`` is its RMS norm times
+    ``offset + weight`` in the activation type (``None`` without ``weight``), or, with a scalar ``alpha``, the element-wise
+    ``tanh(alpha * x) * weight + bias``.  ``routed`` is a mixture block's output: a dense tensor, or
+    :class:`models.qwen3_moe.RoutedRows`, whose weighted sum the kernel takes itself."""
     t = ids if stream is None else stream
+    args = (stream, weight, eps, delta, routed, mult, step, offset, ids, table, dtype, alpha, bias, table_mult)
     if t.is_cuda:
-        return cuda_ops().stream_norm(stream, weight, eps, delta, routed, mult, step, offset, ids, table, dtype)
-    return ref.stream_norm(stream, weight, eps, delta, routed, mult, step, offset, ids, table, dtype)
+        return cuda_ops().stream_norm(*args)
+    return ref.stream_norm(*args)
 
 
 def moe_route_chosen(logits, top_k):
@@ -181,6 +184,45 @@ def mlstm(qkvg, gates, norm_w, state, norm_state, meta, scale, cap, eps, dv_real
     if qkvg.is_cuda:
         return cuda_ops().mlstm(qkvg, gates, norm_w, state, norm_state, meta, scale, cap, eps, dv_real)
     return ref.mlstm(qkvg, gates, norm_w, state, norm_state, meta, scale, cap, eps, dv_real)
+
+
+def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, meta, spec, eps):
+    """Delta-rule mixer with a decay per key channel, from packed projections to gated head outputs ``[T, heads * v_pad]``.
+
+    ``qkv``: packed ``[q | k | v]`` rows of padded heads; ``decay`` (fp32, before bias and softplus), ``gate`` and ``beta`` (fp32) are
+    pre-activations.  ``conv_state`` ``[seats, channels, taps - 1]`` and ``state`` ``[seats, heads, k_pad, v_pad]`` are advanced in
+    place.  ``spec``: :class:`config.ChannelDeltaConfig`."""
+    f = cuda_ops().channel_delta if qkv.is_cuda else ref.channel_delta
+    return f(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, meta, spec, eps)
+
+
+def query_temperature(length, coef, every, device="cpu"):
+    """``[length]`` fp32 factors ``1 + coef * ln(floor((position + 1) / every) + 1)``."""
+    return ref.query_temperature(length, coef, every, device)
+
+
+def unit_kv_write(qkv, kv_layer, meta, temperature, num_q_heads, num_kv_heads, head_dim, real_dim, eps):
+    """Queries and keys over their root mean square (``real_dim`` features of a padded head), queries times the temperature of their
+    position; writes keys and values into the paged cache and returns ``q [T, Hq, D]``."""
+    f = cuda_ops().unit_kv_write if qkv.is_cuda else ref.unit_kv_write
+    return f(qkv, kv_layer, meta, temperature, num_q_heads, num_kv_heads, head_dim, real_dim, eps)
+
+
+def latent_write(rows, kv_layer, meta, cos_sin, norm_w, spec, eps):
+    """Packed ``[q unrotated | q rotated part | latent | rotated key part]`` rows: RMS norm of the latent, interleaved rotation of the
+    rotated parts, and ``[latent | key part]`` written to the paged cache ``[pages, 1, 1, P, row]``.  Returns the rows with their query
+    columns ready (modified in place)."""
+    f = cuda_ops().latent_write if rows.is_cuda else ref.latent_write
+    return f(rows, kv_layer, meta, cos_sin, norm_w, spec, eps)
+
+
+def latent_attention(rows, kv_layer, meta, kv_up, key_up_t, spec):
+    """Causal attention of the queries in ``rows`` (see :func:`latent_write`) over cached latents: ``[T, heads * v_pad]``.
+
+    ``kv_up`` ``[heads * k_pad + heads * v_pad, rank_pad]`` expands a latent into keys and values; ``key_up_t``
+    ``[heads, rank_pad, k_pad]`` is its key part with exchanged axes."""
+    f = cuda_ops().latent_attention if rows.is_cuda else ref.latent_attention
+    return f(rows, kv_layer, meta, kv_up, key_up_t, spec)
 
 
 def kv_fp8_prepare(kv_layer, meta, scales, dtype, window=0):

@@ -177,6 +177,11 @@ def geglu(gate_up: torch.Tensor, tanh_approx: bool = True) -> torch.Tensor:
     rows, two = gate_up.shape
     inter = two // 2
     out = torch.empty(rows, inter, dtype=gate_up.dtype, device=gate_up.device)
+    if gate_up.dtype == torch.float32:
+        if not tanh_approx:
+            raise TypeError("geglu: the fp32 form covers the tanh gelu only")
+        _check(lib().telb_geglu_f32(_p(gate_up.contiguous()), _p(out), c_ll(rows), c_int(inter), _stream()), "geglu_f32")
+        return out
     _check(lib().telb_geglu(_p(gate_up), _p(out), c_ll(rows), c_int(inter), c_int(1 if tanh_approx else 0), c_int(_is_bf16(gate_up)),
                             _stream()), "geglu")
     return out
@@ -282,7 +287,8 @@ def gemm_f32out(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tens
     return out
 
 
-def stream_norm(stream, weight, eps: float, delta, routed, mult: float, step, offset: float, ids, table, dtype):
+def stream_norm(stream, weight, eps: float, delta, routed, mult: float, step, offset: float, ids, table, dtype, alpha=None, bias=None,
+                table_mult: float = 1.0):
     """See :func:`ops.stream_norm`; ``routed`` carries expert rows (``y``, routing tables ``ws``, weights)."""
     if stream is None:
         t, width, dev = ids.numel(), table.shape[1], table.device
@@ -304,7 +310,7 @@ def stream_norm(stream, weight, eps: float, delta, routed, mult: float, step, of
     _check(lib().telb_stream_norm(
         _p(ids), _p(table), c_int(table.shape[0] if table is not None else 0), _p(stream), _p(delta.contiguous() if delta is not None else None), _p(y),
         _p(ws.dst_row if ws is not None else None), _p(w), c_int(w.shape[1] if w is not None else 0), c_int(y.shape[1] if y is not None else 0),
-        c_float(mult), _p(step), _p(weight), c_float(offset), c_float(eps), _p(x), _p(h), c_int(t), c_int(width), c_int(code), _stream()), "stream_norm")
+        c_float(mult), _p(step), _p(weight), c_float(offset), c_float(eps), _p(alpha), _p(bias), c_float(table_mult), _p(x), _p(h), c_int(t), c_int(width), c_int(code), _stream()), "stream_norm")
     return x, h
 
 
@@ -1064,6 +1070,105 @@ def mlstm(qkvg, gates, norm_w, state, norm_state, meta: StepMeta, scale: float, 
     else:
         _check(L.telb_mlstm_scan(ref_p, c_int(meta.num_seqs), c_int(t), c_int(code), _stream()), "mlstm_scan", 2)
     return out
+
+
+class ChannelDeltaParams(ctypes.Structure):
+    """Host mirror of ``ChannelDeltaParams`` (``csrc/kernels/channel_delta.cu``)."""
+    _fields_ = [(n, c_vp) for n in ("qkv", "decay", "gate", "beta", "conv_w", "a_log", "decay_bias", "norm_w", "conv_state", "state", "mixed", "row_scale",
+                                    "g", "b", "o", "out", "q_start", "q_len", "past_len", "slot_ids", "seq_ids")] + \
+               [(n, c_int) for n in ("tokens", "num_seqs", "heads", "kv_heads", "dk", "dv", "dk_real", "dv_real", "taps", "channels", "ld_decay", "ld_gate",
+                                     "gate_f32")] + [("eps", c_float)]
+
+
+def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, meta: StepMeta, spec, eps: float,
+                  kernel: Optional[str] = None) -> torch.Tensor:
+    """See :func:`ops.channel_delta`.  Steps of one row per sequence run the fused decode kernel, longer ones the walk over rows;
+    ``kernel`` forces ``"decode"`` or ``"walk"``."""
+    qkv, beta = qkv.contiguous(), beta.contiguous()
+    t, ch = qkv.shape
+    n, nk, dk, dv = spec.num_heads, spec.num_kv_heads, spec.k_pad, spec.v_pad
+    f32 = torch.float32
+    assert ch == spec.conv_dim and conv_w.shape == (ch, spec.conv_kernel) and conv_w.dtype == conv_state.dtype == qkv.dtype
+    assert state.dtype == decay.dtype == beta.dtype == a_log.dtype == decay_bias.dtype == norm_w.dtype == f32
+    assert state.shape[1:] == (n, dk, dv) and state.is_contiguous() and conv_state.is_contiguous() and conv_w.is_contiguous()
+    assert decay.shape == (t, n * dk) and gate.shape == (t, n * dv) and beta.shape == (t, n) and decay.stride(1) == gate.stride(1) == 1
+    if gate.dtype not in (qkv.dtype, f32) or decay.stride(0) % 4 or gate.stride(0) % 4:
+        raise TypeError(f"channel_delta: gate {gate.dtype} for {qkv.dtype} rows, row pitches {decay.stride(0)}, {gate.stride(0)}")
+    decode_ok = meta.max_q_len == 1 and dk <= 128 and dv <= 128
+    if kernel is None:
+        kernel = "decode" if decode_ok else "walk"
+    if kernel == "decode" and not decode_ok:
+        raise ValueError("the decode kernel does not cover this step")
+    dev, one_launch = qkv.device, kernel == "decode" and n == nk
+    out = torch.empty(t, n * dv, dtype=qkv.dtype, device=dev)
+    mixed = scale = g = b = o = None
+    if not one_launch:
+        mixed, scale = torch.empty_like(qkv), torch.empty(t, 2, nk, dtype=f32, device=dev)
+        g, b = torch.empty(t, n * dk, dtype=f32, device=dev), torch.empty(t, n, dtype=f32, device=dev)
+        o = out if kernel == "decode" else torch.empty_like(out)
+    ptr = lambda x: None if x is None else _p(x).value
+    p = ChannelDeltaParams(*[ptr(x) for x in (qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, mixed, scale, g, b, o, out,
+                                              meta.q_start, meta.q_len, meta.past_len, meta.slot_ids, meta.seq_ids)],
+                           t, meta.num_seqs, n, nk, dk, dv, spec.head_k_dim, spec.head_v_dim, spec.conv_kernel, ch, decay.stride(0), gate.stride(0),
+                           int(gate.dtype == f32), eps)
+    launches = (1 if one_launch else 2) if kernel == "decode" else (4 if spec.conv_kernel > 1 else 3)
+    _check(lib().telb_channel_delta(ctypes.byref(p), c_int(int(kernel == "decode")), c_int(_dtype_code(qkv)), _stream()), "channel_delta", launches)
+    return out
+
+
+# ---- attention with cache rows of its own ---------------------------------------------------------
+
+
+def unit_kv_write(qkv, kv_layer, meta: StepMeta, temperature, num_q_heads: int, num_kv_heads: int, head_dim: int, real_dim: int, eps: float):
+    qkv = qkv.contiguous()
+    t = qkv.shape[0]
+    assert kv_layer.is_contiguous() and kv_layer.dtype == qkv.dtype and kv_layer.shape[1:3] == (2, num_kv_heads) and kv_layer.shape[4] == head_dim
+    q = torch.empty(t, num_q_heads, head_dim, dtype=qkv.dtype, device=qkv.device)
+    _check(lib().telb_unit_kv_write(
+        _p(qkv), _p(q), _p(kv_layer), _p(temperature), _p(meta.positions), _p(meta.seq_ids), _p(meta.q_start), _p(meta.past_len), _p(meta.page_table),
+        c_int(t), c_int(meta.page_table.shape[1]), c_int(meta.page_size), c_int(num_q_heads), c_int(num_kv_heads), c_int(head_dim), c_int(real_dim),
+        c_float(eps), c_int(_dtype_code(qkv)), _stream()), "unit_kv_write")
+    return q
+
+
+def latent_write(rows, kv_layer, meta: StepMeta, cos_sin, norm_w, spec, eps: float):
+    rows = rows.contiguous()
+    n = spec.num_heads
+    assert rows.shape[1] == n * (spec.k_pad + spec.rot_pad) + spec.pad and norm_w.dtype == torch.float32 and norm_w.numel() == spec.rank_pad
+    assert kv_layer.is_contiguous() and kv_layer.dtype == rows.dtype and tuple(kv_layer.shape[1:]) == (1, 1, meta.page_size, spec.pad)
+    _check(lib().telb_latent_write(
+        _p(rows), _p(kv_layer), _p(cos_sin), _p(norm_w), _p(meta.positions), _p(meta.seq_ids), _p(meta.q_start), _p(meta.past_len), _p(meta.page_table),
+        c_int(rows.shape[0]), c_int(meta.page_table.shape[1]), c_int(meta.page_size), c_int(n), c_int(spec.k_pad), c_int(spec.rot_pad),
+        c_int(spec.rank_pad), c_int(spec.rank), c_int(spec.rot_dim), c_int(cos_sin.shape[1]), c_float(eps), c_int(_dtype_code(rows)), _stream()), "latent_write")
+    return rows
+
+
+def head_linear(x, weight, heads: int, x_col: int = 0, tail_col: int = -1, tail: int = 0) -> torch.Tensor:
+    """``y[t, h] = weight[h] · x[t, h]`` for ``weight [H, N, K]`` and the ``H · K`` columns of ``x [T, ld]`` from ``x_col`` on; with ``tail``,
+    ``x``'s columns from ``tail_col`` on (``tail`` per head) follow each head's result.  ``[T, H, N + tail]``."""
+    t, (h, n, k) = x.shape[0], weight.shape
+    assert h == heads and x.is_contiguous() and weight.is_contiguous() and x.dtype == weight.dtype
+    y = torch.empty(t, h, n + tail, dtype=x.dtype, device=x.device)
+    base, es = x.data_ptr(), x.element_size()
+    _p(x)
+    _check(lib().telb_head_linear(c_vp(base + x_col * es), _p(weight), _p(y), c_vp(base + max(tail_col, 0) * es), c_int(t), c_int(h), c_int(n), c_int(k),
+                                  c_int(tail), c_int(x.shape[1]), c_int(x.shape[1]), c_int(h * (n + tail)), c_int(n + tail), c_int(_dtype_code(x)),
+                                  _stream()), "head_linear")
+    return y
+
+
+def latent_attention(rows, kv_layer, meta: StepMeta, kv_up, key_up_t, spec) -> torch.Tensor:
+    """See :func:`ops.latent_attention`."""
+    if meta.tree_mask is not None:
+        raise ValueError("latent attention covers causal masks only")
+    t, n = rows.shape[0], spec.num_heads
+    q = head_linear(rows, key_up_t, n, 0, n * spec.k_pad, spec.rot_pad)
+    o = torch.empty(t, n, spec.rank_pad, dtype=rows.dtype, device=rows.device)
+    _check(lib().telb_latent_attention_simt(
+        _p(q), _p(kv_layer), _p(o), _p(meta.q_start), _p(meta.past_len), _p(meta.seq_ids), _p(meta.page_table), c_int(t), c_int(meta.page_table.shape[1]),
+        c_int(meta.page_size), c_int(n), c_int(spec.pad), c_int(spec.rank_pad), c_float(spec.scale), c_int(_dtype_code(q)), _stream()), "latent_attention_simt")
+    value_up = kv_up[n * spec.k_pad:].view(n, spec.v_pad, spec.rank_pad)
+    return head_linear(o.view(t, -1), value_up, n).view(t, n * spec.v_pad)
 
 
 # ---- speculative decoding -------------------------------------------------------------------------

@@ -590,8 +590,8 @@ def mlstm(qkvg: torch.Tensor, gates: torch.Tensor, norm_w: torch.Tensor, state: 
 # parallel blocks: fp32 residual stream, experts with a clamped unit
 
 
-def stream_norm(stream, weight, eps, delta, routed, mult, step, offset, ids, table, dtype):
-    x = table[ids.long()].float() if stream is None else stream
+def stream_norm(stream, weight, eps, delta, routed, mult, step, offset, ids, table, dtype, alpha=None, bias=None, table_mult=1.0):
+    x = table[ids.long()].float() * table_mult if stream is None else stream
     for d in (delta, routed):
         if d is not None:
             x = x + mult * d.float()
@@ -599,8 +599,105 @@ def stream_norm(stream, weight, eps, delta, routed, mult, step, offset, ids, tab
         x = x + step
     if weight is None:
         return x, None
+    if alpha is not None:
+        return x, (torch.tanh(alpha * x) * weight + bias).to(dtype)
     h = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * (offset + weight.float())
     return x, h.to(dtype)
+
+
+# ------------------------------------------------------------------------------------------
+# channel-decay delta rule, unit-norm attention, latent attention
+
+
+def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, meta: StepMeta, spec, eps):
+    """Row by row in fp32 after the short convolutions (see ``csrc/kernels/channel_delta.cu`` for the equations)."""
+    t, n, nk, dk, dv = qkv.shape[0], spec.num_heads, spec.num_kv_heads, spec.k_pad, spec.v_pad
+    w = conv_w.shape[-1]
+    rep = n // nk
+    g = torch.exp(-torch.exp(a_log)[:, None] * F.softplus((decay.float() + decay_bias).reshape(t, n, dk), threshold=80.0))
+    b = torch.sigmoid(beta.float())
+    o = torch.zeros(t, n, dv)
+    for s in range(meta.num_seqs):
+        r0, ql, past, slot = int(meta.q_start[s]), int(meta.q_len[s]), int(meta.past_len[s]), int(meta.slot_ids[s])
+        if ql == 0:
+            continue
+        hist = conv_state[slot].float() if past > 0 else torch.zeros(qkv.shape[1], w - 1)
+        seq = torch.cat([hist, qkv[r0:r0 + ql].float().t()], dim=1)
+        conv_state[slot] = seq[:, seq.shape[1] - (w - 1):].to(conv_state.dtype)
+        y = F.silu(F.conv1d(seq[None], conv_w.float()[:, None, :], None, groups=qkv.shape[1])[0]).t().to(qkv.dtype).float()
+        q, k, v = y.split([nk * dk, nk * dk, n * dv], dim=-1)
+        q, k, v = q.reshape(ql, nk, dk), k.reshape(ql, nk, dk), v.reshape(ql, n, dv)
+        q = q * torch.rsqrt(q.pow(2).sum(-1, keepdim=True) + 1e-6) * spec.head_k_dim ** -0.5
+        k = k * torch.rsqrt(k.pow(2).sum(-1, keepdim=True) + 1e-6)
+        q, k = q.repeat_interleave(rep, dim=1), k.repeat_interleave(rep, dim=1)
+        m = state[slot].clone() if past > 0 else torch.zeros(n, dk, dv)
+        for i in range(ql):
+            m = m * g[r0 + i][:, :, None]
+            u = b[r0 + i][:, None] * (v[i] - torch.einsum("hkv,hk->hv", m, k[i]))
+            m = m + k[i][:, :, None] * u[:, None, :]
+            o[r0 + i] = torch.einsum("hkv,hk->hv", m, q[i])
+        state[slot] = m
+    o = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / spec.head_v_dim + eps) * norm_w
+    return (o.reshape(t, n * dv) * torch.sigmoid(gate.float())).to(qkv.dtype)
+
+
+def query_temperature(length: int, coef: float, every: float, device="cpu") -> torch.Tensor:
+    p = torch.arange(1, length + 1, dtype=torch.float64)
+    return (1.0 + coef * torch.log(torch.floor(p / every) + 1.0)).float().to(device)
+
+
+def _cache_slots(meta: StepMeta, t: int, device):
+    """``(page, row in page)`` of every row of the step."""
+    sid = meta.seq_ids.long()
+    slot = meta.past_len.long()[sid] + (torch.arange(t, device=device) - meta.q_start.long()[sid])
+    return meta.page_table.long()[sid, slot // meta.page_size], slot % meta.page_size
+
+
+def unit_kv_write(qkv, kv_layer, meta: StepMeta, temperature, num_q_heads, num_kv_heads, head_dim, real_dim, eps):
+    t, d = qkv.shape[0], head_dim
+    q, k, v = (x.reshape(t, -1, d).float() for x in qkv.split([num_q_heads * d, num_kv_heads * d, num_kv_heads * d], dim=-1))
+    q, k = (x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / real_dim + eps) for x in (q, k))
+    page, row = _cache_slots(meta, t, qkv.device)
+    kv_layer[page, 0, :, row] = k.to(kv_layer.dtype)
+    kv_layer[page, 1, :, row] = v.to(kv_layer.dtype)
+    return (q * temperature[meta.positions.long()][:, None, None]).to(qkv.dtype)
+
+
+def _rotate_pairs(x: torch.Tensor, cos_sin: torch.Tensor, positions: torch.Tensor, dims: int) -> torch.Tensor:
+    """Interleaved rotation of the first ``dims`` features of ``x [T, H, D]`` (fp32)."""
+    c, s = cos_sin[positions.long(), :dims].float()[:, None].chunk(2, dim=-1)
+    u, v = x[..., 0:dims:2], x[..., 1:dims:2]
+    x = x.clone()
+    x[..., 0:dims:2], x[..., 1:dims:2] = u * c - v * s, v * c + u * s
+    return x
+
+
+def latent_write(rows, kv_layer, meta: StepMeta, cos_sin, norm_w, spec, eps):
+    t, n = rows.shape[0], spec.num_heads
+    q, qr, c, kr = rows.float().split([n * spec.k_pad, n * spec.rot_pad, spec.rank_pad, spec.rot_pad], dim=-1)
+    qr = _rotate_pairs(qr.reshape(t, n, spec.rot_pad), cos_sin, meta.positions, spec.rot_dim).reshape(t, -1)
+    kr = _rotate_pairs(kr[:, None], cos_sin, meta.positions, spec.rot_dim)[:, 0]
+    c = c * torch.rsqrt(c.pow(2).sum(-1, keepdim=True) / spec.rank + eps) * norm_w
+    page, row = _cache_slots(meta, t, rows.device)
+    kv_layer[page, 0, 0, row] = torch.cat((c, kr), dim=-1).to(kv_layer.dtype)
+    return torch.cat((q, qr, c, kr), dim=-1).to(rows.dtype)
+
+
+def latent_attention(rows, kv_layer, meta: StepMeta, kv_up, key_up_t, spec):
+    t, n, dk, dr, dv, rank = rows.shape[0], spec.num_heads, spec.k_pad, spec.rot_pad, spec.v_pad, spec.rank_pad
+    out = torch.zeros(t, n * dv, dtype=rows.dtype)
+    q = torch.cat((rows[:, :n * dk].reshape(t, n, dk), rows[:, n * dk:n * (dk + dr)].reshape(t, n, dr)), dim=-1).float()
+    for s in range(meta.num_seqs):
+        r0, ql, total = int(meta.q_start[s]), int(meta.q_len[s]), int(meta.past_len[s]) + int(meta.q_len[s])
+        pages = meta.page_table[s, :(total + meta.page_size - 1) // meta.page_size].long()
+        cached = kv_layer[pages, 0, 0].reshape(-1, rank + dr)[:total]
+        kv = linear(cached[:, :rank], kv_up).float()
+        k = torch.cat((kv[:, :n * dk].reshape(total, n, dk), cached[:, None, rank:].float().expand(total, n, dr)), dim=-1)
+        sc = torch.einsum("qhd,khd->hqk", q[r0:r0 + ql], k) * spec.scale
+        hidden = torch.arange(total)[None, :] > total - ql + torch.arange(ql)[:, None]
+        pr = torch.softmax(sc.masked_fill(hidden[None], float("-inf")), dim=-1)
+        out[r0:r0 + ql] = torch.einsum("hqk,khd->qhd", pr, kv[:, n * dk:].reshape(total, n, dv)).reshape(ql, -1).to(rows.dtype)
+    return out
 
 
 def moe_route_chosen(logits: torch.Tensor, top_k: int):

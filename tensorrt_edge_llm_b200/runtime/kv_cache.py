@@ -88,15 +88,18 @@ class KVCacheManager:
             if cfg.head_dim % 16:
                 raise ValueError("an FP8 KV cache needs a head_dim that is a multiple of 16")
             self.dtype = torch.float8_e4m3fn
-        # Stacks whose attention layers have sizes of their own: one tensor per layer, all indexed by the same page table (the pool
-        # tensor is empty then and only names the device, the type and the page count).
+        # Stacks whose attention layers have sizes of their own, or cache one latent row per token instead of keys and values: one
+        # tensor per layer, all indexed by the same page table (the pool tensor is empty then and only names the device, the type and
+        # the page count).
         self._layer_pools: Optional[List[torch.Tensor]] = None
         geometry, head_dim = (cfg.kv_geometry() if num_layers is None else None), cfg.head_dim
         if geometry is not None:
             if self.kv_fp8:
                 raise ValueError("FP8 pages are not built for stacks with per-layer attention sizes")
-            if len(set(geometry)) > 1:
-                self._layer_pools = [torch.zeros(num_pages, 2, h, page_size, d, dtype=self.dtype, device=device) for h, d in geometry]
+            planes = cfg.kv_planes()
+            if len(set(geometry)) > 1 or 1 in planes:
+                self._layer_pools = [torch.zeros(num_pages, n, h, page_size, d, dtype=self.dtype, device=device)
+                                     for n, (h, d) in zip(planes, geometry)]
             elif geometry:
                 hkv, head_dim = geometry[0]
         self.pool = torch.zeros(0 if self._layer_pools else self.num_layers, num_pages, 2, hkv, page_size, head_dim, dtype=self.dtype, device=device)
