@@ -201,8 +201,9 @@ LLMEngineConfig LLMEngineConfig::from_runtime_config(const Json& root) {
         const int n = static_cast<int>(list.size());
         auto pad_head = [](int d) { return d <= 64 ? 64 : d <= 128 ? 128 : d <= 256 ? 256 : (d + 63) / 64 * 64; };
         auto add_run = [&](const Json& spec) {
-            long long kv = 0, state = 0;
+            long long kv = 0, state = 0, window = 0;
             int heads = 0, k = 0, v = 0;
+            auto pad64 = [](int d) { return (d + 63) / 64 * 64; };
             if (spec["attention"].is_object()) {
                 const Json& a = spec["attention"];
                 i(a, "num_kv_heads", heads);
@@ -216,9 +217,26 @@ LLMEngineConfig LLMEngineConfig::from_runtime_config(const Json& root) {
                 i(a, "head_v_dim", v);
                 k = pad_head(k);
                 state = 1LL * heads * (1LL * k * ((v + 127) / 128 * 128) + k + 1);
+            } else if (spec["latent"].is_object()) {
+                i(spec["latent"], "rank", k);
+                i(spec["latent"], "rot_dim", v);
+                kv = pad64(k) + pad64(v);                                          // one row per token
+            } else if (spec["delta"].is_object()) {
+                const Json& a = spec["delta"];
+                int kv_heads = 0, taps = 1;
+                i(a, "num_heads", heads);
+                i(a, "num_kv_heads", kv_heads);
+                i(a, "head_k_dim", k);
+                i(a, "head_v_dim", v);
+                i(a, "conv_kernel", taps);
+                k = k <= 32 ? 32 : pad_head(k);
+                v = v <= 32 ? 32 : pad_head(v);
+                state = 1LL * heads * k * v;
+                window = (2LL * kv_heads * k + 1LL * heads * v) * (taps - 1);      // convolution history
             }
             c.run_kv_elements.push_back(kv);
             c.run_state_values.push_back(state);
+            c.run_window_elements.push_back(window);
         };
         int start = 0, stop = 0, times = 1;
         i(m, "loop_start", start);
@@ -265,7 +283,7 @@ bool LLMEngineConfig::is_hybrid() const {
 
 int LLMEngineConfig::num_recurrent_layers() const {
     int n = 0;
-    for (const auto& t : layer_types) n += (t == "mamba" || t == "gdn" || t == "mlstm") ? 1 : 0;
+    for (const auto& t : layer_types) n += (t == "mamba" || t == "gdn" || t == "mlstm" || t == "channel_delta") ? 1 : 0;
     return n;
 }
 
@@ -299,6 +317,7 @@ long long LLMEngineConfig::recurrent_state_bytes_per_seat() const {
     long long total = 0;
     for (const long long v : run_state_values) total += 4 * v;
     const int eb = element_bytes(dtype), tp = std::max(1, world_size);
+    for (const long long w : run_window_elements) total += eb * w;
     for (const auto& t : layer_types) {
         if (t == "mamba") {
             const long long inner = 1LL * mamba_num_heads * mamba_head_dim;
@@ -325,7 +344,7 @@ std::string LLMEngineConfig::validate() const {
     if (num_experts > 0 && (num_experts_per_tok <= 0 || num_experts_per_tok > num_experts)) return "num_experts_per_tok must be in 1..num_experts";
     for (const auto& t : layer_types) {
         if (t == "mamba" && (mamba_num_heads <= 0 || mamba_d_state <= 0)) return "a mamba layer needs the mamba section";
-        if (t == "mlstm" && run_state_values.size() != layer_types.size()) return "mlstm layers need their layer_specs";
+        if ((t == "mlstm" || t == "channel_delta") && run_state_values.size() != layer_types.size()) return t + " layers need their layer_specs";
         if (t == "gdn" && (gdn_num_v_heads <= 0 || gdn_head_k_dim <= 0)) return "a gdn layer needs the gdn section";
     }
     if (draft_type == "dflash" && dflash_block_size < 2) return "a block draft needs dflash_block_size >= 2";

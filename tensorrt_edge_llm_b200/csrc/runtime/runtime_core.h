@@ -74,7 +74,7 @@ struct LLMEngineConfig {
     bool has_qk_norm = false, attention_bias = false, attention_sink_bias = false, attention_k_eq_v = false, has_value_norm = false;
     int sliding_window = 0;                        // 0 = none
     std::vector<int> layer_windows;                // per layer (empty = sliding_window everywhere)
-    std::vector<std::string> layer_types;          // attention / mamba / gdn / mlstm / none per layer (per layer run of a looped stack)
+    std::vector<std::string> layer_types;          // attention / mamba / gdn / mlstm / channel_delta / none per layer (per layer run of a looped stack)
     std::vector<std::string> mlp_types;            // mlp / moe / none per layer
     int num_kv_shared_layers = 0;
     int num_experts = 0, num_experts_per_tok = 0, moe_intermediate_size = 0, shared_expert_intermediate_size = 0;
@@ -83,8 +83,9 @@ struct LLMEngineConfig {
     std::string lm_head_quantization;
     // recurrent mixers (0 when the model has none)
     int mamba_num_heads = 0, mamba_head_dim = 0, mamba_d_state = 0, mamba_n_groups = 0, mamba_conv_kernel = 0;
-    // stacks described layer by layer: per run, key + value elements per cached token and fp32 state values per seat (padded heads)
-    std::vector<long long> run_kv_elements, run_state_values;
+    // stacks described layer by layer: per run, cached elements per token, fp32 state values and 16-bit convolution history per seat
+    // (padded heads)
+    std::vector<long long> run_kv_elements, run_state_values, run_window_elements;
     int gdn_num_k_heads = 0, gdn_num_v_heads = 0, gdn_head_k_dim = 0, gdn_head_v_dim = 0, gdn_conv_kernel = 0;
     // draft heads
     std::string draft_type, dflash_projector_type;

@@ -1157,18 +1157,129 @@ def head_linear(x, weight, heads: int, x_col: int = 0, tail_col: int = -1, tail:
     return y
 
 
-def latent_attention(rows, kv_layer, meta: StepMeta, kv_up, key_up_t, spec) -> torch.Tensor:
-    """See :func:`ops.latent_attention`."""
+LATENT_FOLDED_COLUMNS = 128      # sequences with at most this many (row, head) pairs in a step read the cached latents directly
+
+
+class LatentPlan:
+    """How a step's sequences run in latent attention: a few rows per sequence against the cached latents themselves (the key expansion
+    folded into the query), prompt portions over keys and values expanded for them.  Built once per step."""
+
+    def __init__(self, meta: StepMeta, heads: int, device, force: Optional[str]):
+        self.key = (heads, force)
+        limit = {None: max(1, LATENT_FOLDED_COLUMNS // heads), "folded": 1 << 30, "expanded": 0}[force]
+        self.rows = self.expand = None                    # rows of the folded sequences (None: all rows), arrays of the expanded ones
+        self.folded = (meta.q_start, meta.q_len, meta.past_len, meta.page_table, meta.seq_ids, meta.num_tokens, meta.num_seqs, meta.max_q_len)
+        self.max_seq_len = meta.max_seq_len
+        if meta.max_q_len <= limit:
+            return
+        lens = meta.lengths()
+        i32 = dict(dtype=torch.int32, device=device)
+        start = [0]
+        for q, _ in lens:
+            start.append(start[-1] + q)
+        short = [i for i, (q, _) in enumerate(lens) if 0 < q <= limit]
+        long = [i for i, (q, _) in enumerate(lens) if q > limit]
+        kv_start, kv_rows = [], 0
+        for i in long:
+            kv_start.append(kv_rows)
+            kv_rows += sum(lens[i])
+        packed = torch.tensor([[start[i] for i in long], [lens[i][0] for i in long], [lens[i][1] for i in long], kv_start], **i32)
+        table = meta.page_table if len(long) == len(lens) else meta.page_table.index_select(0, torch.tensor(long, dtype=torch.int64, device=device))
+        self.expand = (packed[0], packed[1], packed[2], packed[3], table.contiguous(), len(long), max(lens[i][0] for i in long), kv_rows,
+                       max(sum(lens[i]) for i in long))
+        if not short:
+            self.folded = None
+            return
+        rows, q_start, seq_ids = [], [], []
+        for n, i in enumerate(short):
+            q_start.append(len(rows))
+            rows += range(start[i], start[i] + lens[i][0])
+            seq_ids += [n] * lens[i][0]
+        self.rows = torch.tensor(rows, dtype=torch.int64, device=device)
+        arr = torch.tensor([q_start, [lens[i][0] for i in short], [lens[i][1] for i in short]], **i32)
+        table = meta.page_table.index_select(0, torch.tensor(short, dtype=torch.int64, device=device))
+        self.folded = (arr[0], arr[1], arr[2], table, torch.tensor(seq_ids, **i32), len(rows), len(short), max(lens[i][0] for i in short))
+        self.max_seq_len = max(sum(lens[i]) for i in short)
+
+
+def _latent_plan(meta: StepMeta, heads: int, device, force: Optional[str]) -> LatentPlan:
+    for p in meta.plans or ():
+        if p.key == (heads, force):
+            return p
+    p = LatentPlan(meta, heads, device, force)
+    meta.plans = (meta.plans or ()) + (p,)
+    return p
+
+
+def _latent_splits(blocks: int, max_seq_len: int) -> int:
+    """Splits of the cached rows so that the (column block, split, sequence) CTAs, one per SM, come out near whole waves."""
+    tiles = max(1, (max_seq_len + 127) // 128)
+    if blocks >= 2 * 148 or tiles == 1:
+        return 1
+    best, cost = 1, None
+    for s in range(1, min(tiles, 32) + 1):
+        waves = (blocks * s + 147) // 148
+        c = waves * ((tiles + s - 1) // s + 0.7) + (0.4 if s > 1 else 0.0)      # in tiles; start-up and merge in the same unit
+        if cost is None or c < cost - 1e-9:
+            best, cost = s, c
+    return best
+
+
+def latent_attention(rows, kv_layer, meta: StepMeta, kv_up, key_up_t, spec, kernel: Optional[str] = None) -> torch.Tensor:
+    """See :func:`ops.latent_attention`.  16-bit steps run the tcgen05 kernels where the sizes fit (``kernel`` forces ``"folded"`` or
+    ``"expanded"``); fp32 rows and other sizes run on the CUDA cores (``"simt"``)."""
     if meta.tree_mask is not None:
         raise ValueError("latent attention covers causal masks only")
-    t, n = rows.shape[0], spec.num_heads
-    q = head_linear(rows, key_up_t, n, 0, n * spec.k_pad, spec.rot_pad)
-    o = torch.empty(t, n, spec.rank_pad, dtype=rows.dtype, device=rows.device)
-    _check(lib().telb_latent_attention_simt(
-        _p(q), _p(kv_layer), _p(o), _p(meta.q_start), _p(meta.past_len), _p(meta.seq_ids), _p(meta.page_table), c_int(t), c_int(meta.page_table.shape[1]),
-        c_int(meta.page_size), c_int(n), c_int(spec.pad), c_int(spec.rank_pad), c_float(spec.scale), c_int(_dtype_code(q)), _stream()), "latent_attention_simt")
-    value_up = kv_up[n * spec.k_pad:].view(n, spec.v_pad, spec.rank_pad)
-    return head_linear(o.view(t, -1), value_up, n).view(t, n * spec.v_pad)
+    t, n, dev = rows.shape[0], spec.num_heads, rows.device
+    tc = rows.dtype != torch.float32 and meta.page_size == 64 and spec.rank_pad <= 512 and spec.rot_pad == 64
+    expand_ok = tc and spec.v_pad <= 128 and spec.k_pad <= 256 and spec.scale > 0
+    if kernel == "simt" or not tc:
+        tc, kernel = False, "folded"
+    elif not expand_ok:
+        if kernel == "expanded":
+            raise ValueError("the expanded kernel does not cover this layer")
+        kernel = "folded"
+    plan = _latent_plan(meta, n, dev, kernel)
+    ws = Workspace.get(dev)
+    out = None
+    if plan.folded is not None:
+        q_start, q_len, past_len, table, seq_ids, tf, seqs, max_q = plan.folded
+        sub = rows if plan.rows is None else rows[:, :n * (spec.k_pad + spec.rot_pad)].index_select(0, plan.rows)
+        q = head_linear(sub, key_up_t, n, 0, n * spec.k_pad, spec.rot_pad)
+        o = torch.empty(tf, n, spec.rank_pad, dtype=rows.dtype, device=dev)
+        if tc:
+            nc = 16 if max_q * n <= 16 else 32
+            splits = _latent_splits(seqs * ((max_q * n + nc - 1) // nc), plan.max_seq_len)
+            _check(lib().telb_latent_attention_decode(
+                _p(q), _p(kv_layer), _p(o), _p(q_start), _p(q_len), _p(past_len), _p(table), c_int(seqs), c_int(tf), c_int(max_q),
+                c_int(kv_layer.shape[0]), c_int(table.shape[1]), c_int(n), c_int(spec.rank_pad), c_int(spec.rot_pad), c_float(spec.scale), c_int(splits),
+                _p(ws.attn_ws), c_ll(ws.attn_ws.numel()), c_int(_is_bf16(rows)), _p(ws.status), _stream()), "latent_attention_decode", 2 if splits > 1 else 1)
+        else:
+            _check(lib().telb_latent_attention_simt(
+                _p(q), _p(kv_layer), _p(o), _p(q_start), _p(past_len), _p(seq_ids), _p(table), c_int(tf), c_int(table.shape[1]), c_int(meta.page_size),
+                c_int(n), c_int(spec.pad), c_int(spec.rank_pad), c_float(spec.scale), c_int(_dtype_code(q)), _stream()), "latent_attention_simt")
+        value_up = kv_up[n * spec.k_pad:].view(n, spec.v_pad, spec.rank_pad)
+        res = head_linear(o.view(tf, -1), value_up, n).view(tf, n * spec.v_pad)
+        if plan.rows is None:
+            return res
+        out = torch.empty(t, n * spec.v_pad, dtype=rows.dtype, device=dev)
+        out.index_copy_(0, plan.rows, res)
+    if plan.expand is not None:
+        q_start, q_len, past_len, kv_start, table, seqs, max_q, kv_rows, max_total = plan.expand
+        es = rows.element_size()
+        latent = torch.empty(kv_rows, spec.rank_pad, dtype=rows.dtype, device=dev)
+        rot = torch.empty(kv_rows, spec.rot_pad, dtype=rows.dtype, device=dev)
+        _check(lib().telb_latent_gather(_p(kv_layer), _p(latent), _p(rot), _p(kv_start), _p(q_len), _p(past_len), _p(table), c_int(seqs), c_int(max_total),
+                                        c_int(table.shape[1]), c_int(meta.page_size), c_int(spec.rank_pad * es), c_int(spec.rot_pad * es), c_int(0), _stream()),
+               "latent_gather")
+        kv = gemm(latent, kv_up)
+        if out is None:
+            out = torch.empty(t, n * spec.v_pad, dtype=rows.dtype, device=dev)
+        _check(lib().telb_latent_attention_prefill(
+            _p(rows), _p(kv), _p(rot), _p(out), _p(q_start), _p(q_len), _p(past_len), _p(kv_start), c_int(seqs), c_int(t), c_int(max_q), c_int(kv_rows),
+            c_int(rows.shape[1]), c_int(n), c_int(spec.k_pad), c_int(spec.rot_pad), c_int(spec.v_pad), c_float(spec.scale), c_int(_is_bf16(rows)),
+            _p(ws.status), _stream()), "latent_attention_prefill")
+    return out
 
 
 # ---- speculative decoding -------------------------------------------------------------------------

@@ -49,6 +49,16 @@ class StepMeta:
     # Skip-softmax: fp32 [N] log2(lambda) per sequence (lambda = S / sequence length from the deployed scale table; -inf where
     # the sequence is shorter than the first calibrated length), or None when the deployment runs dense.
     skip_thr: Optional[torch.Tensor] = None
+    # What the host knows of the step: (q_len, past_len) per sequence (None: only the device tensors are valid, as in a captured
+    # decode step), and plans that ops derive from it once per step and share between layers.
+    host_lens: Optional[tuple] = None
+    plans: Optional[tuple] = None
+
+    def lengths(self) -> tuple:
+        """``(q_len, past_len)`` per sequence on the host (a device read when the step was built without them)."""
+        if self.host_lens is None:
+            return tuple(zip(self.q_len.tolist(), self.past_len.tolist()))
+        return self.host_lens
 
     @property
     def is_decode(self) -> bool:
@@ -100,4 +110,5 @@ def build_step_meta(q_lens: Sequence[int], past_lens: Sequence[int], page_table:
         logits_idx=torch.tensor(lidx, **i32), page_size=page_size, num_seqs=n, num_tokens=t,
         max_q_len=max(q_lens) if n else 0,
         max_seq_len=max((int(q) + int(p) for q, p in zip(q_lens, past_lens)), default=0),
-        tree_mask=tree_mask.to(device) if tree_mask is not None else None)
+        tree_mask=tree_mask.to(device) if tree_mask is not None else None,
+        host_lens=tuple((int(q), int(p)) for q, p in zip(q_lens, past_lens)))
