@@ -157,7 +157,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
     float* s_red = reinterpret_cast<float*>(tmem_slot + 4);     // [2 parities][4 warps][16] column maxima
     float* s_sum = s_red + 128;                                 // [4 warps][16] column sums (item epilogue)
 
-    pdl_prologue();          // step metadata and Q/KV are produced by earlier kernels
+    pdl_wait();              // step metadata and Q/KV are produced by earlier kernels
     const int warp = threadIdx.x >> 5;
     const int lane = threadIdx.x & 31;
 
@@ -197,6 +197,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
     __syncthreads();
     tc_fence_after_sync();
     const uint32_t tmem_base = *tmem_slot;
+    pdl_launch_dependents(); // after the allocation: a dependent that allocates ahead of its own wait must not take the columns first
     const unsigned long long t_start = p.trace ? global_timer_ns() : 0ull;
 
     if (warp == 0) {

@@ -5,7 +5,8 @@
 //                         Sᵀ[128 tok, NC] = rows[128 tok, rank + rot] · Qᵀ      Oᵀ[rank, NC] += latentᵀ[rank, 128 tok] · Pᵀ
 //                     A tile of rows is loaded once and serves both products (K-major for the scores, MN-major for the output).  It comes
 //                     in pairs of 64-feature chunks through a ring that holds at least one tile: scores start with the first pair, and a
-//                     pair's slot is refilled as soon as its 128 output features are done.
+//                     pair's slot is refilled as soon as its 128 output features are done.  The products are narrow, so consecutive ones go
+//                     to different accumulators (four for the scores, two output blocks in turn) instead of waiting for one another.
 //   latent_prefill    prompt portions, over keys and values expanded from the latents ([rows, heads, k | v], one product per step).  The
 //                     rotated key part is not expanded: a K tile is made of chunks of the head's keys and chunks of the shared rows.
 //                     256 query rows per CTA in two tiles with a softmax warpgroup each; probabilities stay in TMEM (the A operand
@@ -46,21 +47,30 @@ __device__ __forceinline__ float lat_warp_max(float v) {
     return r;
 }
 
+// Whether any of the 128 softmax threads says yes.
+__device__ __forceinline__ bool lat_any(bool yes) {
+    uint32_t r;
+    asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.u32 q, %1, 0;\n\tbar.red.or.pred p, 1, 128, q;\n\tselp.u32 %0, 1, 0, p;\n\t}"
+                 : "=r"(r) : "r"(yes ? 1u : 0u) : "memory");
+    return r != 0;
+}
+
 // grid (column blocks, splits, sequences).  NC: (token, head) columns of a block.
 template <typename T, int NC>
 __global__ void __launch_bounds__(kLatThreads, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_kv, const __grid_constant__ LatentDecParams p) {
     constexpr bool kBf16 = std::is_same<T, __nv_bfloat16>::value;
-    constexpr int kQChunk = NC * 128, kPHalf = 2 * NC * 128;
-    constexpr int kTmemCols = NC == 16 ? 128 : 256;      // S: NC columns, then one block of NC columns per 128 output features
-    static_assert(NC * 5 <= kTmemCols, "scores and four output blocks");
+    constexpr int kQChunk = NC * 128, kPSpan = 2 * NC * 128;         // [high | low rows of the columns][64 tokens]
+    constexpr int kOCol = 4 * NC, kOBlock = 2 * NC;      // TMEM: four partial scores, then per 128 output features high | low columns
+    constexpr int kTmemCols = NC == 16 ? 256 : 512;
+    static_assert(kOCol + 4 * kOBlock <= kTmemCols, "scores and four output blocks");
 
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     uint8_t* s_kv = smem;
     uint8_t* s_q = s_kv + p.slots * kLatSlot;
-    uint8_t* s_p = s_q + p.chunks * kQChunk;             // high half, low half
-    uint64_t* bars = reinterpret_cast<uint64_t*>(s_p + 2 * kPHalf);
+    uint8_t* s_p = s_q + p.chunks * kQChunk;             // two spans of 64 tokens
+    uint64_t* bars = reinterpret_cast<uint64_t*>(s_p + 2 * kPSpan);
     uint64_t* q_full = bars;
     uint64_t* s_full = bars + 1;
     uint64_t* p_full = bars + 2;
@@ -71,7 +81,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
     volatile uint32_t* abort_flag = tmem_slot + 1;
     float* s_red = reinterpret_cast<float*>(tmem_slot + 4);      // [4 warps][NC] maxima, then sums
 
-    pdl_prologue();
+    pdl_wait();                                           // dependents start once TMEM is allocated: theirs must not come first
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int seq = blockIdx.z, split = blockIdx.y, cb = blockIdx.x;
     const int qlen = p.q_len[seq], past = p.past_len[seq];
@@ -102,12 +112,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
         tmem_alloc(tmem_slot, kTmemCols);
         tmem_relinquish();
     }
-    for (int i = threadIdx.x; i < 2 * kPHalf / 16; i += kLatThreads) reinterpret_cast<uint4*>(s_p)[i] = make_uint4(0, 0, 0, 0);
+    for (int i = threadIdx.x; i < 2 * kPSpan / 16; i += kLatThreads) reinterpret_cast<uint4*>(s_p)[i] = make_uint4(0, 0, 0, 0);
     fence_proxy_async_smem();
     tc_fence_before_sync();
     __syncthreads();
     tc_fence_after_sync();
     const uint32_t tmem_base = *tmem_slot;
+    pdl_launch_dependents();
 
     if (warp == 0) {
         // ---- producer ----
@@ -141,7 +152,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
     } else if (warp == 1) {
         // ---- MMA issuer ----
         if (lane == 0 && ntiles > 0) {
-            const uint32_t idesc_s = idesc_f16(128, NC, kBf16), idesc_o = idesc_f16(128, NC, kBf16, true);
+            const uint32_t idesc_s = idesc_f16(128, NC, kBf16), idesc_o = idesc_f16(128, 2 * NC, kBf16, true);
             bool ok = mbar_wait(q_full, 0, abort_flag, p.status, kStatusMmaTimeout);
             for (int j = 0, n = 0; j < ntiles && ok; ++j) {
                 const int first = n;
@@ -155,7 +166,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                         const uint64_t dk = smem_desc_sw128(s_kv + slot * kLatSlot + c * kLatChunk);
                         const uint64_t dq = smem_desc_sw128(s_q + (pr * 2 + c) * kQChunk);
 #pragma unroll
-                        for (int k = 0; k < 4; ++k) umma_f16(tmem_base, dk + 2 * k, dq + 2 * k, idesc_s, (pr | c | k) ? 1u : 0u);
+                        for (int k = 0; k < 4; ++k) umma_f16(tmem_base + k * NC, dk + 2 * k, dq + 2 * k, idesc_s, (pr | c) ? 1u : 0u);
                     }
                     if (pr >= p.vblocks) umma_commit(&kv_empty[slot]);   // keys only
                 }
@@ -165,17 +176,20 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                 if (!ok) break;
                 tc_fence_after_sync();
                 const uint64_t dp = smem_desc_sw128(s_p);
-                for (int b = 0; b < p.vblocks; ++b) {
-                    const int slot = (first + b) % p.slots;
-                    const uint64_t dv = smem_desc_sw128_mn(s_kv + slot * kLatSlot, kLatChunk, 1024);
-                    const uint32_t d_o = tmem_base + NC * (1 + b);
+                for (int b = 0; b < p.vblocks; b += 2) {
+                    const bool two = b + 1 < p.vblocks;
+                    const int slot0 = (first + b) % p.slots, slot1 = (first + b + 1) % p.slots;
+                    const uint64_t dv0 = smem_desc_sw128_mn(s_kv + slot0 * kLatSlot, kLatChunk, 1024);
+                    const uint64_t dv1 = smem_desc_sw128_mn(s_kv + slot1 * kLatSlot, kLatChunk, 1024);
+                    const uint32_t d_o = tmem_base + kOCol + b * kOBlock;
 #pragma unroll
-                    for (int half = 0; half < 2; ++half)
-#pragma unroll
-                        for (int k = 0; k < kLatTile / 16; ++k)
-                            umma_f16(d_o, dv + (uint64_t)((k * 2048) >> 4), dp + (uint64_t)((half * kPHalf + (k >> 2) * (NC * 128)) >> 4) + 2 * (k & 3), idesc_o,
-                                     (j | half | k) ? 1u : 0u);
-                    umma_commit(&kv_empty[slot]);
+                    for (int k = 0; k < kLatTile / 16; ++k) {
+                        const uint64_t db = dp + (uint64_t)(((k >> 2) * kPSpan) >> 4) + 2 * (k & 3);
+                        umma_f16(d_o, dv0 + (uint64_t)((k * 2048) >> 4), db, idesc_o, (j | k) ? 1u : 0u);
+                        if (two) umma_f16(d_o + kOBlock, dv1 + (uint64_t)((k * 2048) >> 4), db, idesc_o, (j | k) ? 1u : 0u);
+                    }
+                    umma_commit(&kv_empty[slot0]);
+                    if (two) umma_commit(&kv_empty[slot1]);
                 }
             }
             if (ok) umma_commit(o_done);
@@ -198,53 +212,66 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
             float s[NC];
 #pragma unroll
             for (int c = 0; c < NC; c += 16) {
-                uint32_t raw[16];
-                tmem_ld_x16(lane_addr + c, raw);
+                uint32_t r0[16], r1[16], r2[16], r3[16];
+                tmem_ld_x16(lane_addr + c, r0);
+                tmem_ld_x16(lane_addr + NC + c, r1);
+                tmem_ld_x16(lane_addr + 2 * NC + c, r2);
+                tmem_ld_x16(lane_addr + 3 * NC + c, r3);
                 tmem_ld_wait();
 #pragma unroll
-                for (int i = 0; i < 16; ++i) s[c + i] = __uint_as_float(raw[i]);
+                for (int i = 0; i < 16; ++i)
+                    s[c + i] = (__uint_as_float(r0[i]) + __uint_as_float(r1[i]) + (__uint_as_float(r2[i]) + __uint_as_float(r3[i]))) * p.scale_log2;
             }
-            const int tk = (j0 + j) * kLatTile + r;
-            float* red = s_red + (j & 1) * 4 * NC;
+            const int t0 = (j0 + j) * kLatTile, tk = t0 + r;
+            if (t0 + kLatTile - 1 > past) {              // the tile reaches the first row's own position: mask
 #pragma unroll
-            for (int c = 0; c < NC; ++c) {
-                if (c < ncol) {
+                for (int c = 0; c < NC; ++c) {
                     const int qi = qlen == 1 ? 0 : (cb * NC + c) / p.heads;
-                    s[c] = tk <= past + qi ? s[c] * p.scale_log2 : -INFINITY;
-                    const float wm = lat_warp_max(s[c]);
-                    if (lane == (c & 31)) red[(warp - 2) * NC + c] = wm;
+                    if (tk > past + qi) s[c] = -INFINITY;
                 }
             }
-            named_barrier_sync(1, 128);
-            bool any_need = false;
-            float f[NC];
+            // the reference of a column moves only when a score exceeds it by 2^8: most tiles need no maximum
+            bool over = false;
 #pragma unroll
-            for (int c = 0; c < NC; ++c) {
-                f[c] = 1.f;
-                if (c < ncol) {
-                    const float mt = fmaxf(fmaxf(red[c], red[NC + c]), fmaxf(red[2 * NC + c], red[3 * NC + c]));
-                    if (mt > m_used[c] + 8.0f) {         // uniform across the four warps
-                        f[c] = m_used[c] == -INFINITY ? 0.f : exp2f(m_used[c] - mt);
-                        l_part[c] *= f[c];
-                        m_used[c] = mt;
-                        any_need = true;
+            for (int c = 0; c < NC; ++c) over = over || (c < ncol && s[c] > m_used[c] + 8.0f);
+            if (lat_any(over)) {
+                float* red = s_red + (j & 1) * 4 * NC;
+                float f[NC];
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    if (c < ncol) {
+                        const float wm = lat_warp_max(s[c]);
+                        if (lane == (c & 31)) red[(warp - 2) * NC + c] = wm;
                     }
                 }
-            }
-            if (j > 0 && any_need) {
-                for (int b = 0; b < p.vblocks; ++b)
+                named_barrier_sync(1, 128);
 #pragma unroll
-                    for (int c = 0; c < NC; c += 16) {
-                        uint32_t o[16];
-                        tmem_ld_x16(lane_addr + NC * (1 + b) + c, o);
-                        tmem_ld_wait();
-#pragma unroll
-                        for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * f[c + i]);
-                        tmem_st_x16(lane_addr + NC * (1 + b) + c, o);
+                for (int c = 0; c < NC; ++c) {
+                    f[c] = 1.f;
+                    if (c < ncol) {
+                        const float mt = fmaxf(fmaxf(red[c], red[NC + c]), fmaxf(red[2 * NC + c], red[3 * NC + c]));
+                        if (mt > m_used[c] + 8.0f) {     // uniform across the four warps
+                            f[c] = m_used[c] == -INFINITY ? 0.f : exp2f(m_used[c] - mt);
+                            l_part[c] *= f[c];
+                            m_used[c] = mt;
+                        }
                     }
-                tmem_st_wait();
+                }
+                if (j > 0) {
+                    for (int b = 0; b < p.vblocks; ++b)
+#pragma unroll
+                        for (int c = 0; c < 2 * NC; c += 16) {
+                            uint32_t o[16];
+                            tmem_ld_x16(lane_addr + kOCol + b * kOBlock + c, o);
+                            tmem_ld_wait();
+#pragma unroll
+                            for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * f[(c + i) % NC]);
+                            tmem_st_x16(lane_addr + kOCol + b * kOBlock + c, o);
+                        }
+                    tmem_st_wait();
+                }
             }
-            uint8_t* pbase = s_p + (r >> 6) * (NC * 128);
+            uint8_t* pbase = s_p + (r >> 6) * kPSpan;
             const int tl = r & 63;
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
@@ -254,7 +281,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                     uint8_t* dst = pbase + (c >> 3) * 1024 + (c & 7) * 128 + ((((tl >> 3) ^ (c & 7)) & 7) << 4) + (tl & 7) * 2;
                     const T hi = Cvt<T>::from_f(e);
                     *reinterpret_cast<T*>(dst) = hi;
-                    *reinterpret_cast<T*>(dst + kPHalf) = Cvt<T>::from_f(e - Cvt<T>::to_f(hi));
+                    *reinterpret_cast<T*>(dst + NC * 128) = Cvt<T>::from_f(e - Cvt<T>::to_f(hi));
                 }
             }
             fence_proxy_async_smem();
@@ -285,14 +312,15 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                 const int feat = b * 128 + r;
 #pragma unroll
                 for (int c = 0; c < NC; c += 16) {
-                    uint32_t o[16];
-                    tmem_ld_x16(lane_addr + NC * (1 + b) + c, o);    // garbage (never used) without tiles
+                    uint32_t o[16], lo[16];
+                    tmem_ld_x16(lane_addr + kOCol + b * kOBlock + c, o);       // garbage (never used) without tiles
+                    tmem_ld_x16(lane_addr + kOCol + b * kOBlock + NC + c, lo);
                     tmem_ld_wait();
                     if (feat >= p.rank_pad) continue;
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
                         if (c + i >= ncol) continue;
-                        const float v = inv[c + i] > 0.f ? __uint_as_float(o[i]) * inv[c + i] : 0.f;
+                        const float v = inv[c + i] > 0.f ? (__uint_as_float(o[i]) + __uint_as_float(lo[i])) * inv[c + i] : 0.f;
                         const size_t row = (size_t)row0 + c + i;
                         if (p.splits == 1) reinterpret_cast<T*>(p.out)[row * p.rank_pad + feat] = Cvt<T>::from_f(v);
                         else p.ws_o[((size_t)split * p.rows + row) * p.rank_pad + feat] = v;
@@ -393,7 +421,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(v_empty + kPreMaxStages);
     volatile uint32_t* abort_flag = tmem_slot + 1;
 
-    pdl_prologue();
+    pdl_wait();                                           // dependents start at the end: a long kernel runs slower under waiting ones
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int qt = gridDim.x - 1 - blockIdx.x;            // long rows first
     const int head = blockIdx.y, seq = blockIdx.z;
@@ -610,6 +638,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
     }
     tc_fence_before_sync();
     __syncthreads();
+    pdl_launch_dependents();
     if (warp == 1) {
         tc_fence_after_sync();
         tmem_dealloc(tmem_base, 512);

@@ -5,13 +5,22 @@
 //   S <- diag(g) S;  u = beta (v - Sᵀ k);  S <- S + k uᵀ;  o = Sᵀ q
 //   y = o / rms(o) · w · sigmoid(gate)
 //
-// Prompt portions run as four launches: `prep` (convolutions, norms as one scale per row and head, decays; parallel over tokens), `walk`
-// (the recurrence, state in registers), `out` (head norm and gate) and `roll` (convolution history).  A step with one row per
-// sequence runs `decode`: everything fused in one launch per layer when q / k heads are not shared, behind `prep` otherwise.
+// Prompt portions run as five launches: `prep` twice (values; q, k and decays: convolutions and norms, parallel over tokens), `walk` (the recurrence, state in
+// registers), `out` (head norm and gate) and `roll` (convolution history).  A step with one row per sequence runs `decode`, everything
+// in one launch (`roll` behind it when several heads share a q / k head).
 //
-// The walk never leaves fp32.  A head's state is cut into column slices that do not talk to each other: a warp owns 4 · CPL columns,
-// eight lanes share the rows of a column and hold RPL rows x CPL columns each, as packed row pairs (fma.rn.f32x2).  Because Sᵀk with
-// the decayed state equals Sᵀ(g ∘ k) with the old one, the decay of S runs beside the reduction that u waits for.
+// The walk takes four tokens at a time and never leaves fp32.  With S the state before a block, D_i = g_1 ∘ .. ∘ g_i and k, q normalised,
+//
+//   u_i = beta_i (v_i - Sᵀ(D_i ∘ k_i) - Σ_{j<i} m_ij u_j)        m_ij = Σ_c k_i k_j g_{j+1} .. g_i
+//   o_i = Sᵀ(D_i ∘ q_i) + Σ_{j<=i} n_ij u_j                      n_ij = Σ_c q_i k_j g_{j+1} .. g_i
+//   S  <- D_4 ∘ S + Σ_j (g_{j+1} .. g_4 ∘ k_j) u_jᵀ
+//
+// so the eight products with S do not wait for one another, and one reduction over lanes serves four tokens.  `prep` writes the three
+// vectors per token, D_4 and the scalars, computed from products of decays only (no quotients).  A head's state is cut into column slices that
+// do not talk to each other: a warp owns 4 · CPL columns, eight lanes share the rows of a column and hold RPL rows x CPL columns each,
+// as packed row pairs (fma.rn.f32x2).
+#include <type_traits>
+
 #include "host_utils.h"
 #include "tc5_common.cuh"
 
@@ -29,10 +38,8 @@ struct ChannelDeltaParams {
     const float* norm_w;       // [dv]
     void* conv_state;          // [slots, channels, taps - 1], oldest first
     float* state;              // [slots, heads, dk, dv]
-    void* mixed;               // [T, channels] scratch: convolved q | k | v
-    float* row_scale;          // [T, 2, kv_heads] scratch: 1 / |q|, 1 / |k|
-    float* g;                  // [T, heads * dk] scratch: decays
-    float* b;                  // [T, heads] scratch: step sizes
+    float* blocks;             // [blocks, heads, 13 dk + 32] scratch: per block of four tokens the vectors and scalars of the walk
+    void* v_blocks;            // [blocks, heads, dv, 4] scratch: convolved values
     void* o;                   // [T, heads * dv] scratch: read-outs
     void* out;                 // [T, heads * dv]
     const int* q_start;
@@ -40,6 +47,7 @@ struct ChannelDeltaParams {
     const int* past_len;
     const int* slot_ids;
     const int* seq_ids;
+    int* status;
     int tokens, num_seqs, heads, kv_heads, dk, dv, dk_real, dv_real, taps, channels, ld_decay, ld_gate, gate_f32;
     float eps;
 };
@@ -49,6 +57,18 @@ constexpr float kUnitEps = 1e-6f;
 __device__ __forceinline__ float cd_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float cd_silu(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float cd_softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// Activations of 16-bit models use the hardware's exponential; their results are rounded to 16 bits, and the decays keep fp32 accuracy:
+// the logarithm of 1 + e carries an absolute error of about 1e-7, no more than the rounding of the decay itself.
+template <typename T>
+__device__ __forceinline__ float cd_silu_as(float x) {
+    if constexpr (sizeof(T) == 4) return cd_silu(x);
+    else return __fdividef(x, 1.f + __expf(-x));
+}
+template <typename T>
+__device__ __forceinline__ float cd_decay_as(float rate, float z) {
+    if constexpr (sizeof(T) == 4) return expf(rate * cd_softplus(z));
+    else return __expf(rate * (fmaxf(z, 0.f) + __logf(1.f + __expf(-fabsf(z)))));
+}
 __device__ __forceinline__ float cd_warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -88,86 +108,183 @@ __device__ __forceinline__ void store_n(T* p, const T (&e)[N]) {
     }
 }
 
-// ---- prep: convolution + silu + norm scales, decays, step sizes ------------------------------------------
-constexpr int kPrepTokens = 8;       // rows per warp
+// ---- prep ------------------------------------------------------------------------------------------------
+constexpr int kBlk = 4;              // tokens of a block
+constexpr int kPrepTokens = 16;      // rows whose blocks a warp takes
+constexpr int kScalars = 32;         // m_21 m_31 m_32 m_41 m_42 m_43 | n_11 n_21 n_22 n_31 .. n_44 | beta_1 .. beta_4, padded
 
-// One head of q, k or v over rows t0 .. t1 - 1; a lane owns C consecutive channels.  W: window size, taps <= W.
+__host__ __device__ inline int block_floats(int dk) { return 13 * dk + kScalars; }
+// First block of a sequence: blocks count from the start of its portion, and those of different sequences never meet.
+__device__ __forceinline__ int first_block(int q_start, int seq) { return q_start / kBlk + seq; }
+
+// fp32 granule m (rows 4 m .. 4 m + 3 of a head) in the order of the walk's lanes: granules that its eight row groups read together lie
+// side by side.
+__device__ __forceinline__ int walk_granule(int dk, int m) { return dk >= 64 ? ((m >> 4) * 2 + (m & 1)) * 8 + ((m & 15) >> 1) : m; }
+
+// Taps of C channels from ch on, right-aligned in a window of W (taps <= W).
 template <typename T, int C, int W>
-__device__ void prep_conv(const ChannelDeltaParams& p, int ch0, int t0, int t1, float* scale, int scale_ld) {
-    const int lane = threadIdx.x & 31;
-    const int ch = ch0 + lane * C;
-    const T* x = reinterpret_cast<const T*>(p.qkv);
-    const T* cw = reinterpret_cast<const T*>(p.conv_w);
-    const T* cs = reinterpret_cast<const T*>(p.conv_state);
-    const int hist = p.taps - 1;
-    float w[W][C], win[W][C];
+__device__ __forceinline__ void load_taps(const ChannelDeltaParams& p, int ch, float (&w)[W][C]) {
+    const T* cw = reinterpret_cast<const T*>(p.conv_w) + (size_t)ch * p.taps;
+    if (p.taps == W) {                                    // C x W values in a row
+        float all[C * W];
+        load_n<T, C * W>(cw, all);
+#pragma unroll
+        for (int j = 0; j < W; ++j)
+#pragma unroll
+            for (int c = 0; c < C; ++c) w[j][c] = all[c * W + j];
+        return;
+    }
 #pragma unroll
     for (int j = 0; j < W; ++j)
 #pragma unroll
         for (int c = 0; c < C; ++c) {
             const int tap = j - (W - p.taps);
-            w[j][c] = tap >= 0 ? Cvt<T>::to_f(cw[(size_t)(ch + c) * p.taps + tap]) : 0.f;
-            win[j][c] = 0.f;
+            w[j][c] = tap >= 0 ? Cvt<T>::to_f(cw[(size_t)c * p.taps + tap]) : 0.f;
         }
-    int prev_seq = -1;
-    for (int t = t0; t < t1; ++t) {
-        const int seq = p.seq_ids[t];
-        const int i = t - p.q_start[seq];
-        if (seq != prev_seq) {                            // fill the window: earlier rows of the portion, then the kept history
-            prev_seq = seq;
-            const bool fresh = p.past_len[seq] == 0;
-            const size_t slot = (size_t)p.slot_ids[seq] * p.channels;
+}
+
+// Convolved and rounded rows i .. i + n - 1 of C channels from ch on (zero behind them).
+template <typename T, int C, int W>
+__device__ __forceinline__ void conv_block(const ChannelDeltaParams& p, const float (&w)[W][C], int ch, size_t t, int i, int n, const T* history, float (&y)[kBlk][C]) {
+    const T* x = reinterpret_cast<const T*>(p.qkv) + ch;
+    const int hist = p.taps - 1;
+    float rows[W - 1 + kBlk][C];
+    if (n == kBlk && i >= W - 1) {                        // inside the portion
 #pragma unroll
-            for (int j = 0; j < W - 1; ++j) {
-                const int back = W - 1 - j, r = i - back;
+        for (int j = 0; j < W - 1 + kBlk; ++j) load_n<T, C>(x + (t + j - (W - 1)) * p.channels, rows[j]);
+    } else {
 #pragma unroll
-                for (int c = 0; c < C; ++c) win[j + 1][c] = 0.f;
-                if (back > hist) continue;
-                if (r >= 0) {
-                    load_n<T, C>(x + (size_t)(t - back) * p.channels + ch, win[j + 1]);
-                } else if (!fresh) {
+        for (int j = 0; j < W - 1 + kBlk; ++j) {
+            const int d = j - (W - 1);                    // row relative to the block's first
 #pragma unroll
-                    for (int c = 0; c < C; ++c) win[j + 1][c] = Cvt<T>::to_f(cs[(slot + ch + c) * hist + hist + r]);
-                }
+            for (int c = 0; c < C; ++c) rows[j][c] = 0.f;
+            if (d < n && i + d >= 0 && d >= -hist) {
+                load_n<T, C>(x + (t + d) * p.channels, rows[j]);
+            } else if (d < 0 && d >= -hist && history) {
+#pragma unroll
+                for (int c = 0; c < C; ++c) rows[j][c] = Cvt<T>::to_f(history[(size_t)(ch + c) * hist + hist + i + d]);
             }
         }
+    }
 #pragma unroll
-        for (int j = 0; j < W - 1; ++j)
-#pragma unroll
-            for (int c = 0; c < C; ++c) win[j][c] = win[j + 1][c];
-        load_n<T, C>(x + (size_t)t * p.channels + ch, win[W - 1]);
-        T y[C];
-        float ss = 0.f;
+    for (int b = 0; b < kBlk; ++b)
 #pragma unroll
         for (int c = 0; c < C; ++c) {
             float acc = 0.f;
 #pragma unroll
-            for (int j = 0; j < W; ++j) acc = fmaf(w[j][c], win[j][c], acc);
-            y[c] = Cvt<T>::from_f(cd_silu(acc));
-            const float r = Cvt<T>::to_f(y[c]);
-            ss += r * r;
+            for (int j = 0; j < W; ++j) acc = fmaf(w[j][c], rows[b + j][c], acc);
+            y[b][c] = b < n ? Cvt<T>::to_f(Cvt<T>::from_f(cd_silu_as<T>(acc))) : 0.f;
         }
-        store_n<T, C>(reinterpret_cast<T*>(p.mixed) + (size_t)t * p.channels + ch, y);
-        if (scale) {
-            ss = cd_warp_sum(ss);
-            if (lane == 0) scale[(size_t)t * scale_ld] = 1.f / sqrtf(ss + kUnitEps);
+}
+
+// Totals of 32 values over the warp; lane l receives that of value l.
+__device__ __forceinline__ float total_of_lane(float (&v)[32], int lane) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const bool hi = lane & o;
+#pragma unroll
+        for (int i = 0; i < o; ++i) {
+            const float give = hi ? v[i] : v[i + o];
+            v[i] = (hi ? v[i + o] : v[i]) + __shfl_xor_sync(0xffffffffu, give, o);
         }
+    }
+    return v[0];
+}
+
+// q, k and decays of one head and block.
+template <typename T, int C, int W>
+__device__ __forceinline__ void prep_head(const ChannelDeltaParams& p, const float (&wq)[W][C], const float (&wk)[W][C], const float (&bias)[C], float rate, int h,
+                                          int seq, size_t t, int i, int n, const T* history) {
+    constexpr int V = C < 4 ? C : 4;
+    const int lane = threadIdx.x & 31, dk = p.dk, hk = h / (p.heads / p.kv_heads);
+    float q[kBlk][C], k[kBlk][C], g[kBlk][C];
+#pragma unroll
+    for (int b = 0; b < kBlk; ++b)
+        if (b < n) load_n<float, C>(p.decay + (t + b) * p.ld_decay + h * dk + lane * C, g[b]);
+    conv_block<T, C, W>(p, wq, hk * dk + lane * C, t, i, n, history, q);
+    conv_block<T, C, W>(p, wk, (p.kv_heads + hk) * dk + lane * C, t, i, n, history, k);
+#pragma unroll
+    for (int b = 0; b < kBlk; ++b)
+#pragma unroll
+        for (int c = 0; c < C; ++c) g[b][c] = b < n ? cd_decay_as<T>(rate, g[b][c] + bias[c]) : 1.f;
+    // values 0-5: m, 6-15: n, 16-19: |k|², 20-23: |q|²; ends[j]: k_j times the decays behind it
+    float sums[32], ends[kBlk][C];
+#pragma unroll
+    for (int x = 0; x < 32; ++x) sums[x] = 0.f;
+#pragma unroll
+    for (int j = 0; j < kBlk; ++j)
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+            float d = k[j][c];
+            sums[16 + j] = fmaf(d, d, sums[16 + j]);
+            sums[20 + j] = fmaf(q[j][c], q[j][c], sums[20 + j]);
+            sums[6 + j * (j + 1) / 2 + j] = fmaf(q[j][c], d, sums[6 + j * (j + 1) / 2 + j]);
+#pragma unroll
+            for (int x = j + 1; x < kBlk; ++x) {
+                d *= g[x][c];
+                sums[x * (x - 1) / 2 + j] = fmaf(k[x][c], d, sums[x * (x - 1) / 2 + j]);
+                sums[6 + x * (x + 1) / 2 + j] = fmaf(q[x][c], d, sums[6 + x * (x + 1) / 2 + j]);
+            }
+            ends[j][c] = d;
+        }
+    float total = total_of_lane(sums, lane);
+    const float inv = 1.f / sqrtf(total + kUnitEps);      // of use on lanes 16-23
+    float rk[kBlk], rq[kBlk];
+#pragma unroll
+    for (int b = 0; b < kBlk; ++b) {
+        rk[b] = __shfl_sync(0xffffffffu, inv, 16 + b);
+        rq[b] = __shfl_sync(0xffffffffu, inv, 20 + b) * rsqrtf((float)p.dk_real);
+    }
+    float* out = p.blocks + ((size_t)(first_block(p.q_start[seq], seq) + i / kBlk) * p.heads + h) * block_floats(dk);
+    // scalars: scale by the norms of their pair
+    float f = 1.f;
+#pragma unroll
+    for (int x = 0; x < kBlk; ++x)
+#pragma unroll
+        for (int j = 0; j <= x; ++j) {
+            if (j < x && lane == x * (x - 1) / 2 + j) f = rk[x] * rk[j];
+            if (lane == 6 + x * (x + 1) / 2 + j) f = rq[x] * rk[j];
+        }
+    total *= f;
+    if (lane >= 16) total = lane < 16 + n ? cd_sigmoid(p.beta[(t + lane - 16) * p.heads + h]) : 0.f;
+    out[13 * dk + lane] = total;
+    float d[C];
+#pragma unroll
+    for (int c = 0; c < C; ++c) d[c] = 1.f;
+#pragma unroll
+    for (int v = 0; v < C; v += V) {
+        const int ch = lane * C + v, at = walk_granule(dk, ch >> 2) * 4 + (ch & 3);
+#pragma unroll
+        for (int b = 0; b < kBlk; ++b) {
+            float x[V], y[V], z[V];
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+                d[v + e] *= g[b][v + e];
+                x[e] = d[v + e] * k[b][v + e] * rk[b];
+                y[e] = d[v + e] * q[b][v + e] * rq[b];
+                z[e] = ends[b][v + e] * rk[b];
+            }
+            store_n<float, V>(out + b * dk + at, x);
+            store_n<float, V>(out + (kBlk + b) * dk + at, y);
+            store_n<float, V>(out + (2 * kBlk + b) * dk + at, z);
+        }
+        float e4[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) e4[e] = d[v + e];
+        store_n<float, V>(out + 3 * kBlk * dk + at, e4);
     }
 }
 
-template <int C>
-__device__ void prep_decay(const ChannelDeltaParams& p, int h, int t0, int t1) {
-    const int lane = threadIdx.x & 31, col = h * p.dk + lane * C;
-    const float rate = -expf(p.a_log[h]);
-    float bias[C];
-    load_n<float, C>(p.decay_bias + col, bias);
-    for (int t = t0; t < t1; ++t) {
-        float z[C];
-        load_n<float, C>(p.decay + (size_t)t * p.ld_decay + col, z);
+template <typename T, int C, int W>
+__device__ __forceinline__ void prep_values(const ChannelDeltaParams& p, const float (&w)[W][C], int h, int seq, size_t t, int i, int n, const T* history) {
+    const int lane = threadIdx.x & 31;
+    float y[kBlk][C];
+    conv_block<T, C, W>(p, w, 2 * p.kv_heads * p.dk + h * p.dv + lane * C, t, i, n, history, y);
+    T* out = reinterpret_cast<T*>(p.v_blocks) + (((size_t)(first_block(p.q_start[seq], seq) + i / kBlk) * p.heads + h) * p.dv + lane * C) * kBlk;
 #pragma unroll
-        for (int c = 0; c < C; ++c) z[c] = expf(rate * cd_softplus(z[c] + bias[c]));
-        store_n<float, C>(p.g + (size_t)t * p.heads * p.dk + col, z);
-        if (lane == 0) p.b[(size_t)t * p.heads + h] = cd_sigmoid(p.beta[(size_t)t * p.heads + h]);
+    for (int c = 0; c < C; ++c) {
+        const T e[kBlk] = {Cvt<T>::from_f(y[0][c]), Cvt<T>::from_f(y[1][c]), Cvt<T>::from_f(y[2][c]), Cvt<T>::from_f(y[3][c])};
+        store_n<T, kBlk>(out + c * kBlk, e);
     }
 }
 
@@ -179,21 +296,40 @@ __device__ void prep_decay(const ChannelDeltaParams& p, int h, int t0, int t1) {
         default: { constexpr int C = 8; CALL; break; } \
     }
 
-template <typename T, int W>
+// The blocks that start in rows t0 .. t1 - 1.
+template <typename T, int C, int W, bool VALUES>
+__device__ void prep_range(const ChannelDeltaParams& p, int h, int t0, int t1) {
+    const int lane = threadIdx.x & 31, hk = h / (p.heads / p.kv_heads);
+    float w0[W][C], w1[VALUES ? 1 : W][C], bias[C];
+    float rate = 0.f;
+    if constexpr (VALUES) {
+        load_taps<T, C, W>(p, 2 * p.kv_heads * p.dk + h * p.dv + lane * C, w0);
+    } else {
+        load_taps<T, C, W>(p, hk * p.dk + lane * C, w0);
+        load_taps<T, C, W>(p, (p.kv_heads + hk) * p.dk + lane * C, w1);
+        load_n<float, C>(p.decay_bias + h * p.dk + lane * C, bias);
+        rate = -expf(p.a_log[h]);
+    }
+    for (int t = t0; t < t1;) {
+        const int seq = p.seq_ids[t], i = t - p.q_start[seq];
+        if (i % kBlk) {
+            t += min(kBlk - i % kBlk, p.q_len[seq] - i);
+            continue;
+        }
+        const int n = min(kBlk, p.q_len[seq] - i);
+        const T* history = p.past_len[seq] > 0 ? reinterpret_cast<const T*>(p.conv_state) + (size_t)p.slot_ids[seq] * p.channels * (p.taps - 1) : nullptr;
+        if constexpr (VALUES) prep_values<T, C, W>(p, w0, h, seq, t, i, n, history);
+        else prep_head<T, C, W>(p, w0, w1, bias, rate, h, seq, t, i, n, history);
+        t += n;
+    }
+}
+
+// grid (row ranges, heads).  VALUES: the value heads, else q, k and decays.
+template <typename T, int C, int W, bool VALUES>
 __global__ void __launch_bounds__(128) channel_delta_prep_kernel(const __grid_constant__ ChannelDeltaParams p) {
     pdl_prologue();
-    const int unit = blockIdx.y;                          // q heads, k heads, v heads, decays
-    const int t0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * kPrepTokens;
-    if (t0 >= p.tokens) return;
-    const int t1 = min(p.tokens, t0 + kPrepTokens);
-    const int nk = p.kv_heads;
-    if (unit < 2 * nk) {
-        TELB_BY_LANES(p.dk, (prep_conv<T, C, W>(p, unit * p.dk, t0, t1, p.row_scale + unit, 2 * nk)))
-    } else if (unit < 2 * nk + p.heads) {
-        TELB_BY_LANES(p.dv, (prep_conv<T, C, W>(p, 2 * nk * p.dk + (unit - 2 * nk) * p.dv, t0, t1, nullptr, 0)))
-    } else {
-        TELB_BY_LANES(p.dk, (prep_decay<C>(p, unit - 2 * nk - p.heads, t0, t1)))
-    }
+    const int t0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * kPrepTokens, t1 = min(p.tokens, t0 + kPrepTokens);
+    prep_range<T, C, W, VALUES>(p, blockIdx.y, t0, t1);
 }
 
 // History of the convolutions after a portion: the last taps - 1 inputs.
@@ -234,142 +370,89 @@ __device__ __forceinline__ f2 f2_mul(f2 a, f2 b) {
     asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
     return r;
 }
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async8(void* dst, const void* src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async4(void* dst, const void* src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
 // Rows of lane group rl (of 8): blocks of BL = min(8, RPL) rows, block j at rows j · 8 BL + rl · BL.
 template <int RPL>
 struct WalkRows {
     static constexpr int BL = RPL < 8 ? RPL : 8;
     static __device__ __forceinline__ int row(int rl, int i) { return (i / BL) * (8 * BL) + rl * BL + i % BL; }
-    // shared-memory place of fp32 granule m (rows 4 m .. 4 m + 3): granules that the eight groups read together lie side by side
-    static __device__ __forceinline__ int granule(int m) { return BL == 8 ? ((m >> 4) * 2 + (m & 1)) * 8 + ((m & 15) >> 1) : m; }
 };
 
-template <typename T, int RPL>
-__device__ __forceinline__ void walk_load(const T* s, int rl, f2 (&v)[RPL / 2]) {
-    constexpr int BL = WalkRows<RPL>::BL;
+// Totals over the eight lanes of a group of a[c][i] (products with k) and b[c][i] (with q), columns c of the lane, tokens i.  Even lanes
+// receive the four k sums of column walk_col, odd lanes the four q sums.
+template <int C>
+__device__ __forceinline__ int walk_col(int rl) { return C == 4 ? rl >> 1 : C == 2 ? (rl >> 1) & 1 : 0; }
+template <int C>
+__device__ __forceinline__ void walk_reduce(const float (&a)[C][kBlk], const float (&b)[C][kBlk], int rl, float (&w)[kBlk]) {
+    constexpr unsigned kAll = 0xffffffffu;
+    float s[C][kBlk];
+    const bool odd = rl & 1;
 #pragma unroll
-    for (int j = 0; j < RPL / BL; ++j) {
-        if constexpr (sizeof(T) == 4) {
+    for (int c = 0; c < C; ++c)
 #pragma unroll
-            for (int h = 0; h < BL / 4; ++h) {
-                const ulonglong2 u = *reinterpret_cast<const ulonglong2*>(s + ((j * (BL / 4) + h) * 8 + rl) * 4);
-                v[j * BL / 2 + h * 2] = u.x;
-                v[j * BL / 2 + h * 2 + 1] = u.y;
-            }
-        } else {
-            uint32_t u[BL / 2];
-            if constexpr (BL == 8) *reinterpret_cast<uint4*>(u) = *reinterpret_cast<const uint4*>(s + j * 64 + rl * 8);
-            else *reinterpret_cast<uint2*>(u) = *reinterpret_cast<const uint2*>(s + j * 32 + rl * 4);
+        for (int i = 0; i < kBlk; ++i) s[c][i] = (odd ? b[c][i] : a[c][i]) + __shfl_xor_sync(kAll, odd ? a[c][i] : b[c][i], 1);
+    const bool h2 = rl & 2, h4 = rl & 4;
+    if constexpr (C == 4) {
+        float x[2][kBlk];
 #pragma unroll
-            for (int i = 0; i < BL / 2; ++i) {
-                if constexpr (std::is_same<T, __nv_bfloat16>::value) {
-                    v[j * BL / 2 + i] = f2_pack(__uint_as_float(u[i] << 16), __uint_as_float(u[i] & 0xffff0000u));
-                } else {
-                    const float2 f = __half22float2(*reinterpret_cast<const __half2*>(&u[i]));
-                    v[j * BL / 2 + i] = f2_pack(f.x, f.y);
-                }
-            }
+        for (int i = 0; i < kBlk; ++i) {
+            x[0][i] = (h4 ? s[2][i] : s[0][i]) + __shfl_xor_sync(kAll, h4 ? s[0][i] : s[2][i], 4);
+            x[1][i] = (h4 ? s[3][i] : s[1][i]) + __shfl_xor_sync(kAll, h4 ? s[1][i] : s[3][i], 4);
+        }
+#pragma unroll
+        for (int i = 0; i < kBlk; ++i) w[i] = (h2 ? x[1][i] : x[0][i]) + __shfl_xor_sync(kAll, h2 ? x[0][i] : x[1][i], 2);
+    } else {
+#pragma unroll
+        for (int i = 0; i < kBlk; ++i) {
+            float x;
+            if constexpr (C == 2) x = (h2 ? s[1][i] : s[0][i]) + __shfl_xor_sync(kAll, h2 ? s[0][i] : s[1][i], 2);
+            else x = s[0][i] + __shfl_xor_sync(kAll, s[0][i], 2);
+            w[i] = x + __shfl_xor_sync(kAll, x, 4);
         }
     }
 }
 
-// Sums of C column values over the eight lanes of a group; a lane receives the sum of column walk_col<C>(rl).
-template <int C>
-__device__ __forceinline__ int walk_col(int rl) { return C == 4 ? rl >> 1 : C == 2 ? rl >> 2 : 0; }
-template <int C>
-__device__ __forceinline__ float walk_reduce(float (&a)[C], int rl) {
-    constexpr unsigned kAll = 0xffffffffu;
-    if constexpr (C == 4) {
-        const bool hi = rl & 4;
-        const float s0 = __shfl_xor_sync(kAll, hi ? a[0] : a[2], 4), s1 = __shfl_xor_sync(kAll, hi ? a[1] : a[3], 4);
-        const float b0 = (hi ? a[2] : a[0]) + s0, b1 = (hi ? a[3] : a[1]) + s1;
-        const bool h2 = rl & 2;
-        float v = (h2 ? b1 : b0) + __shfl_xor_sync(kAll, h2 ? b0 : b1, 2);
-        return v + __shfl_xor_sync(kAll, v, 1);
-    } else if constexpr (C == 2) {
-        const bool hi = rl & 4;
-        float v = (hi ? a[1] : a[0]) + __shfl_xor_sync(kAll, hi ? a[0] : a[1], 4);
-        v += __shfl_xor_sync(kAll, v, 2);
-        return v + __shfl_xor_sync(kAll, v, 1);
-    } else {
-        float v = a[0];
-        v += __shfl_xor_sync(kAll, v, 4);
-        v += __shfl_xor_sync(kAll, v, 2);
-        return v + __shfl_xor_sync(kAll, v, 1);
-    }
-}
-
-constexpr int kWalkTokens = 8;       // rows per stage
-constexpr int kWalkStages = 3;
-
-template <typename T>
-__host__ __device__ inline int walk_row_bytes(int dk, int cols) { return dk * (2 * (int)sizeof(T) + 4) + ((cols * (int)sizeof(T) + 15) & ~15) + 16; }
+constexpr int kWalkStages = 4;
 
 // grid (column slices of a head, heads, sequences); blockDim = warps of one slice
 template <typename T, int RPL, int CPL>
 __global__ void __launch_bounds__(128) channel_delta_walk_kernel(const __grid_constant__ ChannelDeltaParams p) {
-    pdl_prologue();
+    pdl_wait();                                           // dependents start at the end: a long kernel runs slower under waiting ones
     constexpr int DK = RPL * 8;
+    constexpr unsigned kAll = 0xffffffffu;
     extern __shared__ __align__(16) uint8_t walk_smem[];
+    __shared__ uint64_t full[kWalkStages];
+    __shared__ uint32_t abort_word;
+    volatile uint32_t* abort_flag = &abort_word;
     const int seq = blockIdx.z, h = blockIdx.y;
     const int ql = p.q_len[seq];
     if (ql <= 0) return;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nthr = blockDim.x;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int rl = lane & 7, cg = lane >> 3;
-    const int cols = (nthr >> 5) * 4 * CPL;               // columns of this CTA
-    const int col0 = blockIdx.x * cols;                   // within the head
-    const int lcol = warp * 4 * CPL + cg * CPL;           // first column of this lane, within the CTA
-    const int hk = h / (p.heads / p.kv_heads);
-    const size_t r0 = p.q_start[seq];
-    const int row_bytes = walk_row_bytes<T>(DK, cols), stage_bytes = row_bytes * kWalkTokens;
-    const T* mixed = reinterpret_cast<const T*>(p.mixed);
+    const int cols = (blockDim.x >> 5) * 4 * CPL;         // columns of this CTA
+    const int lcol = blockIdx.x * cols + warp * 4 * CPL + cg * CPL;      // first column of this lane, within the head
+    const int r0 = p.q_start[seq], blk0 = first_block(r0, seq);
+    const int chunks = (ql + kBlk - 1) / kBlk;
+    constexpr int kFloats = 13 * DK + kScalars;
+
+    const int v_bytes = cols * kBlk * (int)sizeof(T), stage_bytes = kFloats * 4 + v_bytes;
 
     auto fetch = [&](int chunk) {
-        const int first = chunk * kWalkTokens, n = min(kWalkTokens, ql - first);
+        uint64_t* bar = &full[chunk % kWalkStages];
         uint8_t* st = walk_smem + (chunk % kWalkStages) * stage_bytes;
-        constexpr int kQ = DK * (int)sizeof(T) / 16, kG = DK / 4;
-        const int kV = cols * (int)sizeof(T) / 8;
-        const int per = 2 * kQ + kG + kV + 3;
-        for (int idx = tid; idx < n * per; idx += nthr) {
-            const int i = idx / per;
-            int e = idx - i * per;
-            uint8_t* row = st + i * row_bytes;
-            const size_t t = r0 + first + i;
-            const T* m = mixed + t * p.channels;
-            if (e < 2 * kQ) {
-                const int qk = e >= kQ;
-                e -= qk * kQ;
-                const int dst = sizeof(T) == 4 ? WalkRows<RPL>::granule(e) : e;
-                cp_async16(row + qk * DK * (int)sizeof(T) + dst * 16, reinterpret_cast<const uint8_t*>(m + (qk * p.kv_heads + hk) * DK) + e * 16);
-            } else if (e < 2 * kQ + kG) {
-                e -= 2 * kQ;
-                cp_async16(row + 2 * DK * (int)sizeof(T) + WalkRows<RPL>::granule(e) * 16, p.g + (t * p.heads + h) * DK + e * 4);
-            } else if (e < 2 * kQ + kG + kV) {
-                e -= 2 * kQ + kG;
-                cp_async8(row + DK * (2 * (int)sizeof(T) + 4) + 16 + e * 8,
-                          reinterpret_cast<const uint8_t*>(m + 2 * p.kv_heads * DK + h * p.dv + col0) + e * 8);
-            } else {
-                e -= 2 * kQ + kG + kV;
-                const float* src = e == 2 ? p.b + t * p.heads + h : p.row_scale + t * 2 * p.kv_heads + e * p.kv_heads + hk;
-                cp_async4(row + DK * (2 * (int)sizeof(T) + 4) + e * 4, src);
-            }
-        }
+        const size_t blk = (size_t)(blk0 + chunk) * p.heads + h;
+        mbar_expect_tx(bar, stage_bytes);
+        bulk_load(st, p.blocks + blk * kFloats, kFloats * 4, bar);
+        bulk_load(st + kFloats * 4, reinterpret_cast<const T*>(p.v_blocks) + (blk * p.dv + blockIdx.x * cols) * kBlk, v_bytes, bar);
     };
+    if (tid == 0) {
+        for (int s = 0; s < kWalkStages; ++s) mbar_init(&full[s], 1);
+        abort_word = 0;
+        mbar_fence_init();
+        for (int s = 0; s < kWalkStages && s < chunks; ++s) fetch(s);
+    }
 
     f2 S[RPL / 2][CPL];
-    float* state = p.state + (((size_t)p.slot_ids[seq] * p.heads + h) * DK) * p.dv + col0 + lcol;
+    float* state = p.state + (((size_t)p.slot_ids[seq] * p.heads + h) * DK) * p.dv + lcol;
     if (p.past_len[seq] > 0) {
 #pragma unroll
         for (int i = 0; i < RPL / 2; ++i) {
@@ -385,68 +468,104 @@ __global__ void __launch_bounds__(128) channel_delta_walk_kernel(const __grid_co
 #pragma unroll
             for (int c = 0; c < CPL; ++c) S[i][c] = 0ull;
     }
-
-    const int chunks = (ql + kWalkTokens - 1) / kWalkTokens;
-#pragma unroll
-    for (int s = 0; s < kWalkStages - 1; ++s) {
-        if (s < chunks) fetch(s);
-        cp_async_commit();
-    }
-    const float q_scale = rsqrtf((float)p.dk_real);
     const int my_col = walk_col<CPL>(rl);
-    const bool writer = CPL == 4 ? !(rl & 1) : CPL == 2 ? !(rl & 3) : rl == 0;
-    T* out = reinterpret_cast<T*>(p.o) + r0 * p.heads * p.dv + (size_t)h * p.dv + col0 + lcol + my_col;
+    const bool writer = (rl & 1) && (CPL == 4 || (CPL == 2 ? !(rl & 4) : rl == 1));      // one odd lane per column
+    T* out = reinterpret_cast<T*>(p.o) + (size_t)r0 * p.heads * p.dv + (size_t)h * p.dv + lcol + my_col;
+    __syncthreads();
+    bool ok = true;
     for (int ch = 0; ch < chunks; ++ch) {
-        cp_async_wait<kWalkStages - 2>();
-        __syncthreads();
-        if (ch + kWalkStages - 1 < chunks) fetch(ch + kWalkStages - 1);
-        cp_async_commit();
-        const uint8_t* st = walk_smem + (ch % kWalkStages) * stage_bytes;
-        const int n = min(kWalkTokens, ql - ch * kWalkTokens);
-        for (int i = 0; i < n; ++i) {
-            const uint8_t* row = st + i * row_bytes;
-            const float* sc = reinterpret_cast<const float*>(row + DK * (2 * (int)sizeof(T) + 4));
-            f2 k[RPL / 2], g[RPL / 2];
-            walk_load<T, RPL>(reinterpret_cast<const T*>(row) + DK, rl, k);
-            walk_load<float, RPL>(reinterpret_cast<const float*>(row + 2 * DK * (int)sizeof(T)), rl, g);
-            const float v = Cvt<T>::to_f(reinterpret_cast<const T*>(sc + 4)[lcol + my_col]);
-            const float sk = sc[1], beta = sc[2];
-            f2 acc[CPL];
-            float a[CPL];
+        ok = mbar_wait(&full[ch % kWalkStages], (ch / kWalkStages) & 1, abort_flag, p.status, kStatusEpilogueTimeout);
+        if (!ok) break;
+        const float* st = reinterpret_cast<const float*>(walk_smem + (ch % kWalkStages) * stage_bytes);
+        // eight products with the state before the block: four rows of all vectors at a time, every product with a chain of its own
+        float a[CPL][kBlk], b[CPL][kBlk];
+        {
+            f2 acc[2 * kBlk][CPL];
 #pragma unroll
-            for (int c = 0; c < CPL; ++c) acc[c] = 0ull;
+            for (int j = 0; j < RPL / 4; ++j) {
+                ulonglong2 x[2 * kBlk];
 #pragma unroll
-            for (int r = 0; r < RPL / 2; ++r) {
-                const f2 kg = f2_mul(k[r], g[r]);
+                for (int i = 0; i < 2 * kBlk; ++i) x[i] = *reinterpret_cast<const ulonglong2*>(st + i * DK + (j * 8 + rl) * 4);
 #pragma unroll
-                for (int c = 0; c < CPL; ++c) acc[c] = f2_fma(S[r][c], kg, acc[c]);
+                for (int i = 0; i < 2 * kBlk; ++i)
+#pragma unroll
+                    for (int c = 0; c < CPL; ++c) acc[i][c] = j == 0 ? f2_mul(S[0][c], x[i].x) : f2_fma(S[2 * j][c], x[i].x, acc[i][c]);
+#pragma unroll
+                for (int i = 0; i < 2 * kBlk; ++i)
+#pragma unroll
+                    for (int c = 0; c < CPL; ++c) acc[i][c] = f2_fma(S[2 * j + 1][c], x[i].y, acc[i][c]);
             }
 #pragma unroll
-            for (int c = 0; c < CPL; ++c) a[c] = f2_sum(acc[c]);
-            const float sum = walk_reduce<CPL>(a, rl);
+            for (int c = 0; c < CPL; ++c)
 #pragma unroll
-            for (int r = 0; r < RPL / 2; ++r)
+                for (int i = 0; i < kBlk; ++i) {
+                    a[c][i] = f2_sum(acc[i][c]);
+                    b[c][i] = f2_sum(acc[kBlk + i][c]);
+                }
+        }
+        float w[kBlk];
+        walk_reduce<CPL>(a, b, rl, w);
+        alignas(16) float sc[20];
 #pragma unroll
-                for (int c = 0; c < CPL; ++c) S[r][c] = f2_mul(S[r][c], g[r]);
-            const float us = beta * (v - sk * sum) * sk;          // u times the norm scale of k
-            f2 q[RPL / 2];
-            walk_load<T, RPL>(reinterpret_cast<const T*>(row), rl, q);
+        for (int i = 0; i < 5; ++i) reinterpret_cast<float4*>(sc)[i] = reinterpret_cast<const float4*>(st + 13 * DK)[i];
+        float v[kBlk];
+        load_n<T, kBlk>(reinterpret_cast<const T*>(st + kFloats) + (lcol - (int)blockIdx.x * cols + my_col) * kBlk, v);
+        float u[kBlk];                                    // even lanes
+        u[0] = sc[16] * (v[0] - w[0]);
+        u[1] = sc[17] * (v[1] - w[1] - sc[0] * u[0]);
+        u[2] = sc[18] * (v[2] - w[2] - sc[1] * u[0] - sc[2] * u[1]);
+        u[3] = sc[19] * (v[3] - w[3] - sc[3] * u[0] - sc[4] * u[1] - sc[5] * u[2]);
+        float mine[kBlk];                                 // odd lanes: the steps of their column
+#pragma unroll
+        for (int i = 0; i < kBlk; ++i) mine[i] = __shfl_xor_sync(kAll, u[i], 1);
+        f2 ub[CPL][kBlk];
+#pragma unroll
+        for (int c = 0; c < CPL; ++c)
+#pragma unroll
+            for (int i = 0; i < kBlk; ++i) {
+                const float x = CPL == 1 ? (rl & 1 ? mine[i] : u[i]) : __shfl_sync(kAll, u[i], (lane & 24) | (c * 2));
+                ub[c][i] = f2_pack(x, x);
+            }
+        if (writer) {
+            const int n = min(kBlk, ql - ch * kBlk);
+            float o[kBlk];
+            o[0] = w[0] + sc[6] * mine[0];
+            o[1] = w[1] + sc[7] * mine[0] + sc[8] * mine[1];
+            o[2] = w[2] + sc[9] * mine[0] + sc[10] * mine[1] + sc[11] * mine[2];
+            o[3] = w[3] + sc[12] * mine[0] + sc[13] * mine[1] + sc[14] * mine[2] + sc[15] * mine[3];
+#pragma unroll
+            for (int i = 0; i < kBlk; ++i)
+                if (i < n) out[(size_t)i * p.heads * p.dv] = Cvt<T>::from_f(o[i]);
+        }
+        out += (size_t)kBlk * p.heads * p.dv;
+#pragma unroll
+        for (int j = 0; j < RPL / 4; ++j) {
+            ulonglong2 x[kBlk + 1];                       // D_4 is the vector behind the four
+#pragma unroll
+            for (int i = 0; i <= kBlk; ++i) x[i] = *reinterpret_cast<const ulonglong2*>(st + (2 * kBlk + i) * DK + (j * 8 + rl) * 4);
 #pragma unroll
             for (int c = 0; c < CPL; ++c) {
-                const float uc = __shfl_sync(0xffffffffu, us, (lane & 24) | (CPL == 4 ? c * 2 : CPL == 2 ? c * 4 : 0));
-                const f2 u2 = f2_pack(uc, uc);
-                acc[c] = 0ull;
-#pragma unroll
-                for (int r = 0; r < RPL / 2; ++r) {
-                    S[r][c] = f2_fma(k[r], u2, S[r][c]);
-                    acc[c] = f2_fma(S[r][c], q[r], acc[c]);
-                }
+                S[2 * j][c] = f2_mul(S[2 * j][c], x[kBlk].x);
+                S[2 * j + 1][c] = f2_mul(S[2 * j + 1][c], x[kBlk].y);
             }
 #pragma unroll
-            for (int c = 0; c < CPL; ++c) a[c] = f2_sum(acc[c]);
-            const float o = walk_reduce<CPL>(a, rl) * sc[0] * q_scale;
-            if (writer) out[(size_t)(ch * kWalkTokens + i) * p.heads * p.dv] = Cvt<T>::from_f(o);
+            for (int i = 0; i < kBlk; ++i)
+#pragma unroll
+                for (int c = 0; c < CPL; ++c) {
+                    S[2 * j][c] = f2_fma(x[i].x, ub[c][i], S[2 * j][c]);
+                    S[2 * j + 1][c] = f2_fma(x[i].y, ub[c][i], S[2 * j + 1][c]);
+                }
         }
+        if (ch + kWalkStages < chunks) {                  // every warp is done with the stage: refill it
+            __syncthreads();
+            if (tid == 0) fetch(ch + kWalkStages);
+        }
+    }
+    pdl_launch_dependents();
+    if (!ok) {                                            // a copy never arrived: leave the state alone, let what is in flight land
+        const uint64_t t0 = global_timer_ns();
+        while (global_timer_ns() - t0 < 200000ull) __nanosleep(1000);
+        return;
     }
 #pragma unroll
     for (int i = 0; i < RPL / 2; ++i) {
@@ -473,7 +592,7 @@ __device__ void delta_out(const ChannelDeltaParams& p, size_t t, int h) {
     const float inv = 1.f / sqrtf(cd_warp_sum(ss) / p.dv_real + p.eps);
     T y[C];
 #pragma unroll
-    for (int c = 0; c < C; ++c) y[c] = Cvt<T>::from_f(o[c] * inv * w[c] * cd_sigmoid(z[c]));
+    for (int c = 0; c < C; ++c) y[c] = Cvt<T>::from_f(o[c] * inv * w[c] * (sizeof(T) == 4 ? cd_sigmoid(z[c]) : __fdividef(1.f, 1.f + __expf(-z[c]))));
     store_n<T, C>(reinterpret_cast<T*>(p.out) + t * p.heads * p.dv + col, y);
 }
 
@@ -489,8 +608,8 @@ __global__ void __launch_bounds__(128) channel_delta_out_kernel(const __grid_con
 
 // ---- decode: one row per sequence, everything in one CTA per (head, sequence) -----------------------------
 // Eight warps share the rows of S; a lane owns DV / 32 columns of its warp's DK / 8 rows, in registers from load to store.
-// FUSED: q, k, v are convolved here (their heads are not shared); otherwise `prep` has run.
-template <typename T, int DK, int DV, bool FUSED>
+// The convolution history is rolled here unless heads share q and k (they would read what another CTA rolls).
+template <typename T, int DK, int DV>
 __global__ void __launch_bounds__(256) channel_delta_decode_kernel(const __grid_constant__ ChannelDeltaParams p) {
     pdl_prologue();
     constexpr int R = DK / 8, C = DV / 32;
@@ -512,35 +631,24 @@ __global__ void __launch_bounds__(256) channel_delta_decode_kernel(const __grid_
 #pragma unroll
             for (int c = 0; c < C; ++c) S[r][c] = 0.f;
     }
-    const T* x = reinterpret_cast<const T*>(FUSED ? p.qkv : p.mixed) + t * p.channels;
-    const T* raw = reinterpret_cast<const T*>(p.qkv) + t * p.channels;
+    const T* x = reinterpret_cast<const T*>(p.qkv) + t * p.channels;
     for (int i = tid; i < 2 * DK + DV; i += 256) {
         const int ch = i < DK ? hk * DK + i : i < 2 * DK ? p.kv_heads * DK + hk * DK + i - DK : 2 * p.kv_heads * DK + h * DV + i - 2 * DK;
         T* cs = reinterpret_cast<T*>(p.conv_state) + (slot * p.channels + ch) * hist;
-        float y = Cvt<T>::to_f(x[ch]);
-        if constexpr (FUSED) {
-            const T* cw = reinterpret_cast<const T*>(p.conv_w) + (size_t)ch * p.taps;
-            float acc = 0.f;
-            if (!fresh)
-                for (int j = 0; j < hist; ++j) acc = fmaf(Cvt<T>::to_f(cw[j]), Cvt<T>::to_f(cs[j]), acc);
-            acc = fmaf(Cvt<T>::to_f(cw[hist]), y, acc);
-            y = Cvt<T>::to_f(Cvt<T>::from_f(cd_silu(acc)));
-        }
-        if (hist > 0 && (i >= 2 * DK || h % group == 0)) {             // this CTA keeps the history of the channel
+        const T* cw = reinterpret_cast<const T*>(p.conv_w) + (size_t)ch * p.taps;
+        float acc = 0.f;
+        if (!fresh)
+            for (int j = 0; j < hist; ++j) acc = fmaf(Cvt<T>::to_f(cw[j]), Cvt<T>::to_f(cs[j]), acc);
+        acc = fmaf(Cvt<T>::to_f(cw[hist]), Cvt<T>::to_f(x[ch]), acc);
+        const float y = Cvt<T>::to_f(Cvt<T>::from_f(cd_silu_as<T>(acc)));
+        if (hist > 0 && group == 1) {
             for (int j = 0; j + 1 < hist; ++j) cs[j] = fresh ? Cvt<T>::from_f(0.f) : cs[j + 1];
-            cs[hist - 1] = raw[ch];
+            cs[hist - 1] = x[ch];
         }
         (i < DK ? s_q[i] : i < 2 * DK ? s_k[i - DK] : s_v[i - 2 * DK]) = y;
     }
-    float beta;
-    if constexpr (FUSED) {
-        const float rate = -expf(p.a_log[h]);
-        for (int i = tid; i < DK; i += 256) s_g[i] = expf(rate * cd_softplus(p.decay[t * p.ld_decay + h * DK + i] + p.decay_bias[h * DK + i]));
-        beta = cd_sigmoid(p.beta[t * p.heads + h]);
-    } else {
-        for (int i = tid; i < DK; i += 256) s_g[i] = p.g[(t * p.heads + h) * DK + i];
-        beta = p.b[t * p.heads + h];
-    }
+    const float rate = -expf(p.a_log[h]), beta = cd_sigmoid(p.beta[t * p.heads + h]);
+    for (int i = tid; i < DK; i += 256) s_g[i] = cd_decay_as<T>(rate, p.decay[t * p.ld_decay + h * DK + i] + p.decay_bias[h * DK + i]);
     __syncthreads();
     float qq = 0.f, kk = 0.f, qk = 0.f;                                 // every warp: |q|², |k|², q·k
     for (int i = lane; i < DK; i += 32) {
@@ -613,35 +721,56 @@ __global__ void __launch_bounds__(256) channel_delta_decode_kernel(const __grid_
 template <typename T>
 static int launch_prep(const ChannelDeltaParams& p, cudaStream_t stream) {
     const int warps = (p.tokens + kPrepTokens - 1) / kPrepTokens;
-    const dim3 grid((warps + 3) / 4, 2 * p.kv_heads + 2 * p.heads);
-    if (p.taps <= 4) TELB_LAUNCH("channel_delta_prep_kernel", (channel_delta_prep_kernel<T, 4>), grid, dim3(128), 0, stream, p);
-    else TELB_LAUNCH("channel_delta_prep_kernel", (channel_delta_prep_kernel<T, 8>), grid, dim3(128), 0, stream, p);
+    const dim3 grid((warps + 3) / 4, p.heads);
+#define TELB_PREP(W_, VALUES_) TELB_LAUNCH("channel_delta_prep_kernel", (channel_delta_prep_kernel<T, C, W_, VALUES_>), grid, dim3(128), 0, stream, p)
+    if (p.taps <= 4) {
+        TELB_BY_LANES(p.dv, TELB_PREP(4, true))
+        TELB_BY_LANES(p.dk, TELB_PREP(4, false))
+    } else {
+        TELB_BY_LANES(p.dv, TELB_PREP(8, true))
+        TELB_BY_LANES(p.dk, TELB_PREP(8, false))
+    }
+#undef TELB_PREP
     TELB_CHECK_LAUNCH("channel_delta_prep_kernel");
     return 0;
 }
 
+template <typename T>
+static int launch_roll(const ChannelDeltaParams& p, cudaStream_t stream) {
+    if (p.taps < 2) return 0;
+    TELB_LAUNCH("channel_delta_roll_kernel", (channel_delta_roll_kernel<T>), dim3((p.channels + 127) / 128, p.num_seqs), dim3(128), 0, stream, p);
+    TELB_CHECK_LAUNCH("channel_delta_roll_kernel");
+    return 0;
+}
+
 template <typename T, int RPL, int CPL>
-static int launch_walk_as(const ChannelDeltaParams& p, int warps, cudaStream_t stream) {
-    while (warps > 1 && p.dv % (warps * 4 * CPL)) warps >>= 1;
-    const int cols = warps * 4 * CPL;
-    const size_t smem = (size_t)walk_row_bytes<T>(RPL * 8, cols) * kWalkTokens * kWalkStages;
+static int launch_walk_as(const ChannelDeltaParams& p, cudaStream_t stream) {
+    constexpr int warps = CPL == 1 ? 4 : 2, cols = warps * 4 * CPL;      // 16 or 32: divides every padded head
+    constexpr int smem = ((13 * RPL * 8 + kScalars) * 4 + cols * kBlk * (int)sizeof(T)) * kWalkStages;
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(channel_delta_walk_kernel<T, RPL, CPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return fail("cudaFuncSetAttribute(channel_delta_walk)", e);
+        static bool configured = false;
+        if (!configured) {
+            cudaError_t e = cudaFuncSetAttribute(channel_delta_walk_kernel<T, RPL, CPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+            if (e != cudaSuccess) return fail("cudaFuncSetAttribute(channel_delta_walk)", e);
+            configured = true;
+        }
     }
-    TELB_LAUNCH("channel_delta_walk_kernel", (channel_delta_walk_kernel<T, RPL, CPL>), dim3(p.dv / cols, p.heads, p.num_seqs), dim3(warps * 32), smem,
-                stream, p);
+    TELB_LAUNCH_SERIAL("channel_delta_walk_kernel", (channel_delta_walk_kernel<T, RPL, CPL>), dim3(p.dv / cols, p.heads, p.num_seqs), dim3(warps * 32), smem, stream, p);
     TELB_CHECK_LAUNCH("channel_delta_walk_kernel");
     return 0;
 }
 
+static int g_walk_cols = 0;          // columns per lane; 0 = by the number of columns
+
 template <typename T, int RPL>
 static int launch_walk(const ChannelDeltaParams& p, cudaStream_t stream) {
-    // few (sequence, head) pairs: narrow slices, one warp each, so that every scheduler has a chain of its own
+    // few (sequence, head) pairs: narrow slices, so that every scheduler has a chain of its own; many: wide ones, which read less
     const long long columns = (long long)p.num_seqs * p.heads * p.dv;
-    if (columns / 4 <= 4LL * sm_count()) return launch_walk_as<T, RPL, 1>(p, 1, stream);
-    if (RPL > 16 || columns / 8 <= 4LL * sm_count()) return launch_walk_as<T, RPL, 2>(p, columns / 8 <= 4LL * sm_count() ? 1 : 4, stream);
-    return launch_walk_as<T, RPL, (RPL > 16 ? 2 : 4)>(p, columns / 16 <= 4LL * sm_count() ? 1 : 2, stream);
+    int cpl = columns / 4 <= 8LL * sm_count() ? 1 : (RPL > 16 || columns / 8 <= 8LL * sm_count()) ? 2 : 4;
+    if (g_walk_cols) cpl = g_walk_cols;
+    if (cpl == 1) return launch_walk_as<T, RPL, 1>(p, stream);
+    if (cpl == 2 || RPL > 16) return launch_walk_as<T, RPL, 2>(p, stream);
+    return launch_walk_as<T, RPL, (RPL > 16 ? 2 : 4)>(p, stream);
 }
 
 template <typename T>
@@ -658,24 +787,15 @@ static int channel_delta_rows(const ChannelDeltaParams& p, cudaStream_t stream) 
     const long long warps = (long long)p.tokens * p.heads;
     TELB_LAUNCH("channel_delta_out_kernel", (channel_delta_out_kernel<T>), dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, stream, p);
     TELB_CHECK_LAUNCH("channel_delta_out_kernel");
-    if (p.taps > 1) {
-        TELB_LAUNCH("channel_delta_roll_kernel", (channel_delta_roll_kernel<T>), dim3((p.channels + 127) / 128, p.num_seqs), dim3(128), 0, stream, p);
-        TELB_CHECK_LAUNCH("channel_delta_roll_kernel");
-    }
-    return 0;
+    return launch_roll<T>(p, stream);
 }
 
 template <typename T, int DK, int DV>
 static int launch_decode_step(const ChannelDeltaParams& p, cudaStream_t stream) {
     const dim3 grid(p.heads, p.num_seqs);
-    if (p.heads == p.kv_heads) {
-        TELB_LAUNCH("channel_delta_decode_kernel", (channel_delta_decode_kernel<T, DK, DV, true>), grid, dim3(256), 0, stream, p);
-    } else {
-        if (launch_prep<T>(p, stream)) return -1;
-        TELB_LAUNCH("channel_delta_decode_kernel", (channel_delta_decode_kernel<T, DK, DV, false>), grid, dim3(256), 0, stream, p);
-    }
+    TELB_LAUNCH("channel_delta_decode_kernel", (channel_delta_decode_kernel<T, DK, DV>), grid, dim3(256), 0, stream, p);
     TELB_CHECK_LAUNCH("channel_delta_decode_kernel");
-    return 0;
+    return p.heads == p.kv_heads ? 0 : launch_roll<T>(p, stream);
 }
 
 template <typename T, int DK>
@@ -696,7 +816,14 @@ static int channel_delta_step(const ChannelDeltaParams& p, cudaStream_t stream) 
 
 using namespace telb;
 
-// dtype: 0 fp16, 1 bf16, 2 fp32 (of qkv, conv_w, conv_state, mixed, o, out and, unless gate_f32, gate).
+// Columns per lane of the walk: 1, 2 or 4; 0 picks by the number of columns.  Process-wide.
+extern "C" int telb_set_delta_walk_columns(int n) {
+    if (n != 0 && n != 1 && n != 2 && n != 4) return fail("telb_set_delta_walk_columns: 0, 1, 2 or 4");
+    g_walk_cols = n;
+    return 0;
+}
+
+// dtype: 0 fp16, 1 bf16, 2 fp32 (of qkv, conv_w, conv_state, v_blocks, o, out and, unless gate_f32, gate).
 // decode != 0: every sequence has at most one row and dk, dv <= 128.
 extern "C" int telb_channel_delta(const ChannelDeltaParams* pp, int decode, int dtype, cudaStream_t stream) {
     const ChannelDeltaParams& p = *pp;
@@ -705,7 +832,7 @@ extern "C" int telb_channel_delta(const ChannelDeltaParams* pp, int decode, int 
     if (!size_ok(p.dk) || !size_ok(p.dv)) return fail("telb_channel_delta: padded head sizes are 32, 64, 128 or 256");
     if (p.taps < 1 || p.taps > 8) return fail("telb_channel_delta: convolutions have 1 to 8 taps");
     if (p.kv_heads <= 0 || p.heads % p.kv_heads) return fail("telb_channel_delta: heads must be a multiple of the q / k heads");
-    if (p.num_seqs > 65535 || p.heads > 65535 / 4) return fail("telb_channel_delta: too many sequences or heads");
+    if (p.num_seqs > 65535 || p.heads > 65535) return fail("telb_channel_delta: too many sequences or heads");
     if (decode) {
         if (p.dk > 128 || p.dv > 128) return fail("telb_channel_delta: the decode step covers heads up to 128");
         if (dtype == 2) return channel_delta_step<float>(p, stream);

@@ -176,6 +176,24 @@ inline cudaError_t launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, s
         if (e__ != cudaSuccess) return ::telb::fail(name, e__);                                     \
     } while (0)
 
+// The same without programmatic dependent launch: the grid starts on an empty device.  For long kernels of few CTAs, which would
+// otherwise settle on the few SMs that the kernel before leaves first and share those while others idle.
+template <typename... KArgs, typename... Args>
+inline cudaError_t launch_serial(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args&&... args) {
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = stream;
+    return cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
+}
+
+#define TELB_LAUNCH_SERIAL(name, kernel, grid, block, smem, stream, ...)                            \
+    do {                                                                                            \
+        cudaError_t e__ = ::telb::launch_serial(kernel, grid, block, smem, stream, __VA_ARGS__);    \
+        if (e__ != cudaSuccess) return ::telb::fail(name, e__);                                     \
+    } while (0)
+
 inline int sm_count() {
     static int n = 0;
     if (!n) {

@@ -6,6 +6,8 @@
 //   latent_gather    cached latent rows of the step's sequences, back to back (input of the key / value expansion)
 //
 // Norms, rotation and sums are fp32; inputs and outputs have the activation type.
+#include <type_traits>
+
 #include "host_utils.h"
 #include "tc5_common.cuh"
 
@@ -17,90 +19,122 @@ __device__ __forceinline__ T* cache_row(T* kv, const int* page_table, int max_pa
     return page < 0 ? nullptr : kv + ((size_t)page * page_rows + slot % page_size) * width;
 }
 
-// One CTA per row.  Columns: q [heads * kp] | q rotated [heads * rp] | latent [rank_pad] | key rotated [rp].
+// One CTA per row.  Columns: q [heads * kp] | q rotated [heads * rp] | latent [rank_pad] | key rotated [rp].  A thread takes one pair of
+// neighbours (one rotation) at a time.
+constexpr int kLatWriteThreads = 256;
+
+template <typename T> struct Pair;
+template <> struct Pair<float> { typedef float2 word; };
+template <> struct Pair<__nv_bfloat16> { typedef uint32_t word; };
+template <> struct Pair<__half> { typedef uint32_t word; };
+
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kLatWriteThreads)
 latent_write_kernel(T* rows, T* kv, const float* cos_sin, const float* norm_w, const int* positions, const int* seq_ids, const int* q_start,
                     const int* past_len, const int* page_table, int max_pages, int page_size, int heads, int kp, int rp, int rank_pad, int rank, int rot,
                     int table_ld, float eps) {
     pdl_prologue();
-    __shared__ float red[4];
+    typedef typename Pair<T>::word Word;
+    __shared__ float red[kLatWriteThreads / 32];
     const int t = blockIdx.x, tid = threadIdx.x;
     const size_t ld = (size_t)heads * (kp + rp) + rank_pad + rp;
     T* qr = rows + t * ld + (size_t)heads * kp;
     const T* c = qr + (size_t)heads * rp;
     const T* kr = c + rank_pad;
+    const int s = seq_ids[t];
+    T* dst = cache_row(kv, page_table, max_pages, page_size, s, past_len[s] + t - q_start[s], page_size, rank_pad + rp);
     const float* cs = cos_sin + (size_t)positions[t] * table_ld;
-    const int half = rot / 2;
-    for (int i = tid; i < heads * half; i += 128) {
-        const int h = i / half, j = i - h * half;
-        T* pair = qr + h * rp + 2 * j;
-        const float u = Cvt<T>::to_f(pair[0]), v = Cvt<T>::to_f(pair[1]), co = cs[j], si = cs[half + j];
-        pair[0] = Cvt<T>::from_f(u * co - v * si);
-        pair[1] = Cvt<T>::from_f(v * co + u * si);
-    }
+    const int half = rot / 2, hp = rp / 2;
+    auto turn = [&](Word w, int j) {                      // pair j of a head
+        alignas(8) T e[2];
+        *reinterpret_cast<Word*>(e) = w;
+        if (j < half) {
+            const float u = Cvt<T>::to_f(e[0]), v = Cvt<T>::to_f(e[1]), co = cs[j], si = cs[half + j];
+            e[0] = Cvt<T>::from_f(u * co - v * si);
+            e[1] = Cvt<T>::from_f(v * co + u * si);
+        }
+        return *reinterpret_cast<Word*>(e);
+    };
     float ss = 0.f;
-    for (int i = tid; i < rank_pad; i += 128) {
-        const float x = Cvt<T>::to_f(c[i]);
-        ss += x * x;
+    for (int i = tid; i < rank_pad / 2; i += kLatWriteThreads) {
+        alignas(8) T e[2];
+        *reinterpret_cast<Word*>(e) = reinterpret_cast<const Word*>(c)[i];
+        const float a = Cvt<T>::to_f(e[0]), b = Cvt<T>::to_f(e[1]);
+        ss += a * a + b * b;
+    }
+    for (int i = tid; i < heads * hp; i += kLatWriteThreads) {
+        Word* w = reinterpret_cast<Word*>(qr) + i;
+        *w = turn(*w, i % hp);
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     if ((tid & 31) == 0) red[tid >> 5] = ss;
     __syncthreads();
-    const float inv = 1.f / sqrtf((red[0] + red[1] + red[2] + red[3]) / rank + eps);
-    const int s = seq_ids[t];
-    T* dst = cache_row(kv, page_table, max_pages, page_size, s, past_len[s] + t - q_start[s], page_size, rank_pad + rp);
+    float tot = 0.f;
+#pragma unroll
+    for (int w = 0; w < kLatWriteThreads / 32; ++w) tot += red[w];
+    const float inv = 1.f / sqrtf(tot / rank + eps);
     if (!dst) return;
-    for (int i = tid; i < rank_pad; i += 128) dst[i] = Cvt<T>::from_f(Cvt<T>::to_f(c[i]) * inv * norm_w[i]);
-    dst += rank_pad;
-    for (int j = tid; j < rp / 2; j += 128) {
-        float u = Cvt<T>::to_f(kr[2 * j]), v = Cvt<T>::to_f(kr[2 * j + 1]);
-        if (j < half) {
-            const float co = cs[j], si = cs[half + j], a = u * co - v * si;
-            v = v * co + u * si;
-            u = a;
-        }
-        dst[2 * j] = Cvt<T>::from_f(u);
-        dst[2 * j + 1] = Cvt<T>::from_f(v);
+    for (int i = tid; i < rank_pad / 2; i += kLatWriteThreads) {
+        alignas(8) T e[2];
+        *reinterpret_cast<Word*>(e) = reinterpret_cast<const Word*>(c)[i];
+        e[0] = Cvt<T>::from_f(Cvt<T>::to_f(e[0]) * inv * norm_w[2 * i]);
+        e[1] = Cvt<T>::from_f(Cvt<T>::to_f(e[1]) * inv * norm_w[2 * i + 1]);
+        reinterpret_cast<Word*>(dst)[i] = *reinterpret_cast<Word*>(e);
     }
+    for (int j = tid; j < hp; j += kLatWriteThreads) reinterpret_cast<Word*>(dst + rank_pad)[j] = turn(reinterpret_cast<const Word*>(kr)[j], j);
 }
 
-// One warp per (row, head) of packed q | k | v; d: padded head, real: features that count in the mean.
+// One warp per row and group of heads of packed q | k | v: a lane holds eight consecutive features, d / 8 lanes a head, so a warp takes
+// 256 / d heads at once (wider heads in turns of 256 features).  d: padded head, real: features that count in the mean.
 template <typename T>
 __global__ void __launch_bounds__(128)
 unit_kv_write_kernel(const T* qkv, T* q_out, T* kv, const float* temperature, const int* positions, const int* seq_ids, const int* q_start,
-                     const int* past_len, const int* page_table, int max_pages, int page_size, int tokens, int hq, int hkv, int d, int real, float eps) {
+                     const int* past_len, const int* page_table, int max_pages, int page_size, int tokens, int hq, int hkv, int d, int real, float eps,
+                     int lanes) {
     pdl_prologue();
-    const int heads = hq + 2 * hkv, lane = threadIdx.x & 31;
+    constexpr int kV = 8 * sizeof(T) / 16;
+    const int heads = hq + 2 * hkv, lane = threadIdx.x & 31, per = 32 / lanes, groups = (heads + per - 1) / per;
     const long long wid = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
-    if (wid >= (long long)tokens * heads) return;
-    const int t = (int)(wid / heads), h = (int)(wid - (long long)t * heads);
-    const T* src = qkv + ((size_t)t * heads + h) * d;
-    float f = 1.f;
-    if (h < hq + hkv) {
-        float ss = 0.f;
-        for (int i = lane * 2; i < d; i += 64) {
-            const float a = Cvt<T>::to_f(src[i]), b = Cvt<T>::to_f(src[i + 1]);
-            ss += a * a + b * b;
-        }
+    if (wid >= (long long)tokens * groups) return;
+    const int t = (int)(wid / groups), h = (int)(wid - (long long)t * groups) * per + lane / lanes, li = lane % lanes;
+    const bool live = h < heads;
+    const T* src = qkv + ((size_t)t * heads + (live ? h : 0)) * d;
+    float ss = 0.f;
+    alignas(16) T e[8];
+    for (int c = li * 8; c < d; c += lanes * 8) {
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        f = 1.f / sqrtf(ss / real + eps);
+        for (int v = 0; v < kV; ++v) reinterpret_cast<uint4*>(e)[v] = reinterpret_cast<const uint4*>(src + c)[v];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const float x = Cvt<T>::to_f(e[i]);
+            ss = fmaf(x, x, ss);
+        }
     }
+    for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!live) return;
+    float f = h < hq + hkv ? 1.f / sqrtf(ss / real + eps) : 1.f;
     T* dst;
     if (h < hq) {
         f *= temperature[positions[t]];
         dst = q_out + ((size_t)t * hq + h) * d;
     } else {
-        const int s = seq_ids[t], g = h - hq;             // planes keys | values: g counts through both
+        const int s = seq_ids[t];                         // planes keys | values: h - hq counts through both
         dst = cache_row(kv, page_table, max_pages, page_size, s, past_len[s] + t - q_start[s], 2 * hkv * page_size, d);
         if (!dst) return;
-        dst += (size_t)g * page_size * d;
+        dst += (size_t)(h - hq) * page_size * d;
     }
-    for (int i = lane * 2; i < d; i += 64) {
-        dst[i] = Cvt<T>::from_f(Cvt<T>::to_f(src[i]) * f);
-        dst[i + 1] = Cvt<T>::from_f(Cvt<T>::to_f(src[i + 1]) * f);
+    for (int c = li * 8; c < d; c += lanes * 8) {
+        if (d > lanes * 8) {                              // several turns: read again
+#pragma unroll
+            for (int v = 0; v < kV; ++v) reinterpret_cast<uint4*>(e)[v] = reinterpret_cast<const uint4*>(src + c)[v];
+        }
+        if (h < hq + hkv) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) e[i] = Cvt<T>::from_f(Cvt<T>::to_f(e[i]) * f);
+        }
+#pragma unroll
+        for (int v = 0; v < kV; ++v) reinterpret_cast<uint4*>(dst + c)[v] = reinterpret_cast<const uint4*>(e)[v];
     }
 }
 
@@ -158,6 +192,112 @@ head_linear_kernel(const T* x, const T* w, T* y, const T* x2, int tokens, int n,
     }
 }
 
+// The same product for 16-bit rows on tcgen05: Yᵀ[64 outputs, 64 rows] = W[h] (A, K-major) · X[:, h]ᵀ (B, K-major).  A CTA keeps its 64 rows
+// of one head's matrix in shared memory and walks the row tiles.  The upper half of the 128-row A tile is never loaded; what it holds only
+// reaches accumulator rows that nobody reads.  Warps 0-1: results; warp 2: copies and MMA; warp 3: TMEM, tail columns.
+template <typename T>
+__global__ void __launch_bounds__(128)
+head_linear_tc5_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_constant__ CUtensorMap tma_x, T* y, const T* x2, int tokens, int n, int kc, int tail,
+                       int ldx2, int ldy, int hy, int* status) {
+    constexpr bool kBf16 = std::is_same<T, __nv_bfloat16>::value;
+    constexpr int kWChunk = 128 * 128, kXChunk = 64 * 128;
+    extern __shared__ uint8_t hl_raw[];
+    __shared__ uint64_t bar_w, bar_x, bar_d, bar_free;
+    __shared__ uint32_t tmem_word, abort_word;
+    uint8_t* s_w = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(hl_raw) + 1023) & ~uintptr_t(1023));
+    uint8_t* s_x = s_w + kc * kWChunk;
+    volatile uint32_t* abort_flag = &abort_word;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y, n0 = blockIdx.x * 64;
+    const int tiles = (tokens + 63) / 64;
+    if (threadIdx.x == 0) {
+        mbar_init(&bar_w, 1);
+        mbar_init(&bar_x, 1);
+        mbar_init(&bar_d, 1);
+        mbar_init(&bar_free, 64);
+        abort_word = 0;
+        mbar_fence_init();
+    }
+    __syncthreads();
+    if (warp == 2 && lane == 0) {                         // the matrix does not depend on earlier kernels
+        mbar_expect_tx(&bar_w, kc * 64 * 128);
+        for (int c = 0; c < kc; ++c) tma_load_2d(s_w + c * kWChunk, &tma_w, &bar_w, c * 64, h * n + n0);
+    }
+    pdl_wait();                                           // before TMEM: a kernel that is still running may be about to allocate its own
+    if (warp == 3) {
+        tmem_alloc(&tmem_word, 64);
+        tmem_relinquish();
+    }
+    tc_fence_before_sync();
+    __syncthreads();
+    tc_fence_after_sync();
+    const uint32_t tmem = tmem_word;
+    pdl_launch_dependents();
+    if (warp == 2) {
+        if (lane == 0) {
+            const uint32_t idesc = idesc_f16(128, 64, kBf16);
+            bool ok = true;
+            int it = 0;
+            for (int t = blockIdx.z; t < tiles && ok; t += gridDim.z, ++it) {
+                // the tile before has been read out: its product is complete and its accumulator free
+                if (it > 0) ok = mbar_wait(&bar_free, (it - 1) & 1, abort_flag, status, kStatusProducerTimeout);
+                if (!ok) break;
+                tc_fence_after_sync();
+                mbar_expect_tx(&bar_x, kc * kXChunk);
+                for (int c = 0; c < kc; ++c) tma_load_3d(s_x + c * kXChunk, &tma_x, &bar_x, c * 64, h, t * 64);
+                if (it == 0) ok = mbar_wait(&bar_w, 0, abort_flag, status, kStatusMmaTimeout);
+                ok = ok && mbar_wait(&bar_x, it & 1, abort_flag, status, kStatusMmaTimeout);
+                if (!ok) break;
+                tc_fence_after_sync();
+                for (int c = 0; c < kc; ++c) {
+                    const uint64_t dw = smem_desc_sw128(s_w + c * kWChunk), dx = smem_desc_sw128(s_x + c * kXChunk);
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) umma_f16(tmem, dw + 2 * k, dx + 2 * k, idesc, (c | k) ? 1u : 0u);
+                }
+                umma_commit(&bar_d);
+            }
+        }
+    } else if (warp < 2) {
+        const int r = warp * 32 + lane;
+        int it = 0;
+        for (int t = blockIdx.z; t < tiles; t += gridDim.z, ++it) {
+            if (!mbar_wait(&bar_d, it & 1, abort_flag, status, kStatusEpilogueTimeout)) break;
+            tc_fence_after_sync();
+            uint32_t a[32], b[32];
+            tmem_ld_x32(tmem + (static_cast<uint32_t>(warp * 32) << 16), a);
+            tmem_ld_x32(tmem + (static_cast<uint32_t>(warp * 32) << 16) + 32, b);
+            tmem_ld_wait();
+            tc_fence_before_sync();
+            mbar_arrive(&bar_free);
+            T* dst = y + (size_t)t * 64 * ldy + (size_t)h * hy + n0 + r;
+            const int cnt = min(64, tokens - t * 64);
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+                if (i < cnt) dst[(size_t)i * ldy] = Cvt<T>::from_f(__uint_as_float(a[i]));
+                if (i + 32 < cnt) dst[(size_t)(i + 32) * ldy] = Cvt<T>::from_f(__uint_as_float(b[i]));
+            }
+        }
+    } else if (tail > 0 && n0 == 0) {
+        const int v = tail / 8;                           // 16-byte pieces
+        for (int t = blockIdx.z; t < tiles; t += gridDim.z)
+            for (int i = lane; i < 64 * v; i += 32) {
+                const int row = t * 64 + i / v, c = i % v * 8;
+                if (row < tokens)
+                    *reinterpret_cast<uint4*>(y + (size_t)row * ldy + (size_t)h * hy + n + c) =
+                        *reinterpret_cast<const uint4*>(x2 + (size_t)row * ldx2 + (size_t)h * tail + c);
+            }
+    }
+    if (*abort_flag) {
+        const uint64_t t0 = global_timer_ns();
+        while (global_timer_ns() - t0 < 200000ull) __nanosleep(1000);
+    }
+    tc_fence_before_sync();
+    __syncthreads();
+    if (warp == 3) {
+        tc_fence_after_sync();
+        tmem_dealloc(tmem, 64);
+    }
+}
+
 // Cached rows [0, past + q_len) of every sequence, sequence s from row out_start[s]; one warp per row, 16 bytes per lane and turn.
 // Sequences with at most min_q rows in the step are left out.
 __global__ void __launch_bounds__(128)
@@ -193,7 +333,7 @@ extern "C" int telb_latent_write(void* rows, void* kv_layer, const float* cos_si
                                  int rp, int rank_pad, int rank, int rot, int table_ld, float eps, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (rot % 2 || rot > rp || rank > rank_pad || rank <= 0) return fail("telb_latent_write: sizes");
-    TELB_BY_TYPE(dtype, TELB_LAUNCH("latent_write_kernel", (latent_write_kernel<T>), dim3(tokens), dim3(128), 0, stream, (T*)rows, (T*)kv_layer, cos_sin, norm_w,
+    TELB_BY_TYPE(dtype, TELB_LAUNCH("latent_write_kernel", (latent_write_kernel<T>), dim3(tokens), dim3(kLatWriteThreads), 0, stream, (T*)rows, (T*)kv_layer, cos_sin, norm_w,
                                     positions, seq_ids, q_start, past_len, page_table, max_pages, page_size, heads, kp, rp, rank_pad, rank, rot, table_ld, eps))
     TELB_CHECK_LAUNCH("latent_write_kernel");
     return 0;
@@ -204,18 +344,45 @@ extern "C" int telb_unit_kv_write(const void* qkv, void* q_out, void* kv_layer, 
                                   int d, int real, float eps, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (d % 64 || real <= 0 || real > d) return fail("telb_unit_kv_write: padded heads are multiples of 64");
-    const long long warps = (long long)tokens * (hq + 2 * hkv);
+    const int lanes = d <= 64 ? 8 : d <= 128 ? 16 : 32;
+    const long long warps = (long long)tokens * ((hq + 2 * hkv + 32 / lanes - 1) / (32 / lanes));
     TELB_BY_TYPE(dtype, TELB_LAUNCH("unit_kv_write_kernel", (unit_kv_write_kernel<T>), dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, stream, (const T*)qkv, (T*)q_out,
-                                    (T*)kv_layer, temperature, positions, seq_ids, q_start, past_len, page_table, max_pages, page_size, tokens, hq, hkv, d, real, eps))
+                                    (T*)kv_layer, temperature, positions, seq_ids, q_start, past_len, page_table, max_pages, page_size, tokens, hq, hkv, d, real, eps, lanes))
     TELB_CHECK_LAUNCH("unit_kv_write_kernel");
     return 0;
 }
 
+template <typename T>
+static int launch_head_linear_tc5(const void* x, const void* w, void* y, const void* x2, int tokens, int heads, int n, int k, int tail, int ldx, int ldx2, int ldy,
+                                  int hy, int* status, cudaStream_t stream) {
+    const int kc = k / 64, smem = kc * (128 + 64) * 128 + 1024;
+    static int configured = 0;
+    if (smem > configured) {
+        cudaError_t e = cudaFuncSetAttribute(head_linear_tc5_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        if (e != cudaSuccess) return fail("cudaFuncSetAttribute(head_linear_tc5)", e);
+        configured = smem;
+    }
+    const CUtensorMapDataType dt = std::is_same<T, __nv_bfloat16>::value ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
+    CUtensorMap mw, mx;
+    if (make_tmap_2d(&mw, dt, 2, w, (uint64_t)heads * n, k, (uint64_t)k * 2, 64, 64, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
+    const uint64_t dims[3] = {(uint64_t)k, (uint64_t)heads, (uint64_t)tokens}, strides[2] = {(uint64_t)k * 2, (uint64_t)ldx * 2};
+    const uint32_t box[3] = {64, 1, 64};
+    if (make_tmap_nd(&mx, dt, 3, x, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
+    const int tiles = (tokens + 63) / 64, want = (2 * sm_count() + heads * (n / 64) - 1) / (heads * (n / 64));
+    TELB_LAUNCH("head_linear_tc5_kernel", (head_linear_tc5_kernel<T>), dim3(n / 64, heads, tiles < want ? tiles : want), dim3(128), smem, stream, mw, mx, (T*)y,
+                (const T*)x2, tokens, n, kc, tail, ldx2, ldy, hy, status);
+    TELB_CHECK_LAUNCH("head_linear_tc5_kernel");
+    return 0;
+}
+
 extern "C" int telb_head_linear(const void* x, const void* w, void* y, const void* x2, int tokens, int heads, int n, int k, int tail, int ldx, int ldx2,
-                                int ldy, int hy, int dtype, cudaStream_t stream) {
+                                int ldy, int hy, int dtype, int* status, cudaStream_t stream) {
     if (tokens <= 0 || heads <= 0) return 0;
     if (n % 64 || k % 64 || ldx % 8) return fail("telb_head_linear: sizes must be multiples of 64 and the row pitch of 8");
     if (heads > 65535 || tokens > 65535 * 64) return fail("telb_head_linear: too many heads or rows");
+    if (dtype != 2 && k <= 576 && ldx2 % 8 == 0 && ldy % 8 == 0 && hy % 8 == 0 && tail % 8 == 0)
+        return dtype == 1 ? launch_head_linear_tc5<__nv_bfloat16>(x, w, y, x2, tokens, heads, n, k, tail, ldx, ldx2, ldy, hy, status, stream)
+                          : launch_head_linear_tc5<__half>(x, w, y, x2, tokens, heads, n, k, tail, ldx, ldx2, ldy, hy, status, stream);
     const dim3 grid(n / 64 + (tail > 0 ? 1 : 0), (tokens + 63) / 64, heads);
     TELB_BY_TYPE(dtype, TELB_LAUNCH("head_linear_kernel", (head_linear_kernel<T>), grid, dim3(256), 0, stream, (const T*)x, (const T*)w, (T*)y, (const T*)x2,
                                     tokens, n, k, tail, ldx, ldx2, ldy, hy))

@@ -1074,8 +1074,8 @@ def mlstm(qkvg, gates, norm_w, state, norm_state, meta: StepMeta, scale: float, 
 
 class ChannelDeltaParams(ctypes.Structure):
     """Host mirror of ``ChannelDeltaParams`` (``csrc/kernels/channel_delta.cu``)."""
-    _fields_ = [(n, c_vp) for n in ("qkv", "decay", "gate", "beta", "conv_w", "a_log", "decay_bias", "norm_w", "conv_state", "state", "mixed", "row_scale",
-                                    "g", "b", "o", "out", "q_start", "q_len", "past_len", "slot_ids", "seq_ids")] + \
+    _fields_ = [(n, c_vp) for n in ("qkv", "decay", "gate", "beta", "conv_w", "a_log", "decay_bias", "norm_w", "conv_state", "state", "blocks",
+                                    "v_blocks", "o", "out", "q_start", "q_len", "past_len", "slot_ids", "seq_ids", "status")] + \
                [(n, c_int) for n in ("tokens", "num_seqs", "heads", "kv_heads", "dk", "dv", "dk_real", "dv_real", "taps", "channels", "ld_decay", "ld_gate",
                                      "gate_f32")] + [("eps", c_float)]
 
@@ -1099,19 +1099,19 @@ def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, con
         kernel = "decode" if decode_ok else "walk"
     if kernel == "decode" and not decode_ok:
         raise ValueError("the decode kernel does not cover this step")
-    dev, one_launch = qkv.device, kernel == "decode" and n == nk
+    dev = qkv.device
     out = torch.empty(t, n * dv, dtype=qkv.dtype, device=dev)
-    mixed = scale = g = b = o = None
-    if not one_launch:
-        mixed, scale = torch.empty_like(qkv), torch.empty(t, 2, nk, dtype=f32, device=dev)
-        g, b = torch.empty(t, n * dk, dtype=f32, device=dev), torch.empty(t, n, dtype=f32, device=dev)
-        o = out if kernel == "decode" else torch.empty_like(out)
+    blocks = v_blocks = o = None
+    if kernel == "walk":                       # blocks of four tokens, counted from the start of every portion
+        nb = t // 4 + meta.num_seqs + 1
+        blocks, v_blocks = torch.empty(nb, n, 13 * dk + 32, dtype=f32, device=dev), torch.empty(nb, n, dv, 4, dtype=qkv.dtype, device=dev)
+        o = torch.empty_like(out)
     ptr = lambda x: None if x is None else _p(x).value
-    p = ChannelDeltaParams(*[ptr(x) for x in (qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, mixed, scale, g, b, o, out,
-                                              meta.q_start, meta.q_len, meta.past_len, meta.slot_ids, meta.seq_ids)],
+    p = ChannelDeltaParams(*[ptr(x) for x in (qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, blocks, v_blocks, o, out,
+                                              meta.q_start, meta.q_len, meta.past_len, meta.slot_ids, meta.seq_ids, Workspace.get(dev).status)],
                            t, meta.num_seqs, n, nk, dk, dv, spec.head_k_dim, spec.head_v_dim, spec.conv_kernel, ch, decay.stride(0), gate.stride(0),
                            int(gate.dtype == f32), eps)
-    launches = (1 if one_launch else 2) if kernel == "decode" else (4 if spec.conv_kernel > 1 else 3)
+    launches = (1 if kernel == "decode" else 4) + int(spec.conv_kernel > 1 and (kernel == "walk" or n != nk))
     _check(lib().telb_channel_delta(ctypes.byref(p), c_int(int(kernel == "decode")), c_int(_dtype_code(qkv)), _stream()), "channel_delta", launches)
     return out
 
@@ -1153,7 +1153,7 @@ def head_linear(x, weight, heads: int, x_col: int = 0, tail_col: int = -1, tail:
     _p(x)
     _check(lib().telb_head_linear(c_vp(base + x_col * es), _p(weight), _p(y), c_vp(base + max(tail_col, 0) * es), c_int(t), c_int(h), c_int(n), c_int(k),
                                   c_int(tail), c_int(x.shape[1]), c_int(x.shape[1]), c_int(h * (n + tail)), c_int(n + tail), c_int(_dtype_code(x)),
-                                  _stream()), "head_linear")
+                                  _p(Workspace.get(x.device).status), _stream()), "head_linear")
     return y
 
 
