@@ -2,15 +2,20 @@
 //
 //   latent_decode     few rows per sequence.  The key expansion has been folded into the query (one [rank + rot] row per token and head),
 //                     so every (token, head) pair is a column against the same cached rows:
-//                         Sᵀ[128 tok, NC] = rows[128 tok, rank + rot] · Qᵀ      Oᵀ[rank, NC] += latentᵀ[rank, 128 tok] · Pᵀ
+//                         Sᵀ[64 tok, NC] = rows[64 tok, rank + rot] · Qᵀ        Oᵀ[rank, NC] += latentᵀ[rank, 64 tok] · Pᵀ
 //                     A tile of rows is loaded once and serves both products (K-major for the scores, MN-major for the output).  It comes
 //                     in pairs of 64-feature chunks through a ring that holds at least one tile: scores start with the first pair, and a
 //                     pair's slot is refilled as soon as its 128 output features are done.  The products are narrow, so consecutive ones go
 //                     to different accumulators (four for the scores, two output blocks in turn) instead of waiting for one another.
+//                     A tile is one page, so that two CTAs fit on an SM and one computes while the other loads; the upper half of the
+//                     128-row score MMA reads whatever lies behind the chunk, and nobody reads its results.
 //   latent_prefill    prompt portions, over keys and values expanded from the latents ([rows, heads, k | v], one product per step).  The
 //                     rotated key part is not expanded: a K tile is made of chunks of the head's keys and chunks of the shared rows.
 //                     256 query rows per CTA in two tiles with a softmax warpgroup each; probabilities stay in TMEM (the A operand
 //                     of P·V), over the scores they were made from.
+//
+// The producer and the MMA warp walk their loops as whole warps and elect a lane only for the instructions themselves: descriptors then
+// live in uniform registers (under a divergent branch every issue costs about 100 cycles, more than these narrow products take).
 //
 // Probabilities enter P·V as a high and a low 16-bit half (2^-17).  Scores, maxima and sums are fp32.  All waits are bounded.
 #include <type_traits>
@@ -21,6 +26,7 @@
 namespace telb {
 
 constexpr int kLatMaxSlots = 16;
+constexpr int kLatMaxSplits = 64;
 
 struct LatentDecParams {
     void* out;                 // [rows, rank_pad] 16-bit, rows = T * heads
@@ -36,9 +42,8 @@ struct LatentDecParams {
 };
 
 constexpr int kLatThreads = 192;
-constexpr int kLatTile = 128;                // cached rows per tile = 2 pages
-constexpr int kLatPage = 64;
-constexpr int kLatChunk = kLatTile * 128;    // bytes of [128 rows x 64 features]
+constexpr int kLatTile = 64;                 // cached rows per tile = 1 page
+constexpr int kLatChunk = kLatTile * 128;    // bytes of [64 rows x 64 features]
 constexpr int kLatSlot = 2 * kLatChunk;
 
 __device__ __forceinline__ float lat_warp_max(float v) {
@@ -57,10 +62,10 @@ __device__ __forceinline__ bool lat_any(bool yes) {
 
 // grid (column blocks, splits, sequences).  NC: (token, head) columns of a block.
 template <typename T, int NC>
-__global__ void __launch_bounds__(kLatThreads, 1)
+__global__ void __launch_bounds__(kLatThreads, NC == 16 ? 2 : 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_kv, const __grid_constant__ LatentDecParams p) {
     constexpr bool kBf16 = std::is_same<T, __nv_bfloat16>::value;
-    constexpr int kQChunk = NC * 128, kPSpan = 2 * NC * 128;         // [high | low rows of the columns][64 tokens]
+    constexpr int kQChunk = NC * 128, kPBytes = 2 * NC * 128;        // [high | low rows of the columns][64 tokens]
     constexpr int kOCol = 4 * NC, kOBlock = 2 * NC;      // TMEM: four partial scores, then per 128 output features high | low columns
     constexpr int kTmemCols = NC == 16 ? 256 : 512;
     static_assert(kOCol + 4 * kOBlock <= kTmemCols, "scores and four output blocks");
@@ -69,8 +74,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     uint8_t* s_kv = smem;
     uint8_t* s_q = s_kv + p.slots * kLatSlot;
-    uint8_t* s_p = s_q + p.chunks * kQChunk;             // two spans of 64 tokens
-    uint64_t* bars = reinterpret_cast<uint64_t*>(s_p + 2 * kPSpan);
+    uint8_t* s_p = s_q + p.chunks * kQChunk;
+    uint64_t* bars = reinterpret_cast<uint64_t*>(s_p + kPBytes);
     uint64_t* q_full = bars;
     uint64_t* s_full = bars + 1;
     uint64_t* p_full = bars + 2;
@@ -112,7 +117,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
         tmem_alloc(tmem_slot, kTmemCols);
         tmem_relinquish();
     }
-    for (int i = threadIdx.x; i < 2 * kPSpan / 16; i += kLatThreads) reinterpret_cast<uint4*>(s_p)[i] = make_uint4(0, 0, 0, 0);
+    for (int i = threadIdx.x; i < kPBytes / 16; i += kLatThreads) reinterpret_cast<uint4*>(s_p)[i] = make_uint4(0, 0, 0, 0);
     fence_proxy_async_smem();
     tc_fence_before_sync();
     __syncthreads();
@@ -122,77 +127,100 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
 
     if (warp == 0) {
         // ---- producer ----
-        if (lane == 0 && ntiles > 0) {
-            mbar_expect_tx(q_full, p.chunks * kQChunk);
-            for (int c = 0; c < p.chunks; ++c) tma_load_2d(s_q + c * kQChunk, &tma_q, q_full, c * 64, row0);
+        if (ntiles > 0) {
+            const bool leader = elect_one();
+            if (leader) {
+                mbar_expect_tx(q_full, p.chunks * kQChunk);
+                for (int c = 0; c < p.chunks; ++c) tma_load_2d(s_q + c * kQChunk, &tma_q, q_full, c * 64, row0);
+            }
             const int* pages = p.page_table + (size_t)seq * p.max_pages;
             bool ok = true;
-            for (int j = 0, n = 0; j < ntiles && ok; ++j) {
-                int page[2];
-#pragma unroll
-                for (int h = 0; h < 2; ++h) {
-                    const int lp = (j0 + j) * 2 + h;
-                    const int pg = lp < p.max_pages ? pages[lp] : -1;
-                    page[h] = pg < 0 ? 0 : pg;           // rows past the end are masked
+            int slot = 0;
+            uint32_t ph = 1;
+            int next = 0;                                // pages are fetched 32 tiles at a time
+            for (int j = 0; j < ntiles && ok; ++j) {
+                if ((j & 31) == 0) {
+                    const int lp = j0 + j + lane;
+                    next = lp < p.max_pages ? pages[lp] : -1;
                 }
-                for (int pr = 0; pr < p.pairs; ++pr, ++n) {
-                    const int slot = n % p.slots;
-                    ok = mbar_wait(&kv_empty[slot], ((n / p.slots) & 1) ^ 1, abort_flag, p.status, kStatusProducerTimeout);
+                const int row = max(__shfl_sync(0xffffffffu, next, j & 31), 0) * kLatTile;      // rows past the end are masked
+                for (int pr = 0; pr < p.pairs; ++pr) {
+                    ok = mbar_wait(&kv_empty[slot], ph, abort_flag, p.status, kStatusProducerTimeout);
+                    ok = __all_sync(0xffffffffu, ok);
                     if (!ok) break;
-                    const int cnt = min(2, p.chunks - pr * 2);
-                    mbar_expect_tx(&kv_full[slot], cnt * kLatChunk);
-                    for (int c = 0; c < cnt; ++c)
-#pragma unroll
-                        for (int h = 0; h < 2; ++h)
-                            tma_load_2d(s_kv + slot * kLatSlot + c * kLatChunk + h * (kLatPage * 128), &tma_kv, &kv_full[slot], (pr * 2 + c) * 64,
-                                        page[h] * kLatPage);
+                    uint8_t* dst = s_kv + slot * kLatSlot;
+                    const bool two = pr * 2 + 1 < p.chunks;
+                    if (leader) {
+                        mbar_expect_tx(&kv_full[slot], two ? 2 * kLatChunk : kLatChunk);
+                        tma_load_2d(dst, &tma_kv, &kv_full[slot], pr * 128, row);
+                        if (two) tma_load_2d(dst + kLatChunk, &tma_kv, &kv_full[slot], pr * 128 + 64, row);
+                    }
+                    if (++slot == p.slots) {
+                        slot = 0;
+                        ph ^= 1;
+                    }
                 }
             }
         }
     } else if (warp == 1) {
         // ---- MMA issuer ----
-        if (lane == 0 && ntiles > 0) {
-            const uint32_t idesc_s = idesc_f16(128, NC, kBf16), idesc_o = idesc_f16(128, 2 * NC, kBf16, true);
-            bool ok = mbar_wait(q_full, 0, abort_flag, p.status, kStatusMmaTimeout);
-            for (int j = 0, n = 0; j < ntiles && ok; ++j) {
-                const int first = n;
-                for (int pr = 0; pr < p.pairs && ok; ++pr, ++n) {
-                    const int slot = n % p.slots;
-                    ok = mbar_wait(&kv_full[slot], (n / p.slots) & 1, abort_flag, p.status, kStatusMmaTimeout);
+        if (ntiles > 0) {
+            const bool leader = elect_one();
+            constexpr uint32_t idesc_s = idesc_f16(128, NC, kBf16), idesc_o = idesc_f16(128, 2 * NC, kBf16, true);
+            const uint64_t desc_kv = smem_desc_sw128(s_kv), desc_v = smem_desc_sw128_mn(s_kv, kLatChunk, 1024), desc_q = smem_desc_sw128(s_q),
+                           desc_p = smem_desc_sw128(s_p);
+            bool ok = __all_sync(0xffffffffu, mbar_wait(q_full, 0, abort_flag, p.status, kStatusMmaTimeout));
+            int slot = 0;
+            uint32_t ph = 0;
+            for (int j = 0; j < ntiles && ok; ++j) {
+                const int first = slot;
+                for (int pr = 0; pr < p.pairs; ++pr) {
+                    ok = __all_sync(0xffffffffu, mbar_wait(&kv_full[slot], ph, abort_flag, p.status, kStatusMmaTimeout));
                     if (!ok) break;
                     tc_fence_after_sync();
-                    const int cnt = min(2, p.chunks - pr * 2);
-                    for (int c = 0; c < cnt; ++c) {
-                        const uint64_t dk = smem_desc_sw128(s_kv + slot * kLatSlot + c * kLatChunk);
-                        const uint64_t dq = smem_desc_sw128(s_q + (pr * 2 + c) * kQChunk);
+                    const bool two = pr * 2 + 1 < p.chunks;
+                    const uint64_t dk = desc_kv + (uint64_t)((slot * kLatSlot) >> 4), dq = desc_q + (uint64_t)((pr * 2 * kQChunk) >> 4);
+                    if (leader) {
 #pragma unroll
-                        for (int k = 0; k < 4; ++k) umma_f16(tmem_base + k * NC, dk + 2 * k, dq + 2 * k, idesc_s, (pr | c) ? 1u : 0u);
+                        for (int k = 0; k < 4; ++k) umma_f16(tmem_base + k * NC, dk + 2 * k, dq + 2 * k, idesc_s, pr ? 1u : 0u);
+                        if (two) {
+#pragma unroll
+                            for (int k = 0; k < 4; ++k)
+                                umma_f16(tmem_base + k * NC, dk + (kLatChunk >> 4) + 2 * k, dq + (kQChunk >> 4) + 2 * k, idesc_s, 1u);
+                        }
+                        if (pr >= p.vblocks) umma_commit(&kv_empty[slot]);       // keys only
+                        if (pr == p.pairs - 1) umma_commit(s_full);
                     }
-                    if (pr >= p.vblocks) umma_commit(&kv_empty[slot]);   // keys only
+                    __syncwarp();
+                    if (++slot == p.slots) {
+                        slot = 0;
+                        ph ^= 1;
+                    }
                 }
                 if (!ok) break;
-                umma_commit(s_full);
-                ok = mbar_wait(p_full, j & 1, abort_flag, p.status, kStatusMmaTimeout);
+                ok = __all_sync(0xffffffffu, mbar_wait(p_full, j & 1, abort_flag, p.status, kStatusMmaTimeout));
                 if (!ok) break;
                 tc_fence_after_sync();
-                const uint64_t dp = smem_desc_sw128(s_p);
+                int s0 = first;
                 for (int b = 0; b < p.vblocks; b += 2) {
                     const bool two = b + 1 < p.vblocks;
-                    const int slot0 = (first + b) % p.slots, slot1 = (first + b + 1) % p.slots;
-                    const uint64_t dv0 = smem_desc_sw128_mn(s_kv + slot0 * kLatSlot, kLatChunk, 1024);
-                    const uint64_t dv1 = smem_desc_sw128_mn(s_kv + slot1 * kLatSlot, kLatChunk, 1024);
+                    const int s1 = s0 + 1 == p.slots ? 0 : s0 + 1;
+                    const uint64_t dv0 = desc_v + (uint64_t)((s0 * kLatSlot) >> 4), dv1 = desc_v + (uint64_t)((s1 * kLatSlot) >> 4);
                     const uint32_t d_o = tmem_base + kOCol + b * kOBlock;
+                    if (leader) {
 #pragma unroll
-                    for (int k = 0; k < kLatTile / 16; ++k) {
-                        const uint64_t db = dp + (uint64_t)(((k >> 2) * kPSpan) >> 4) + 2 * (k & 3);
-                        umma_f16(d_o, dv0 + (uint64_t)((k * 2048) >> 4), db, idesc_o, (j | k) ? 1u : 0u);
-                        if (two) umma_f16(d_o + kOBlock, dv1 + (uint64_t)((k * 2048) >> 4), db, idesc_o, (j | k) ? 1u : 0u);
+                        for (int k = 0; k < kLatTile / 16; ++k) {
+                            umma_f16(d_o, dv0 + (uint64_t)((k * 2048) >> 4), desc_p + 2 * k, idesc_o, (j | k) ? 1u : 0u);
+                            if (two) umma_f16(d_o + kOBlock, dv1 + (uint64_t)((k * 2048) >> 4), desc_p + 2 * k, idesc_o, (j | k) ? 1u : 0u);
+                        }
+                        umma_commit(&kv_empty[s0]);
+                        if (two) umma_commit(&kv_empty[s1]);
+                        if (j == ntiles - 1 && b + 2 >= p.vblocks) umma_commit(o_done);
                     }
-                    umma_commit(&kv_empty[slot0]);
-                    if (two) umma_commit(&kv_empty[slot1]);
+                    __syncwarp();
+                    s0 = s1 + 1 == p.slots ? 0 : s1 + 1;
                 }
             }
-            if (ok) umma_commit(o_done);
         }
     } else {
         // ---- softmax / epilogue ----
@@ -201,7 +229,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
         float m_used[NC], l_part[NC];
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
-            m_used[c] = -INFINITY;
+            m_used[c] = c < ncol ? -INFINITY : INFINITY;
             l_part[c] = 0.f;
         }
         bool ok = true;
@@ -223,7 +251,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                     s[c + i] = (__uint_as_float(r0[i]) + __uint_as_float(r1[i]) + (__uint_as_float(r2[i]) + __uint_as_float(r3[i]))) * p.scale_log2;
             }
             const int t0 = (j0 + j) * kLatTile, tk = t0 + r;
-            if (t0 + kLatTile - 1 > past) {              // the tile reaches the first row's own position: mask
+            if (r >= kLatTile) {                         // lanes behind the tile only help to rescale and to write the output
+#pragma unroll
+                for (int c = 0; c < NC; ++c) s[c] = -INFINITY;
+            } else if (t0 + kLatTile - 1 > past) {       // the tile reaches the first row's own position: mask
 #pragma unroll
                 for (int c = 0; c < NC; ++c) {
                     const int qi = qlen == 1 ? 0 : (cb * NC + c) / p.heads;
@@ -233,7 +264,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
             // the reference of a column moves only when a score exceeds it by 2^8: most tiles need no maximum
             bool over = false;
 #pragma unroll
-            for (int c = 0; c < NC; ++c) over = over || (c < ncol && s[c] > m_used[c] + 8.0f);
+            for (int c = 0; c < NC; ++c) over = over || s[c] > m_used[c] + 8.0f;
             if (lat_any(over)) {
                 float* red = s_red + (j & 1) * 4 * NC;
                 float f[NC];
@@ -271,14 +302,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                     tmem_st_wait();
                 }
             }
-            uint8_t* pbase = s_p + (r >> 6) * kPSpan;
-            const int tl = r & 63;
+            if (r < kLatTile) {
+                uint8_t* prow = s_p + (r & 7) * 2;
+                const int unit = r >> 3;
 #pragma unroll
-            for (int c = 0; c < NC; ++c) {
-                if (c < ncol) {
+                for (int c = 0; c < NC; ++c) {           // columns beyond ncol: reference +inf, probability zero
                     const float e = exp2f(s[c] - (m_used[c] == -INFINITY ? 0.f : m_used[c]));
                     l_part[c] += e;
-                    uint8_t* dst = pbase + (c >> 3) * 1024 + (c & 7) * 128 + ((((tl >> 3) ^ (c & 7)) & 7) << 4) + (tl & 7) * 2;
+                    uint8_t* dst = prow + (c >> 3) * 1024 + (c & 7) * 128 + ((unit ^ (c & 7)) << 4);
                     const T hi = Cvt<T>::from_f(e);
                     *reinterpret_cast<T*>(dst) = hi;
                     *reinterpret_cast<T*>(dst + NC * 128) = Cvt<T>::from_f(e - Cvt<T>::to_f(hi));
@@ -346,22 +377,32 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
 template <typename T>
 __global__ void __launch_bounds__(128) latent_combine_kernel(const float* ws_o, const float* ws_lse, T* out, int rows, int splits, int d) {
     pdl_prologue();
-    __shared__ float w[32];
+    __shared__ float w[kLatMaxSplits];
     const int row = blockIdx.x;
     if (threadIdx.x < 32) {
-        const float l = threadIdx.x < splits ? ws_lse[(size_t)threadIdx.x * rows + row] : -INFINITY;
-        float mx = l;
+        float l[kLatMaxSplits / 32], mx = -INFINITY, den = 0.f;
+#pragma unroll
+        for (int i = 0; i < kLatMaxSplits / 32; ++i) {
+            const int sp = i * 32 + threadIdx.x;
+            l[i] = sp < splits ? ws_lse[(size_t)sp * rows + row] : -INFINITY;
+            mx = fmaxf(mx, l[i]);
+        }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-        const float e = l == -INFINITY ? 0.f : exp2f(l - mx);
-        float den = e;
+#pragma unroll
+        for (int i = 0; i < kLatMaxSplits / 32; ++i) {
+            l[i] = l[i] == -INFINITY ? 0.f : exp2f(l[i] - mx);
+            den += l[i];
+        }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
-        w[threadIdx.x] = den > 0.f ? e / den : 0.f;
+#pragma unroll
+        for (int i = 0; i < kLatMaxSplits / 32; ++i) w[i * 32 + threadIdx.x] = den > 0.f ? l[i] / den : 0.f;
     }
     __syncthreads();
     for (int i = threadIdx.x * 4; i < d; i += 512) {
         float a[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
         for (int s = 0; s < splits; ++s) {
             const float4 v = __ldcg(reinterpret_cast<const float4*>(ws_o + ((size_t)s * rows + row) * d + i));
             a[0] = fmaf(w[s], v.x, a[0]);
@@ -461,7 +502,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
 
     if (warp == 0) {
         // ---- producer ----
-        if (lane == 0) {
+        const bool leader = elect_one();
+        if (leader) {
             mbar_expect_tx(q_full, qtiles * kc * kPreQChunk);
             for (int t = 0; t < qtiles; ++t)
                 for (int c = 0; c < kc; ++c) {
@@ -469,58 +511,77 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
                     if (c < p.kn) tma_load_3d(dst, &tma_q, q_full, c * 64, head, qrow0 + t * 128);
                     else tma_load_3d(dst, &tma_qr, q_full, (c - p.kn) * 64, head, qrow0 + t * 128);
                 }
-            for (int j = 0; j < nt; ++j) {
-                const int st = j % p.stages;
-                const uint32_t ph = ((j / p.stages) & 1) ^ 1;
-                uint8_t* sk = s_kv + st * stage_bytes;
-                const int row = kvrow0 + j * kPreTile;
-                if (!mbar_wait(&k_empty[st], ph, abort_flag, p.status, kStatusProducerTimeout)) break;
+        }
+        int st = 0;
+        uint32_t ph = 1;
+        for (int j = 0; j < nt; ++j) {
+            uint8_t* sk = s_kv + st * stage_bytes;
+            const int row = kvrow0 + j * kPreTile;
+            if (!__all_sync(0xffffffffu, mbar_wait(&k_empty[st], ph, abort_flag, p.status, kStatusProducerTimeout))) break;
+            if (leader) {
                 mbar_expect_tx(&k_full[st], k_bytes);
-                for (int c = 0; c < kc; ++c) {
-                    if (c < p.kn) tma_load_3d(sk + c * kPreChunk, &tma_k, &k_full[st], c * 64, head, row);
-                    else tma_load_2d(sk + c * kPreChunk, &tma_kr, &k_full[st], (c - p.kn) * 64, row);
-                }
-                if (!mbar_wait(&v_empty[st], ph, abort_flag, p.status, kStatusProducerTimeout)) break;
+                for (int c = 0; c < p.kn; ++c) tma_load_3d(sk + c * kPreChunk, &tma_k, &k_full[st], c * 64, head, row);
+                for (int c = 0; c < p.rc; ++c) tma_load_2d(sk + (p.kn + c) * kPreChunk, &tma_kr, &k_full[st], c * 64, row);
+            }
+            if (!__all_sync(0xffffffffu, mbar_wait(&v_empty[st], ph, abort_flag, p.status, kStatusProducerTimeout))) break;
+            if (leader) {
                 mbar_expect_tx(&v_full[st], VC * kPreChunk);
 #pragma unroll
                 for (int c = 0; c < VC; ++c) tma_load_3d(sk + k_bytes + c * kPreChunk, &tma_v, &v_full[st], c * 64, head, row);
             }
+            if (++st == p.stages) {
+                st = 0;
+                ph ^= 1;
+            }
         }
     } else if (warp == 1) {
         // ---- MMA issuer: S(0); then S(j + 1), P·V(j) ----
-        if (lane == 0) {
-            const uint32_t idesc_s = idesc_f16(128, kPreTile, kBf16), idesc_o = idesc_f16(128, VP, kBf16, false, true);
-            auto tiles_of = [&](int t) { return t == 0 ? nt0 : nt1; };
-            auto issue_s = [&](int j) {
-                const int st = j % p.stages;
-                if (!mbar_wait(&k_full[st], (j / p.stages) & 1, abort_flag, p.status, kStatusMmaTimeout)) return false;
-                tc_fence_after_sync();
-                for (int t = 0; t < 2; ++t) {
-                    if (j >= tiles_of(t)) continue;
-                    const uint32_t d = tmem_base + t * kTileCols + (j & 1) * 64;
-                    for (int c = 0; c < kc; ++c) {
-                        const uint64_t dq = smem_desc_sw128(s_q + (t * kc + c) * kPreQChunk);
-                        const uint64_t dk = smem_desc_sw128(s_kv + st * stage_bytes + c * kPreChunk);
+        const bool leader = elect_one();
+        constexpr uint32_t idesc_s = idesc_f16(128, kPreTile, kBf16), idesc_o = idesc_f16(128, VP, kBf16, false, true);
+        const uint64_t desc_q = smem_desc_sw128(s_q), desc_k = smem_desc_sw128(s_kv), desc_v = smem_desc_sw128_mn(s_kv + k_bytes, kPreChunk, 1024);
+        auto wait = [&](uint64_t* bar, uint32_t parity) {
+            const bool got = __all_sync(0xffffffffu, mbar_wait(bar, parity, abort_flag, p.status, kStatusMmaTimeout));
+            tc_fence_after_sync();
+            return got;
+        };
+        int ks = 0, vs = 0;                               // ring positions of the next key and value tile
+        uint32_t kph = 0, vph = 0;
+        auto issue_s = [&](int j) {
+            if (!wait(&k_full[ks], kph)) return false;
+            const uint64_t dk = desc_k + (uint64_t)((ks * stage_bytes) >> 4);
+            const uint32_t d = tmem_base + (j & 1) * 64;
 #pragma unroll
-                        for (int k = 0; k < 4; ++k) umma_f16(d, dq + 2 * k, dk + 2 * k, idesc_s, (c | k) ? 1u : 0u);
-                    }
+            for (int t = 0; t < 2; ++t) {
+                if (j >= (t == 0 ? nt0 : nt1)) continue;
+                const uint64_t dq = desc_q + (uint64_t)((t * kc * kPreQChunk) >> 4);
+                if (leader) {
+                    for (int c = 0; c < kc; ++c)
+#pragma unroll
+                        for (int k = 0; k < 4; ++k)
+                            umma_f16(d + t * kTileCols, dq + (uint64_t)((c * kPreQChunk) >> 4) + 2 * k, dk + (uint64_t)((c * kPreChunk) >> 4) + 2 * k, idesc_s,
+                                     (c | k) ? 1u : 0u);
                     umma_commit(&s_full[t * 2 + (j & 1)]);
                 }
-                umma_commit(&k_empty[st]);
-                return true;
-            };
-            bool ok = mbar_wait(q_full, 0, abort_flag, p.status, kStatusMmaTimeout) && issue_s(0);
-            for (int j = 0; j < nt && ok; ++j) {
-                if (j + 1 < nt) ok = issue_s(j + 1);
-                const int st = j % p.stages;
-                ok = ok && mbar_wait(&v_full[st], (j / p.stages) & 1, abort_flag, p.status, kStatusMmaTimeout);
-                const uint64_t dv = smem_desc_sw128_mn(s_kv + st * stage_bytes + k_bytes, kPreChunk, 1024);
-                for (int t = 0; t < 2 && ok; ++t) {
-                    if (j >= tiles_of(t)) continue;
-                    ok = mbar_wait(&p_full[t * 2 + (j & 1)], (j >> 1) & 1, abort_flag, p.status, kStatusMmaTimeout);
-                    if (!ok) break;
-                    tc_fence_after_sync();
-                    const uint32_t a = tmem_base + t * kTileCols + (j & 1) * 64, d = tmem_base + t * kTileCols + kOCol;
+            }
+            if (leader) umma_commit(&k_empty[ks]);
+            if (++ks == p.stages) {
+                ks = 0;
+                kph ^= 1;
+            }
+            return true;
+        };
+        bool ok = wait(q_full, 0) && issue_s(0);
+        for (int j = 0; j < nt && ok; ++j) {
+            if (j + 1 < nt) ok = issue_s(j + 1);
+            ok = ok && wait(&v_full[vs], vph);
+            const uint64_t dv = desc_v + (uint64_t)((vs * stage_bytes) >> 4);
+#pragma unroll
+            for (int t = 0; t < 2; ++t) {
+                if (!ok || j >= (t == 0 ? nt0 : nt1)) continue;
+                ok = wait(&p_full[t * 2 + (j & 1)], (j >> 1) & 1);
+                if (!ok) continue;
+                const uint32_t a = tmem_base + t * kTileCols + (j & 1) * 64, d = tmem_base + t * kTileCols + kOCol;
+                if (leader) {
 #pragma unroll
                     for (int half = 0; half < 2; ++half)
 #pragma unroll
@@ -528,7 +589,11 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
                             umma_f16_ts(d, a + half * 32 + k * 8, dv + (uint64_t)((k * 2048) >> 4), idesc_o, (j | half | k) ? 1u : 0u);
                     umma_commit(&o_done[t * 2 + (j & 1)]);
                 }
-                if (ok) umma_commit(&v_empty[st]);
+            }
+            if (ok && leader) umma_commit(&v_empty[vs]);
+            if (++vs == p.stages) {
+                vs = 0;
+                vph ^= 1;
             }
         }
     } else {
@@ -649,8 +714,10 @@ constexpr int kSmemLimit = 227 * 1024;
 
 template <typename T, int NC>
 static int launch_latent_decode(const CUtensorMap& tq, const CUtensorMap& tkv, LatentDecParams p, int nseq, int max_cols, cudaStream_t stream) {
-    const int fixed = p.chunks * NC * 128 + 4 * NC * 128 + (4 + 2 * kLatMaxSlots) * 8 + 16 + 8 * NC * 4 + 1024;
-    p.slots = (kSmemLimit - fixed) / kLatSlot;
+    // two CTAs per SM where a tile leaves room for that.  The score MMA reads one chunk beyond the last slot: Q and P, and a spare
+    const int fixed = p.chunks * NC * 128 + 2 * NC * 128 + (4 + 2 * kLatMaxSlots) * 8 + 16 + 8 * NC * 4 + 1024 + kLatChunk;
+    p.slots = (kSmemLimit / (NC == 16 ? 2 : 1) - 1024 - fixed) / kLatSlot;
+    if (p.slots < p.pairs) p.slots = (kSmemLimit - fixed) / kLatSlot;
     if (p.slots > kLatMaxSlots) p.slots = kLatMaxSlots;
     if (p.slots > 3 * p.pairs) p.slots = 3 * p.pairs;
     if (p.slots < p.pairs) return fail("telb_latent_attention_decode: rows too wide for shared memory");
@@ -718,7 +785,7 @@ extern "C" int telb_latent_attention_decode(const void* q, const void* kv_layer,
     p.scale_log2 = scale * 1.4426950408889634f;
     p.status = status;
     if (splits < 1) splits = 1;
-    if (splits > 32) splits = 32;
+    if (splits > kLatMaxSplits) splits = kLatMaxSplits;
     while (splits > 1 && (long long)splits * p.rows * (rank_pad + 1) > ws_floats) --splits;
     p.splits = splits;
     p.ws_o = ws;
@@ -728,7 +795,7 @@ extern "C" int telb_latent_attention_decode(const void* q, const void* kv_layer,
     const int nc = max_cols <= 16 ? 16 : 32;
     CUtensorMap tq, tkv;
     if (make_tmap_2d(&tq, dt, 2, q, p.rows, row, (uint64_t)row * 2, nc, 64, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
-    if (make_tmap_2d(&tkv, dt, 2, kv_layer, (uint64_t)num_pages * kLatPage, row, (uint64_t)row * 2, kLatPage, 64, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
+    if (make_tmap_2d(&tkv, dt, 2, kv_layer, (uint64_t)num_pages * kLatTile, row, (uint64_t)row * 2, kLatTile, 64, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
     if (nc == 16)
         return is_bf16 ? launch_latent_decode<__nv_bfloat16, 16>(tq, tkv, p, num_seqs, max_cols, stream) : launch_latent_decode<__half, 16>(tq, tkv, p, num_seqs, max_cols, stream);
     return is_bf16 ? launch_latent_decode<__nv_bfloat16, 32>(tq, tkv, p, num_seqs, max_cols, stream) : launch_latent_decode<__half, 32>(tq, tkv, p, num_seqs, max_cols, stream);

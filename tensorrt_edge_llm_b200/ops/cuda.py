@@ -1211,15 +1211,13 @@ def _latent_plan(meta: StepMeta, heads: int, device, force: Optional[str]) -> La
     return p
 
 
-def _latent_splits(blocks: int, max_seq_len: int) -> int:
-    """Splits of the cached rows so that the (column block, split, sequence) CTAs, one per SM, come out near whole waves."""
-    tiles = max(1, (max_seq_len + 127) // 128)
-    if blocks >= 2 * 148 or tiles == 1:
-        return 1
+def _latent_splits(blocks: int, max_seq_len: int, slots: int) -> int:
+    """Splits of the cached rows so that the (column block, split, sequence) CTAs come out near whole waves of ``slots`` CTAs."""
+    tiles = max(1, (max_seq_len + 63) // 64)
     best, cost = 1, None
-    for s in range(1, min(tiles, 32) + 1):
-        waves = (blocks * s + 147) // 148
-        c = waves * ((tiles + s - 1) // s + 0.7) + (0.4 if s > 1 else 0.0)      # in tiles; start-up and merge in the same unit
+    for s in range(1, min(tiles, 64) + 1):
+        waves = (blocks * s + slots - 1) // slots
+        c = waves * ((tiles + s - 1) // s + 1.0) + (1.0 + s / 32 if s > 1 else 0.0)      # in tiles; start-up and merge in the same unit
         if cost is None or c < cost - 1e-9:
             best, cost = s, c
     return best
@@ -1249,7 +1247,7 @@ def latent_attention(rows, kv_layer, meta: StepMeta, kv_up, key_up_t, spec, kern
         o = torch.empty(tf, n, spec.rank_pad, dtype=rows.dtype, device=dev)
         if tc:
             nc = 16 if max_q * n <= 16 else 32
-            splits = _latent_splits(seqs * ((max_q * n + nc - 1) // nc), plan.max_seq_len)
+            splits = _latent_splits(seqs * ((max_q * n + nc - 1) // nc), plan.max_seq_len, 296 if nc == 16 else 148)
             _check(lib().telb_latent_attention_decode(
                 _p(q), _p(kv_layer), _p(o), _p(q_start), _p(q_len), _p(past_len), _p(table), c_int(seqs), c_int(tf), c_int(max_q),
                 c_int(kv_layer.shape[0]), c_int(table.shape[1]), c_int(n), c_int(spec.rank_pad), c_int(spec.rot_pad), c_float(spec.scale), c_int(splits),
