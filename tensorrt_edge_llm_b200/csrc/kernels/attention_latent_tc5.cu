@@ -46,10 +46,20 @@ constexpr int kLatTile = 64;                 // cached rows per tile = 1 page
 constexpr int kLatChunk = kLatTile * 128;    // bytes of [64 rows x 64 features]
 constexpr int kLatSlot = 2 * kLatChunk;
 
-__device__ __forceinline__ float lat_warp_max(float v) {
-    float r;
-    asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(r) : "f"(v));
-    return r;
+// Maxima of N column values over the warp; lane l receives that of column l % N.
+template <int N>
+__device__ __forceinline__ float lat_column_max(const float (&s)[N], int lane) {
+    float v[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = s[i];
+#pragma unroll
+    for (int o = N / 2; o > 0; o >>= 1) {
+        const bool hi = lane & o;
+#pragma unroll
+        for (int i = 0; i < o; ++i) v[i] = fmaxf(hi ? v[i + o] : v[i], __shfl_xor_sync(0xffffffffu, hi ? v[i] : v[i + o], o));
+    }
+    if constexpr (N == 16) v[0] = fmaxf(v[0], __shfl_xor_sync(0xffffffffu, v[0], 16));
+    return v[0];
 }
 
 // Whether any of the 128 softmax threads says yes.
@@ -149,11 +159,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                     ok = __all_sync(0xffffffffu, ok);
                     if (!ok) break;
                     uint8_t* dst = s_kv + slot * kLatSlot;
-                    const bool two = pr * 2 + 1 < p.chunks;
                     if (leader) {
-                        mbar_expect_tx(&kv_full[slot], two ? 2 * kLatChunk : kLatChunk);
-                        tma_load_2d(dst, &tma_kv, &kv_full[slot], pr * 128, row);
-                        if (two) tma_load_2d(dst + kLatChunk, &tma_kv, &kv_full[slot], pr * 128 + 64, row);
+                        mbar_expect_tx(&kv_full[slot], kLatSlot);                 // a missing second chunk arrives as zeros
+                        tma_load_3d(dst, &tma_kv, &kv_full[slot], 0, row, pr * 2);
                     }
                     if (++slot == p.slots) {
                         slot = 0;
@@ -268,25 +276,16 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
             if (lat_any(over)) {
                 float* red = s_red + (j & 1) * 4 * NC;
                 float f[NC];
-#pragma unroll
-                for (int c = 0; c < NC; ++c) {
-                    if (c < ncol) {
-                        const float wm = lat_warp_max(s[c]);
-                        if (lane == (c & 31)) red[(warp - 2) * NC + c] = wm;
-                    }
-                }
+                const float wm = lat_column_max<NC>(s, lane);
+                if (lane < NC) red[(warp - 2) * NC + lane] = wm;
                 named_barrier_sync(1, 128);
 #pragma unroll
                 for (int c = 0; c < NC; ++c) {
-                    f[c] = 1.f;
-                    if (c < ncol) {
-                        const float mt = fmaxf(fmaxf(red[c], red[NC + c]), fmaxf(red[2 * NC + c], red[3 * NC + c]));
-                        if (mt > m_used[c] + 8.0f) {     // uniform across the four warps
-                            f[c] = m_used[c] == -INFINITY ? 0.f : exp2f(m_used[c] - mt);
-                            l_part[c] *= f[c];
-                            m_used[c] = mt;
-                        }
-                    }
+                    const float mt = fmaxf(fmaxf(red[c], red[NC + c]), fmaxf(red[2 * NC + c], red[3 * NC + c]));
+                    const bool move = mt > m_used[c] + 8.0f;                      // uniform across the four warps
+                    f[c] = !move ? 1.f : m_used[c] == -INFINITY ? 0.f : exp2f(m_used[c] - mt);
+                    l_part[c] *= f[c];
+                    if (move) m_used[c] = mt;
                 }
                 if (j > 0) {
                     for (int b = 0; b < p.vblocks; ++b)
@@ -795,7 +794,11 @@ extern "C" int telb_latent_attention_decode(const void* q, const void* kv_layer,
     const int nc = max_cols <= 16 ? 16 : 32;
     CUtensorMap tq, tkv;
     if (make_tmap_2d(&tq, dt, 2, q, p.rows, row, (uint64_t)row * 2, nc, 64, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
-    if (make_tmap_2d(&tkv, dt, 2, kv_layer, (uint64_t)num_pages * kLatTile, row, (uint64_t)row * 2, kLatTile, 64, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
+    {   // cached rows as [chunk][row][64 features]: one copy brings a page's rows for a pair of chunks
+        const uint64_t dims[3] = {64, (uint64_t)num_pages * kLatTile, (uint64_t)row / 64}, strides[2] = {(uint64_t)row * 2, 128};
+        const uint32_t box[3] = {64, kLatTile, 2};
+        if (make_tmap_nd(&tkv, dt, 3, kv_layer, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
+    }
     if (nc == 16)
         return is_bf16 ? launch_latent_decode<__nv_bfloat16, 16>(tq, tkv, p, num_seqs, max_cols, stream) : launch_latent_decode<__half, 16>(tq, tkv, p, num_seqs, max_cols, stream);
     return is_bf16 ? launch_latent_decode<__nv_bfloat16, 32>(tq, tkv, p, num_seqs, max_cols, stream) : launch_latent_decode<__half, 32>(tq, tkv, p, num_seqs, max_cols, stream);

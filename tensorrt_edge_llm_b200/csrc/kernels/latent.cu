@@ -19,70 +19,85 @@ __device__ __forceinline__ T* cache_row(T* kv, const int* page_table, int max_pa
     return page < 0 ? nullptr : kv + ((size_t)page * page_rows + slot % page_size) * width;
 }
 
-// One CTA per row.  Columns: q [heads * kp] | q rotated [heads * rp] | latent [rank_pad] | key rotated [rp].  A thread takes one pair of
-// neighbours (one rotation) at a time.
-constexpr int kLatWriteThreads = 256;
-
-template <typename T> struct Pair;
-template <> struct Pair<float> { typedef float2 word; };
-template <> struct Pair<__nv_bfloat16> { typedef uint32_t word; };
-template <> struct Pair<__half> { typedef uint32_t word; };
-
+// Eight consecutive values, moved as 16-byte words.
 template <typename T>
-__global__ void __launch_bounds__(kLatWriteThreads)
+struct Eight {
+    alignas(16) T e[8];
+    __device__ __forceinline__ void load(const T* p) {
+#pragma unroll
+        for (int v = 0; v < (int)(8 * sizeof(T) / 16); ++v) reinterpret_cast<uint4*>(e)[v] = reinterpret_cast<const uint4*>(p)[v];
+    }
+    __device__ __forceinline__ void store(T* p) const {
+#pragma unroll
+        for (int v = 0; v < (int)(8 * sizeof(T) / 16); ++v) reinterpret_cast<uint4*>(p)[v] = reinterpret_cast<const uint4*>(e)[v];
+    }
+    // pairs j .. j + 3 of a head; those from `half` on pass
+    __device__ __forceinline__ void turn(const float* cs, int j, int half) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            if (j + i >= half) break;
+            const float u = Cvt<T>::to_f(e[2 * i]), v = Cvt<T>::to_f(e[2 * i + 1]), co = cs[j + i], si = cs[half + j + i];
+            e[2 * i] = Cvt<T>::from_f(u * co - v * si);
+            e[2 * i + 1] = Cvt<T>::from_f(v * co + u * si);
+        }
+    }
+};
+
+// Columns of a row: q [heads * kp] | q rotated [heads * rp] | latent [rank_pad] | key rotated [rp].  Two kinds of warps: one per row for
+// the latent and the key part, and one per row and 1024 rotated query features.
+template <typename T>
+__global__ void __launch_bounds__(128)
 latent_write_kernel(T* rows, T* kv, const float* cos_sin, const float* norm_w, const int* positions, const int* seq_ids, const int* q_start,
-                    const int* past_len, const int* page_table, int max_pages, int page_size, int heads, int kp, int rp, int rank_pad, int rank, int rot,
-                    int table_ld, float eps) {
+                    const int* past_len, const int* page_table, int max_pages, int page_size, int tokens, int heads, int kp, int rp, int rank_pad, int rank,
+                    int rot, int table_ld, float eps, int parts) {
     pdl_prologue();
-    typedef typename Pair<T>::word Word;
-    __shared__ float red[kLatWriteThreads / 32];
-    const int t = blockIdx.x, tid = threadIdx.x;
+    const int lane = threadIdx.x & 31;
+    const long long wid = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (wid >= (long long)tokens * parts) return;
+    const int t = (int)(wid / parts), part = (int)(wid - (long long)t * parts);
     const size_t ld = (size_t)heads * (kp + rp) + rank_pad + rp;
     T* qr = rows + t * ld + (size_t)heads * kp;
-    const T* c = qr + (size_t)heads * rp;
-    const T* kr = c + rank_pad;
-    const int s = seq_ids[t];
-    T* dst = cache_row(kv, page_table, max_pages, page_size, s, past_len[s] + t - q_start[s], page_size, rank_pad + rp);
     const float* cs = cos_sin + (size_t)positions[t] * table_ld;
-    const int half = rot / 2, hp = rp / 2;
-    auto turn = [&](Word w, int j) {                      // pair j of a head
-        alignas(8) T e[2];
-        *reinterpret_cast<Word*>(e) = w;
-        if (j < half) {
-            const float u = Cvt<T>::to_f(e[0]), v = Cvt<T>::to_f(e[1]), co = cs[j], si = cs[half + j];
-            e[0] = Cvt<T>::from_f(u * co - v * si);
-            e[1] = Cvt<T>::from_f(v * co + u * si);
+    const int half = rot / 2;
+    Eight<T> x;
+    if (part > 0) {
+        const int end = min(heads * rp, part * 1024);
+        for (int i = (part - 1) * 1024 + lane * 8; i < end; i += 256) {
+            const int j = i % rp / 2;
+            if (j >= half) continue;                      // padding
+            x.load(qr + i);
+            x.turn(cs, j, half);
+            x.store(qr + i);
         }
-        return *reinterpret_cast<Word*>(e);
-    };
-    float ss = 0.f;
-    for (int i = tid; i < rank_pad / 2; i += kLatWriteThreads) {
-        alignas(8) T e[2];
-        *reinterpret_cast<Word*>(e) = reinterpret_cast<const Word*>(c)[i];
-        const float a = Cvt<T>::to_f(e[0]), b = Cvt<T>::to_f(e[1]);
-        ss += a * a + b * b;
+        return;
     }
-    for (int i = tid; i < heads * hp; i += kLatWriteThreads) {
-        Word* w = reinterpret_cast<Word*>(qr) + i;
-        *w = turn(*w, i % hp);
+    const T* c = qr + (size_t)heads * rp;
+    float ss = 0.f;
+    for (int i = lane * 8; i < rank_pad; i += 256) {
+        x.load(c + i);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+            const float v = Cvt<T>::to_f(x.e[k]);
+            ss = fmaf(v, v, ss);
+        }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
-    __syncthreads();
-    float tot = 0.f;
-#pragma unroll
-    for (int w = 0; w < kLatWriteThreads / 32; ++w) tot += red[w];
-    const float inv = 1.f / sqrtf(tot / rank + eps);
+    const float inv = 1.f / sqrtf(ss / rank + eps);
+    const int s = seq_ids[t];
+    T* dst = cache_row(kv, page_table, max_pages, page_size, s, past_len[s] + t - q_start[s], page_size, rank_pad + rp);
     if (!dst) return;
-    for (int i = tid; i < rank_pad / 2; i += kLatWriteThreads) {
-        alignas(8) T e[2];
-        *reinterpret_cast<Word*>(e) = reinterpret_cast<const Word*>(c)[i];
-        e[0] = Cvt<T>::from_f(Cvt<T>::to_f(e[0]) * inv * norm_w[2 * i]);
-        e[1] = Cvt<T>::from_f(Cvt<T>::to_f(e[1]) * inv * norm_w[2 * i + 1]);
-        reinterpret_cast<Word*>(dst)[i] = *reinterpret_cast<Word*>(e);
+    for (int i = lane * 8; i < rank_pad; i += 256) {
+        x.load(c + i);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) x.e[k] = Cvt<T>::from_f(Cvt<T>::to_f(x.e[k]) * inv * norm_w[i + k]);
+        x.store(dst + i);
     }
-    for (int j = tid; j < hp; j += kLatWriteThreads) reinterpret_cast<Word*>(dst + rank_pad)[j] = turn(reinterpret_cast<const Word*>(kr)[j], j);
+    for (int i = lane * 8; i < rp; i += 256) {
+        x.load(c + rank_pad + i);
+        x.turn(cs, i / 2, half);
+        x.store(dst + rank_pad + i);
+    }
 }
 
 // One warp per row and group of heads of packed q | k | v: a lane holds eight consecutive features, d / 8 lanes a head, so a warp takes
@@ -332,9 +347,12 @@ extern "C" int telb_latent_write(void* rows, void* kv_layer, const float* cos_si
                                  const int* q_start, const int* past_len, const int* page_table, int tokens, int max_pages, int page_size, int heads, int kp,
                                  int rp, int rank_pad, int rank, int rot, int table_ld, float eps, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (rot % 2 || rot > rp || rank > rank_pad || rank <= 0) return fail("telb_latent_write: sizes");
-    TELB_BY_TYPE(dtype, TELB_LAUNCH("latent_write_kernel", (latent_write_kernel<T>), dim3(tokens), dim3(kLatWriteThreads), 0, stream, (T*)rows, (T*)kv_layer, cos_sin, norm_w,
-                                    positions, seq_ids, q_start, past_len, page_table, max_pages, page_size, heads, kp, rp, rank_pad, rank, rot, table_ld, eps))
+    if (rot % 2 || rot > rp || rp % 8 || kp % 8 || rank_pad % 8 || rank > rank_pad || rank <= 0) return fail("telb_latent_write: sizes");
+    const int parts = 1 + (heads * rp + 1023) / 1024;
+    const long long warps = (long long)tokens * parts;
+    TELB_BY_TYPE(dtype, TELB_LAUNCH("latent_write_kernel", (latent_write_kernel<T>), dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, stream, (T*)rows, (T*)kv_layer,
+                                    cos_sin, norm_w, positions, seq_ids, q_start, past_len, page_table, max_pages, page_size, tokens, heads, kp, rp, rank_pad, rank,
+                                    rot, table_ld, eps, parts))
     TELB_CHECK_LAUNCH("latent_write_kernel");
     return 0;
 }
