@@ -2,13 +2,14 @@
 //
 //   latent_decode     few rows per sequence.  The key expansion has been folded into the query (one [rank + rot] row per token and head),
 //                     so every (token, head) pair is a column against the same cached rows:
-//                         Sᵀ[64 tok, NC] = rows[64 tok, rank + rot] · Qᵀ        Oᵀ[rank, NC] += latentᵀ[rank, 64 tok] · Pᵀ
+//                         Sᵀ[TILE tok, NC] = rows[TILE tok, rank + rot] · Qᵀ    Oᵀ[rank, NC] += latentᵀ[rank, TILE tok] · Pᵀ
 //                     A tile of rows is loaded once and serves both products (K-major for the scores, MN-major for the output).  It comes
 //                     in pairs of 64-feature chunks through a ring that holds at least one tile: scores start with the first pair, and a
 //                     pair's slot is refilled as soon as its 128 output features are done.  The products are narrow, so consecutive ones go
 //                     to different accumulators (four for the scores, two output blocks in turn) instead of waiting for one another.
-//                     A tile is one page, so that two CTAs fit on an SM and one computes while the other loads; the upper half of the
-//                     128-row score MMA reads whatever lies behind the chunk, and nobody reads its results.
+//                     Tiles of two pages use the tensor cores best and fill the ring of the one CTA that an SM holds.  With few rows
+//                     in flight tiles of one page spread the work over more CTAs, two per SM; the upper half of their 128-row score
+//                     MMA reads whatever lies behind the chunk, and nobody reads its results.
 //   latent_prefill    prompt portions, over keys and values expanded from the latents ([rows, heads, k | v], one product per step).  The
 //                     rotated key part is not expanded: a K tile is made of chunks of the head's keys and chunks of the shared rows.
 //                     256 query rows per CTA in two tiles with a softmax warpgroup each; probabilities stay in TMEM (the A operand
@@ -42,9 +43,7 @@ struct LatentDecParams {
 };
 
 constexpr int kLatThreads = 192;
-constexpr int kLatTile = 64;                 // cached rows per tile = 1 page
-constexpr int kLatChunk = kLatTile * 128;    // bytes of [64 rows x 64 features]
-constexpr int kLatSlot = 2 * kLatChunk;
+constexpr int kLatPage = 64;
 
 // Maxima of N column values over the warp; lane l receives that of column l % N.
 template <int N>
@@ -70,12 +69,14 @@ __device__ __forceinline__ bool lat_any(bool yes) {
     return r != 0;
 }
 
-// grid (column blocks, splits, sequences).  NC: (token, head) columns of a block.
-template <typename T, int NC>
-__global__ void __launch_bounds__(kLatThreads, NC == 16 ? 2 : 1)
+// grid (column blocks, splits, sequences).  NC: (token, head) columns of a block; TILE: cached rows of a tile, one or two pages.
+template <typename T, int NC, int TILE>
+__global__ void __launch_bounds__(kLatThreads, NC == 16 && TILE == 64 ? 2 : 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_kv, const __grid_constant__ LatentDecParams p) {
     constexpr bool kBf16 = std::is_same<T, __nv_bfloat16>::value;
-    constexpr int kQChunk = NC * 128, kPBytes = 2 * NC * 128;        // [high | low rows of the columns][64 tokens]
+    constexpr int kQChunk = NC * 128, kPSpan = 2 * NC * 128;         // [high | low rows of the columns][64 tokens]
+    constexpr int kPBytes = TILE / 64 * kPSpan;
+    constexpr int kLatTile = TILE, kLatChunk = TILE * 128, kLatSlot = 2 * kLatChunk;      // chunk: bytes of [TILE rows x 64 features]
     constexpr int kOCol = 4 * NC, kOBlock = 2 * NC;      // TMEM: four partial scores, then per 128 output features high | low columns
     constexpr int kTmemCols = NC == 16 ? 256 : 512;
     static_assert(kOCol + 4 * kOBlock <= kTmemCols, "scores and four output blocks");
@@ -147,13 +148,16 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
             bool ok = true;
             int slot = 0;
             uint32_t ph = 1;
-            int next = 0;                                // pages are fetched 32 tiles at a time
+            constexpr int kPages = TILE / kLatPage, kAhead = 32 / kPages;
+            int next = 0;                                // the pages of kAhead tiles are fetched at a time
             for (int j = 0; j < ntiles && ok; ++j) {
-                if ((j & 31) == 0) {
-                    const int lp = j0 + j + lane;
+                if (j % kAhead == 0) {
+                    const int lp = (j0 + j) * kPages + lane;
                     next = lp < p.max_pages ? pages[lp] : -1;
                 }
-                const int row = max(__shfl_sync(0xffffffffu, next, j & 31), 0) * kLatTile;      // rows past the end are masked
+                int row[kPages];                         // rows past the end are masked
+#pragma unroll
+                for (int h = 0; h < kPages; ++h) row[h] = max(__shfl_sync(0xffffffffu, next, j % kAhead * kPages + h), 0) * kLatPage;
                 for (int pr = 0; pr < p.pairs; ++pr) {
                     ok = mbar_wait(&kv_empty[slot], ph, abort_flag, p.status, kStatusProducerTimeout);
                     ok = __all_sync(0xffffffffu, ok);
@@ -161,7 +165,15 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                     uint8_t* dst = s_kv + slot * kLatSlot;
                     if (leader) {
                         mbar_expect_tx(&kv_full[slot], kLatSlot);                 // a missing second chunk arrives as zeros
-                        tma_load_3d(dst, &tma_kv, &kv_full[slot], 0, row, pr * 2);
+                        if constexpr (kPages == 1) {                              // both chunks in one copy
+                            tma_load_3d(dst, &tma_kv, &kv_full[slot], 0, row[0], pr * 2);
+                        } else {
+#pragma unroll
+                            for (int c = 0; c < 2; ++c)
+#pragma unroll
+                                for (int h = 0; h < kPages; ++h)
+                                    tma_load_3d(dst + c * kLatChunk + h * (kLatPage * 128), &tma_kv, &kv_full[slot], 0, row[h], pr * 2 + c);
+                        }
                     }
                     if (++slot == p.slots) {
                         slot = 0;
@@ -218,8 +230,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                     if (leader) {
 #pragma unroll
                         for (int k = 0; k < kLatTile / 16; ++k) {
-                            umma_f16(d_o, dv0 + (uint64_t)((k * 2048) >> 4), desc_p + 2 * k, idesc_o, (j | k) ? 1u : 0u);
-                            if (two) umma_f16(d_o + kOBlock, dv1 + (uint64_t)((k * 2048) >> 4), desc_p + 2 * k, idesc_o, (j | k) ? 1u : 0u);
+                            const uint64_t db = desc_p + (uint64_t)(((k >> 2) * kPSpan) >> 4) + 2 * (k & 3);
+                            umma_f16(d_o, dv0 + (uint64_t)((k * 2048) >> 4), db, idesc_o, (j | k) ? 1u : 0u);
+                            if (two) umma_f16(d_o + kOBlock, dv1 + (uint64_t)((k * 2048) >> 4), db, idesc_o, (j | k) ? 1u : 0u);
                         }
                         umma_commit(&kv_empty[s0]);
                         if (two) umma_commit(&kv_empty[s1]);
@@ -302,8 +315,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                 }
             }
             if (r < kLatTile) {
-                uint8_t* prow = s_p + (r & 7) * 2;
-                const int unit = r >> 3;
+                uint8_t* prow = s_p + (r >> 6) * kPSpan + (r & 7) * 2;
+                const int unit = (r & 63) >> 3;
 #pragma unroll
                 for (int c = 0; c < NC; ++c) {           // columns beyond ncol: reference +inf, probability zero
                     const float e = exp2f(s[c] - (m_used[c] == -INFINITY ? 0.f : m_used[c]));
@@ -711,23 +724,24 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
 
 constexpr int kSmemLimit = 227 * 1024;
 
-template <typename T, int NC>
+template <typename T, int NC, int TILE>
 static int launch_latent_decode(const CUtensorMap& tq, const CUtensorMap& tkv, LatentDecParams p, int nseq, int max_cols, cudaStream_t stream) {
-    // two CTAs per SM where a tile leaves room for that.  The score MMA reads one chunk beyond the last slot: Q and P, and a spare
-    const int fixed = p.chunks * NC * 128 + 2 * NC * 128 + (4 + 2 * kLatMaxSlots) * 8 + 16 + 8 * NC * 4 + 1024 + kLatChunk;
-    p.slots = (kSmemLimit / (NC == 16 ? 2 : 1) - 1024 - fixed) / kLatSlot;
-    if (p.slots < p.pairs) p.slots = (kSmemLimit - fixed) / kLatSlot;
+    // the score MMA of one-page tiles reads one chunk beyond the last slot: Q and P, and a spare
+    constexpr int chunk = TILE * 128, slot = 2 * chunk, ctas = NC == 16 && TILE == 64 ? 2 : 1;
+    const int fixed = p.chunks * NC * 128 + TILE / 64 * 2 * NC * 128 + (4 + 2 * kLatMaxSlots) * 8 + 16 + 8 * NC * 4 + 1024 + (TILE == 64 ? chunk : 0);
+    p.slots = (kSmemLimit / ctas - (ctas - 1) * 1024 - fixed) / slot;
+    if (p.slots < p.pairs) p.slots = (kSmemLimit - fixed) / slot;
     if (p.slots > kLatMaxSlots) p.slots = kLatMaxSlots;
     if (p.slots > 3 * p.pairs) p.slots = 3 * p.pairs;
     if (p.slots < p.pairs) return fail("telb_latent_attention_decode: rows too wide for shared memory");
-    const int smem = fixed + p.slots * kLatSlot;
+    const int smem = fixed + p.slots * slot;
     static int configured = 0;
     if (smem > configured) {
-        cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<T, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<T, NC, TILE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return fail("cudaFuncSetAttribute(latent_decode)", e);
         configured = smem;
     }
-    TELB_LAUNCH("latent_decode_kernel", (latent_decode_kernel<T, NC>), dim3((max_cols + NC - 1) / NC, p.splits, nseq), dim3(kLatThreads), smem, stream, tq, tkv, p);
+    TELB_LAUNCH("latent_decode_kernel", (latent_decode_kernel<T, NC, TILE>), dim3((max_cols + NC - 1) / NC, p.splits, nseq), dim3(kLatThreads), smem, stream, tq, tkv, p);
     TELB_CHECK_LAUNCH("latent_decode_kernel");
     if (p.splits > 1) {
         TELB_LAUNCH("latent_combine_kernel", (latent_combine_kernel<T>), dim3(p.rows), dim3(128), 0, stream, p.ws_o, p.ws_lse, (T*)p.out, p.rows, p.splits, p.rank_pad);
@@ -761,11 +775,13 @@ static int launch_latent_prefill(const CUtensorMap (&m)[5], LatentPrefillParams 
 using namespace telb;
 
 // q [rows = T * heads, rank_pad + rot_pad] with the key expansion folded in, cached rows [pages, 64, rank_pad + rot_pad] → out [rows, rank_pad].
-// Sizes are multiples of 64, rank_pad at most 512.  ws holds splits * rows * (rank_pad + 1) floats.
+// Sizes are multiples of 64, rank_pad at most 512; tile: 64 or 128 cached rows at a time.  ws holds splits * rows * (rank_pad + 1) floats.
 extern "C" int telb_latent_attention_decode(const void* q, const void* kv_layer, void* out, const int* q_start, const int* q_len, const int* past_len,
                                             const int* page_table, int num_seqs, int tokens, int max_q_len, int num_pages, int max_pages, int heads, int rank_pad,
-                                            int rot_pad, float scale, int splits, float* ws, long long ws_floats, int is_bf16, int* status, cudaStream_t stream) {
+                                            int rot_pad, float scale, int splits, int tile, float* ws, long long ws_floats, int is_bf16, int* status,
+                                            cudaStream_t stream) {
     if (num_seqs <= 0 || tokens <= 0) return 0;
+    if (tile != 64 && tile != 128) return fail("telb_latent_attention_decode: tiles of 64 or 128 rows");
     if (rank_pad % 64 || rot_pad % 64 || rank_pad < 64 || rank_pad > 512 || rot_pad < 64) return fail("telb_latent_attention_decode: sizes");
     if (num_seqs > 65535) return fail("telb_latent_attention_decode: too many sequences");
     LatentDecParams p{};
@@ -795,13 +811,16 @@ extern "C" int telb_latent_attention_decode(const void* q, const void* kv_layer,
     CUtensorMap tq, tkv;
     if (make_tmap_2d(&tq, dt, 2, q, p.rows, row, (uint64_t)row * 2, nc, 64, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
     {   // cached rows as [chunk][row][64 features]: one copy brings a page's rows for a pair of chunks
-        const uint64_t dims[3] = {64, (uint64_t)num_pages * kLatTile, (uint64_t)row / 64}, strides[2] = {(uint64_t)row * 2, 128};
-        const uint32_t box[3] = {64, kLatTile, 2};
+        const uint64_t dims[3] = {64, (uint64_t)num_pages * kLatPage, (uint64_t)row / 64}, strides[2] = {(uint64_t)row * 2, 128};
+        const uint32_t box[3] = {64, kLatPage, tile == 64 ? 2u : 1u};
         if (make_tmap_nd(&tkv, dt, 3, kv_layer, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
     }
-    if (nc == 16)
-        return is_bf16 ? launch_latent_decode<__nv_bfloat16, 16>(tq, tkv, p, num_seqs, max_cols, stream) : launch_latent_decode<__half, 16>(tq, tkv, p, num_seqs, max_cols, stream);
-    return is_bf16 ? launch_latent_decode<__nv_bfloat16, 32>(tq, tkv, p, num_seqs, max_cols, stream) : launch_latent_decode<__half, 32>(tq, tkv, p, num_seqs, max_cols, stream);
+#define TELB_LATENT(NC_, TILE_)                                                                                          \
+    (is_bf16 ? launch_latent_decode<__nv_bfloat16, NC_, TILE_>(tq, tkv, p, num_seqs, max_cols, stream)                   \
+             : launch_latent_decode<__half, NC_, TILE_>(tq, tkv, p, num_seqs, max_cols, stream))
+    if (nc == 16) return tile == 64 ? TELB_LATENT(16, 64) : TELB_LATENT(16, 128);
+    return tile == 64 ? TELB_LATENT(32, 64) : TELB_LATENT(32, 128);
+#undef TELB_LATENT
 }
 
 // q: packed rows of pitch ldq whose first heads * k_pad columns are the unrotated and next heads * rot_pad the rotated query parts; kv

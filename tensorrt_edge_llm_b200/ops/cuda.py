@@ -1211,21 +1211,28 @@ def _latent_plan(meta: StepMeta, heads: int, device, force: Optional[str]) -> La
     return p
 
 
-def _latent_splits(blocks: int, max_seq_len: int, slots: int) -> int:
-    """Splits of the cached rows so that the (column block, split, sequence) CTAs come out near whole waves of ``slots`` CTAs."""
-    tiles = max(1, (max_seq_len + 63) // 64)
-    best, cost = 1, None
-    for s in range(1, min(tiles, 64) + 1):
-        waves = (blocks * s + slots - 1) // slots
-        c = waves * ((tiles + s - 1) // s + 1.0) + (1.0 + s / 32 if s > 1 else 0.0)      # in tiles; start-up and merge in the same unit
-        if cost is None or c < cost - 1e-9:
-            best, cost = s, c
+def _latent_splits(blocks: int, max_seq_len: int, columns: int) -> Tuple[int, int]:
+    """``(splits, rows per tile)`` of the cached rows for ``blocks`` (column block, sequence) pairs, so that the CTAs come out near whole
+    waves.  Costs in the time of a one-page tile; a two-page tile takes little longer than that while an SM has a CTA to itself."""
+    best, cost = (1, 128), None
+    for tile, slots, unit in ((64, 296 if columns == 16 else 148, 1.7 if columns == 16 else 1.0), (128, 148, 1.0)):
+        tiles = max(1, (max_seq_len + tile - 1) // tile)
+        for s in range(1, min(tiles, 64) + 1):
+            ctas = blocks * s
+            waves = (ctas + slots - 1) // slots
+            alone = ctas <= 148                              # one CTA per SM: it does not share the tensor cores
+            c = waves * ((tiles + s - 1) // s * ((0.9 if tile == 64 else 1.0) if alone else unit) + 1.0) + (1.0 + s / 32 if s > 1 else 0.0)
+            if cost is None or c < cost - 1e-9:
+                best, cost = (s, tile), c
     return best
 
 
 def latent_attention(rows, kv_layer, meta: StepMeta, kv_up, key_up_t, spec, kernel: Optional[str] = None) -> torch.Tensor:
     """See :func:`ops.latent_attention`.  16-bit steps run the tcgen05 kernels where the sizes fit (``kernel`` forces ``"folded"`` or
-    ``"expanded"``); fp32 rows and other sizes run on the CUDA cores (``"simt"``)."""
+    ``"expanded"``, ``"folded-64"`` / ``"folded-128"`` also the tile); fp32 rows and other sizes run on the CUDA cores (``"simt"``)."""
+    force_tile = 0
+    if kernel in ("folded-64", "folded-128"):
+        kernel, force_tile = "folded", int(kernel[7:])
     if meta.tree_mask is not None:
         raise ValueError("latent attention covers causal masks only")
     t, n, dev = rows.shape[0], spec.num_heads, rows.device
@@ -1247,10 +1254,11 @@ def latent_attention(rows, kv_layer, meta: StepMeta, kv_up, key_up_t, spec, kern
         o = torch.empty(tf, n, spec.rank_pad, dtype=rows.dtype, device=dev)
         if tc:
             nc = 16 if max_q * n <= 16 else 32
-            splits = _latent_splits(seqs * ((max_q * n + nc - 1) // nc), plan.max_seq_len, 296 if nc == 16 else 148)
+            splits, tile = _latent_splits(seqs * ((max_q * n + nc - 1) // nc), plan.max_seq_len, nc)
+            tile = force_tile or tile
             _check(lib().telb_latent_attention_decode(
                 _p(q), _p(kv_layer), _p(o), _p(q_start), _p(q_len), _p(past_len), _p(table), c_int(seqs), c_int(tf), c_int(max_q),
-                c_int(kv_layer.shape[0]), c_int(table.shape[1]), c_int(n), c_int(spec.rank_pad), c_int(spec.rot_pad), c_float(spec.scale), c_int(splits),
+                c_int(kv_layer.shape[0]), c_int(table.shape[1]), c_int(n), c_int(spec.rank_pad), c_int(spec.rot_pad), c_float(spec.scale), c_int(splits), c_int(tile),
                 _p(ws.attn_ws), c_ll(ws.attn_ws.numel()), c_int(_is_bf16(rows)), _p(ws.status), _stream()), "latent_attention_decode", 2 if splits > 1 else 1)
         else:
             _check(lib().telb_latent_attention_simt(

@@ -88,7 +88,7 @@ def test_channel_delta_slices(heads):
 LATENT = [(16, 128, 64, 128, 512), (3, 40, 24, 56, 72), (5, 64, 32, 64, 192), (40, 64, 64, 128, 256), (2, 200, 8, 96, 64)]
 
 
-@pytest.mark.parametrize("kernel", ["folded", "expanded", "simt"])
+@pytest.mark.parametrize("kernel", ["folded", "folded-64", "folded-128", "expanded", "simt"])
 @pytest.mark.parametrize("heads, dim, rot, dv, rank", LATENT)
 def test_latent_attention_kernels(heads, dim, rot, dv, rank, kernel):
     """Both tensor-core forms and the CUDA-core one: prompts, portions behind a past, page borders, single rows."""
@@ -97,6 +97,13 @@ def test_latent_attention_kernels(heads, dim, rot, dv, rank, kernel):
         if kernel == "expanded" and max(lens) == 1:
             continue
         assert cases.latent_case(DEV, torch.bfloat16, heads, dim, rot, dv, rank, lens, past, kernel) < tol, (lens, past)
+
+
+@pytest.mark.parametrize("needle", [0, 63, 64, 127, 128, 255])
+@pytest.mark.parametrize("kernel", ["folded-64", "folded-128"])
+def test_latent_needle_in_tiles(needle, kernel):
+    for past in ([needle, 700, 256], [needle + 1, 129, 383]):
+        assert cases.latent_case(DEV, torch.bfloat16, 4, 64, 32, 64, 128, [1, 3, 2], past, kernel, needle=needle) < 8e-2
 
 
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
