@@ -5,9 +5,9 @@
 //   S <- diag(g) S;  u = beta (v - Sᵀ k);  S <- S + k uᵀ;  o = Sᵀ q
 //   y = o / rms(o) · w · sigmoid(gate)
 //
-// Prompt portions run as five launches: `prep` twice (values; q, k and decays: convolutions and norms, parallel over tokens), `walk` (the recurrence, state in
-// registers), `out` (head norm and gate) and `roll` (convolution history).  A step with one row per sequence runs `decode`, everything
-// in one launch (`roll` behind it when several heads share a q / k head).
+// Prompt portions run as five launches: `prep` twice (values; q, k and decays: convolutions and norms, parallel over tokens), `walk` (the
+// recurrence, state in registers), `out` (head norm and gate) and `roll` (convolution history).  A step with one row per sequence runs
+// `decode`, everything in one launch (`roll` behind it when several heads share a q / k head).
 //
 // The walk takes four tokens at a time and never leaves fp32.  With S the state before a block, D_i = g_1 ∘ .. ∘ g_i and k, q normalised,
 //
@@ -577,6 +577,150 @@ __global__ void __launch_bounds__(128) channel_delta_walk_kernel(const __grid_co
     }
 }
 
+// The walk for few (sequence, head) pairs and keys of 128 or 256: all 32 lanes share the rows of four columns (four rows, G granules each),
+// so a vector costs one shared-memory read per warp and granule instead of four and the chain of a block is short.  The 32 products of
+// a block (columns x (k, q) x tokens) are reduced so that lane 8 c + 4 a + i holds product a of column c and token i.
+template <typename T, int G>
+__global__ void __launch_bounds__(128) channel_delta_walk_narrow_kernel(const __grid_constant__ ChannelDeltaParams p) {
+    pdl_wait();
+    constexpr int DK = G * 128, C = 4, kCols = 16;
+    constexpr unsigned kAll = 0xffffffffu;
+    constexpr int kFloats = 13 * DK + kScalars, kVBytes = kCols * kBlk * (int)sizeof(T), kStage = kFloats * 4 + kVBytes;
+    extern __shared__ __align__(16) uint8_t walk_smem[];
+    __shared__ uint64_t full[kWalkStages];
+    __shared__ uint32_t abort_word;
+    volatile uint32_t* abort_flag = &abort_word;
+    const int seq = blockIdx.z, h = blockIdx.y;
+    const int ql = p.q_len[seq];
+    if (ql <= 0) return;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int col0 = blockIdx.x * kCols + warp * C, c_own = lane >> 3, i_own = lane & 3;
+    const int r0 = p.q_start[seq], blk0 = first_block(r0, seq), chunks = (ql + kBlk - 1) / kBlk;
+    auto fetch = [&](int chunk) {
+        uint64_t* bar = &full[chunk % kWalkStages];
+        uint8_t* st = walk_smem + (chunk % kWalkStages) * kStage;
+        const size_t blk = (size_t)(blk0 + chunk) * p.heads + h;
+        mbar_expect_tx(bar, kStage);
+        bulk_load(st, p.blocks + blk * kFloats, kFloats * 4, bar);
+        bulk_load(st + kFloats * 4, reinterpret_cast<const T*>(p.v_blocks) + (blk * p.dv + blockIdx.x * kCols) * kBlk, kVBytes, bar);
+    };
+    if (tid == 0) {
+        for (int s = 0; s < kWalkStages; ++s) mbar_init(&full[s], 1);
+        abort_word = 0;
+        mbar_fence_init();
+        for (int s = 0; s < kWalkStages && s < chunks; ++s) fetch(s);
+    }
+    // granule at place x of a vector in lane order holds rows 4 m .. 4 m + 3 with m = place_granule(x)
+    auto first_row = [&](int g) {
+        const int x = lane + 32 * g, j = x >> 3;
+        return 4 * ((j >> 1) * 16 + 2 * (x & 7) + (j & 1));
+    };
+    f2 S[2 * G][C];
+    float* state = p.state + (((size_t)p.slot_ids[seq] * p.heads + h) * DK) * p.dv + col0;
+    const bool fresh = p.past_len[seq] == 0;
+#pragma unroll
+    for (int r = 0; r < 2 * G; ++r) {
+        float a[C] = {}, b[C] = {};
+        if (!fresh) {
+            const size_t row = first_row(r >> 1) + 2 * (r & 1);
+            load_n<float, C>(state + row * p.dv, a);
+            load_n<float, C>(state + (row + 1) * p.dv, b);
+        }
+#pragma unroll
+        for (int c = 0; c < C; ++c) S[r][c] = f2_pack(a[c], b[c]);
+    }
+    T* out = reinterpret_cast<T*>(p.o) + ((size_t)r0 + i_own) * p.heads * p.dv + (size_t)h * p.dv + col0 + c_own;
+    const int n_row = 13 * DK + 6 + i_own * (i_own + 1) / 2;
+    __syncthreads();
+    bool ok = true;
+    for (int ch = 0; ch < chunks; ++ch) {
+        ok = mbar_wait(&full[ch % kWalkStages], (ch / kWalkStages) & 1, abort_flag, p.status, kStatusEpilogueTimeout);
+        if (!ok) break;
+        const float* st = reinterpret_cast<const float*>(walk_smem + (ch % kWalkStages) * kStage);
+        f2 acc[2 * kBlk][C];
+#pragma unroll
+        for (int g = 0; g < G; ++g)
+#pragma unroll
+            for (int i = 0; i < 2 * kBlk; ++i) {
+                const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(st + i * DK + (lane + 32 * g) * 4);
+#pragma unroll
+                for (int c = 0; c < C; ++c) {
+                    acc[i][c] = g == 0 ? f2_mul(S[0][c], x.x) : f2_fma(S[2 * g][c], x.x, acc[i][c]);
+                    acc[i][c] = f2_fma(S[2 * g + 1][c], x.y, acc[i][c]);
+                }
+            }
+        float sums[32];
+#pragma unroll
+        for (int c = 0; c < C; ++c)
+#pragma unroll
+            for (int i = 0; i < 2 * kBlk; ++i) sums[c * 8 + i] = f2_sum(acc[i][c]);
+        const float total = total_of_lane(sums, lane);
+        float w[kBlk], v[kBlk], u[kBlk];
+        load_n<T, kBlk>(reinterpret_cast<const T*>(st + kFloats) + (warp * C + c_own) * kBlk, v);
+        alignas(16) float m[8], beta[kBlk];
+        reinterpret_cast<float4*>(m)[0] = *reinterpret_cast<const float4*>(st + 13 * DK);
+        reinterpret_cast<float4*>(m)[1] = *reinterpret_cast<const float4*>(st + 13 * DK + 4);
+        *reinterpret_cast<float4*>(beta) = *reinterpret_cast<const float4*>(st + 13 * DK + 16);
+        float nr[kBlk];
+#pragma unroll
+        for (int j = 0; j < kBlk; ++j) nr[j] = j <= i_own ? st[n_row + j] : 0.f;
+#pragma unroll
+        for (int i = 0; i < kBlk; ++i) w[i] = __shfl_sync(kAll, total, (lane & 24) + i);
+        u[0] = beta[0] * (v[0] - w[0]);
+        u[1] = beta[1] * (v[1] - w[1] - m[0] * u[0]);
+        u[2] = beta[2] * (v[2] - w[2] - m[1] * u[0] - m[2] * u[1]);
+        u[3] = beta[3] * (v[3] - w[3] - m[3] * u[0] - m[4] * u[1] - m[5] * u[2]);
+        if ((lane & 4) && i_own < ql - ch * kBlk)
+            *out = Cvt<T>::from_f(total + nr[0] * u[0] + nr[1] * u[1] + (nr[2] * u[2] + nr[3] * u[3]));
+        out += (size_t)kBlk * p.heads * p.dv;
+        f2 ub[C][kBlk];
+#pragma unroll
+        for (int c = 0; c < C; ++c)
+#pragma unroll
+            for (int i = 0; i < kBlk; ++i) {
+                const float x = __shfl_sync(kAll, u[i], c * 8);
+                ub[c][i] = f2_pack(x, x);
+            }
+#pragma unroll
+        for (int g = 0; g < G; ++g) {
+            ulonglong2 x[kBlk + 1];
+#pragma unroll
+            for (int i = 0; i <= kBlk; ++i) x[i] = *reinterpret_cast<const ulonglong2*>(st + (2 * kBlk + i) * DK + (lane + 32 * g) * 4);
+#pragma unroll
+            for (int c = 0; c < C; ++c) {
+                S[2 * g][c] = f2_mul(S[2 * g][c], x[kBlk].x);
+                S[2 * g + 1][c] = f2_mul(S[2 * g + 1][c], x[kBlk].y);
+            }
+#pragma unroll
+            for (int i = 0; i < kBlk; ++i)
+#pragma unroll
+                for (int c = 0; c < C; ++c) {
+                    S[2 * g][c] = f2_fma(x[i].x, ub[c][i], S[2 * g][c]);
+                    S[2 * g + 1][c] = f2_fma(x[i].y, ub[c][i], S[2 * g + 1][c]);
+                }
+        }
+        if (ch + kWalkStages < chunks) {                  // every warp is done with the stage: refill it
+            __syncthreads();
+            if (tid == 0) fetch(ch + kWalkStages);
+        }
+    }
+    pdl_launch_dependents();
+    if (!ok) {                                            // a copy never arrived: leave the state alone, let what is in flight land
+        const uint64_t t0 = global_timer_ns();
+        while (global_timer_ns() - t0 < 200000ull) __nanosleep(1000);
+        return;
+    }
+#pragma unroll
+    for (int r = 0; r < 2 * G; ++r) {
+        float a[C], b[C];
+#pragma unroll
+        for (int c = 0; c < C; ++c) asm("mov.b64 {%0, %1}, %2;" : "=f"(a[c]), "=f"(b[c]) : "l"(S[r][c]));
+        const size_t row = first_row(r >> 1) + 2 * (r & 1);
+        store_n<float, C>(state + row * p.dv, a);
+        store_n<float, C>(state + (row + 1) * p.dv, b);
+    }
+}
+
 // ---- out: head norm and gate, one warp per (row, head) ---------------------------------------------------
 template <typename T, int C>
 __device__ void delta_out(const ChannelDeltaParams& p, size_t t, int h) {
@@ -760,15 +904,35 @@ static int launch_walk_as(const ChannelDeltaParams& p, cudaStream_t stream) {
     return 0;
 }
 
+template <typename T, int G>
+static int launch_walk_narrow(const ChannelDeltaParams& p, cudaStream_t stream) {
+    constexpr int smem = ((13 * G * 128 + kScalars) * 4 + 16 * kBlk * (int)sizeof(T)) * kWalkStages;
+    if (smem > 48 * 1024) {
+        static bool configured = false;
+        if (!configured) {
+            cudaError_t e = cudaFuncSetAttribute(channel_delta_walk_narrow_kernel<T, G>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+            if (e != cudaSuccess) return fail("cudaFuncSetAttribute(channel_delta_walk_narrow)", e);
+            configured = true;
+        }
+    }
+    TELB_LAUNCH_SERIAL("channel_delta_walk_narrow_kernel", (channel_delta_walk_narrow_kernel<T, G>), dim3(p.dv / 16, p.heads, p.num_seqs), dim3(128), smem, stream, p);
+    TELB_CHECK_LAUNCH("channel_delta_walk_narrow_kernel");
+    return 0;
+}
+
 static int g_walk_cols = 0;          // columns per lane; 0 = by the number of columns
 
 template <typename T, int RPL>
 static int launch_walk(const ChannelDeltaParams& p, cudaStream_t stream) {
     // few (sequence, head) pairs: narrow slices, so that every scheduler has a chain of its own; many: wide ones, which read less
     const long long columns = (long long)p.num_seqs * p.heads * p.dv;
-    int cpl = columns / 4 <= 8LL * sm_count() ? 1 : (RPL > 16 || columns / 8 <= 8LL * sm_count()) ? 2 : 4;
+    int cpl = columns / 4 <= 8LL * sm_count() ? 1 : RPL > 16 ? 2 : 4;
     if (g_walk_cols) cpl = g_walk_cols;
-    if (cpl == 1) return launch_walk_as<T, RPL, 1>(p, stream);
+    if constexpr (RPL >= 16) {
+        if (cpl == 1) return launch_walk_narrow<T, RPL / 16>(p, stream);
+    } else {
+        if (cpl == 1) return launch_walk_as<T, RPL, 1>(p, stream);
+    }
     if (cpl == 2 || RPL > 16) return launch_walk_as<T, RPL, 2>(p, stream);
     return launch_walk_as<T, RPL, (RPL > 16 ? 2 : 4)>(p, stream);
 }
