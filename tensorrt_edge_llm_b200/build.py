@@ -29,7 +29,8 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
               "-Xcompiler", "-fPIC", "-Xcompiler", "-Wall", "--expt-relaxed-constexpr",
               "-diag-suppress", "177", "-diag-suppress", "550"]
 # sources compiled without --use_fast_math: their exponentials, tanh and divisions feed routers, norms and recurrences
-NO_FAST_MATH: set = {"attention_simt.cu", "channel_delta.cu", "gemm_f32.cu", "latent.cu", "mlstm.cu", "mlstm_tc5.cu", "moe.cu", "stream_norm.cu"}
+NO_FAST_MATH: set = {"attention_simt.cu", "channel_delta.cu", "gemm_f32.cu", "latent.cu", "lightning.cu", "lightning_tc5.cu", "mlstm.cu",
+                      "mlstm_tc5.cu", "moe.cu", "stream_norm.cu", "stream_post.cu"}
 
 
 def _newer(src: str, dst: str, deps: List[str]) -> bool:
@@ -49,6 +50,8 @@ def _run(cmd: List[str]) -> str:
 # Kernel sources of one model family, for a process that serves only that family from a tree without built libraries: they link
 # into a library of their own (`libtelb_kernels-<family>.so`) in a fraction of the time of the whole set.
 KERNEL_SETS = {
+    "begupel": ["attention_decode_tc5.cu", "attention_simt.cu", "attention_tc5.cu", "attention_tc5_extra.cu", "channel_delta.cu", "elementwise.cu",
+                "gemm_f32.cu", "gemm_skinny_tc5.cu", "gemm_tc5.cu", "latent.cu", "lightning.cu", "nvfp4_host.cu", "stream_post.cu"],
     "debonex": ["attention_decode_tc5.cu", "attention_latent_tc5.cu", "attention_simt.cu", "attention_tc5.cu", "attention_tc5_extra.cu",
                 "channel_delta.cu", "elementwise.cu", "gemm_f32.cu", "gemm_skinny_tc5.cu", "gemm_tc5.cu", "latent.cu", "nvfp4_host.cu", "stream_norm.cu"],
     "dimesun": ["attention_decode_tc5.cu", "attention_simt.cu", "attention_tc5.cu", "attention_tc5_extra.cu", "elementwise.cu", "gemm_f32.cu",

@@ -39,8 +39,11 @@ LAYER_MAMBA = "mamba"
 LAYER_GDN = "gdn"
 LAYER_MLSTM = "mlstm"
 LAYER_CHANNEL_DELTA = "channel_delta"
+LAYER_LIGHTNING = "lightning"
+LAYER_PARALLEL = "parallel"        # attention and a delta rule side by side on the same input
 LAYER_MLP = "mlp"
 LAYER_MOE = "moe"
+KV_LAYERS = (LAYER_ATTENTION, LAYER_PARALLEL)     # kinds that keep rows in the paged cache
 
 
 @dataclass
@@ -221,6 +224,11 @@ class AttentionConfig:
     unit_qk: bool = False            # queries and keys divided by their root mean square over the head, without a weight
     temp_coef: float = 0.0           # query temperature: q times 1 + coef * ln(floor((position + 1) / every) + 1)
     temp_every: float = 1.0
+    window: int = 0                  # > 0: position i sees itself and the window - 1 positions before it
+    row_norm: bool = False           # RMS norm with a weight over all heads of a query (key) row at once, before rotation
+    interleaved: bool = False        # rotated pairs are neighbours (2i, 2i + 1)
+    rope_factor: float = 1.0         # linear scaling: every frequency of queries and keys over this
+    rotated_values: bool = False     # values turn by their position over all v_head_dim features, outputs turn back by theirs
 
     @property
     def pad(self) -> int:
@@ -284,6 +292,8 @@ class ChannelDeltaConfig:
     conv_kernel: int = 4
     decay_rank: int = 128            # inner size of the two-step projection behind the decays
     gate_rank: int = 128             # the same for the output gate
+    head_decay: bool = False         # one decay per head instead of one per key channel
+    silu_gate: bool = False          # the output gate is silu instead of a sigmoid
 
     @property
     def k_pad(self) -> int:
@@ -297,6 +307,24 @@ class ChannelDeltaConfig:
     def conv_dim(self) -> int:
         """Channels of the packed q | k | v rows."""
         return 2 * self.num_kv_heads * self.k_pad + self.num_heads * self.v_pad
+
+
+@dataclass
+class LightningConfig:
+    """Linear attention with a constant decay per head: ``S <- decay S + k v^T``, read by q, with silu on q, k and v."""
+
+    num_heads: int = 8
+    head_k_dim: int = 128
+    head_v_dim: int = 128
+    decay: List[float] = field(default_factory=list)
+
+    @property
+    def k_pad(self) -> int:
+        return pad_head(self.head_k_dim)
+
+    @property
+    def v_pad(self) -> int:
+        return (self.head_v_dim + 127) // 128 * 128
 
 
 @dataclass
@@ -325,6 +353,11 @@ class LayerConfig:
     latent: Optional[LatentConfig] = None              # kind "attention" over cached latents
     delta: Optional[ChannelDeltaConfig] = None
     ff: int = 0                                        # dense gated feed-forward of this size
+    ff_act: str = "gelu_tanh"                          # its gate: "gelu_tanh" or "relu"
+    ff_bias: bool = False                              # its projections have biases
+    lightning: Optional[LightningConfig] = None
+    attention_mult: float = 1.0                        # kind "parallel": the layer's output is attention_mult * attention
+    delta_mult: float = 1.0                            # + delta_mult * delta rule
 
     @property
     def cached(self):
@@ -335,7 +368,9 @@ class LayerConfig:
     def from_dict(cls, d: Dict[str, Any]) -> "LayerConfig":
         sub = lambda c, v: c(**v) if isinstance(v, dict) else v
         return cls(d["kind"], sub(AttentionConfig, d.get("attention")), sub(MlstmConfig, d.get("mlstm")), sub(MoeConfig, d.get("moe")),
-                   sub(LatentConfig, d.get("latent")), sub(ChannelDeltaConfig, d.get("delta")), int(d.get("ff", 0)))
+                   sub(LatentConfig, d.get("latent")), sub(ChannelDeltaConfig, d.get("delta")), int(d.get("ff", 0)), d.get("ff_act", "gelu_tanh"),
+                   bool(d.get("ff_bias", False)), sub(LightningConfig, d.get("lightning")), float(d.get("attention_mult", 1.0)),
+                   float(d.get("delta_mult", 1.0)))
 
 
 @dataclass
@@ -405,6 +440,13 @@ class ModelConfig:
     residual_mult: float = 1.0              # the residual stream advances by this multiple of a layer's output
     embedding_mult: float = 1.0             # looked-up embedding rows times this enter the residual stream
     logits_mult: float = 1.0                # logits are this multiple of the head's output
+    norm_groups: int = 1                    # RMS norms of the stream go over this many equal parts of a row
+    input_conv: int = 0                     # taps of the causal convolution that every mixer's input is added to (0 = none)
+    # bigram table: row (previous token * bigram_mul_prev + token * bigram_mul_cur) mod bigram_buckets joins the token's embedding,
+    # row bigram_buckets for a sequence's first token (0 = none)
+    bigram_buckets: int = 0
+    bigram_mul_prev: int = 0
+    bigram_mul_cur: int = 0
     diffusion: Optional[DiffusionConfig] = None      # block-diffusion checkpoints (model_type "diffusion_gemma")
     # draft heads
     draft_type: Optional[str] = None        # "eagle3" / "mtp"
@@ -503,11 +545,11 @@ class ModelConfig:
         if not self.layer_specs:
             return None
         specs = [self.layer_specs[i] for i in self.layer_run_ids]
-        return [(sp.cached.num_kv_heads, sp.cached.pad) for sp in specs if sp.kind == LAYER_ATTENTION]
+        return [(sp.cached.num_kv_heads, sp.cached.pad) for sp in specs if sp.kind in KV_LAYERS]
 
     def kv_planes(self) -> List[int]:
         """Cached planes per attention layer of such a stack: 2 (keys, values) or 1 (latent rows)."""
-        return [self.layer_specs[i].cached.cache_planes for i in self.layer_run_ids if self.layer_specs[i].kind == LAYER_ATTENTION]
+        return [self.layer_specs[i].cached.cache_planes for i in self.layer_run_ids if self.layer_specs[i].kind in KV_LAYERS]
 
     def kv_donor(self, layer_idx: int) -> int:
         """The layer whose KV cache ``layer_idx`` attends over, or -1 when it writes and reads its own."""
@@ -542,7 +584,7 @@ class ModelConfig:
 
     @property
     def num_attn_layers(self) -> int:
-        return sum(t == LAYER_ATTENTION for t in self.layer_types)
+        return sum(t in KV_LAYERS for t in self.layer_types)
 
     @property
     def num_mamba_layers(self) -> int:
@@ -607,6 +649,8 @@ class ModelConfig:
             return _parse_dimesun(cls, hf, quant)
         if str(hf.get("architecture", "")) == "Debonex":
             return _parse_debonex(cls, hf, quant)
+        if str(hf.get("architecture", "")) == "Begupel":
+            return _parse_begupel(cls, hf, quant)
         llm = hf.get("text_config", hf)
         model_type = llm.get("model_type", hf.get("model_type", "llama"))
         heads = int(llm["num_attention_heads"])
@@ -974,6 +1018,63 @@ def _debonex_stack(specs: List[LayerConfig]) -> Dict[str, Any]:
                 layer_types=[sp.kind for sp in specs], mlp_types=[LAYER_MLP if sp.ff else "none" for sp in specs], layer_specs=specs)
 
 
+def _parse_begupel(cls, hf: Dict[str, Any], quant: Optional["QuantConfig"]) -> "ModelConfig":
+    """Begupel: layers listed one by one, norms on the sublayers' outputs only, in groups; a short convolution in front of every mixer;
+    lightning attention, or windowed attention with rotated values beside a gated delta rule; relu-gated feed-forwards with biases;
+    bigram embeddings and capped logits."""
+    specs: List[LayerConfig] = []
+    for i, entry in enumerate(hf["layers"]):
+        m, f, kind = entry["mixer"], entry.get("mlp"), str(entry["type"])
+        spec = LayerConfig(kind=kind)
+        if kind == LAYER_LIGHTNING:
+            spec.lightning = l = LightningConfig(int(m["heads"]), int(m["dim"]), int(m["vdim"]), [float(x) for x in m["decay"]])
+            if len(l.decay) != l.num_heads or any(not 0.0 <= x <= 1.0 for x in l.decay):
+                raise ValueError(f"layer {i}: one decay between 0 and 1 per head")
+        elif kind == LAYER_PARALLEL:
+            a, d = m["left"], m["right"]
+            rot = a.get("rot") or {}
+            spec.attention = at = AttentionConfig(
+                num_heads=int(a["heads"]), num_kv_heads=int(a["kv_heads"]), head_dim=int(a["dim"]), v_head_dim=int(a["vdim"]),
+                rotary_dim=int(rot.get("dims", 0)), rope_theta=float(rot.get("base", 10000.0)), scale=float(a["scale"]), fp32_weights=True,
+                window=int(a["mask"]["size"]), row_norm=True, interleaved=True, rope_factor=float((rot.get("scaling") or {}).get("factor", 1.0)),
+                rotated_values=True)
+            if at.num_heads % at.num_kv_heads or at.rotary_dim % 2 or at.rotary_dim > at.head_dim or at.v_head_dim % 2:
+                raise ValueError(f"layer {i}: query heads must be a multiple of the KV heads, and the rotated features pairs within the head")
+            if at.window < 1 or at.rope_factor <= 0:
+                raise ValueError(f"layer {i}: a position sees at least itself, and frequencies scale by a positive factor")
+            spec.delta = de = ChannelDeltaConfig(
+                num_heads=int(d["heads"]), num_kv_heads=int(d["kv_heads"]), head_k_dim=int(d["dim"]), head_v_dim=int(d["vdim"]),
+                conv_kernel=int(d["conv"]), decay_rank=0, gate_rank=0, head_decay=True, silu_gate=True)
+            if de.num_heads % de.num_kv_heads or de.conv_kernel < 1:
+                raise ValueError(f"layer {i}: heads must be a multiple of the q / k heads, and the convolution needs a tap")
+            spec.attention_mult, spec.delta_mult = float(m["left_scale"]), float(m["right_scale"])
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        if f:
+            if f.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+            spec.ff, spec.ff_act, spec.ff_bias = int(f["ff"]), "relu", True
+        specs.append(spec)
+    bigram = (hf.get("embedding") or {}).get("bigram") or {}
+    torch_dtype = str(hf.get("torch_dtype", hf.get("dtype", "bfloat16"))).replace("torch.", "")
+    base = dict(vocab_size=int(hf["vocab"]), hidden_size=int(hf["width"]), rms_norm_eps=float(hf["norm"]["eps"]),
+                norm_groups=int(hf["norm"]["groups"]), input_conv=int(hf["canon"]["taps"]), final_logit_softcapping=float(hf.get("logit_softcap") or 0.0),
+                bigram_buckets=int(bigram.get("buckets", 0)), bigram_mul_prev=int(bigram.get("mul_prev", 0)), bigram_mul_cur=int(bigram.get("mul_cur", 0)),
+                dtype=torch_dtype if torch_dtype in ("bfloat16", "float16", "float32") else "bfloat16",
+                quant=quant or QuantConfig(), bos_token_id=hf.get("bos_token_id"), eos_token_id=hf.get("eos_token_id"))
+    if base["hidden_size"] % base["norm_groups"] or base["input_conv"] < 1:
+        raise ValueError("the norm's groups must divide the width, and the input convolution needs a tap")
+    return cls(**base, **_begupel_stack(specs))
+
+
+def _begupel_stack(specs: List[LayerConfig]) -> Dict[str, Any]:
+    """Model-wide fields that follow from the layers."""
+    attn = next((sp.cached for sp in specs if sp.cached), AttentionConfig(1, 1, 64, 64))
+    return dict(model_type="begupel", intermediate_size=max((sp.ff for sp in specs), default=0), num_hidden_layers=len(specs),
+                num_attention_heads=attn.num_heads, num_key_value_heads=attn.num_kv_heads, head_dim=attn.pad, hidden_act="relu",
+                layer_types=[sp.kind for sp in specs], mlp_types=[LAYER_MLP if sp.ff else "none" for sp in specs], layer_specs=specs)
+
+
 def _parse_dspark(llm: dict, hf: dict) -> dict:
     """DSpark draft fields (``dspark_config``, a top-level ``markov_head_type`` or an architecture named ``…DSparkModel``;
     ``tensorrt_edgellm/config.py:1880-1905``): the block geometry may sit at the top level instead of in ``dflash_config``, labels
@@ -1219,6 +1320,26 @@ def debonex_config(layers: int = 12, hidden: int = 2048, vocab: int = 32768, hea
     base = dict(vocab_size=vocab, hidden_size=hidden, rms_norm_eps=1e-6, embedding_mult=2.0, logits_mult=1.0)
     base.update(over)
     return ModelConfig(**{**_debonex_stack(specs), **base})
+
+
+def begupel_config(layers: int = 12, hidden: int = 2048, vocab: int = 32768, heads: int = 16, inter: int = 6144, window: int = 1024,
+                   **over: Any) -> ModelConfig:
+    """Begupel at the sizes of a small production model: parallel layers (attention with four query heads per KV head beside a delta rule,
+    d 128) with feed-forwards and lightning layers without one in turn."""
+    specs = []
+    for i in range(layers):
+        if i % 2 == 0:
+            specs.append(LayerConfig(
+                LAYER_PARALLEL, ff=inter, ff_act="relu", ff_bias=True, attention_mult=0.7, delta_mult=0.7,
+                attention=AttentionConfig(heads, max(heads // 4, 1), 128, 128, 128, 1e6, 128 ** -0.5, fp32_weights=True, window=window, row_norm=True,
+                                          interleaved=True, rope_factor=2.0, rotated_values=True),
+                delta=ChannelDeltaConfig(heads, heads, 128, 128, 4, 0, 0, head_decay=True, silu_gate=True)))
+        else:
+            specs.append(LayerConfig(LAYER_LIGHTNING, lightning=LightningConfig(heads, 128, 128, [1 - 2.0 ** -(2 + 6 * h / heads) for h in range(heads)])))
+    base = dict(vocab_size=vocab, hidden_size=hidden, rms_norm_eps=1e-6, norm_groups=4, input_conv=4, final_logit_softcapping=30.0,
+                bigram_buckets=65536, bigram_mul_prev=1000003, bigram_mul_cur=8191)
+    base.update(over)
+    return ModelConfig(**{**_begupel_stack(specs), **base})
 
 
 def hybrid_nemotron_config(**over: Any) -> ModelConfig:

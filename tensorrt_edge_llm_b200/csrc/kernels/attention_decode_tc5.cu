@@ -45,6 +45,10 @@ struct DecParams {
     int chunk;                      // chunked mask: a token sees only keys of its own `chunk`-token block (0 = none)
     int num_seqs, num_items;        // items = sequences x KV heads x splits, walked by persistent CTAs
     float scale_log2;
+    // rotated values: outputs turn back by their position (neighbouring features form the pairs) and are multiplied, or null
+    const float* back;              // [positions, D]: D / 2 cos | D / 2 sin
+    float back_mult;
+    long long ld_out;               // row pitch of out
     const float* sinks;             // [Hq] fp32 per-head sink logits (natural-log units), or null
     // FP8 (E4M3) cache pages read directly (KV8 kernels): kv_scales[0] multiplies the scores (K dequantisation scale),
     // kv_scales[1] the output (V scale); probabilities enter the P·V product as E4M3 of 256 x p.
@@ -548,7 +552,13 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
                             if ((lane & 7) == 0) *reinterpret_cast<uint32_t*>(p.oq + tok * (size_t)(p.hq * D / 2) + col / 2) = w4;
                             if ((lane & 15) == 0) p.osf[sf_atom_offset((long long)tok, col >> 4, p.ok64)] = s8;
                         } else if (p.splits == 1) {
-                            reinterpret_cast<T*>(p.out)[(tok * p.hq + head) * D + r] = Cvt<T>::from_f(val);
+                            float y = val;
+                            if (p.back) {                   // the pair's other half sits on the next lane
+                                const float other = __shfl_xor_sync(0xffffffffu, val, 1);
+                                const float* cs = p.back + (size_t)(it.past + qi) * D + r / 2;
+                                y = (val * cs[0] + ((r & 1) ? -other : other) * cs[D / 2]) * p.back_mult;
+                            }
+                            reinterpret_cast<T*>(p.out)[tok * p.ld_out + head * D + r] = Cvt<T>::from_f(y);
                         } else {
                             p.ws_o[(((size_t)it.split * p.total_tokens + tok) * p.hq + head) * D + r] = val;
                             if (r == 0) p.ws_lse[((size_t)it.split * p.total_tokens + tok) * p.hq + head] = lse;
@@ -623,6 +633,8 @@ extern "C" int telb_attn_combine(const float* ws_o, const float* ws_lse, void* o
                                  cudaStream_t stream);
 extern "C" int telb_attn_combine_quant(const float* ws_o, const float* ws_lse, void* oq, void* osf, const float* ogs, int tokens, int hq,
                                        int splits, int d, int is_bf16, cudaStream_t stream);
+extern "C" int telb_attn_combine_back(const float* ws_o, const float* ws_lse, void* out, int tokens, int hq, int splits, int d, const float* back,
+                                      float mult, const int* positions, long long ld_out, int is_bf16, cudaStream_t stream);
 extern "C" int telb_nvfp4_k64_pad(int k);
 
 // Ring depth / residency variant of the decode kernel (0, 1 or 2: see launch_decode); process-wide.
@@ -637,7 +649,8 @@ extern "C" int telb_paged_attention_decode_traced(const void* q, const void* kv_
                                                   int total_tokens, int max_q_len, int num_pages, int max_pages, int page_size,
                                                   int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                                                   long long ws_floats, int is_bf16, int* status, unsigned long long* trace,
-                                                  const float* sinks, int chunk, int split_p, cudaStream_t stream);
+                                                  const float* sinks, int chunk, int split_p, const float* back, float back_mult,
+                                                  const int* positions, long long ld_out, cudaStream_t stream);
 
 // Decode-shaped steps only: max_q_len * (Hq/Hkv) <= 16.  Same tensors as telb_paged_attention.
 extern "C" int telb_paged_attention_decode(const void* q, const void* kv_layer, void* out, const int* q_start,
@@ -647,14 +660,14 @@ extern "C" int telb_paged_attention_decode(const void* q, const void* kv_layer, 
                                            long long ws_floats, int is_bf16, int* status, cudaStream_t stream) {
     return telb_paged_attention_decode_traced(q, kv_layer, out, q_start, q_len, past_len, page_table, num_seqs, total_tokens, max_q_len,
                                               num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16,
-                                              status, nullptr, nullptr, 0, 0, stream);
+                                              status, nullptr, nullptr, 0, 0, nullptr, 1.f, nullptr, (long long)hq * d, stream);
 }
 
 static int decode_impl(const void* q, const void* kv_layer, void* out, void* oq, void* osf, const float* ogs, const int* q_start,
                        const int* q_len, const int* past_len, const int* page_table, int num_seqs, int total_tokens, int max_q_len,
                        int num_pages, int max_pages, int page_size, int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                        long long ws_floats, int is_bf16, int* status, unsigned long long* trace, const float* sinks, const float* kv_scales,
-                       int chunk, int split_p, cudaStream_t stream);
+                       int chunk, int split_p, const float* back, float back_mult, const int* positions, long long ld_out, cudaStream_t stream);
 
 // Same call with a timeline buffer (3 x 64 x 4 u64, zeroed by the caller) filled by the first CTA.
 extern "C" int telb_paged_attention_decode_traced(const void* q, const void* kv_layer, void* out, const int* q_start,
@@ -662,9 +675,11 @@ extern "C" int telb_paged_attention_decode_traced(const void* q, const void* kv_
                                                   int total_tokens, int max_q_len, int num_pages, int max_pages, int page_size,
                                                   int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                                                   long long ws_floats, int is_bf16, int* status, unsigned long long* trace,
-                                                  const float* sinks, int chunk, int split_p, cudaStream_t stream) {
+                                                  const float* sinks, int chunk, int split_p, const float* back, float back_mult,
+                                                  const int* positions, long long ld_out, cudaStream_t stream) {
     return decode_impl(q, kv_layer, out, nullptr, nullptr, nullptr, q_start, q_len, past_len, page_table, num_seqs, total_tokens, max_q_len,
-                       num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, trace, sinks, nullptr, chunk, split_p, stream);
+                       num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, trace, sinks, nullptr, chunk, split_p,
+                       back, back_mult, positions, ld_out, stream);
 }
 
 // Decode attention whose output is written as NVFP4 only (packed codes out_xq [T, Hq * D / 2], atom-layout scales out_sf over
@@ -677,7 +692,8 @@ extern "C" int telb_paged_attention_decode_quant(const void* q, const void* kv_l
                                                  int is_bf16, int* status, const float* sinks, cudaStream_t stream) {
     if (!out_xq || !out_sf || !out_global_scale) return fail("telb_paged_attention_decode_quant: output buffers and scale are required");
     return decode_impl(q, kv_layer, nullptr, out_xq, out_sf, out_global_scale, q_start, q_len, past_len, page_table, num_seqs, total_tokens,
-                       max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, nullptr, sinks, nullptr, 0, 0, stream);
+                       max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, nullptr, sinks, nullptr, 0, 0, nullptr, 1.f, nullptr,
+                       (long long)hq * d, stream);
 }
 
 // Decode attention over FP8 (E4M3) cache pages read in place: `q8` is the query tensor cast to E4M3 [T, Hq, D], `kv_layer` the
@@ -694,14 +710,14 @@ extern "C" int telb_paged_attention_decode_fp8(const void* q8, const void* kv_la
     if (out_xq && (!out_sf || !out_global_scale)) return fail("telb_paged_attention_decode_fp8: NVFP4 output needs its scale buffers");
     return decode_impl(q8, kv_layer, out, out_xq, out_sf, out_global_scale, q_start, q_len, past_len, page_table, num_seqs, total_tokens,
                        max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits, ws, ws_floats, is_bf16, status, nullptr,
-                       sinks, kv_scales, 0, 0, stream);
+                       sinks, kv_scales, 0, 0, nullptr, 1.f, nullptr, (long long)hq * d, stream);
 }
 
 static int decode_impl(const void* q, const void* kv_layer, void* out, void* oq, void* osf, const float* ogs, const int* q_start,
                        const int* q_len, const int* past_len, const int* page_table, int num_seqs, int total_tokens, int max_q_len,
                        int num_pages, int max_pages, int page_size, int hq, int hkv, int d, float scale, int window, int splits, float* ws,
                        long long ws_floats, int is_bf16, int* status, unsigned long long* trace, const float* sinks, const float* kv_scales,
-                       int chunk, int split_p, cudaStream_t stream) {
+                       int chunk, int split_p, const float* back, float back_mult, const int* positions, long long ld_out, cudaStream_t stream) {
     if (num_seqs <= 0 || total_tokens <= 0) return 0;
     if (d != 128) return fail("telb_paged_attention_decode: head_dim must be 128");
     if (page_size != 64 && page_size != 128) return fail("telb_paged_attention_decode: page size must be 64 or 128");
@@ -715,6 +731,11 @@ static int decode_impl(const void* q, const void* kv_layer, void* out, void* oq,
     p.osf = static_cast<uint8_t*>(osf);
     p.ogs = ogs;
     p.ok64 = telb_nvfp4_k64_pad(hq * d);
+    if (back && !positions) return fail("telb_paged_attention_decode: rotated values need the positions of the rows");
+    if (!back && ld_out != (long long)hq * d) return fail("telb_paged_attention_decode: rows further apart are built for rotated values");
+    p.back = back;
+    p.back_mult = back_mult;
+    p.ld_out = ld_out;
     p.sinks = sinks;
     p.kv_scales = kv_scales;
     p.q_start = q_start;
@@ -766,6 +787,8 @@ static int decode_impl(const void* q, const void* kv_layer, void* out, void* oq,
         rc = is_bf16 ? launch_decode<128, __nv_bfloat16>(tq, tkv, p, num_seqs, max_q_len * group, stream)
                      : launch_decode<128, __half>(tq, tkv, p, num_seqs, max_q_len * group, stream);
     if (rc) return rc;
+    if (splits > 1 && back)
+        return telb_attn_combine_back(p.ws_o, p.ws_lse, out, total_tokens, hq, splits, d, back, back_mult, positions, ld_out, is_bf16, stream);
     if (splits > 1 && oq) return telb_attn_combine_quant(p.ws_o, p.ws_lse, oq, osf, ogs, total_tokens, hq, splits, d, is_bf16, stream);
     if (splits > 1) return telb_attn_combine(p.ws_o, p.ws_lse, out, total_tokens * hq, splits, d, is_bf16, stream);
     return 0;

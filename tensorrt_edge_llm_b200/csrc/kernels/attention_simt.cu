@@ -23,6 +23,9 @@ struct SimtAttnParams {
     int dv, planes;              // value features; 2 = key and value planes, 1 = values are the first dv features of the keys
     float scale;
     const float* sinks;
+    const float* back;           // [positions, d] cos | sin: outputs turn back by their position, pairs of neighbours; or null
+    float mult;                  // factor of the outputs, with back
+    long long ld_out;            // row pitch of out
 };
 
 template <typename T, int E>                             // E: value features per lane, dv <= 32 E
@@ -87,10 +90,20 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(const __grid_constant__ 
         }
     }
     const float inv = l > 0.f ? 1.f / l : 0.f;
-    T* out = reinterpret_cast<T*>(p.out) + ((size_t)t * p.hq + h) * p.dv;
+    T* out = reinterpret_cast<T*>(p.out) + (size_t)t * p.ld_out + (size_t)h * p.dv;
 #pragma unroll
-    for (int e = 0; e < E; ++e)
-        if (e * 32 + lane < p.dv) out[e * 32 + lane] = Cvt<T>::from_f(acc[e] * inv);
+    for (int e = 0; e < E; ++e) {
+        const int c = e * 32 + lane;
+        float o = acc[e] * inv;
+        if (p.back) {                                        // uniform: the pair's other half sits on the next lane
+            const float other = __shfl_xor_sync(0xffffffffu, o, 1);
+            if (c < p.dv) {
+                const float* cs = p.back + (size_t)pos * p.dv + c / 2;
+                o = (o * cs[0] + ((lane & 1) ? -other : other) * cs[p.dv / 2]) * p.mult;
+            }
+        }
+        if (c < p.dv) out[c] = Cvt<T>::from_f(o);
+    }
 }
 
 template <typename T>
@@ -115,11 +128,12 @@ using namespace telb;
 
 extern "C" int telb_paged_attention_simt(const void* q, const void* kv_layer, void* out, const int* q_start, const int* past_len, const int* seq_ids,
                                          const int* page_table, int total_tokens, int max_pages, int page_size, int hq, int hkv, int d, float scale,
-                                         int window, int chunk, const float* sinks, int dtype, cudaStream_t stream) {
+                                         int window, int chunk, const float* sinks, const float* back, float mult, long long ld_out, int dtype,
+                                         cudaStream_t stream) {
     if (total_tokens <= 0) return 0;
     if (d > 1024) return fail("telb_paged_attention_simt: head_dim must be at most 1024");
     if (hkv <= 0 || hq % hkv) return fail("telb_paged_attention_simt: Hq must be a multiple of Hkv");
-    SimtAttnParams p{q, kv_layer, out, q_start, past_len, seq_ids, page_table, total_tokens, max_pages, page_size, hq, hkv, d, window, chunk, d, 2, scale, sinks};
+    SimtAttnParams p{q, kv_layer, out, q_start, past_len, seq_ids, page_table, total_tokens, max_pages, page_size, hq, hkv, d, window, chunk, d, 2, scale, sinks, back, mult, ld_out};
     if (dtype == 2) return launch_simt<float>(p, stream);
     return dtype == 1 ? launch_simt<__nv_bfloat16>(p, stream) : launch_simt<__half>(p, stream);
 }
@@ -130,7 +144,7 @@ extern "C" int telb_latent_attention_simt(const void* q, const void* kv_layer, v
                                           int dtype, cudaStream_t stream) {
     if (total_tokens <= 0) return 0;
     if (dv > 1024 || dv > row || row > 2048) return fail("telb_latent_attention_simt: at most 1024 latent features");
-    SimtAttnParams p{q, kv_layer, out, q_start, past_len, seq_ids, page_table, total_tokens, max_pages, page_size, hq, 1, row, 0, 0, dv, 1, scale, nullptr};
+    SimtAttnParams p{q, kv_layer, out, q_start, past_len, seq_ids, page_table, total_tokens, max_pages, page_size, hq, 1, row, 0, 0, dv, 1, scale, nullptr, nullptr, 1.f, (long long)hq * dv};
     if (dtype == 2) return launch_simt<float>(p, stream);
     return dtype == 1 ? launch_simt<__nv_bfloat16>(p, stream) : launch_simt<__half>(p, stream);
 }

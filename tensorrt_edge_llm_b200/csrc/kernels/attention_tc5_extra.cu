@@ -37,6 +37,11 @@ struct AttnParams {
     // A KV tile whose largest score lies more than that below the running maximum for every query row of a warp is not
     // exponentiated (its P rows are zeros); when all four warps vote so, the tile's P·V products are not issued either.
     const float* skip_thr;
+    // Rotated values: outputs turn back by their position (neighbouring features form the pairs) and are multiplied, or null
+    const float* back;         // [positions, D]: D / 2 cos | D / 2 sin
+    float back_mult;
+    const int* positions;      // [T], for the split merge
+    long long ld_out;          // row pitch of out
     int* skip_stats;           // optional [2]: tiles processed, tiles whose P·V was skipped (diagnostics / tests), or null
     int out_bf16;
     int* status;
@@ -127,6 +132,45 @@ __global__ void attn_combine_quant_kernel(const float* __restrict__ ws_o, const 
     if ((d & 15) == 0) osf[sf_atom_offset((long long)tok, col >> 4, k64)] = s8;
 }
 
+// The merge of outputs that turn back by their position; rows of out may lie further apart than their heads.
+template <int D, typename T>
+__global__ void attn_combine_back_kernel(const float* __restrict__ ws_o, const float* __restrict__ ws_lse, T* __restrict__ out, int total_rows /* T*Hq */,
+                                         int hq, int splits, const float* __restrict__ back, float mult, const int* __restrict__ positions,
+                                         long long ld_out) {
+    pdl_prologue();
+    __shared__ float w[32];
+    const int row = blockIdx.x, d = threadIdx.x;
+    if (d < 32) {
+        const float l = d < splits ? ws_lse[(size_t)d * total_rows + row] : -INFINITY;
+        float mx = l;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float e = l == -INFINITY ? 0.f : exp2f(l - mx);
+        float den = e;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
+        w[d] = den > 0.f ? e / den : 0.f;
+    }
+    const int tok = row / hq, head = row - tok * hq;
+    const float* cs = back + (size_t)positions[tok] * D + d / 2;
+    const float c = cs[0], s = (d & 1) ? -cs[D / 2] : cs[D / 2];
+    __syncthreads();
+    float acc = 0.f;
+#pragma unroll 8
+    for (int i = 0; i < splits; ++i) acc += w[i] * __ldcg(&ws_o[((size_t)i * total_rows + row) * D + d]);
+    const float other = __shfl_xor_sync(0xffffffffu, acc, 1);
+    out[(size_t)tok * ld_out + head * D + d] = Cvt<T>::from_f((acc * c + other * s) * mult);
+}
+
+template <int D, typename T>
+static int launch_combine_back(const float* ws_o, const float* ws_lse, void* out, int tokens, int hq, int splits, const float* back, float mult,
+                               const int* positions, long long ld_out, cudaStream_t stream) {
+    TELB_LAUNCH("attn_combine_back_kernel", (attn_combine_back_kernel<D, T>), dim3(tokens * hq), dim3(D), 0, stream, ws_o, ws_lse, (T*)out, tokens * hq, hq, splits,
+                back, mult, positions, ld_out);
+    TELB_CHECK_LAUNCH("attn_combine_back_kernel");
+    return 0;
+}
+
 template <int D, typename T, int KVS, int MINB>
 static int launch_attn_extra(const CUtensorMap& tq, const CUtensorMap& tkv, const AttnParams& p, int qtiles, int nseq, cudaStream_t stream) {
     constexpr int smem = 128 * D * 2 + 2 * KVS * kKvTile * D * 2 + 2 * 128 * kKvTile * 2 + 1024 + 512;
@@ -139,6 +183,8 @@ static int launch_attn_extra(const CUtensorMap& tq, const CUtensorMap& tkv, cons
     dim3 grid(qtiles, p.hkv, nseq * p.splits);
     TELB_LAUNCH("attn_tc5_extra_kernel", (attn_tc5_extra_kernel<D, T, KVS, MINB>), dim3(grid), dim3(kAttnThreads), smem, stream, tq, tkv, p);
     TELB_CHECK_LAUNCH("attn_tc5_extra_kernel");
+    if (p.splits > 1 && p.back)
+        return launch_combine_back<D, T>(p.ws_o, p.ws_lse, p.out, p.total_tokens, p.hq, p.splits, p.back, p.back_mult, p.positions, p.ld_out, stream);
     if (p.splits > 1) {
         const int rows = p.total_tokens * p.hq;
         TELB_LAUNCH("attn_combine_kernel", (attn_combine_kernel<D, T>), dim3(rows), dim3(D), 0, stream, p.ws_o, p.ws_lse, reinterpret_cast<T*>(p.out), rows, p.splits);
@@ -178,6 +224,14 @@ extern "C" int telb_attn_combine(const float* ws_o, const float* ws_lse, void* o
     return 0;
 }
 
+extern "C" int telb_attn_combine_back(const float* ws_o, const float* ws_lse, void* out, int tokens, int hq, int splits, int d, const float* back,
+                                      float mult, const int* positions, long long ld_out, int is_bf16, cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (d != 128 || splits > 32) return fail("telb_attn_combine_back: heads of 128 and at most 32 splits");
+    if (is_bf16) return launch_combine_back<128, __nv_bfloat16>(ws_o, ws_lse, out, tokens, hq, splits, back, mult, positions, ld_out, stream);
+    return launch_combine_back<128, __half>(ws_o, ws_lse, out, tokens, hq, splits, back, mult, positions, ld_out, stream);
+}
+
 extern "C" int telb_nvfp4_k64_pad(int k);
 
 // The merge with an NVFP4 result: packed codes oq [tokens, hq * d / 2] and atom-layout scales osf over hq * d columns.
@@ -201,10 +255,13 @@ extern "C" int telb_paged_attention(const void* q, const void* kv_layer, void* o
                                     const int* tree_mask, int mask_words, int num_seqs, int total_tokens,
                                     int max_q_len, int num_pages, int max_pages, int page_size, int hq, int hkv, int d,
                                     float scale, int window, int splits, float* ws, long long ws_floats, int is_bf16,
-                                    int* status, const float* sinks, const float* skip_thr, int* skip_stats, int chunk, int split_p, cudaStream_t stream) {
+                                    int* status, const float* sinks, const float* skip_thr, int* skip_stats, int chunk, int split_p,
+                                    const float* back, float back_mult, const int* positions, long long ld_out, cudaStream_t stream) {
     if (num_seqs <= 0 || total_tokens <= 0) return 0;
     const int group = hkv > 0 ? hq / hkv : 0;
-    if (sinks == nullptr && skip_thr == nullptr && chunk <= 0 && !split_p && d != 256 && group > 0 && 128 % group == 0)
+    if (!back && ld_out != (long long)hq * d) return fail("telb_paged_attention: rows further apart are built for rotated values");
+    if (back && !positions) return fail("telb_paged_attention: rotated values need the positions of the rows");
+    if (sinks == nullptr && skip_thr == nullptr && chunk <= 0 && !split_p && !back && d != 256 && group > 0 && 128 % group == 0)
         return telb_paged_attention_dense(q, kv_layer, out, q_start, q_len, past_len, page_table, tree_mask, mask_words, num_seqs,
                                           total_tokens, max_q_len, num_pages, max_pages, page_size, hq, hkv, d, scale, window, splits,
                                           ws, ws_floats, is_bf16, status, stream);
@@ -235,6 +292,10 @@ extern "C" int telb_paged_attention(const void* q, const void* kv_layer, void* o
     p.sinks = sinks;
     p.skip_thr = skip_thr;
     p.skip_stats = skip_stats;
+    p.back = back;
+    p.back_mult = back_mult;
+    p.positions = positions;
+    p.ld_out = ld_out;
     p.status = status;
     if (splits < 1) splits = 1;
     while (splits > 1 && (long long)splits * total_tokens * hq * (d + 1) > ws_floats) --splits;

@@ -1,9 +1,9 @@
-// Delta-rule mixer with one decay per head and key channel, over the packed ragged step.  Per head (S: keys x values, fp32):
+// Delta-rule mixer with one decay per head and key channel (or one per head), over the packed ragged step.  Per head (S: keys x values, fp32):
 //
 //   q, k, v <- silu(short causal convolution)            q, k <- x / sqrt(sum x² + 1e-6), q also times dim^-1/2
 //   g = exp(-exp(a_log) · softplus(decay + bias))        beta = sigmoid(beta)
 //   S <- diag(g) S;  u = beta (v - Sᵀ k);  S <- S + k uᵀ;  o = Sᵀ q
-//   y = o / rms(o) · w · sigmoid(gate)
+//   y = o / rms(o) · w · sigmoid(gate)                   (or silu(gate))
 //
 // Prompt portions run as five launches: `prep` twice (values; q, k and decays: convolutions and norms, parallel over tokens), `walk` (the
 // recurrence, state in registers), `out` (head norm and gate) and `roll` (convolution history).  A step with one row per sequence runs
@@ -28,10 +28,10 @@ namespace telb {
 
 // Host mirror: ops/cuda.py (ChannelDeltaParams).
 struct ChannelDeltaParams {
-    const void* qkv;           // [T, channels] projections: q [kv_heads * dk] | k [kv_heads * dk] | v [heads * dv]
-    const float* decay;        // [T, ld_decay] pre-activations [heads * dk]
+    const void* qkv;           // [T, ld_qkv] projections: q [kv_heads * dk] | k [kv_heads * dk] | v [heads * dv]
+    const float* decay;        // [T, ld_decay] pre-activations [heads * dk] (head_decay: [heads])
     const void* gate;          // [T, ld_gate] pre-activations [heads * dv], fp32 when gate_f32
-    const float* beta;         // [T, heads] pre-activations
+    const float* beta;         // [T, ld_beta] pre-activations [heads]
     const void* conv_w;        // [channels, taps]
     const float* a_log;        // [heads]
     const float* decay_bias;   // [heads * dk]
@@ -41,7 +41,7 @@ struct ChannelDeltaParams {
     float* blocks;             // [blocks, heads, 13 dk + 32] scratch: per block of four tokens the vectors and scalars of the walk
     void* v_blocks;            // [blocks, heads, dv, 4] scratch: convolved values
     void* o;                   // [T, heads * dv] scratch: read-outs
-    void* out;                 // [T, heads * dv]
+    void* out;                 // [T, ld_out]: heads * dv
     const int* q_start;
     const int* q_len;
     const int* past_len;
@@ -49,7 +49,8 @@ struct ChannelDeltaParams {
     const int* seq_ids;
     int* status;
     int tokens, num_seqs, heads, kv_heads, dk, dv, dk_real, dv_real, taps, channels, ld_decay, ld_gate, gate_f32;
-    float eps;
+    int ld_qkv, ld_beta, ld_out, head_decay, gate_silu;      // head_decay: decay [T, heads] and decay_bias [heads]; gate_silu: silu instead of a sigmoid
+    float eps, mult;             // mult: factor of the outputs
 };
 
 constexpr float kUnitEps = 1e-6f;
@@ -151,7 +152,7 @@ __device__ __forceinline__ void conv_block(const ChannelDeltaParams& p, const fl
     float rows[W - 1 + kBlk][C];
     if (n == kBlk && i >= W - 1) {                        // inside the portion
 #pragma unroll
-        for (int j = 0; j < W - 1 + kBlk; ++j) load_n<T, C>(x + (t + j - (W - 1)) * p.channels, rows[j]);
+        for (int j = 0; j < W - 1 + kBlk; ++j) load_n<T, C>(x + (t + j - (W - 1)) * p.ld_qkv, rows[j]);
     } else {
 #pragma unroll
         for (int j = 0; j < W - 1 + kBlk; ++j) {
@@ -159,7 +160,7 @@ __device__ __forceinline__ void conv_block(const ChannelDeltaParams& p, const fl
 #pragma unroll
             for (int c = 0; c < C; ++c) rows[j][c] = 0.f;
             if (d < n && i + d >= 0 && d >= -hist) {
-                load_n<T, C>(x + (t + d) * p.channels, rows[j]);
+                load_n<T, C>(x + (t + d) * p.ld_qkv, rows[j]);
             } else if (d < 0 && d >= -hist && history) {
 #pragma unroll
                 for (int c = 0; c < C; ++c) rows[j][c] = Cvt<T>::to_f(history[(size_t)(ch + c) * hist + hist + i + d]);
@@ -199,8 +200,16 @@ __device__ __forceinline__ void prep_head(const ChannelDeltaParams& p, const flo
     const int lane = threadIdx.x & 31, dk = p.dk, hk = h / (p.heads / p.kv_heads);
     float q[kBlk][C], k[kBlk][C], g[kBlk][C];
 #pragma unroll
-    for (int b = 0; b < kBlk; ++b)
-        if (b < n) load_n<float, C>(p.decay + (t + b) * p.ld_decay + h * dk + lane * C, g[b]);
+    for (int b = 0; b < kBlk; ++b) {
+        if (b >= n) continue;
+        if (p.head_decay) {
+            const float z = p.decay[(t + b) * p.ld_decay + h];
+#pragma unroll
+            for (int c = 0; c < C; ++c) g[b][c] = z;
+        } else {
+            load_n<float, C>(p.decay + (t + b) * p.ld_decay + h * dk + lane * C, g[b]);
+        }
+    }
     conv_block<T, C, W>(p, wq, hk * dk + lane * C, t, i, n, history, q);
     conv_block<T, C, W>(p, wk, (p.kv_heads + hk) * dk + lane * C, t, i, n, history, k);
 #pragma unroll
@@ -246,7 +255,7 @@ __device__ __forceinline__ void prep_head(const ChannelDeltaParams& p, const flo
             if (lane == 6 + x * (x + 1) / 2 + j) f = rq[x] * rk[j];
         }
     total *= f;
-    if (lane >= 16) total = lane < 16 + n ? cd_sigmoid(p.beta[(t + lane - 16) * p.heads + h]) : 0.f;
+    if (lane >= 16) total = lane < 16 + n ? cd_sigmoid(p.beta[(t + lane - 16) * p.ld_beta + h]) : 0.f;
     out[13 * dk + lane] = total;
     float d[C];
 #pragma unroll
@@ -307,7 +316,12 @@ __device__ void prep_range(const ChannelDeltaParams& p, int h, int t0, int t1) {
     } else {
         load_taps<T, C, W>(p, hk * p.dk + lane * C, w0);
         load_taps<T, C, W>(p, (p.kv_heads + hk) * p.dk + lane * C, w1);
-        load_n<float, C>(p.decay_bias + h * p.dk + lane * C, bias);
+        if (p.head_decay) {
+#pragma unroll
+            for (int c = 0; c < C; ++c) bias[c] = p.decay_bias[h];
+        } else {
+            load_n<float, C>(p.decay_bias + h * p.dk + lane * C, bias);
+        }
         rate = -expf(p.a_log[h]);
     }
     for (int t = t0; t < t1;) {
@@ -339,12 +353,12 @@ __global__ void __launch_bounds__(128) channel_delta_roll_kernel(const __grid_co
     const int seq = blockIdx.y, ch = blockIdx.x * 128 + threadIdx.x;
     const int ql = p.q_len[seq], hist = p.taps - 1;
     if (ch >= p.channels || ql <= 0) return;
-    const T* x = reinterpret_cast<const T*>(p.qkv) + (size_t)p.q_start[seq] * p.channels + ch;
+    const T* x = reinterpret_cast<const T*>(p.qkv) + (size_t)p.q_start[seq] * p.ld_qkv + ch;
     T* cs = reinterpret_cast<T*>(p.conv_state) + ((size_t)p.slot_ids[seq] * p.channels + ch) * hist;
     const bool fresh = p.past_len[seq] == 0;
     for (int j = 0; j < hist; ++j) {                      // ascending: an old value is read before its place is written
         const int r = ql - hist + j;
-        cs[j] = r >= 0 ? x[(size_t)r * p.channels] : (fresh ? Cvt<T>::from_f(0.f) : cs[j + ql]);
+        cs[j] = r >= 0 ? x[(size_t)r * p.ld_qkv] : (fresh ? Cvt<T>::from_f(0.f) : cs[j + ql]);
     }
 }
 
@@ -736,8 +750,11 @@ __device__ void delta_out(const ChannelDeltaParams& p, size_t t, int h) {
     const float inv = 1.f / sqrtf(cd_warp_sum(ss) / p.dv_real + p.eps);
     T y[C];
 #pragma unroll
-    for (int c = 0; c < C; ++c) y[c] = Cvt<T>::from_f(o[c] * inv * w[c] * (sizeof(T) == 4 ? cd_sigmoid(z[c]) : __fdividef(1.f, 1.f + __expf(-z[c]))));
-    store_n<T, C>(reinterpret_cast<T*>(p.out) + t * p.heads * p.dv + col, y);
+    for (int c = 0; c < C; ++c) {
+        const float s = sizeof(T) == 4 ? cd_sigmoid(z[c]) : __fdividef(1.f, 1.f + __expf(-z[c]));
+        y[c] = Cvt<T>::from_f(o[c] * inv * w[c] * (p.gate_silu ? s * z[c] : s) * p.mult);
+    }
+    store_n<T, C>(reinterpret_cast<T*>(p.out) + t * p.ld_out + col, y);
 }
 
 template <typename T>
@@ -775,7 +792,7 @@ __global__ void __launch_bounds__(256) channel_delta_decode_kernel(const __grid_
 #pragma unroll
             for (int c = 0; c < C; ++c) S[r][c] = 0.f;
     }
-    const T* x = reinterpret_cast<const T*>(p.qkv) + t * p.channels;
+    const T* x = reinterpret_cast<const T*>(p.qkv) + t * p.ld_qkv;
     for (int i = tid; i < 2 * DK + DV; i += 256) {
         const int ch = i < DK ? hk * DK + i : i < 2 * DK ? p.kv_heads * DK + hk * DK + i - DK : 2 * p.kv_heads * DK + h * DV + i - 2 * DK;
         T* cs = reinterpret_cast<T*>(p.conv_state) + (slot * p.channels + ch) * hist;
@@ -791,8 +808,11 @@ __global__ void __launch_bounds__(256) channel_delta_decode_kernel(const __grid_
         }
         (i < DK ? s_q[i] : i < 2 * DK ? s_k[i - DK] : s_v[i - 2 * DK]) = y;
     }
-    const float rate = -expf(p.a_log[h]), beta = cd_sigmoid(p.beta[t * p.heads + h]);
-    for (int i = tid; i < DK; i += 256) s_g[i] = cd_decay_as<T>(rate, p.decay[t * p.ld_decay + h * DK + i] + p.decay_bias[h * DK + i]);
+    const float rate = -expf(p.a_log[h]), beta = cd_sigmoid(p.beta[t * p.ld_beta + h]);
+    for (int i = tid; i < DK; i += 256) {
+        const int at = p.head_decay ? h : h * DK + i;
+        s_g[i] = cd_decay_as<T>(rate, p.decay[t * p.ld_decay + at] + p.decay_bias[at]);
+    }
     __syncthreads();
     float qq = 0.f, kk = 0.f, qk = 0.f;                                 // every warp: |q|², |k|², q·k
     for (int i = lane; i < DK; i += 32) {
@@ -857,7 +877,7 @@ __global__ void __launch_bounds__(256) channel_delta_decode_kernel(const __grid_
         const float inv = 1.f / sqrtf(tot / p.dv_real + p.eps);
         const size_t gi = t * p.ld_gate + h * DV + tid;
         const float z = p.gate_f32 ? reinterpret_cast<const float*>(p.gate)[gi] : Cvt<T>::to_f(reinterpret_cast<const T*>(p.gate)[gi]);
-        reinterpret_cast<T*>(p.out)[(t * p.heads + h) * DV + tid] = Cvt<T>::from_f(o * inv * p.norm_w[tid] * cd_sigmoid(z));
+        reinterpret_cast<T*>(p.out)[t * p.ld_out + h * DV + tid] = Cvt<T>::from_f(o * inv * p.norm_w[tid] * cd_sigmoid(z) * (p.gate_silu ? z : 1.f) * p.mult);
     }
 }
 
@@ -996,6 +1016,7 @@ extern "C" int telb_channel_delta(const ChannelDeltaParams* pp, int decode, int 
     if (!size_ok(p.dk) || !size_ok(p.dv)) return fail("telb_channel_delta: padded head sizes are 32, 64, 128 or 256");
     if (p.taps < 1 || p.taps > 8) return fail("telb_channel_delta: convolutions have 1 to 8 taps");
     if (p.kv_heads <= 0 || p.heads % p.kv_heads) return fail("telb_channel_delta: heads must be a multiple of the q / k heads");
+    if (p.ld_qkv % 8 || p.ld_out % 8) return fail("telb_channel_delta: row pitches are multiples of 8");
     if (p.num_seqs > 65535 || p.heads > 65535) return fail("telb_channel_delta: too many sequences or heads");
     if (decode) {
         if (p.dk > 128 || p.dv > 128) return fail("telb_channel_delta: the decode step covers heads up to 128");

@@ -180,9 +180,9 @@ __global__ void swiglu_kernel(const T* __restrict__ in, T* __restrict__ out, lon
     }
 }
 
-// out[t, i] = gelu(in[t, i]) * in[t, inter + i]   (tanh form or exact erf form)
+// out[t, i] = act(in[t, i]) * in[t, inter + i]; kind: 0 gelu (exact erf form), 1 gelu (tanh form), 2 relu
 template <typename T>
-__global__ void geglu_kernel(const T* __restrict__ in, T* __restrict__ out, long long rows, int inter, int tanh_approx) {
+__global__ void geglu_kernel(const T* __restrict__ in, T* __restrict__ out, long long rows, int inter, int kind) {
     pdl_prologue();
     const long long nvec = rows * (inter / 8);
     for (long long idx = blockIdx.x * (long long)blockDim.x + threadIdx.x; idx < nvec;
@@ -195,7 +195,8 @@ __global__ void geglu_kernel(const T* __restrict__ in, T* __restrict__ out, long
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
             const float x = g.get(j);
-            const float act = tanh_approx ? 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)))
+            const float act = kind == 2   ? fmaxf(x, 0.f)
+                              : kind == 1 ? 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)))
                                           : 0.5f * x * (1.f + erff(x * 0.7071067811865476f));
             o.set(j, act * u.get(j));
         }
@@ -708,13 +709,14 @@ extern "C" int telb_swiglu(const void* in, void* out, long long rows, int inter,
     return 0;
 }
 
-extern "C" int telb_geglu(const void* in, void* out, long long rows, int inter, int tanh_approx, int is_bf16, cudaStream_t stream) {
+// kind: 0 gelu (erf), 1 gelu (tanh form), 2 relu
+extern "C" int telb_geglu(const void* in, void* out, long long rows, int inter, int kind, int is_bf16, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (inter % 8) return fail("telb_geglu: intermediate size must be a multiple of 8");
     const long long nvec = rows * (inter / 8);
     long long blocks = (nvec + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
-    DISPATCH_T(is_bf16, { TELB_LAUNCH("geglu_kernel", (geglu_kernel<T>), dim3((int)blocks), dim3(256), 0, stream, (const T*)in, (T*)out, rows, inter, tanh_approx); })
+    DISPATCH_T(is_bf16, { TELB_LAUNCH("geglu_kernel", (geglu_kernel<T>), dim3((int)blocks), dim3(256), 0, stream, (const T*)in, (T*)out, rows, inter, kind); })
     TELB_CHECK_LAUNCH("geglu_kernel");
     return 0;
 }

@@ -66,26 +66,43 @@ gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, float*
     }
 }
 
-// out[t, i] = gelu(in[t, i]) * in[t, inter + i], tanh form, for the models whose products above feed it.
-__global__ void __launch_bounds__(256) geglu_f32_kernel(const float* __restrict__ in, float* __restrict__ out, long long rows, int inter) {
+// out[t, i] = act(in[t, i]) * in[t, inter + i] for the models whose products above feed it; act: gelu in tanh form, or relu.
+__global__ void __launch_bounds__(256) glu_f32_kernel(const float* __restrict__ in, float* __restrict__ out, long long rows, int inter, int relu) {
     pdl_prologue();
     const long long n = rows * inter;
     for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
         const long long r = i / inter;
         const float x = in[r * 2 * inter + i - r * inter], u = in[r * 2 * inter + inter + i - r * inter];
-        out[i] = 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x))) * u;
+        out[i] = (relu ? fmaxf(x, 0.f) : 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)))) * u;
     }
+}
+
+// Logit cap in place: x <- cap tanh(x / cap).
+__global__ void __launch_bounds__(256) softcap_kernel(float* x, long long n, float cap) {
+    pdl_prologue();
+    for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) x[i] = cap * tanhf(x[i] / cap);
+}
+
+static unsigned grid_for(long long n) {
+    const long long blocks = (n + 255) / 256;
+    return (unsigned)(blocks < 148 * 16 ? blocks : 148 * 16);
 }
 
 }  // namespace telb
 
 using namespace telb;
 
-extern "C" int telb_geglu_f32(const float* in, float* out, long long rows, int inter, cudaStream_t stream) {
+extern "C" int telb_glu_f32(const float* in, float* out, long long rows, int inter, int relu, cudaStream_t stream) {
     if (rows <= 0 || inter <= 0) return 0;
-    const long long blocks = (rows * inter + 255) / 256;
-    TELB_LAUNCH("geglu_f32_kernel", geglu_f32_kernel, dim3((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0, stream, in, out, rows, inter);
-    TELB_CHECK_LAUNCH("geglu_f32_kernel");
+    TELB_LAUNCH("glu_f32_kernel", glu_f32_kernel, dim3(grid_for(rows * inter)), dim3(256), 0, stream, in, out, rows, inter, relu);
+    TELB_CHECK_LAUNCH("glu_f32_kernel");
+    return 0;
+}
+
+extern "C" int telb_softcap(float* x, long long n, float cap, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    TELB_LAUNCH("softcap_kernel", softcap_kernel, dim3(grid_for(n)), dim3(256), 0, stream, x, n, cap);
+    TELB_CHECK_LAUNCH("softcap_kernel");
     return 0;
 }
 

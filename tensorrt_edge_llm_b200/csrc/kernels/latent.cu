@@ -2,6 +2,7 @@
 //
 //   latent_write     latent attention: RMS norm of the latent, interleaved rotation of the query and key parts, cache row
 //   unit_kv_write    queries and keys over their root mean square, query temperature, cache rows
+//   turned_kv_write  norms over whole query and key rows, interleaved rotation of queries, keys and values, cache rows
 //   head_linear      one small matrix per head, y[t,h] = W[h] x[t,h]: carries queries into latent space and results out of it
 //   latent_gather    cached latent rows of the step's sequences, back to back (input of the key / value expansion)
 //
@@ -97,6 +98,89 @@ latent_write_kernel(T* rows, T* kv, const float* cos_sin, const float* norm_w, c
         x.load(c + rank_pad + i);
         x.turn(cs, i / 2, half);
         x.store(dst + rank_pad + i);
+    }
+}
+
+// One CTA per row of packed q | k | v.  The norms divide by the real features of all heads together; every pair of a padded head turns
+// by its own row of the table (features that do not rotate have angle zero).
+struct TurnedKvParams {
+    const void* rows;            // [T, ld]
+    void* q_out;                 // [T, hq, d]
+    void* kv;                    // [pages, 2, hkv, P, d]
+    const float* key_table;      // [positions, d]: d / 2 cos | d / 2 sin
+    const float* value_table;
+    const float* q_norm;         // [hq * d]
+    const float* k_norm;         // [hkv * d]
+    const int* positions;
+    const int* seq_ids;
+    const int* q_start;
+    const int* past_len;
+    const int* page_table;
+    int ld, tokens, max_pages, page_size, hq, hkv, d, real;
+    float eps;
+};
+
+constexpr int kTurnThreads = 128;
+
+template <typename T>
+__global__ void __launch_bounds__(kTurnThreads) turned_kv_write_kernel(const __grid_constant__ TurnedKvParams p) {
+    pdl_prologue();
+    __shared__ float red[2][kTurnThreads / 32];
+    const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const T* src = reinterpret_cast<const T*>(p.rows) + (size_t)t * p.ld;
+    const int qn = p.hq * p.d, kn = p.hkv * p.d;
+    float ss[2] = {0.f, 0.f};
+    Eight<T> x;
+    for (int c = tid * 8; c < qn + kn; c += kTurnThreads * 8) {
+        x.load(src + c);
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const float v = Cvt<T>::to_f(x.e[i]);
+            s = fmaf(v, v, s);
+        }
+        ss[c < qn ? 0 : 1] += s;
+    }
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) ss[k] += __shfl_xor_sync(0xffffffffu, ss[k], o);
+        if (lane == 0) red[k][warp] = ss[k];
+    }
+    __syncthreads();
+    float inv[2];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        float s = 0.f;
+#pragma unroll
+        for (int w = 0; w < kTurnThreads / 32; ++w) s += red[k][w];
+        inv[k] = 1.f / sqrtf(s / ((k ? p.hkv : p.hq) * p.real) + p.eps);
+    }
+    const int seq = p.seq_ids[t], pos = p.positions[t], half = p.d / 2;
+    T* dst = cache_row(reinterpret_cast<T*>(p.kv), p.page_table, p.max_pages, p.page_size, seq, p.past_len[seq] + t - p.q_start[seq], 2 * p.hkv * p.page_size, p.d);
+    for (int c = tid * 8; c < qn + 2 * kn; c += kTurnThreads * 8) {
+        const int kind = c < qn ? 0 : c < qn + kn ? 1 : 2, f = c % p.d;
+        const float* cs = (kind == 2 ? p.value_table : p.key_table) + (size_t)pos * p.d + f / 2;
+        const float4 co4 = *reinterpret_cast<const float4*>(cs), si4 = *reinterpret_cast<const float4*>(cs + half);
+        const float co[4] = {co4.x, co4.y, co4.z, co4.w}, si[4] = {si4.x, si4.y, si4.z, si4.w};
+        x.load(src + c);
+        float v[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = Cvt<T>::to_f(x.e[i]);
+        if (kind < 2) {
+            const float* w = kind ? p.k_norm + c - qn : p.q_norm + c;
+            const float4 w0 = *reinterpret_cast<const float4*>(w), w1 = *reinterpret_cast<const float4*>(w + 4);
+            const float g[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] *= inv[kind] * g[i];
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            x.e[2 * i] = Cvt<T>::from_f(v[2 * i] * co[i] - v[2 * i + 1] * si[i]);
+            x.e[2 * i + 1] = Cvt<T>::from_f(v[2 * i + 1] * co[i] + v[2 * i] * si[i]);
+        }
+        if (kind == 0) x.store(reinterpret_cast<T*>(p.q_out) + (size_t)t * qn + c);
+        else if (dst) x.store(dst + (size_t)((c - qn) / p.d) * p.page_size * p.d + f);      // planes keys | values: heads count through both
     }
 }
 
@@ -417,5 +501,18 @@ extern "C" int telb_latent_gather(const void* kv_layer, void* latent, void* rot,
     TELB_LAUNCH("latent_gather_kernel", latent_gather_kernel, dim3(blocks, num_seqs), dim3(128), 0, stream, (const uint4*)kv_layer, (uint4*)latent, (uint4*)rot,
                 out_start, q_len, past_len, page_table, max_pages, page_size, rank_bytes / 16, rot_bytes / 16, min_q);
     TELB_CHECK_LAUNCH("latent_gather_kernel");
+    return 0;
+}
+
+// dtype: 0 fp16, 1 bf16, 2 fp32.  Heads are padded to multiples of 8, row pitches likewise.
+extern "C" int telb_turned_kv_write(const TurnedKvParams* pp, int dtype, cudaStream_t stream) {
+    const TurnedKvParams& p = *pp;
+    if (p.tokens <= 0) return 0;
+    if (p.d % 8 || p.ld % 8 || p.hq < 1 || p.hkv < 1) return fail("telb_turned_kv_write: head and row sizes are multiples of 8");
+    const dim3 grid(p.tokens), block(kTurnThreads);
+    if (dtype == 2) TELB_LAUNCH("turned_kv_write_kernel", (turned_kv_write_kernel<float>), grid, block, 0, stream, p);
+    else if (dtype == 1) TELB_LAUNCH("turned_kv_write_kernel", (turned_kv_write_kernel<__nv_bfloat16>), grid, block, 0, stream, p);
+    else TELB_LAUNCH("turned_kv_write_kernel", (turned_kv_write_kernel<__half>), grid, block, 0, stream, p);
+    TELB_CHECK_LAUNCH("turned_kv_write_kernel");
     return 0;
 }

@@ -199,6 +199,9 @@ LLMEngineConfig LLMEngineConfig::from_runtime_config(const Json& root) {
     if (specs.is_array() && !specs.items().empty()) {
         const auto& list = specs.items();
         const int n = static_cast<int>(list.size());
+        int input_taps = 0, bigram_buckets = 0;
+        i(m, "input_conv", input_taps);
+        i(m, "bigram_buckets", bigram_buckets);
         auto pad_head = [](int d) { return d <= 64 ? 64 : d <= 128 ? 128 : d <= 256 ? 256 : (d + 63) / 64 * 64; };
         auto add_run = [&](const Json& spec) {
             long long kv = 0, state = 0, window = 0;
@@ -209,19 +212,22 @@ LLMEngineConfig LLMEngineConfig::from_runtime_config(const Json& root) {
                 i(a, "num_kv_heads", heads);
                 i(a, "head_dim", k);
                 i(a, "v_head_dim", v);
-                kv = 2LL * heads * pad_head(std::max(k, v));
-            } else if (spec["mlstm"].is_object()) {
+                kv += 2LL * heads * pad_head(std::max(k, v));
+            }
+            if (spec["mlstm"].is_object()) {
                 const Json& a = spec["mlstm"];
                 i(a, "num_heads", heads);
                 i(a, "head_k_dim", k);
                 i(a, "head_v_dim", v);
                 k = pad_head(k);
-                state = 1LL * heads * (1LL * k * ((v + 127) / 128 * 128) + k + 1);
-            } else if (spec["latent"].is_object()) {
+                state += 1LL * heads * (1LL * k * ((v + 127) / 128 * 128) + k + 1);
+            }
+            if (spec["latent"].is_object()) {
                 i(spec["latent"], "rank", k);
                 i(spec["latent"], "rot_dim", v);
-                kv = pad64(k) + pad64(v);                                          // one row per token
-            } else if (spec["delta"].is_object()) {
+                kv += pad64(k) + pad64(v);                                         // one row per token
+            }
+            if (spec["delta"].is_object()) {
                 const Json& a = spec["delta"];
                 int kv_heads = 0, taps = 1;
                 i(a, "num_heads", heads);
@@ -231,9 +237,18 @@ LLMEngineConfig LLMEngineConfig::from_runtime_config(const Json& root) {
                 i(a, "conv_kernel", taps);
                 k = k <= 32 ? 32 : pad_head(k);
                 v = v <= 32 ? 32 : pad_head(v);
-                state = 1LL * heads * k * v;
-                window = (2LL * kv_heads * k + 1LL * heads * v) * (taps - 1);      // convolution history
+                state += 1LL * heads * k * v;
+                window += (2LL * kv_heads * k + 1LL * heads * v) * (taps - 1);     // convolution history
             }
+            if (spec["lightning"].is_object()) {
+                const Json& a = spec["lightning"];
+                i(a, "num_heads", heads);
+                i(a, "head_k_dim", k);
+                i(a, "head_v_dim", v);
+                state += 1LL * heads * pad_head(k) * ((v + 127) / 128 * 128);
+            }
+            if (input_taps > 1) state += 1LL * c.hidden_size * (input_taps - 1);   // fp32 rows in front of the mixer's input convolution
+            if (c.run_state_values.empty() && bigram_buckets > 0) state += 1;      // the sequence's last token
             c.run_kv_elements.push_back(kv);
             c.run_state_values.push_back(state);
             c.run_window_elements.push_back(window);
@@ -283,7 +298,7 @@ bool LLMEngineConfig::is_hybrid() const {
 
 int LLMEngineConfig::num_recurrent_layers() const {
     int n = 0;
-    for (const auto& t : layer_types) n += (t == "mamba" || t == "gdn" || t == "mlstm" || t == "channel_delta") ? 1 : 0;
+    for (const auto& t : layer_types) n += (t == "mamba" || t == "gdn" || t == "mlstm" || t == "channel_delta" || t == "lightning" || t == "parallel") ? 1 : 0;
     return n;
 }
 
@@ -291,7 +306,7 @@ int LLMEngineConfig::num_attention_layers() const {
     int n = 0;
     if (layer_types.empty()) n = num_layers;
     else
-        for (const auto& t : layer_types) n += t == "attention" ? 1 : 0;
+        for (const auto& t : layer_types) n += (t == "attention" || t == "parallel") ? 1 : 0;
     return std::max(0, n - num_kv_shared_layers);
 }
 
@@ -344,7 +359,7 @@ std::string LLMEngineConfig::validate() const {
     if (num_experts > 0 && (num_experts_per_tok <= 0 || num_experts_per_tok > num_experts)) return "num_experts_per_tok must be in 1..num_experts";
     for (const auto& t : layer_types) {
         if (t == "mamba" && (mamba_num_heads <= 0 || mamba_d_state <= 0)) return "a mamba layer needs the mamba section";
-        if ((t == "mlstm" || t == "channel_delta") && run_state_values.size() != layer_types.size()) return t + " layers need their layer_specs";
+        if ((t == "mlstm" || t == "channel_delta" || t == "lightning" || t == "parallel") && run_state_values.size() != layer_types.size()) return t + " layers need their layer_specs";
         if (t == "gdn" && (gdn_num_v_heads <= 0 || gdn_head_k_dim <= 0)) return "a gdn layer needs the gdn section";
     }
     if (draft_type == "dflash" && dflash_block_size < 2) return "a block draft needs dflash_block_size >= 2";

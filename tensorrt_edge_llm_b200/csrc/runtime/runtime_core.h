@@ -74,7 +74,7 @@ struct LLMEngineConfig {
     bool has_qk_norm = false, attention_bias = false, attention_sink_bias = false, attention_k_eq_v = false, has_value_norm = false;
     int sliding_window = 0;                        // 0 = none
     std::vector<int> layer_windows;                // per layer (empty = sliding_window everywhere)
-    std::vector<std::string> layer_types;          // attention / mamba / gdn / mlstm / channel_delta / none per layer (per layer run of a looped stack)
+    std::vector<std::string> layer_types;          // attention / mamba / gdn / mlstm / channel_delta / lightning / parallel / none per layer (per layer run of a looped stack)
     std::vector<std::string> mlp_types;            // mlp / moe / none per layer
     int num_kv_shared_layers = 0;
     int num_experts = 0, num_experts_per_tok = 0, moe_intermediate_size = 0, shared_expert_intermediate_size = 0;

@@ -157,31 +157,59 @@ class Attention(nn.Module):
 
 class LayerAttention(nn.Module):
     """Attention with a geometry of its own (``AttentionConfig``): key and value sizes that may differ, partial rotary, a score scale,
-    chunked causal masking and a zero sink; or, without rotary, unit queries and keys and a query temperature.  Heads are padded to a
-    size the kernels take and share the paged cache layout; the model hands in the position table (cos / sin per (base, rotary size),
-    or the temperature per position)."""
+    chunked or windowed causal masking and a zero sink; or, without rotary, unit queries and keys and a query temperature; or norms over
+    whole query and key rows, interleaved rotation and values that turn with their positions.  Heads are padded to a size the kernels
+    take and share the paged cache layout; the model hands in the position table (cos / sin per (base, rotary size), or the
+    temperature per position; with rotated values a pair of tables, keys and values).
 
-    def __init__(self, cfg: ModelConfig, spec, prefix: str):
+    ``bare``: no projections of its own; a surrounding mixer hands packed q | k | v rows to :meth:`attend`."""
+
+    def __init__(self, cfg: ModelConfig, spec, prefix: str, bare: bool = False):
         super().__init__()
         self.spec, self.prefix, self.eps = spec, prefix, cfg.rms_norm_eps
         h, d = cfg.hidden_size, spec.pad
-        self.qkv_proj = HeadLinear(h, 0, out_heads=[(spec.num_heads, spec.head_dim, d), (spec.num_kv_heads, spec.head_dim, d),
-                                                    (spec.num_kv_heads, spec.v_head_dim, d)],
-                                   sources=["q_proj", "k_proj", "v_proj"], dtype=cfg.compute_dtype)
-        self.o_proj = HeadLinear(0, h, in_heads=(spec.num_heads, spec.v_head_dim, d), dtype=cfg.compute_dtype)
+        # heads of q, k and v in a packed row, and the input heads of the output projection
+        self.row_heads = [(spec.num_heads, spec.head_dim, d), (spec.num_kv_heads, spec.head_dim, d), (spec.num_kv_heads, spec.v_head_dim, d)]
+        self.out_heads = (spec.num_heads, spec.v_head_dim, d)
+        if not bare:
+            self.qkv_proj = HeadLinear(h, 0, out_heads=self.row_heads, sources=["q_proj", "k_proj", "v_proj"], dtype=cfg.compute_dtype)
+            self.o_proj = HeadLinear(0, h, in_heads=self.out_heads, dtype=cfg.compute_dtype)
         if spec.zero_sink:
             self.register_buffer("sinks", torch.zeros(spec.num_heads, dtype=torch.float32), persistent=False)
         else:
             self.sinks = None
+        if spec.row_norm:
+            self.q_norm = nn.Parameter(torch.ones(spec.num_heads * d, dtype=torch.float32), requires_grad=False)
+            self.k_norm = nn.Parameter(torch.ones(spec.num_kv_heads * d, dtype=torch.float32), requires_grad=False)
 
-    def forward(self, x: torch.Tensor, meta: StepMeta, kv_layer: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
+    @torch.no_grad()
+    def load_checkpoint(self, fetch) -> bool:
         sp = self.spec
-        if sp.unit_qk:
-            q = ops.unit_kv_write(self.qkv_proj(x), kv_layer, meta, table, sp.num_heads, sp.num_kv_heads, sp.pad, sp.head_dim, self.eps)
+        if sp.row_norm:
+            for name, p, heads in (("q_norm", self.q_norm, sp.num_heads), ("k_norm", self.k_norm, sp.num_kv_heads)):
+                w = fetch(f"{self.prefix}.{name}.weight")
+                if w is not None:
+                    p.zero_()
+                    p.view(heads, sp.pad)[:, :sp.head_dim] = w.float().reshape(heads, sp.head_dim)
+        return False        # the projections are loaded by the generic path
+
+    def attend(self, rows: torch.Tensor, meta: StepMeta, kv_layer: torch.Tensor, table, out: Optional[torch.Tensor] = None, mult: float = 1.0):
+        """Cache write and attention of packed q | k | v rows: head outputs ``[T, heads * pad]`` (into ``out`` and times ``mult``, with
+        rotated values)."""
+        sp, back = self.spec, None
+        if sp.row_norm:
+            keys, values = table
+            q = ops.turned_kv_write(rows, kv_layer, meta, keys, values, self.q_norm, self.k_norm, sp, self.eps)
+            back = (values, mult)
+        elif sp.unit_qk:
+            q = ops.unit_kv_write(rows, kv_layer, meta, table, sp.num_heads, sp.num_kv_heads, sp.pad, sp.head_dim, self.eps)
         else:
-            q = ops.rope_kv_write(self.qkv_proj(x), kv_layer, meta, table, sp.num_heads, sp.num_kv_heads, sp.pad)
-        o = ops.paged_attention(q, kv_layer, meta, sp.scale, None, self.sinks, chunk=sp.chunk, fp32_weights=sp.fp32_weights)
-        return self.o_proj(o.reshape(o.shape[0], -1))
+            q = ops.rope_kv_write(rows, kv_layer, meta, table, sp.num_heads, sp.num_kv_heads, sp.pad)
+        o = ops.paged_attention(q, kv_layer, meta, sp.scale, sp.window or None, self.sinks, chunk=sp.chunk, fp32_weights=sp.fp32_weights, back=back, out=out)
+        return o.reshape(o.shape[0], -1)
+
+    def forward(self, x: torch.Tensor, meta: StepMeta, kv_layer: torch.Tensor, table) -> torch.Tensor:
+        return self.o_proj(self.attend(self.qkv_proj(x), meta, kv_layer, table))
 
 
 class LatentAttention(nn.Module):
@@ -225,16 +253,18 @@ class LatentAttention(nn.Module):
 
 
 class GatedMLP(nn.Module):
-    """``down(act(gate x) * up x)`` with a size of its own (tanh-form gelu); the inner size is padded to what the kernels take."""
+    """``down(act(gate x) * up x)`` with a size of its own (tanh-form gelu or relu, with or without biases); the inner size is padded to
+    what the kernels take."""
 
-    def __init__(self, cfg: ModelConfig, size: int):
+    def __init__(self, cfg: ModelConfig, size: int, act: str = "gelu_tanh", bias: bool = False):
         super().__init__()
         pad = (1, size, (size + 63) // 64 * 64)
-        self.gate_up_proj = HeadLinear(cfg.hidden_size, 0, out_heads=[pad, pad], sources=["gate_proj", "up_proj"], dtype=cfg.compute_dtype)
-        self.down_proj = HeadLinear(0, cfg.hidden_size, in_heads=pad, dtype=cfg.compute_dtype)
+        self.act = act
+        self.gate_up_proj = HeadLinear(cfg.hidden_size, 0, out_heads=[pad, pad], sources=["gate_proj", "up_proj"], dtype=cfg.compute_dtype, bias=bias)
+        self.down_proj = HeadLinear(0, cfg.hidden_size, in_heads=pad, dtype=cfg.compute_dtype, bias=bias)
 
     def forward(self, x):
-        return self.down_proj(ops.geglu(self.gate_up_proj(x), True))
+        return self.down_proj(ops.glu(self.gate_up_proj(x), self.act))
 
 
 class MLP(nn.Module):

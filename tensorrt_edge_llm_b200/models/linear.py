@@ -132,11 +132,11 @@ class HeadLinear(Linear):
     ``in_heads``: the same for the input features.  Padding rows and columns are zero, so padded features are zeros on the
     way out and ignored on the way in."""
 
-    def __init__(self, in_features: int, out_features: int, out_heads=None, in_heads=None, sources=None, dtype=torch.bfloat16):
+    def __init__(self, in_features: int, out_features: int, out_heads=None, in_heads=None, sources=None, dtype=torch.bfloat16, bias: bool = False):
         self.out_heads, self.in_heads = out_heads, in_heads
         n_in = in_features if in_heads is None else in_heads[0] * in_heads[2]
         outs = [out_features] if out_heads is None else [h * pad for h, _, pad in out_heads]
-        super().__init__(n_in, outs, dtype=dtype, sources=sources)
+        super().__init__(n_in, outs, dtype=dtype, sources=sources, bias=bias)
 
     def _pad_in(self, w: torch.Tensor) -> torch.Tensor:
         if self.in_heads is None:
@@ -144,15 +144,16 @@ class HeadLinear(Linear):
         h, real, pad = self.in_heads
         return torch.nn.functional.pad(w.reshape(w.shape[0], h, real), (0, pad - real)).reshape(w.shape[0], h * pad)
 
+    def _pad_out(self, w: torch.Tensor, i: int) -> torch.Tensor:
+        if self.out_heads is None:
+            return w
+        h, real, pad = self.out_heads[i]
+        return torch.nn.functional.pad(w.reshape(h, real, -1), (0, 0, 0, pad - real)).reshape(h * pad, -1)
+
     def load_from(self, tensors):
-        parts = []
-        for i, t in enumerate(tensors):
-            w = self._pad_in(t["weight"])
-            if self.out_heads is not None:
-                h, real, pad = self.out_heads[i]
-                w = torch.nn.functional.pad(w.reshape(h, real, -1), (0, 0, 0, pad - real)).reshape(h * pad, -1)
-            parts.append(w)
-        self.weight.data.copy_(torch.cat(parts, 0).to(self.weight.dtype))
+        self.weight.data.copy_(torch.cat([self._pad_out(self._pad_in(t["weight"]), i) for i, t in enumerate(tensors)], 0).to(self.weight.dtype))
+        if self.bias is not None:
+            self.bias.data.copy_(torch.cat([self._pad_out(t["bias"].reshape(-1, 1), i) for i, t in enumerate(tensors)])[:, 0].to(self.bias.dtype))
 
     @torch.no_grad()
     def zero_padding(self) -> None:
@@ -165,6 +166,26 @@ class HeadLinear(Linear):
         for h, real, pad in self.out_heads or ():
             w[r0:r0 + h * pad].view(h, pad, -1)[:, real:] = 0
             r0 += h * pad
+
+
+class JoinedLinear(Linear):
+    """Sum of several linears over inputs that lie side by side in one row, as one product: source ``i`` reads the columns of
+    ``in_heads[i]`` (``(heads, real size, padded size)``)."""
+
+    def __init__(self, in_heads, out_features: int, sources, dtype=torch.bfloat16):
+        self.in_heads = in_heads
+        super().__init__(sum(h * pad for h, _, pad in in_heads), [out_features], dtype=dtype, sources=sources)
+
+    def load_from(self, tensors):
+        self.weight.data.copy_(torch.cat([torch.nn.functional.pad(t["weight"].reshape(-1, h, real), (0, pad - real)).reshape(-1, h * pad)
+                                          for t, (h, real, pad) in zip(tensors, self.in_heads)], 1).to(self.weight.dtype))
+
+    @torch.no_grad()
+    def zero_padding(self) -> None:
+        c0 = 0
+        for h, real, pad in self.in_heads:
+            self.weight.data[:, c0:c0 + h * pad].unflatten(1, (h, pad))[:, :, real:] = 0
+            c0 += h * pad
 
 
 class Fp32OutLinear(Linear):

@@ -20,11 +20,12 @@ import torch
 from torch import nn
 
 from .. import ops
-from ..config import LAYER_ATTENTION, LAYER_CHANNEL_DELTA, LAYER_GDN, LAYER_MAMBA, LAYER_MLP, LAYER_MLSTM, LAYER_MOE, ModelConfig
+from ..config import (LAYER_ATTENTION, LAYER_CHANNEL_DELTA, LAYER_GDN, LAYER_LIGHTNING, LAYER_MAMBA, LAYER_MLP, LAYER_MLSTM, LAYER_MOE, LAYER_PARALLEL,
+                      ModelConfig)
 from ..model import register_model
 from ..ops.meta import StepMeta
-from .default import MLP, Attention, CausalLM, RMSNorm
-from .linear import Fp32OutLinear, HeadLinear, StackedRankLinear, TPMode, make_linear
+from .default import MLP, Attention, CausalLM, LayerAttention, RMSNorm
+from .linear import Fp32OutLinear, HeadLinear, JoinedLinear, StackedRankLinear, TPMode, make_linear
 
 
 class RecurrentState:
@@ -34,7 +35,10 @@ class RecurrentState:
         tp = cfg.tp_size
         self.conv, self.ssm, self.gdn = {}, {}, {}
         self.mlstm, self.mlstm_norm = {}, {}      # matrix memory; normaliser and running maximum
-        self.delta = {}                           # channel-decay delta rule
+        self.delta = {}                           # delta rule with a decay per key channel or head
+        self.lightning = {}                       # linear attention with constant decays
+        self.inputs = {}                          # last rows of the stream in front of each mixer's input convolution, fp32
+        self.tokens = {}                          # the sequence's last token (bigram embeddings)
         runs = cfg.layer_run_ids if cfg.layer_specs else None
         for i, t in enumerate(cfg.layer_types):
             if t == LAYER_MAMBA:
@@ -51,16 +55,23 @@ class RecurrentState:
                 m = cfg.layer_specs[runs[i]].mlstm
                 self.mlstm[i] = torch.zeros(seats, m.num_heads, m.k_pad, m.v_pad, dtype=torch.float32, device=device)
                 self.mlstm_norm[i] = torch.zeros(seats, m.num_heads, m.k_pad + 1, dtype=torch.float32, device=device)
-            elif t == LAYER_CHANNEL_DELTA:
+            elif t in (LAYER_CHANNEL_DELTA, LAYER_PARALLEL):
                 d = cfg.layer_specs[runs[i]].delta
                 self.conv[i] = torch.zeros(seats, d.conv_dim, d.conv_kernel - 1, dtype=dtype, device=device)
                 self.delta[i] = torch.zeros(seats, d.num_heads, d.k_pad, d.v_pad, dtype=torch.float32, device=device)
+            elif t == LAYER_LIGHTNING:
+                l = cfg.layer_specs[runs[i]].lightning
+                self.lightning[i] = torch.zeros(seats, l.num_heads, l.k_pad, l.v_pad, dtype=torch.float32, device=device)
+            if cfg.input_conv > 1:
+                self.inputs[i] = torch.zeros(seats, cfg.input_conv - 1, cfg.hidden_size, dtype=torch.float32, device=device)
+        if cfg.bigram_buckets:
+            self.tokens[0] = torch.zeros(seats, 1, dtype=torch.int32, device=device)
 
     def bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in self.pools())
 
     def pools(self):
-        for d in (self.conv, self.ssm, self.gdn, self.mlstm, self.mlstm_norm, self.delta):
+        for d in (self.conv, self.ssm, self.gdn, self.mlstm, self.mlstm_norm, self.delta, self.lightning, self.inputs, self.tokens):
             yield from d.values()
 
     # ---- replay data -------------------------------------------------------------------------------------------------
@@ -301,25 +312,36 @@ class MLstmMixer(nn.Module):
 
 
 class ChannelDeltaMixer(nn.Module):
-    """Delta rule with one decay per head and key channel.  q, k and v come from one product; the inner rows of the two low-rank
-    projections (decays, output gate) from a second, their outer halves and the step sizes with fp32 results.  Short convolutions,
-    unit norms, decays, recurrence, head norm and output gate are one op over the step's rows (``ops.channel_delta``)."""
+    """Delta rule with one decay per head and key channel, or (``head_decay``) one per head.
 
-    def __init__(self, cfg: ModelConfig, spec, prefix: str):
+    Per channel: q, k and v come from one product; the inner rows of the two low-rank projections (decays, output gate) from a second,
+    their outer halves and the step sizes with fp32 results.  Per head: q, k, v and the gate from one product, step sizes and decays from a
+    second with fp32 results.  Short convolutions, unit norms, decays, recurrence, head norm and output gate are one op over the
+    step's rows (``ops.channel_delta``).  ``bare``: no projections; a surrounding mixer hands the rows to :meth:`recur`."""
+
+    def __init__(self, cfg: ModelConfig, spec, prefix: str, bare: bool = False):
         super().__init__()
         self.spec, self.prefix, self.eps = spec, prefix, cfg.rms_norm_eps
         h, n, nk, dt = cfg.hidden_size, spec.num_heads, spec.num_kv_heads, cfg.compute_dtype
-        self.qkv_proj = HeadLinear(h, 0, out_heads=[(nk, spec.head_k_dim, spec.k_pad), (nk, spec.head_k_dim, spec.k_pad),
-                                                    (n, spec.head_v_dim, spec.v_pad)], sources=["q_proj", "k_proj", "v_proj"], dtype=dt)
-        ranks = [(1, r, (r + 7) // 8 * 8) for r in (spec.decay_rank, spec.gate_rank)]
-        self.rank_proj = HeadLinear(h, 0, out_heads=ranks, sources=["decay_in_proj", "gate_in_proj"], dtype=dt)
-        self.up_proj = StackedRankLinear(ranks, [(n, spec.head_k_dim, spec.k_pad), (n, spec.head_v_dim, spec.v_pad)],
-                                         sources=["decay_out_proj", "gate_out_proj"], dtype=dt)
-        self.beta_proj = Fp32OutLinear(h, [n], dtype=dt)
-        self.o_proj = HeadLinear(0, h, in_heads=(n, spec.head_v_dim, spec.v_pad), dtype=dt)
+        self.row_heads = [(nk, spec.head_k_dim, spec.k_pad), (nk, spec.head_k_dim, spec.k_pad), (n, spec.head_v_dim, spec.v_pad)]
+        self.out_heads = (n, spec.head_v_dim, spec.v_pad)
+        if bare:
+            pass
+        elif spec.head_decay:
+            self.qkvg_proj = HeadLinear(h, 0, out_heads=self.row_heads + [self.out_heads], sources=["q_proj", "k_proj", "v_proj", "g_proj"], dtype=dt)
+            self.beta_decay_proj = Fp32OutLinear(h, [n, n], sources=["beta_proj", "decay_proj"], dtype=dt)
+        else:
+            self.qkv_proj = HeadLinear(h, 0, out_heads=self.row_heads, sources=["q_proj", "k_proj", "v_proj"], dtype=dt)
+            ranks = [(1, r, (r + 7) // 8 * 8) for r in (spec.decay_rank, spec.gate_rank)]
+            self.rank_proj = HeadLinear(h, 0, out_heads=ranks, sources=["decay_in_proj", "gate_in_proj"], dtype=dt)
+            self.up_proj = StackedRankLinear(ranks, [(n, spec.head_k_dim, spec.k_pad), self.out_heads],
+                                             sources=["decay_out_proj", "gate_out_proj"], dtype=dt)
+            self.beta_proj = Fp32OutLinear(h, [n], dtype=dt)
+        if not bare:
+            self.o_proj = HeadLinear(0, h, in_heads=self.out_heads, dtype=dt)
         self.conv_weight = nn.Parameter(torch.zeros(spec.conv_dim, spec.conv_kernel, dtype=dt), requires_grad=False)
         self.a_log = nn.Parameter(torch.zeros(n, dtype=torch.float32), requires_grad=False)
-        self.decay_bias = nn.Parameter(torch.zeros(n * spec.k_pad, dtype=torch.float32), requires_grad=False)
+        self.decay_bias = nn.Parameter(torch.zeros(n if spec.head_decay else n * spec.k_pad, dtype=torch.float32), requires_grad=False)
         self.norm_weight = nn.Parameter(torch.ones(spec.v_pad, dtype=torch.float32), requires_grad=False)
 
     def _heads(self, t: torch.Tensor, heads: int, real: int, pad: int) -> torch.Tensor:
@@ -330,12 +352,12 @@ class ChannelDeltaMixer(nn.Module):
     @torch.no_grad()
     def load_checkpoint(self, fetch) -> bool:
         sp = self.spec
-        sizes = ((sp.num_kv_heads, sp.head_k_dim, sp.k_pad), (sp.num_kv_heads, sp.head_k_dim, sp.k_pad), (sp.num_heads, sp.head_v_dim, sp.v_pad))
         taps = [fetch(f"{self.prefix}.{n}_conv") for n in "qkv"]
         if any(t is None for t in taps):
             return False
-        self.conv_weight.copy_(torch.cat([self._heads(t, *z) for t, z in zip(taps, sizes)]).to(self.conv_weight.dtype))
-        self.decay_bias.copy_(self._heads(fetch(f"{self.prefix}.dt_bias").float(), sp.num_heads, sp.head_k_dim, sp.k_pad)[:, 0])
+        self.conv_weight.copy_(torch.cat([self._heads(t, *z) for t, z in zip(taps, self.row_heads)]).to(self.conv_weight.dtype))
+        bias = fetch(f"{self.prefix}.dt_bias").float()
+        self.decay_bias.copy_(bias if sp.head_decay else self._heads(bias, sp.num_heads, sp.head_k_dim, sp.k_pad)[:, 0])
         self.norm_weight.zero_()
         self.norm_weight[:sp.head_v_dim] = fetch(f"{self.prefix}.head_norm.weight").float()
         return False        # the projections and a_log are loaded by the generic path
@@ -347,19 +369,103 @@ class ChannelDeltaMixer(nn.Module):
         self.decay_bias.copy_(torch.rand(self.decay_bias.shape, generator=gen) - 4.0)
 
     def forward(self, x, meta: StepMeta, state: RecurrentState, run: int):
-        qkv, beta = self.qkv_proj(x), self.beta_proj(x)
-        decay, gate = self.up_proj(self.rank_proj(x))
+        n, sp = self.spec.num_heads, self.spec
+        if sp.head_decay:
+            rows, small = self.qkvg_proj(x), self.beta_decay_proj(x)
+            saved = (rows[:, :sp.conv_dim], small[:, n:], rows[:, sp.conv_dim:], small[:, :n])
+        else:
+            qkv, beta = self.qkv_proj(x), self.beta_proj(x)
+            decay, gate = self.up_proj(self.rank_proj(x))
+            saved = (qkv, decay, gate, beta)
         if state.record is not None:
-            state.record[run] = (qkv, decay, gate, beta)
-        return self.o_proj(self._recur(qkv, decay, gate, beta, meta, state, run))
+            state.record[run] = saved
+        return self.o_proj(self.recur(*saved, meta, state, run))
 
-    def _recur(self, qkv, decay, gate, beta, meta, state, run):
+    def recur(self, qkv, decay, gate, beta, meta, state, run, out: Optional[torch.Tensor] = None, mult: float = 1.0):
+        """Gated head outputs of packed rows and pre-activations (into ``out``, times ``mult``)."""
         return ops.channel_delta(qkv, decay, gate, beta, self.conv_weight, self.a_log, self.decay_bias, self.norm_weight, state.conv[run],
-                                 state.delta[run], meta, self.spec, self.eps)
+                                 state.delta[run], meta, self.spec, self.eps, out=out, mult=mult)
 
     @torch.no_grad()
     def replay(self, saved, rows: torch.Tensor, meta: StepMeta, state: RecurrentState, run: int) -> None:
-        self._recur(*(t.index_select(0, rows) for t in saved), meta, state, run)
+        self.recur(*(t.index_select(0, rows) for t in saved), meta, state, run)
+
+
+class LightningMixer(nn.Module):
+    """Linear attention with a constant decay per head: q, k, v and the output gate from one product; silu, recurrence, the norm over
+    all heads and the gate are one op (``ops.lightning``); state in fp32 rows indexed by seat."""
+
+    POWERS = 256          # decay^0 .. decay^POWERS, rounded once from double
+
+    def __init__(self, cfg: ModelConfig, spec, prefix: str):
+        super().__init__()
+        self.spec, self.prefix, self.eps = spec, prefix, cfg.rms_norm_eps
+        h, n, dt = cfg.hidden_size, spec.num_heads, cfg.compute_dtype
+        self.qkvg_proj = HeadLinear(h, 0, out_heads=[(n, spec.head_k_dim, spec.k_pad), (n, spec.head_k_dim, spec.k_pad),
+                                                     (n, spec.head_v_dim, spec.v_pad), (n, spec.head_v_dim, spec.v_pad)],
+                                    sources=["q_proj", "k_proj", "v_proj", "g_proj"], dtype=dt)
+        self.o_proj = HeadLinear(0, h, in_heads=(n, spec.head_v_dim, spec.v_pad), dtype=dt)
+        self.out_norm = nn.Parameter(torch.ones(n * spec.v_pad, dtype=torch.float32), requires_grad=False)
+        decay = torch.tensor([float(x) for x in spec.decay], dtype=torch.float64)[:, None]
+        steps = torch.arange(self.POWERS + 1, dtype=torch.float64, device=decay.device)
+        self.register_buffer("decay_powers", (decay ** steps).float(), persistent=False)
+
+    @torch.no_grad()
+    def load_checkpoint(self, fetch) -> bool:
+        w = fetch(f"{self.prefix}.head_norm.weight")
+        if w is not None:
+            sp = self.spec
+            self.out_norm.zero_()
+            self.out_norm.view(sp.num_heads, sp.v_pad)[:, :sp.head_v_dim] = w.float().reshape(sp.num_heads, sp.head_v_dim)
+        return False        # the projections are loaded by the generic path
+
+    def forward(self, x, meta: StepMeta, state: RecurrentState, run: int):
+        rows = self.qkvg_proj(x)
+        if state.record is not None:
+            state.record[run] = rows
+        return self.o_proj(self._recur(rows, meta, state, run))
+
+    def _recur(self, rows, meta, state, run):
+        return ops.lightning(rows, self.out_norm, self.decay_powers, state.lightning[run], meta, self.spec.head_v_dim, self.eps)
+
+    @torch.no_grad()
+    def replay(self, saved, rows: torch.Tensor, meta: StepMeta, state: RecurrentState, run: int) -> None:
+        self._recur(saved.index_select(0, rows), meta, state, run)
+
+
+class ParallelMixer(nn.Module):
+    """Attention and a delta rule on the same input, ``attention_mult * attention + delta_mult * delta``.  One product gives the rows of both,
+    a small one with fp32 results the step sizes and decays; both write their heads into one row, and one product over it is the
+    weighted sum of the two output projections (the multipliers join the heads in fp32)."""
+
+    def __init__(self, cfg: ModelConfig, spec, prefix: str):
+        super().__init__()
+        self.spec, h, dt = spec, cfg.hidden_size, cfg.compute_dtype
+        self.left = LayerAttention(cfg, spec.attention, f"{prefix}.left", bare=True)
+        self.right = ChannelDeltaMixer(cfg, spec.delta, f"{prefix}.right", bare=True)
+        heads = self.left.row_heads + self.right.row_heads + [self.right.out_heads]
+        self.in_proj = HeadLinear(h, 0, out_heads=heads, dtype=dt, sources=[f"left.{n}_proj" for n in "qkv"] + [f"right.{n}_proj" for n in "qkvg"])
+        n = spec.delta.num_heads
+        self.beta_decay_proj = Fp32OutLinear(h, [n, n], sources=["right.beta_proj", "right.decay_proj"], dtype=dt)
+        self.out_proj = JoinedLinear([self.left.out_heads, self.right.out_heads], h, sources=["left.o_proj", "right.o_proj"], dtype=dt)
+        width = lambda heads: sum(h * pad for h, _, pad in heads)
+        self.left_cols, self.right_cols = width(self.left.row_heads), width(self.right.row_heads)
+        self.left_out = width([self.left.out_heads])
+
+    def forward(self, x, meta: StepMeta, cache, table, run: int):
+        rows, small, state = self.in_proj(x), self.beta_decay_proj(x), cache.recurrent
+        n, c = self.spec.delta.num_heads, self.left_cols + self.right_cols
+        delta_in = (rows[:, self.left_cols:c], small[:, n:], rows[:, c:], small[:, :n])
+        if state.record is not None:
+            state.record[run] = delta_in
+        y = torch.empty(x.shape[0], self.out_proj.in_features, dtype=x.dtype, device=x.device)
+        self.left.attend(rows[:, :self.left_cols], meta, cache.kv_layer(run), table, out=y[:, :self.left_out], mult=self.spec.attention_mult)
+        self.right.recur(*delta_in, meta, state, run, out=y[:, self.left_out:], mult=self.spec.delta_mult)
+        return self.out_proj(y)
+
+    @torch.no_grad()
+    def replay(self, saved, rows: torch.Tensor, meta: StepMeta, state: RecurrentState, run: int) -> None:
+        self.right.replay(saved, rows, meta, state, run)
 
 
 class HybridLayer(nn.Module):

@@ -10,6 +10,7 @@ MoE plugins :2017-2209, all_reduce :2754) expressed as directly executable funct
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional, Tuple
 
 import torch
@@ -80,6 +81,25 @@ def geglu(gate_up, tanh_approx=True):
     return (g * gate_up[..., inter:].float()).to(gate_up.dtype)
 
 
+def glu(gate_up, act="gelu_tanh"):
+    """``act(gate) * up`` over the fused ``[T, 2·I]`` projection output; ``act``: ``"gelu_tanh"`` or ``"relu"``."""
+    if act == "gelu_tanh":
+        return geglu(gate_up, True)
+    if act != "relu":
+        raise ValueError(f"unknown gate activation {act!r}")
+    if gate_up.is_cuda:
+        return cuda_ops().reglu(gate_up)
+    inter = gate_up.shape[-1] // 2
+    return (torch.relu(gate_up[..., :inter].float()) * gate_up[..., inter:].float()).to(gate_up.dtype)
+
+
+def softcap_(logits, cap):
+    """``cap * tanh(logits / cap)`` of fp32 logits, in place."""
+    if logits.is_cuda:
+        return cuda_ops().softcap_(logits, cap)
+    return logits.div_(cap).tanh_().mul_(cap)
+
+
 def relu2(x):
     if x.is_cuda:
         return cuda_ops().relu2(x)
@@ -115,14 +135,21 @@ def rope_kv_write(qkv, kv_layer, meta, cos_sin, num_q_heads, num_kv_heads, head_
                              q_norm_w, k_norm_w, eps)
 
 
-def rope_cos_sin(max_pos, rotary_dim, theta, scaling=None, device="cpu"):
+def rope_cos_sin(max_pos, rotary_dim, theta, scaling=None, device="cpu", pairs=0):
     """RoPE ``[max_pos, rotary_dim]`` cos | sin table (fp32, angles in fp64) with the frequency scaling of the checkpoint; built by
-    a kernel when the table lives on a GPU."""
+    a kernel when the table lives on a GPU.  ``pairs`` > ``rotary_dim / 2``: the table goes on to that many pairs, of angle zero."""
     dev = torch.device(device)
     if dev.type == "cuda":
         inv, att = ref.rope_frequencies(max_pos, rotary_dim, theta, scaling)
+        if pairs:
+            inv = torch.nn.functional.pad(inv, (0, pairs - inv.numel()))
         return cuda_ops().rope_table(inv, att, max_pos, dev)
-    return ref.rope_cos_sin(max_pos, rotary_dim, theta, scaling, device=device)
+    t = ref.rope_cos_sin(max_pos, rotary_dim, theta, scaling, device=device)
+    if pairs:
+        c, s = t.chunk(2, dim=-1)
+        fill = pairs - c.shape[-1]
+        t = torch.cat([torch.nn.functional.pad(c, (0, fill), value=1.0), torch.nn.functional.pad(s, (0, fill))], dim=-1)
+    return t
 
 
 def mrope_rows(cos_sin, positions3, sections):
@@ -140,12 +167,16 @@ def rope_q(q, kv_layer, meta, cos_sin, num_q_heads, head_dim, q_norm_w=None, eps
     return ref.rope_q(q, meta, cos_sin, num_q_heads, head_dim, q_norm_w, eps)
 
 
-def paged_attention(q, kv_layer, meta, scale, sliding_window=None, sinks=None, causal=True, chunk=0, fp32_weights=False):
+def paged_attention(q, kv_layer, meta, scale, sliding_window=None, sinks=None, causal=True, chunk=0, fp32_weights=False, back=None, out=None):
     """``chunk`` > 0: row at position ``i`` sees only keys ``j`` with ``j // chunk == i // chunk`` (and ``j <= i``).
-    ``fp32_weights``: the softmax weights keep fp32 precision in the weighted sum of 16-bit values."""
+    ``fp32_weights``: the softmax weights keep fp32 precision in the weighted sum of 16-bit values.
+    ``back``: ``(cos | sin table, factor)``; every output is turned back by its position (neighbouring features form the pairs) and
+    multiplied, before it is rounded.  ``out``: where the rows go (``[T, heads * head]``, its rows may lie further apart)."""
     if q.is_cuda:
-        return cuda_ops().paged_attention(q, kv_layer, meta, scale, sliding_window, sinks, causal=causal, chunk=chunk, fp32_weights=fp32_weights)
-    return ref.paged_attention(q, kv_layer, meta, scale, sliding_window, sinks, causal=causal, chunk=chunk)
+        return cuda_ops().paged_attention(q, kv_layer, meta, scale, sliding_window, sinks, causal=causal, chunk=chunk, fp32_weights=fp32_weights,
+                                          back=back, out=out)
+    o = ref.paged_attention(q, kv_layer, meta, scale, sliding_window, sinks, causal=causal, chunk=chunk, back=back)
+    return o if out is None else out.copy_(o.reshape(out.shape))
 
 
 def linear_f32(x, weight, bias=None):
@@ -171,6 +202,38 @@ def stream_norm(stream, weight, eps, *, delta=None, routed=None, mult=1.0, step=
     return ref.stream_norm(*args)
 
 
+@dataclass
+class Bigram:
+    """Second embedding of a token: row ``(previous * mul_prev + token * mul_cur) mod buckets`` of ``table``, row ``buckets`` where a
+    sequence starts.  ``last``: ``[seats, 1]`` int32, the last token of every sequence."""
+
+    table: torch.Tensor
+    last: torch.Tensor
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+def stream_post(stream, delta, weight, groups, eps, meta, dtype, *, ids=None, table=None, bigram=None, conv=None, history=None, out_norm=None):
+    """Advance the fp32 residual stream by a normed sublayer output and write what the next sublayer reads: ``(stream, h)``.
+
+    ``stream`` (or ``table[ids]`` plus the row of ``bigram`` when it is ``None``) ``+ norm(delta) * weight``; the norm divides each of ``groups``
+    equal parts of a row by its own root mean square.  ``h`` in ``dtype`` is the stream itself; with ``conv`` ``[taps, width]`` (fp32) the
+    stream plus its causal convolution over time, whose ``history`` ``[seats, taps - 1, width]`` (fp32) is advanced; with ``out_norm`` the norm
+    of the stream times that weight."""
+    t = ids if stream is None else stream
+    f = cuda_ops().stream_post if t.is_cuda else ref.stream_post
+    return f(stream, delta, weight, groups, eps, meta, dtype, ids, table, bigram, conv, history, out_norm)
+
+
+def lightning(rows, norm_w, powers, state, meta, dv_real, eps):
+    """Linear attention with a constant decay per head over packed ``[q | k | v | g]`` rows: silu on q, k and v, the recurrence, an RMS norm
+    over all heads of a row, and the sigmoid of g: ``[T, heads · dv]``.  ``powers`` ``[heads, n + 1]``: powers of the decays from 0 on;
+    ``state`` ``[seats, heads, dk, dv]`` is advanced in place; ``dv_real``: value features of a padded head."""
+    f = cuda_ops().lightning if rows.is_cuda else ref.lightning
+    return f(rows, norm_w, powers, state, meta, dv_real, eps)
+
+
 def moe_route_chosen(logits, top_k):
     """The ``top_k`` largest fp32 logits per row and the softmax over them: ``(weights, indices)``."""
     if logits.is_cuda:
@@ -186,14 +249,15 @@ def mlstm(qkvg, gates, norm_w, state, norm_state, meta, scale, cap, eps, dv_real
     return ref.mlstm(qkvg, gates, norm_w, state, norm_state, meta, scale, cap, eps, dv_real)
 
 
-def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, meta, spec, eps):
-    """Delta-rule mixer with a decay per key channel, from packed projections to gated head outputs ``[T, heads * v_pad]``.
+def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, meta, spec, eps, out=None, mult=1.0):
+    """Delta-rule mixer with a decay per key channel (or per head), from packed projections to gated head outputs ``[T, heads * v_pad]``
+    times ``mult``.
 
-    ``qkv``: packed ``[q | k | v]`` rows of padded heads; ``decay`` (fp32, before bias and softplus), ``gate`` and ``beta`` (fp32) are
-    pre-activations.  ``conv_state`` ``[seats, channels, taps - 1]`` and ``state`` ``[seats, heads, k_pad, v_pad]`` are advanced in
-    place.  ``spec``: :class:`config.ChannelDeltaConfig`."""
+    ``qkv``: packed ``[q | k | v]`` rows of padded heads; ``decay`` (fp32, before bias and softplus; ``[T, heads]`` with one decay per
+    head), ``gate`` and ``beta`` (fp32) are pre-activations.  ``conv_state`` ``[seats, channels, taps - 1]`` and ``state``
+    ``[seats, heads, k_pad, v_pad]`` are advanced in place.  ``spec``: :class:`config.ChannelDeltaConfig`.  ``out``: where the rows go."""
     f = cuda_ops().channel_delta if qkv.is_cuda else ref.channel_delta
-    return f(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, meta, spec, eps)
+    return f(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, meta, spec, eps, out=out, mult=mult)
 
 
 def query_temperature(length, coef, every, device="cpu"):
@@ -206,6 +270,14 @@ def unit_kv_write(qkv, kv_layer, meta, temperature, num_q_heads, num_kv_heads, h
     position; writes keys and values into the paged cache and returns ``q [T, Hq, D]``."""
     f = cuda_ops().unit_kv_write if qkv.is_cuda else ref.unit_kv_write
     return f(qkv, kv_layer, meta, temperature, num_q_heads, num_kv_heads, head_dim, real_dim, eps)
+
+
+def turned_kv_write(rows, kv_layer, meta, key_table, value_table, q_norm, k_norm, spec, eps):
+    """Packed q | k | v rows: RMS norms over all heads of the queries and of the keys, interleaved rotation of both by ``key_table`` and of the
+    values by ``value_table`` (cos | sin, a pair per two padded features); keys and values go to the paged cache.  Returns ``q [T, Hq, D]``.
+    ``spec``: :class:`config.AttentionConfig`."""
+    f = cuda_ops().turned_kv_write if rows.is_cuda else ref.turned_kv_write
+    return f(rows, kv_layer, meta, key_table, value_table, q_norm, k_norm, spec, eps)
 
 
 def latent_write(rows, kv_layer, meta, cos_sin, norm_w, spec, eps):

@@ -180,11 +180,30 @@ def geglu(gate_up: torch.Tensor, tanh_approx: bool = True) -> torch.Tensor:
     if gate_up.dtype == torch.float32:
         if not tanh_approx:
             raise TypeError("geglu: the fp32 form covers the tanh gelu only")
-        _check(lib().telb_geglu_f32(_p(gate_up.contiguous()), _p(out), c_ll(rows), c_int(inter), _stream()), "geglu_f32")
+        _check(lib().telb_glu_f32(_p(gate_up.contiguous()), _p(out), c_ll(rows), c_int(inter), c_int(0), _stream()), "glu_f32")
         return out
     _check(lib().telb_geglu(_p(gate_up), _p(out), c_ll(rows), c_int(inter), c_int(1 if tanh_approx else 0), c_int(_is_bf16(gate_up)),
                             _stream()), "geglu")
     return out
+
+
+def reglu(gate_up: torch.Tensor) -> torch.Tensor:
+    """``relu(gate) * up``."""
+    gate_up = gate_up.contiguous()
+    rows, two = gate_up.shape
+    out = torch.empty(rows, two // 2, dtype=gate_up.dtype, device=gate_up.device)
+    if gate_up.dtype == torch.float32:
+        _check(lib().telb_glu_f32(_p(gate_up), _p(out), c_ll(rows), c_int(two // 2), c_int(1), _stream()), "glu_f32")
+    else:
+        _check(lib().telb_geglu(_p(gate_up), _p(out), c_ll(rows), c_int(two // 2), c_int(2), c_int(_is_bf16(gate_up)), _stream()), "reglu")
+    return out
+
+
+def softcap_(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    if logits.dtype != torch.float32 or not logits.is_contiguous():
+        raise TypeError("softcap_: contiguous fp32 logits")
+    _check(lib().telb_softcap(_p(logits), c_ll(logits.numel()), c_float(cap), _stream()), "softcap")
+    return logits
 
 
 def swiglu(gate_up: torch.Tensor) -> torch.Tensor:
@@ -314,6 +333,56 @@ def stream_norm(stream, weight, eps: float, delta, routed, mult: float, step, of
     return x, h
 
 
+class StreamPostParams(ctypes.Structure):
+    """Host mirror of ``StreamPostParams`` (``csrc/kernels/stream_post.cu``)."""
+    _fields_ = [(n, c_vp) for n in ("ids", "table", "bigram", "last", "x_in", "delta", "weight", "conv", "history", "out_norm", "x_out", "h", "q_start",
+                                    "q_len", "past_len", "slot_ids", "seq_ids")] + \
+               [(n, c_ll) for n in ("buckets", "mul_prev", "mul_cur")] + \
+               [(n, c_int) for n in ("vocab", "width", "groups", "tokens", "taps", "block_rows")] + [("eps", c_float)]
+
+
+def _conv_block_rows(meta: StepMeta, tokens: int) -> int:
+    """Rows per CTA of the convolution form: every block reads the rows in front of it once more, so long steps take long blocks."""
+    if meta.max_q_len == 1:
+        return 1
+    return 8 if tokens <= 148 * 2 * 8 else 16 if tokens <= 148 * 4 * 16 else 32
+
+
+def stream_post(stream, delta, weight, groups: int, eps: float, meta: StepMeta, dtype, ids, table, bigram, conv, history, out_norm):
+    """See :func:`ops.stream_post`."""
+    f32 = torch.float32
+    if stream is None:
+        t, width, dev = ids.numel(), table.shape[1], table.device
+        ids = ids.to(torch.int32).contiguous()
+        if table.dtype != dtype or (bigram is not None and (bigram.table.dtype != dtype or bigram.table.shape != (bigram.buckets + 1, width))):
+            raise TypeError(f"stream_post: embedding tables of {table.dtype}, activations {dtype}")
+        if bigram is not None:
+            assert bigram.last.dtype == torch.int32 and bigram.last.is_contiguous() and bigram.table.is_contiguous()
+    else:
+        (t, width), dev = stream.shape, stream.device
+        assert stream.dtype == f32 and stream.is_contiguous()
+        ids = table = bigram = None
+    if delta is not None:
+        delta = delta.contiguous()
+        assert delta.dtype == dtype and delta.shape == (t, width) and weight.dtype == f32 and weight.numel() == width
+    taps = 0 if conv is None else conv.shape[0]
+    if conv is not None:
+        assert conv.dtype == f32 and conv.is_contiguous() and conv.shape[1] == width and out_norm is None
+        assert taps == 1 or (history.dtype == f32 and history.is_contiguous() and history.shape[1:] == (taps - 1, width))
+    x = torch.empty(t, width, dtype=f32, device=dev)
+    h = torch.empty(t, width, dtype=dtype, device=dev)
+    ptr = lambda v: None if v is None else _p(v).value
+    b = bigram
+    p = StreamPostParams(*[ptr(v) for v in (ids, table, None if b is None else b.table, None if b is None else b.last, stream, delta, weight, conv,
+                                            history if taps > 1 else None, out_norm, x, h, meta.q_start, meta.q_len, meta.past_len, meta.slot_ids,
+                                            meta.seq_ids)],
+                         *((0, 0, 0) if b is None else (b.buckets, b.mul_prev, b.mul_cur)), 0 if table is None else table.shape[0], width, groups, t, taps,
+                         _conv_block_rows(meta, t) if taps else 1, eps)
+    code = 2 if dtype == f32 else int(dtype == torch.bfloat16)
+    _check(lib().telb_stream_post(ctypes.byref(p), c_int(code), _stream()), "stream_post")
+    return x, h
+
+
 def rope_table(inv_freq: torch.Tensor, attention_factor: float, max_pos: int, device) -> torch.Tensor:
     """``[max_pos, 2 * len(inv_freq)]`` fp32 cos | sin table from fp64 inverse frequencies, built on the device."""
     inv = inv_freq.to(device=device, dtype=torch.float64).contiguous()
@@ -426,33 +495,34 @@ def paged_attention_decode_fp8(q8: torch.Tensor, kv_layer: torch.Tensor, meta: S
     return out if out_scale is None else QuantActs(xq, sf, (t, hq * d), out_dtype)
 
 
-def _visible_len(meta: StepMeta, chunk: int) -> int:
-    """Most keys one row of the step can see."""
-    return min(meta.max_seq_len, chunk) if chunk > 0 else meta.max_seq_len
+def _visible_len(meta: StepMeta, chunk: int, window: int = 0) -> int:
+    """Most keys that rows of one tile of the step can see."""
+    n = min(meta.max_seq_len, chunk) if chunk > 0 else meta.max_seq_len
+    return min(n, window + 128) if window > 0 else n
 
 
-def _attn_splits(meta: StepMeta, hkv: int, group: int, chunk: int = 0) -> int:
+def _attn_splits(meta: StepMeta, hkv: int, group: int, chunk: int = 0, window: int = 0) -> int:
     tq = 128 // group
     qtiles = (meta.max_q_len + tq - 1) // tq
     ctas = meta.num_seqs * hkv * qtiles
     if ctas >= 148 or meta.max_q_len > 4 * tq:
         return 1
-    kv_tiles = max(1, (_visible_len(meta, chunk) + 63) // 64)
+    kv_tiles = max(1, (_visible_len(meta, chunk, window) + 63) // 64)
     return max(1, min((2 * 148 + ctas - 1) // ctas, kv_tiles, 32))
 
 
-def _decode_splits(meta: StepMeta, hkv: int, chunk: int = 0) -> int:
+def _decode_splits(meta: StepMeta, hkv: int, chunk: int = 0, window: int = 0) -> int:
     ctas = meta.num_seqs * hkv
     if ctas >= 148:
         return 1
-    tiles = max(1, (_visible_len(meta, chunk) + 127) // 128)
+    tiles = max(1, (_visible_len(meta, chunk, window) + 127) // 128)
     return max(1, min((148 + ctas - 1) // ctas, tiles, 32))
 
 
 def paged_attention(q, kv_layer, meta: StepMeta, scale, sliding_window=None, sinks=None, splits: Optional[int] = None,
                     kernel: Optional[str] = None, trace: Optional[torch.Tensor] = None, causal: bool = True,
                     skip_thr: Optional[torch.Tensor] = None, skip_stats: Optional[torch.Tensor] = None, chunk: int = 0,
-                    fp32_weights: bool = False) -> torch.Tensor:
+                    fp32_weights: bool = False, back: Optional[tuple] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Paged GQA attention.  Decode-shaped steps (``max_q_len * Hq/Hkv <= 16``, head_dim 128, causal)
     run the token-major XQA-style kernel; everything else the row-major tile kernel.
     ``kernel`` forces ``"decode"`` or ``"tile"``; ``causal=False`` lets every row see every token of its sequence; ``chunk`` > 0 limits
@@ -466,7 +536,16 @@ def paged_attention(q, kv_layer, meta: StepMeta, scale, sliding_window=None, sin
     t, hq, d = q.shape
     hkv = kv_layer.shape[2]
     group = hq // hkv
-    out = torch.empty_like(q)
+    table, mult = back if back is not None else (None, 1.0)
+    if out is None:
+        out = torch.empty_like(q)
+        ld_out = hq * d
+    else:                                   # rows of a wider buffer
+        assert out.shape == (t, hq * d) and out.dtype == q.dtype and out.stride(1) == 1 and out.stride(0) % 8 == 0 and (back is not None or out.is_contiguous())
+        ld_out = out.stride(0)
+    if back is not None and (table.dtype != torch.float32 or not table.is_contiguous() or table.shape[1] != d or meta.tree_mask is not None):
+        raise ValueError("rotated values: an fp32 table row per position and causal steps")
+    win = sliding_window if sliding_window and sliding_window > 0 else 0
     tm = meta.tree_mask
     if q.dtype == torch.float32 or d not in (64, 128, 256):
         if tm is not None or not causal or skip_thr is not None or meta.skip_thr is not None:
@@ -474,7 +553,7 @@ def paged_attention(q, kv_layer, meta: StepMeta, scale, sliding_window=None, sin
         _check(lib().telb_paged_attention_simt(
             _p(q), _p(kv_layer), _p(out), _p(meta.q_start), _p(meta.past_len), _p(meta.seq_ids), _p(meta.page_table), c_int(t),
             c_int(meta.page_table.shape[1]), c_int(meta.page_size), c_int(hq), c_int(hkv), c_int(d), c_float(scale), c_int(sliding_window or 0),
-            c_int(chunk), _p(sinks), c_int(_dtype_code(q)), _stream()), "paged_attention_simt")
+            c_int(chunk), _p(sinks), _p(table), c_float(mult), c_ll(ld_out), c_int(_dtype_code(q)), _stream()), "paged_attention_simt")
         return out
     ws = Workspace.get(q.device)
     decode_ok = (tm is None and d == 128 and meta.max_q_len * group <= 16 and 16 % group == 0)
@@ -489,22 +568,24 @@ def paged_attention(q, kv_layer, meta: StepMeta, scale, sliding_window=None, sin
         if not decode_ok:
             raise ValueError("step is not decode-shaped")
         if splits is None:
-            splits = _decode_splits(meta, hkv, chunk)
+            splits = _decode_splits(meta, hkv, chunk, win)
         _check(lib().telb_paged_attention_decode_traced(
             _p(q), _p(kv_layer), _p(out), _p(meta.q_start), _p(meta.q_len), _p(meta.past_len), _p(meta.page_table),
             c_int(meta.num_seqs), c_int(t), c_int(meta.max_q_len), c_int(kv_layer.shape[0]), c_int(meta.page_table.shape[1]),
             c_int(meta.page_size), c_int(hq), c_int(hkv), c_int(d), c_float(scale), c_int(sliding_window or 0), c_int(splits),
-            _p(ws.attn_ws), c_ll(ws.attn_ws.numel()), c_int(_is_bf16(q)), _p(ws.status), _p(trace), _p(sinks), c_int(chunk), c_int(int(fp32_weights)), _stream()),
+            _p(ws.attn_ws), c_ll(ws.attn_ws.numel()), c_int(_is_bf16(q)), _p(ws.status), _p(trace), _p(sinks), c_int(chunk), c_int(int(fp32_weights)),
+            _p(table), c_float(mult), _p(meta.positions), c_ll(ld_out), _stream()),
             "paged_attention_decode", 2 if splits > 1 else 1)
         return out
     if splits is None:
-        splits = _attn_splits(meta, hkv, group, chunk)
+        splits = _attn_splits(meta, hkv, group, chunk, win)
     _check(lib().telb_paged_attention(
         _p(q), _p(kv_layer), _p(out), _p(meta.q_start), _p(meta.q_len), _p(meta.past_len), _p(meta.page_table),
         _p(tm), c_int(tm.shape[1] if tm is not None else 0), c_int(meta.num_seqs), c_int(t), c_int(meta.max_q_len),
         c_int(kv_layer.shape[0]), c_int(meta.page_table.shape[1]), c_int(meta.page_size), c_int(hq), c_int(hkv),
         c_int(d), c_float(scale), c_int(sliding_window or 0), c_int(splits), _p(ws.attn_ws), c_ll(ws.attn_ws.numel()),
-        c_int(_is_bf16(q)), _p(ws.status), _p(sinks), _p(skip_thr), _p(skip_stats), c_int(chunk), c_int(int(fp32_weights)), _stream()), "paged_attention", 2 if splits > 1 else 1)
+        c_int(_is_bf16(q)), _p(ws.status), _p(sinks), _p(skip_thr), _p(skip_stats), c_int(chunk), c_int(int(fp32_weights)),
+        _p(table), c_float(mult), _p(meta.positions), c_ll(ld_out), _stream()), "paged_attention", 2 if splits > 1 else 1)
     return out
 
 
@@ -1072,27 +1153,67 @@ def mlstm(qkvg, gates, norm_w, state, norm_state, meta: StepMeta, scale: float, 
     return out
 
 
+class LightningParams(ctypes.Structure):
+    """Host mirror of ``LightningParams`` (``csrc/kernels/lightning_common.cuh``)."""
+    _fields_ = [(n, c_vp) for n in ("rows", "act", "powers", "state", "norm_w", "out", "o32", "carry", "q_start", "q_len", "past_len", "slot_ids", "status")] + \
+               [(n, c_int) for n in ("ld", "heads", "dk", "dv", "k_off", "v_off", "g_off", "dv_real", "n_powers", "tokens", "num_seqs", "segments",
+                                     "seg_chunks")] + [("eps", c_float)]
+
+
+def lightning(rows, norm_w, powers, state, meta: StepMeta, dv_real: int, eps: float, kernel: Optional[str] = None) -> torch.Tensor:
+    """See :func:`ops.lightning`.  Steps of one row per sequence run the decode kernel, longer ones the walk row by row; ``kernel`` forces
+    ``"step"`` or ``"walk"``."""
+    rows = rows.contiguous()
+    t = rows.shape[0]
+    _, n, dk, dv = state.shape
+    f32, dev = torch.float32, rows.device
+    assert state.dtype == norm_w.dtype == powers.dtype == f32 and state.is_contiguous() and powers.is_contiguous()
+    assert rows.shape[1] == 2 * n * (dk + dv) and norm_w.numel() == n * dv and powers.shape[0] == n
+    if kernel is None:
+        kernel = "step" if meta.max_q_len == 1 else "walk"
+    if kernel == "step" and meta.max_q_len != 1:
+        raise ValueError("the decode kernel does not cover this step")
+    out = torch.empty(t, n * dv, dtype=rows.dtype, device=dev)
+    o32 = torch.empty(t, n * dv, dtype=f32, device=dev)
+    ptr = lambda x: None if x is None else _p(x).value
+    p = LightningParams(*[ptr(x) for x in (rows, None, powers, state, norm_w, out, o32, None, meta.q_start, meta.q_len, meta.past_len, meta.slot_ids,
+                                           Workspace.get(dev).status)],
+                        rows.shape[1], n, dk, dv, n * dk, 2 * n * dk, n * (2 * dk + dv), dv_real, powers.shape[1], t, meta.num_seqs, 1, 0, eps)
+    code, L, ref_p = _dtype_code(rows), lib(), ctypes.byref(p)
+    if kernel == "step":
+        _check(L.telb_lightning_step(ref_p, c_int(code), _stream()), "lightning_step", 2)
+    else:
+        _check(L.telb_lightning_walk(ref_p, c_int(code), _stream()), "lightning_walk", 2)
+    return out
+
+
 class ChannelDeltaParams(ctypes.Structure):
     """Host mirror of ``ChannelDeltaParams`` (``csrc/kernels/channel_delta.cu``)."""
     _fields_ = [(n, c_vp) for n in ("qkv", "decay", "gate", "beta", "conv_w", "a_log", "decay_bias", "norm_w", "conv_state", "state", "blocks",
                                     "v_blocks", "o", "out", "q_start", "q_len", "past_len", "slot_ids", "seq_ids", "status")] + \
                [(n, c_int) for n in ("tokens", "num_seqs", "heads", "kv_heads", "dk", "dv", "dk_real", "dv_real", "taps", "channels", "ld_decay", "ld_gate",
-                                     "gate_f32")] + [("eps", c_float)]
+                                     "gate_f32", "ld_qkv", "ld_beta", "ld_out", "head_decay", "gate_silu")] + [("eps", c_float), ("mult", c_float)]
+
+
+def _pitched(x: torch.Tensor) -> torch.Tensor:
+    """``x`` itself when its rows are contiguous and 16-byte aligned (they may lie further apart), else a copy."""
+    return x if x.stride(1) == 1 and x.stride(0) % 8 == 0 and x.storage_offset() % 8 == 0 else x.contiguous()
 
 
 def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, meta: StepMeta, spec, eps: float,
-                  kernel: Optional[str] = None) -> torch.Tensor:
+                  kernel: Optional[str] = None, out: Optional[torch.Tensor] = None, mult: float = 1.0) -> torch.Tensor:
     """See :func:`ops.channel_delta`.  Steps of one row per sequence run the fused decode kernel, longer ones the walk over rows;
     ``kernel`` forces ``"decode"`` or ``"walk"``."""
-    qkv, beta = qkv.contiguous(), beta.contiguous()
+    qkv = _pitched(qkv)
     t, ch = qkv.shape
     n, nk, dk, dv = spec.num_heads, spec.num_kv_heads, spec.k_pad, spec.v_pad
     f32 = torch.float32
     assert ch == spec.conv_dim and conv_w.shape == (ch, spec.conv_kernel) and conv_w.dtype == conv_state.dtype == qkv.dtype
     assert state.dtype == decay.dtype == beta.dtype == a_log.dtype == decay_bias.dtype == norm_w.dtype == f32
     assert state.shape[1:] == (n, dk, dv) and state.is_contiguous() and conv_state.is_contiguous() and conv_w.is_contiguous()
-    assert decay.shape == (t, n * dk) and gate.shape == (t, n * dv) and beta.shape == (t, n) and decay.stride(1) == gate.stride(1) == 1
-    if gate.dtype not in (qkv.dtype, f32) or decay.stride(0) % 4 or gate.stride(0) % 4:
+    assert decay.shape == (t, n if spec.head_decay else n * dk) and decay_bias.numel() == decay.shape[1]
+    assert gate.shape == (t, n * dv) and beta.shape == (t, n) and decay.stride(1) == gate.stride(1) == beta.stride(1) == 1
+    if gate.dtype not in (qkv.dtype, f32) or (not spec.head_decay and decay.stride(0) % 4) or gate.stride(0) % 4:
         raise TypeError(f"channel_delta: gate {gate.dtype} for {qkv.dtype} rows, row pitches {decay.stride(0)}, {gate.stride(0)}")
     decode_ok = meta.max_q_len == 1 and dk <= 128 and dv <= 128
     if kernel is None:
@@ -1100,17 +1221,19 @@ def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, con
     if kernel == "decode" and not decode_ok:
         raise ValueError("the decode kernel does not cover this step")
     dev = qkv.device
-    out = torch.empty(t, n * dv, dtype=qkv.dtype, device=dev)
+    if out is None:
+        out = torch.empty(t, n * dv, dtype=qkv.dtype, device=dev)
+    assert out.shape == (t, n * dv) and out.dtype == qkv.dtype and out.stride(1) == 1 and out.stride(0) % 8 == 0
     blocks = v_blocks = o = None
     if kernel == "walk":                       # blocks of four tokens, counted from the start of every portion
         nb = t // 4 + meta.num_seqs + 1
         blocks, v_blocks = torch.empty(nb, n, 13 * dk + 32, dtype=f32, device=dev), torch.empty(nb, n, dv, 4, dtype=qkv.dtype, device=dev)
-        o = torch.empty_like(out)
+        o = torch.empty(t, n * dv, dtype=qkv.dtype, device=dev)
     ptr = lambda x: None if x is None else _p(x).value
     p = ChannelDeltaParams(*[ptr(x) for x in (qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, blocks, v_blocks, o, out,
                                               meta.q_start, meta.q_len, meta.past_len, meta.slot_ids, meta.seq_ids, Workspace.get(dev).status)],
                            t, meta.num_seqs, n, nk, dk, dv, spec.head_k_dim, spec.head_v_dim, spec.conv_kernel, ch, decay.stride(0), gate.stride(0),
-                           int(gate.dtype == f32), eps)
+                           int(gate.dtype == f32), qkv.stride(0), beta.stride(0), out.stride(0), int(spec.head_decay), int(spec.silu_gate), eps, mult)
     launches = (1 if kernel == "decode" else 4) + int(spec.conv_kernel > 1 and (kernel == "walk" or n != nk))
     _check(lib().telb_channel_delta(ctypes.byref(p), c_int(int(kernel == "decode")), c_int(_dtype_code(qkv)), _stream()), "channel_delta", launches)
     return out
@@ -1128,6 +1251,29 @@ def unit_kv_write(qkv, kv_layer, meta: StepMeta, temperature, num_q_heads: int, 
         _p(qkv), _p(q), _p(kv_layer), _p(temperature), _p(meta.positions), _p(meta.seq_ids), _p(meta.q_start), _p(meta.past_len), _p(meta.page_table),
         c_int(t), c_int(meta.page_table.shape[1]), c_int(meta.page_size), c_int(num_q_heads), c_int(num_kv_heads), c_int(head_dim), c_int(real_dim),
         c_float(eps), c_int(_dtype_code(qkv)), _stream()), "unit_kv_write")
+    return q
+
+
+class TurnedKvParams(ctypes.Structure):
+    """Host mirror of ``TurnedKvParams`` (``csrc/kernels/latent.cu``)."""
+    _fields_ = [(n, c_vp) for n in ("rows", "q_out", "kv", "key_table", "value_table", "q_norm", "k_norm", "positions", "seq_ids", "q_start", "past_len",
+                                    "page_table")] + \
+               [(n, c_int) for n in ("ld", "tokens", "max_pages", "page_size", "hq", "hkv", "d", "real")] + [("eps", c_float)]
+
+
+def turned_kv_write(rows, kv_layer, meta: StepMeta, key_table, value_table, q_norm, k_norm, spec, eps: float):
+    rows = _pitched(rows)
+    t, hq, hkv, d = rows.shape[0], spec.num_heads, spec.num_kv_heads, spec.pad
+    f32 = torch.float32
+    assert rows.shape[1] == (hq + 2 * hkv) * d and kv_layer.is_contiguous() and kv_layer.dtype == rows.dtype
+    assert kv_layer.shape[1:] == (2, hkv, meta.page_size, d)
+    assert all(x.dtype == f32 and x.is_contiguous() for x in (key_table, value_table, q_norm, k_norm))
+    assert key_table.shape[1] == value_table.shape[1] == d and q_norm.numel() == hq * d and k_norm.numel() == hkv * d
+    q = torch.empty(t, hq, d, dtype=rows.dtype, device=rows.device)
+    p = TurnedKvParams(*[_p(x).value for x in (rows, q, kv_layer, key_table, value_table, q_norm, k_norm, meta.positions, meta.seq_ids, meta.q_start,
+                                               meta.past_len, meta.page_table)],
+                       rows.stride(0), t, meta.page_table.shape[1], meta.page_size, hq, hkv, d, spec.head_dim, eps)
+    _check(lib().telb_turned_kv_write(ctypes.byref(p), c_int(_dtype_code(rows)), _stream()), "turned_kv_write")
     return q
 
 

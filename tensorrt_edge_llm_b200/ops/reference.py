@@ -260,7 +260,7 @@ def gather_kv(kv_layer: torch.Tensor, page_table_row: torch.Tensor, length: int,
 
 def paged_attention(q: torch.Tensor, kv_layer: torch.Tensor, meta: StepMeta, scale: float,
                     sliding_window: Optional[int] = None, sinks: Optional[torch.Tensor] = None, causal: bool = True,
-                    chunk: int = 0) -> torch.Tensor:
+                    chunk: int = 0, back: Optional[tuple] = None) -> torch.Tensor:
     """Causal GQA attention of the step's rows over the paged cache (which already holds this
     step's keys/values).  Row ``i`` of a sequence sees cache slots ``[0, past + i]``
     (bottom-right aligned causal mask), optionally limited to a sliding window, or the tree
@@ -300,7 +300,12 @@ def paged_attention(q: torch.Tensor, kv_layer: torch.Tensor, meta: StepMeta, sca
             pr = torch.softmax(torch.cat([sc, sink], dim=-1), dim=-1)[..., :-1]
         else:
             pr = torch.softmax(sc, dim=-1)
-        out[r0:r0 + ql] = torch.matmul(pr, vf).permute(1, 0, 2).to(q.dtype)
+        o = torch.matmul(pr, vf).permute(1, 0, 2)
+        if back is not None:
+            table, factor = back
+            c, sn = table[past:total].chunk(2, dim=-1)
+            o = _rotate_pairs(o, torch.cat([c, -sn], dim=-1), torch.arange(ql), d) * factor
+        out[r0:r0 + ql] = o.to(q.dtype)
     return out
 
 
@@ -605,16 +610,75 @@ def stream_norm(stream, weight, eps, delta, routed, mult, step, offset, ids, tab
     return x, h.to(dtype)
 
 
+def _part_norm(x, weight, groups, eps):
+    parts = x.reshape(x.shape[0], groups, -1)
+    return (parts * torch.rsqrt(parts.pow(2).mean(-1, keepdim=True) + eps)).reshape(x.shape) * weight
+
+
+def stream_post(stream, delta, weight, groups, eps, meta: StepMeta, dtype, ids, table, bigram, conv, history, out_norm):
+    """See :func:`ops.stream_post`."""
+    seqs = [(int(a), int(n), int(p), int(s)) for a, n, p, s in zip(meta.q_start, meta.q_len, meta.past_len, meta.slot_ids) if int(n)]
+    if stream is None:
+        x = table[ids.long()].float()
+        if bigram is not None:
+            rows = torch.empty(ids.numel(), dtype=torch.int64)
+            for r0, n, past, slot in seqs:
+                cur = ids[r0:r0 + n].long()
+                first = bigram.last[slot].long() if past > 0 else cur[:1]
+                rows[r0:r0 + n] = (torch.cat([first, cur[:-1]]) * bigram.mul_prev + cur * bigram.mul_cur) % bigram.buckets
+                if past == 0:
+                    rows[r0] = bigram.buckets
+                bigram.last[slot] = ids[r0 + n - 1].to(torch.int32)
+            x = x + bigram.table[rows].float()
+    else:
+        x = stream
+    if delta is not None:
+        x = x + _part_norm(delta.float(), weight, groups, eps)
+    if out_norm is not None:
+        return x, _part_norm(x, out_norm, groups, eps).to(dtype)
+    if conv is None:
+        return x, x.to(dtype)
+    h, taps = x.clone(), conv.shape[0]
+    for r0, n, past, slot in seqs:
+        before = history[slot] if taps > 1 and past > 0 else torch.zeros(taps - 1, x.shape[1])
+        seq = torch.cat([before, x[r0:r0 + n]])
+        for j in range(taps):
+            h[r0:r0 + n] += conv[j] * seq[j:j + n]
+        if taps > 1:
+            history[slot] = seq[n:]
+    return x, h.to(dtype)
+
+
+def lightning(rows, norm_w, powers, state, meta: StepMeta, dv_real, eps):
+    """Row by row in fp32 (see :func:`ops.lightning`)."""
+    t, (_, n, dk, dv) = rows.shape[0], state.shape
+    q, k, v, g = rows.float().split([n * dk, n * dk, n * dv, n * dv], dim=-1)
+    q, k, v = (F.silu(x).to(rows.dtype).float().reshape(t, n, -1) for x in (q, k, v))
+    o = torch.zeros(t, n, dv)
+    for s in range(meta.num_seqs):
+        r0, ql, past, slot = int(meta.q_start[s]), int(meta.q_len[s]), int(meta.past_len[s]), int(meta.slot_ids[s])
+        S = state[slot].clone() if past > 0 else torch.zeros(n, dk, dv)
+        for i in range(r0, r0 + ql):
+            S = powers[:, 1, None, None] * S + k[i][:, :, None] * v[i][:, None, :]
+            o[i] = torch.einsum("hkv,hk->hv", S, q[i])
+        if ql:
+            state[slot] = S
+    o = o.reshape(t, n * dv)
+    o = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / (n * dv_real) + eps) * norm_w
+    return (o * torch.sigmoid(g)).to(rows.dtype)
+
+
 # ------------------------------------------------------------------------------------------
 # channel-decay delta rule, unit-norm attention, latent attention
 
 
-def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, meta: StepMeta, spec, eps):
+def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, meta: StepMeta, spec, eps, out=None, mult=1.0):
     """Row by row in fp32 after the short convolutions (see ``csrc/kernels/channel_delta.cu`` for the equations)."""
     t, n, nk, dk, dv = qkv.shape[0], spec.num_heads, spec.num_kv_heads, spec.k_pad, spec.v_pad
     w = conv_w.shape[-1]
     rep = n // nk
-    g = torch.exp(-torch.exp(a_log)[:, None] * F.softplus((decay.float() + decay_bias).reshape(t, n, dk), threshold=80.0))
+    z = (decay.float() + decay_bias).reshape(t, n, -1).expand(t, n, dk)
+    g = torch.exp(-torch.exp(a_log)[:, None] * F.softplus(z, threshold=80.0))
     b = torch.sigmoid(beta.float())
     o = torch.zeros(t, n, dv)
     for s in range(meta.num_seqs):
@@ -638,7 +702,8 @@ def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, con
             o[r0 + i] = torch.einsum("hkv,hk->hv", m, q[i])
         state[slot] = m
     o = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / spec.head_v_dim + eps) * norm_w
-    return (o.reshape(t, n * dv) * torch.sigmoid(gate.float())).to(qkv.dtype)
+    y = (o.reshape(t, n * dv) * (F.silu if spec.silu_gate else torch.sigmoid)(gate.float()) * mult).to(qkv.dtype)
+    return y if out is None else out.copy_(y)
 
 
 def query_temperature(length: int, coef: float, every: float, device="cpu") -> torch.Tensor:
@@ -670,6 +735,17 @@ def _rotate_pairs(x: torch.Tensor, cos_sin: torch.Tensor, positions: torch.Tenso
     x = x.clone()
     x[..., 0:dims:2], x[..., 1:dims:2] = u * c - v * s, v * c + u * s
     return x
+
+
+def turned_kv_write(rows, kv_layer, meta: StepMeta, key_table, value_table, q_norm, k_norm, spec, eps):
+    t, d, hq, hkv, real = rows.shape[0], spec.pad, spec.num_heads, spec.num_kv_heads, spec.head_dim
+    q, k, v = rows.float().split([hq * d, hkv * d, hkv * d], dim=-1)
+    q, k = (x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / (n * real) + eps) * w for x, n, w in ((q, hq, q_norm), (k, hkv, k_norm)))
+    q, k, v = (_rotate_pairs(x.reshape(t, -1, d), table, meta.positions, d) for x, table in ((q, key_table), (k, key_table), (v, value_table)))
+    page, row = _cache_slots(meta, t, rows.device)
+    kv_layer[page, 0, :, row] = k.to(kv_layer.dtype)
+    kv_layer[page, 1, :, row] = v.to(kv_layer.dtype)
+    return q.to(rows.dtype)
 
 
 def latent_write(rows, kv_layer, meta: StepMeta, cos_sin, norm_w, spec, eps):

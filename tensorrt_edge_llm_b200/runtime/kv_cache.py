@@ -16,7 +16,7 @@ from typing import Dict, List, Optional, Sequence
 
 import torch
 
-from ..config import ModelConfig, LAYER_ATTENTION
+from ..config import KV_LAYERS, ModelConfig
 
 
 class PageAllocator:
@@ -78,7 +78,7 @@ class KVCacheManager:
         self.page_size = page_size
         self.max_seats = max_seats
         self.max_pages_per_seq = max_pages_per_seq
-        self.num_layers = num_layers if num_layers is not None else sum(t == LAYER_ATTENTION for t in cfg.layer_types)
+        self.num_layers = num_layers if num_layers is not None else sum(t in KV_LAYERS for t in cfg.layer_types)
         hkv = max(cfg.num_key_value_heads // cfg.tp_size, 1)
         self.dtype = dtype or cfg.compute_dtype
         if kv_dtype in (None, "auto"):
@@ -106,7 +106,7 @@ class KVCacheManager:
         # hybrid models: model layer index → attention pool index, plus the recurrent state pools
         self._attn_index = {}
         for i, t in enumerate(cfg.layer_types):
-            if t == LAYER_ATTENTION:
+            if t in KV_LAYERS:
                 self._attn_index[i] = len(self._attn_index)
         self.recurrent = None
         if cfg.is_hybrid:
