@@ -51,7 +51,8 @@ def _run(cmd: List[str]) -> str:
 # into a library of their own (`libtelb_kernels-<family>.so`) in a fraction of the time of the whole set.
 KERNEL_SETS = {
     "begupel": ["attention_decode_tc5.cu", "attention_simt.cu", "attention_tc5.cu", "attention_tc5_extra.cu", "channel_delta.cu", "elementwise.cu",
-                "gemm_f32.cu", "gemm_skinny_tc5.cu", "gemm_tc5.cu", "latent.cu", "lightning.cu", "nvfp4_host.cu", "stream_post.cu"],
+                "gemm_f32.cu", "gemm_skinny_tc5.cu", "gemm_tc5.cu", "latent.cu", "lightning.cu", "lightning_tc5.cu", "nvfp4_host.cu",
+                "stream_post.cu"],
     "debonex": ["attention_decode_tc5.cu", "attention_latent_tc5.cu", "attention_simt.cu", "attention_tc5.cu", "attention_tc5_extra.cu",
                 "channel_delta.cu", "elementwise.cu", "gemm_f32.cu", "gemm_skinny_tc5.cu", "gemm_tc5.cu", "latent.cu", "nvfp4_host.cu", "stream_norm.cu"],
     "dimesun": ["attention_decode_tc5.cu", "attention_simt.cu", "attention_tc5.cu", "attention_tc5_extra.cu", "elementwise.cu", "gemm_f32.cu",

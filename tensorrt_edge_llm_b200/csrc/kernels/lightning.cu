@@ -4,15 +4,25 @@
 //   S = decay S + k vᵀ,   o = Sᵀ q                       per head; S starts at zero
 //   y = o / rms(o) · w · σ(g)                            rms over all heads of a row together
 //
-// Projections arrive packed as [q | k | v | g] rows in the activation type; state, read-outs and the norm are fp32.  Heads may be padded
-// at the end (zero projection rows): `dv_real` is the number of value features per head that the norm averages over.
+// Projections arrive packed as [q | k | v | g] rows in the activation type; state and read-outs are fp32.  Heads may be padded at the end
+// (zero projection rows).
+//
+// The kernels write u = o · w · σ(g) and the sums of squares of o.  The rms is one number per row, so it commutes with the output
+// projection: whoever adds the projected row to the residual stream divides by it (stream_post.cu), and no pass over the heads of a
+// row is needed here.
 //
 // Here: the walk over the rows of a sequence in order (any size, any type; state tile in shared memory), the decode step (one row per
-// sequence), the norm with its gate, and the activation pass in front of the chunked tensor-core form (lightning_tc5.cu).
+// sequence) and the activation pass in front of the chunked tensor-core form (lightning_tc5.cu).
 #include "host_utils.h"
 #include "lightning_common.cuh"
 
 namespace telb {
+
+__device__ __forceinline__ float lightning_warp_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
 
 constexpr int kWalkCols = 64;          // value columns per CTA of the walk
 constexpr int kWalkThreads = 256;
@@ -26,6 +36,7 @@ __global__ void __launch_bounds__(kWalkThreads) lightning_walk_kernel(const __gr
     float* sq = S + (size_t)p.dk * kWalkCols;        // [dk]
     float* sk = sq + p.dk;                           // [dk]
     float* part = sk + p.dk;                         // [4][64]
+    float* red = part + 4 * kWalkCols;               // [2]
     const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kWalkCols;
     const int ql = p.q_len[seq];
     if (ql <= 0) return;
@@ -51,7 +62,15 @@ __global__ void __launch_bounds__(kWalkThreads) lightning_walk_kernel(const __gr
         }
         part[rg * kWalkCols + c] = acc;
         __syncthreads();
-        if (tid < kWalkCols) p.o32[(t * p.heads + h) * p.dv + c0 + c] = (part[c] + part[64 + c]) + (part[128 + c] + part[192 + c]);
+        if (tid < kWalkCols) {
+            const float o = (part[c] + part[64 + c]) + (part[128 + c] + part[192 + c]);
+            const size_t col = (size_t)h * p.dv + c0 + c;
+            reinterpret_cast<T*>(p.out)[t * p.heads * p.dv + col] = Cvt<T>::from_f(lightning_gate<T>(o, p.norm_w[col], Cvt<T>::to_f(row[p.g_off + col])));
+            const float ss = lightning_warp_sum(o * o);
+            if ((tid & 31) == 0) red[tid >> 5] = ss;
+            named_barrier_sync(1, kWalkCols);
+            if (tid == 0) p.sums[(t * p.heads * p.dv + (size_t)h * p.dv + c0) / 64] = red[0] + red[1];
+        }
     }
     for (int r = rg; r < p.dk; r += 4) gs[(size_t)r * p.dv] = S[r * kWalkCols + c];
 }
@@ -60,12 +79,13 @@ __global__ void __launch_bounds__(kWalkThreads) lightning_walk_kernel(const __gr
 // them, K rows in flight at a time.
 constexpr int kStepThreads = 256;
 template <typename T, int K>
-__global__ void __launch_bounds__(kStepThreads) lightning_step_kernel(const __grid_constant__ LightningParams p) {
+__global__ void __launch_bounds__(kStepThreads, 2) lightning_step_kernel(const __grid_constant__ LightningParams p) {
     pdl_prologue();
     extern __shared__ float sm[];
     float* sq = sm;                                  // [dk]
     float* sk = sq + p.dk;                           // [dk]
     float* part = sk + p.dk;                         // [8][128]
+    __shared__ float red[4];
     const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * 128;
     if (p.q_len[seq] <= 0) return;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -110,69 +130,13 @@ __global__ void __launch_bounds__(kStepThreads) lightning_step_kernel(const __gr
         float o = 0.f;
 #pragma unroll
         for (int w = 0; w < kStepThreads / 32; ++w) o += part[w * 128 + tid];
-        p.o32[(t * p.heads + h) * p.dv + c0 + tid] = o;
+        const size_t col = (size_t)h * p.dv + c0 + tid;
+        reinterpret_cast<T*>(p.out)[t * p.heads * p.dv + col] = Cvt<T>::from_f(lightning_gate<T>(o, p.norm_w[col], Cvt<T>::to_f(row[p.g_off + col])));
+        const float ss = lightning_warp_sum(o * o);
+        if (lane == 0) red[warp] = ss;
+        named_barrier_sync(1, 128);
+        if (tid < 2) p.sums[(t * p.heads * p.dv + (size_t)h * p.dv + c0) / 64 + tid] = red[tid * 2] + red[tid * 2 + 1];
     }
-}
-
-// Norm over all heads of a row, weight and gate; one CTA per row.
-constexpr int kNormThreads = 256;
-template <typename T>
-__global__ void __launch_bounds__(kNormThreads) lightning_norm_kernel(const __grid_constant__ LightningParams p) {
-    pdl_prologue();
-    __shared__ float red[kNormThreads / 32];
-    constexpr int kKeep = 4;                         // four-feature vectors a thread keeps between the passes
-    const int tid = threadIdx.x, width = p.heads * p.dv;
-    const float* o = p.o32 + (size_t)blockIdx.x * width;
-    const T* g = reinterpret_cast<const T*>(p.rows) + (size_t)blockIdx.x * p.ld + p.g_off;
-    T* out = reinterpret_cast<T*>(p.out) + (size_t)blockIdx.x * width;
-    float4 kept[kKeep];
-    float ss = 0.f;
-#pragma unroll
-    for (int k = 0; k < kKeep; ++k) {
-        const int c = (k * kNormThreads + tid) * 4;
-        if (c >= width) break;
-        kept[k] = *reinterpret_cast<const float4*>(o + c);
-        ss += kept[k].x * kept[k].x + kept[k].y * kept[k].y + kept[k].z * kept[k].z + kept[k].w * kept[k].w;
-    }
-    for (int c = (kKeep * kNormThreads + tid) * 4; c < width; c += kNormThreads * 4) {
-        const float4 v = *reinterpret_cast<const float4*>(o + c);
-        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-    }
-#pragma unroll
-    for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
-    __syncthreads();
-    float tot = 0.f;
-#pragma unroll
-    for (int w = 0; w < kNormThreads / 32; ++w) tot += red[w];
-    const float inv = 1.f / sqrtf(tot / (p.heads * p.dv_real) + p.eps);
-    auto finish = [&](int c, const float4& v) {
-        const float4 w = *reinterpret_cast<const float4*>(p.norm_w + c);
-        const float e[4] = {v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w};
-        T y[4];
-        if constexpr (sizeof(T) == 4) {
-#pragma unroll
-            for (int i = 0; i < 4; ++i) y[i] = e[i] / (1.f + expf(-g[c + i]));
-            *reinterpret_cast<float4*>(out + c) = *reinterpret_cast<const float4*>(y);
-        } else {
-            const uint2 u = *reinterpret_cast<const uint2*>(g + c);
-            const T* z = reinterpret_cast<const T*>(&u);
-            float f[4];
-#pragma unroll
-            for (int i = 0; i < 4; ++i) f[i] = __fdividef(e[i], 1.f + __expf(-Cvt<T>::to_f(z[i])));
-            uint2 r;
-            r.x = Cvt<T>::pack2(f[0], f[1]);
-            r.y = Cvt<T>::pack2(f[2], f[3]);
-            *reinterpret_cast<uint2*>(out + c) = r;
-        }
-    };
-#pragma unroll
-    for (int k = 0; k < kKeep; ++k) {
-        const int c = (k * kNormThreads + tid) * 4;
-        if (c >= width) break;
-        finish(c, kept[k]);
-    }
-    for (int c = (kKeep * kNormThreads + tid) * 4; c < width; c += kNormThreads * 4) finish(c, *reinterpret_cast<const float4*>(o + c));
 }
 
 // act = silu(q | k | v), rounded to the activation type: the operands of the chunk kernel's products.
@@ -202,15 +166,8 @@ __global__ void __launch_bounds__(256) lightning_act_kernel(const __grid_constan
 }
 
 template <typename T>
-static int run_norm(const LightningParams& p, cudaStream_t stream) {
-    TELB_LAUNCH("lightning_norm_kernel", (lightning_norm_kernel<T>), dim3(p.tokens), dim3(kNormThreads), 0, stream, p);
-    TELB_CHECK_LAUNCH("lightning_norm_kernel");
-    return 0;
-}
-
-template <typename T>
 static int run_walk(const LightningParams& p, cudaStream_t stream) {
-    const size_t smem = ((size_t)p.dk * kWalkCols + 2 * p.dk + 4 * kWalkCols) * sizeof(float);
+    const size_t smem = ((size_t)p.dk * kWalkCols + 2 * p.dk + 4 * kWalkCols + 2) * sizeof(float);
     static size_t configured = 48 * 1024;
     if (smem > configured) {
         cudaError_t e = cudaFuncSetAttribute(lightning_walk_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -219,7 +176,7 @@ static int run_walk(const LightningParams& p, cudaStream_t stream) {
     }
     TELB_LAUNCH("lightning_walk_kernel", (lightning_walk_kernel<T>), dim3(p.num_seqs, p.heads, p.dv / kWalkCols), dim3(kWalkThreads), smem, stream, p);
     TELB_CHECK_LAUNCH("lightning_walk_kernel");
-    return run_norm<T>(p, stream);
+    return 0;
 }
 
 template <typename T>
@@ -229,7 +186,7 @@ static int run_step(const LightningParams& p, cudaStream_t stream) {
     if (p.dk % 128 == 0) TELB_LAUNCH("lightning_step_kernel", (lightning_step_kernel<T, 16>), grid, dim3(kStepThreads), smem, stream, p);
     else TELB_LAUNCH("lightning_step_kernel", (lightning_step_kernel<T, 8>), grid, dim3(kStepThreads), smem, stream, p);
     TELB_CHECK_LAUNCH("lightning_step_kernel");
-    return run_norm<T>(p, stream);
+    return 0;
 }
 
 }  // namespace telb
@@ -242,36 +199,26 @@ static int check_sizes(const LightningParams* p) {
     return 0;
 }
 
-// Walk over every sequence's rows, then norm and gate.  dtype: 0 fp16, 1 bf16, 2 fp32.
+// Walk over every sequence's rows.  dtype: 1 bf16, 2 fp32 (un-normed rows need bf16's range).
 extern "C" int telb_lightning_walk(const LightningParams* p, int dtype, cudaStream_t stream) {
     if (p->num_seqs <= 0 || p->tokens <= 0) return 0;
     if (check_sizes(p)) return -1;
-    if (dtype == 2) return run_walk<float>(*p, stream);
-    return dtype == 1 ? run_walk<__nv_bfloat16>(*p, stream) : run_walk<__half>(*p, stream);
+    return dtype == 2 ? run_walk<float>(*p, stream) : run_walk<__nv_bfloat16>(*p, stream);
 }
 
 // Every sequence has at most one row (decode).
 extern "C" int telb_lightning_step(const LightningParams* p, int dtype, cudaStream_t stream) {
     if (p->num_seqs <= 0 || p->tokens <= 0) return 0;
     if (check_sizes(p)) return -1;
-    if (dtype == 2) return run_step<float>(*p, stream);
-    return dtype == 1 ? run_step<__nv_bfloat16>(*p, stream) : run_step<__half>(*p, stream);
+    return dtype == 2 ? run_step<float>(*p, stream) : run_step<__nv_bfloat16>(*p, stream);
 }
 
-// Norm and gate of the read-outs in p->o32.
-extern "C" int telb_lightning_norm(const LightningParams* p, int dtype, cudaStream_t stream) {
-    if (p->tokens <= 0) return 0;
-    if (dtype == 2) return run_norm<float>(*p, stream);
-    return dtype == 1 ? run_norm<__nv_bfloat16>(*p, stream) : run_norm<__half>(*p, stream);
-}
-
-// p->act = silu(q | k | v), 16-bit types.
-extern "C" int telb_lightning_act(const LightningParams* p, int is_bf16, cudaStream_t stream) {
+// p->act = silu(q | k | v), bf16.
+extern "C" int telb_lightning_act(const LightningParams* p, cudaStream_t stream) {
     if (p->tokens <= 0) return 0;
     const long long blocks = ((long long)p->tokens * (p->g_off / 8) + 255) / 256;
     const dim3 grid((unsigned)(blocks < 148 * 32 ? blocks : 148 * 32));
-    if (is_bf16) TELB_LAUNCH("lightning_act_kernel", (lightning_act_kernel<__nv_bfloat16>), grid, dim3(256), 0, stream, *p);
-    else TELB_LAUNCH("lightning_act_kernel", (lightning_act_kernel<__half>), grid, dim3(256), 0, stream, *p);
+    TELB_LAUNCH("lightning_act_kernel", (lightning_act_kernel<__nv_bfloat16>), grid, dim3(256), 0, stream, *p);
     TELB_CHECK_LAUNCH("lightning_act_kernel");
     return 0;
 }

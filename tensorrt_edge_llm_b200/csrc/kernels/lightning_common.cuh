@@ -14,16 +14,15 @@ struct LightningParams {
     const float* powers;       // [heads, n_powers]: decay^0, decay^1, ...
     float* state;              // [slots, heads, dk, dv] fp32
     const float* norm_w;       // [heads * dv] fp32
-    void* out;                 // [T, heads * dv]
-    float* o32;                // [T, heads * dv] fp32 scratch: read-outs
+    void* out;                 // [T, heads * dv]: read-outs times weight and gate
+    float* sums;               // [T, heads * dv / 64]: squares of 64 read-outs each
     float* carry;              // [sequences, heads, segments, dk, dv] fp32 scratch: states in front of the segments (chunk kernel)
     const int* q_start;
     const int* q_len;
     const int* past_len;
     const int* slot_ids;
     int* status;
-    int ld, heads, dk, dv, k_off, v_off, g_off, dv_real, n_powers, tokens, num_seqs, segments, seg_chunks;
-    float eps;
+    int ld, heads, dk, dv, k_off, v_off, g_off, n_powers, tokens, num_seqs, segments, seg_chunks;
 };
 
 // silu in the precision of the projection it belongs to
@@ -31,6 +30,13 @@ template <typename T>
 __device__ __forceinline__ float lightning_silu(float x) {
     if constexpr (sizeof(T) == 4) return x / (1.f + expf(-x));
     else return Cvt<T>::to_f(Cvt<T>::from_f(__fdividef(x, 1.f + __expf(-x))));
+}
+
+// weight and sigmoid gate of a read-out
+template <typename T>
+__device__ __forceinline__ float lightning_gate(float o, float w, float g) {
+    if constexpr (sizeof(T) == 4) return o * w / (1.f + expf(-g));
+    else return __fdividef(o * w, 1.f + __expf(-g));
 }
 
 }  // namespace telb

@@ -1,7 +1,8 @@
 // The fp32 residual stream of blocks that are normed behind their sublayers.  Everything that lies between two sublayers is one kernel:
 //
 //   source   x = table[id] + bigram[row(previous id, id)] (first call) or the running fp32 stream
-//   update   x += y / rms(y) * w                       y: sublayer output; each of `groups` equal parts of a row has its own rms
+//   update   x += y / rms(y) * w                       y: sublayer output; each of `groups` equal parts of a row has its own rms.  With
+//                                                       `sums` the row is first divided by the rms of the row that was projected to y
 //   output   h = x                                     for a feed-forward                                  (post_row_kernel)
 //            h = x / rms(x) * w'                       same parts, for the head                            (post_row_kernel)
 //            h = x + Σ_j c[j] ∘ x_{t - taps + 1 + j}   causal convolution over time, for a mixer           (post_conv_kernel)
@@ -26,6 +27,7 @@ struct StreamPostParams {
     const float* x_in;           // [T, width] when ids is null
     const void* delta;           // [T, width] or null
     const float* weight;         // [width], with delta
+    const float* sums;           // [T, n_sums]: sums of squares of the row behind delta, or null
     const float* conv;           // [taps, width] or null
     float* history;              // [slots, taps - 1, width], oldest first
     const float* out_norm;       // [width] or null
@@ -37,7 +39,7 @@ struct StreamPostParams {
     const int* slot_ids;
     const int* seq_ids;
     long long buckets, mul_prev, mul_cur;
-    int vocab, width, groups, tokens, taps, block_rows;
+    int vocab, width, groups, tokens, taps, block_rows, n_sums, sum_count;      // sum_count: features of that row
     float eps;
 };
 
@@ -71,6 +73,14 @@ __device__ __forceinline__ float post_warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
     return v;
+}
+
+// One over the root mean square of the row that was projected to row `row` of delta (every warp computes it).
+__device__ __forceinline__ float row_scale(const StreamPostParams& p, size_t row) {
+    if (!p.sums) return 1.f;
+    float s = 0.f;
+    for (int i = threadIdx.x & 31; i < p.n_sums; i += 32) s += p.sums[row * p.n_sums + i];
+    return 1.f / sqrtf(post_warp_sum(s) / p.sum_count + p.eps);
 }
 
 // Divide every part of R rows by its root mean square, in place.  Thread i of N holds features 4 (e N + i) .. + 3 of each row.  Parts that are
@@ -156,6 +166,7 @@ __global__ void __launch_bounds__(N) post_row_kernel(const __grid_constant__ Str
     const size_t row = (size_t)blockIdx.x * p.width;
     const int tid = threadIdx.x;
     float x[1][E][4], d[1][E][4];
+    const float scale = row_scale(p, blockIdx.x);
 #pragma unroll
     for (int e = 0; e < E; ++e) {
         const int c = (e * N + tid) * 4;
@@ -164,6 +175,8 @@ __global__ void __launch_bounds__(N) post_row_kernel(const __grid_constant__ Str
         if (c >= p.width) continue;
         get4(p.x_in + row + c, x[0][e]);
         if (p.delta) get4(reinterpret_cast<const T*>(p.delta) + row + c, d[0][e]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) d[0][e][i] *= scale;
     }
     if (p.delta) norm_parts<N, E, 1>(p, d, red, 0);
 #pragma unroll
@@ -244,6 +257,7 @@ __global__ void __launch_bounds__(N) post_conv_kernel(const __grid_constant__ St
                 for (int r = 0; r < R; ++r) {
                     const bool live = j + r < j1;
                     const size_t row = (size_t)(t0 + j + r) * p.width;
+                    const float scale = live ? row_scale(p, t0 + j + r) : 1.f;
                     int id = 0;
                     long long pair = 0;
                     if (p.ids && live) {
@@ -275,6 +289,8 @@ __global__ void __launch_bounds__(N) post_conv_kernel(const __grid_constant__ St
                             get4(p.x_in + row + c, x[r][e]);
                         }
                         if (p.delta) get4(reinterpret_cast<const T*>(p.delta) + row + c, d[r][e]);
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) d[r][e][i] *= scale;
                     }
                 }
                 if (p.delta) norm_parts<N, E, R>(p, d, red, turn++);
@@ -378,7 +394,7 @@ static int run_post(const StreamPostParams& p, cudaStream_t stream) {
 
 using namespace telb;
 
-// dtype: 0 fp16, 1 bf16, 2 fp32 (of the tables, delta and h).  With a convolution, p->block_rows is 1 (then every sequence has at most one
+// dtype: 1 bf16, 2 fp32 (of the tables, delta and h; the un-normed stream needs bf16's range).  With a convolution, p->block_rows is 1 (then every sequence has at most one
 // row) or at least 8.
 extern "C" int telb_stream_post(const StreamPostParams* pp, int dtype, cudaStream_t stream) {
     const StreamPostParams& p = *pp;
@@ -397,6 +413,6 @@ extern "C" int telb_stream_post(const StreamPostParams* pp, int dtype, cudaStrea
     } else if (p.ids) {
         return fail("telb_stream_post: token ids enter through the convolution form");
     }
-    if (dtype == 2) return run_post<float>(p, stream);
-    return dtype == 1 ? run_post<__nv_bfloat16>(p, stream) : run_post<__half>(p, stream);
+    if (p.sums && (!p.delta || p.n_sums < 1 || p.sum_count < 1)) return fail("telb_stream_post: sums belong to an update");
+    return dtype == 2 ? run_post<float>(p, stream) : run_post<__nv_bfloat16>(p, stream);
 }

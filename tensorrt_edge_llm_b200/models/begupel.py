@@ -67,10 +67,11 @@ class BegupelLayer(nn.Module):
             self.mlp_norm = PartNorm(cfg.hidden_size)
             self.mlp = GatedMLP(cfg, spec.ff, act=spec.ff_act, bias=spec.ff_bias)
 
-    def mix(self, h: torch.Tensor, meta: StepMeta, cache, table) -> torch.Tensor:
+    def mix(self, h: torch.Tensor, meta: StepMeta, cache, table):
+        """``(output, sums of the row behind it that it still has to be divided by, or None)``."""
         if self.kind == LAYER_LIGHTNING:
             return self.mixer(h, meta, cache.recurrent, self.idx)
-        return self.mixer(h, meta, cache, table, self.idx)
+        return self.mixer(h, meta, cache, table, self.idx), None
 
 
 class BegupelTransformer(nn.Module):
@@ -108,11 +109,11 @@ class BegupelTransformer(nn.Module):
         x, h = step(None, None, None, **self.source(ids, state), **self.conv_args(0, state))
         taps, last = [], len(self.layers) - 1
         for i, layer in enumerate(self.layers):
-            y, norm = layer.mix(h, meta, cache, tables.get(i)), layer.norm
+            (y, sums), norm = layer.mix(h, meta, cache, tables.get(i)), layer.norm
             if layer.mlp is not None:
-                x, h = step(x, y, norm)
-                y, norm = layer.mlp(h), layer.mlp_norm
-            x, h = step(x, y, norm, **(dict(out_norm=self.norm.weight) if i == last else self.conv_args(i + 1, state)))
+                x, h = step(x, y, norm, sums=sums)
+                y, sums, norm = layer.mlp(h), None, layer.mlp_norm
+            x, h = step(x, y, norm, sums=sums, **(dict(out_norm=self.norm.weight) if i == last else self.conv_args(i + 1, state)))
             if rec is not None and i < last:
                 rec["inputs", i + 1] = x
             if i in capture_layers:
@@ -131,6 +132,8 @@ class BegupelCausalLM(HybridCausalLM):
             raise NotImplementedError("quantised weights are not built for the begupel family")
         if cfg.hidden_size % 8:
             raise ValueError("the model width must be a multiple of 8")
+        if cfg.dtype == "float16":
+            raise ValueError("the begupel family runs in bfloat16 or float32: rows that no norm has scaled leave the range of float16")
         super().__init__(cfg, comm)
         self.lm_head = Fp32OutLinear(cfg.hidden_size, [cfg.vocab_size], dtype=cfg.compute_dtype)
         self._tables: Dict[tuple, torch.Tensor] = {}

@@ -392,14 +392,15 @@ class ChannelDeltaMixer(nn.Module):
 
 
 class LightningMixer(nn.Module):
-    """Linear attention with a constant decay per head: q, k, v and the output gate from one product; silu, recurrence, the norm over
-    all heads and the gate are one op (``ops.lightning``); state in fp32 rows indexed by seat."""
+    """Linear attention with a constant decay per head: q, k, v and the output gate from one product; silu, recurrence, norm weight and
+    gate are one op (``ops.lightning``); state in fp32 rows indexed by seat.  The root mean square over all heads of a row commutes with
+    the output projection: ``forward`` returns the projected rows and the sums that their consumer divides by."""
 
     POWERS = 256          # decay^0 .. decay^POWERS, rounded once from double
 
     def __init__(self, cfg: ModelConfig, spec, prefix: str):
         super().__init__()
-        self.spec, self.prefix, self.eps = spec, prefix, cfg.rms_norm_eps
+        self.spec, self.prefix = spec, prefix
         h, n, dt = cfg.hidden_size, spec.num_heads, cfg.compute_dtype
         self.qkvg_proj = HeadLinear(h, 0, out_heads=[(n, spec.head_k_dim, spec.k_pad), (n, spec.head_k_dim, spec.k_pad),
                                                      (n, spec.head_v_dim, spec.v_pad), (n, spec.head_v_dim, spec.v_pad)],
@@ -423,10 +424,11 @@ class LightningMixer(nn.Module):
         rows = self.qkvg_proj(x)
         if state.record is not None:
             state.record[run] = rows
-        return self.o_proj(self._recur(rows, meta, state, run))
+        u, sums = self._recur(rows, meta, state, run)
+        return self.o_proj(u), (sums, self.spec.num_heads * self.spec.head_v_dim)
 
     def _recur(self, rows, meta, state, run):
-        return ops.lightning(rows, self.out_norm, self.decay_powers, state.lightning[run], meta, self.spec.head_v_dim, self.eps)
+        return ops.lightning(rows, self.out_norm, self.decay_powers, state.lightning[run], meta)
 
     @torch.no_grad()
     def replay(self, saved, rows: torch.Tensor, meta: StepMeta, state: RecurrentState, run: int) -> None:

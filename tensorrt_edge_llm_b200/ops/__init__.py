@@ -214,24 +214,27 @@ class Bigram:
     mul_cur: int
 
 
-def stream_post(stream, delta, weight, groups, eps, meta, dtype, *, ids=None, table=None, bigram=None, conv=None, history=None, out_norm=None):
+def stream_post(stream, delta, weight, groups, eps, meta, dtype, *, ids=None, table=None, bigram=None, conv=None, history=None, out_norm=None, sums=None):
     """Advance the fp32 residual stream by a normed sublayer output and write what the next sublayer reads: ``(stream, h)``.
 
     ``stream`` (or ``table[ids]`` plus the row of ``bigram`` when it is ``None``) ``+ norm(delta) * weight``; the norm divides each of ``groups``
-    equal parts of a row by its own root mean square.  ``h`` in ``dtype`` is the stream itself; with ``conv`` ``[taps, width]`` (fp32) the
+    equal parts of a row by its own root mean square.  ``sums``: ``(partial sums of squares [T, n], features)`` of the row that was projected
+    to ``delta``, which still has to be divided by that row's root mean square.  ``h`` in ``dtype`` is the stream itself; with ``conv`` ``[taps, width]`` (fp32) the
     stream plus its causal convolution over time, whose ``history`` ``[seats, taps - 1, width]`` (fp32) is advanced; with ``out_norm`` the norm
     of the stream times that weight."""
     t = ids if stream is None else stream
     f = cuda_ops().stream_post if t.is_cuda else ref.stream_post
-    return f(stream, delta, weight, groups, eps, meta, dtype, ids, table, bigram, conv, history, out_norm)
+    return f(stream, delta, weight, groups, eps, meta, dtype, ids, table, bigram, conv, history, out_norm, sums)
 
 
-def lightning(rows, norm_w, powers, state, meta, dv_real, eps):
-    """Linear attention with a constant decay per head over packed ``[q | k | v | g]`` rows: silu on q, k and v, the recurrence, an RMS norm
-    over all heads of a row, and the sigmoid of g: ``[T, heads · dv]``.  ``powers`` ``[heads, n + 1]``: powers of the decays from 0 on;
-    ``state`` ``[seats, heads, dk, dv]`` is advanced in place; ``dv_real``: value features of a padded head."""
+def lightning(rows, norm_w, powers, state, meta):
+    """Linear attention with a constant decay per head over packed ``[q | k | v | g]`` rows: silu on q, k and v, the recurrence, weight and
+    sigmoid gate.  Returns ``(u [T, heads · dv], sums [T, heads · dv / 64])``: the gated read-outs before the RMS norm over all heads of a
+    row, and sums of squares of the read-outs; the norm's division commutes with the output projection and is left to the consumer
+    (:func:`stream_post`).  ``powers`` ``[heads, n + 1]``: powers of the decays from 0 on; ``state`` ``[seats, heads, dk, dv]`` is
+    advanced in place."""
     f = cuda_ops().lightning if rows.is_cuda else ref.lightning
-    return f(rows, norm_w, powers, state, meta, dv_real, eps)
+    return f(rows, norm_w, powers, state, meta)
 
 
 def moe_route_chosen(logits, top_k):

@@ -335,10 +335,10 @@ def stream_norm(stream, weight, eps: float, delta, routed, mult: float, step, of
 
 class StreamPostParams(ctypes.Structure):
     """Host mirror of ``StreamPostParams`` (``csrc/kernels/stream_post.cu``)."""
-    _fields_ = [(n, c_vp) for n in ("ids", "table", "bigram", "last", "x_in", "delta", "weight", "conv", "history", "out_norm", "x_out", "h", "q_start",
+    _fields_ = [(n, c_vp) for n in ("ids", "table", "bigram", "last", "x_in", "delta", "weight", "sums", "conv", "history", "out_norm", "x_out", "h", "q_start",
                                     "q_len", "past_len", "slot_ids", "seq_ids")] + \
                [(n, c_ll) for n in ("buckets", "mul_prev", "mul_cur")] + \
-               [(n, c_int) for n in ("vocab", "width", "groups", "tokens", "taps", "block_rows")] + [("eps", c_float)]
+               [(n, c_int) for n in ("vocab", "width", "groups", "tokens", "taps", "block_rows", "n_sums", "sum_count")] + [("eps", c_float)]
 
 
 def _conv_block_rows(meta: StepMeta, tokens: int) -> int:
@@ -348,9 +348,12 @@ def _conv_block_rows(meta: StepMeta, tokens: int) -> int:
     return 8 if tokens <= 148 * 2 * 8 else 16 if tokens <= 148 * 4 * 16 else 32
 
 
-def stream_post(stream, delta, weight, groups: int, eps: float, meta: StepMeta, dtype, ids, table, bigram, conv, history, out_norm):
+def stream_post(stream, delta, weight, groups: int, eps: float, meta: StepMeta, dtype, ids, table, bigram, conv, history, out_norm,
+                sums=None):
     """See :func:`ops.stream_post`."""
     f32 = torch.float32
+    if dtype not in (torch.bfloat16, f32):
+        raise TypeError(f"stream_post: the un-normed stream leaves in bf16 or fp32, not {dtype}")
     if stream is None:
         t, width, dev = ids.numel(), table.shape[1], table.device
         ids = ids.to(torch.int32).contiguous()
@@ -365,6 +368,8 @@ def stream_post(stream, delta, weight, groups: int, eps: float, meta: StepMeta, 
     if delta is not None:
         delta = delta.contiguous()
         assert delta.dtype == dtype and delta.shape == (t, width) and weight.dtype == f32 and weight.numel() == width
+    partial, count = sums if sums is not None else (None, 0)
+    assert partial is None or (partial.dtype == f32 and partial.is_contiguous() and partial.shape[0] == t and delta is not None)
     taps = 0 if conv is None else conv.shape[0]
     if conv is not None:
         assert conv.dtype == f32 and conv.is_contiguous() and conv.shape[1] == width and out_norm is None
@@ -373,12 +378,12 @@ def stream_post(stream, delta, weight, groups: int, eps: float, meta: StepMeta, 
     h = torch.empty(t, width, dtype=dtype, device=dev)
     ptr = lambda v: None if v is None else _p(v).value
     b = bigram
-    p = StreamPostParams(*[ptr(v) for v in (ids, table, None if b is None else b.table, None if b is None else b.last, stream, delta, weight, conv,
+    p = StreamPostParams(*[ptr(v) for v in (ids, table, None if b is None else b.table, None if b is None else b.last, stream, delta, weight, partial, conv,
                                             history if taps > 1 else None, out_norm, x, h, meta.q_start, meta.q_len, meta.past_len, meta.slot_ids,
                                             meta.seq_ids)],
                          *((0, 0, 0) if b is None else (b.buckets, b.mul_prev, b.mul_cur)), 0 if table is None else table.shape[0], width, groups, t, taps,
-                         _conv_block_rows(meta, t) if taps else 1, eps)
-    code = 2 if dtype == f32 else int(dtype == torch.bfloat16)
+                         _conv_block_rows(meta, t) if taps else 1, 0 if partial is None else partial.shape[1], count, eps)
+    code = 2 if dtype == f32 else 1
     _check(lib().telb_stream_post(ctypes.byref(p), c_int(code), _stream()), "stream_post")
     return x, h
 
@@ -1155,36 +1160,60 @@ def mlstm(qkvg, gates, norm_w, state, norm_state, meta: StepMeta, scale: float, 
 
 class LightningParams(ctypes.Structure):
     """Host mirror of ``LightningParams`` (``csrc/kernels/lightning_common.cuh``)."""
-    _fields_ = [(n, c_vp) for n in ("rows", "act", "powers", "state", "norm_w", "out", "o32", "carry", "q_start", "q_len", "past_len", "slot_ids", "status")] + \
-               [(n, c_int) for n in ("ld", "heads", "dk", "dv", "k_off", "v_off", "g_off", "dv_real", "n_powers", "tokens", "num_seqs", "segments",
-                                     "seg_chunks")] + [("eps", c_float)]
+    _fields_ = [(n, c_vp) for n in ("rows", "act", "powers", "state", "norm_w", "out", "sums", "carry", "q_start", "q_len", "past_len", "slot_ids", "status")] + \
+               [(n, c_int) for n in ("ld", "heads", "dk", "dv", "k_off", "v_off", "g_off", "n_powers", "tokens", "num_seqs", "segments", "seg_chunks")]
 
 
-def lightning(rows, norm_w, powers, state, meta: StepMeta, dv_real: int, eps: float, kernel: Optional[str] = None) -> torch.Tensor:
-    """See :func:`ops.lightning`.  Steps of one row per sequence run the decode kernel, longer ones the walk row by row; ``kernel`` forces
-    ``"step"`` or ``"walk"``."""
+LIGHTNING_TC_MIN_Q = 16      # steps whose longest sequence has at least this many new rows take the chunked tensor-core kernel
+
+
+def _lightning_segments(meta: StepMeta, tiles: int) -> Tuple[int, int]:
+    """``(segments, chunks per segment)`` of the longest sequence: few (sequence, head, value tile) triples are cut until about every SM has one."""
+    chunks = (meta.max_q_len + 127) // 128
+    want = max(1, 148 // tiles)
+    if want < 2 or chunks < 4:
+        return 1, chunks
+    per = max(2, (chunks + want - 1) // want)
+    return (chunks + per - 1) // per, per
+
+
+def lightning(rows, norm_w, powers, state, meta: StepMeta, kernel: Optional[str] = None, segments: Optional[Tuple[int, int]] = None):
+    """See :func:`ops.lightning`.  Steps of one row per sequence run the decode kernel, longer ones the chunked tensor-core kernel (bf16) or
+    the walk row by row; ``kernel`` forces ``"step"``, ``"chunk"`` or ``"walk"``."""
     rows = rows.contiguous()
     t = rows.shape[0]
     _, n, dk, dv = state.shape
     f32, dev = torch.float32, rows.device
+    if rows.dtype not in (torch.bfloat16, f32):
+        raise TypeError(f"lightning: un-normed rows leave in bf16 or fp32, not {rows.dtype}")
     assert state.dtype == norm_w.dtype == powers.dtype == f32 and state.is_contiguous() and powers.is_contiguous()
     assert rows.shape[1] == 2 * n * (dk + dv) and norm_w.numel() == n * dv and powers.shape[0] == n
+    chunk_ok = rows.dtype == torch.bfloat16 and dk in (64, 128) and powers.shape[1] > 128
     if kernel is None:
-        kernel = "step" if meta.max_q_len == 1 else "walk"
-    if kernel == "step" and meta.max_q_len != 1:
-        raise ValueError("the decode kernel does not cover this step")
+        kernel = "step" if meta.max_q_len == 1 else "chunk" if chunk_ok and meta.max_q_len >= LIGHTNING_TC_MIN_Q else "walk"
+    if (kernel == "step" and meta.max_q_len != 1) or (kernel == "chunk" and not chunk_ok):
+        raise ValueError(f"the {kernel} kernel does not cover this step")
     out = torch.empty(t, n * dv, dtype=rows.dtype, device=dev)
-    o32 = torch.empty(t, n * dv, dtype=f32, device=dev)
+    sums = torch.empty(t, n * dv // 64, dtype=f32, device=dev)
+    act = carry = None
+    segs, per, launches = 1, 0, 1
+    if kernel == "chunk":
+        segs, per = segments or _lightning_segments(meta, meta.num_seqs * n * (dv // 128))
+        act = torch.empty(t, n * (2 * dk + dv), dtype=rows.dtype, device=dev)
+        if segs > 1:
+            carry = torch.empty(meta.num_seqs, n, segs, dk, dv, dtype=f32, device=dev)
+        launches = 2 if segs == 1 else 4
     ptr = lambda x: None if x is None else _p(x).value
-    p = LightningParams(*[ptr(x) for x in (rows, None, powers, state, norm_w, out, o32, None, meta.q_start, meta.q_len, meta.past_len, meta.slot_ids,
+    p = LightningParams(*[ptr(x) for x in (rows, act, powers, state, norm_w, out, sums, carry, meta.q_start, meta.q_len, meta.past_len, meta.slot_ids,
                                            Workspace.get(dev).status)],
-                        rows.shape[1], n, dk, dv, n * dk, 2 * n * dk, n * (2 * dk + dv), dv_real, powers.shape[1], t, meta.num_seqs, 1, 0, eps)
-    code, L, ref_p = _dtype_code(rows), lib(), ctypes.byref(p)
-    if kernel == "step":
-        _check(L.telb_lightning_step(ref_p, c_int(code), _stream()), "lightning_step", 2)
+                        rows.shape[1], n, dk, dv, n * dk, 2 * n * dk, n * (2 * dk + dv), powers.shape[1], t, meta.num_seqs, segs, per)
+    L, ref_p = lib(), ctypes.byref(p)
+    if kernel == "chunk":
+        _check(L.telb_lightning_chunk(ref_p, _stream()), "lightning_chunk", launches)
     else:
-        _check(L.telb_lightning_walk(ref_p, c_int(code), _stream()), "lightning_walk", 2)
-    return out
+        f = L.telb_lightning_step if kernel == "step" else L.telb_lightning_walk
+        _check(f(ref_p, c_int(_dtype_code(rows)), _stream()), f"lightning_{kernel}")
+    return out, sums
 
 
 class ChannelDeltaParams(ctypes.Structure):

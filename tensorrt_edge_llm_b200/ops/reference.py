@@ -615,7 +615,7 @@ def _part_norm(x, weight, groups, eps):
     return (parts * torch.rsqrt(parts.pow(2).mean(-1, keepdim=True) + eps)).reshape(x.shape) * weight
 
 
-def stream_post(stream, delta, weight, groups, eps, meta: StepMeta, dtype, ids, table, bigram, conv, history, out_norm):
+def stream_post(stream, delta, weight, groups, eps, meta: StepMeta, dtype, ids, table, bigram, conv, history, out_norm, sums=None):
     """See :func:`ops.stream_post`."""
     seqs = [(int(a), int(n), int(p), int(s)) for a, n, p, s in zip(meta.q_start, meta.q_len, meta.past_len, meta.slot_ids) if int(n)]
     if stream is None:
@@ -633,7 +633,10 @@ def stream_post(stream, delta, weight, groups, eps, meta: StepMeta, dtype, ids, 
     else:
         x = stream
     if delta is not None:
-        x = x + _part_norm(delta.float(), weight, groups, eps)
+        d = delta.float()
+        if sums is not None:
+            d = d * torch.rsqrt(sums[0].sum(-1, keepdim=True) / sums[1] + eps)
+        x = x + _part_norm(d, weight, groups, eps)
     if out_norm is not None:
         return x, _part_norm(x, out_norm, groups, eps).to(dtype)
     if conv is None:
@@ -649,7 +652,7 @@ def stream_post(stream, delta, weight, groups, eps, meta: StepMeta, dtype, ids, 
     return x, h.to(dtype)
 
 
-def lightning(rows, norm_w, powers, state, meta: StepMeta, dv_real, eps):
+def lightning(rows, norm_w, powers, state, meta: StepMeta):
     """Row by row in fp32 (see :func:`ops.lightning`)."""
     t, (_, n, dk, dv) = rows.shape[0], state.shape
     q, k, v, g = rows.float().split([n * dk, n * dk, n * dv, n * dv], dim=-1)
@@ -664,8 +667,7 @@ def lightning(rows, norm_w, powers, state, meta: StepMeta, dv_real, eps):
         if ql:
             state[slot] = S
     o = o.reshape(t, n * dv)
-    o = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / (n * dv_real) + eps) * norm_w
-    return (o * torch.sigmoid(g)).to(rows.dtype)
+    return (o * norm_w * torch.sigmoid(g)).to(rows.dtype), o.pow(2).reshape(t, -1, 64).sum(-1)
 
 
 # ------------------------------------------------------------------------------------------

@@ -185,22 +185,26 @@ def _meta(lo, hi, slots, device, table=None):
                            slot_ids=slots, device=device)
 
 
-def stream_case(device, dtype, width, groups, taps, lens, past=None, ids=False, buckets=37, mul=(1000003, 77)):
-    """:func:`ops.stream_post` with a convolution: worst errors of the stream and of the convolved rows.  State rows hold leftovers."""
+def stream_case(device, dtype, width, groups, taps, lens, past=None, ids=False, buckets=37, mul=(1000003, 77), behind=0):
+    """:func:`ops.stream_post` with a convolution: worst errors of the stream and of the convolved rows.  State rows hold leftovers.
+    ``behind``: that many partial sums of squares per row, by whose root mean square (over 100 features) the update is divided."""
     from tensorrt_edge_llm_b200 import ops
     g, t, eps = torch.Generator().manual_seed(3), sum(lens), 1e-4
     starts = [sum(lens[:i]) for i in range(len(lens))]
     x, d = torch.randn(t, width, generator=g), (torch.randn(t, width, generator=g) * 3).to(dtype)
     w, conv = torch.randn(width, generator=g), torch.randn(taps, width, generator=g) * 0.5
     table, big = torch.randn(50, width, generator=g).to(dtype), torch.randn(buckets + 1, width, generator=g).to(dtype)
-    toks = torch.randint(0, 50, (t,), generator=g)
+    toks, sums = torch.randint(0, 50, (t,), generator=g), torch.rand(t, max(behind, 1), generator=g) * 50
     f, want_x, want_h = lambda v: v.double(), [], []
     for s, n in zip(starts, lens):
         if ids:
             y = [int(v) for v in toks[s:s + n]]
             y = f(table)[y] + f(big)[oracle.bigram_rows(y, buckets, *mul)]
         else:
-            y = f(x[s:s + n]) + oracle.group_norm(f(d[s:s + n]), f(w), groups, eps)
+            y = f(d[s:s + n])
+            if behind:
+                y = y / torch.sqrt(f(sums[s:s + n]).sum(-1, keepdim=True) / 100 + eps)
+            y = f(x[s:s + n]) + oracle.group_norm(y, f(w), groups, eps)
         want_x.append(y)
         want_h.append(y + oracle.causal_conv(y, f(conv).t()))
     dev = lambda v: v.to(device)
@@ -215,7 +219,8 @@ def stream_case(device, dtype, width, groups, taps, lens, past=None, ids=False, 
             a, b = ops.stream_post(None, None, None, groups, eps, _meta(lo, hi, slots, device), dtype, ids=dev(toks[idx].int()), table=dev(table),
                                    bigram=ops.Bigram(dev(big), last, buckets, *mul), **kw)
         else:
-            a, b = ops.stream_post(dev(x[idx]), dev(d[idx]), dev(w), groups, eps, _meta(lo, hi, slots, device), dtype, **kw)
+            a, b = ops.stream_post(dev(x[idx]), dev(d[idx]), dev(w), groups, eps, _meta(lo, hi, slots, device), dtype,
+                                   sums=(dev(sums[idx]), 100) if behind else None, **kw)
         got_x[idx], got_h[idx] = a.float().cpu(), b.float().cpu()
     want_x, want_h = torch.cat(want_x), torch.cat(want_h)
     return _worst_row(got_x - want_x, want_x), _worst_row(got_h - want_h, want_h)
@@ -335,9 +340,9 @@ def delta_case(device, dtype, heads, kv, dk, dv, conv, lens, past=None, kernel=N
     return float((got[:, :, :dv].double() - w).pow(2).mean().sqrt() / w.std())
 
 
-def lightning_case(device, dtype, heads, dk, dv, lens, past=None, decay=None, kernel=None, loud=None):
-    """:func:`ops.lightning` at padded sizes against the memory of the oracle: worst row error of the outputs, and the error of the states.
-    ``loud``: a row whose key and value are large, so that it has to be carried (decayed) through every later row."""
+def lightning_case(device, dtype, heads, dk, dv, lens, past=None, decay=None, kernel=None, loud=None, **force):
+    """:func:`ops.lightning` at padded sizes against the memory of the oracle: worst row error of the normed outputs, and the error of the
+    states.  ``loud``: a row whose key and value are large, so that it has to be carried (decayed) through every later row."""
     from tensorrt_edge_llm_b200 import ops
     from tensorrt_edge_llm_b200.config import LightningConfig
     decay = decay or [1 - 2.0 ** -(2 + 3 * h) for h in range(heads)]
@@ -364,11 +369,15 @@ def lightning_case(device, dtype, heads, dk, dv, lens, past=None, decay=None, ke
     powers = (dd[:, None] ** torch.arange(257, dtype=torch.float64)).float()
     state = torch.full((6, heads, kp, vp), 9.0, device=device)
     slots = [4, 1, 3, 0, 5, 2][:len(lens)]
-    fn = ops.lightning if kernel is None else functools.partial(ops.cuda_ops().lightning, kernel=kernel)
+    if kernel is not None:
+        force["kernel"] = kernel
+    fn = functools.partial(ops.cuda_ops().lightning, **force) if force else ops.lightning
     dev, got = (lambda x: x.to(device)), torch.zeros(t, heads, vp)
     for lo, hi in _steps(lens, past):
         idx = _rows(starts, lo, hi)
-        got[idx] = fn(dev(packed[idx]), dev(_pad(nw, vp).reshape(-1)), dev(powers), state, _meta(lo, hi, slots, device), dv, eps).float().cpu().view(-1, heads, vp)
+        u, sums = fn(dev(packed[idx]), dev(_pad(nw, vp).reshape(-1)), dev(powers), state, _meta(lo, hi, slots, device))
+        rms = torch.sqrt(sums.double().cpu().sum(-1) / (heads * dv) + eps)
+        got[idx] = (u.double().cpu() / rms[:, None]).float().view(-1, heads, vp)
     assert vp == dv or float(got[:, :, dv:].abs().max()) == 0.0
     w, st = torch.cat(want), torch.stack(states)
     err = torch.stack([(state[s].cpu().double()[:, :dk, :dv] - x).pow(2).mean((-1, -2)).sqrt() / x.pow(2).mean((-1, -2)).sqrt() for s, x in zip(slots, st)])

@@ -91,6 +91,7 @@ def test_config_refuses_what_it_does_not_know(change):
 
 @pytest.mark.parametrize("width, groups, taps", [(24, 3, 4), (40, 4, 1), (256, 2, 3), (64, 1, 8)])
 def test_stream_conv_and_bigram(width, groups, taps):
+    assert max(cases.stream_case("cpu", torch.float32, width, groups, taps, [9, 1, 20], behind=3)) < 1e-5
     for ids in (False, True):
         for lens, past in (([9, 1, 20], None), ([12, 3, 30], [5, 2, 1]), ([2, 2], [1, 1])):
             assert max(cases.stream_case("cpu", torch.float32, width, groups, taps, lens, past, ids=ids)) < 1e-5
@@ -324,6 +325,8 @@ def test_deployments_that_are_refused(ckpt):
     cfg = ModelConfig.from_hf_dict(cases.CONFIGS["wide"]())
     with pytest.raises((NotImplementedError, ValueError)):
         AutoModel.from_config(cfg.for_rank(0, 2))
+    with pytest.raises(ValueError, match="range of float16"):
+        cases.make_runner(ckpt("wide"), "cpu", "float16")
     r = cases.make_runner(ckpt("wide"), "cpu", "float32")
     with pytest.raises(NotImplementedError):
         r.prefill_embeds([0], [torch.zeros(3, cfg.hidden_size)])

@@ -36,6 +36,7 @@ def no_timed_out_waits():
 def test_stream_conv_and_bigram(width, groups, taps, dtype):
     """Rows of one portion in several blocks, portions shorter than the convolution, single rows; state rows held other requests."""
     tol = (1e-5, 1e-5) if dtype == "float32" else (1e-5, 8e-3)
+    assert max(cases.stream_case(DEV, DTYPES[dtype], width, groups, taps, [40, 1, 20], behind=37)) < tol[1]
     for ids in (False, True):
         for lens, past in (([40, 1, 20], None), ([33, 9, 30], [17, 2, 1]), ([2, 2], [1, 1]), ([7, 100, 3], [6, 99, 2])):
             x, h = cases.stream_case(DEV, DTYPES[dtype], width, groups, taps, lens, past, ids=ids)
@@ -131,23 +132,38 @@ LIGHTNING = [(3, 24, 40), (1, 72, 136), (4, 64, 128), (2, 128, 128), (2, 200, 26
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
 @pytest.mark.parametrize("shape", LIGHTNING)
 def test_lightning_prompts(shape, dtype):
-    """Ragged prompts and portions; constant, forgetting and everything between; an early row that has to be carried along."""
+    """Ragged prompts and portions; constant, forgetting and everything between; an early row that has to be carried along.  The state is
+    fp32 whatever the rows are: it agrees with the plain memory over the same rows."""
     tol = 1e-2 if dtype == "bfloat16" else 2e-5
-    run = lambda *a, **k: max(cases.lightning_case(DEV, DTYPES[dtype], *shape, *a, **k)[0:1])
-    assert run([150, 17, 300, 2]) < tol
-    assert run([150, 20, 275], past=[71, 18, 130]) < tol
-    assert run([290, 129], loud=3, decay=[0.999] * shape[0]) < tol
-    assert run([140, 260], past=[128, 129], decay=([0.0, 1.0, 0.5, 0.97] * 4)[:shape[0]]) < tol
+
+    def run(*a, **k):
+        out, state = cases.lightning_case(DEV, DTYPES[dtype], *shape, *a, **k)
+        assert out < tol and state < 2e-5, (a, k, out, state)
+    run([150, 17, 300, 2])
+    run([150, 20, 275], past=[71, 18, 130])
+    run([290, 129], loud=3, decay=[0.999] * shape[0])
+    run([140, 260], past=[128, 129], decay=([0.0, 1.0, 0.5, 0.97] * 4)[:shape[0]])
+
+
+@pytest.mark.parametrize("shape", [s for s in LIGHTNING if s[1] <= 128])
+def test_lightning_segments(shape):
+    """Long sequences cut into segments that run side by side: the same numbers, also where sequences end inside an early segment."""
+    lens, past = [1000, 130, 2, 513], [300, 1, 1, 128]
+    for segs in ((1, 8), (8, 1), (4, 2), (3, 3)):
+        for kw in (dict(), dict(past=past), dict(loud=3, decay=[0.9995] * shape[0])):
+            out, state = cases.lightning_case(DEV, torch.bfloat16, *shape, lens, kernel="chunk", segments=segs, **kw)
+            assert out < 1e-2 and state < 2e-5, (segs, kw, out, state)
 
 
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
 @pytest.mark.parametrize("shape", LIGHTNING)
-def test_lightning_state_and_decoding(shape, dtype):
-    """The state is fp32 whatever the rows are: after a prompt it agrees with the plain memory over the same rows; single rows go on from it."""
+def test_lightning_decoding(shape, dtype):
     tol = 1e-2 if dtype == "bfloat16" else 2e-5
-    for lens, past in (([300, 65, 2], None), ([1, 1, 1], None), ([141, 18, 2], [140, 17, 1])):
+    for lens, past in (([1, 1, 1], None), ([141, 18, 2], [140, 17, 1]), ([30, 18], [15, 17])):
         out, state = cases.lightning_case(DEV, DTYPES[dtype], *shape, lens, past)
         assert out < tol and state < 2e-5, (lens, past, out, state)
+    if dtype == "bfloat16":
+        assert max(cases.lightning_case(DEV, DTYPES[dtype], *shape, [40, 33], kernel="walk")) < tol
 
 
 # ---- the model through the runner ---------------------------------------------------------------------------
