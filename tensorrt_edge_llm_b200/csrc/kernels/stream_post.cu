@@ -1,18 +1,18 @@
-// The fp32 residual stream of blocks that are normed behind their sublayers.  Everything that lies between two sublayers is one kernel:
+// The fp32 residual stream of blocks that are normed behind their sublayers.  What lies between two sublayers:
 //
 //   source   x = table[id] + bigram[row(previous id, id)] (first call) or the running fp32 stream
 //   update   x += y / rms(y) * w                       y: sublayer output; each of `groups` equal parts of a row has its own rms.  With
 //                                                       `sums` the row is first divided by the rms of the row that was projected to y
-//   output   h = x                                     for a feed-forward                                  (post_row_kernel)
-//            h = x / rms(x) * w'                       same parts, for the head                            (post_row_kernel)
-//            h = x + Σ_j c[j] ∘ x_{t - taps + 1 + j}   causal convolution over time, for a mixer           (post_conv_kernel)
+//   output   h = x                                     for a feed-forward
+//            h = x / rms(x) * w'                       same parts, for the head
+//            h = x + Σ_j c[j] ∘ x_{t - taps + 1 + j}   causal convolution over time, for a mixer
 //
 // Stream, norms, convolution and its history are fp32; y, the tables and h have the activation type.
 //
-// The convolution looks at rows that other CTAs advance, so a CTA takes a block of rows and advances the taps - 1 rows in front of it
-// once more (reads only).  Blocks count from the start of a sequence's portion: only the first block of a portion needs the history
-// row of its seat, and the CTA that owns it also writes the new history (the last rows of the portion, advanced once more when they
-// lie in another block), so no CTA reads what another one writes.  The same holds for the last token of the sequence.
+// post_row_kernel does all of it for one row per CTA, the convolution included when every sequence has one row (decoding: the rows in front
+// are the history of its seat).  Longer portions take the convolution from the advanced stream in a second launch (post_conv_kernel):
+// blocks of rows count from the start of a sequence's portion, only the first one needs the history row of the seat, and the CTA that owns
+// it also writes the new history, so no CTA reads what another one of its launch writes.  The last token of a sequence is kept likewise.
 #include "host_utils.h"
 #include "tc5_common.cuh"
 
@@ -77,7 +77,6 @@ __device__ __forceinline__ float post_warp_sum(float v) {
 
 // One over the root mean square of the row that was projected to row `row` of delta (every warp computes it).
 __device__ __forceinline__ float row_scale(const StreamPostParams& p, size_t row) {
-    if (!p.sums) return 1.f;
     float s = 0.f;
     for (int i = threadIdx.x & 31; i < p.n_sums; i += 32) s += p.sums[row * p.n_sums + i];
     return 1.f / sqrtf(post_warp_sum(s) / p.sum_count + p.eps);
@@ -158,74 +157,152 @@ __device__ __forceinline__ void norm_parts(const StreamPostParams& p, float (&d)
         }
 }
 
-// One CTA per row: x += norm(y) w, h = x or norm(x) w'.
-template <typename T, int N, int E>
+// One CTA per row.  IDS: the stream starts from token ids.  CONV: every sequence has at most one row, h is the convolved stream.
+template <typename T, int N, int E, bool CONV, bool IDS>
 __global__ void __launch_bounds__(N) post_row_kernel(const __grid_constant__ StreamPostParams p) {
     pdl_prologue();
     extern __shared__ float red[];
     const size_t row = (size_t)blockIdx.x * p.width;
-    const int tid = threadIdx.x;
-    float x[1][E][4], d[1][E][4];
-    const float scale = row_scale(p, blockIdx.x);
+    const int tid = threadIdx.x, t = blockIdx.x;
+    float x[1][E][4], d[1][E][4], w[E][4], conv[E][4];
+    int slot = 0;
+    bool fresh = true;
+    if (CONV || IDS) {
+        const int seq = p.seq_ids[t];
+        slot = p.slot_ids[seq];
+        fresh = p.past_len[seq] <= 0;
+    }
+    float* hist = CONV ? p.history + (size_t)slot * (p.taps - 1) * p.width : nullptr;
+    if constexpr (CONV) {                                 // what the convolution takes from the rows in front; the history moves up
+#pragma unroll
+        for (int e = 0; e < E; ++e) {
+            const int c = (e * N + tid) * 4;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) conv[e][i] = 0.f;
+            if (c >= p.width) continue;
+            float old[kPostMaxTaps - 1][4], tap[kPostMaxTaps - 1][4];
+#pragma unroll
+            for (int j = 0; j < kPostMaxTaps - 1; ++j) {
+                if (j >= p.taps - 1) break;
+                get4(p.conv + (size_t)j * p.width + c, tap[j]);
+                if (fresh) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) old[j][i] = 0.f;
+                } else {
+                    get4(hist + (size_t)j * p.width + c, old[j]);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < kPostMaxTaps - 1; ++j) {
+                if (j >= p.taps - 1) break;
+#pragma unroll
+                for (int i = 0; i < 4; ++i) conv[e][i] = fmaf(tap[j][i], old[j][i], conv[e][i]);
+                if (j > 0) put4(hist + (size_t)(j - 1) * p.width + c, old[j]);
+            }
+        }
+    }
+    int id = 0;
+    long long pair = 0;
+    if constexpr (IDS) {
+        const int seq = p.seq_ids[t], t0 = p.q_start[seq];
+        id = min(max(p.ids[t], 0), p.vocab - 1);
+        if (p.bigram) {
+            const int prev = t > t0 ? p.ids[t - 1] : fresh ? -1 : p.last[slot];
+            pair = p.buckets;
+            if (prev >= 0) {
+                pair = (prev * p.mul_prev + id * p.mul_cur) % p.buckets;
+                if (pair < 0) pair += p.buckets;
+            }
+            if (t == t0) {                                // the CTA that reads the last token also replaces it
+                __syncthreads();
+                if (tid == 0) p.last[slot] = p.ids[t0 + p.q_len[seq] - 1];
+            }
+        }
+    }
 #pragma unroll
     for (int e = 0; e < E; ++e) {
         const int c = (e * N + tid) * 4;
 #pragma unroll
         for (int i = 0; i < 4; ++i) x[0][e][i] = d[0][e][i] = 0.f;
         if (c >= p.width) continue;
-        get4(p.x_in + row + c, x[0][e]);
-        if (p.delta) get4(reinterpret_cast<const T*>(p.delta) + row + c, d[0][e]);
+        if constexpr (IDS) {
+            get4(reinterpret_cast<const T*>(p.table) + (size_t)id * p.width + c, x[0][e]);
+            if (p.bigram) {
+                float b[4];
+                get4(reinterpret_cast<const T*>(p.bigram) + (size_t)pair * p.width + c, b);
 #pragma unroll
-        for (int i = 0; i < 4; ++i) d[0][e][i] *= scale;
+                for (int i = 0; i < 4; ++i) x[0][e][i] += b[i];
+            }
+        } else {
+            get4(p.x_in + row + c, x[0][e]);
+            if (p.delta) {
+                get4(reinterpret_cast<const T*>(p.delta) + row + c, d[0][e]);
+                get4(p.weight + c, w[e]);
+            }
+        }
     }
-    if (p.delta) norm_parts<N, E, 1>(p, d, red, 0);
+    if constexpr (!IDS) {
+        if (p.delta) {
+            if (p.sums) {
+                const float scale = row_scale(p, t);
+#pragma unroll
+                for (int e = 0; e < E; ++e)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) d[0][e][i] *= scale;
+            }
+            norm_parts<N, E, 1>(p, d, red, 0);
+        }
+    }
 #pragma unroll
     for (int e = 0; e < E; ++e) {
         const int c = (e * N + tid) * 4;
         if (c >= p.width) break;
-        if (p.delta) {
-            float w[4];
-            get4(p.weight + c, w);
+        if (!IDS && p.delta) {
 #pragma unroll
-            for (int i = 0; i < 4; ++i) x[0][e][i] = fmaf(d[0][e][i], w[i], x[0][e][i]);
+            for (int i = 0; i < 4; ++i) x[0][e][i] = fmaf(d[0][e][i], w[e][i], x[0][e][i]);
         }
         put4(p.x_out + row + c, x[0][e]);
-        if (!p.out_norm) put4(reinterpret_cast<T*>(p.h) + row + c, x[0][e]);
+        if constexpr (CONV) {
+            float tap[4], y[4];
+            get4(p.conv + (size_t)(p.taps - 1) * p.width + c, tap);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) y[i] = x[0][e][i] + fmaf(tap[i], x[0][e][i], conv[e][i]);
+            put4(reinterpret_cast<T*>(p.h) + row + c, y);
+            if (p.taps > 1) put4(hist + (size_t)(p.taps - 2) * p.width + c, x[0][e]);
+        } else if (p.h && !p.out_norm) {
+            put4(reinterpret_cast<T*>(p.h) + row + c, x[0][e]);
+        }
     }
-    if (!p.out_norm) return;
+    if (CONV || !p.out_norm) return;
     norm_parts<N, E, 1>(p, x, red, 1);
 #pragma unroll
     for (int e = 0; e < E; ++e) {
         const int c = (e * N + tid) * 4;
         if (c >= p.width) break;
-        float w[4];
-        get4(p.out_norm + c, w);
+        float g[4];
+        get4(p.out_norm + c, g);
 #pragma unroll
-        for (int i = 0; i < 4; ++i) w[i] *= x[0][e][i];
-        put4(reinterpret_cast<T*>(p.h) + row + c, w);
+        for (int i = 0; i < 4; ++i) g[i] *= x[0][e][i];
+        put4(reinterpret_cast<T*>(p.h) + row + c, g);
     }
 }
 
-// Blocks of rows with the convolution; W: window of the taps (right-aligned), R: rows at a time.
-template <typename T, int N, int E, int W>
-__global__ void __launch_bounds__(N) post_conv_kernel(const __grid_constant__ StreamPostParams p) {
-    constexpr int R = 2;
+// Convolution of the advanced stream (p.x_out) over blocks of rows; a thread walks four features down a block.  W: window of the taps
+// (right-aligned), R: rows whose loads are in flight together.
+constexpr int kConvThreads = 128;
+template <typename T, int W>
+__global__ void __launch_bounds__(kConvThreads) post_conv_kernel(const __grid_constant__ StreamPostParams p) {
+    constexpr int R = 8;
     pdl_prologue();
-    extern __shared__ float red[];
-    const int tid = threadIdx.x, pad = W - p.taps, past_rows = p.taps - 1;
-    float taps[W][E][4], nw[E][4];
+    const int c = (blockIdx.y * kConvThreads + threadIdx.x) * 4, pad = W - p.taps, front = p.taps - 1;
+    if (c >= p.width) return;
+    float taps[W][4];
 #pragma unroll
-    for (int e = 0; e < E; ++e) {
-        const int c = (e * N + tid) * 4;
+    for (int j = 0; j < W; ++j) {
 #pragma unroll
-        for (int j = 0; j < W; ++j) {
-#pragma unroll
-            for (int i = 0; i < 4; ++i) taps[j][e][i] = 0.f;
-            if (j >= pad && c < p.width) get4(p.conv + (size_t)(j - pad) * p.width + c, taps[j][e]);
-        }
-        if (p.delta && c < p.width) get4(p.weight + c, nw[e]);
+        for (int i = 0; i < 4; ++i) taps[j][i] = 0.f;
+        if (j >= pad) get4(p.conv + (size_t)(j - pad) * p.width + c, taps[j]);
     }
-    int turn = 0;
     const int lo = blockIdx.x * p.block_rows, hi = min(p.tokens, lo + p.block_rows);
     for (int t = lo; t < hi;) {
         const int seq = p.seq_ids[t], t0 = p.q_start[seq], i0 = t - t0, ql = p.q_len[seq];
@@ -235,184 +312,114 @@ __global__ void __launch_bounds__(N) post_conv_kernel(const __grid_constant__ St
         }
         const int n = min(p.block_rows, ql - i0), slot = p.slot_ids[seq];
         const bool first = i0 == 0, fresh = p.past_len[seq] <= 0;
-        float* hist_row = p.history + (size_t)slot * past_rows * p.width;
-        float hist[W - 1][E][4];                          // the rows in front, newest last
+        const float* src = p.x_out + (size_t)t0 * p.width + c;
+        T* dst = reinterpret_cast<T*>(p.h) + (size_t)t0 * p.width + c;
+        float* state = p.history + (size_t)slot * front * p.width + c;
+        // row of the portion, or of the history in front of it
+        auto row_at = [&](int j, float (&v)[4]) {
+            if (j >= 0) {
+                get4(src + (size_t)j * p.width, v);
+            } else if (!fresh && j >= -front) {
+                get4(state + (size_t)(front + j) * p.width, v);
+            } else {
 #pragma unroll
-        for (int j = 0; j < W - 1; ++j)
-#pragma unroll
-            for (int e = 0; e < E; ++e) {
-                const int c = (e * N + tid) * 4;
-#pragma unroll
-                for (int i = 0; i < 4; ++i) hist[j][e][i] = 0.f;
-                if (first && !fresh && j >= pad && c < p.width) get4(hist_row + (size_t)(j - pad) * p.width + c, hist[j][e]);
+                for (int i = 0; i < 4; ++i) v[i] = 0.f;
             }
-        // rows j0 .. j1 - 1 of the portion pass through, those from `emit` on are written: the block behind the rows in front of it, then,
-        // for the history, the portion's last rows when they lie in another block
-        for (int pass = 0; pass < (first && n < ql ? 2 : 1); ++pass) {
-            const int j0 = pass ? ql - past_rows : first ? i0 : i0 - past_rows;
-            const int j1 = pass ? ql : i0 + n, emit = pass ? ql : i0;
-            for (int j = j0; j < j1; j += R) {
-                float x[R][E][4], d[R][E][4];
+        };
+        float rows[W - 1 + R][4];
 #pragma unroll
-                for (int r = 0; r < R; ++r) {
-                    const bool live = j + r < j1;
-                    const size_t row = (size_t)(t0 + j + r) * p.width;
-                    const float scale = live ? row_scale(p, t0 + j + r) : 1.f;
-                    int id = 0;
-                    long long pair = 0;
-                    if (p.ids && live) {
-                        id = min(max(p.ids[t0 + j + r], 0), p.vocab - 1);
-                        if (p.bigram) {
-                            const int prev = j + r > 0 ? p.ids[t0 + j + r - 1] : fresh ? -1 : p.last[slot];
-                            pair = p.buckets;
-                            if (prev >= 0) {
-                                pair = (prev * p.mul_prev + id * p.mul_cur) % p.buckets;
-                                if (pair < 0) pair += p.buckets;
-                            }
-                        }
-                    }
+        for (int j = 0; j < W - 1; ++j) row_at(i0 - (W - 1) + j, rows[j]);
+        for (int j0 = i0; j0 < i0 + n; j0 += R) {
 #pragma unroll
-                    for (int e = 0; e < E; ++e) {
-                        const int c = (e * N + tid) * 4;
+            for (int r = 0; r < R; ++r)
+                if (j0 + r < i0 + n) get4(src + (size_t)(j0 + r) * p.width, rows[W - 1 + r]);
 #pragma unroll
-                        for (int i = 0; i < 4; ++i) x[r][e][i] = d[r][e][i] = 0.f;
-                        if (!live || c >= p.width) continue;
-                        if (p.ids) {
-                            get4(reinterpret_cast<const T*>(p.table) + (size_t)id * p.width + c, x[r][e]);
-                            if (p.bigram) {
-                                float b[4];
-                                get4(reinterpret_cast<const T*>(p.bigram) + (size_t)pair * p.width + c, b);
+            for (int r = 0; r < R; ++r) {
+                if (j0 + r >= i0 + n) break;
+                float y[4];
 #pragma unroll
-                                for (int i = 0; i < 4; ++i) x[r][e][i] += b[i];
-                            }
-                        } else {
-                            get4(p.x_in + row + c, x[r][e]);
-                        }
-                        if (p.delta) get4(reinterpret_cast<const T*>(p.delta) + row + c, d[r][e]);
+                for (int i = 0; i < 4; ++i) {
+                    float s = 0.f;
 #pragma unroll
-                        for (int i = 0; i < 4; ++i) d[r][e][i] *= scale;
-                    }
+                    for (int k = 0; k < W; ++k) s = fmaf(taps[k][i], rows[r + k][i], s);
+                    y[i] = rows[r + W - 1][i] + s;
                 }
-                if (p.delta) norm_parts<N, E, R>(p, d, red, turn++);
-#pragma unroll
-                for (int r = 0; r < R; ++r) {
-                    if (j + r >= j1) break;
-                    const size_t row = (size_t)(t0 + j + r) * p.width;
-                    const bool out = j + r >= emit;
-#pragma unroll
-                    for (int e = 0; e < E; ++e) {
-                        const int c = (e * N + tid) * 4;
-                        if (c >= p.width) break;
-                        if (p.delta) {
-#pragma unroll
-                            for (int i = 0; i < 4; ++i) x[r][e][i] = fmaf(d[r][e][i], nw[e][i], x[r][e][i]);
-                        }
-                        if (out) {
-                            put4(p.x_out + row + c, x[r][e]);
-                            float y[4];
-#pragma unroll
-                            for (int i = 0; i < 4; ++i) {
-                                float s = 0.f;
-#pragma unroll
-                                for (int k = 0; k < W - 1; ++k) s = fmaf(taps[k][e][i], hist[k][e][i], s);
-                                y[i] = x[r][e][i] + fmaf(taps[W - 1][e][i], x[r][e][i], s);
-                            }
-                            put4(reinterpret_cast<T*>(p.h) + row + c, y);
-                        }
-#pragma unroll
-                        for (int k = 0; k + 1 < W - 1; ++k)
-#pragma unroll
-                            for (int i = 0; i < 4; ++i) hist[k][e][i] = hist[k + 1][e][i];
-#pragma unroll
-                        for (int i = 0; i < 4; ++i) hist[W - 2][e][i] = x[r][e][i];
-                    }
-                }
+                put4(dst + (size_t)(j0 + r) * p.width, y);
             }
-        }
-        if (first) {
 #pragma unroll
             for (int j = 0; j < W - 1; ++j)
 #pragma unroll
-                for (int e = 0; e < E; ++e) {
-                    const int c = (e * N + tid) * 4;
-                    if (j >= pad && c < p.width) put4(hist_row + (size_t)(j - pad) * p.width + c, hist[j][e]);
-                }
-            if (p.ids && p.bigram) {
-                __syncthreads();                          // everyone has read the old last token
-                if (tid == 0) p.last[slot] = p.ids[t0 + ql - 1];
-            }
+                for (int i = 0; i < 4; ++i) rows[j][i] = rows[j + R][i];
+        }
+        if (first) {                                      // new history: the last rows of the portion, behind it what is left of the old one
+            float keep[W - 1][4];
+#pragma unroll
+            for (int j = 0; j < W - 1; ++j)
+                if (j >= pad) row_at(ql - (W - 1) + j, keep[j]);
+#pragma unroll
+            for (int j = 0; j < W - 1; ++j)
+                if (j >= pad) put4(state + (size_t)(j - pad) * p.width, keep[j]);
         }
         t += n;
     }
 }
 
-template <int N, int E, int R>
-static size_t post_smem(const StreamPostParams& p) {
-    const int part = p.width / p.groups;
-    if (part % 128 == 0) return (size_t)2 * R * E * (N / 32) * sizeof(float);
-    return (size_t)R * ((part % 4 == 0 ? p.width / 4 : p.width) + p.groups) * sizeof(float);
-}
-
 template <typename T, int N, int E>
-static int launch_row(const StreamPostParams& p, cudaStream_t stream) {
-    const size_t smem = post_smem<N, E, 1>(p);
+static int launch_row(const StreamPostParams& p, bool conv, cudaStream_t stream) {
+    const int part = p.width / p.groups;
+    const size_t smem = (part % 128 == 0 ? (size_t)2 * E * (N / 32) : (size_t)(part % 4 == 0 ? p.width / 4 : p.width) + p.groups) * sizeof(float);
     if (smem > 48 * 1024) return fail("telb_stream_post: parts of this size are not built for rows this wide");
-    TELB_LAUNCH("post_row_kernel", (post_row_kernel<T, N, E>), dim3(p.tokens), dim3(N), smem, stream, p);
+#define TELB_ROW(CONV_, IDS_) TELB_LAUNCH("post_row_kernel", (post_row_kernel<T, N, E, CONV_, IDS_>), dim3(p.tokens), dim3(N), smem, stream, p)
+    if (conv && p.ids) TELB_ROW(true, true);
+    else if (conv) TELB_ROW(true, false);
+    else if (p.ids) TELB_ROW(false, true);
+    else TELB_ROW(false, false);
+#undef TELB_ROW
     TELB_CHECK_LAUNCH("post_row_kernel");
     return 0;
 }
 
-template <typename T, int N, int E, int W>
-static int launch_conv(const StreamPostParams& p, cudaStream_t stream) {
-    const size_t smem = post_smem<N, E, 2>(p);
-    if (smem > 48 * 1024) return fail("telb_stream_post: parts of this size are not built for rows this wide");
-    TELB_LAUNCH("post_conv_kernel", (post_conv_kernel<T, N, E, W>), dim3((p.tokens + p.block_rows - 1) / p.block_rows), dim3(N), smem, stream, p);
-    TELB_CHECK_LAUNCH("post_conv_kernel");
-    return 0;
+template <typename T>
+static int run_row(const StreamPostParams& p, bool conv, cudaStream_t stream) {
+    if (p.width <= 1024) return launch_row<T, 256, 1>(p, conv, stream);
+    if (p.width <= 2048) return launch_row<T, 256, 2>(p, conv, stream);
+    if (p.width <= 4096) return launch_row<T, 512, 2>(p, conv, stream);
+    return launch_row<T, 1024, 4>(p, conv, stream);
 }
 
 template <typename T>
-static int run_post(const StreamPostParams& p, cudaStream_t stream) {
-    if (!p.conv) {
-        if (p.width <= 1024) return launch_row<T, 256, 1>(p, stream);
-        if (p.width <= 2048) return launch_row<T, 256, 2>(p, stream);
-        if (p.width <= 4096) return launch_row<T, 256, 4>(p, stream);
-        return launch_row<T, 1024, 4>(p, stream);
-    }
-    if (p.taps <= 4) {
-        if (p.width <= 1024) return launch_conv<T, 256, 1, 4>(p, stream);
-        if (p.width <= 2048) return launch_conv<T, 256, 2, 4>(p, stream);
-        if (p.width <= 4096) return launch_conv<T, 512, 2, 4>(p, stream);
-        return launch_conv<T, 512, 4, 4>(p, stream);
-    }
-    if (p.width <= 1024) return launch_conv<T, 256, 1, 8>(p, stream);
-    if (p.width <= 4096) return launch_conv<T, 512, 2, 8>(p, stream);
-    return launch_conv<T, 512, 4, 8>(p, stream);
+static int run_post(const StreamPostParams& p, int one_row, cudaStream_t stream) {
+    if (!p.conv || one_row) return run_row<T>(p, p.conv != nullptr, stream);
+    StreamPostParams first = p;
+    first.h = nullptr;
+    if (run_row<T>(first, false, stream)) return -1;
+    const dim3 grid((p.tokens + p.block_rows - 1) / p.block_rows, (p.width / 4 + kConvThreads - 1) / kConvThreads);
+    if (p.taps <= 4) TELB_LAUNCH("post_conv_kernel", (post_conv_kernel<T, 4>), grid, dim3(kConvThreads), 0, stream, p);
+    else TELB_LAUNCH("post_conv_kernel", (post_conv_kernel<T, 8>), grid, dim3(kConvThreads), 0, stream, p);
+    TELB_CHECK_LAUNCH("post_conv_kernel");
+    return 0;
 }
 
 }  // namespace telb
 
 using namespace telb;
 
-// dtype: 1 bf16, 2 fp32 (of the tables, delta and h; the un-normed stream needs bf16's range).  With a convolution, p->block_rows is 1 (then every sequence has at most one
-// row) or at least 8.
-extern "C" int telb_stream_post(const StreamPostParams* pp, int dtype, cudaStream_t stream) {
+// dtype: 1 bf16, 2 fp32 (of the tables, delta and h; the un-normed stream needs bf16's range).  one_row: every sequence has at most one row.
+// Otherwise a convolution goes over blocks of p->block_rows rows (at least 8).
+extern "C" int telb_stream_post(const StreamPostParams* pp, int one_row, int dtype, cudaStream_t stream) {
     const StreamPostParams& p = *pp;
     if (p.tokens <= 0) return 0;
     if (p.width % 4 || p.width > 16 * 1024) return fail("telb_stream_post: width must be a multiple of 4 and at most 16384");
     if (p.groups < 1 || p.groups > kPostMaxGroups || p.width % p.groups) return fail("telb_stream_post: 1 to 256 groups that divide the width");
     if (!p.ids == !p.x_in) return fail("telb_stream_post: either ids or a stream");
-    if (p.delta && !p.weight) return fail("telb_stream_post: the update has a weight");
+    if (p.delta && (!p.weight || p.ids)) return fail("telb_stream_post: an update has a weight and a stream to join");
+    if (p.sums && (!p.delta || p.n_sums < 1 || p.sum_count < 1)) return fail("telb_stream_post: sums belong to an update");
+    if (p.bigram && (!p.last || p.buckets < 1)) return fail("telb_stream_post: the bigram table needs buckets and last tokens");
     if (p.conv) {
-        if (p.width > 8 * 1024) return fail("telb_stream_post: the convolution covers rows up to 8192 wide");
         if (p.taps < 1 || p.taps > kPostMaxTaps) return fail("telb_stream_post: convolutions have 1 to 8 taps");
         if (p.taps > 1 && !p.history) return fail("telb_stream_post: the convolution keeps a history");
-        if (p.block_rows != 1 && p.block_rows < kPostMaxTaps) return fail("telb_stream_post: blocks of 1 or at least 8 rows");
-        if (p.bigram && (!p.last || p.buckets < 1)) return fail("telb_stream_post: the bigram table needs buckets and last tokens");
+        if (!one_row && p.block_rows < kPostMaxTaps) return fail("telb_stream_post: blocks of at least 8 rows");
         if (p.out_norm) return fail("telb_stream_post: a convolution or a norm, not both");
-    } else if (p.ids) {
-        return fail("telb_stream_post: token ids enter through the convolution form");
     }
-    if (p.sums && (!p.delta || p.n_sums < 1 || p.sum_count < 1)) return fail("telb_stream_post: sums belong to an update");
-    return dtype == 2 ? run_post<float>(p, stream) : run_post<__nv_bfloat16>(p, stream);
+    return dtype == 2 ? run_post<float>(p, one_row, stream) : run_post<__nv_bfloat16>(p, one_row, stream);
 }

@@ -341,11 +341,9 @@ class StreamPostParams(ctypes.Structure):
                [(n, c_int) for n in ("vocab", "width", "groups", "tokens", "taps", "block_rows", "n_sums", "sum_count")] + [("eps", c_float)]
 
 
-def _conv_block_rows(meta: StepMeta, tokens: int) -> int:
-    """Rows per CTA of the convolution form: every block reads the rows in front of it once more, so long steps take long blocks."""
-    if meta.max_q_len == 1:
-        return 1
-    return 8 if tokens <= 148 * 2 * 8 else 16 if tokens <= 148 * 4 * 16 else 32
+def _conv_block_rows(tokens: int) -> int:
+    """Rows per CTA of the convolution: every block reads the rows in front of it once more, so long steps take longer blocks."""
+    return 8 if tokens <= 148 * 8 else 16 if tokens <= 148 * 4 * 16 else 32
 
 
 def stream_post(stream, delta, weight, groups: int, eps: float, meta: StepMeta, dtype, ids, table, bigram, conv, history, out_norm,
@@ -382,9 +380,10 @@ def stream_post(stream, delta, weight, groups: int, eps: float, meta: StepMeta, 
                                             history if taps > 1 else None, out_norm, x, h, meta.q_start, meta.q_len, meta.past_len, meta.slot_ids,
                                             meta.seq_ids)],
                          *((0, 0, 0) if b is None else (b.buckets, b.mul_prev, b.mul_cur)), 0 if table is None else table.shape[0], width, groups, t, taps,
-                         _conv_block_rows(meta, t) if taps else 1, 0 if partial is None else partial.shape[1], count, eps)
+                         _conv_block_rows(t), 0 if partial is None else partial.shape[1], count, eps)
     code = 2 if dtype == f32 else 1
-    _check(lib().telb_stream_post(ctypes.byref(p), c_int(code), _stream()), "stream_post")
+    one_row = meta.max_q_len == 1
+    _check(lib().telb_stream_post(ctypes.byref(p), c_int(int(one_row)), c_int(code), _stream()), "stream_post", 1 if one_row or not taps else 2)
     return x, h
 
 
