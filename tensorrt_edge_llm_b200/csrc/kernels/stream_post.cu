@@ -9,7 +9,8 @@
 //
 // Stream, norms, convolution and its history are fp32; y, the tables and h have the activation type.
 //
-// post_row_kernel does all of it for one row per CTA, the convolution included when every sequence has one row (decoding: the rows in front
+// post_row_kernel does all of it for one row per CTA (steps of many rows update the stream with one row per warp instead: post_warp_kernel),
+// the convolution included when every sequence has one row (decoding: the rows in front
 // are the history of its seat).  Longer portions take the convolution from the advanced stream in a second launch (post_conv_kernel):
 // blocks of rows count from the start of a sequence's portion, only the first one needs the history row of the seat, and the CTA that owns
 // it also writes the new history, so no CTA reads what another one of its launch writes.  The last token of a sequence is kept likewise.
@@ -287,6 +288,63 @@ __global__ void __launch_bounds__(N) post_row_kernel(const __grid_constant__ Str
     }
 }
 
+// Many rows: one warp per row, x += norm(y) w, h = x.  Parts are multiples of 128 features, so a vector of a warp (four features per lane)
+// lies in one part; E vectors of the row stay in registers.
+constexpr int kPostWarps = 8;
+template <typename T, int E>
+__global__ void __launch_bounds__(kPostWarps * 32, 2) post_warp_kernel(const __grid_constant__ StreamPostParams p) {
+    pdl_prologue();
+    __shared__ float part_inv[kPostWarps][E];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t = blockIdx.x * kPostWarps + warp;
+    if (t >= p.tokens) return;
+    const size_t row = (size_t)t * p.width + lane * 4;
+    const int live = p.width / 128, n = live / p.groups;  // vectors of a row and of a part
+    T raw[E][4];
+    float x[E][4];
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+        if (e >= live) break;
+        const T* src = reinterpret_cast<const T*>(p.delta) + row + e * 128;
+        if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(raw[e]) = *reinterpret_cast<const float4*>(src);
+        else *reinterpret_cast<uint2*>(raw[e]) = *reinterpret_cast<const uint2*>(src);
+        get4(p.x_in + row + e * 128, x[e]);
+    }
+    const float scale = p.sums ? row_scale(p, t) : 1.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+        if (e >= live) break;
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float v = Cvt<T>::to_f(raw[e][i]) * scale;
+            s = fmaf(v, v, s);
+        }
+        s = post_warp_sum(s);
+        if (lane == 0) part_inv[warp][e] = s;
+    }
+    __syncwarp();
+    float inv = 0.f;
+    if (lane < live) {
+        for (int i = lane / n * n; i < lane / n * n + n; ++i) inv += part_inv[warp][i];
+        inv = scale / sqrtf(inv / (n * 128) + p.eps);
+    }
+    __syncwarp();
+    if (lane < live) part_inv[warp][lane] = inv;
+    __syncwarp();
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+        if (e >= live) break;
+        const float f = part_inv[warp][e];
+        float w[4];
+        get4(p.weight + lane * 4 + e * 128, w);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) x[e][i] = fmaf(Cvt<T>::to_f(raw[e][i]) * f, w[i], x[e][i]);
+        put4(p.x_out + row + e * 128, x[e]);
+        if (p.h) put4(reinterpret_cast<T*>(p.h) + row + e * 128, x[e]);
+    }
+}
+
 // Convolution of the advanced stream (p.x_out) over blocks of rows; a thread walks four features down a block.  W: window of the taps
 // (right-aligned), R: rows whose loads are in flight together.
 constexpr int kConvThreads = 128;
@@ -379,8 +437,20 @@ static int launch_row(const StreamPostParams& p, bool conv, cudaStream_t stream)
     return 0;
 }
 
+template <typename T, int E>
+static int launch_warp(const StreamPostParams& p, cudaStream_t stream) {
+    TELB_LAUNCH("post_warp_kernel", (post_warp_kernel<T, E>), dim3((p.tokens + kPostWarps - 1) / kPostWarps), dim3(kPostWarps * 32), 0, stream, p);
+    TELB_CHECK_LAUNCH("post_warp_kernel");
+    return 0;
+}
+
 template <typename T>
 static int run_row(const StreamPostParams& p, bool conv, cudaStream_t stream) {
+    if (p.tokens >= kPostWarps * sm_count() && p.delta && !conv && !p.out_norm && p.width / p.groups % 128 == 0 && p.width <= 4096) {
+        if (p.width <= 1024) return launch_warp<T, 8>(p, stream);
+        if (p.width <= 2048) return launch_warp<T, 16>(p, stream);
+        return launch_warp<T, 32>(p, stream);
+    }
     if (p.width <= 1024) return launch_row<T, 256, 1>(p, conv, stream);
     if (p.width <= 2048) return launch_row<T, 256, 2>(p, conv, stream);
     if (p.width <= 4096) return launch_row<T, 512, 2>(p, conv, stream);

@@ -50,6 +50,15 @@ def test_stream_long_blocks():
 
 
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
+@pytest.mark.parametrize("width, groups", [(128, 1), (768, 3), (2048, 4), (4096, 1)])
+def test_stream_many_rows(width, groups, dtype):
+    """One row per warp."""
+    for behind in (0, 40):
+        x, h = cases.stream_case(DEV, DTYPES[dtype], width, groups, 4, [1203, 5], behind=behind)
+        assert x < 1e-5 and h < (8e-3 if dtype == "bfloat16" else 1e-5)
+
+
+@pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
 @pytest.mark.parametrize("t, width, groups", [(1, 64, 2), (9, 72, 12), (130, 2048, 4), (3, 5120, 1), (5, 40, 4)])
 def test_stream_norms(t, width, groups, dtype):
     from tensorrt_edge_llm_b200 import ops
