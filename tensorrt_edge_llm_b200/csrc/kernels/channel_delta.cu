@@ -16,7 +16,8 @@
 //   S  <- D_4 ∘ S + Σ_j (g_{j+1} .. g_4 ∘ k_j) u_jᵀ
 //
 // so the eight products with S do not wait for one another, and one reduction over lanes serves four tokens.  `prep` writes the three
-// vectors per token, D_4 and the scalars, computed from products of decays only (no quotients).  A head's state is cut into column slices that
+// vectors per token, D_4 and the scalars, computed from products of decays only (no quotients).  With one decay per head the products leave
+// the vectors: a block then is k_1 .. k_4, q_1 .. q_4 and scalars (D_i joins the products with S, g_{j+1} .. g_4 the steps u_j).  A head's state is cut into column slices that
 // do not talk to each other: a warp owns 4 · CPL columns, eight lanes share the rows of a column and hold RPL rows x CPL columns each,
 // as packed row pairs (fma.rn.f32x2).
 #include <type_traits>
@@ -38,7 +39,7 @@ struct ChannelDeltaParams {
     const float* norm_w;       // [dv]
     void* conv_state;          // [slots, channels, taps - 1], oldest first
     float* state;              // [slots, heads, dk, dv]
-    float* blocks;             // [blocks, heads, 13 dk + 32] scratch: per block of four tokens the vectors and scalars of the walk
+    float* blocks;             // [blocks, heads, 13 dk + 32] scratch (8 dk + 32 with head_decay): per block of four tokens the vectors and scalars of the walk
     void* v_blocks;            // [blocks, heads, dv, 4] scratch: convolved values
     void* o;                   // [T, heads * dv] scratch: read-outs
     void* out;                 // [T, ld_out]: heads * dv
@@ -112,9 +113,14 @@ __device__ __forceinline__ void store_n(T* p, const T (&e)[N]) {
 // ---- prep ------------------------------------------------------------------------------------------------
 constexpr int kBlk = 4;              // tokens of a block
 constexpr int kPrepTokens = 16;      // rows whose blocks a warp takes
-constexpr int kScalars = 32;         // m_21 m_31 m_32 m_41 m_42 m_43 | n_11 n_21 n_22 n_31 .. n_44 | beta_1 .. beta_4, padded
+constexpr int kScalars = 32;         // m_21 m_31 m_32 m_41 m_42 m_43 | n_11 n_21 n_22 n_31 .. n_44 | beta_1 .. beta_4 | head decays: D_1 .. D_4 |
+                                     // head decays: g_{j+1} .. g_4 for j = 1 .. 4; padded
 
-__host__ __device__ inline int block_floats(int dk) { return 13 * dk + kScalars; }
+// vectors of a block: D_i k_i, D_i q_i, k_j times the decays behind it, D_4; or k_i, q_i
+template <bool HEAD>
+struct BlockVectors {
+    static constexpr int value = HEAD ? 8 : 13;
+};
 // First block of a sequence: blocks count from the start of its portion, and those of different sequences never meet.
 __device__ __forceinline__ int first_block(int q_start, int seq) { return q_start / kBlk + seq; }
 
@@ -192,8 +198,8 @@ __device__ __forceinline__ float total_of_lane(float (&v)[32], int lane) {
     return v[0];
 }
 
-// q, k and decays of one head and block.
-template <typename T, int C, int W>
+// q, k and decays of one head and block; HEAD: one decay per head.
+template <typename T, int C, int W, bool HEAD>
 __device__ __forceinline__ void prep_head(const ChannelDeltaParams& p, const float (&wq)[W][C], const float (&wk)[W][C], const float (&bias)[C], float rate, int h,
                                           int seq, size_t t, int i, int n, const T* history) {
     constexpr int V = C < 4 ? C : 4;
@@ -202,20 +208,15 @@ __device__ __forceinline__ void prep_head(const ChannelDeltaParams& p, const flo
 #pragma unroll
     for (int b = 0; b < kBlk; ++b) {
         if (b >= n) continue;
-        if (p.head_decay) {
-            const float z = p.decay[(t + b) * p.ld_decay + h];
-#pragma unroll
-            for (int c = 0; c < C; ++c) g[b][c] = z;
-        } else {
-            load_n<float, C>(p.decay + (t + b) * p.ld_decay + h * dk + lane * C, g[b]);
-        }
+        if constexpr (HEAD) g[b][0] = p.decay[(t + b) * p.ld_decay + h];
+        else load_n<float, C>(p.decay + (t + b) * p.ld_decay + h * dk + lane * C, g[b]);
     }
     conv_block<T, C, W>(p, wq, hk * dk + lane * C, t, i, n, history, q);
     conv_block<T, C, W>(p, wk, (p.kv_heads + hk) * dk + lane * C, t, i, n, history, k);
 #pragma unroll
     for (int b = 0; b < kBlk; ++b)
 #pragma unroll
-        for (int c = 0; c < C; ++c) g[b][c] = b < n ? cd_decay_as<T>(rate, g[b][c] + bias[c]) : 1.f;
+        for (int c = 0; c < (HEAD ? 1 : C); ++c) g[b][c] = b < n ? cd_decay_as<T>(rate, g[b][c] + bias[c]) : 1.f;
     // values 0-5: m, 6-15: n, 16-19: |k|², 20-23: |q|²; ends[j]: k_j times the decays behind it
     float sums[32], ends[kBlk][C];
 #pragma unroll
@@ -230,7 +231,7 @@ __device__ __forceinline__ void prep_head(const ChannelDeltaParams& p, const flo
             sums[6 + j * (j + 1) / 2 + j] = fmaf(q[j][c], d, sums[6 + j * (j + 1) / 2 + j]);
 #pragma unroll
             for (int x = j + 1; x < kBlk; ++x) {
-                d *= g[x][c];
+                if constexpr (!HEAD) d *= g[x][c];
                 sums[x * (x - 1) / 2 + j] = fmaf(k[x][c], d, sums[x * (x - 1) / 2 + j]);
                 sums[6 + x * (x + 1) / 2 + j] = fmaf(q[x][c], d, sums[6 + x * (x + 1) / 2 + j]);
             }
@@ -244,19 +245,51 @@ __device__ __forceinline__ void prep_head(const ChannelDeltaParams& p, const flo
         rk[b] = __shfl_sync(0xffffffffu, inv, 16 + b);
         rq[b] = __shfl_sync(0xffffffffu, inv, 20 + b) * rsqrtf((float)p.dk_real);
     }
-    float* out = p.blocks + ((size_t)(first_block(p.q_start[seq], seq) + i / kBlk) * p.heads + h) * block_floats(dk);
+    constexpr int kVecs = BlockVectors<HEAD>::value;
+    float* out = p.blocks + ((size_t)(first_block(p.q_start[seq], seq) + i / kBlk) * p.heads + h) * (kVecs * dk + kScalars);
     // scalars: scale by the norms of their pair
     float f = 1.f;
 #pragma unroll
-    for (int x = 0; x < kBlk; ++x)
+    for (int j = 0; j < kBlk; ++j) {
+        float between = 1.f;                              // g_{j+1} .. g_x (in the sums already with one decay per channel)
 #pragma unroll
-        for (int j = 0; j <= x; ++j) {
-            if (j < x && lane == x * (x - 1) / 2 + j) f = rk[x] * rk[j];
-            if (lane == 6 + x * (x + 1) / 2 + j) f = rq[x] * rk[j];
+        for (int x = j; x < kBlk; ++x) {
+            if (HEAD && x > j) between *= g[x][0];
+            if (j < x && lane == x * (x - 1) / 2 + j) f = rk[x] * rk[j] * between;
+            if (lane == 6 + x * (x + 1) / 2 + j) f = rq[x] * rk[j] * between;
         }
+    }
     total *= f;
     if (lane >= 16) total = lane < 16 + n ? cd_sigmoid(p.beta[(t + lane - 16) * p.ld_beta + h]) : 0.f;
-    out[13 * dk + lane] = total;
+    if constexpr (HEAD) {
+        float up = 1.f, behind = 1.f;
+#pragma unroll
+        for (int b = 0; b < kBlk; ++b) {
+            up *= g[b][0];
+            if (lane == 20 + b) total = up;
+            if (lane == 24 + kBlk - 1 - b) total = behind;
+            behind *= g[kBlk - 1 - b][0];
+        }
+    }
+    out[kVecs * dk + lane] = total;
+    if constexpr (HEAD) {
+#pragma unroll
+        for (int v = 0; v < C; v += V) {
+            const int ch = lane * C + v, at = walk_granule(dk, ch >> 2) * 4 + (ch & 3);
+#pragma unroll
+            for (int b = 0; b < kBlk; ++b) {
+                float x[V], y[V];
+#pragma unroll
+                for (int e = 0; e < V; ++e) {
+                    x[e] = k[b][v + e] * rk[b];
+                    y[e] = q[b][v + e] * rq[b];
+                }
+                store_n<float, V>(out + b * dk + at, x);
+                store_n<float, V>(out + (kBlk + b) * dk + at, y);
+            }
+        }
+        return;
+    }
     float d[C];
 #pragma unroll
     for (int c = 0; c < C; ++c) d[c] = 1.f;
@@ -306,7 +339,7 @@ __device__ __forceinline__ void prep_values(const ChannelDeltaParams& p, const f
     }
 
 // The blocks that start in rows t0 .. t1 - 1.
-template <typename T, int C, int W, bool VALUES>
+template <typename T, int C, int W, bool VALUES, bool HEAD>
 __device__ void prep_range(const ChannelDeltaParams& p, int h, int t0, int t1) {
     const int lane = threadIdx.x & 31, hk = h / (p.heads / p.kv_heads);
     float w0[W][C], w1[VALUES ? 1 : W][C], bias[C];
@@ -316,12 +349,8 @@ __device__ void prep_range(const ChannelDeltaParams& p, int h, int t0, int t1) {
     } else {
         load_taps<T, C, W>(p, hk * p.dk + lane * C, w0);
         load_taps<T, C, W>(p, (p.kv_heads + hk) * p.dk + lane * C, w1);
-        if (p.head_decay) {
-#pragma unroll
-            for (int c = 0; c < C; ++c) bias[c] = p.decay_bias[h];
-        } else {
-            load_n<float, C>(p.decay_bias + h * p.dk + lane * C, bias);
-        }
+        if constexpr (HEAD) bias[0] = p.decay_bias[h];
+        else load_n<float, C>(p.decay_bias + h * p.dk + lane * C, bias);
         rate = -expf(p.a_log[h]);
     }
     for (int t = t0; t < t1;) {
@@ -333,17 +362,17 @@ __device__ void prep_range(const ChannelDeltaParams& p, int h, int t0, int t1) {
         const int n = min(kBlk, p.q_len[seq] - i);
         const T* history = p.past_len[seq] > 0 ? reinterpret_cast<const T*>(p.conv_state) + (size_t)p.slot_ids[seq] * p.channels * (p.taps - 1) : nullptr;
         if constexpr (VALUES) prep_values<T, C, W>(p, w0, h, seq, t, i, n, history);
-        else prep_head<T, C, W>(p, w0, w1, bias, rate, h, seq, t, i, n, history);
+        else prep_head<T, C, W, HEAD>(p, w0, w1, bias, rate, h, seq, t, i, n, history);
         t += n;
     }
 }
 
 // grid (row ranges, heads).  VALUES: the value heads, else q, k and decays.
-template <typename T, int C, int W, bool VALUES>
+template <typename T, int C, int W, bool VALUES, bool HEAD>
 __global__ void __launch_bounds__(128) channel_delta_prep_kernel(const __grid_constant__ ChannelDeltaParams p) {
     pdl_prologue();
     const int t0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * kPrepTokens, t1 = min(p.tokens, t0 + kPrepTokens);
-    prep_range<T, C, W, VALUES>(p, blockIdx.y, t0, t1);
+    prep_range<T, C, W, VALUES, HEAD>(p, blockIdx.y, t0, t1);
 }
 
 // History of the convolutions after a portion: the last taps - 1 inputs.
@@ -428,7 +457,7 @@ __device__ __forceinline__ void walk_reduce(const float (&a)[C][kBlk], const flo
 constexpr int kWalkStages = 4;
 
 // grid (column slices of a head, heads, sequences); blockDim = warps of one slice
-template <typename T, int RPL, int CPL>
+template <typename T, int RPL, int CPL, bool HEAD>
 __global__ void __launch_bounds__(128) channel_delta_walk_kernel(const __grid_constant__ ChannelDeltaParams p) {
     pdl_wait();                                           // dependents start at the end: a long kernel runs slower under waiting ones
     constexpr int DK = RPL * 8;
@@ -446,7 +475,7 @@ __global__ void __launch_bounds__(128) channel_delta_walk_kernel(const __grid_co
     const int lcol = blockIdx.x * cols + warp * 4 * CPL + cg * CPL;      // first column of this lane, within the head
     const int r0 = p.q_start[seq], blk0 = first_block(r0, seq);
     const int chunks = (ql + kBlk - 1) / kBlk;
-    constexpr int kFloats = 13 * DK + kScalars;
+    constexpr int kVecs = BlockVectors<HEAD>::value, kFloats = kVecs * DK + kScalars;
 
     const int v_bytes = cols * kBlk * (int)sizeof(T), stage_bytes = kFloats * 4 + v_bytes;
 
@@ -519,9 +548,13 @@ __global__ void __launch_bounds__(128) channel_delta_walk_kernel(const __grid_co
         }
         float w[kBlk];
         walk_reduce<CPL>(a, b, rl, w);
-        alignas(16) float sc[20];
+        alignas(16) float sc[HEAD ? 28 : 20];
 #pragma unroll
-        for (int i = 0; i < 5; ++i) reinterpret_cast<float4*>(sc)[i] = reinterpret_cast<const float4*>(st + 13 * DK)[i];
+        for (int i = 0; i < (HEAD ? 7 : 5); ++i) reinterpret_cast<float4*>(sc)[i] = reinterpret_cast<const float4*>(st + kVecs * DK)[i];
+        if constexpr (HEAD) {
+#pragma unroll
+            for (int i = 0; i < kBlk; ++i) w[i] *= sc[20 + i];
+        }
         float v[kBlk];
         load_n<T, kBlk>(reinterpret_cast<const T*>(st + kFloats) + (lcol - (int)blockIdx.x * cols + my_col) * kBlk, v);
         float u[kBlk];                                    // even lanes
@@ -537,7 +570,8 @@ __global__ void __launch_bounds__(128) channel_delta_walk_kernel(const __grid_co
         for (int c = 0; c < CPL; ++c)
 #pragma unroll
             for (int i = 0; i < kBlk; ++i) {
-                const float x = CPL == 1 ? (rl & 1 ? mine[i] : u[i]) : __shfl_sync(kAll, u[i], (lane & 24) | (c * 2));
+                float x = CPL == 1 ? (rl & 1 ? mine[i] : u[i]) : __shfl_sync(kAll, u[i], (lane & 24) | (c * 2));
+                if constexpr (HEAD) x *= sc[24 + i];
                 ub[c][i] = f2_pack(x, x);
             }
         if (writer) {
@@ -554,9 +588,10 @@ __global__ void __launch_bounds__(128) channel_delta_walk_kernel(const __grid_co
         out += (size_t)kBlk * p.heads * p.dv;
 #pragma unroll
         for (int j = 0; j < RPL / 4; ++j) {
-            ulonglong2 x[kBlk + 1];                       // D_4 is the vector behind the four
+            ulonglong2 x[kBlk + 1];                       // D_4 is the vector behind the four (one number with head decays)
 #pragma unroll
-            for (int i = 0; i <= kBlk; ++i) x[i] = *reinterpret_cast<const ulonglong2*>(st + (2 * kBlk + i) * DK + (j * 8 + rl) * 4);
+            for (int i = 0; i < (HEAD ? kBlk : kBlk + 1); ++i) x[i] = *reinterpret_cast<const ulonglong2*>(st + ((HEAD ? 0 : 2 * kBlk) + i) * DK + (j * 8 + rl) * 4);
+            if constexpr (HEAD) x[kBlk].x = x[kBlk].y = f2_pack(sc[23], sc[23]);
 #pragma unroll
             for (int c = 0; c < CPL; ++c) {
                 S[2 * j][c] = f2_mul(S[2 * j][c], x[kBlk].x);
@@ -594,12 +629,12 @@ __global__ void __launch_bounds__(128) channel_delta_walk_kernel(const __grid_co
 // The walk for few (sequence, head) pairs and keys of 128 or 256: all 32 lanes share the rows of four columns (four rows, G granules each),
 // so a vector costs one shared-memory read per warp and granule instead of four and the chain of a block is short.  The 32 products of
 // a block (columns x (k, q) x tokens) are reduced so that lane 8 c + 4 a + i holds product a of column c and token i.
-template <typename T, int G>
+template <typename T, int G, bool HEAD>
 __global__ void __launch_bounds__(128) channel_delta_walk_narrow_kernel(const __grid_constant__ ChannelDeltaParams p) {
     pdl_wait();
     constexpr int DK = G * 128, C = 4, kCols = 16;
     constexpr unsigned kAll = 0xffffffffu;
-    constexpr int kFloats = 13 * DK + kScalars, kVBytes = kCols * kBlk * (int)sizeof(T), kStage = kFloats * 4 + kVBytes;
+    constexpr int kVecs = BlockVectors<HEAD>::value, kFloats = kVecs * DK + kScalars, kVBytes = kCols * kBlk * (int)sizeof(T), kStage = kFloats * 4 + kVBytes;
     extern __shared__ __align__(16) uint8_t walk_smem[];
     __shared__ uint64_t full[kWalkStages];
     __shared__ uint32_t abort_word;
@@ -644,7 +679,7 @@ __global__ void __launch_bounds__(128) channel_delta_walk_narrow_kernel(const __
         for (int c = 0; c < C; ++c) S[r][c] = f2_pack(a[c], b[c]);
     }
     T* out = reinterpret_cast<T*>(p.o) + ((size_t)r0 + i_own) * p.heads * p.dv + (size_t)h * p.dv + col0 + c_own;
-    const int n_row = 13 * DK + 6 + i_own * (i_own + 1) / 2;
+    const int n_row = kVecs * DK + 6 + i_own * (i_own + 1) / 2;
     __syncthreads();
     bool ok = true;
     for (int ch = 0; ch < chunks; ++ch) {
@@ -668,13 +703,16 @@ __global__ void __launch_bounds__(128) channel_delta_walk_narrow_kernel(const __
         for (int c = 0; c < C; ++c)
 #pragma unroll
             for (int i = 0; i < 2 * kBlk; ++i) sums[c * 8 + i] = f2_sum(acc[i][c]);
-        const float total = total_of_lane(sums, lane);
+        float total = total_of_lane(sums, lane);
+        if constexpr (HEAD) total *= st[kVecs * DK + 20 + i_own];
         float w[kBlk], v[kBlk], u[kBlk];
         load_n<T, kBlk>(reinterpret_cast<const T*>(st + kFloats) + (warp * C + c_own) * kBlk, v);
-        alignas(16) float m[8], beta[kBlk];
-        reinterpret_cast<float4*>(m)[0] = *reinterpret_cast<const float4*>(st + 13 * DK);
-        reinterpret_cast<float4*>(m)[1] = *reinterpret_cast<const float4*>(st + 13 * DK + 4);
-        *reinterpret_cast<float4*>(beta) = *reinterpret_cast<const float4*>(st + 13 * DK + 16);
+        alignas(16) float m[8], beta[kBlk], behind[kBlk];
+        reinterpret_cast<float4*>(m)[0] = *reinterpret_cast<const float4*>(st + kVecs * DK);
+        reinterpret_cast<float4*>(m)[1] = *reinterpret_cast<const float4*>(st + kVecs * DK + 4);
+        *reinterpret_cast<float4*>(beta) = *reinterpret_cast<const float4*>(st + kVecs * DK + 16);
+        if constexpr (HEAD) *reinterpret_cast<float4*>(behind) = *reinterpret_cast<const float4*>(st + kVecs * DK + 24);
+        const float all = HEAD ? st[kVecs * DK + 23] : 1.f;
         float nr[kBlk];
 #pragma unroll
         for (int j = 0; j < kBlk; ++j) nr[j] = j <= i_own ? st[n_row + j] : 0.f;
@@ -692,14 +730,16 @@ __global__ void __launch_bounds__(128) channel_delta_walk_narrow_kernel(const __
         for (int c = 0; c < C; ++c)
 #pragma unroll
             for (int i = 0; i < kBlk; ++i) {
-                const float x = __shfl_sync(kAll, u[i], c * 8);
+                float x = __shfl_sync(kAll, u[i], c * 8);
+                if constexpr (HEAD) x *= behind[i];
                 ub[c][i] = f2_pack(x, x);
             }
 #pragma unroll
         for (int g = 0; g < G; ++g) {
             ulonglong2 x[kBlk + 1];
 #pragma unroll
-            for (int i = 0; i <= kBlk; ++i) x[i] = *reinterpret_cast<const ulonglong2*>(st + (2 * kBlk + i) * DK + (lane + 32 * g) * 4);
+            for (int i = 0; i < (HEAD ? kBlk : kBlk + 1); ++i) x[i] = *reinterpret_cast<const ulonglong2*>(st + ((HEAD ? 0 : 2 * kBlk) + i) * DK + (lane + 32 * g) * 4);
+            if constexpr (HEAD) x[kBlk].x = x[kBlk].y = f2_pack(all, all);
 #pragma unroll
             for (int c = 0; c < C; ++c) {
                 S[2 * g][c] = f2_mul(S[2 * g][c], x[kBlk].x);
@@ -882,17 +922,18 @@ __global__ void __launch_bounds__(256) channel_delta_decode_kernel(const __grid_
 }
 
 // ---- launchers ---------------------------------------------------------------------------------------------
-template <typename T>
+template <typename T, bool HEAD>
 static int launch_prep(const ChannelDeltaParams& p, cudaStream_t stream) {
     const int warps = (p.tokens + kPrepTokens - 1) / kPrepTokens;
     const dim3 grid((warps + 3) / 4, p.heads);
-#define TELB_PREP(W_, VALUES_) TELB_LAUNCH("channel_delta_prep_kernel", (channel_delta_prep_kernel<T, C, W_, VALUES_>), grid, dim3(128), 0, stream, p)
+#define TELB_PREP(W_, VALUES_, HEAD_) \
+    TELB_LAUNCH("channel_delta_prep_kernel", (channel_delta_prep_kernel<T, C, W_, VALUES_, HEAD_>), grid, dim3(128), 0, stream, p)
     if (p.taps <= 4) {
-        TELB_BY_LANES(p.dv, TELB_PREP(4, true))
-        TELB_BY_LANES(p.dk, TELB_PREP(4, false))
+        TELB_BY_LANES(p.dv, TELB_PREP(4, true, false))
+        TELB_BY_LANES(p.dk, TELB_PREP(4, false, HEAD))
     } else {
-        TELB_BY_LANES(p.dv, TELB_PREP(8, true))
-        TELB_BY_LANES(p.dk, TELB_PREP(8, false))
+        TELB_BY_LANES(p.dv, TELB_PREP(8, true, false))
+        TELB_BY_LANES(p.dk, TELB_PREP(8, false, HEAD))
     }
 #undef TELB_PREP
     TELB_CHECK_LAUNCH("channel_delta_prep_kernel");
@@ -907,65 +948,65 @@ static int launch_roll(const ChannelDeltaParams& p, cudaStream_t stream) {
     return 0;
 }
 
-template <typename T, int RPL, int CPL>
+template <typename T, int RPL, int CPL, bool HEAD>
 static int launch_walk_as(const ChannelDeltaParams& p, cudaStream_t stream) {
     constexpr int warps = CPL == 1 ? 4 : 2, cols = warps * 4 * CPL;      // 16 or 32: divides every padded head
-    constexpr int smem = ((13 * RPL * 8 + kScalars) * 4 + cols * kBlk * (int)sizeof(T)) * kWalkStages;
+    constexpr int smem = ((BlockVectors<HEAD>::value * RPL * 8 + kScalars) * 4 + cols * kBlk * (int)sizeof(T)) * kWalkStages;
     if (smem > 48 * 1024) {
         static bool configured = false;
         if (!configured) {
-            cudaError_t e = cudaFuncSetAttribute(channel_delta_walk_kernel<T, RPL, CPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+            cudaError_t e = cudaFuncSetAttribute(channel_delta_walk_kernel<T, RPL, CPL, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
             if (e != cudaSuccess) return fail("cudaFuncSetAttribute(channel_delta_walk)", e);
             configured = true;
         }
     }
-    TELB_LAUNCH_SERIAL("channel_delta_walk_kernel", (channel_delta_walk_kernel<T, RPL, CPL>), dim3(p.dv / cols, p.heads, p.num_seqs), dim3(warps * 32), smem, stream, p);
+    TELB_LAUNCH_SERIAL("channel_delta_walk_kernel", (channel_delta_walk_kernel<T, RPL, CPL, HEAD>), dim3(p.dv / cols, p.heads, p.num_seqs), dim3(warps * 32), smem, stream, p);
     TELB_CHECK_LAUNCH("channel_delta_walk_kernel");
     return 0;
 }
 
-template <typename T, int G>
+template <typename T, int G, bool HEAD>
 static int launch_walk_narrow(const ChannelDeltaParams& p, cudaStream_t stream) {
-    constexpr int smem = ((13 * G * 128 + kScalars) * 4 + 16 * kBlk * (int)sizeof(T)) * kWalkStages;
+    constexpr int smem = ((BlockVectors<HEAD>::value * G * 128 + kScalars) * 4 + 16 * kBlk * (int)sizeof(T)) * kWalkStages;
     if (smem > 48 * 1024) {
         static bool configured = false;
         if (!configured) {
-            cudaError_t e = cudaFuncSetAttribute(channel_delta_walk_narrow_kernel<T, G>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+            cudaError_t e = cudaFuncSetAttribute(channel_delta_walk_narrow_kernel<T, G, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
             if (e != cudaSuccess) return fail("cudaFuncSetAttribute(channel_delta_walk_narrow)", e);
             configured = true;
         }
     }
-    TELB_LAUNCH_SERIAL("channel_delta_walk_narrow_kernel", (channel_delta_walk_narrow_kernel<T, G>), dim3(p.dv / 16, p.heads, p.num_seqs), dim3(128), smem, stream, p);
+    TELB_LAUNCH_SERIAL("channel_delta_walk_narrow_kernel", (channel_delta_walk_narrow_kernel<T, G, HEAD>), dim3(p.dv / 16, p.heads, p.num_seqs), dim3(128), smem, stream, p);
     TELB_CHECK_LAUNCH("channel_delta_walk_narrow_kernel");
     return 0;
 }
 
 static int g_walk_cols = 0;          // columns per lane; 0 = by the number of columns
 
-template <typename T, int RPL>
+template <typename T, int RPL, bool HEAD>
 static int launch_walk(const ChannelDeltaParams& p, cudaStream_t stream) {
     // few (sequence, head) pairs: narrow slices, so that every scheduler has a chain of its own; many: wide ones, which read less
     const long long columns = (long long)p.num_seqs * p.heads * p.dv;
     int cpl = columns / 4 <= 8LL * sm_count() ? 1 : RPL > 16 ? 2 : 4;
     if (g_walk_cols) cpl = g_walk_cols;
     if constexpr (RPL >= 16) {
-        if (cpl == 1) return launch_walk_narrow<T, RPL / 16>(p, stream);
+        if (cpl == 1) return launch_walk_narrow<T, RPL / 16, HEAD>(p, stream);
     } else {
-        if (cpl == 1) return launch_walk_as<T, RPL, 1>(p, stream);
+        if (cpl == 1) return launch_walk_as<T, RPL, 1, HEAD>(p, stream);
     }
-    if (cpl == 2 || RPL > 16) return launch_walk_as<T, RPL, 2>(p, stream);
-    return launch_walk_as<T, RPL, (RPL > 16 ? 2 : 4)>(p, stream);
+    if (cpl == 2 || RPL > 16) return launch_walk_as<T, RPL, 2, HEAD>(p, stream);
+    return launch_walk_as<T, RPL, (RPL > 16 ? 2 : 4), HEAD>(p, stream);
 }
 
-template <typename T>
+template <typename T, bool HEAD>
 static int channel_delta_rows(const ChannelDeltaParams& p, cudaStream_t stream) {
-    if (launch_prep<T>(p, stream)) return -1;
+    if (launch_prep<T, HEAD>(p, stream)) return -1;
     int rc = 0;
     switch (p.dk) {
-        case 32: rc = launch_walk<T, 4>(p, stream); break;
-        case 64: rc = launch_walk<T, 8>(p, stream); break;
-        case 128: rc = launch_walk<T, 16>(p, stream); break;
-        default: rc = launch_walk<T, 32>(p, stream); break;
+        case 32: rc = launch_walk<T, 4, HEAD>(p, stream); break;
+        case 64: rc = launch_walk<T, 8, HEAD>(p, stream); break;
+        case 128: rc = launch_walk<T, 16, HEAD>(p, stream); break;
+        default: rc = launch_walk<T, 32, HEAD>(p, stream); break;
     }
     if (rc) return rc;
     const long long warps = (long long)p.tokens * p.heads;
@@ -1023,6 +1064,10 @@ extern "C" int telb_channel_delta(const ChannelDeltaParams* pp, int decode, int 
         if (dtype == 2) return channel_delta_step<float>(p, stream);
         return dtype == 1 ? channel_delta_step<__nv_bfloat16>(p, stream) : channel_delta_step<__half>(p, stream);
     }
-    if (dtype == 2) return channel_delta_rows<float>(p, stream);
-    return dtype == 1 ? channel_delta_rows<__nv_bfloat16>(p, stream) : channel_delta_rows<__half>(p, stream);
+    if (p.head_decay) {
+        if (dtype == 0) return fail("telb_channel_delta: prompts with one decay per head are built for bf16 and fp32");
+        return dtype == 2 ? channel_delta_rows<float, true>(p, stream) : channel_delta_rows<__nv_bfloat16, true>(p, stream);
+    }
+    if (dtype == 2) return channel_delta_rows<float, false>(p, stream);
+    return dtype == 1 ? channel_delta_rows<__nv_bfloat16, false>(p, stream) : channel_delta_rows<__half, false>(p, stream);
 }

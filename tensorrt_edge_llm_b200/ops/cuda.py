@@ -1255,7 +1255,7 @@ def channel_delta(qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, con
     blocks = v_blocks = o = None
     if kernel == "walk":                       # blocks of four tokens, counted from the start of every portion
         nb = t // 4 + meta.num_seqs + 1
-        blocks, v_blocks = torch.empty(nb, n, 13 * dk + 32, dtype=f32, device=dev), torch.empty(nb, n, dv, 4, dtype=qkv.dtype, device=dev)
+        blocks, v_blocks = torch.empty(nb, n, (8 if spec.head_decay else 13) * dk + 32, dtype=f32, device=dev), torch.empty(nb, n, dv, 4, dtype=qkv.dtype, device=dev)
         o = torch.empty(t, n * dv, dtype=qkv.dtype, device=dev)
     ptr = lambda x: None if x is None else _p(x).value
     p = ChannelDeltaParams(*[ptr(x) for x in (qkv, decay, gate, beta, conv_w, a_log, decay_bias, norm_w, conv_state, state, blocks, v_blocks, o, out,
