@@ -120,7 +120,7 @@ def kernel_pairs(device) -> list:
         # ---- stream and feed-forward element-wise steps ----
         x, y, res = [rnd(t, h) for _ in range(sets)], [rnd(t, h).to(dt) for _ in range(sets)], [rnd(t, h).to(dt) for _ in range(sets)]
         ww, wb, alpha = torch.ones(h, device=device), torch.ones(h, device=device, dtype=dt), torch.ones((), device=device)
-        taps, hist, sums = rnd(4, h) * 0.2, [torch.zeros(b, 3, h, device=device) for _ in range(sets)], [rnd(t, n * d // 64).abs() for _ in range(sets)]
+        taps, hist, sums = rnd(4, h) * 0.2, [torch.zeros(b, 3, h, device=device) for _ in range(sets)], [rnd(t, n * d // 32).abs() for _ in range(sets)]
         post = lambda i, **kw: cu.stream_post(x[i], y[i], ww, 4, 1e-6, meta, dt, None, None, None, kw.get("conv"), kw.get("history"), kw.get("out_norm"),
                                               kw.get("sums"))
         us_tanh = timer(lambda i: cu.stream_norm(x[i], ww, 1e-6, y[i], None, 1.0, None, 0.0, None, None, dt, alpha, ww))
@@ -129,7 +129,7 @@ def kernel_pairs(device) -> list:
         hb_ = 2 * b * 3 * h * 4
         for nm, u, by in (("output norm in parts + stream update (fp32)", timer(post), row),
                           ("output norm in parts + stream update (fp32) + input convolution", timer(lambda i: post(i, conv=taps, history=hist[i])), row + hb_),
-                          ("the same behind lightning attention", timer(lambda i: post(i, conv=taps, history=hist[i], sums=(sums[i], n * d))), row + hb_ + t * n * 8)):
+                          ("the same behind lightning attention", timer(lambda i: post(i, conv=taps, history=hist[i], sums=(sums[i], n * d))), row + hb_ + t * n * d // 8)):
             add(f"{nm}, {label}", u, by, 0.0, "stream update (fp32) + tanh norm", us_tanh, row, 0.0)
             add(f"{nm}, {label}", u, by, 0.0, "residual (16-bit) + RMS norm", us_add, t * h * 8, 0.0)
         ids, table, big = torch.randint(0, 32768, (t,), device=device, dtype=torch.int32), rnd(32768, h).to(dt), rnd(65537, h).to(dt)

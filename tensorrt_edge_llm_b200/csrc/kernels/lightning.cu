@@ -36,7 +36,6 @@ __global__ void __launch_bounds__(kWalkThreads) lightning_walk_kernel(const __gr
     float* sq = S + (size_t)p.dk * kWalkCols;        // [dk]
     float* sk = sq + p.dk;                           // [dk]
     float* part = sk + p.dk;                         // [4][64]
-    float* red = part + 4 * kWalkCols;               // [2]
     const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kWalkCols;
     const int ql = p.q_len[seq];
     if (ql <= 0) return;
@@ -67,9 +66,7 @@ __global__ void __launch_bounds__(kWalkThreads) lightning_walk_kernel(const __gr
             const size_t col = (size_t)h * p.dv + c0 + c;
             reinterpret_cast<T*>(p.out)[t * p.heads * p.dv + col] = Cvt<T>::from_f(lightning_gate<T>(o, p.norm_w[col], Cvt<T>::to_f(row[p.g_off + col])));
             const float ss = lightning_warp_sum(o * o);
-            if ((tid & 31) == 0) red[tid >> 5] = ss;
-            named_barrier_sync(1, kWalkCols);
-            if (tid == 0) p.sums[(t * p.heads * p.dv + (size_t)h * p.dv + c0) / 64] = red[0] + red[1];
+            if ((tid & 31) == 0) p.sums[(t * p.heads * p.dv + col) / 32] = ss;
         }
     }
     for (int r = rg; r < p.dk; r += 4) gs[(size_t)r * p.dv] = S[r * kWalkCols + c];
@@ -85,7 +82,6 @@ __global__ void __launch_bounds__(kStepThreads, 2) lightning_step_kernel(const _
     float* sq = sm;                                  // [dk]
     float* sk = sq + p.dk;                           // [dk]
     float* part = sk + p.dk;                         // [8][128]
-    __shared__ float red[4];
     const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * 128;
     if (p.q_len[seq] <= 0) return;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -133,9 +129,7 @@ __global__ void __launch_bounds__(kStepThreads, 2) lightning_step_kernel(const _
         const size_t col = (size_t)h * p.dv + c0 + tid;
         reinterpret_cast<T*>(p.out)[t * p.heads * p.dv + col] = Cvt<T>::from_f(lightning_gate<T>(o, p.norm_w[col], Cvt<T>::to_f(row[p.g_off + col])));
         const float ss = lightning_warp_sum(o * o);
-        if (lane == 0) red[warp] = ss;
-        named_barrier_sync(1, 128);
-        if (tid < 2) p.sums[(t * p.heads * p.dv + (size_t)h * p.dv + c0) / 64 + tid] = red[tid * 2] + red[tid * 2 + 1];
+        if (lane == 0) p.sums[(t * p.heads * p.dv + col) / 32] = ss;
     }
 }
 
@@ -167,7 +161,7 @@ __global__ void __launch_bounds__(256) lightning_act_kernel(const __grid_constan
 
 template <typename T>
 static int run_walk(const LightningParams& p, cudaStream_t stream) {
-    const size_t smem = ((size_t)p.dk * kWalkCols + 2 * p.dk + 4 * kWalkCols + 2) * sizeof(float);
+    const size_t smem = ((size_t)p.dk * kWalkCols + 2 * p.dk + 4 * kWalkCols) * sizeof(float);
     static size_t configured = 48 * 1024;
     if (smem > configured) {
         cudaError_t e = cudaFuncSetAttribute(lightning_walk_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);

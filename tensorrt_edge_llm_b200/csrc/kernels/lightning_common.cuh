@@ -15,7 +15,7 @@ struct LightningParams {
     float* state;              // [slots, heads, dk, dv] fp32
     const float* norm_w;       // [heads * dv] fp32
     void* out;                 // [T, heads * dv]: read-outs times weight and gate
-    float* sums;               // [T, heads * dv / 64]: squares of 64 read-outs each
+    float* sums;               // [T, heads * dv / 32]: squares of 32 read-outs each
     float* carry;              // [sequences, heads, segments, dk, dv] fp32 scratch: states in front of the segments (chunk kernel)
     const int* q_start;
     const int* q_len;

@@ -12,7 +12,8 @@
 // registers.
 //
 // One CTA owns (sequence, head, 128 value features, segment of chunks) and walks its chunks in order.  The state is kept transposed,
-// Sᵀ [128 v, DK]: thread (row r, half) of the eight compute warps holds half of value row r, and serves half of token row r elsewhere.
+// Sᵀ [128 v, DK]: thread (row r, quarter) of the sixteen compute warps holds a quarter of value row r, and serves a quarter of token row r
+// elsewhere.
 // Weighted V needs nothing but V, so the state update is issued before P is ready; the loads of the next chunk start when the last
 // product of this one is done, and run under the state's bookkeeping, the outputs and their gates.
 //
@@ -29,23 +30,20 @@
 namespace telb {
 
 constexpr int kLtL = 128;              // chunk length
-constexpr int kLtThreads = 64 + 256;   // producer, MMA issuer, eight compute warps
-constexpr int kLtCompute = 256;
+constexpr int kLtCompute = 512;        // sixteen compute warps
+constexpr int kLtThreads = 64 + kLtCompute;
 
-// Split eight fp32 values into high and low 16-bit halves of one swizzled 16-byte unit each.
-template <typename T>
+// Split eight fp32 values into high and low bf16 halves of one swizzled 16-byte unit each.  A packed pair is widened by shifts: conversions
+// are the slow instructions here.
+__device__ __forceinline__ void lightning_split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+    hi = Cvt<__nv_bfloat16>::pack2(a, b);
+    lo = Cvt<__nv_bfloat16>::pack2(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
+}
 __device__ __forceinline__ void lightning_split8(const float (&x)[8], uint4& hi, uint4& lo) {
-    float l[8];
-#pragma unroll
-    for (int i = 0; i < 8; ++i) l[i] = x[i] - Cvt<T>::to_f(Cvt<T>::from_f(x[i]));
-    hi.x = Cvt<T>::pack2(x[0], x[1]);
-    hi.y = Cvt<T>::pack2(x[2], x[3]);
-    hi.z = Cvt<T>::pack2(x[4], x[5]);
-    hi.w = Cvt<T>::pack2(x[6], x[7]);
-    lo.x = Cvt<T>::pack2(l[0], l[1]);
-    lo.y = Cvt<T>::pack2(l[2], l[3]);
-    lo.z = Cvt<T>::pack2(l[4], l[5]);
-    lo.w = Cvt<T>::pack2(l[6], l[7]);
+    lightning_split2(x[0], x[1], hi.x, lo.x);
+    lightning_split2(x[2], x[3], hi.y, lo.y);
+    lightning_split2(x[4], x[5], hi.z, lo.z);
+    lightning_split2(x[6], x[7], hi.w, lo.w);
 }
 
 template <int DK, bool STATE_ONLY>
@@ -74,14 +72,16 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_con
     uint8_t* sS = sQ + 32768;                            // Sᵀ hi | Sᵀ lo (at least 32 KB); P lo overlays the first 32 KB
     uint8_t* tail = STATE_ONLY ? sQ : sS + 2 * kAtoms * 16384;
     float* sPw = reinterpret_cast<float*>(tail);         // λ^0 .. λ^128
-    uint64_t* bars = reinterpret_cast<uint64_t*>(tail + 544);
+    float* sNw = sPw + 132;                              // norm weights of the tile's features
+    float* sNear = sNw + 128;                            // λ^31 .. λ^0
+    uint64_t* bars = reinterpret_cast<uint64_t*>(tail + 528 + 512 + 128);
     uint64_t* full_bar = bars;        // inputs of the chunk have landed (TMA)
     uint64_t* g_bar = bars + 1;       // G is in TMEM
     uint64_t* yi_bar = bars + 2;      // Q S_prev is in TMEM
-    uint64_t* w_full = bars + 3;      // weighted V is in shared memory (256 arrivals)
-    uint64_t* p_full = bars + 4;      // P hi, lo are in shared memory (256 arrivals)
+    uint64_t* w_full = bars + 3;      // weighted V is in shared memory (512 arrivals)
+    uint64_t* p_full = bars + 4;      // P hi, lo are in shared memory (512 arrivals)
     uint64_t* y_bar = bars + 5;       // every product of the chunk is done
-    uint64_t* s_ready = bars + 6;     // state copies of the chunk written, TMEM of the chunk before it read (256 arrivals)
+    uint64_t* s_ready = bars + 6;     // state copies of the chunk written, TMEM of the chunk before it read (512 arrivals)
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 8);
     volatile uint32_t* abort_flag = tmem_slot + 1;
 
@@ -100,6 +100,8 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_con
         prefetch_tensormap(&tma);
     }
     for (int i = threadIdx.x; i <= kLtL; i += kLtThreads) sPw[i] = p.powers[(size_t)h * p.n_powers + i];
+    if (threadIdx.x < 32) sNear[threadIdx.x] = p.powers[(size_t)h * p.n_powers + 31 - threadIdx.x];
+    if (!STATE_ONLY && threadIdx.x < 128) sNw[threadIdx.x] = p.norm_w[(size_t)h * p.dv + vt * 128 + threadIdx.x];
     if (warp == 1) {
         tmem_alloc(tmem_slot, 512);
         tmem_relinquish();
@@ -200,11 +202,10 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_con
             __syncwarp();
         }
     } else {
-        // ---------------- compute threads: token row r of the chunk, value row r of the state, half of the columns ----------------
-        const int quad = warp & 3, half = (warp - 2) >> 2;
+        // ---------------- compute threads: token row r of the chunk, value row r of the state, a quarter of the columns ----------------
+        const int quad = warp & 3, quarter = (warp - 2) >> 2;
         const int r = quad * 32 + lane;
         const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(quad * 32) << 16);
-        const uint32_t row_off = (r >> 3) * 1024 + (r & 7) * 128;
         bool ok = true;
         auto wait = [&](uint64_t* bar, uint32_t parity) {
             const bool got = ok && mbar_wait(bar, parity, abort_flag, p.status, kStatusEpilogueTimeout);
@@ -212,8 +213,11 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_con
             if (ok) tc_fence_after_sync();
             return ok;
         };
-        auto unit = [&](int c8) { return row_off + (((c8 & 7) ^ (r & 7)) << 4); };      // 16-byte unit c8 of row r within its atom
-        constexpr int kOwn = DK / 2;                                     // key features of the state row that this thread holds
+        // 16-byte unit j (of four) of this quarter in row `row` of a 128-column tile
+        auto unit = [&](int row, int j) {
+            return (quarter >> 1) * 16384 + (row >> 3) * 1024 + (row & 7) * 128 + ((((quarter & 1) * 4 + j) ^ (row & 7)) << 4);
+        };
+        constexpr int kOwn = DK / 4;                                     // key features of the state row that this thread holds
         const size_t sh_off = (size_t)h * DK * p.dv + vt * 128 + r;      // column r of this tile, rows p.dv apart
         const size_t per_seq = (size_t)p.heads * DK * p.dv;
         float* carry = p.carry + ((size_t)(seq * p.heads + h) * p.segments + seg) * DK * p.dv + vt * 128 + r;
@@ -223,7 +227,7 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_con
             const float* src = p.segments > 1 ? carry : slot;
             const bool zero = STATE_ONLY || (p.segments == 1 && p.past_len[seq] <= 0);
 #pragma unroll
-            for (int j = 0; j < kOwn; ++j) S[j] = zero ? 0.f : src[(size_t)(half * kOwn + j) * p.dv];
+            for (int j = 0; j < kOwn; ++j) S[j] = zero ? 0.f : src[(size_t)(quarter * kOwn + j) * p.dv];
         }
         auto publish_state = [&]() {
             if (!STATE_ONLY) {
@@ -233,9 +237,9 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_con
 #pragma unroll
                     for (int i = 0; i < 8; ++i) x[i] = S[q * 8 + i];
                     uint4 hi, lo;
-                    lightning_split8<T>(x, hi, lo);
-                    const int c8 = half * (kOwn / 8) + q;
-                    uint8_t* dst = sS + (c8 >> 3) * 16384 + unit(c8);
+                    lightning_split8(x, hi, lo);
+                    const int c8 = quarter * (kOwn / 8) + q;
+                    uint8_t* dst = sS + (c8 >> 3) * 16384 + (r >> 3) * 1024 + (r & 7) * 128 + (((c8 & 7) ^ (r & 7)) << 4);
                     *reinterpret_cast<uint4*>(dst) = hi;
                     *reinterpret_cast<uint4*>(dst + kAtoms * 16384) = lo;
                 }
@@ -250,126 +254,156 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tma, const __grid_con
             const int len = min(kLtL, ql - c * kLtL);
             const size_t t = (size_t)t_first + (size_t)c * kLtL + r;
             const bool valid = r < len;
-            // ---- weighted V (64 features of token r) ----
+            // ---- weighted V (32 features of token r) ----
             if (!wait(full_bar, par)) break;
             {
                 const float wgt = valid ? sPw[len - 1 - r] : 0.f;
 #pragma unroll
-                for (int q = 0; q < 8; ++q) {
-                    const uint32_t off = half * 16384 + unit(q);
+                for (int q = 0; q < 4; ++q) {
+                    const uint32_t off = unit(r, q);
                     const uint4 vu = *reinterpret_cast<const uint4*>(sV + off);
                     const T* ve = reinterpret_cast<const T*>(&vu);
                     float x[8];
 #pragma unroll
                     for (int i = 0; i < 8; ++i) x[i] = valid ? Cvt<T>::to_f(ve[i]) * wgt : 0.f;
                     uint4 hi, lo;
-                    lightning_split8<T>(x, hi, lo);
+                    lightning_split8(x, hi, lo);
                     *reinterpret_cast<uint4*>(sW + off) = hi;
                     *reinterpret_cast<uint4*>(sW + 32768 + off) = lo;
                 }
                 fence_proxy_async_smem();
                 mbar_arrive(w_full);
             }
-            float o[STATE_ONLY ? 1 : 64];
+            // gates of this warp's 32 rows, fetched under the products: four lanes share a row, eight rows at a time
+            uint4 gate[STATE_ONLY ? 1 : 4];
+            const size_t col = (size_t)h * p.dv + vt * 128 + quarter * 32;
+            const int row_first = c * kLtL + quad * 32 + (lane >> 2);       // this lane's first row of the segment
             if constexpr (!STATE_ONLY) {
                 // ---- P = G ∘ decays: computed under Q S, stored when that has read Q and the state copies ----
                 if (!wait(g_bar, par)) break;
-                uint4 hi[8], lo[8];
+                uint4 hi[4], lo[4];
+                const int c0 = quarter * 32;
+                if (c0 > quad * 32) {                               // wholly above the diagonal
 #pragma unroll
-                for (int g = 0; g < 2; ++g) {
-                    const int c0 = half * 64 + g * 32;              // 32 chunk columns at a time
-                    if (c0 > quad * 32 + 31) {                      // wholly above the diagonal for this warp
+                    for (int q = 0; q < 4; ++q) hi[q] = lo[q] = make_uint4(0, 0, 0, 0);
+                } else {
 #pragma unroll
-                        for (int q = 0; q < 4; ++q) hi[g * 4 + q] = lo[g * 4 + q] = make_uint4(0, 0, 0, 0);
-                        continue;
-                    }
-                    uint32_t gr[32];
-                    tmem_ld_x32(lane_addr + kColG + c0, gr);
-                    tmem_ld_wait();
+                    for (int g = 0; g < 2; ++g) {
+                        uint32_t gr[16];
+                        tmem_ld_x16(lane_addr + kColG + c0 + g * 16, gr);
+                        tmem_ld_wait();
+                        if (c0 == quad * 32) {                      // the diagonal runs through these columns
 #pragma unroll
-                    for (int q = 0; q < 4; ++q) {
-                        float e[8];
+                            for (int q = 0; q < 2; ++q) {
+                                float e[8];
 #pragma unroll
-                        for (int i = 0; i < 8; ++i) {
-                            const int s = c0 + q * 8 + i;
-                            e[i] = s <= r ? __uint_as_float(gr[q * 8 + i]) * sPw[max(r - s, 0)] : 0.f;
+                                for (int i = 0; i < 8; ++i) {
+                                    const int s = g * 16 + q * 8 + i;
+                                    e[i] = s <= lane ? __uint_as_float(gr[q * 8 + i]) * sPw[max(lane - s, 0)] : 0.f;
+                                }
+                                lightning_split8(e, hi[g * 2 + q], lo[g * 2 + q]);
+                            }
+                        } else {                                    // λ^{r-s} = λ^{r-c0-31} λ^{c0+31-s}, the second the same for all rows
+                            const float far = sPw[r - c0 - 31];
+#pragma unroll
+                            for (int q = 0; q < 2; ++q) {
+                                float e[8];
+                                const float4* np = reinterpret_cast<const float4*>(sNear + g * 16 + q * 8);
+                                const float4 d0 = np[0], d1 = np[1];
+                                const float d[8] = {d0.x, d0.y, d0.z, d0.w, d1.x, d1.y, d1.z, d1.w};
+#pragma unroll
+                                for (int i = 0; i < 8; ++i) e[i] = __uint_as_float(gr[q * 8 + i]) * (far * d[i]);
+                                lightning_split8(e, hi[g * 2 + q], lo[g * 2 + q]);
+                            }
                         }
-                        lightning_split8<T>(e, hi[g * 4 + q], lo[g * 4 + q]);
                     }
                 }
                 tc_fence_before_sync();
                 if (!wait(yi_bar, par)) break;
 #pragma unroll
-                for (int q = 0; q < 8; ++q) {
-                    const uint32_t off = half * 16384 + unit(q);
+                for (int q = 0; q < 4; ++q) {
+                    const uint32_t off = unit(r, q);
                     *reinterpret_cast<uint4*>(sQ + off) = hi[q];
                     *reinterpret_cast<uint4*>(sS + off) = lo[q];
                 }
                 fence_proxy_async_smem();
                 mbar_arrive(p_full);
+                const T* gp = reinterpret_cast<const T*>(p.rows) + ((size_t)t_first + row_first) * p.ld + p.g_off + col + (lane & 3) * 8;
+#pragma unroll
+                for (int q = 0; q < 4; ++q)
+                    gate[q] = row_first + q * 8 < ql ? __ldg(reinterpret_cast<const uint4*>(gp + (size_t)q * 8 * p.ld)) : make_uint4(0, 0, 0, 0);
             }
             if (!wait(y_bar, par)) break;
+            float o[STATE_ONLY ? 1 : 32];
             if constexpr (!STATE_ONLY) {
                 // ---- read-outs: P V + λ^{r+1} Q S ----
                 const float carry_in = sPw[r + 1];
 #pragma unroll
                 for (int g = 0; g < 2; ++g) {
-                    uint32_t y[32], yi[32];
-                    tmem_ld_x32(lane_addr + kColY + half * 64 + g * 32, y);
-                    tmem_ld_x32(lane_addr + kColYI + half * 64 + g * 32, yi);
+                    uint32_t y[16], yi[16];
+                    tmem_ld_x16(lane_addr + kColY + quarter * 32 + g * 16, y);
+                    tmem_ld_x16(lane_addr + kColYI + quarter * 32 + g * 16, yi);
                     tmem_ld_wait();
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) o[g * 32 + i] = fmaf(carry_in, __uint_as_float(yi[i]), __uint_as_float(y[i]));
+                    for (int i = 0; i < 16; ++i) o[g * 16 + i] = fmaf(carry_in, __uint_as_float(yi[i]), __uint_as_float(y[i]));
                 }
             }
             // ---- state: decayed in registers, plus the update ----
             {
                 const float keep = sPw[len];
 #pragma unroll
-                for (int g = 0; g < kOwn / 32; ++g) {
-                    uint32_t u[32];
-                    tmem_ld_x32(lane_addr + kColS + half * kOwn + g * 32, u);
+                for (int g = 0; g < kOwn / 16; ++g) {
+                    uint32_t u[16];
+                    tmem_ld_x16(lane_addr + kColS + quarter * kOwn + g * 16, u);
                     tmem_ld_wait();
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) S[g * 32 + i] = fmaf(keep, S[g * 32 + i], __uint_as_float(u[i]));
+                    for (int i = 0; i < 16; ++i) S[g * 16 + i] = fmaf(keep, S[g * 16 + i], __uint_as_float(u[i]));
                 }
             }
             if (c + 1 < nchunks) publish_state();
             if constexpr (!STATE_ONLY) {
-                // ---- outputs, under the next chunk's loads and first products ----
-                if (valid) {
-                    const size_t col = (size_t)h * p.dv + vt * 128 + half * 64, width = (size_t)p.heads * p.dv;
-                    const uint4* gp = reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(p.rows) + t * p.ld + p.g_off + col);
-                    const float4* wp = reinterpret_cast<const float4*>(p.norm_w + col);
-                    uint4* op = reinterpret_cast<uint4*>(reinterpret_cast<T*>(p.out) + t * width + col);
-                    float part[4] = {0.f, 0.f, 0.f, 0.f};
+                // ---- outputs, under the next chunk's loads and first products.  The products have read the weighted V; in the units that
+                // only this warp writes there, lanes that fetched pieces of rows pass them to the rows' lanes and take the results back ----
+                const size_t width = (size_t)p.heads * p.dv;
 #pragma unroll
-                    for (int q = 0; q < 8; ++q) {
-                        const uint4 gu = gp[q];
-                        const T* ge = reinterpret_cast<const T*>(&gu);
-                        const float4 w0 = wp[q * 2], w1 = wp[q * 2 + 1];
-                        const float w8[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
-                        float y[8];
+                for (int q = 0; q < 4; ++q) *reinterpret_cast<uint4*>(sW + unit(quad * 32 + q * 8 + (lane >> 2), lane & 3)) = gate[q];
+                __syncwarp();
+                float part[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-                        for (int i = 0; i < 8; ++i) {
-                            part[i & 3] = fmaf(o[q * 8 + i], o[q * 8 + i], part[i & 3]);
-                            y[i] = lightning_gate<T>(o[q * 8 + i], w8[i], Cvt<T>::to_f(ge[i]));
-                        }
-                        uint4 ou;
-                        ou.x = Cvt<T>::pack2(y[0], y[1]);
-                        ou.y = Cvt<T>::pack2(y[2], y[3]);
-                        ou.z = Cvt<T>::pack2(y[4], y[5]);
-                        ou.w = Cvt<T>::pack2(y[6], y[7]);
-                        op[q] = ou;
+                for (int q = 0; q < 4; ++q) {
+                    uint4* mine = reinterpret_cast<uint4*>(sW + unit(r, q));
+                    const uint4 gu = *mine;
+                    const T* ge = reinterpret_cast<const T*>(&gu);
+                    const float4* wp = reinterpret_cast<const float4*>(sNw + quarter * 32 + q * 8);
+                    const float4 w0 = wp[0], w1 = wp[1];
+                    const float w8[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+                    float y[8];
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {
+                        part[i & 3] = fmaf(o[q * 8 + i], o[q * 8 + i], part[i & 3]);
+                        y[i] = lightning_gate<T>(o[q * 8 + i], w8[i], Cvt<T>::to_f(ge[i]));
                     }
-                    p.sums[(t * width + col) / 64] = (part[0] + part[1]) + (part[2] + part[3]);
+                    uint4 ou;
+                    ou.x = Cvt<T>::pack2(y[0], y[1]);
+                    ou.y = Cvt<T>::pack2(y[2], y[3]);
+                    ou.z = Cvt<T>::pack2(y[4], y[5]);
+                    ou.w = Cvt<T>::pack2(y[6], y[7]);
+                    *mine = ou;
                 }
+                if (valid) p.sums[(t * width + col) / 32] = (part[0] + part[1]) + (part[2] + part[3]);
+                __syncwarp();
+                T* op = reinterpret_cast<T*>(p.out) + ((size_t)t_first + row_first) * width + col + (lane & 3) * 8;
+#pragma unroll
+                for (int q = 0; q < 4; ++q)
+                    if (row_first + q * 8 < ql)
+                        *reinterpret_cast<uint4*>(op + (size_t)q * 8 * width) = *reinterpret_cast<const uint4*>(sW + unit(quad * 32 + q * 8 + (lane >> 2), lane & 3));
+                __syncwarp();                             // before this warp's next weighted V
             }
         }
         if (ok && (STATE_ONLY || last_seg)) {
             float* dst = STATE_ONLY ? carry : slot;
 #pragma unroll
-            for (int j = 0; j < kOwn; ++j) dst[(size_t)(half * kOwn + j) * p.dv] = S[j];
+            for (int j = 0; j < kOwn; ++j) dst[(size_t)(quarter * kOwn + j) * p.dv] = S[j];
         }
     }
 
@@ -400,17 +434,26 @@ __global__ void __launch_bounds__(256) lightning_carry_kernel(const __grid_const
     float4 cur = make_float4(0.f, 0.f, 0.f, 0.f);
     if (p.past_len[seq] > 0) cur = *reinterpret_cast<const float4*>(p.state + ((size_t)p.slot_ids[seq] * p.heads + h) * size + e);
     float* seg = p.carry + (size_t)sh * p.segments * size + e;
-    for (int s = 0; s < n; ++s, seg += size) {
-        float4 local = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (s + 1 < n) local = *reinterpret_cast<const float4*>(seg);
-        *reinterpret_cast<float4*>(seg) = cur;
-        cur = make_float4(fmaf(cur.x, keep, local.x), fmaf(cur.y, keep, local.y), fmaf(cur.z, keep, local.z), fmaf(cur.w, keep, local.w));
+    constexpr int kAhead = 8;                             // segments whose loads are in flight together
+    for (int s0 = 0; s0 < n; s0 += kAhead) {
+        float4 local[kAhead];
+#pragma unroll
+        for (int i = 0; i < kAhead; ++i) {
+            local[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (s0 + i + 1 < n) local[i] = *reinterpret_cast<const float4*>(seg + (size_t)(s0 + i) * size);
+        }
+#pragma unroll
+        for (int i = 0; i < kAhead; ++i) {
+            if (s0 + i >= n) break;
+            *reinterpret_cast<float4*>(seg + (size_t)(s0 + i) * size) = cur;
+            cur = make_float4(fmaf(cur.x, keep, local[i].x), fmaf(cur.y, keep, local[i].y), fmaf(cur.z, keep, local[i].z), fmaf(cur.w, keep, local[i].w));
+        }
     }
 }
 
 template <int DK, bool STATE_ONLY>
 static int launch_lightning(const CUtensorMap& tma, const LightningParams& p, cudaStream_t stream) {
-    constexpr int smem = DK / 64 * 16384 + 32768 + 65536 + (STATE_ONLY ? 0 : 32768 + DK / 64 * 32768) + 544 + 128 + 1024;
+    constexpr int smem = DK / 64 * 16384 + 32768 + 65536 + (STATE_ONLY ? 0 : 32768 + DK / 64 * 32768) + 528 + 512 + 128 + 128 + 1024;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(lightning_chunk_kernel<DK, STATE_ONLY>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);

@@ -229,7 +229,7 @@ def stream_post(stream, delta, weight, groups, eps, meta, dtype, *, ids=None, ta
 
 def lightning(rows, norm_w, powers, state, meta):
     """Linear attention with a constant decay per head over packed ``[q | k | v | g]`` rows: silu on q, k and v, the recurrence, weight and
-    sigmoid gate.  Returns ``(u [T, heads · dv], sums [T, heads · dv / 64])``: the gated read-outs before the RMS norm over all heads of a
+    sigmoid gate.  Returns ``(u [T, heads · dv], sums [T, heads · dv / 32])``: the gated read-outs before the RMS norm over all heads of a
     row, and sums of squares of the read-outs; the norm's division commutes with the output projection and is left to the consumer
     (:func:`stream_post`).  ``powers`` ``[heads, n + 1]``: powers of the decays from 0 on; ``state`` ``[seats, heads, dk, dv]`` is
     advanced in place."""

@@ -1193,7 +1193,7 @@ def lightning(rows, norm_w, powers, state, meta: StepMeta, kernel: Optional[str]
     if (kernel == "step" and meta.max_q_len != 1) or (kernel == "chunk" and not chunk_ok):
         raise ValueError(f"the {kernel} kernel does not cover this step")
     out = torch.empty(t, n * dv, dtype=rows.dtype, device=dev)
-    sums = torch.empty(t, n * dv // 64, dtype=f32, device=dev)
+    sums = torch.empty(t, n * dv // 32, dtype=f32, device=dev)
     act = carry = None
     segs, per, launches = 1, 0, 1
     if kernel == "chunk":

@@ -667,7 +667,7 @@ def lightning(rows, norm_w, powers, state, meta: StepMeta):
         if ql:
             state[slot] = S
     o = o.reshape(t, n * dv)
-    return (o * norm_w * torch.sigmoid(g)).to(rows.dtype), o.pow(2).reshape(t, -1, 64).sum(-1)
+    return (o * norm_w * torch.sigmoid(g)).to(rows.dtype), o.pow(2).reshape(t, -1, 32).sum(-1)
 
 
 # ------------------------------------------------------------------------------------------
