@@ -75,7 +75,7 @@ def _meta(q_lens, past, device):
 def kernel_pairs(device) -> list:
     """One row per kernel or kernel group: time, roofline and the counterpart's."""
     from ..config import MoeConfig, qwen3_30b_a3b_config
-    from ..models.qwen3_moe import ClampedExperts, MoEBlock
+    from ..models.qwen3_moe import GatedExperts, MoEBlock
     from ..ops import cuda as cu
     bw, fl = peaks()
     s, dt, n, d = SIZES, torch.bfloat16, SIZES["heads"], 128
@@ -148,7 +148,7 @@ def kernel_pairs(device) -> list:
                                     num_hidden_layers=1)
         gen = torch.Generator().manual_seed(0)
         with torch.device(device):
-            ours = [ClampedExperts(cfg, MoeConfig(s["experts"], s["top_k"], s["inter"], 7.0), "m") for _ in range(2)]
+            ours = [GatedExperts(cfg, MoeConfig(s["experts"], s["top_k"], s["inter"], 7.0), "m") for _ in range(2)]
             theirs = [MoEBlock(qcfg, "m") for _ in range(2)]
         for m in ours + theirs:
             m.random_init(gen)

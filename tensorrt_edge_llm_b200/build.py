@@ -30,7 +30,7 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
               "-diag-suppress", "177", "-diag-suppress", "550"]
 # sources compiled without --use_fast_math: their exponentials, tanh and divisions feed routers, norms and recurrences
 NO_FAST_MATH: set = {"attention_simt.cu", "channel_delta.cu", "gemm_f32.cu", "latent.cu", "lightning.cu", "lightning_tc5.cu", "mlstm.cu",
-                      "mlstm_tc5.cu", "moe.cu", "stream_norm.cu", "stream_post.cu"}
+                      "mlstm_tc5.cu", "moe.cu", "stream_norm.cu", "stream_post.cu", "stream_sandwich.cu"}
 
 
 def _newer(src: str, dst: str, deps: List[str]) -> bool:
@@ -55,6 +55,8 @@ KERNEL_SETS = {
                 "stream_post.cu"],
     "debonex": ["attention_decode_tc5.cu", "attention_latent_tc5.cu", "attention_simt.cu", "attention_tc5.cu", "attention_tc5_extra.cu",
                 "channel_delta.cu", "elementwise.cu", "gemm_f32.cu", "gemm_skinny_tc5.cu", "gemm_tc5.cu", "latent.cu", "nvfp4_host.cu", "stream_norm.cu"],
+    "ditenex": ["attention_mixed_tc5.cu", "attention_simt.cu", "elementwise.cu", "gemm_f32.cu", "gemm_skinny_tc5.cu", "gemm_tc5.cu", "mixed_heads.cu", "moe.cu",
+                "nvfp4_host.cu", "stream_sandwich.cu"],
     "dimesun": ["attention_decode_tc5.cu", "attention_simt.cu", "attention_tc5.cu", "attention_tc5_extra.cu", "elementwise.cu", "gemm_f32.cu",
                 "gemm_skinny_tc5.cu", "gemm_tc5.cu", "mlstm.cu", "mlstm_tc5.cu", "moe.cu", "nvfp4_host.cu", "stream_norm.cu"],
 }

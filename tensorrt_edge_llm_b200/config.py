@@ -229,6 +229,11 @@ class AttentionConfig:
     interleaved: bool = False        # rotated pairs are neighbours (2i, 2i + 1)
     rope_factor: float = 1.0         # linear scaling: every frequency of queries and keys over this
     rotated_values: bool = False     # values turn by their position over all v_head_dim features, outputs turn back by theirs
+    mixed_scores: bool = False       # a head's scores are a learned combination of all heads' scores, taken before the softmax
+    distance_bias: bool = False      # scores lose slope * distance, slope 2^(-8 (h + 1) / heads) for head h (before they are mixed)
+    value_mix: bool = False          # values join with those of the first such layer, by a learned share
+    qkv_bias: bool = False           # the query, key and value projections have biases
+    out_gate: bool = False           # heads times sigmoid(gate projection of the layer's input) before the output projection
 
     @property
     def pad(self) -> int:
@@ -334,8 +339,16 @@ class MoeConfig:
     num_experts: int = 8
     top_k: int = 2
     intermediate_size: int = 64
-    limit: float = 7.0               # clamped gated unit: gate <= limit, |up| <= limit
-    alpha: float = 1.702             # gate * sigmoid(alpha * gate) * (up + 1)
+    limit: float = 7.0               # clamped gated unit: gate <= limit, |up| <= limit (0 = no clamp)
+    alpha: float = 1.702             # gate * sigmoid(alpha * gate) * (up + up_offset)
+    up_offset: float = 1.0
+    # "chosen": weights are the softmax over the chosen logits.  "sigmoid_groups": scores sigmoid(logit); choice by score + correction
+    # within the keep_groups best of `groups` equal groups (a group's worth: its two best); weights weight_scale * score
+    router: str = "chosen"
+    groups: int = 1
+    keep_groups: int = 1
+    weight_scale: float = 1.0
+    shared_size: int = 0             # one more gated unit (silu) of this size that every token passes through
 
     @property
     def inter_pad(self) -> int:
@@ -352,8 +365,8 @@ class LayerConfig:
     moe: Optional[MoeConfig] = None
     latent: Optional[LatentConfig] = None              # kind "attention" over cached latents
     delta: Optional[ChannelDeltaConfig] = None
-    ff: int = 0                                        # dense gated feed-forward of this size
-    ff_act: str = "gelu_tanh"                          # its gate: "gelu_tanh" or "relu"
+    ff: int = 0                                        # dense feed-forward of this size
+    ff_act: str = "gelu_tanh"                          # gated by "gelu_tanh" or "relu", or "xielu" without a gate
     ff_bias: bool = False                              # its projections have biases
     lightning: Optional[LightningConfig] = None
     attention_mult: float = 1.0                        # kind "parallel": the layer's output is attention_mult * attention
@@ -442,6 +455,8 @@ class ModelConfig:
     logits_mult: float = 1.0                # logits are this multiple of the head's output
     norm_groups: int = 1                    # RMS norms of the stream go over this many equal parts of a row
     input_conv: int = 0                     # taps of the causal convolution that every mixer's input is added to (0 = none)
+    token_shift: bool = False               # features of a mixer's input move by learned shares towards the row before
+    learned_positions: bool = False         # a table row per position joins the token's embedding: no position beyond the table exists
     # bigram table: row (previous token * bigram_mul_prev + token * bigram_mul_cur) mod bigram_buckets joins the token's embedding,
     # row bigram_buckets for a sequence's first token (0 = none)
     bigram_buckets: int = 0
@@ -576,7 +591,8 @@ class ModelConfig:
 
     @property
     def is_hybrid(self) -> bool:
-        return any(t != LAYER_ATTENTION for t in self.layer_types)
+        """Sequences have state rows besides their pages."""
+        return self.token_shift or any(t != LAYER_ATTENTION for t in self.layer_types)
 
     @property
     def is_moe(self) -> bool:
@@ -651,6 +667,8 @@ class ModelConfig:
             return _parse_debonex(cls, hf, quant)
         if str(hf.get("architecture", "")) == "Begupel":
             return _parse_begupel(cls, hf, quant)
+        if str(hf.get("architecture", "")) == "Ditenex":
+            return _parse_ditenex(cls, hf, quant)
         llm = hf.get("text_config", hf)
         model_type = llm.get("model_type", hf.get("model_type", "llama"))
         heads = int(llm["num_attention_heads"])
@@ -1075,6 +1093,59 @@ def _begupel_stack(specs: List[LayerConfig]) -> Dict[str, Any]:
                 layer_types=[sp.kind for sp in specs], mlp_types=[LAYER_MLP if sp.ff else "none" for sp in specs], layer_specs=specs)
 
 
+def _parse_ditenex(cls, hf: Dict[str, Any], quant: Optional["QuantConfig"]) -> "ModelConfig":
+    """Ditenex: layers listed one by one with a norm in front of and behind every sublayer and a token shift before every mixer; windowed
+    attention with mixed scores, a distance bias, mixed values and an output gate; dense xIELU feed-forwards or experts behind a
+    group-limited sigmoid router beside a shared one; learned positions, tied embeddings."""
+    specs: List[LayerConfig] = []
+    for i, entry in enumerate(hf["layers"]):
+        m, f, kind = entry["mixer"], entry.get("mlp"), str(entry["type"])
+        if kind != LAYER_ATTENTION:
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        spec = LayerConfig(kind=kind)
+        spec.attention = a = AttentionConfig(
+            num_heads=int(m["heads"]), num_kv_heads=int(m["kv_heads"]), head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]), rotary_dim=0,
+            scale=float(m["scale"]), fp32_weights=True, window=int(m["mask"]["size"]), mixed_scores=True, distance_bias=True,
+            value_mix=bool(m.get("v_mix", False)), qkv_bias=True, out_gate=True)
+        if a.num_heads % a.num_kv_heads or a.window < 1:
+            raise ValueError(f"layer {i}: query heads must be a multiple of the KV heads, and a position sees at least itself")
+        if f:
+            what = str(f.get("kind", "dense"))
+            if what == "dense":
+                spec.ff, spec.ff_act = int(f["ff"]), "xielu"
+            elif what == "moe":
+                r = f["router"]
+                g = r.get("groups") or {}
+                spec.moe = e = MoeConfig(int(r["experts"]), int(r["top"]), int(f["expert"]["ff"]), 0.0, 1.0, 0.0, router="sigmoid_groups",
+                                         groups=int(g.get("count", 1)), keep_groups=int(g.get("keep", 1)), weight_scale=float(r.get("scale", 1.0)),
+                                         shared_size=int((f.get("shared") or {}).get("ff", 0)))
+                if e.groups < 1 or e.num_experts % e.groups or not 1 <= e.keep_groups <= e.groups:
+                    raise ValueError(f"layer {i}: experts fall into equal groups, of which at least one is kept")
+                if not 1 <= e.top_k <= e.num_experts // e.groups * e.keep_groups:
+                    raise ValueError(f"layer {i}: the kept groups must hold the experts that a token uses")
+            else:
+                raise ValueError(f"layer {i}: unknown feed-forward kind {what!r}")
+        specs.append(spec)
+    mixing = [(sp.attention.num_kv_heads, sp.attention.v_head_dim) for sp in specs if sp.attention.value_mix]
+    if len(set(mixing)) > 1:
+        raise ValueError("layers that mix values have equally many value heads of one size")
+    torch_dtype = str(hf.get("torch_dtype", hf.get("dtype", "bfloat16"))).replace("torch.", "")
+    base = dict(vocab_size=int(hf["vocab"]), hidden_size=int(hf["width"]), rms_norm_eps=float(hf["norm"]["eps"]),
+                residual_mult=float(hf.get("residual_mult", 1.0)), max_position_embeddings=int(hf["max_positions"]),
+                dtype=torch_dtype if torch_dtype in ("bfloat16", "float16", "float32") else "bfloat16",
+                quant=quant or QuantConfig(), bos_token_id=hf.get("bos_token_id"), eos_token_id=hf.get("eos_token_id"))
+    return cls(**base, **_ditenex_stack(specs))
+
+
+def _ditenex_stack(specs: List[LayerConfig]) -> Dict[str, Any]:
+    """Model-wide fields that follow from the layers."""
+    a = specs[0].attention
+    return dict(model_type="ditenex", intermediate_size=max((sp.ff for sp in specs), default=0), num_hidden_layers=len(specs),
+                num_attention_heads=a.num_heads, num_key_value_heads=a.num_kv_heads, head_dim=a.pad, hidden_act="xielu", token_shift=True,
+                learned_positions=True, tie_word_embeddings=True, layer_types=[sp.kind for sp in specs],
+                mlp_types=[LAYER_MLP if sp.ff else LAYER_MOE if sp.moe else "none" for sp in specs], layer_specs=specs)
+
+
 def _parse_dspark(llm: dict, hf: dict) -> dict:
     """DSpark draft fields (``dspark_config``, a top-level ``markov_head_type`` or an architecture named ``…DSparkModel``;
     ``tensorrt_edgellm/config.py:1880-1905``): the block geometry may sit at the top level instead of in ``dflash_config``, labels
@@ -1340,6 +1411,24 @@ def begupel_config(layers: int = 12, hidden: int = 2048, vocab: int = 32768, hea
                 bigram_buckets=65536, bigram_mul_prev=1000003, bigram_mul_cur=8191)
     base.update(over)
     return ModelConfig(**{**_begupel_stack(specs), **base})
+
+
+def ditenex_config(layers: int = 12, hidden: int = 2048, vocab: int = 32768, heads: int = 16, inter: int = 6144, experts: int = 64, top_k: int = 4,
+                   expert_inter: int = 768, window: int = 1024, **over: Any) -> ModelConfig:
+    """Ditenex at the sizes of a small production model: four query heads per KV head, d 128; dense feed-forwards and experts (eight groups,
+    four kept) with a shared one in turn."""
+    specs = []
+    for i in range(layers):
+        a = AttentionConfig(heads, max(heads // 4, 1), 128, 128, 0, 1e4, 128 ** -0.5, fp32_weights=True, window=window, mixed_scores=True,
+                            distance_bias=True, value_mix=True, qkv_bias=True, out_gate=True)
+        if i % 2 == 0:
+            specs.append(LayerConfig(LAYER_ATTENTION, attention=a, ff=inter, ff_act="xielu"))
+        else:
+            specs.append(LayerConfig(LAYER_ATTENTION, attention=a, moe=MoeConfig(
+                experts, top_k, expert_inter, 0.0, 1.0, 0.0, router="sigmoid_groups", groups=8, keep_groups=4, weight_scale=2.0, shared_size=expert_inter)))
+    base = dict(vocab_size=vocab, hidden_size=hidden, rms_norm_eps=1e-6, residual_mult=0.5, max_position_embeddings=16384)
+    base.update(over)
+    return ModelConfig(**{**_ditenex_stack(specs), **base})
 
 
 def hybrid_nemotron_config(**over: Any) -> ModelConfig:

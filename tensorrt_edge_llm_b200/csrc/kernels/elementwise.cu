@@ -204,6 +204,31 @@ __global__ void geglu_kernel(const T* __restrict__ in, T* __restrict__ out, long
     }
 }
 
+// xIELU: coef[0] x² + x / 2 above zero, coef[1] (exp(x) - 1 - x) + x / 2 below.
+__global__ void xielu_f32_kernel(const float* __restrict__ in, float* __restrict__ out, long long n, const float* __restrict__ coef) {
+    pdl_prologue();
+    const float a = coef[0], b = coef[1];
+    for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+        const float x = in[i], pos = fmaxf(x, 0.f), neg = fminf(x, 0.f);
+        out[i] = fmaf(a * pos, pos, fmaf(b, expm1f(neg) - neg, 0.5f * x));
+    }
+}
+template <typename T>
+__global__ void xielu_kernel(const T* __restrict__ in, T* __restrict__ out, long long n, const float* __restrict__ coef) {
+    pdl_prologue();
+    const float a = coef[0], b = coef[1];
+    for (long long i = (blockIdx.x * (long long)blockDim.x + threadIdx.x) * 8; i < n; i += (long long)gridDim.x * blockDim.x * 8) {
+        Vec8<T> v, o;
+        v.load(in + i);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const float x = v.get(j), pos = fmaxf(x, 0.f), neg = fminf(x, 0.f);
+            o.set(j, fmaf(a * pos, pos, fmaf(b, __expf(neg) - 1.f - neg, 0.5f * x)));
+        }
+        o.store(out + i);
+    }
+}
+
 template <typename T>
 __global__ void relu2_kernel(const T* __restrict__ in, T* __restrict__ out, long long n) {
     pdl_prologue();
@@ -718,6 +743,21 @@ extern "C" int telb_geglu(const void* in, void* out, long long rows, int inter, 
     if (blocks > 148 * 16) blocks = 148 * 16;
     DISPATCH_T(is_bf16, { TELB_LAUNCH("geglu_kernel", (geglu_kernel<T>), dim3((int)blocks), dim3(256), 0, stream, (const T*)in, (T*)out, rows, inter, kind); })
     TELB_CHECK_LAUNCH("geglu_kernel");
+    return 0;
+}
+
+// dtype: 0 fp16, 1 bf16, 2 fp32.  coef: two fp32 factors on the device.
+extern "C" int telb_xielu(const void* in, void* out, long long n, const float* coef, int dtype, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (n % 8) return fail("telb_xielu: element count must be a multiple of 8");
+    const long long units = dtype == 2 ? n : n / 8;
+    long long blocks = (units + 255) / 256;
+    if (blocks > 148 * 16) blocks = 148 * 16;
+    if (dtype == 2)
+        TELB_LAUNCH("xielu_f32_kernel", xielu_f32_kernel, dim3((int)blocks), dim3(256), 0, stream, (const float*)in, (float*)out, n, coef);
+    else
+        DISPATCH_T(dtype, { TELB_LAUNCH("xielu_kernel", (xielu_kernel<T>), dim3((int)blocks), dim3(256), 0, stream, (const T*)in, (T*)out, n, coef); })
+    TELB_CHECK_LAUNCH("xielu_kernel");
     return 0;
 }
 

@@ -44,7 +44,7 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, float* __restrict
     for (int e = lane; e < experts; e += 32) {
         const float x = Cvt<T>::to_f(row[e]);
         float p;
-        if (sigmoid) p = 1.f / (1.f + __expf(-x));
+        if (sigmoid) p = 1.f / (1.f + expf(-x));
         else { p = __expf(x - mx); sum += p; }
         prob[e] = p;
     }
@@ -102,6 +102,7 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, float* __restrict
             const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
         }
+        bi = min(bi, experts - 1);                            // no number among the logits: any expert
         const float w = prob[bi];
         my_w[r] = w;
         my_i[r] = bi;
@@ -157,11 +158,12 @@ __global__ void moe_route_chosen_kernel(const float* __restrict__ logits, int ld
 }
 
 // Clamped gated unit over [gate I | up I] rows of the padded expert layout (or plain rows): with g = min(gate, limit) and
-// u = clamp(up, ±limit), out = g · σ(alpha g) · (u + 1).  Rows that hold no routed token are skipped.
+// u = clamp(up, ±limit) (limit 0: as they are), out = g · σ(alpha g) · (u + up_offset).  Rows that hold no routed token are skipped.
 template <typename T>
 __global__ void clamped_glu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, const int* __restrict__ tile_rows, int rows, int inter,
-                                   float limit, float alpha) {
+                                   float limit, float alpha, float up_offset) {
     pdl_prologue();
+    if (limit <= 0.f) limit = INFINITY;
     const int groups = inter >> 3;
     const long long total = (long long)rows * groups;
     for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
@@ -181,7 +183,7 @@ __global__ void clamped_glu_kernel(const T* __restrict__ gate_up, T* __restrict_
         for (int j = 0; j < 8; ++j) {
             const float g = fminf(Cvt<T>::to_f(gv[j]), limit);
             const float u = fminf(fmaxf(Cvt<T>::to_f(uv[j]), -limit), limit);
-            y[j] = g / (1.f + expf(-alpha * g)) * (u + 1.f);
+            y[j] = g / (1.f + expf(-alpha * g)) * (u + up_offset);
         }
         alignas(16) T ov[8];
 #pragma unroll
@@ -359,21 +361,21 @@ extern "C" int telb_moe_route_chosen(const float* logits, int ld, float* topk_w,
 }
 
 // dtype: 0 fp16, 1 bf16, 2 fp32.  tile_rows (rows in use of every 128-row tile) may be null.
-extern "C" int telb_clamped_glu(const void* gate_up, void* out, const int* tile_rows, int rows, int inter, float limit, float alpha, int dtype,
-                                cudaStream_t stream) {
+extern "C" int telb_clamped_glu(const void* gate_up, void* out, const int* tile_rows, int rows, int inter, float limit, float alpha, float up_offset,
+                                int dtype, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (inter % 8) return fail("telb_clamped_glu: the width must be a multiple of 8");
     const long long total = (long long)rows * (inter / 8);
     const long long blocks = (total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16;
     if (dtype == 2)
         TELB_LAUNCH("clamped_glu_kernel", (clamped_glu_kernel<float>), dim3((unsigned)blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out,
-                    tile_rows, rows, inter, limit, alpha);
+                    tile_rows, rows, inter, limit, alpha, up_offset);
     else if (dtype == 1)
         TELB_LAUNCH("clamped_glu_kernel", (clamped_glu_kernel<__nv_bfloat16>), dim3((unsigned)blocks), dim3(256), 0, stream,
-                    (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, tile_rows, rows, inter, limit, alpha);
+                    (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, tile_rows, rows, inter, limit, alpha, up_offset);
     else
         TELB_LAUNCH("clamped_glu_kernel", (clamped_glu_kernel<__half>), dim3((unsigned)blocks), dim3(256), 0, stream, (const __half*)gate_up, (__half*)out,
-                    tile_rows, rows, inter, limit, alpha);
+                    tile_rows, rows, inter, limit, alpha, up_offset);
     TELB_CHECK_LAUNCH("clamped_glu_kernel");
     return 0;
 }

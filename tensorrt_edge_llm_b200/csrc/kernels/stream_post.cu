@@ -15,7 +15,7 @@
 // blocks of rows count from the start of a sequence's portion, only the first one needs the history row of the seat, and the CTA that owns
 // it also writes the new history, so no CTA reads what another one of its launch writes.  The last token of a sequence is kept likewise.
 #include "host_utils.h"
-#include "tc5_common.cuh"
+#include "stream_common.cuh"
 
 namespace telb {
 
@@ -46,35 +46,6 @@ struct StreamPostParams {
 
 constexpr int kPostMaxGroups = 256;
 constexpr int kPostMaxTaps = 8;
-
-template <typename T>
-__device__ __forceinline__ void get4(const T* p, float (&v)[4]) {
-    if constexpr (sizeof(T) == 4) {
-        const float4 f = *reinterpret_cast<const float4*>(p);
-        v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
-    } else {
-        const uint2 u = *reinterpret_cast<const uint2*>(p);
-        const T* e = reinterpret_cast<const T*>(&u);
-#pragma unroll
-        for (int i = 0; i < 4; ++i) v[i] = Cvt<T>::to_f(e[i]);
-    }
-}
-template <typename T>
-__device__ __forceinline__ void put4(T* p, const float (&v)[4]) {
-    if constexpr (sizeof(T) == 4) {
-        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-    } else {
-        uint2 u;
-        u.x = Cvt<T>::pack2(v[0], v[1]);
-        u.y = Cvt<T>::pack2(v[2], v[3]);
-        *reinterpret_cast<uint2*>(p) = u;
-    }
-}
-__device__ __forceinline__ float post_warp_sum(float v) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
 
 // One over the root mean square of the row that was projected to row `row` of delta (every warp computes it).
 __device__ __forceinline__ float row_scale(const StreamPostParams& p, size_t row) {

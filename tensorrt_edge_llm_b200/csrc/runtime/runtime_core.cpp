@@ -200,6 +200,8 @@ LLMEngineConfig LLMEngineConfig::from_runtime_config(const Json& root) {
         const auto& list = specs.items();
         const int n = static_cast<int>(list.size());
         int input_taps = 0, bigram_buckets = 0;
+        bool token_shift = false;
+        b(m, "token_shift", token_shift);
         i(m, "input_conv", input_taps);
         i(m, "bigram_buckets", bigram_buckets);
         auto pad_head = [](int d) { return d <= 64 ? 64 : d <= 128 ? 128 : d <= 256 ? 256 : (d + 63) / 64 * 64; };
@@ -248,6 +250,7 @@ LLMEngineConfig LLMEngineConfig::from_runtime_config(const Json& root) {
                 state += 1LL * heads * pad_head(k) * ((v + 127) / 128 * 128);
             }
             if (input_taps > 1) state += 1LL * c.hidden_size * (input_taps - 1);   // fp32 rows in front of the mixer's input convolution
+            if (token_shift) state += c.hidden_size;                               // last normed row in front of the mixer
             if (c.run_state_values.empty() && bigram_buckets > 0) state += 1;      // the sequence's last token
             c.run_kv_elements.push_back(kv);
             c.run_state_values.push_back(state);
@@ -291,6 +294,8 @@ LLMEngineConfig LLMEngineConfig::from_runtime_config(const Json& root) {
 }
 
 bool LLMEngineConfig::is_hybrid() const {
+    for (const long long v : run_state_values)
+        if (v > 0) return true;                    // attention layers may keep state rows too
     for (const auto& t : layer_types)
         if (t != "attention") return true;
     return false;

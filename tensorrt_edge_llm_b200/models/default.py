@@ -252,9 +252,82 @@ class LatentAttention(nn.Module):
         return self.o_proj(ops.latent_attention(q, kv_layer, meta, self.kv_up_proj.weight, self._key_up_t, self.spec))
 
 
+class MixedAttention(nn.Module):
+    """Windowed attention whose heads read learned combinations of all heads' scores (``AttentionConfig.mixed_scores``), with a distance bias,
+    values that join with those of the first such layer, and a gate on the heads.
+
+    Scores are linear in the queries, so the combination is taken on their side, in fp32: head ``h`` attends with one query over the keys
+    of all KV heads side by side, ``[T[h, g] q_g summed over the heads g of KV head c]_c``, and loses ``(T slope)_h * distance``.  One
+    product gives q, k, v and the gate; ``ops.mixed_kv_write`` makes the wide queries, mixes the values and writes the cache;
+    ``ops.mixed_attention`` attends and applies the gate before its one rounding."""
+
+    def __init__(self, cfg: ModelConfig, spec, prefix: str):
+        super().__init__()
+        self.spec, self.prefix = spec, prefix
+        h, d, n = cfg.hidden_size, spec.pad, spec.num_heads
+        out = (n, spec.v_head_dim, d)
+        heads = [(n, spec.head_dim, d), (spec.num_kv_heads, spec.head_dim, d), (spec.num_kv_heads, spec.v_head_dim, d), out]
+        self.qkvg_proj = HeadLinear(h, 0, out_heads=heads, sources=["q_proj", "k_proj", "v_proj", "g_proj"], dtype=cfg.compute_dtype, bias=spec.qkv_bias)
+        self.o_proj = HeadLinear(0, h, in_heads=out, dtype=cfg.compute_dtype)
+        self.v_col, self.g_col = (n + spec.num_kv_heads) * d, (n + 2 * spec.num_kv_heads) * d
+        f32 = dict(dtype=torch.float32)
+        self.mix = nn.Parameter(torch.eye(n, **f32), requires_grad=False)
+        self.share = nn.Parameter(torch.zeros((), **f32), requires_grad=False)     # of the first layer's values
+        self._slopes: Optional[torch.Tensor] = None
+
+    @torch.no_grad()
+    def random_init(self, gen, std=0.02):
+        n = self.spec.num_heads
+        self.mix.copy_(torch.eye(n) + torch.randn(n, n, generator=gen) * 0.2)
+        self.share.fill_(0.4)
+
+    def finalize(self):
+        """Slopes of the mixed scores, rounded once from double."""
+        n = self.spec.num_heads
+        slope = torch.tensor([2.0 ** (-8.0 * (h + 1) / n) if self.spec.distance_bias else 0.0 for h in range(n)], dtype=torch.float64)
+        self._slopes = (self.mix.detach().double().cpu() @ slope).float().to(self.mix.device)
+
+    def forward(self, x: torch.Tensor, meta: StepMeta, kv_layer: torch.Tensor, first: Optional[torch.Tensor]):
+        """``(output, values for the layers behind)``; ``first``: the value columns of the first layer that mixes, None until it has run."""
+        if meta.tree_mask is not None:
+            raise NotImplementedError("attention with mixed scores covers causal windows only (no draft trees)")
+        if self._slopes is None or self._slopes.device != x.device:
+            self.finalize()
+        sp = self.spec
+        rows = self.qkvg_proj(x)
+        join = first if sp.value_mix else None
+        q = ops.mixed_kv_write(rows, kv_layer, meta, self.mix, join, self.share, sp)
+        o = ops.mixed_attention(q, kv_layer, meta, self._slopes, rows[:, self.g_col:] if sp.out_gate else None, sp)
+        if sp.value_mix and first is None:
+            first = rows[:, self.v_col:self.g_col]
+        return self.o_proj(o), first
+
+
+class XieluMLP(nn.Module):
+    """``down(xielu(up x))`` without a gate; the activation's two numbers are learned."""
+
+    def __init__(self, cfg: ModelConfig, size: int):
+        super().__init__()
+        pad = (1, size, (size + 63) // 64 * 64)
+        self.up_proj = HeadLinear(cfg.hidden_size, 0, out_heads=[pad], dtype=cfg.compute_dtype)
+        self.down_proj = HeadLinear(0, cfg.hidden_size, in_heads=pad, dtype=cfg.compute_dtype)
+        self.act = nn.Parameter(torch.zeros(2, dtype=torch.float32), requires_grad=False)
+        self._coef: Optional[torch.Tensor] = None
+
+    def finalize(self):
+        """Factors of the two branches, rounded once from double: softplus(p), 1/2 + softplus(q)."""
+        p = torch.nn.functional.softplus(self.act.detach().double().cpu(), threshold=700.0)
+        self._coef = (p + torch.tensor([0.0, 0.5], dtype=torch.float64)).float().to(self.act.device)
+
+    def forward(self, x):
+        if self._coef is None or self._coef.device != x.device:
+            self.finalize()
+        return self.down_proj(ops.xielu(self.up_proj(x), self._coef))
+
+
 class GatedMLP(nn.Module):
-    """``down(act(gate x) * up x)`` with a size of its own (tanh-form gelu or relu, with or without biases); the inner size is padded to
-    what the kernels take."""
+    """``down(act(gate x) * up x)`` with a size of its own (tanh-form gelu, relu or silu, with or without biases); the inner size is padded
+    to what the kernels take."""
 
     def __init__(self, cfg: ModelConfig, size: int, act: str = "gelu_tanh", bias: bool = False):
         super().__init__()

@@ -24,7 +24,7 @@ from ..ops.meta import StepMeta
 from .default import LayerAttention
 from .linear import Fp32OutLinear
 from .nemotron_h import HybridCausalLM, MLstmMixer
-from .qwen3_moe import ClampedExperts
+from .qwen3_moe import GatedExperts
 
 
 class OffsetRMSNorm(nn.Module):
@@ -53,7 +53,7 @@ class ParallelLayer(nn.Module):
         self.router_col = sum(sizes)
         self.mlp = None
         if spec.moe is not None:
-            self.mlp = ClampedExperts(cfg, spec.moe, f"{p}.mlp")
+            self.mlp = GatedExperts(cfg, spec.moe, f"{p}.mlp")
             sizes.append(spec.moe.num_experts)
             sources.append("mlp.router")
         # gate pre-activations and router logits: one product with fp32 results

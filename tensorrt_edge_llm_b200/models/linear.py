@@ -130,7 +130,7 @@ class HeadLinear(Linear):
 
     ``out_heads``: one ``(heads, real size, padded size)`` per source module (its checkpoint rows are ``heads x real``);
     ``in_heads``: the same for the input features.  Padding rows and columns are zero, so padded features are zeros on the
-    way out and ignored on the way in."""
+    way out and ignored on the way in.  ``bias``: sources without one have zeros."""
 
     def __init__(self, in_features: int, out_features: int, out_heads=None, in_heads=None, sources=None, dtype=torch.bfloat16, bias: bool = False):
         self.out_heads, self.in_heads = out_heads, in_heads
@@ -153,7 +153,8 @@ class HeadLinear(Linear):
     def load_from(self, tensors):
         self.weight.data.copy_(torch.cat([self._pad_out(self._pad_in(t["weight"]), i) for i, t in enumerate(tensors)], 0).to(self.weight.dtype))
         if self.bias is not None:
-            self.bias.data.copy_(torch.cat([self._pad_out(t["bias"].reshape(-1, 1), i) for i, t in enumerate(tensors)])[:, 0].to(self.bias.dtype))
+            self.bias.data.copy_(torch.cat([self._pad_out(t["bias"].reshape(-1, 1) if "bias" in t else torch.zeros(t["weight"].shape[0], 1), i)
+                                            for i, t in enumerate(tensors)])[:, 0].to(self.bias.dtype))
 
     @torch.no_grad()
     def zero_padding(self) -> None:

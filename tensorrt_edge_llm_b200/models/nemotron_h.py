@@ -37,7 +37,7 @@ class RecurrentState:
         self.mlstm, self.mlstm_norm = {}, {}      # matrix memory; normaliser and running maximum
         self.delta = {}                           # delta rule with a decay per key channel or head
         self.lightning = {}                       # linear attention with constant decays
-        self.inputs = {}                          # last rows of the stream in front of each mixer's input convolution, fp32
+        self.inputs = {}                          # last rows in front of each mixer (of the stream: input convolution; normed: token shift), fp32
         self.tokens = {}                          # the sequence's last token (bigram embeddings)
         runs = cfg.layer_run_ids if cfg.layer_specs else None
         for i, t in enumerate(cfg.layer_types):
@@ -62,8 +62,9 @@ class RecurrentState:
             elif t == LAYER_LIGHTNING:
                 l = cfg.layer_specs[runs[i]].lightning
                 self.lightning[i] = torch.zeros(seats, l.num_heads, l.k_pad, l.v_pad, dtype=torch.float32, device=device)
-            if cfg.input_conv > 1:
-                self.inputs[i] = torch.zeros(seats, cfg.input_conv - 1, cfg.hidden_size, dtype=torch.float32, device=device)
+            if cfg.input_conv > 1 or cfg.token_shift:
+                rows = 1 if cfg.token_shift else cfg.input_conv - 1
+                self.inputs[i] = torch.zeros(seats, rows, cfg.hidden_size, dtype=torch.float32, device=device)
         if cfg.bigram_buckets:
             self.tokens[0] = torch.zeros(seats, 1, dtype=torch.int32, device=device)
 

@@ -26,8 +26,8 @@ from .. import ops
 from ..config import QUANT_NVFP4, ModelConfig
 from ..model import register_model
 from ..ops import reference as ref
-from .default import Attention, CausalLM, RMSNorm, Transformer
-from .linear import Linear, TPMode
+from .default import Attention, CausalLM, GatedMLP, RMSNorm, Transformer
+from .linear import Fp32OutLinear, Linear, TPMode
 
 
 class MoEBlock(nn.Module):
@@ -283,9 +283,9 @@ class RoutedRows:
         self.y, self.ws, self.weights = y, ws, weights
 
 
-class ClampedExperts(nn.Module):
-    """Experts with a clamped gated unit (``MoeConfig``) and a router whose weights are the softmax over the chosen logits.  The fp32
-    logits come from the layer (its fp32 projection), the weighted sum is left to the consumer."""
+class GatedExperts(nn.Module):
+    """Experts with a (clamped) gated unit and one of two routers (``MoeConfig``).  The fp32 logits come from the layer (its fp32
+    projection), the weighted sum is left to the consumer."""
 
     def __init__(self, cfg: ModelConfig, spec, prefix: str):
         super().__init__()
@@ -295,6 +295,15 @@ class ClampedExperts(nn.Module):
         # rows of an expert: gate, then up; the intermediate size is padded with zero rows / columns (a zero gate gives a zero unit)
         self.w13 = nn.Parameter(torch.zeros(e * 2 * i, cfg.hidden_size, dtype=dt), requires_grad=False)
         self.w2 = nn.Parameter(torch.zeros(e * cfg.hidden_size, i, dtype=dt), requires_grad=False)
+        if spec.router == "sigmoid_groups":               # joins the scores in the choice, not in the weights
+            self.correction = nn.Parameter(torch.zeros(e, dtype=torch.float32), requires_grad=False)
+
+    def route(self, logits: torch.Tensor):
+        """``(weights, indices)`` of the chosen experts per row."""
+        sp = self.spec
+        if sp.router == "sigmoid_groups":
+            return ops.moe_route_sigmoid_groups(logits, self.correction, sp.top_k, sp.groups, sp.keep_groups, sp.weight_scale)
+        return ops.moe_route_chosen(logits, sp.top_k)
 
     @torch.no_grad()
     def load_checkpoint(self, fetch) -> bool:
@@ -326,15 +335,30 @@ class ClampedExperts(nn.Module):
     def forward(self, x: torch.Tensor, logits: torch.Tensor):
         """``x`` ``[T, hidden]`` and fp32 router logits ``[T, experts]`` (may be a column slice) → :class:`RoutedRows`."""
         sp = self.spec
-        w, idx = ops.moe_route_chosen(logits, sp.top_k)
+        w, idx = self.route(logits)
         if not x.is_cuda:
             return ops.ref.clamped_experts(x, self.w13.view(sp.num_experts, -1, self.hidden), self.w2.view(sp.num_experts, self.hidden, -1), w, idx,
-                                           sp.limit, sp.alpha)
+                                           sp.limit, sp.alpha, sp.up_offset)
         cu = ops.cuda_ops()
         ws = cu.moe_align(idx, sp.num_experts, 0, sp.num_experts)
         h1 = cu.gemm_grouped(cu.moe_gather(x, ws, sp.top_k, None), self.w13, ws, sp.num_experts)
-        y = cu.gemm_grouped(cu.clamped_glu(h1, sp.limit, sp.alpha, ws), self.w2, ws, sp.num_experts)
+        y = cu.gemm_grouped(cu.clamped_glu(h1, sp.limit, sp.alpha, ws, sp.up_offset), self.w2, ws, sp.num_experts)
         return RoutedRows(y, ws, w)
+
+
+class SharedExpertsBlock(nn.Module):
+    """Routed experts behind a router of their own, beside a gated unit that every token passes through (``MoeConfig.shared_size``, or
+    none).  Returns ``(shared output or None, RoutedRows)``; the kernel that advances the residual stream takes the sum."""
+
+    def __init__(self, cfg: ModelConfig, spec, prefix: str):
+        super().__init__()
+        self.router = Fp32OutLinear(cfg.hidden_size, [spec.num_experts], dtype=cfg.compute_dtype)
+        self.routed = GatedExperts(cfg, spec, prefix)
+        self.shared = GatedMLP(cfg, spec.shared_size, act="silu") if spec.shared_size else None
+
+    def forward(self, x: torch.Tensor):
+        routed = self.routed(x, self.router(x))
+        return (None if self.shared is None else self.shared(x)), routed
 
 
 class MoEDecoderLayer(nn.Module):

@@ -82,15 +82,26 @@ def geglu(gate_up, tanh_approx=True):
 
 
 def glu(gate_up, act="gelu_tanh"):
-    """``act(gate) * up`` over the fused ``[T, 2·I]`` projection output; ``act``: ``"gelu_tanh"`` or ``"relu"``."""
+    """``act(gate) * up`` over the fused ``[T, 2·I]`` projection output; ``act``: ``"gelu_tanh"``, ``"relu"`` or ``"silu"``."""
     if act == "gelu_tanh":
         return geglu(gate_up, True)
+    if act == "silu":
+        if gate_up.is_cuda and gate_up.dtype == torch.float32:
+            return cuda_ops().clamped_glu(gate_up, 0.0, 1.0, up_offset=0.0)
+        return swiglu(gate_up)
     if act != "relu":
         raise ValueError(f"unknown gate activation {act!r}")
     if gate_up.is_cuda:
         return cuda_ops().reglu(gate_up)
     inter = gate_up.shape[-1] // 2
     return (torch.relu(gate_up[..., :inter].float()) * gate_up[..., inter:].float()).to(gate_up.dtype)
+
+
+def xielu(x, coef):
+    """``coef[0] x² + x / 2`` above zero, ``coef[1] (exp(x) - 1 - x) + x / 2`` below; ``coef`` fp32 ``[2]``."""
+    if x.is_cuda:
+        return cuda_ops().xielu(x, coef)
+    return ref.xielu(x, coef)
 
 
 def softcap_(logits, cap):
@@ -227,6 +238,19 @@ def stream_post(stream, delta, weight, groups, eps, meta, dtype, *, ids=None, ta
     return f(stream, delta, weight, groups, eps, meta, dtype, ids, table, bigram, conv, history, out_norm, sums)
 
 
+def stream_sandwich(stream, eps, meta, dtype, *, ids=None, table=None, positions=None, delta=None, routed=None, post=None, mult=1.0, norm=None,
+                    shift=None, state=None):
+    """The fp32 residual stream of blocks with a norm in front of and behind every sublayer: ``(stream, h)``.
+
+    ``stream`` (or ``table[ids]`` when it is ``None``), plus the row of ``positions`` of every token's position when given, ``+ mult * rms_norm(delta
+    + routed) * post``; ``h`` in ``dtype`` is its RMS norm times ``norm``.  ``shift`` ``[width]``: features of ``h`` move by these shares towards
+    the row before it in its sequence; ``state`` ``[seats, 1, width]`` (fp32) holds the last normed row of every sequence and is
+    advanced.  ``routed``: a dense tensor, or :class:`models.qwen3_moe.RoutedRows`, whose weighted sum the kernel takes itself."""
+    t = ids if stream is None else stream
+    f = cuda_ops().stream_sandwich if t.is_cuda else ref.stream_sandwich
+    return f(stream, eps, meta, dtype, ids, table, positions, delta, routed, post, mult, norm, shift, state)
+
+
 def lightning(rows, norm_w, powers, state, meta):
     """Linear attention with a constant decay per head over packed ``[q | k | v | g]`` rows: silu on q, k and v, the recurrence, weight and
     sigmoid gate.  Returns ``(u [T, heads · dv], sums [T, heads · dv / 32])``: the gated read-outs before the RMS norm over all heads of a
@@ -242,6 +266,14 @@ def moe_route_chosen(logits, top_k):
     if logits.is_cuda:
         return cuda_ops().moe_route_chosen(logits, top_k)
     return ref.moe_route_chosen(logits, top_k)
+
+
+def moe_route_sigmoid_groups(logits, correction, top_k, groups, keep, scale):
+    """Scores ``sigmoid(logits)``; the ``top_k`` largest ``score + correction`` inside the ``keep`` best of ``groups`` equal groups of neighbours (a
+    group's worth: the sum of its two largest).  Returns ``(scale * scores, indices)`` of the chosen."""
+    if logits.is_cuda:
+        return cuda_ops().moe_route_softmax_topk(logits, top_k, False, correction, True, groups, keep, scale)
+    return ref.moe_route_sigmoid_group_topk(logits, correction, top_k, groups, keep, False, scale)
 
 
 def mlstm(qkvg, gates, norm_w, state, norm_state, meta, scale, cap, eps, dv_real):
@@ -281,6 +313,21 @@ def turned_kv_write(rows, kv_layer, meta, key_table, value_table, q_norm, k_norm
     ``spec``: :class:`config.AttentionConfig`."""
     f = cuda_ops().turned_kv_write if rows.is_cuda else ref.turned_kv_write
     return f(rows, kv_layer, meta, key_table, value_table, q_norm, k_norm, spec, eps)
+
+
+def mixed_kv_write(rows, kv_layer, meta, mix, first, share, spec):
+    """Packed q | k | v rows (and what lies behind them) of padded heads: keys go to the paged cache, values too, ``(1 - share) v + share *
+    first`` when ``first`` ``[T, kv heads * pad]`` is given.  Returns the wide queries: head ``h`` holds, for every KV head ``c``, the sum of
+    ``mix[h, g] q_g`` over the query heads ``g`` of ``c``.  ``spec``: :class:`config.AttentionConfig`."""
+    f = cuda_ops().mixed_kv_write if rows.is_cuda else ref.mixed_kv_write
+    return f(rows, kv_layer, meta, mix, first, share, spec)
+
+
+def mixed_attention(q, kv_layer, meta, slopes, gate, spec):
+    """Windowed attention of wide queries (see :func:`mixed_kv_write`) over the keys of all KV heads at once; head ``h`` loses ``slopes[h]`` times
+    the distance and reads the values of its own KV head; heads times ``sigmoid(gate)`` (``[T, heads * pad]``, or None).  ``[T, heads * pad]``."""
+    f = cuda_ops().mixed_attention if kv_layer.is_cuda else ref.mixed_attention
+    return f(q, kv_layer, meta, slopes, gate, spec)
 
 
 def latent_write(rows, kv_layer, meta, cos_sin, norm_w, spec, eps):

@@ -199,6 +199,14 @@ def reglu(gate_up: torch.Tensor) -> torch.Tensor:
     return out
 
 
+def xielu(x: torch.Tensor, coef: torch.Tensor) -> torch.Tensor:
+    x = x.contiguous()
+    assert coef.dtype == torch.float32 and coef.numel() == 2
+    out = torch.empty_like(x)
+    _check(lib().telb_xielu(_p(x), _p(out), c_ll(x.numel()), _p(coef), c_int(_dtype_code(x)), _stream()), "xielu")
+    return out
+
+
 def softcap_(logits: torch.Tensor, cap: float) -> torch.Tensor:
     if logits.dtype != torch.float32 or not logits.is_contiguous():
         raise TypeError("softcap_: contiguous fp32 logits")
@@ -384,6 +392,56 @@ def stream_post(stream, delta, weight, groups: int, eps: float, meta: StepMeta, 
     code = 2 if dtype == f32 else 1
     one_row = meta.max_q_len == 1
     _check(lib().telb_stream_post(ctypes.byref(p), c_int(int(one_row)), c_int(code), _stream()), "stream_post", 1 if one_row or not taps else 2)
+    return x, h
+
+
+class StreamSandwichParams(ctypes.Structure):
+    """Host mirror of ``StreamSandwichParams`` (``csrc/kernels/stream_sandwich.cu``)."""
+    _fields_ = [(n, c_vp) for n in ("ids", "table", "pos_table", "x_in", "y", "e", "dst_row", "topk_w", "post", "norm", "shift", "state", "x_out", "h", "positions",
+                                    "q_start", "q_len", "past_len", "slot_ids", "seq_ids")] + \
+               [(n, c_int) for n in ("vocab", "max_pos", "width", "tokens", "block_rows", "top_k", "lde")] + [("mult", c_float), ("eps", c_float)]
+
+
+def _sandwich_block_rows(tokens: int, shifted: bool) -> int:
+    """Rows per CTA.  Shifted blocks compute the row in front of them once more, so long steps take longer blocks."""
+    if not shifted:
+        return 1 if tokens <= 148 * 8 else 2
+    return 1 if tokens <= 148 * 2 else 4 if tokens <= 148 * 16 else 8
+
+
+def stream_sandwich(stream, eps: float, meta: StepMeta, dtype, ids, table, positions, delta, routed, post, mult: float, norm, shift, state):
+    """See :func:`ops.stream_sandwich`; ``routed`` carries expert rows (``y``, routing tables ``ws``, weights)."""
+    f32 = torch.float32
+    if stream is None:
+        t, width, dev = ids.numel(), table.shape[1], table.device
+        ids = ids.to(torch.int32).contiguous()
+    else:
+        (t, width), dev = stream.shape, stream.device
+        assert stream.dtype == f32 and stream.is_contiguous()
+        ids = table = None
+    y = ws = w = None
+    if routed is not None:
+        y, ws, w = routed.y, routed.ws, routed.weights
+        assert y.is_contiguous() and y.shape[1] == width and w.shape[0] == t and w.dtype == f32
+    if delta is not None:
+        delta = delta.contiguous()
+        assert delta.shape == (t, width)
+    for v in (table, positions, delta, y):
+        if v is not None and v.dtype != dtype:
+            raise TypeError(f"stream_sandwich: rows of {v.dtype}, activations {dtype}")
+    for v in (post, norm, shift):
+        assert v is None or (v.dtype == f32 and v.numel() == width and v.is_contiguous())
+    assert shift is None or (state.dtype == f32 and state.is_contiguous() and state.shape[1:] == (1, width))
+    assert positions is None or (positions.is_contiguous() and positions.shape[1] == width)
+    x = torch.empty(t, width, dtype=f32, device=dev)
+    h = None if norm is None else torch.empty(t, width, dtype=dtype, device=dev)
+    rows = 1 if shift is not None and meta.max_q_len == 1 else _sandwich_block_rows(t, shift is not None)
+    p = StreamSandwichParams(*[None if v is None else _p(v).value for v in (
+        ids, table, positions, stream, delta, y, None if ws is None else ws.dst_row, w, post, norm, shift, state, x, h, meta.positions, meta.q_start, meta.q_len,
+        meta.past_len, meta.slot_ids, meta.seq_ids)], 0 if table is None else table.shape[0], 0 if positions is None else positions.shape[0], width, t, rows,
+        0 if w is None else w.shape[1], 0 if y is None else y.shape[1], mult, eps)
+    code = 2 if dtype == f32 else int(dtype == torch.bfloat16)
+    _check(lib().telb_stream_sandwich(ctypes.byref(p), c_int(code), _stream()), "stream_sandwich")
     return x, h
 
 
@@ -930,12 +988,13 @@ def moe_route_chosen(logits: torch.Tensor, top_k: int):
     return w, idx
 
 
-def clamped_glu(gate_up: torch.Tensor, limit: float, alpha: float, ws: Optional["MoeWorkspace"] = None) -> torch.Tensor:
-    """Clamped gated unit over ``[gate | up]`` rows; with ``ws`` the rows of the padded expert layout that hold no token are skipped."""
+def clamped_glu(gate_up: torch.Tensor, limit: float, alpha: float, ws: Optional["MoeWorkspace"] = None, up_offset: float = 1.0) -> torch.Tensor:
+    """``g σ(alpha g) (u + up_offset)`` over ``[gate | up]`` rows, both clamped unless ``limit`` is 0; with ``ws`` the rows of the padded expert
+    layout that hold no token are skipped."""
     rows, two = gate_up.shape
     out = torch.empty(rows, two // 2, dtype=gate_up.dtype, device=gate_up.device)
     tile_rows = c_vp(ws.tile_expert.data_ptr() + 4 * ws.max_tiles) if ws is not None else c_vp(0)
-    _check(lib().telb_clamped_glu(_p(gate_up), _p(out), tile_rows, c_int(rows), c_int(two // 2), c_float(limit), c_float(alpha),
+    _check(lib().telb_clamped_glu(_p(gate_up), _p(out), tile_rows, c_int(rows), c_int(two // 2), c_float(limit), c_float(alpha), c_float(up_offset),
                                   c_int(_dtype_code(gate_up)), _stream()), "clamped_glu")
     return out
 
@@ -1303,6 +1362,121 @@ def turned_kv_write(rows, kv_layer, meta: StepMeta, key_table, value_table, q_no
                        rows.stride(0), t, meta.page_table.shape[1], meta.page_size, hq, hkv, d, spec.head_dim, eps)
     _check(lib().telb_turned_kv_write(ctypes.byref(p), c_int(_dtype_code(rows)), _stream()), "turned_kv_write")
     return q
+
+
+MIXED_DECODE_COLUMNS = 64       # sequences with at most this many (row, head) pairs in a step run the token-major kernel
+
+
+class RowSplit:
+    """A step's sequences by how many rows they bring: ``short`` (up to ``limit``) and ``long``, each ``(q_start, q_len, past_len, page_table,
+    sequences, most rows, longest sequence)`` over the rows of the whole step, or None.  Built once per step."""
+
+    def __init__(self, meta: StepMeta, limit: int, device):
+        self.key = ("rows", limit)
+        everything = (meta.q_start, meta.q_len, meta.past_len, meta.page_table, meta.num_seqs, meta.max_q_len, meta.max_seq_len)
+        self.short = self.long = None
+        if meta.max_q_len <= limit:
+            self.short = everything
+            return
+        lens, start = meta.lengths(), [0]
+        for q, _ in lens:
+            start.append(start[-1] + q)
+        parts = [[i for i, (q, _) in enumerate(lens) if 0 < q <= limit], [i for i, (q, _) in enumerate(lens) if q > limit]]
+        if len(parts[1]) == len(lens):
+            self.long = everything
+            return
+        out = []
+        for part in parts:
+            if not part:
+                out.append(None)
+                continue
+            arr = torch.tensor([[start[i] for i in part], [lens[i][0] for i in part], [lens[i][1] for i in part]], dtype=torch.int32, device=device)
+            table = meta.page_table.index_select(0, torch.tensor(part, dtype=torch.int64, device=device))
+            out.append((arr[0], arr[1], arr[2], table, len(part), max(lens[i][0] for i in part), max(sum(lens[i]) for i in part)))
+        self.short, self.long = out
+
+
+def _row_split(meta: StepMeta, limit: int, device) -> RowSplit:
+    for p in meta.plans or ():
+        if p.key == ("rows", limit):
+            return p
+    p = RowSplit(meta, limit, device)
+    meta.plans = (meta.plans or ()) + (p,)
+    return p
+
+
+class MixedKvParams(ctypes.Structure):
+    """Host mirror of ``MixedKvParams`` (``csrc/kernels/mixed_heads.cu``)."""
+    _fields_ = [(n, c_vp) for n in ("rows", "first", "q_out", "kv", "mix", "share", "seq_ids", "q_start", "past_len", "page_table")] + \
+               [(n, c_ll) for n in ("ld", "ld_first")] + [(n, c_int) for n in ("tokens", "max_pages", "page_size", "hq", "hkv", "d", "halves")]
+
+
+def _mixed_tc(spec, dtype, page_size: int) -> bool:
+    """Whether the tensor-core kernels take this layer."""
+    return dtype == torch.bfloat16 and page_size == 64 and spec.pad in (64, 128) and spec.num_kv_heads * spec.pad <= 512
+
+
+def _mixed_plan(meta: StepMeta, heads: int, device) -> RowSplit:
+    return _row_split(meta, max(1, MIXED_DECODE_COLUMNS // heads), device)
+
+
+def mixed_kv_write(rows, kv_layer, meta: StepMeta, mix, first, share, spec):
+    """See :func:`ops.mixed_kv_write`; 16-bit wide queries come as high | low halves where the kernels behind can use both."""
+    t, n, g, d = rows.shape[0], spec.num_heads, spec.num_kv_heads, spec.pad
+    rows = _pitched(rows)
+    assert rows.shape[1] >= (n + 2 * g) * d and kv_layer.is_contiguous() and kv_layer.dtype == rows.dtype and kv_layer.shape[1:] == (2, g, meta.page_size, d)
+    assert mix.dtype == torch.float32 and mix.is_contiguous() and mix.shape == (n, n) and share.dtype == torch.float32
+    if first is not None:
+        first = _pitched(first)
+        assert first.dtype == rows.dtype and first.shape == (t, g * d)
+    halves = 1
+    if _mixed_tc(spec, rows.dtype, meta.page_size) and (g * d <= 256 or _mixed_plan(meta, n, rows.device).long is None):
+        halves = 2
+    q = torch.empty(t, n, halves * g * d, dtype=rows.dtype, device=rows.device)
+    p = MixedKvParams(*[None if x is None else _p(x).value for x in (rows, first, q, kv_layer, mix, share, meta.seq_ids, meta.q_start, meta.past_len, meta.page_table)],
+                      rows.stride(0), 0 if first is None else first.stride(0), t, meta.page_table.shape[1], meta.page_size, n, g, d, halves)
+    _check(lib().telb_mixed_kv_write(ctypes.byref(p), c_int(_dtype_code(rows)), _stream()), "mixed_kv_write")
+    return q
+
+
+def mixed_attention(q, kv_layer, meta: StepMeta, slopes, gate, spec, kernel: Optional[str] = None, splits: Optional[int] = None, tile: Optional[int] = None):
+    """See :func:`ops.mixed_attention`.  Sequences with few rows run the token-major kernel, prompt portions the row-major one (``kernel``
+    forces ``"decode"``, ``"prefill"`` or ``"simt"`` for all); fp32 rows and sizes without a tensor-core form run on the CUDA cores."""
+    if meta.tree_mask is not None:
+        raise ValueError("mixed attention covers causal windows only")
+    (t, n, width), g, d, dev = q.shape, spec.num_kv_heads, spec.pad, q.device
+    halves = width // (g * d)
+    out = torch.empty(t, n * d, dtype=q.dtype, device=dev)
+    ld_gate = 0
+    if gate is not None:
+        assert gate.shape == (t, n * d) and gate.dtype == q.dtype and gate.stride(1) == 1
+        ld_gate = gate.stride(0)
+    assert slopes.dtype == torch.float32 and slopes.numel() == n and spec.window >= 1
+    if kernel == "simt" or not _mixed_tc(spec, q.dtype, meta.page_size):
+        q = q[:, :, :g * d].contiguous()
+        _check(lib().telb_mixed_attention_simt(
+            _p(q), _p(kv_layer), _p(out), _p(meta.q_start), _p(meta.past_len), _p(meta.seq_ids), _p(meta.page_table), c_int(t), c_int(meta.page_table.shape[1]),
+            c_int(meta.page_size), c_int(n), c_int(g), c_int(d), c_float(spec.scale), c_int(spec.window), _p(slopes), _p(gate), c_ll(ld_gate),
+            c_int(_dtype_code(q)), _stream()), "mixed_attention_simt")
+        return out
+    everything = (meta.q_start, meta.q_len, meta.past_len, meta.page_table, meta.num_seqs, meta.max_q_len, meta.max_seq_len)
+    if kernel is None:
+        plan = _mixed_plan(meta, n, dev)
+        short, long = plan.short, plan.long
+    else:
+        short, long = (everything, None) if kernel == "decode" else (None, everything)
+    ws = Workspace.get(dev)
+    common = lambda s: (_p(q), _p(kv_layer), _p(out), _p(s[0]), _p(s[1]), _p(s[2]), _p(s[3]), c_int(s[4]), c_int(t), c_int(s[5]), c_int(kv_layer.shape[0]),
+                        c_int(s[3].shape[1]), c_int(n), c_int(g), c_int(d), c_int(halves), c_float(spec.scale), c_int(spec.window), _p(slopes), _p(gate), c_ll(ld_gate))
+    if long is not None:
+        _check(lib().telb_mixed_attention_prefill(*common(long), _p(ws.status), _stream()), "mixed_attention_prefill")
+    if short is not None:
+        nc = 16 if short[5] * n <= 16 else 32
+        sp, tl = _latent_splits(short[4] * ((short[5] * n + nc - 1) // nc), min(short[6], spec.window + short[5] + 63), nc)
+        sp, tl = splits or sp, tile or tl
+        _check(lib().telb_mixed_attention_decode(*common(short), c_int(sp), c_int(tl), _p(ws.attn_ws), c_ll(ws.attn_ws.numel()), _p(ws.status), _stream()),
+               "mixed_attention_decode", 2 if sp > 1 else 1)
+    return out
 
 
 def latent_write(rows, kv_layer, meta: StepMeta, cos_sin, norm_w, spec, eps: float):

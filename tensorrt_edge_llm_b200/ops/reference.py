@@ -652,6 +652,34 @@ def stream_post(stream, delta, weight, groups, eps, meta: StepMeta, dtype, ids, 
     return x, h.to(dtype)
 
 
+def stream_sandwich(stream, eps, meta: StepMeta, dtype, ids, table, positions, delta, routed, post, mult, norm, shift, state):
+    """See :func:`ops.stream_sandwich`."""
+    unit = lambda v: v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)
+    x = table[ids.long()].float() if stream is None else stream
+    if positions is not None:
+        x = x + positions[meta.positions.long()].float()
+    if delta is not None or routed is not None:
+        x = x + mult * (unit(sum(d.float() for d in (delta, routed) if d is not None)) * post)
+    if norm is None:
+        return x, None
+    h = unit(x) * norm
+    if shift is not None:
+        before = torch.empty_like(h)
+        before[1:] = h[:-1]
+        for r0, n, past, slot in zip(*(v.tolist() for v in (meta.q_start[:meta.num_seqs], meta.q_len, meta.past_len, meta.slot_ids))):
+            if n:
+                before[r0] = state[slot, 0] if past > 0 else 0.0
+                state[slot, 0] = h[r0 + n - 1]
+        h = h + (before - h) * shift
+    return x, h.to(dtype)
+
+
+def xielu(x, coef):
+    z = x.float()
+    neg = z.clamp(max=0)
+    return (torch.where(z > 0, coef[0] * z * z, coef[1] * (torch.expm1(neg) - neg)) + z / 2).to(x.dtype)
+
+
 def lightning(rows, norm_w, powers, state, meta: StepMeta):
     """Row by row in fp32 (see :func:`ops.lightning`)."""
     t, (_, n, dk, dv) = rows.shape[0], state.shape
@@ -750,6 +778,37 @@ def turned_kv_write(rows, kv_layer, meta: StepMeta, key_table, value_table, q_no
     return q.to(rows.dtype)
 
 
+def mixed_kv_write(rows, kv_layer, meta: StepMeta, mix, first, share, spec):
+    t, d, n, g = rows.shape[0], spec.pad, spec.num_heads, spec.num_kv_heads
+    q, k, v = rows[:, :(n + 2 * g) * d].float().split([n * d, g * d, g * d], dim=-1)
+    if first is not None:
+        v = (1 - share) * v + share * first.float()
+    page, row = _cache_slots(meta, t, rows.device)
+    kv_layer[page, 0, :, row] = k.reshape(t, g, d).to(kv_layer.dtype)
+    kv_layer[page, 1, :, row] = v.reshape(t, g, d).to(kv_layer.dtype)
+    return torch.einsum("hcg,tcgd->thcd", mix.view(n, g, n // g), q.reshape(t, g, n // g, d)).reshape(t, n, g * d)
+
+
+def mixed_attention(q, kv_layer, meta: StepMeta, slopes, gate, spec):
+    """``q`` fp32 ``[T, heads, kv heads * pad]``."""
+    t, n, g, d = q.shape[0], spec.num_heads, spec.num_kv_heads, spec.pad
+    out = torch.zeros(t, n * d, dtype=kv_layer.dtype)
+    for s in range(meta.num_seqs):
+        r0, ql, past = int(meta.q_start[s]), int(meta.q_len[s]), int(meta.past_len[s])
+        if ql == 0:
+            continue
+        k, v = gather_kv(kv_layer, meta.page_table[s], past + ql, meta.page_size)                # [G, total, d]
+        sc = torch.einsum("qhx,kx->hqk", q[r0:r0 + ql].float(), k.float().transpose(0, 1).reshape(past + ql, g * d)) * spec.scale
+        gap = (past + torch.arange(ql))[:, None] - torch.arange(past + ql)[None, :]
+        sc = sc - slopes[:, None, None] * gap
+        pr = torch.softmax(sc.masked_fill((gap < 0) | (gap >= spec.window), float("-inf")), dim=-1)
+        o = torch.einsum("hqk,hkd->qhd", pr, v.float().repeat_interleave(n // g, dim=0)).reshape(ql, -1)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[r0:r0 + ql].float())
+        out[r0:r0 + ql] = o.to(out.dtype)
+    return out
+
+
 def latent_write(rows, kv_layer, meta: StepMeta, cos_sin, norm_w, spec, eps):
     t, n = rows.shape[0], spec.num_heads
     q, qr, c, kr = rows.float().split([n * spec.k_pad, n * spec.rot_pad, spec.rank_pad, spec.rot_pad], dim=-1)
@@ -783,19 +842,20 @@ def moe_route_chosen(logits: torch.Tensor, top_k: int):
     return torch.softmax(logits.float().gather(1, order), dim=-1), order.to(torch.int32)
 
 
-def clamped_glu(gate_up: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+def clamped_glu(gate_up: torch.Tensor, limit: float, alpha: float, up_offset: float = 1.0) -> torch.Tensor:
     g, u = gate_up.float().chunk(2, dim=-1)
-    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
-    return (g * torch.sigmoid(alpha * g) * (u + 1)).to(gate_up.dtype)
+    if limit > 0:
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return (g * torch.sigmoid(alpha * g) * (u + up_offset)).to(gate_up.dtype)
 
 
-def clamped_experts(x, w13, w2, weights, idx, limit, alpha):
+def clamped_experts(x, w13, w2, weights, idx, limit, alpha, up_offset=1.0):
     """Weighted sum of the chosen experts' outputs: ``w13 [E, 2I, H]`` (gate rows, then up rows), ``w2 [E, H, I]``."""
     out = torch.zeros(x.shape[0], x.shape[1], dtype=torch.float32)
     for e in range(w13.shape[0]):
         rows, slot = (idx == e).nonzero(as_tuple=True)
         if rows.numel():
-            a = clamped_glu(linear(x[rows], w13[e]), limit, alpha)
+            a = clamped_glu(linear(x[rows], w13[e]), limit, alpha, up_offset)
             out.index_add_(0, rows, linear(a, w2[e]).float() * weights[rows, slot][:, None])
     return out
 

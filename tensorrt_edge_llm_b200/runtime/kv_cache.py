@@ -78,6 +78,10 @@ class KVCacheManager:
         self.page_size = page_size
         self.max_seats = max_seats
         self.max_pages_per_seq = max_pages_per_seq
+        # most tokens of one sequence: its pages, and the positions that the model has a table row for
+        self.max_tokens = max_pages_per_seq * page_size
+        if cfg.learned_positions:
+            self.max_tokens = min(self.max_tokens, cfg.max_position_embeddings)
         self.num_layers = num_layers if num_layers is not None else sum(t in KV_LAYERS for t in cfg.layer_types)
         hkv = max(cfg.num_key_value_heads // cfg.tp_size, 1)
         self.dtype = dtype or cfg.compute_dtype
@@ -145,6 +149,8 @@ class KVCacheManager:
         have = self._pages.setdefault(seat, [])
         if need > self.max_pages_per_seq:
             raise ValueError(f"sequence of {total_tokens} tokens exceeds {self.max_pages_per_seq} pages")
+        if total_tokens > self.max_tokens:
+            raise ValueError(f"sequence of {total_tokens} tokens exceeds the model's {self.max_tokens} positions")
         if need > len(have):
             if self.native is not None:
                 self.native.reserve(seat, total_tokens)

@@ -110,14 +110,14 @@ class ModelSession(rt.RuntimeSession):
         c.max_batch_size = self.kv.max_seats
         c.max_input_length = self.max_input_len
         c.kv_page_size = self.kv.page_size
-        c.max_kv_tokens = self.kv.max_pages_per_seq * self.kv.page_size
+        c.max_kv_tokens = self.kv.max_tokens
         return c
 
     def admit(self, request_id, req):
         r = rt.AdmissionResult()
         n = len(req.prompt_ids)
         need = n + req.max_tokens
-        if n > self.max_input_len or need > self.kv.max_pages_per_seq * self.kv.page_size:
+        if n > self.max_input_len or need > self.kv.max_tokens:
             r.admitted, r.retry_later, r.reason = False, False, "EDGELLM_INPUT_TOO_LONG: prompt + max_tokens exceed the KV capacity"
             return r
         row_state = None

@@ -218,7 +218,7 @@ def create_app(llm: LLM, api: Optional[ApiConfig] = None, chat_template: Optiona
         vision = multimodal is not None and multimodal.vision is not None
         return {"chat": True, "transcription": audio, "speech": False,
                 "input_modalities": ["text"] + (["image"] if vision else []) + (["audio"] if audio else []), "output_modalities": ["text"],
-                "max_model_len": llm.kv.max_pages_per_seq * llm.kv.page_size, "max_input_len": llm.max_input_len,
+                "max_model_len": llm.kv.max_tokens, "max_input_len": llm.max_input_len,
                 "max_batch_size": llm.max_batch_size, "max_num_seqs": llm.max_batch_size, "kv_cache_dtype": str(llm.kv.pool.dtype).replace("torch.", ""),
                 "speculative_decoding": spec is not None or llm.diffusion_decoder is not None,
                 "speculative_method": getattr(spec, "name", "eagle3" if spec is not None else ("block_diffusion" if llm.diffusion_decoder is not None else None)),

@@ -130,14 +130,14 @@ def test_products_with_fp32_results(t, width, n, dtype):
 def test_experts_into_the_stream(t, width, e, top, ff, dtype):
     from tensorrt_edge_llm_b200 import ops
     from tensorrt_edge_llm_b200.config import LAYER_ATTENTION, AttentionConfig, LayerConfig, ModelConfig, MoeConfig
-    from tensorrt_edge_llm_b200.models.qwen3_moe import ClampedExperts
+    from tensorrt_edge_llm_b200.models.qwen3_moe import GatedExperts
     dt = DTYPES[dtype]
     spec = MoeConfig(e, top, ff, 0.7)
     cfg = ModelConfig(model_type="dimesun", hidden_size=width, num_hidden_layers=1, dtype=dtype, layer_types=[LAYER_ATTENTION],
                       layer_specs=[LayerConfig(LAYER_ATTENTION, AttentionConfig(), None, spec)])
     c = cases.moe(e, top, ff, 0.7)
     w = {k: v.to(dt) for k, v in oracle.random_weights(cases.small_config([("attention", cases.attn_mixer(1, 1, 64), c)], width=width)).items()}
-    m = ClampedExperts(cfg, spec, "m")
+    m = GatedExperts(cfg, spec, "m")
     assert m.load_checkpoint(lambda n: w["l0.mlp.e{}.{}".format(n.split(".")[2], n.split(".")[3][:-5])])
     m = m.to(DEV)
     g = torch.Generator().manual_seed(4)
