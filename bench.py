@@ -94,10 +94,10 @@ def main() -> int:
     ap.add_argument("--steps", type=int, default=3)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="dense", choices=["dense", "moe", "hybrid", "eagle", "serve", "dimesun", "debonex", "begupel"],
+    ap.add_argument("--workload", default="dense", choices=["dense", "moe", "hybrid", "eagle", "serve", "dimesun", "debonex", "begupel", "ditenex"],
                     help="dense = the headline benchmark; moe / hybrid / eagle are the secondary configurations; dimesun = the mLSTM / chunked "
                          "attention family, debonex = the channel-decay delta rule / latent attention family, begupel = the lightning attention / parallel "
-                         "attention and delta rule family, each beside the closest other model at equal "
+                         "attention and delta rule family, ditenex = the mixed-score attention family, each beside the closest other model at equal "
                          "size; serve = the request engine "
                          "with staggered arrivals (in-flight batching)")
     ap.add_argument("--batch", type=int, default=None)

@@ -7,6 +7,7 @@ warm-up, synthetic seeded token ids, random-init weights of the named architectu
     python bench.py --workload eagle    # EAGLE-3 tree speculative decoding on the Qwen3-8B shape, forced accept lengths
     python bench.py --workload begupel  # windowed attention beside a delta rule, lightning attention, beside a like-sized hybrid
     python bench.py --workload debonex  # channel-decay delta rule + latent attention beside a like-sized GDN / attention hybrid
+    python bench.py --workload ditenex  # attention with mixed scores, dense / expert feed-forwards, beside a like-sized windowed attention stack
     python bench.py --workload dimesun  # looped-stack hybrid (mLSTM + chunked attention + experts) beside a like-sized GDN hybrid
     python bench.py --workload serve    # the served path: native request engine, staggered arrivals, in-flight batching
 """
@@ -263,6 +264,11 @@ def run_begupel(args) -> dict:
     return run(args)
 
 
+def run_ditenex(args) -> dict:
+    from .ditenex import run
+    return run(args)
+
+
 def run_debonex(args) -> dict:
     from .debonex import run
     return run(args)
@@ -274,7 +280,7 @@ def run_dimesun(args) -> dict:
 
 
 def main(args) -> int:
-    fn = {"begupel": run_begupel, "debonex": run_debonex, "dimesun": run_dimesun, "moe": run_moe, "hybrid": run_hybrid, "eagle": run_eagle, "serve": run_serve}[args.workload]
+    fn = {"begupel": run_begupel, "debonex": run_debonex, "dimesun": run_dimesun, "ditenex": run_ditenex, "moe": run_moe, "hybrid": run_hybrid, "eagle": run_eagle, "serve": run_serve}[args.workload]
     out = fn(args)
     rank, world, llm = out.pop("_rank", 0), out.pop("_world", 1), out.pop("_llm", None)
     out.update({"steps": args.steps, "warmup": args.warmup, "higher_is_better": True})
