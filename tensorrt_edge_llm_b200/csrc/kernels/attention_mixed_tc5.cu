@@ -7,9 +7,10 @@
 //                   A tile's keys, then its values stream through one ring in pairs of 64-feature chunks; a pair's slot is refilled as
 //                   soon as its products are done.  All columns meet all value heads (the products are as narrow as they get); a
 //                   column's output is read from the block of its own head.
-//   mixed_prefill   prompt portions.  QT query tiles of 128 rows of one head per CTA, a softmax warpgroup each.  Wide queries stay in shared
-//                   memory; key chunks of 64 features stream through a ring, so that scores of the next tile start while chunks of it
-//                   still arrive; probabilities stay in TMEM (the A operand of P·V), over the scores they were made from.
+//   mixed_prefill   prompt portions.  128 rows of one head per CTA; wide queries stay in shared memory, chunks of 128 keys x 64 features stream
+//                   through a ring, so that scores of the next tile start while chunks of it still arrive.  Two softmax warpgroups take
+//                   64 keys of a tile each, with maxima, sums and outputs of their own, which join at the end; probabilities stay in
+//                   TMEM (the A operand of P·V), over the scores they were made from.
 //
 // HQ = 2: queries come as a high and a low half (2^-17 together), in mixed_decode as further columns, in mixed_prefill as further products.
 // Probabilities enter P·V as a high and a low half.  Scores, bias, maxima and sums are fp32.  The producer and the MMA warp walk their loops
@@ -441,79 +442,67 @@ struct MixedPreParams {
     const int* q_len;
     const int* past_len;
     const int* page_table;
-    int max_pages, heads, hkv, chunks, window, kslots;
+    int max_pages, heads, hkv, chunks, window, kslots, vstages;
     long long ld_gate;
     float scale_log2;
     int* status;
 };
 
-constexpr int kMixTile = 64;                 // keys per tile: a page
-constexpr int kMixKChunk = kMixTile * 128;   // bytes of [64 keys x 64 features]
+constexpr int kMixTile = 128;                // keys per tile: two pages, one per softmax warpgroup
+constexpr int kMixKChunk = kMixTile * 128;   // bytes of [128 keys x 64 features]
 constexpr int kMixQChunk = 128 * 128;        // bytes of [128 rows x 64 features]
-constexpr int kMixKSlots = 16;
-constexpr int kMixVStages = 2;
+constexpr int kMixKSlots = 8;
+constexpr int kMixThreadsPre = 320;          // producer, MMA issuer, two softmax warpgroups
 
-// grid (query tiles of QT * 128 rows, heads, sequences).  VC: 64-feature chunks of a head.
-template <int VC, int QT, int HQ>
-__global__ void __launch_bounds__(64 + QT * 128, 1)
+// grid (query tiles of 128 rows, heads, sequences).  VC: 64-feature chunks of a head.
+template <int VC, int HQ>
+__global__ void __launch_bounds__(kMixThreadsPre, 1)
 mixed_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_kv, const __grid_constant__ MixedPreParams p) {
     constexpr int VP = VC * 64, kVStage = VC * kMixKChunk;
-    // TMEM per query tile: two score buffers of 64 columns (each turns into high | low probabilities), then the output
-    constexpr uint32_t kTileCols = 256, kOCol = 128, kTmemCols = QT * kTileCols;
+    // TMEM: two score buffers of 128 columns (64 of each warpgroup, which turn into its high | low probabilities), then an output per warpgroup
+    constexpr uint32_t kOCol = 256, kTmemCols = 512;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-    const int chunks = p.chunks, q_tile = HQ * chunks * kMixQChunk;
-    uint8_t* s_q = smem;                                  // [QT][HQ][chunks]
-    uint8_t* s_k = s_q + QT * q_tile;
+    const int chunks = p.chunks;
+    uint8_t* s_q = smem;                                  // [HQ][chunks]; at the end the warpgroups exchange halves of their outputs here
+    uint8_t* s_k = s_q + HQ * chunks * kMixQChunk;
     uint8_t* s_v = s_k + p.kslots * kMixKChunk;
-    uint64_t* bars = reinterpret_cast<uint64_t*>(s_v + kMixVStages * kVStage);
+    uint64_t* bars = reinterpret_cast<uint64_t*>(s_v + p.vstages * kVStage);
     uint64_t* q_full = bars;
-    uint64_t* s_full = bars + 1;                          // [tile][buffer]
-    uint64_t* p_full = s_full + 4;
-    uint64_t* o_done = p_full + 4;                        // [tile][buffer]: two in turn, so that a wait never meets the phase after next
+    uint64_t* s_full = bars + 1;                          // [buffer]
+    uint64_t* p_full = s_full + 2;                        // [warpgroup][buffer]
+    uint64_t* o_done = p_full + 4;                        // [warpgroup][buffer]: two in turn, so that a wait never meets the phase after next
     uint64_t* k_full = o_done + 4;
     uint64_t* k_empty = k_full + kMixKSlots;
     uint64_t* v_full = k_empty + kMixKSlots;
-    uint64_t* v_empty = v_full + kMixVStages;
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(v_empty + kMixVStages);
+    uint64_t* v_empty = v_full + 2;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(v_empty + 2);
     volatile uint32_t* abort_flag = tmem_slot + 1;
 
     pdl_wait();                                           // dependents start at the end: a long kernel runs slower under waiting ones
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int qt = gridDim.x - 1 - blockIdx.x;            // long rows first
     const int head = blockIdx.y, seq = blockIdx.z;
-    const int qlen = p.q_len[seq], past = p.past_len[seq], tok0 = qt * QT * 128;
+    const int qlen = p.q_len[seq], past = p.past_len[seq], tok0 = qt * 128;
     if (tok0 >= qlen) return;                             // uniform, before any barrier or TMEM use
     const int qrow0 = p.q_start[seq] + tok0, kvh = head / (p.heads / p.hkv);
-    // key tiles [lo, hi) that a query tile sees (none: the tile has no rows)
-    int lo[QT], hi[QT];
-    int live = 0, jlo = 0, jhi = 0;
-#pragma unroll
-    for (int t = 0; t < QT; ++t) {
-        const int r0 = tok0 + t * 128;
-        lo[t] = hi[t] = 0;
-        if (r0 >= qlen) continue;
-        lo[t] = max(0, past + r0 - p.window + 1) / kMixTile;
-        hi[t] = (past + min(qlen, r0 + 128) + kMixTile - 1) / kMixTile;
-        if (live == 0) jlo = lo[t];
-        jhi = hi[t];
-        ++live;
-    }
+    const int row_first = past + tok0, row_last = past + min(qlen, tok0 + 128) - 1;
+    const int jlo = max(0, row_first - p.window + 1) / kMixTile, jhi = row_last / kMixTile + 1;      // key tiles [jlo, jhi)
 
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
-        for (int i = 0; i < 4; ++i) {
+        for (int i = 0; i < 2; ++i) {
             mbar_init(&s_full[i], 1);
+            mbar_init(&v_full[i], 1);
+            mbar_init(&v_empty[i], 1);
+        }
+        for (int i = 0; i < 4; ++i) {
             mbar_init(&p_full[i], 128);
             mbar_init(&o_done[i], 1);
         }
         for (int s = 0; s < p.kslots; ++s) {
             mbar_init(&k_full[s], 1);
             mbar_init(&k_empty[s], 1);
-        }
-        for (int s = 0; s < kMixVStages; ++s) {
-            mbar_init(&v_full[s], 1);
-            mbar_init(&v_empty[s], 1);
         }
         *abort_flag = 0;
         mbar_fence_init();
@@ -530,20 +519,23 @@ mixed_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
     if (warp == 0) {
         // ---- producer: K(jlo); then K(j + 1), V(j) ----
         const bool leader = elect_one();
-        if (leader) {
-            mbar_expect_tx(q_full, live * q_tile);
-            for (int t = 0; t < live; ++t)
-                for (int c = 0; c < HQ * chunks; ++c) tma_load_3d(s_q + t * q_tile + c * kMixQChunk, &tma_q, q_full, c * 64, head, qrow0 + t * 128);
-        }
         const int* pages = p.page_table + (size_t)seq * p.max_pages;
+        const int last_page = row_last / kMixPage;        // pages behind it hold nothing that a row sees: they read page 0, masked
+        auto page_of = [&](int j, int half) { return 2 * j + half <= last_page ? max(pages[2 * j + half], 0) : 0; };
         int ks = 0, vs = 0;
         uint32_t kph = 1, vph = 1;
-        auto load_keys = [&](int page) {
+        auto load_keys = [&](int p0, int p1) {
+            int part = 0, h = 0;
             for (int c = 0; c < chunks; ++c) {
                 if (!__all_sync(0xffffffffu, mbar_wait(&k_empty[ks], kph, abort_flag, p.status, kStatusProducerTimeout))) return false;
                 if (leader) {
                     mbar_expect_tx(&k_full[ks], kMixKChunk);
-                    tma_load_4d(s_k + ks * kMixKChunk, &tma_kv, &k_full[ks], 0, 0, c % VC, page * 2 * p.hkv + c / VC);
+                    tma_load_4d(s_k + ks * kMixKChunk, &tma_kv, &k_full[ks], 0, 0, part, p0 * 2 * p.hkv + h);
+                    tma_load_4d(s_k + ks * kMixKChunk + kMixKChunk / 2, &tma_kv, &k_full[ks], 0, 0, part, p1 * 2 * p.hkv + h);
+                }
+                if (++part == VC) {
+                    part = 0;
+                    ++h;
                 }
                 if (++ks == p.kslots) {
                     ks = 0;
@@ -552,25 +544,31 @@ mixed_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
             }
             return true;
         };
-        int page = max(pages[jlo], 0), ahead = jlo + 1 < jhi ? pages[jlo + 1] : 0;
-        bool ok = load_keys(page);
+        int p0 = page_of(jlo, 0), p1 = page_of(jlo, 1), n0 = page_of(jlo + 1, 0), n1 = page_of(jlo + 1, 1);
+        if (leader) {
+            mbar_expect_tx(q_full, HQ * chunks * kMixQChunk);
+            for (int c = 0; c < HQ * chunks; ++c) tma_load_3d(s_q + c * kMixQChunk, &tma_q, q_full, c * 64, head, qrow0);
+        }
+        bool ok = load_keys(p0, p1);
         for (int j = jlo; j < jhi && ok; ++j) {
-            const int next = max(ahead, 0);
-            if (j + 2 < jhi) ahead = pages[j + 2];        // fetched a tile before it is used
-            if (j + 1 < jhi) ok = load_keys(next);
+            const int f0 = page_of(j + 2, 0), f1 = page_of(j + 2, 1);            // fetched a tile before they are used
+            if (j + 1 < jhi) ok = load_keys(n0, n1);
             ok = ok && __all_sync(0xffffffffu, mbar_wait(&v_empty[vs], vph, abort_flag, p.status, kStatusProducerTimeout));
             if (!ok) break;
             if (leader) {
                 mbar_expect_tx(&v_full[vs], kVStage);
 #pragma unroll
-                for (int c = 0; c < VC; ++c)
-                    tma_load_4d(s_v + vs * kVStage + c * kMixKChunk, &tma_kv, &v_full[vs], 0, 0, c, (page * 2 + 1) * p.hkv + kvh);
+                for (int c = 0; c < VC; ++c) {
+                    uint8_t* dst = s_v + vs * kVStage + c * kMixKChunk;
+                    tma_load_4d(dst, &tma_kv, &v_full[vs], 0, 0, c, (p0 * 2 + 1) * p.hkv + kvh);
+                    tma_load_4d(dst + kMixKChunk / 2, &tma_kv, &v_full[vs], 0, 0, c, (p1 * 2 + 1) * p.hkv + kvh);
+                }
             }
-            if (++vs == kMixVStages) {
+            if (++vs == p.vstages) {
                 vs = 0;
                 vph ^= 1;
             }
-            page = next;
+            p0 = n0, p1 = n1, n0 = f0, n1 = f1;
         }
     } else if (warp == 1) {
         // ---- MMA issuer: S(jlo); then S(j + 1), P·V(j) ----
@@ -584,28 +582,19 @@ mixed_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
         };
         int ks = 0, vs = 0;                               // ring positions of the next key chunk and value tile
         uint32_t kph = 0, vph = 0;
-        auto issue_s = [&](int j) {
+        auto issue_s = [&](int n) {                       // n: tile counted from jlo
+            const uint32_t d = tmem_base + (n & 1) * kMixTile;
             for (int c = 0; c < chunks; ++c) {
                 if (!wait(&k_full[ks], kph)) return false;
-                const uint64_t dk = desc_k + (uint64_t)((ks * kMixKChunk) >> 4);
+                const uint64_t dk = desc_k + (uint64_t)((ks * kMixKChunk) >> 4), dq = desc_q + (uint64_t)((c * kMixQChunk) >> 4);
                 if (leader) {
 #pragma unroll
-                    for (int t = 0; t < QT; ++t) {
-                        if (j < lo[t] || j >= hi[t]) continue;
-                        const uint32_t d = tmem_base + t * kTileCols + ((j - lo[t]) & 1) * 64;
-                        const uint64_t dq = desc_q + (uint64_t)((t * q_tile + c * kMixQChunk) >> 4);
+                    for (int h = 0; h < HQ; ++h)
 #pragma unroll
-                        for (int h = 0; h < HQ; ++h)
-#pragma unroll
-                            for (int k = 0; k < 4; ++k)
-                                umma_f16(d, dq + (uint64_t)((h * chunks * kMixQChunk) >> 4) + 2 * k, dk + 2 * k, idesc_s, (c | h | k) ? 1u : 0u);
-                    }
+                        for (int k = 0; k < 4; ++k)
+                            umma_f16(d, dq + (uint64_t)((h * chunks * kMixQChunk) >> 4) + 2 * k, dk + 2 * k, idesc_s, (c | h | k) ? 1u : 0u);
                     umma_commit(&k_empty[ks]);
-                    if (c == chunks - 1) {
-#pragma unroll
-                        for (int t = 0; t < QT; ++t)
-                            if (j >= lo[t] && j < hi[t]) umma_commit(&s_full[t * 2 + ((j - lo[t]) & 1)]);
-                    }
+                    if (c == chunks - 1) umma_commit(&s_full[n & 1]);
                 }
                 __syncwarp();
                 if (++ks == p.kslots) {
@@ -615,55 +604,51 @@ mixed_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
             }
             return true;
         };
-        bool ok = wait(q_full, 0) && issue_s(jlo);
-        for (int j = jlo; j < jhi && ok; ++j) {
-            if (j + 1 < jhi) ok = issue_s(j + 1);
+        const int ntiles = jhi - jlo;
+        bool ok = wait(q_full, 0) && issue_s(0);
+        for (int n = 0; n < ntiles && ok; ++n) {
+            if (n + 1 < ntiles) ok = issue_s(n + 1);
             ok = ok && wait(&v_full[vs], vph);
             const uint64_t dv = desc_v + (uint64_t)((vs * kVStage) >> 4);
 #pragma unroll
-            for (int t = 0; t < QT; ++t) {
-                if (!ok || j < lo[t] || j >= hi[t]) continue;
-                const int n = j - lo[t];
-                ok = wait(&p_full[t * 2 + (n & 1)], (n >> 1) & 1);
-                if (!ok) continue;
-                const uint32_t a = tmem_base + t * kTileCols + (n & 1) * 64, d = tmem_base + t * kTileCols + kOCol;
+            for (int g = 0; g < 2; ++g) {
+                ok = ok && wait(&p_full[g * 2 + (n & 1)], (n >> 1) & 1);
+                if (!ok) break;
+                const uint32_t a = tmem_base + (n & 1) * kMixTile + g * 64, d = tmem_base + kOCol + g * 128;
                 if (leader) {
 #pragma unroll
                     for (int half = 0; half < 2; ++half)
 #pragma unroll
-                        for (int k = 0; k < kMixTile / 16; ++k)
-                            umma_f16_ts(d, a + half * 32 + k * 8, dv + (uint64_t)((k * 2048) >> 4), idesc_o, (n | half | k) ? 1u : 0u);
-                    umma_commit(&o_done[t * 2 + (n & 1)]);
+                        for (int k = 0; k < 4; ++k)
+                            umma_f16_ts(d, a + half * 32 + k * 8, dv + (uint64_t)(((g * 4 + k) * 2048) >> 4), idesc_o, (n | half | k) ? 1u : 0u);
+                    umma_commit(&o_done[g * 2 + (n & 1)]);
+                    if (g == 1) umma_commit(&v_empty[vs]);
                 }
                 __syncwarp();
             }
-            if (ok && leader) umma_commit(&v_empty[vs]);
-            __syncwarp();
-            if (++vs == kMixVStages) {
+            if (++vs == p.vstages) {
                 vs = 0;
                 vph ^= 1;
             }
         }
     } else {
-        // ---- softmax / epilogue: one thread per query row ----
-        const int t = (warp - 2) >> 2, quad = warp & 3;
-        const int r = quad * 32 + lane, qi = tok0 + t * 128 + r;
-        const int from = t == 0 ? lo[0] : lo[QT - 1], mine = (t == 0 ? hi[0] : hi[QT - 1]) - from;
-        const uint32_t base = tmem_base + t * kTileCols + (static_cast<uint32_t>(quad * 32) << 16);
+        // ---- softmax / epilogue: warpgroup g takes keys g * 64 .. + 63 of every tile, one thread per query row ----
+        const int g = (warp - 2) >> 2, quad = warp & 3;
+        const int r = quad * 32 + lane, qi = tok0 + r, ntiles = jhi - jlo;
+        const uint32_t base = tmem_base + (static_cast<uint32_t>(quad * 32) << 16), s_col = base + g * 64, o_col = base + kOCol + g * 128;
         const int limit = past + qi;                      // last visible key
-        const int row_first = past + tok0 + t * 128, row_last = past + min(qlen, tok0 + t * 128 + 128) - 1;
         const float slope = p.slopes[head] * kLog2e;
         float m_used = -INFINITY, l_sum = 0.f;
         bool ok = true;
-        for (int n = 0; n < mine && ok; ++n) {
+        for (int n = 0; n < ntiles && ok; ++n) {
             const int b = n & 1;
-            if (!mbar_wait(&s_full[t * 2 + b], (n >> 1) & 1, abort_flag, p.status, kStatusEpilogueTimeout)) { ok = false; break; }
+            if (!mbar_wait(&s_full[b], (n >> 1) & 1, abort_flag, p.status, kStatusEpilogueTimeout)) { ok = false; break; }
             tc_fence_after_sync();
-            float s[kMixTile];
+            float s[64];
             {
                 uint32_t r0[32], r1[32];
-                tmem_ld_x32(base + b * 64, r0);
-                tmem_ld_x32(base + b * 64 + 32, r1);
+                tmem_ld_x32(s_col + b * kMixTile, r0);
+                tmem_ld_x32(s_col + b * kMixTile + 32, r1);
                 tmem_ld_wait();
 #pragma unroll
                 for (int i = 0; i < 32; ++i) {
@@ -671,34 +656,34 @@ mixed_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                     s[32 + i] = __uint_as_float(r1[i]);
                 }
             }
-            const int c0 = (from + n) * kMixTile;
+            const int c0 = (jlo + n) * kMixTile + g * 64;
             const float bias = slope * (float)(c0 - limit);
 #pragma unroll
-            for (int i = 0; i < kMixTile; ++i) s[i] = fmaf(s[i], p.scale_log2, fmaf(slope, (float)i, bias));
-            if (c0 + kMixTile - 1 > row_first || c0 <= row_last - p.window) {       // the tile reaches the diagonal or the window's start
+            for (int i = 0; i < 64; ++i) s[i] = fmaf(s[i], p.scale_log2, fmaf(slope, (float)i, bias));
+            if (c0 + 63 > row_first || c0 <= row_last - p.window) {                 // the keys reach the diagonal or the window's start
 #pragma unroll
-                for (int i = 0; i < kMixTile; ++i) s[i] = c0 + i <= limit && c0 + i > limit - p.window ? s[i] : -INFINITY;
+                for (int i = 0; i < 64; ++i) s[i] = c0 + i <= limit && c0 + i > limit - p.window ? s[i] : -INFINITY;
             }
-            float mx = s[0];
+            float mx[4] = {s[0], s[1], s[2], s[3]};
 #pragma unroll
-            for (int i = 1; i < kMixTile; ++i) mx = fmaxf(mx, s[i]);
-            const float m_new = fmaxf(m_used, mx);
+            for (int i = 4; i < 64; ++i) mx[i & 3] = fmaxf(mx[i & 3], s[i]);
+            const float m_new = fmaxf(m_used, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])));
             const bool need = m_new > m_used + 8.0f;
             if (n == 0) {
                 m_used = m_new;
             } else if (__any_sync(0xffffffffu, need)) {
                 // P·V of tile n - 1 (that of tile n - 2 was issued ahead of these scores and is complete)
-                if (!mbar_wait(&o_done[t * 2 + (b ^ 1)], ((n - 1) >> 1) & 1, abort_flag, p.status, kStatusEpilogueTimeout)) { ok = false; break; }
+                if (!mbar_wait(&o_done[g * 2 + (b ^ 1)], ((n - 1) >> 1) & 1, abort_flag, p.status, kStatusEpilogueTimeout)) { ok = false; break; }
                 tc_fence_after_sync();
                 const float f = need ? exp2f(m_used - m_new) : 1.f;
 #pragma unroll 1
                 for (int c = 0; c < VP / 16; ++c) {
                     uint32_t o[16];
-                    tmem_ld_x16(base + kOCol + c * 16, o);
+                    tmem_ld_x16(o_col + c * 16, o);
                     tmem_ld_wait();
 #pragma unroll
                     for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * f);
-                    tmem_st_x16(base + kOCol + c * 16, o);
+                    tmem_st_x16(o_col + c * 16, o);
                 }
                 if (need) {
                     l_sum *= f;
@@ -706,60 +691,91 @@ mixed_prefill_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_con
                 }
             }
             const float mref = m_used == -INFINITY ? 0.f : m_used;
-            float acc = 0.f;
+            float acc[2] = {0.f, 0.f};
 #pragma unroll
             for (int h = 0; h < 2; ++h) {                             // 32 keys at a time: 16 columns of high halves, 16 of low ones
                 uint32_t hw[16], lw[16];
 #pragma unroll
                 for (int i = 0; i < 16; ++i) {
                     const float e0 = exp2f(s[h * 32 + 2 * i] - mref), e1 = exp2f(s[h * 32 + 2 * i + 1] - mref);
-                    acc += e0 + e1;
+                    acc[0] += e0;
+                    acc[1] += e1;
                     hw[i] = Cvt<MixT>::pack2(e0, e1);
                     const MixT* q = reinterpret_cast<const MixT*>(&hw[i]);
                     lw[i] = Cvt<MixT>::pack2(e0 - Cvt<MixT>::to_f(q[0]), e1 - Cvt<MixT>::to_f(q[1]));
                 }
-                tmem_st_x16(base + b * 64 + h * 16, hw);
-                tmem_st_x16(base + b * 64 + 32 + h * 16, lw);
+                tmem_st_x16(s_col + b * kMixTile + h * 16, hw);
+                tmem_st_x16(s_col + b * kMixTile + 32 + h * 16, lw);
             }
-            l_sum += acc;
+            l_sum += acc[0] + acc[1];
             tmem_st_wait();
             tc_fence_before_sync();
-            mbar_arrive(&p_full[t * 2 + b]);
+            mbar_arrive(&p_full[g * 2 + b]);
         }
-        if (ok && mine > 0) {
-            ok = mbar_wait(&o_done[t * 2 + ((mine - 1) & 1)], ((mine - 1) >> 1) & 1, abort_flag, p.status, kStatusEpilogueTimeout);
-            if (ok) {
-                tc_fence_after_sync();
-                const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
-                const size_t tok = (size_t)p.q_start[seq] + qi;
-                MixT* dst = reinterpret_cast<MixT*>(p.out) + (tok * p.heads + head) * VP;
-                const MixT* gate = p.gate ? reinterpret_cast<const MixT*>(p.gate) + tok * p.ld_gate + head * VP : nullptr;
+        // ---- the two halves of a row join: each warpgroup hands over the features that the other one writes ----
+        constexpr int kHalf = VP / 2, kPitch = kHalf + 4;             // fp32 words of a row's half in shared memory, padded
+        const size_t tok = (size_t)p.q_start[seq] + qi;
+        const MixT* gate = p.gate && qi < qlen ? reinterpret_cast<const MixT*>(p.gate) + tok * p.ld_gate + head * VP + g * kHalf : nullptr;
+        if (ok) ok = mbar_wait(&o_done[g * 2 + ((ntiles - 1) & 1)], ((ntiles - 1) >> 1) & 1, abort_flag, p.status, kStatusEpilogueTimeout);
+        // Q is read by score products only, and those of the last tile are complete: its room is free
+        float* mine = reinterpret_cast<float*>(s_q) + ((size_t)g * 128 + r) * kPitch;
+        const float* theirs = reinterpret_cast<const float*>(s_q) + ((size_t)(g ^ 1) * 128 + r) * kPitch;
+        float* s_ml = reinterpret_cast<float*>(s_q) + 256 * kPitch;   // [warpgroup][maximum | sum][row]
+        if (ok) {
+            tc_fence_after_sync();
+            s_ml[g * 256 + r] = m_used;
+            s_ml[g * 256 + 128 + r] = l_sum;
 #pragma unroll 1
-                for (int c = 0; c < VP / 16; ++c) {
-                    uint32_t o[16];
-                    tmem_ld_x16(base + kOCol + c * 16, o);
-                    tmem_ld_wait();
-                    if (qi < qlen) {
-                        float v[16];
+            for (int c = 0; c < kHalf / 16; ++c) {
+                uint32_t o[16];
+                tmem_ld_x16(o_col + (g ^ 1) * kHalf + c * 16, o);
+                tmem_ld_wait();
 #pragma unroll
-                        for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(o[i]) * inv;
-                        if (gate) {
-                            alignas(16) MixT g[16];
-#pragma unroll
-                            for (int i = 0; i < 2; ++i) reinterpret_cast<uint4*>(g)[i] = reinterpret_cast<const uint4*>(gate + c * 16)[i];
-#pragma unroll
-                            for (int i = 0; i < 16; ++i) v[i] *= mix_sigmoid(Cvt<MixT>::to_f(g[i]));
-                        }
-                        uint32_t w[8];
-#pragma unroll
-                        for (int i = 0; i < 8; ++i) w[i] = Cvt<MixT>::pack2(v[2 * i], v[2 * i + 1]);
-                        reinterpret_cast<uint4*>(dst + c * 16)[0] = make_uint4(w[0], w[1], w[2], w[3]);
-                        reinterpret_cast<uint4*>(dst + c * 16)[1] = make_uint4(w[4], w[5], w[6], w[7]);
-                    }
-                    __syncwarp();
-                }
-                tc_fence_before_sync();
+                for (int i = 0; i < 4; ++i)
+                    *reinterpret_cast<uint4*>(mine + c * 16 + i * 4) = make_uint4(o[i * 4], o[i * 4 + 1], o[i * 4 + 2], o[i * 4 + 3]);
             }
+        }
+        named_barrier_sync(1, 256);
+        if (ok && *abort_flag == 0) {
+            const float om = s_ml[(g ^ 1) * 256 + r], ol = s_ml[(g ^ 1) * 256 + 128 + r], m = fmaxf(m_used, om);
+            float f0 = m_used == -INFINITY ? 0.f : exp2f(m_used - m), f1 = om == -INFINITY ? 0.f : exp2f(om - m);
+            const float l = l_sum * f0 + ol * f1, inv = l > 0.f ? 1.f / l : 0.f;
+            f0 *= inv;
+            f1 *= inv;
+            MixT* dst = reinterpret_cast<MixT*>(p.out) + (tok * p.heads + head) * VP + g * kHalf;
+#pragma unroll
+            for (int c = 0; c < kHalf / 16; ++c) {
+                uint32_t o[16];
+                tmem_ld_x16(o_col + g * kHalf + c * 16, o);
+                alignas(16) MixT gv[16];
+                if (gate) {
+#pragma unroll
+                    for (int i = 0; i < 2; ++i) reinterpret_cast<uint4*>(gv)[i] = reinterpret_cast<const uint4*>(gate + c * 16)[i];
+                }
+                tmem_ld_wait();
+                if (qi < qlen) {
+                    float v[16];
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const float4 t = *reinterpret_cast<const float4*>(theirs + c * 16 + i * 4);
+                        v[i * 4] = __uint_as_float(o[i * 4]) * f0 + t.x * f1;
+                        v[i * 4 + 1] = __uint_as_float(o[i * 4 + 1]) * f0 + t.y * f1;
+                        v[i * 4 + 2] = __uint_as_float(o[i * 4 + 2]) * f0 + t.z * f1;
+                        v[i * 4 + 3] = __uint_as_float(o[i * 4 + 3]) * f0 + t.w * f1;
+                    }
+                    if (gate) {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) v[i] *= mix_sigmoid(Cvt<MixT>::to_f(gv[i]));
+                    }
+                    uint32_t w[8];
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) w[i] = Cvt<MixT>::pack2(v[2 * i], v[2 * i + 1]);
+                    reinterpret_cast<uint4*>(dst + c * 16)[0] = make_uint4(w[0], w[1], w[2], w[3]);
+                    reinterpret_cast<uint4*>(dst + c * 16)[1] = make_uint4(w[4], w[5], w[6], w[7]);
+                }
+                __syncwarp();
+            }
+            tc_fence_before_sync();
         }
     }
     if (*abort_flag) {
@@ -800,20 +816,22 @@ static int launch_mixed_decode(const CUtensorMap& tq, const CUtensorMap& tkv, Mi
     return 0;
 }
 
-template <int VC, int QT, int HQ>
+template <int VC, int HQ>
 static int launch_mixed_prefill(const CUtensorMap& tq, const CUtensorMap& tkv, MixedPreParams p, int nseq, int max_q, cudaStream_t stream) {
-    const int fixed = QT * HQ * p.chunks * kMixQChunk + kMixVStages * VC * kMixKChunk + (13 + 2 * kMixKSlots + 2 * kMixVStages) * 8 + 16 + 1024;
-    p.kslots = (kMixSmemLimit - fixed) / kMixKChunk;
+    // the exchange of outputs at the end takes the room of the queries and, where those are narrow, of the keys behind them
+    const int fixed = HQ * p.chunks * kMixQChunk + (15 + 2 * kMixKSlots) * 8 + 16 + 1024, v_stage = VC * kMixKChunk;
+    p.vstages = kMixSmemLimit - fixed - 2 * v_stage >= 6 * kMixKChunk ? 2 : 1;
+    p.kslots = (kMixSmemLimit - fixed - p.vstages * v_stage) / kMixKChunk;
     if (p.kslots > kMixKSlots) p.kslots = kMixKSlots;
     if (p.kslots < 2) return fail("telb_mixed_attention_prefill: queries too wide for shared memory");
-    const int smem = fixed + p.kslots * kMixKChunk;
+    const int smem = fixed + p.kslots * kMixKChunk + p.vstages * v_stage;
     static int configured = 0;
     if (smem > configured) {
-        cudaError_t e = cudaFuncSetAttribute(mixed_prefill_kernel<VC, QT, HQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        cudaError_t e = cudaFuncSetAttribute(mixed_prefill_kernel<VC, HQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return fail("cudaFuncSetAttribute(mixed_prefill)", e);
         configured = smem;
     }
-    TELB_LAUNCH("mixed_prefill_kernel", (mixed_prefill_kernel<VC, QT, HQ>), dim3((max_q + QT * 128 - 1) / (QT * 128), p.heads, nseq), dim3(64 + QT * 128), smem, stream, tq, tkv, p);
+    TELB_LAUNCH("mixed_prefill_kernel", (mixed_prefill_kernel<VC, HQ>), dim3((max_q + 127) / 128, p.heads, nseq), dim3(kMixThreadsPre), smem, stream, tq, tkv, p);
     TELB_CHECK_LAUNCH("mixed_prefill_kernel");
     return 0;
 }
@@ -885,7 +903,7 @@ extern "C" int telb_mixed_attention_prefill(const void* q, const void* kv_layer,
     if ((pad != 64 && pad != 128) || hkv < 1 || hkv * pad > 512 || heads % hkv || (halves != 1 && halves != 2)) return fail("telb_mixed_attention_prefill: sizes");
     if (halves == 1 && hkv * pad <= 256) return fail("telb_mixed_attention_prefill: narrow queries come in two halves");
     if (window < 1 || num_seqs > 65535 || heads > 65535 || (gate && ld_gate % 8)) return fail("telb_mixed_attention_prefill: window, sequences, heads or gate pitch");
-    MixedPreParams p{out, gate, slopes, q_start, q_len, past_len, page_table, max_pages, heads, hkv, hkv * pad / 64, window, 0, ld_gate, scale * kLog2e, status};
+    MixedPreParams p{out, gate, slopes, q_start, q_len, past_len, page_table, max_pages, heads, hkv, hkv * pad / 64, window, 0, 0, ld_gate, scale * kLog2e, status};
     CUtensorMap tq, tkv;
     {
         const uint64_t width = (uint64_t)halves * hkv * pad;
@@ -894,11 +912,7 @@ extern "C" int telb_mixed_attention_prefill(const void* q, const void* kv_layer,
         if (make_tmap_nd(&tq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, q, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -1;
     }
     if (mixed_kv_map(&tkv, kv_layer, num_pages, hkv, pad)) return -1;
-#define TELB_MIXED(QT_, HQ_)                                                                            \
-    (pad == 64 ? launch_mixed_prefill<1, QT_, HQ_>(tq, tkv, p, num_seqs, max_q_len, stream)             \
-               : launch_mixed_prefill<2, QT_, HQ_>(tq, tkv, p, num_seqs, max_q_len, stream))
-    if (p.chunks <= 2) return TELB_MIXED(2, 2);
-    if (p.chunks <= 4) return TELB_MIXED(1, 2);
-    return TELB_MIXED(1, 1);
-#undef TELB_MIXED
+    if (p.chunks <= 4)
+        return pad == 64 ? launch_mixed_prefill<1, 2>(tq, tkv, p, num_seqs, max_q_len, stream) : launch_mixed_prefill<2, 2>(tq, tkv, p, num_seqs, max_q_len, stream);
+    return pad == 64 ? launch_mixed_prefill<1, 1>(tq, tkv, p, num_seqs, max_q_len, stream) : launch_mixed_prefill<2, 1>(tq, tkv, p, num_seqs, max_q_len, stream);
 }

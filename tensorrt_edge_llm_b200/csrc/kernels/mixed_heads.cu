@@ -47,79 +47,83 @@ __device__ __forceinline__ void store8(T* p, const float (&v)[8]) {
     for (int i = 0; i < (int)(8 * sizeof(T) / 16); ++i) reinterpret_cast<uint4*>(p)[i] = reinterpret_cast<const uint4*>(e)[i];
 }
 
+// One CTA per row.  An item is (part of the query heads, KV head, eight features); the threads behind the items only help with keys and values.
 // GS: query heads per KV head kept in registers (0: any number, read again for every result).
 template <typename T, int GS>
 __global__ void __launch_bounds__(kMixThreads) mixed_kv_write_kernel(const __grid_constant__ MixedKvParams p) {
-    extern __shared__ float s_mix[];                      // [hq, hq]
     pdl_prologue();
-    const int tid = threadIdx.x, hq = p.hq, d = p.d, gs = hq / p.hkv, vecs = d / 8, units = p.hkv * vecs;
-    for (int i = tid; i < hq * hq; i += kMixThreads) s_mix[i] = p.mix[i];
-    __syncthreads();
-    // items of a row: (part of the heads, KV head, eight features); the parts share the units among spare threads
-    const int parts = min(hq, max(1, kMixThreads / units)), per = (hq + parts - 1) / parts, wide = p.hkv * d;
-    for (int t = blockIdx.x; t < p.tokens; t += gridDim.x) {
-        const T* row = reinterpret_cast<const T*>(p.rows) + (size_t)t * p.ld;
-        T* out = reinterpret_cast<T*>(p.q_out) + (size_t)t * hq * wide * p.halves;
-        for (int w = tid; w < units * parts; w += kMixThreads) {
-            const int part = w / units, u = w - part * units, c = u / vecs, f = (u - c * vecs) * 8;
-            const T* src = row + (size_t)c * gs * d + f;
-            float q[GS > 0 ? GS : 1][8];
+    const int tid = threadIdx.x, t = blockIdx.x, hq = p.hq, d = p.d, gs = GS > 0 ? GS : hq / p.hkv, vecs = d / 8, units = p.hkv * vecs;
+    const int parts = min(hq, max(1, (int)blockDim.x / units)), per = (hq + parts - 1) / parts, wide = p.hkv * d;
+    const T* row = reinterpret_cast<const T*>(p.rows) + (size_t)t * p.ld;
+    T* out = reinterpret_cast<T*>(p.q_out) + (size_t)t * hq * wide * p.halves;
+    for (int w = tid; w < units * parts; w += blockDim.x) {
+        const int part = w / units, u = w - part * units, c = u / vecs, f = (u - c * vecs) * 8;
+        const T* src = row + (size_t)c * gs * d + f;
+        float q[GS > 0 ? GS : 1][8];
+        if constexpr (GS > 0) {
+#pragma unroll
+            for (int i = 0; i < GS; ++i) load8(src + (size_t)i * d, q[i]);
+        }
+        const int h1 = min(hq, (part + 1) * per);
+#pragma unroll 4
+        for (int h = part * per; h < h1; ++h) {
+            const float* m = p.mix + h * hq + c * gs;
+            float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
             if constexpr (GS > 0) {
+                alignas(16) float mm[GS];
+                if constexpr (GS % 4 == 0) {             // hq and c * gs are multiples of 4 then
 #pragma unroll
-                for (int i = 0; i < GS; ++i) load8(src + (size_t)i * d, q[i]);
-            }
-            const int h1 = min(hq, (part + 1) * per);
-            for (int h = part * per; h < h1; ++h) {
-                const float* m = s_mix + h * hq + c * gs;
-                float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-                if constexpr (GS > 0) {
-#pragma unroll
-                    for (int i = 0; i < GS; ++i)
-#pragma unroll
-                        for (int k = 0; k < 8; ++k) v[k] = fmaf(m[i], q[i][k], v[k]);
+                    for (int i = 0; i < GS; i += 4) *reinterpret_cast<float4*>(mm + i) = __ldg(reinterpret_cast<const float4*>(m + i));
                 } else {
-                    for (int i = 0; i < gs; ++i) {
-                        load8(src + (size_t)i * d, q[0]);
 #pragma unroll
-                        for (int k = 0; k < 8; ++k) v[k] = fmaf(m[i], q[0][k], v[k]);
-                    }
+                    for (int i = 0; i < GS; ++i) mm[i] = __ldg(m + i);
                 }
-                T* dst = out + (size_t)h * wide * p.halves + c * d + f;
-                store8(dst, v);
-                if constexpr (sizeof(T) == 2) {
-                    if (p.halves == 2) {
 #pragma unroll
-                        for (int k = 0; k < 8; ++k) v[k] -= Cvt<T>::to_f(Cvt<T>::from_f(v[k]));
-                        store8(dst + wide, v);
-                    }
+                for (int i = 0; i < GS; ++i)
+#pragma unroll
+                    for (int k = 0; k < 8; ++k) v[k] = fmaf(mm[i], q[i][k], v[k]);
+            } else {
+                for (int i = 0; i < gs; ++i) {
+                    load8(src + (size_t)i * d, q[0]);
+#pragma unroll
+                    for (int k = 0; k < 8; ++k) v[k] = fmaf(__ldg(m + i), q[0][k], v[k]);
+                }
+            }
+            T* dst = out + (size_t)h * wide * p.halves + c * d + f;
+            store8(dst, v);
+            if constexpr (sizeof(T) == 2) {
+                if (p.halves == 2) {
+#pragma unroll
+                    for (int k = 0; k < 8; ++k) v[k] -= Cvt<T>::to_f(Cvt<T>::from_f(v[k]));
+                    store8(dst + wide, v);
                 }
             }
         }
-        const int seq = p.seq_ids[t], slot = p.past_len[seq] + t - p.q_start[seq];
-        const int page = p.page_table[(size_t)seq * p.max_pages + slot / p.page_size];
-        if (page < 0) continue;
-        T* kv = reinterpret_cast<T*>(p.kv) + ((size_t)page * 2 * p.hkv * p.page_size + slot % p.page_size) * d;
-        const float share = p.first ? *p.share : 0.f;
-        for (int w = tid; w < 2 * units; w += kMixThreads) {             // heads count through both planes
-            const int c = w / vecs, f = (w - c * vecs) * 8;
-            float v[8];
-            load8(row + (size_t)hq * d + (size_t)w * 8, v);
-            if (p.first && w >= units) {
-                float o[8];
-                load8(reinterpret_cast<const T*>(p.first) + (size_t)t * p.ld_first + (size_t)(w - units) * 8, o);
+    }
+    const int seq = p.seq_ids[t], slot = p.past_len[seq] + t - p.q_start[seq];
+    const int page = p.page_table[(size_t)seq * p.max_pages + slot / p.page_size];
+    if (page < 0) return;
+    T* kv = reinterpret_cast<T*>(p.kv) + ((size_t)page * 2 * p.hkv * p.page_size + slot % p.page_size) * d;
+    const float share = p.first ? *p.share : 0.f;
+    for (int w = tid; w < 2 * units; w += blockDim.x) {                  // heads count through both planes
+        const int c = w / vecs, f = (w - c * vecs) * 8;
+        float v[8];
+        load8(row + (size_t)hq * d + (size_t)w * 8, v);
+        if (p.first && w >= units) {
+            float o[8];
+            load8(reinterpret_cast<const T*>(p.first) + (size_t)t * p.ld_first + (size_t)(w - units) * 8, o);
 #pragma unroll
-                for (int k = 0; k < 8; ++k) v[k] = fmaf(share, o[k], (1.f - share) * v[k]);
-            }
-            store8(kv + (size_t)c * p.page_size * d + f, v);
+            for (int k = 0; k < 8; ++k) v[k] = fmaf(share, o[k], (1.f - share) * v[k]);
         }
+        store8(kv + (size_t)c * p.page_size * d + f, v);
     }
 }
 
 template <typename T>
 static int launch_mixed_kv(const MixedKvParams& p, cudaStream_t stream) {
-    const int slots = 8 * sm_count(), grid = p.tokens < slots ? p.tokens : slots;
-    const size_t smem = (size_t)p.hq * p.hq * sizeof(float);
-#define TELB_MIX(GS_) TELB_LAUNCH("mixed_kv_write_kernel", (mixed_kv_write_kernel<T, GS_>), dim3(grid), dim3(kMixThreads), smem, stream, p)
+    const int units = p.hkv * p.d / 8;
+    const int threads = 2 * units > kMixThreads ? kMixThreads : 2 * units < 64 ? 64 : (2 * units + 31) / 32 * 32;
+#define TELB_MIX(GS_) TELB_LAUNCH("mixed_kv_write_kernel", (mixed_kv_write_kernel<T, GS_>), dim3(p.tokens), dim3(threads), 0, stream, p)
     switch (p.hq / p.hkv) {
         case 1: TELB_MIX(1); break;
         case 2: TELB_MIX(2); break;
@@ -140,7 +144,7 @@ using namespace telb;
 extern "C" int telb_mixed_kv_write(const MixedKvParams* pp, int dtype, cudaStream_t stream) {
     const MixedKvParams& p = *pp;
     if (p.tokens <= 0) return 0;
-    if (p.hkv <= 0 || p.hq % p.hkv || p.hq > 104) return fail("telb_mixed_kv_write: at most 104 query heads, a multiple of the KV heads");
+    if (p.hkv <= 0 || p.hq % p.hkv) return fail("telb_mixed_kv_write: query heads are a multiple of the KV heads");
     if (p.d % 8 || p.ld % 8 || p.ld_first % 8) return fail("telb_mixed_kv_write: heads and row pitches in multiples of 8");
     if (p.halves != 1 && (p.halves != 2 || dtype == 2)) return fail("telb_mixed_kv_write: one or (16-bit) two halves");
     if (p.first && !p.share) return fail("telb_mixed_kv_write: mixed values have a share");

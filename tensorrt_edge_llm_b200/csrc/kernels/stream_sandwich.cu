@@ -9,7 +9,8 @@
 // Stream, norms, shift and state are fp32; tables, y, e and the written h have the activation type.  One CTA walks a block of rows of one
 // sequence.  A shifted block starts with the row before it: inside a portion that row is computed once more, the first row of a portion
 // takes the state.  The CTA that reads a sequence's state also writes it (it computes the portion's last row for that), so no CTA reads
-// what another one of its launch writes, and the rows x are never advanced in place.
+// what another one of its launch writes, and the rows x are never advanced in place.  Steps of
+// many rows run a warp per block instead.
 #include "host_utils.h"
 #include "stream_common.cuh"
 
@@ -41,192 +42,253 @@ struct StreamSandwichParams {
     float mult, eps;
 };
 
-// Sum over the CTA's N threads; `red` holds two turns of N / 32 warp sums, used alternately (one barrier per sum).
+// How a row lies on threads: N threads hold E vectors of four features each, thread i features 4 (e N + i) .. + 3.  N = 32: a warp per row,
+// several rows' blocks per CTA, widths of exactly 128 E (no guards, no barriers); else the whole CTA.
 template <int N>
-__device__ __forceinline__ float block_total(float v, float* red, int& turn) {
-    v = post_warp_sum(v);
-    float* buf = red + (turn & 1) * (N / 32);
-    ++turn;
-    if ((threadIdx.x & 31) == 0) buf[threadIdx.x >> 5] = v;
-    __syncthreads();
-    float s = 0.f;
+struct RowThreads {
+    static constexpr bool kWarp = N == 32;
+    static constexpr int kBlocks = kWarp ? 4 : 1;                    // row blocks of a CTA
+    float* red;                                                      // [2][N / 32], used alternately: one barrier per sum
+    int turn = 0;
+    __device__ __forceinline__ int idx() const { return kWarp ? threadIdx.x & 31 : threadIdx.x; }
+    __device__ __forceinline__ int block() const { return kWarp ? blockIdx.x * kBlocks + (threadIdx.x >> 5) : blockIdx.x; }
+    __device__ __forceinline__ int col(int e) const { return (e * N + idx()) * 4; }
+    __device__ __forceinline__ bool in(int e, int width) const { return kWarp || col(e) < width; }
+    __device__ __forceinline__ float sum(float v) {
+        v = post_warp_sum(v);
+        if constexpr (kWarp) return v;
+        float* buf = red + (turn & 1) * (N / 32);
+        ++turn;
+        if ((threadIdx.x & 31) == 0) buf[threadIdx.x >> 5] = v;
+        __syncthreads();
+        float s = 0.f;
 #pragma unroll
-    for (int w = 0; w < N / 32; ++w) s += buf[w];
-    return s;
+        for (int w = 0; w < N / 32; ++w) s += buf[w];
+        return s;
+    }
+};
+
+template <typename T>
+__device__ __forceinline__ void raw4(const T* p, T (&v)[4]) {
+    if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
+    else *reinterpret_cast<uint2*>(v) = *reinterpret_cast<const uint2*>(p);
 }
 
-// What a row is made of, fetched ahead of the sums of the row before.
+// A row as it lies in memory, so that fetching it waits for nothing: the stream and the sublayer's output, or the token's table row.
 template <typename T, int E>
-struct RowParts {
-    float x[E][4], d[E][4];
+struct RowRaw {
+    float x[E][4];
+    alignas(16) T y[E][4];
 };
 
 template <typename T, int N, int E>
-__device__ __forceinline__ void fetch_row(const StreamSandwichParams& p, int t, RowParts<T, E>& r) {
-    const int id = p.ids ? min(max(p.ids[t], 0), p.vocab - 1) : 0;
-    const int pos = p.pos_table ? min(max(p.positions[t], 0), p.max_pos - 1) : 0;
+__device__ __forceinline__ void fetch_row(const StreamSandwichParams& p, const RowThreads<N>& th, int t, RowRaw<T, E>& r) {
+    const T* y = reinterpret_cast<const T*>(p.y) + (size_t)t * p.width;
+    if (p.ids) y = reinterpret_cast<const T*>(p.table) + (size_t)min(max(p.ids[t], 0), p.vocab - 1) * p.width;
+    const float* x = p.x_in + (size_t)t * p.width;
+    if (!p.ids) {
 #pragma unroll
-    for (int e = 0; e < E; ++e) {
-        const int c = (e * N + threadIdx.x) * 4;
-#pragma unroll
-        for (int i = 0; i < 4; ++i) r.x[e][i] = r.d[e][i] = 0.f;
-        if (c >= p.width) continue;
-        if (p.ids) get4(reinterpret_cast<const T*>(p.table) + (size_t)id * p.width + c, r.x[e]);
-        else get4(p.x_in + (size_t)t * p.width + c, r.x[e]);
-        if (p.pos_table) {
-            float v[4];
-            get4(reinterpret_cast<const T*>(p.pos_table) + (size_t)pos * p.width + c, v);
-#pragma unroll
-            for (int i = 0; i < 4; ++i) r.x[e][i] += v[i];
-        }
-        if (p.y) get4(reinterpret_cast<const T*>(p.y) + (size_t)t * p.width + c, r.d[e]);
+        for (int e = 0; e < E; ++e)
+            if (th.in(e, p.width)) get4(x + th.col(e), r.x[e]);
     }
-    if (p.e) {
-        for (int k = 0; k < p.top_k; ++k) {
-            const int row = p.dst_row[(size_t)t * p.top_k + k];
-            if (row < 0) continue;
-            const float w = p.topk_w[(size_t)t * p.top_k + k];
+    if (p.ids || p.y) {
 #pragma unroll
-            for (int e = 0; e < E; ++e) {
-                const int c = (e * N + threadIdx.x) * 4;
-                if (c >= p.width) break;
-                float v[4];
-                get4(reinterpret_cast<const T*>(p.e) + (size_t)row * p.lde + c, v);
-#pragma unroll
-                for (int i = 0; i < 4; ++i) r.d[e][i] = fmaf(w, v[i], r.d[e][i]);
-            }
-        }
+        for (int e = 0; e < E; ++e)
+            if (th.in(e, p.width)) raw4(y + th.col(e), r.y[e]);
     }
 }
 
-// Advances the row in place (stored when `own`) and leaves its norm, without the weight, in r.d.
-template <typename T, int N, int E>
-__device__ __forceinline__ void advance_row(const StreamSandwichParams& p, int t, bool own, RowParts<T, E>& r, const float (&post)[E][4], float* red, int& turn) {
-    if (p.y || p.e) {
+// Advances the row in r.x (stored when `own`) and returns one over its root mean square.
+template <typename T, int N, int E, bool EXPERTS>
+__device__ __forceinline__ float advance_row(const StreamSandwichParams& p, RowThreads<N>& th, int t, bool own, RowRaw<T, E>& r) {
+    if (p.ids) {
+#pragma unroll
+        for (int e = 0; e < E; ++e)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) r.x[e][i] = th.in(e, p.width) ? Cvt<T>::to_f(r.y[e][i]) : 0.f;
+    }
+    if (!EXPERTS && p.pos_table) {
+        const T* row = reinterpret_cast<const T*>(p.pos_table) + (size_t)min(max(p.positions[t], 0), p.max_pos - 1) * p.width;
+#pragma unroll
+        for (int e = 0; e < E; ++e)
+            if (th.in(e, p.width)) raw4(row + th.col(e), r.y[e]);
+#pragma unroll
+        for (int e = 0; e < E; ++e)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) r.x[e][i] += th.in(e, p.width) ? Cvt<T>::to_f(r.y[e][i]) : 0.f;
+    } else if constexpr (EXPERTS) {
+        float d[E][4];
+#pragma unroll
+        for (int e = 0; e < E; ++e)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) d[e][i] = p.y && th.in(e, p.width) ? Cvt<T>::to_f(r.y[e][i]) : 0.f;
+        for (int k0 = 0; k0 < p.top_k; k0 += 4) {                    // four expert rows in flight
+            const T* src[4];
+            float w[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const int row = k0 + k < p.top_k ? p.dst_row[(size_t)t * p.top_k + k0 + k] : -1;
+                w[k] = row < 0 ? 0.f : p.topk_w[(size_t)t * p.top_k + k0 + k];
+                src[k] = reinterpret_cast<const T*>(p.e) + (size_t)max(row, 0) * p.lde;
+            }
+#pragma unroll
+            for (int e = 0; e < E; ++e) {
+                if (!th.in(e, p.width)) continue;
+                alignas(16) T v[4][4];
+#pragma unroll
+                for (int k = 0; k < 4; ++k)
+                    if (w[k] != 0.f) raw4(src[k] + th.col(e), v[k]);
+#pragma unroll
+                for (int k = 0; k < 4; ++k)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i)
+                        if (w[k] != 0.f) d[e][i] = fmaf(w[k], Cvt<T>::to_f(v[k][i]), d[e][i]);
+            }
+        }
         float ss = 0.f;
 #pragma unroll
         for (int e = 0; e < E; ++e)
 #pragma unroll
-            for (int i = 0; i < 4; ++i) ss = fmaf(r.d[e][i], r.d[e][i], ss);
-        const float f = p.mult / sqrtf(block_total<N>(ss, red, turn) / p.width + p.eps);
-#pragma unroll
-        for (int e = 0; e < E; ++e)
-#pragma unroll
-            for (int i = 0; i < 4; ++i) r.x[e][i] = fmaf(r.d[e][i] * f, post[e][i], r.x[e][i]);
-    }
-    if (own && p.x_out) {
+            for (int i = 0; i < 4; ++i) ss = fmaf(d[e][i], d[e][i], ss);
+        const float f = p.mult / sqrtf(th.sum(ss) / p.width + p.eps);
 #pragma unroll
         for (int e = 0; e < E; ++e) {
-            const int c = (e * N + threadIdx.x) * 4;
-            if (c < p.width) put4(p.x_out + (size_t)t * p.width + c, r.x[e]);
+            if (!th.in(e, p.width)) continue;
+            float w[4];
+            get4(p.post + th.col(e), w);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) r.x[e][i] = fmaf(d[e][i] * f, w[i], r.x[e][i]);
+        }
+    } else if (p.y) {
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < E; ++e)
+            if (th.in(e, p.width)) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const float v = Cvt<T>::to_f(r.y[e][i]);
+                    ss = fmaf(v, v, ss);
+                }
+            }
+        const float f = p.mult / sqrtf(th.sum(ss) / p.width + p.eps);
+#pragma unroll
+        for (int e = 0; e < E; ++e) {
+            if (!th.in(e, p.width)) continue;
+            float w[4];
+            get4(p.post + th.col(e), w);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) r.x[e][i] = fmaf(Cvt<T>::to_f(r.y[e][i]) * f, w[i], r.x[e][i]);
         }
     }
-    if (!p.norm) return;
     float ss = 0.f;
 #pragma unroll
-    for (int e = 0; e < E; ++e)
+    for (int e = 0; e < E; ++e) {
+        if (!th.in(e, p.width)) continue;
+        if (own && p.x_out) put4(p.x_out + (size_t)t * p.width + th.col(e), r.x[e]);
 #pragma unroll
         for (int i = 0; i < 4; ++i) ss = fmaf(r.x[e][i], r.x[e][i], ss);
-    const float inv = 1.f / sqrtf(block_total<N>(ss, red, turn) / p.width + p.eps);
-#pragma unroll
-    for (int e = 0; e < E; ++e)
-#pragma unroll
-        for (int i = 0; i < 4; ++i) r.d[e][i] = r.x[e][i] * inv;
-}
-
-template <int N, int E>
-__device__ __forceinline__ void load_weight(const float* w, int width, float (&v)[E][4]) {
-#pragma unroll
-    for (int e = 0; e < E; ++e) {
-        const int c = (e * N + threadIdx.x) * 4;
-#pragma unroll
-        for (int i = 0; i < 4; ++i) v[e][i] = 0.f;
-        if (w && c < width) get4(w + c, v[e]);
     }
+    return p.norm ? 1.f / sqrtf(th.sum(ss) / p.width + p.eps) : 0.f;
 }
 
-// Every CTA takes the blocks that start in its range of block_rows rows (blocks count from the start of a sequence's portion).
-template <typename T, int N, int E, bool SHIFT>
-__global__ void __launch_bounds__(N) stream_sandwich_kernel(const __grid_constant__ StreamSandwichParams p) {
+// Every block index takes the blocks that start in its range of block_rows rows (blocks count from the start of a sequence's portion).
+template <typename T, int N, int E, bool SHIFT, bool EXPERTS>
+__global__ void __launch_bounds__(N * RowThreads<N>::kBlocks) stream_sandwich_kernel(const __grid_constant__ StreamSandwichParams p) {
     pdl_prologue();
     __shared__ float red[2 * (N / 32)];
-    const int tid = threadIdx.x;
-    int turn = 0;
-    float post[E][4], norm[E][4], shift[E][4];
-    load_weight<N, E>(p.post, p.width, post);
-    load_weight<N, E>(p.norm, p.width, norm);
-    if constexpr (SHIFT) load_weight<N, E>(p.shift, p.width, shift);
-    RowParts<T, E> r, next;
-    const int lo = blockIdx.x * p.block_rows, hi = min(p.tokens, lo + p.block_rows);
+    RowThreads<N> th;
+    th.red = red;
+    RowRaw<T, E> r, next;
+    constexpr bool kAhead = !RowThreads<N>::kWarp;                   // warps overlap one another instead
+    const int lo = th.block() * p.block_rows, hi = min(p.tokens, lo + p.block_rows);
+    T* h = reinterpret_cast<T*>(p.h);
+    if (lo >= hi) return;                                            // whole rows of threads at once
     if constexpr (!SHIFT) {
-        fetch_row<T, N, E>(p, lo, next);
+        if (kAhead) fetch_row<T, N, E>(p, th, lo, next);
         for (int t = lo; t < hi; ++t) {
-            r = next;
-            if (t + 1 < hi) fetch_row<T, N, E>(p, t + 1, next);
-            advance_row<T, N, E>(p, t, true, r, post, red, turn);
+            if (kAhead) {
+                r = next;
+                if (t + 1 < hi) fetch_row<T, N, E>(p, th, t + 1, next);
+            } else {
+                fetch_row<T, N, E>(p, th, t, r);
+            }
+            const float inv = advance_row<T, N, E, EXPERTS>(p, th, t, true, r);
             if (!p.norm) continue;
 #pragma unroll
             for (int e = 0; e < E; ++e) {
-                const int c = (e * N + tid) * 4;
-                if (c >= p.width) break;
+                if (!th.in(e, p.width)) continue;
+                float w[4];
+                get4(p.norm + th.col(e), w);
 #pragma unroll
-                for (int i = 0; i < 4; ++i) r.d[e][i] *= norm[e][i];
-                put4(reinterpret_cast<T*>(p.h) + (size_t)t * p.width + c, r.d[e]);
+                for (int i = 0; i < 4; ++i) w[i] *= r.x[e][i] * inv;
+                put4(h + (size_t)t * p.width + th.col(e), w);
             }
         }
     } else {
-        float before[E][4];                               // normed row in front of the current one, with its weight
-        auto keep = [&](const RowParts<T, E>& row) {
+        float before[E][4];                                          // normed row in front of the current one
+        auto keep = [&](float inv) {
 #pragma unroll
-            for (int e = 0; e < E; ++e)
+            for (int e = 0; e < E; ++e) {
+                if (!th.in(e, p.width)) continue;
+                float w[4];
+                get4(p.norm + th.col(e), w);
 #pragma unroll
-                for (int i = 0; i < 4; ++i) before[e][i] = row.d[e][i] * norm[e][i];
+                for (int i = 0; i < 4; ++i) before[e][i] = r.x[e][i] * inv * w[i];
+            }
         };
         for (int t = lo; t < hi;) {
             const int seq = p.seq_ids[t], t0 = p.q_start[seq], i0 = t - t0, ql = p.q_len[seq];
-            if (i0 % p.block_rows) {                      // inside a block that starts in an earlier range
+            if (i0 % p.block_rows) {                                 // inside a block that starts in an earlier range
                 t += min(p.block_rows - i0 % p.block_rows, ql - i0);
                 continue;
             }
             const int end = t + min(p.block_rows, ql - i0);
             float* state = p.state + (size_t)p.slot_ids[seq] * p.width;
             if (i0 > 0) {
-                fetch_row<T, N, E>(p, t - 1, r);
-                fetch_row<T, N, E>(p, t, next);
-                advance_row<T, N, E>(p, t - 1, false, r, post, red, turn);
-                keep(r);
+                fetch_row<T, N, E>(p, th, t - 1, r);
+                if (kAhead) fetch_row<T, N, E>(p, th, t, next);
+                keep(advance_row<T, N, E, EXPERTS>(p, th, t - 1, false, r));
             } else {
-                fetch_row<T, N, E>(p, t, next);
-                load_weight<N, E>(p.past_len[seq] > 0 ? state : nullptr, p.width, before);
+                const bool fresh = p.past_len[seq] <= 0;
+                if (kAhead) fetch_row<T, N, E>(p, th, t, next);
+#pragma unroll
+                for (int e = 0; e < E; ++e) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) before[e][i] = 0.f;
+                    if (!fresh && th.in(e, p.width)) get4(state + th.col(e), before[e]);
+                }
             }
             for (int u = t; u < end; ++u) {
-                r = next;
-                if (u + 1 < end) fetch_row<T, N, E>(p, u + 1, next);
-                advance_row<T, N, E>(p, u, true, r, post, red, turn);
+                if (kAhead) {
+                    r = next;
+                    if (u + 1 < end) fetch_row<T, N, E>(p, th, u + 1, next);
+                } else {
+                    fetch_row<T, N, E>(p, th, u, r);
+                }
+                const float inv = advance_row<T, N, E, EXPERTS>(p, th, u, true, r);
 #pragma unroll
                 for (int e = 0; e < E; ++e) {
-                    const int c = (e * N + tid) * 4;
-                    float v[4];
+                    if (!th.in(e, p.width)) continue;
+                    float w[4], sh[4];
+                    get4(p.norm + th.col(e), w);
+                    get4(p.shift + th.col(e), sh);
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
-                        const float h = r.d[e][i] * norm[e][i];
-                        v[i] = fmaf(before[e][i] - h, shift[e][i], h);
-                        before[e][i] = h;
+                        const float v = r.x[e][i] * inv * w[i];
+                        w[i] = fmaf(before[e][i] - v, sh[i], v);
+                        before[e][i] = v;
                     }
-                    if (c < p.width) put4(reinterpret_cast<T*>(p.h) + (size_t)u * p.width + c, v);
+                    put4(h + (size_t)u * p.width + th.col(e), w);
                 }
             }
-            if (i0 == 0) {                                // the state moves to the portion's last row
+            if (i0 == 0) {                                           // the state moves to the portion's last row
                 if (end < t0 + ql) {
-                    fetch_row<T, N, E>(p, t0 + ql - 1, r);
-                    advance_row<T, N, E>(p, t0 + ql - 1, false, r, post, red, turn);
-                    keep(r);
+                    fetch_row<T, N, E>(p, th, t0 + ql - 1, r);
+                    keep(advance_row<T, N, E, EXPERTS>(p, th, t0 + ql - 1, false, r));
                 }
 #pragma unroll
-                for (int e = 0; e < E; ++e) {
-                    const int c = (e * N + tid) * 4;
-                    if (c < p.width) put4(state + c, before[e]);
-                }
+                for (int e = 0; e < E; ++e)
+                    if (th.in(e, p.width)) put4(state + th.col(e), before[e]);
             }
             t = end;
         }
@@ -235,15 +297,28 @@ __global__ void __launch_bounds__(N) stream_sandwich_kernel(const __grid_constan
 
 template <typename T, int N, int E>
 static int launch_sandwich(const StreamSandwichParams& p, cudaStream_t stream) {
-    const dim3 grid((p.tokens + p.block_rows - 1) / p.block_rows);
-    if (p.shift) TELB_LAUNCH("stream_sandwich_kernel", (stream_sandwich_kernel<T, N, E, true>), grid, dim3(N), 0, stream, p);
-    else TELB_LAUNCH("stream_sandwich_kernel", (stream_sandwich_kernel<T, N, E, false>), grid, dim3(N), 0, stream, p);
+    constexpr int kBlocks = RowThreads<N>::kBlocks;
+    const int blocks = (p.tokens + p.block_rows - 1) / p.block_rows;
+    const dim3 grid((blocks + kBlocks - 1) / kBlocks), threads(N * kBlocks);
+#define TELB_SANDWICH(SHIFT_, EXPERTS_) TELB_LAUNCH("stream_sandwich_kernel", (stream_sandwich_kernel<T, N, E, SHIFT_, EXPERTS_>), grid, threads, 0, stream, p)
+    if (p.shift && p.e) TELB_SANDWICH(true, true);
+    else if (p.shift) TELB_SANDWICH(true, false);
+    else if (p.e) TELB_SANDWICH(false, true);
+    else TELB_SANDWICH(false, false);
+#undef TELB_SANDWICH
     TELB_CHECK_LAUNCH("stream_sandwich_kernel");
     return 0;
 }
 
 template <typename T>
-static int run_sandwich(const StreamSandwichParams& p, cudaStream_t stream) {
+static int run_sandwich(const StreamSandwichParams& p, int warp_rows, cudaStream_t stream) {
+    if (sizeof(T) == 2 && warp_rows > 0) {
+        StreamSandwichParams w = p;
+        w.block_rows = warp_rows;
+        if (p.width == 1024) return launch_sandwich<T, 32, 8>(w, stream);
+        if (p.width == 1536) return launch_sandwich<T, 32, 12>(w, stream);
+        if (p.width == 2048) return launch_sandwich<T, 32, 16>(w, stream);
+    }
     if (p.width <= 512) return launch_sandwich<T, 128, 1>(p, stream);
     if (p.width <= 1024) return launch_sandwich<T, 256, 1>(p, stream);
     if (p.width <= 2048) return launch_sandwich<T, 256, 2>(p, stream);
@@ -255,19 +330,20 @@ static int run_sandwich(const StreamSandwichParams& p, cudaStream_t stream) {
 
 using namespace telb;
 
-// dtype: 0 fp16, 1 bf16, 2 fp32 (of the tables, y, e and h).
-extern "C" int telb_stream_sandwich(const StreamSandwichParams* pp, int dtype, cudaStream_t stream) {
+// dtype: 1 bf16, 2 fp32 (of the tables, y, e and h).  warp_rows > 0: blocks of that many rows run on a warp each where the width allows.
+extern "C" int telb_stream_sandwich(const StreamSandwichParams* pp, int warp_rows, int dtype, cudaStream_t stream) {
     const StreamSandwichParams& p = *pp;
     if (p.tokens <= 0) return 0;
     if (p.width % 4 || p.width > 16 * 1024) return fail("telb_stream_sandwich: width must be a multiple of 4 and at most 16384");
     if (!p.ids == !p.x_in) return fail("telb_stream_sandwich: either ids or a stream");
     if (p.block_rows < 1) return fail("telb_stream_sandwich: blocks of at least one row");
+    if (p.ids && (p.y || p.e)) return fail("telb_stream_sandwich: a stream that starts from ids has no update");
+    if (p.pos_table && (p.y || p.e)) return fail("telb_stream_sandwich: position rows join before the first update");
     if ((p.y || p.e) && !p.post) return fail("telb_stream_sandwich: an update has a weight");
     if (p.e && (!p.dst_row || !p.topk_w || p.lde % 4)) return fail("telb_stream_sandwich: expert rows come with their tables");
     if (p.pos_table && (!p.positions || p.max_pos < 1)) return fail("telb_stream_sandwich: position rows need positions");
     if (p.norm && !p.h) return fail("telb_stream_sandwich: a norm has an output");
     if (p.shift && (!p.norm || !p.state)) return fail("telb_stream_sandwich: a shift has a norm and a state");
     if (p.x_out && p.x_out == p.x_in) return fail("telb_stream_sandwich: rows are not advanced in place");
-    if (dtype == 2) return run_sandwich<float>(p, stream);
-    return dtype == 1 ? run_sandwich<__nv_bfloat16>(p, stream) : run_sandwich<__half>(p, stream);
+    return dtype == 2 ? run_sandwich<float>(p, warp_rows, stream) : run_sandwich<__nv_bfloat16>(p, warp_rows, stream);
 }

@@ -409,9 +409,14 @@ def _sandwich_block_rows(tokens: int, shifted: bool) -> int:
     return 1 if tokens <= 148 * 2 else 4 if tokens <= 148 * 16 else 8
 
 
+SANDWICH_WARP_ROWS = (1, 8)      # rows per warp of long steps: as they are, with a shift
+
+
 def stream_sandwich(stream, eps: float, meta: StepMeta, dtype, ids, table, positions, delta, routed, post, mult: float, norm, shift, state):
     """See :func:`ops.stream_sandwich`; ``routed`` carries expert rows (``y``, routing tables ``ws``, weights)."""
     f32 = torch.float32
+    if dtype not in (torch.bfloat16, f32):
+        raise TypeError(f"stream_sandwich: rows in bf16 or fp32, not {dtype}")
     if stream is None:
         t, width, dev = ids.numel(), table.shape[1], table.device
         ids = ids.to(torch.int32).contiguous()
@@ -440,8 +445,9 @@ def stream_sandwich(stream, eps: float, meta: StepMeta, dtype, ids, table, posit
         ids, table, positions, stream, delta, y, None if ws is None else ws.dst_row, w, post, norm, shift, state, x, h, meta.positions, meta.q_start, meta.q_len,
         meta.past_len, meta.slot_ids, meta.seq_ids)], 0 if table is None else table.shape[0], 0 if positions is None else positions.shape[0], width, t, rows,
         0 if w is None else w.shape[1], 0 if y is None else y.shape[1], mult, eps)
-    code = 2 if dtype == f32 else int(dtype == torch.bfloat16)
-    _check(lib().telb_stream_sandwich(ctypes.byref(p), c_int(code), _stream()), "stream_sandwich")
+    code = 2 if dtype == f32 else 1
+    warp_rows = SANDWICH_WARP_ROWS[shift is not None] if t >= 148 * 8 else 0
+    _check(lib().telb_stream_sandwich(ctypes.byref(p), c_int(warp_rows), c_int(code), _stream()), "stream_sandwich")
     return x, h
 
 

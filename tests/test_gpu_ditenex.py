@@ -7,7 +7,7 @@ import ditenex_oracle as oracle
 
 pytestmark = pytest.mark.gpu
 DEV = "cuda"
-DTYPES = {"bfloat16": torch.bfloat16, "float16": torch.float16, "float32": torch.float32}
+DTYPES = {"bfloat16": torch.bfloat16, "float32": torch.float32}
 
 
 @pytest.fixture(scope="module")
@@ -31,7 +31,7 @@ def no_timed_out_waits():
 # ---- kernels ------------------------------------------------------------------------------------------------
 
 
-@pytest.mark.parametrize("dtype", ["bfloat16", "float16", "float32"])
+@pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
 @pytest.mark.parametrize("width", [24, 40, 520, 1032, 2048, 4096, 5120])
 def test_stream_norms_and_token_shift(width, dtype):
     """Rows of one portion in several blocks, portions of one and two rows; state rows held other requests."""
@@ -45,7 +45,12 @@ def test_stream_norms_and_token_shift(width, dtype):
 
 
 def test_stream_long_blocks():
-    """Enough rows for blocks of four and of eight, sequences that start inside another one's range."""
+    """Enough rows for longer blocks and for a warp per block, sequences that start inside another one's range."""
+    for width in (1024, 1536, 2048, 2056):
+        for kw in (dict(), dict(top=5), dict(top=2, dense=False), dict(ids=True), dict(shift=False), dict(shift=False, top=4)):
+            x, h = cases.sandwich_case(DEV, torch.bfloat16, width, [1300, 5, 700, 3], [1290, 2, 90, 1], **kw)
+            assert x < 1e-5 and h < 8e-3, (width, kw)
+            assert cases.sandwich_case(DEV, torch.bfloat16, width, [1300, 5, 700, 3], **kw)[0] < 1e-5
     for n in (900, 5000):
         for kw in (dict(), dict(shift=False)):
             assert max(cases.sandwich_case(DEV, torch.float32, 64, [n, 5, 700, 3], [n - 9, 2, 300, 1], **kw)) < 1e-5
