@@ -15,7 +15,7 @@ namespace telb {
 // Host mirror: ops/cuda.py (MixedKvParams).
 struct MixedKvParams {
     const void* rows;            // [T, ld]: q [hq * d] | k [hkv * d] | v [hkv * d] | ...
-    const void* first;           // [T, ld_first] values of another layer, or null
+    const void* first;           // [T, ld_first] values of another layer, heads of d_first features (padded unlike d perhaps), or null
     void* q_out;                 // [T, hq, halves * hkv * d]
     void* kv;                    // [pages, 2, hkv, P, d]
     const float* mix;            // [hq, hq]
@@ -25,7 +25,7 @@ struct MixedKvParams {
     const int* past_len;
     const int* page_table;
     long long ld, ld_first;
-    int tokens, max_pages, page_size, hq, hkv, d, halves;
+    int tokens, max_pages, page_size, hq, hkv, d, halves, d_first;
 };
 
 constexpr int kMixThreads = 256;
@@ -110,8 +110,8 @@ __global__ void __launch_bounds__(kMixThreads) mixed_kv_write_kernel(const __gri
         float v[8];
         load8(row + (size_t)hq * d + (size_t)w * 8, v);
         if (p.first && w >= units) {
-            float o[8];
-            load8(reinterpret_cast<const T*>(p.first) + (size_t)t * p.ld_first + (size_t)(w - units) * 8, o);
+            float o[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+            if (f < p.d_first) load8(reinterpret_cast<const T*>(p.first) + (size_t)t * p.ld_first + (size_t)(c - p.hkv) * p.d_first + f, o);
 #pragma unroll
             for (int k = 0; k < 8; ++k) v[k] = fmaf(share, o[k], (1.f - share) * v[k]);
         }
@@ -145,7 +145,7 @@ extern "C" int telb_mixed_kv_write(const MixedKvParams* pp, int dtype, cudaStrea
     const MixedKvParams& p = *pp;
     if (p.tokens <= 0) return 0;
     if (p.hkv <= 0 || p.hq % p.hkv) return fail("telb_mixed_kv_write: query heads are a multiple of the KV heads");
-    if (p.d % 8 || p.ld % 8 || p.ld_first % 8) return fail("telb_mixed_kv_write: heads and row pitches in multiples of 8");
+    if (p.d % 8 || p.ld % 8 || p.ld_first % 8 || p.d_first % 8) return fail("telb_mixed_kv_write: heads and row pitches in multiples of 8");
     if (p.halves != 1 && (p.halves != 2 || dtype == 2)) return fail("telb_mixed_kv_write: one or (16-bit) two halves");
     if (p.first && !p.share) return fail("telb_mixed_kv_write: mixed values have a share");
     if (dtype == 2) return launch_mixed_kv<float>(p, stream);

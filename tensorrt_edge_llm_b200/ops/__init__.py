@@ -317,7 +317,7 @@ def turned_kv_write(rows, kv_layer, meta, key_table, value_table, q_norm, k_norm
 
 def mixed_kv_write(rows, kv_layer, meta, mix, first, share, spec):
     """Packed q | k | v rows (and what lies behind them) of padded heads: keys go to the paged cache, values too, ``(1 - share) v + share *
-    first`` when ``first`` ``[T, kv heads * pad]`` is given.  Returns the wide queries: head ``h`` holds, for every KV head ``c``, the sum of
+    first`` when ``first`` ``[T, kv heads * its pad]`` is given (its heads may be padded to another size).  Returns the wide queries: head ``h`` holds, for every KV head ``c``, the sum of
     ``mix[h, g] q_g`` over the query heads ``g`` of ``c``.  ``spec``: :class:`config.AttentionConfig`."""
     f = cuda_ops().mixed_kv_write if rows.is_cuda else ref.mixed_kv_write
     return f(rows, kv_layer, meta, mix, first, share, spec)

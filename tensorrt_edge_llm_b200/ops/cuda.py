@@ -1414,7 +1414,7 @@ def _row_split(meta: StepMeta, limit: int, device) -> RowSplit:
 class MixedKvParams(ctypes.Structure):
     """Host mirror of ``MixedKvParams`` (``csrc/kernels/mixed_heads.cu``)."""
     _fields_ = [(n, c_vp) for n in ("rows", "first", "q_out", "kv", "mix", "share", "seq_ids", "q_start", "past_len", "page_table")] + \
-               [(n, c_ll) for n in ("ld", "ld_first")] + [(n, c_int) for n in ("tokens", "max_pages", "page_size", "hq", "hkv", "d", "halves")]
+               [(n, c_ll) for n in ("ld", "ld_first")] + [(n, c_int) for n in ("tokens", "max_pages", "page_size", "hq", "hkv", "d", "halves", "d_first")]
 
 
 def _mixed_tc(spec, dtype, page_size: int) -> bool:
@@ -1434,13 +1434,13 @@ def mixed_kv_write(rows, kv_layer, meta: StepMeta, mix, first, share, spec):
     assert mix.dtype == torch.float32 and mix.is_contiguous() and mix.shape == (n, n) and share.dtype == torch.float32
     if first is not None:
         first = _pitched(first)
-        assert first.dtype == rows.dtype and first.shape == (t, g * d)
+        assert first.dtype == rows.dtype and first.shape[0] == t and first.shape[1] % (8 * g) == 0
     halves = 1
     if _mixed_tc(spec, rows.dtype, meta.page_size) and (g * d <= 256 or _mixed_plan(meta, n, rows.device).long is None):
         halves = 2
     q = torch.empty(t, n, halves * g * d, dtype=rows.dtype, device=rows.device)
     p = MixedKvParams(*[None if x is None else _p(x).value for x in (rows, first, q, kv_layer, mix, share, meta.seq_ids, meta.q_start, meta.past_len, meta.page_table)],
-                      rows.stride(0), 0 if first is None else first.stride(0), t, meta.page_table.shape[1], meta.page_size, n, g, d, halves)
+                      rows.stride(0), 0 if first is None else first.stride(0), t, meta.page_table.shape[1], meta.page_size, n, g, d, halves, 0 if first is None else first.shape[1] // g)
     _check(lib().telb_mixed_kv_write(ctypes.byref(p), c_int(_dtype_code(rows)), _stream()), "mixed_kv_write")
     return q
 

@@ -782,7 +782,8 @@ def mixed_kv_write(rows, kv_layer, meta: StepMeta, mix, first, share, spec):
     t, d, n, g = rows.shape[0], spec.pad, spec.num_heads, spec.num_kv_heads
     q, k, v = rows[:, :(n + 2 * g) * d].float().split([n * d, g * d, g * d], dim=-1)
     if first is not None:
-        v = (1 - share) * v + share * first.float()
+        f = first.float().reshape(t, g, -1)
+        v = (1 - share) * v + share * F.pad(f, (0, d - f.shape[2])).reshape(t, g * d)        # a negative pad cuts padding off
     page, row = _cache_slots(meta, t, rows.device)
     kv_layer[page, 0, :, row] = k.reshape(t, g, d).to(kv_layer.dtype)
     kv_layer[page, 1, :, row] = v.reshape(t, g, d).to(kv_layer.dtype)

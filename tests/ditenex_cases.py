@@ -36,10 +36,10 @@ def small_config(layers, width=64, vocab=96, eps=1e-5, mult=0.4, positions=400):
 
 def _cfg_mixed():
     """Uneven sizes everywhere: padded heads, value sizes unlike key sizes, three query heads per KV head; the first layer does not mix
-    values and one in between neither; a layer without a feed-forward, experts with and without a shared one."""
+    values and one in between neither; layers that mix values pad their heads differently; a layer without a feed-forward, experts with and without a shared one."""
     return small_config([(attn(6, 2, 40, 56, 37, v_mix=False), dense(72)), (attn(6, 3, 40, 24, 20), moe(9, 3, 40, 3, 2, 1.7, 48)),
                          (attn(3, 3, 24, 24, 70), None), (attn(2, 1, 72, 16, 33, v_mix=False), moe(6, 2, 24, 2, 1, 2.5)),
-                         (attn(12, 3, 16, 24, 90), dense(40))], width=72, vocab=101)
+                         (attn(12, 3, 72, 24, 90), dense(40))], width=72, vocab=101)
 
 
 def _cfg_wide():
@@ -56,7 +56,7 @@ def _cfg_ones():
 
 def _cfg_long():
     """Windows that lie far inside a prompt, one key head for all, as many key heads as query heads, experts of which all are used."""
-    return small_config([(attn(8, 1, 64, 64, 100), moe(4, 4, 24, 2, 2, 0.7, 24)), (attn(4, 2, 64, 40, 300, v_mix=False), dense(64)),
+    return small_config([(attn(8, 1, 80, 64, 100), moe(4, 4, 24, 2, 2, 0.7, 24)), (attn(4, 2, 64, 40, 300, v_mix=False), dense(64)),
                          (attn(5, 1, 64, 64, 65), None), (attn(10, 10, 48, 32, 50, v_mix=False), dense(32))], width=40, vocab=72, mult=0.6)
 
 

@@ -39,7 +39,7 @@ def test_config_round_trip(ckpt):
     assert (e.router, e.limit, e.alpha, e.up_offset) == ("sigmoid_groups", 0.0, 1.0, 0.0) and cfg.layer_specs[3].moe.shared_size == 0
     assert (cfg.layer_specs[0].ff, cfg.layer_specs[0].ff_act, cfg.residual_mult, cfg.max_position_embeddings) == (72, "xielu", 0.4, 400)
     assert cfg.token_shift and cfg.learned_positions and cfg.is_hybrid and cfg.tie_word_embeddings
-    assert cfg.kv_geometry() == [(2, 64), (3, 64), (3, 64), (1, 128), (3, 64)] and cfg.num_attn_layers == 5
+    assert cfg.kv_geometry() == [(2, 64), (3, 64), (3, 64), (1, 128), (3, 128)] and cfg.num_attn_layers == 5
     again = ModelConfig.from_dict(json.loads(json.dumps(cfg.to_dict())))
     assert again.layer_specs == cfg.layer_specs and again.token_shift
 
